@@ -71,13 +71,25 @@ def build_host(force: bool = False) -> Path:
     return HOST_LIB
 
 
-def build_cuda(force: bool = False) -> Path:
+# Kernel sources a dense / recurrent graph needs without experts, DeltaNet, EXL3 or sharded prefill.  A checkout without the full library
+# can compile just these (``_lib.use_components("core")``); the full library, when it is there, serves every graph.
+COMPONENTS = {
+    "core": ("common", "comm", "elementwise", "gemm_tcgen05", "gemv", "gemv_stream", "linear_f32", "attention", "attention_tc", "mingru", "sampling"),
+}
+
+
+def build_cuda(force: bool = False, component: str | None = None) -> Path:
+    """The sm_100a kernel library; ``component`` builds only that subset, into a library of its own."""
     srcs = sorted((CSRC / "cuda").glob("*.cu"))
+    lib = CUDA_LIB
+    if component is not None:
+        srcs = [s for s in srcs if s.stem in COMPONENTS[component]]
+        lib = CUDA_LIB.with_name(f"libmx_cuda_{component}.so")
     hdrs = sorted((CSRC / "cuda").glob("*.cuh")) + sorted((CSRC / "cuda").glob("*.h"))
     OUT.mkdir(exist_ok=True)
-    stale, dg = _stale(CUDA_LIB, srcs + hdrs, " ".join(NVCC_FLAGS))
+    stale, dg = _stale(lib, srcs + hdrs, " ".join(NVCC_FLAGS))
     if not (stale or force):
-        return CUDA_LIB
+        return lib
     nvcc = _nvcc()
     if nvcc is None:
         raise RuntimeError("nvcc not found: cannot build the sm_100a kernels")
@@ -96,9 +108,9 @@ def build_cuda(force: bool = False) -> Path:
 
     with ThreadPoolExecutor(max_workers=min(8, len(srcs) or 1)) as ex:
         objs = list(ex.map(compile_one, srcs))
-    _run([nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", *map(str, objs), "-o", str(CUDA_LIB)])
-    CUDA_LIB.with_suffix(".stamp").write_text(dg)
-    return CUDA_LIB
+    _run([nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", *map(str, objs), "-o", str(lib)])
+    lib.with_suffix(".stamp").write_text(dg)
+    return lib
 
 
 def build_all(force: bool = False) -> None:

@@ -15,6 +15,7 @@ from . import _build
 _lock = threading.Lock()
 _host = None
 _cuda = None
+_component = None
 
 
 class NativeError(RuntimeError):
@@ -33,6 +34,13 @@ def host() -> C.CDLL:
     return _host
 
 
+def use_components(name: str) -> None:
+    """Before the first kernel: this process needs only the ``name`` subset of the kernels.  It is built (and loaded) when the checkout has no
+    full library; a full library is used as it is."""
+    global _component
+    _component = name
+
+
 def cuda() -> C.CDLL:
     global _cuda
     if _cuda is None:
@@ -40,7 +48,7 @@ def cuda() -> C.CDLL:
             if _cuda is None:
                 path = _build.CUDA_LIB
                 if not path.exists():
-                    path = _build.build_cuda()
+                    path = _build.build_cuda(component=_component)
                 try:
                     lib = C.CDLL(str(path))
                 except OSError as e:  # pragma: no cover - needs a broken install

@@ -1,6 +1,6 @@
 """``ie`` command line: ``run`` (REPL), ``serve`` (OpenAI server on :11435), ``bench`` (ie-bench), ``import``
-(AWQ / GPTQ safetensors -> GGUF), ``pull`` (model fetch helper), ``inspect`` (GGUF listing), ``synth`` (write a
-random-init GGUF of a named architecture).
+(AWQ / GPTQ safetensors -> GGUF), ``pull`` (model fetch helper), ``inspect`` (checkpoint listing), ``synth`` (write a
+random-init checkpoint of a named architecture).
 
 Reference parity: src/cli/main.cpp:13-157 (sub-commands and the flags ``--ctx --port --host --gpus --int8-kv
 --spec --spec-k --spec-head``; REPL commands ``/reset`` ``/quit``; ``IE_PERF`` per-turn statistics).
@@ -42,7 +42,7 @@ def _load(a):
     from ..formats.memory_plan import plan_placement
     if par.rank == 0:
         print(plan_placement(a.model, n_gpus=max(par.world, 1), ctx=a.ctx).describe(), file=sys.stderr)
-    return Engine.load(a.model, dev, _engine_options(a), par, spec_head=a.spec_head), par
+    return Engine.load(a.model, dev, _engine_options(a), par, spec_head=a.spec_head, dtype=a.dtype), par
 
 
 def main(argv=None) -> int:
@@ -60,6 +60,7 @@ def main(argv=None) -> int:
         p.add_argument("--spec", action="store_true")
         p.add_argument("--spec-k", type=int, default=3)
         p.add_argument("--spec-head", default=None, help="draft-head GGUF for --spec (Gemma-4: the gemma4-assistant file)")
+        p.add_argument("--dtype", default="bf16", choices=("bf16", "fp32"), help="fp32: run in 32-bit throughout (graphs that support it)")
         p.add_argument("--cpu", action="store_true")
 
     p = sub.add_parser("run"); common(p)
@@ -93,9 +94,9 @@ def main(argv=None) -> int:
         from .inspect_gguf import inspect
         return inspect(a.gguf, a.tensors)
     if a.cmd == "synth":
-        from ..formats.synth import write_synthetic_gguf
+        from ..formats.synth import write_synthetic
         from ..formats.model_config import preset
-        write_synthetic_gguf(preset(a.preset), a.out, quant=a.quant, seed=a.seed)
+        write_synthetic(preset(a.preset), a.out, quant=a.quant, seed=a.seed)
         print(f"wrote {a.out}")
         return 0
 
@@ -126,6 +127,15 @@ def main(argv=None) -> int:
             break
         if line.strip() == "/reset":
             turns = []
+            continue
+        if eng.tok is None:                # a checkpoint without a tokenizer: token ids in, token ids out
+            try:
+                ids = [int(t) for t in line.split()]
+            except ValueError:
+                print("this checkpoint has no tokenizer: type token ids", file=sys.stderr)
+                continue
+            res = eng.generate(ids, SamplingParams(temperature=a.temperature, max_tokens=a.max_tokens))
+            print(" ".join(str(t) for t in res.token_ids) if not res.error else f"error: {res.error}")
             continue
         turns.append(ChatTurn("user", line))
         res = eng.chat(turns, SamplingParams(temperature=a.temperature, max_tokens=a.max_tokens), on_text=lambda s: (sys.stdout.write(s), sys.stdout.flush()))

@@ -10,7 +10,12 @@
 // launch.  Splits that would get no key tile exit at once and are not counted.  The separate
 // combine kernel remains for batches with more groups than there are tickets.
 //
-// KV cache layout: [block][kv_head][block_size][head_dim] bf16, block_size a multiple of 64.  An int8 cache has the
+// Keys and values may have different widths (multiples of 8, at most 512), the score scale may depend on the query's position
+// (a table over positions: query temperature) and the output may be multiplied by the sigmoid of a gate.  Shapes with equal widths of
+// 64 / 128 / 256 / 512 run on instances whose widths are compile-time constants; all other shapes, and caches in fp32, run on
+// instances that take the widths at run time and only round the value width up to 64 / 128 / 256 / 512 (accumulator registers).
+//
+// KV cache layout: [block][kv_head][block_size][head_dim] bf16 (or fp32), block_size a multiple of 64.  An int8 cache has the
 // same layout with one byte per element plus an fp32 scale per (block, kv head, token) row (value = q * scale); the
 // staging loop widens it to bf16, so the math below is shared.  kv_dequant_pages_kernel expands the pages of a prefill
 // batch into a bf16 scratch cache for the tensor-core prefill kernel.
@@ -18,6 +23,7 @@
 // Reference parity: src/ops/attention.cpp:229-454 (naive / gpt-oss window + sink),
 // :685-1036 (split-K flash decode, sink folded in combine), :2456-2714 (wide tile prefill with
 // causal + window masks and whole-tile skipping).
+#include "act.cuh"
 #include "common.cuh"
 #include "host_util.h"
 #include "mx_noalloc.h"
@@ -30,19 +36,22 @@ constexpr int ATT_WARPS = 8;
 constexpr int ATT_TILE = 64;
 
 struct AttnParams {
-  const __nv_bfloat16* q;      // [Tq][n_q][hd]
-  const __nv_bfloat16* k_cache;
-  const __nv_bfloat16* v_cache;
+  const void* q;               // [Tq] rows of [n_q][dk], q_ld elements apart
+  const void* k_cache;
+  const void* v_cache;
   const float* k_scale;        // non-null: the caches hold int8 and these are the per-row scales [block][kv_head][block_size]
   const float* v_scale;
   const int* block_table;      // [B][max_blocks]
   const int* seq_lens;         // [B] kv length including this step's tokens
   const int* cu_q;             // [B+1]
-  float* o_part;               // [splits][Tq][n_q][hd]
+  const float* q_scale;        // [q_scale_n] factor on the scores of a query at that position, or null
+  const void* gate;            // out is multiplied by sigmoid(gate): [Tq] rows of [n_q][dv], gate_ld elements apart, or null
+  int q_scale_n, q_ld, gate_ld, dk, dv;
+  float* o_part;               // [splits][Tq][n_q][dv]
   float* ml_part;              // [splits][Tq][n_q][2]
   int* tickets;                // non-null: one counter per (batch entry, query tile, kv head) group; the last split merges
   const float* sinks;          // [n_q] or null (used by the merging CTA)
-  __nv_bfloat16* out;          // [Tq][n_q][hd] (written by the merging CTA)
+  void* out;                   // [Tq][n_q][dv] (written by the merging CTA)
   int B, n_q, n_kv, max_blocks, block_size;
   int q_tile;                  // query tokens per CTA
   int max_q_tiles;             // per sequence
@@ -85,15 +94,28 @@ __global__ void __launch_bounds__(256) kv_dequant_pages_kernel(const int8_t* __r
   }
 }
 
-template <int HD, int PPW>
-__global__ void __launch_bounds__(ATT_WARPS * 32) attn_partial_kernel(const AttnParams p) {
+// elements by which a K row is padded in shared memory: an odd number of words apart, conflict-free one-key-per-lane reads
+template <typename T> __host__ __device__ constexpr int att_kpad() { return sizeof(T) == 2 ? 2 : 1; }
+// two consecutive K elements of a padded row (an fp32 row may start on an odd word)
+__device__ __forceinline__ float2 k_pair(const __nv_bfloat16* r, int c) { return load2(r + 2 * c); }
+__device__ __forceinline__ float2 k_pair(const float* r, int c) { return make_float2(r[2 * c], r[2 * c + 1]); }
+template <bool PRECISE> __device__ __forceinline__ float att_exp(float x) { return PRECISE ? expf(x) : __expf(x); }
+
+// EXACT: keys and values are both HD wide; otherwise the widths come from the parameters (dv <= HD)
+template <typename T, int HD, int PPW, bool EXACT>
+__global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 : (PPW == 2 || HD <= 128) ? 3 : 2) attn_partial_kernel(const AttnParams p) {
   pdl_prologue();
   constexpr int PAIRS = ATT_WARPS * PPW;
-  constexpr int KSTR = HD + 2;   // padded K row (elements): conflict-free one-key-per-lane reads
+  constexpr bool PRECISE = sizeof(T) == 4;
+  constexpr int VE = 16 / sizeof(T);                                               // elements per 16-byte access
+  const int DK = EXACT ? HD : p.dk, DV = EXACT ? HD : p.dv;
+  const int KSTR = DK + att_kpad<T>();
   extern __shared__ uint8_t smem_raw[];
-  float* sq = reinterpret_cast<float*>(smem_raw);                                  // [PAIRS][HD]
-  __nv_bfloat16* sk = reinterpret_cast<__nv_bfloat16*>(sq + PAIRS * HD);           // [64][KSTR]
-  __nv_bfloat16* sv = sk + ATT_TILE * KSTR;                                        // [64][HD]
+  float* sq = reinterpret_cast<float*>(smem_raw);                                  // [PAIRS][DK]
+  T* sv = reinterpret_cast<T*>(sq + PAIRS * DK);                                   // [64][DV]
+  T* sk = sv + ATT_TILE * DV;                                                      // [64][KSTR]
+  const T* kc = reinterpret_cast<const T*>(p.k_cache);
+  const T* vc = reinterpret_cast<const T*>(p.v_cache);
 
   const int b = blockIdx.x / p.max_q_tiles, qt = blockIdx.x % p.max_q_tiles;
   const int kvh = blockIdx.y, split = blockIdx.z;
@@ -121,12 +143,14 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attn_partial_kernel(const Attn
   for (int round0 = 0; round0 < total_pairs; round0 += PAIRS) {
     __syncthreads();
     // stage the queries of this round as fp32, pre-scaled
-    for (int i = threadIdx.x; i < PAIRS * HD; i += blockDim.x) {
-      const int pr = round0 + i / HD, d = i % HD;
+    for (int i = threadIdx.x; i < PAIRS * DK; i += blockDim.x) {
+      const int pr = round0 + i / DK, d = i % DK;
       float v = 0.f;
       if (pr < total_pairs) {
         const int tq = pr / gqa, hq = kvh * gqa + pr % gqa;
-        v = __bfloat162float(p.q[((size_t)(q_begin + t0 + tq) * p.n_q + hq) * HD + d]) * p.scale;
+        float sc = p.scale;
+        if (p.q_scale) sc *= p.q_scale[min(pos0 + tq, p.q_scale_n - 1)];
+        v = to_f32(reinterpret_cast<const T*>(p.q)[(size_t)(q_begin + t0 + tq) * p.q_ld + (size_t)hq * DK + d]) * sc;
       }
       sq[i] = v;
     }
@@ -141,11 +165,12 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attn_partial_kernel(const Attn
       __syncthreads();
       const int key0 = tile * ATT_TILE;
       const int blk = p.block_table[(size_t)b * p.max_blocks + key0 / p.block_size];
-      const size_t base = (((size_t)blk * p.n_kv + kvh) * p.block_size + key0 % p.block_size) * HD;
-      if (p.k_scale) {
+      const size_t row0 = ((size_t)blk * p.n_kv + kvh) * p.block_size + key0 % p.block_size;
+      if (EXACT && sizeof(T) == 2 && p.k_scale) {
+        const size_t base = row0 * HD;
         const int8_t* k8 = reinterpret_cast<const int8_t*>(p.k_cache);
         const int8_t* v8 = reinterpret_cast<const int8_t*>(p.v_cache);
-        const size_t srow = ((size_t)blk * p.n_kv + kvh) * p.block_size + key0 % p.block_size;
+        const size_t srow = row0;
         for (int i = threadIdx.x; i < ATT_TILE * HD / 8; i += blockDim.x) {
           const int r = i / (HD / 8), c = (i % (HD / 8)) * 8;
           const uint2 kq = *reinterpret_cast<const uint2*>(k8 + base + (size_t)r * HD + c);
@@ -160,12 +185,26 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attn_partial_kernel(const Attn
           *reinterpret_cast<uint4*>(sv + r * HD + c) = vv;
         }
       } else {
-        for (int i = threadIdx.x; i < ATT_TILE * HD / 8; i += blockDim.x) {
-          const int r = i / (HD / 8), c = (i % (HD / 8)) * 8;
-          const uint4 kv4 = *reinterpret_cast<const uint4*>(p.k_cache + base + (size_t)r * HD + c);
-          uint32_t* kd = reinterpret_cast<uint32_t*>(sk + r * KSTR + c);
-          kd[0] = kv4.x; kd[1] = kv4.y; kd[2] = kv4.z; kd[3] = kv4.w;
-          *reinterpret_cast<uint4*>(sv + r * HD + c) = *reinterpret_cast<const uint4*>(p.v_cache + base + (size_t)r * HD + c);
+        const int pk = DK / VE, pv = DV / VE;
+        const T* kp = kc + row0 * DK;
+        const T* vp = vc + row0 * DV;
+        if constexpr (EXACT) {
+          for (int i = threadIdx.x; i < ATT_TILE * pk; i += blockDim.x) {
+            const int r = i / pk, c = (i % pk) * VE;
+            const uint4 kv4 = *reinterpret_cast<const uint4*>(kp + (size_t)r * DK + c);
+            uint32_t* kd = reinterpret_cast<uint32_t*>(sk + r * KSTR + c);
+            kd[0] = kv4.x; kd[1] = kv4.y; kd[2] = kv4.z; kd[3] = kv4.w;
+            *reinterpret_cast<uint4*>(sv + r * DV + c) = *reinterpret_cast<const uint4*>(vp + (size_t)r * DV + c);
+          }
+        } else {
+          for (int i = threadIdx.x; i < ATT_TILE * pk; i += blockDim.x) {
+            const int r = i / pk, c = (i % pk) * VE;
+            const uint4 kv4 = *reinterpret_cast<const uint4*>(kp + (size_t)r * DK + c);
+            uint32_t* kd = reinterpret_cast<uint32_t*>(sk + r * KSTR + c);
+            kd[0] = kv4.x; kd[1] = kv4.y; kd[2] = kv4.z; kd[3] = kv4.w;
+          }
+          for (int i = threadIdx.x; i < ATT_TILE * pv; i += blockDim.x)            // the tile's rows are one dense run
+            reinterpret_cast<uint4*>(sv)[i] = reinterpret_cast<const uint4*>(vp)[i];
         }
       }
       __syncthreads();
@@ -177,19 +216,19 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attn_partial_kernel(const Attn
         float sc[PPW][2];
         {
           // both keys of the lane in one pass: a query element read from shared memory feeds two dot products
-          const uint32_t* kr0 = reinterpret_cast<const uint32_t*>(sk + lane * KSTR);
-          const uint32_t* kr1 = reinterpret_cast<const uint32_t*>(sk + (lane + 32) * KSTR);
-          const float* qv = sq + warp * PPW * HD;
+          const T* kr0 = sk + lane * KSTR;
+          const T* kr1 = sk + (lane + 32) * KSTR;
+          const float* qv = sq + warp * PPW * DK;
           float d0[PPW], d1[PPW];
 #pragma unroll
           for (int pi = 0; pi < PPW; ++pi) d0[pi] = d1[pi] = 0.f;
 #pragma unroll 8
-          for (int c = 0; c < HD / 2; ++c) {
-            const uint32_t ka = kr0[c], kb = kr1[c];
-            const float a0 = bf16_lo(ka), a1 = bf16_hi(ka), b0 = bf16_lo(kb), b1 = bf16_hi(kb);
+          for (int c = 0; c < DK / 2; ++c) {
+            const float2 ka = k_pair(kr0, c), kb = k_pair(kr1, c);
+            const float a0 = ka.x, a1 = ka.y, b0 = kb.x, b1 = kb.y;
 #pragma unroll
             for (int pi = 0; pi < PPW; ++pi) {
-              const float2 qq = *reinterpret_cast<const float2*>(qv + pi * HD + 2 * c);
+              const float2 qq = *reinterpret_cast<const float2*>(qv + pi * DK + 2 * c);
               d0[pi] = fmaf(qq.x, a0, d0[pi]); d0[pi] = fmaf(qq.y, a1, d0[pi]);
               d1[pi] = fmaf(qq.x, b0, d1[pi]); d1[pi] = fmaf(qq.y, b1, d1[pi]);
             }
@@ -212,9 +251,9 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attn_partial_kernel(const Attn
         for (int pi = 0; pi < PPW; ++pi) {
           const float tmax = warp_max(fmaxf(sc[pi][0], sc[pi][1]));
           const float m_new = fmaxf(m[pi], tmax);
-          const float corr = __expf(m[pi] - m_new);
-          p0[pi] = __expf(sc[pi][0] - m_new);
-          p1[pi] = __expf(sc[pi][1] - m_new);
+          const float corr = att_exp<PRECISE>(m[pi] - m_new);
+          p0[pi] = att_exp<PRECISE>(sc[pi][0] - m_new);
+          p1[pi] = att_exp<PRECISE>(sc[pi][1] - m_new);
           l[pi] = l[pi] * corr + warp_sum(p0[pi] + p1[pi]);
           m[pi] = m_new;
 #pragma unroll
@@ -224,10 +263,10 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attn_partial_kernel(const Attn
       // P V: a value element is read once per key and feeds all PPW pairs
 #pragma unroll 2
       for (int j = 0; j < ATT_TILE; ++j) {
-        const __nv_bfloat16* vr = sv + j * HD;
+        const T* vr = sv + j * DV;
         float vv[HD / 32];
 #pragma unroll
-        for (int c = 0; c < HD / 32; ++c) vv[c] = __bfloat162float(vr[lane + 32 * c]);
+        for (int c = 0; c < HD / 32; ++c) vv[c] = (EXACT || lane + 32 * c < DV) ? to_f32(vr[lane + 32 * c]) : 0.f;
 #pragma unroll
         for (int pi = 0; pi < PPW; ++pi) {
           const float pj = __shfl_sync(0xffffffffu, j < 32 ? p0[pi] : p1[pi], j & 31);
@@ -244,7 +283,8 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attn_partial_kernel(const Attn
       const int tq = pr / gqa, hq = kvh * gqa + pr % gqa;
       const size_t row = ((size_t)split * p.Tq + (q_begin + t0 + tq)) * p.n_q + hq;
 #pragma unroll
-      for (int c = 0; c < HD / 32; ++c) p.o_part[row * HD + lane + 32 * c] = acc[pi][c];
+      for (int c = 0; c < HD / 32; ++c)
+        if (EXACT || lane + 32 * c < DV) p.o_part[row * DV + lane + 32 * c] = acc[pi][c];
       if (lane == 0) { p.ml_part[row * 2] = m[pi]; p.ml_part[row * 2 + 1] = l[pi]; }
     }
   }
@@ -272,52 +312,63 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attn_partial_kernel(const Attn
     float L = 0.f;
     for (int s = lane; s < eff; s += 32) {
       const float2 ml = __ldcg(reinterpret_cast<const float2*>(p.ml_part + (s * sstride + r) * 2));
-      L += ml.y * __expf(ml.x - M);
+      L += ml.y * att_exp<PRECISE>(ml.x - M);
     }
-    L = warp_sum(L) + (p.sinks ? __expf(p.sinks[hq] - M) : 0.f);
+    L = warp_sum(L) + (p.sinks ? att_exp<PRECISE>(p.sinks[hq] - M) : 0.f);
     const float inv = L > 0.f ? 1.f / L : 0.f;
     float acc[HD / 32];
 #pragma unroll
     for (int c = 0; c < HD / 32; ++c) acc[c] = 0.f;
     for (int s0 = 0; s0 < eff; s0 += 32) {
-      const float sc_l = s0 + lane < eff ? __expf(__ldcg(p.ml_part + ((s0 + lane) * sstride + r) * 2) - M) : 0.f;
+      const float sc_l = s0 + lane < eff ? att_exp<PRECISE>(__ldcg(p.ml_part + ((s0 + lane) * sstride + r) * 2) - M) : 0.f;
       const int cnt = min(32, eff - s0);
 #pragma unroll 4
       for (int j = 0; j < cnt; ++j) {
         const float sc = __shfl_sync(0xffffffffu, sc_l, j);
-        const float* op = p.o_part + ((s0 + j) * sstride + r) * HD;
+        const float* op = p.o_part + ((s0 + j) * sstride + r) * DV;
 #pragma unroll
-        for (int c = 0; c < HD / 32; ++c) acc[c] = fmaf(__ldcg(op + lane + 32 * c), sc, acc[c]);
+        for (int c = 0; c < HD / 32; ++c)
+          if (EXACT || lane + 32 * c < DV) acc[c] = fmaf(__ldcg(op + lane + 32 * c), sc, acc[c]);
       }
     }
 #pragma unroll
-    for (int c = 0; c < HD / 32; ++c) p.out[r * HD + lane + 32 * c] = __float2bfloat16(acc[c] * inv);
+    for (int c = 0; c < HD / 32; ++c) {
+      const int d = lane + 32 * c;
+      if (!EXACT && d >= DV) continue;
+      float o = acc[c] * inv;
+      if (p.gate) o *= sigmoid_f<PRECISE>(to_f32(reinterpret_cast<const T*>(p.gate)[(size_t)(q_begin + t0 + tq) * p.gate_ld + (size_t)hq * DV + d]));
+      reinterpret_cast<T*>(p.out)[r * DV + d] = from_f32<T>(o);
+    }
   }
 }
 
-// out[t][h][:] = sum_s acc_s e^{m_s - M} / (sum_s l_s e^{m_s - M} + e^{sink_h - M})
+// out[t][h][:] = sum_s acc_s e^{m_s - M} / (sum_s l_s e^{m_s - M} + e^{sink_h - M}) [* sigmoid(gate)]
+template <typename T>
 __global__ void __launch_bounds__(128) attn_combine_kernel(const float* __restrict__ o_part, const float* __restrict__ ml_part,
-                                                           const float* __restrict__ sinks, __nv_bfloat16* __restrict__ out, int Tq, int n_q,
-                                                           int hd, int n_splits) {
+                                                           const float* __restrict__ sinks, const T* __restrict__ gate, int gate_ld, T* __restrict__ out,
+                                                           int Tq, int n_q, int hd, int n_splits) {
+  constexpr bool PRECISE = sizeof(T) == 4;
   pdl_prologue();
   const int r = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (r >= Tq * n_q) return;
   const int h = r % n_q;
   float M = sinks ? sinks[h] : -1e30f;
   for (int s = 0; s < n_splits; ++s) M = fmaxf(M, ml_part[((size_t)s * Tq * n_q + r) * 2]);
-  float L = sinks ? __expf(sinks[h] - M) : 0.f;
+  float L = sinks ? att_exp<PRECISE>(sinks[h] - M) : 0.f;
   for (int s = 0; s < n_splits; ++s) {
     const float* ml = ml_part + ((size_t)s * Tq * n_q + r) * 2;
-    L += ml[1] * __expf(ml[0] - M);
+    L += ml[1] * att_exp<PRECISE>(ml[0] - M);
   }
   const float inv = L > 0.f ? 1.f / L : 0.f;
   for (int d = lane; d < hd; d += 32) {
     float a = 0.f;
     for (int s = 0; s < n_splits; ++s) {
       const size_t row = (size_t)s * Tq * n_q + r;
-      a += o_part[row * hd + d] * __expf(ml_part[row * 2] - M);
+      a += o_part[row * hd + d] * att_exp<PRECISE>(ml_part[row * 2] - M);
     }
-    out[(size_t)r * hd + d] = __float2bfloat16(a * inv);
+    a *= inv;
+    if (gate) a *= sigmoid_f<PRECISE>(to_f32(gate[(size_t)(r / n_q) * gate_ld + (size_t)h * hd + d]));
+    out[(size_t)r * hd + d] = from_f32<T>(a);
   }
 }
 
@@ -327,14 +378,16 @@ __global__ void __launch_bounds__(128) attn_combine_kernel(const float* __restri
 constexpr int ATT_TICKET_SLOTS = 8, ATT_TICKETS_PER_SLOT = 2048;
 static __device__ int g_attn_tickets[ATT_TICKET_SLOTS * ATT_TICKETS_PER_SLOT];
 
-template <int HD, int PPW>
+template <typename T, int HD, int PPW, bool EXACT>
 static int launch_partial(const AttnParams& p, cudaStream_t st) {
   constexpr int PAIRS = ATT_WARPS * PPW;
-  const size_t smem = (size_t)PAIRS * HD * 4 + (size_t)ATT_TILE * (HD + 2) * 2 + (size_t)ATT_TILE * HD * 2;
-  auto kern = attn_partial_kernel<HD, PPW>;
+  constexpr size_t SMEM_MAX = 227 * 1024;
+  const size_t smem = (size_t)PAIRS * p.dk * 4 + (size_t)ATT_TILE * (p.dk + att_kpad<T>()) * sizeof(T) + (size_t)ATT_TILE * p.dv * sizeof(T);
+  if (smem > SMEM_MAX) return -112;
+  auto kern = attn_partial_kernel<T, HD, PPW, EXACT>;
   static DeviceOnce configured;
   if (configured.pending()) {
-    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, EXACT ? (int)smem : (int)SMEM_MAX);
     if (e != cudaSuccess) return (int)e;
     configured.mark();
   }
@@ -365,23 +418,32 @@ MX_HOST_API int mx_attention_launches(int B, int max_q_len, int n_q, int n_kv) {
 
 // Scratch: o_part needs n_splits*Tq*n_q*hd floats, ml_part n_splits*Tq*n_q*2 floats.
 // max_q_len is the longest query segment of the batch (host knows it from cu_q).
+struct AttnShape {            // what the plain entry points leave at its default
+  int dk, dv, q_ld;           // q_ld: elements between the query rows
+  const void* gate = nullptr;
+  int gate_ld = 0;
+  const float* q_scale = nullptr;
+  int q_scale_n = 0;
+  int elem_f32 = 0;           // queries, cache, gate and output in fp32
+};
 static int attention_impl(const void* q, const void* k_cache, const void* v_cache, const float* k_scale, const float* v_scale,
                           const int* block_table, const int* seq_lens, const int* cu_q, const float* sinks, void* out, float* o_part,
-                          float* ml_part, int B, int Tq, int max_q_len, int n_q, int n_kv, int hd, int max_blocks, int block_size, int window,
-                          float scale, float softcap, int n_splits, cudaStream_t st) {
+                          float* ml_part, int B, int Tq, int max_q_len, int n_q, int n_kv, const AttnShape& sh, int max_blocks, int block_size,
+                          int window, float scale, float softcap, int n_splits, cudaStream_t st) {
   if (B <= 0 || Tq <= 0) return 0;
   if (block_size % ATT_TILE) return -110;
   if (n_q % n_kv) return -111;
   const int gqa = n_q / n_kv;
   AttnParams p;
-  p.q = (const __nv_bfloat16*)q; p.k_cache = (const __nv_bfloat16*)k_cache; p.v_cache = (const __nv_bfloat16*)v_cache;
+  p.q = q; p.k_cache = k_cache; p.v_cache = v_cache;
+  p.dk = sh.dk; p.dv = sh.dv; p.q_ld = sh.q_ld; p.gate = sh.gate; p.gate_ld = sh.gate_ld; p.q_scale = sh.q_scale; p.q_scale_n = sh.q_scale_n;
   p.k_scale = k_scale; p.v_scale = k_scale ? v_scale : nullptr;
   p.block_table = block_table; p.seq_lens = seq_lens; p.cu_q = cu_q; p.o_part = o_part; p.ml_part = ml_part;
   p.B = B; p.n_q = n_q; p.n_kv = n_kv; p.max_blocks = max_blocks; p.block_size = block_size;
   p.n_splits = n_splits < 1 ? 1 : n_splits; p.Tq = Tq; p.window = window; p.scale = scale; p.softcap = softcap;
   int ppw;
   att_tiling(max_q_len, gqa, ppw, p.q_tile, p.max_q_tiles);
-  p.tickets = nullptr; p.sinks = sinks; p.out = (__nv_bfloat16*)out;
+  p.tickets = nullptr; p.sinks = sinks; p.out = out;
   const long long groups = (long long)B * p.max_q_tiles * n_kv;
   if (groups <= ATT_TICKETS_PER_SLOT) {
     static int* base[64] = {nullptr};
@@ -397,19 +459,54 @@ static int attention_impl(const void* q, const void* k_cache, const void* v_cach
     p.tickets = base[dev] + (size_t)(turn[dev]++ % ATT_TICKET_SLOTS) * ATT_TICKETS_PER_SLOT;
   }
   int rc;
-#define MX_ATT(HD_)                                                        \
-  (ppw == 4 ? launch_partial<HD_, 4>(p, st) : ppw == 2 ? launch_partial<HD_, 2>(p, st) : launch_partial<HD_, 1>(p, st))
-  switch (hd) {
-    case 64: rc = MX_ATT(64); break;
-    case 128: rc = MX_ATT(128); break;
-    case 256: rc = MX_ATT(256); break;
-    case 512: rc = MX_ATT(512); break;      // Gemma-4 global layers
-    default: return -112;
+#define MX_ATT(T_, HD_, EX_) \
+  (ppw == 4 ? launch_partial<T_, HD_, 4, EX_>(p, st) : ppw == 2 ? launch_partial<T_, HD_, 2, EX_>(p, st) : launch_partial<T_, HD_, 1, EX_>(p, st))
+  const int dk = sh.dk, dv = sh.dv, ve = sh.elem_f32 ? 4 : 8;
+  if (dk < 1 || dv < 1 || dk > 512 || dv > 512 || dk % ve || dv % ve) return -112;
+  if (!sh.elem_f32 && dk == dv && (dk == 64 || dk == 128 || dk == 256 || dk == 512)) {
+    switch (dk) {
+      case 64: rc = MX_ATT(__nv_bfloat16, 64, true); break;
+      case 128: rc = MX_ATT(__nv_bfloat16, 128, true); break;
+      case 256: rc = MX_ATT(__nv_bfloat16, 256, true); break;
+      default: rc = MX_ATT(__nv_bfloat16, 512, true); break;      // Gemma-4 global layers
+    }
+  } else if (k_scale) {
+    return -112;                                                  // int8 rows: instances with fixed widths only
+  } else if (sh.elem_f32) {
+    rc = dv <= 64 ? MX_ATT(float, 64, false) : dv <= 128 ? MX_ATT(float, 128, false) : dv <= 256 ? MX_ATT(float, 256, false) : MX_ATT(float, 512, false);
+  } else {
+    rc = dv <= 64 ? MX_ATT(__nv_bfloat16, 64, false) : dv <= 128 ? MX_ATT(__nv_bfloat16, 128, false)
+         : dv <= 256 ? MX_ATT(__nv_bfloat16, 256, false) : MX_ATT(__nv_bfloat16, 512, false);
   }
 #undef MX_ATT
   if (rc || p.tickets) return rc;
-  launch_pdl(attn_combine_kernel, dim3((Tq * n_q + 3) / 4), dim3(128), 0, st, o_part, ml_part, sinks, (__nv_bfloat16*)out, Tq, n_q, hd, p.n_splits);
+  const dim3 cgrid((Tq * n_q + 3) / 4);
+  if (sh.elem_f32)
+    launch_pdl(attn_combine_kernel<float>, cgrid, dim3(128), 0, st, o_part, ml_part, sinks, (const float*)sh.gate, sh.gate_ld, (float*)out, Tq, n_q, dv, p.n_splits);
+  else
+    launch_pdl(attn_combine_kernel<__nv_bfloat16>, cgrid, dim3(128), 0, st, o_part, ml_part, sinks, (const __nv_bfloat16*)sh.gate, sh.gate_ld,
+               (__nv_bfloat16*)out, Tq, n_q, dv, p.n_splits);
   return (int)cudaGetLastError();
+}
+
+static AttnShape plain_shape(int n_q, int hd) {
+  AttnShape sh;
+  sh.dk = sh.dv = hd;
+  sh.q_ld = n_q * hd;
+  return sh;
+}
+
+// Queries [Tq] rows of [n_q][dk] (q_ld elements apart), cache pages of dk- / dv-wide rows, out [Tq][n_q][dv]; optional gate (rows of
+// [n_q][dv], gate_ld apart; out *= sigmoid(gate)) and per-position score factors q_scale [q_scale_n].  elem_f32: everything in fp32.
+// o_part needs n_splits*Tq*n_q*dv floats.  Rows, widths and strides are multiples of 16 bytes.
+MX_HOST_API int mx_attention_ext(const void* q, int q_ld, const void* k_cache, const void* v_cache, const int* block_table, const int* seq_lens,
+                                 const int* cu_q, const float* sinks, const void* gate, int gate_ld, const float* q_scale, int q_scale_n, void* out,
+                                 float* o_part, float* ml_part, int B, int Tq, int max_q_len, int n_q, int n_kv, int dk, int dv, int max_blocks,
+                                 int block_size, int window, float scale, float softcap, int n_splits, int elem_f32, cudaStream_t st) {
+  AttnShape sh;
+  sh.dk = dk; sh.dv = dv; sh.q_ld = q_ld; sh.gate = gate; sh.gate_ld = gate_ld; sh.q_scale = q_scale; sh.q_scale_n = q_scale_n; sh.elem_f32 = elem_f32;
+  return attention_impl(q, k_cache, v_cache, nullptr, nullptr, block_table, seq_lens, cu_q, sinks, out, o_part, ml_part, B, Tq, max_q_len, n_q, n_kv,
+                        sh, max_blocks, block_size, window, scale, softcap, n_splits, st);
 }
 
 MX_HOST_API int mx_attention(const void* q, const void* k_cache, const void* v_cache, const int* block_table, const int* seq_lens,
@@ -417,7 +514,7 @@ MX_HOST_API int mx_attention(const void* q, const void* k_cache, const void* v_c
                              int n_q, int n_kv, int hd, int max_blocks, int block_size, int window, float scale, float softcap,
                              int n_splits, cudaStream_t st) {
   return attention_impl(q, k_cache, v_cache, nullptr, nullptr, block_table, seq_lens, cu_q, sinks, out, o_part, ml_part, B, Tq, max_q_len, n_q,
-                        n_kv, hd, max_blocks, block_size, window, scale, softcap, n_splits, st);
+                        n_kv, plain_shape(n_q, hd), max_blocks, block_size, window, scale, softcap, n_splits, st);
 }
 
 // The same over an int8 cache with per-row scales (see the layout note at the top of this file).
@@ -427,7 +524,7 @@ MX_HOST_API int mx_attention_kv8(const void* q, const void* k_cache, const void*
                                  int window, float scale, float softcap, int n_splits, cudaStream_t st) {
   if (!k_scale || !v_scale) return -113;
   return attention_impl(q, k_cache, v_cache, k_scale, v_scale, block_table, seq_lens, cu_q, sinks, out, o_part, ml_part, B, Tq, max_q_len, n_q,
-                        n_kv, hd, max_blocks, block_size, window, scale, softcap, n_splits, st);
+                        n_kv, plain_shape(n_q, hd), max_blocks, block_size, window, scale, softcap, n_splits, st);
 }
 
 // dst_k / dst_v: bf16 [B * nb][n_kv][block_size][hd]; page (b, j) is filled when j * block_size < seq_lens[b].

@@ -1,5 +1,7 @@
-// Prefill FlashAttention on the sm_100a tensor cores: head_dim 64, 128 or 256, paged KV, causal, sliding window with
-// whole-tile skipping, attention sinks, logit soft-cap, GQA.
+// Prefill FlashAttention on the sm_100a tensor cores: paged KV, causal, sliding window with whole-tile skipping, attention sinks,
+// logit soft-cap, GQA, score factors per query position (query temperature), sigmoid output gate.  Keys and values may have different
+// widths (multiples of 8 up to 256): the shared tiles are 64 / 128 / 256 columns wide and the tensor maps, whose rows end at the real
+// width, fill the rest with zeros, so the cache itself is not padded.
 //
 // One CTA owns 128 query tokens of one query head and walks the key tiles of its range (128 keys per tile, 64 for
 // head_dim 256 so that two K and two V tiles still fit in shared memory):
@@ -16,6 +18,7 @@
 // Reference parity: src/ops/attention.cpp:2456-2815 (fa2_tile_wide_impl<HD,Bc,REGDOT,SG,SINK> for HD 64..512 and its
 // dispatcher: causal and window masks per key, whole-tile skip outside the window, sink folded at row end); the soft-cap
 // of src/model/gemma4.cpp's attention is applied to the scores here.
+#include "act.cuh"
 #include "common.cuh"
 #include "host_util.h"
 
@@ -29,31 +32,34 @@ struct FaParams {
   const int* seq_lens;     // [B]
   const int* cu_q;         // [B+1]
   const float* sinks;      // [n_q] or null
-  __nv_bfloat16* out;      // [Tq][n_q][hd]
+  const float* q_scale;    // [q_scale_n] factor on the scores of a query at that position, or null
+  const __nv_bfloat16* gate;   // out *= sigmoid(gate): [Tq] rows of [n_q][dv], gate_ld elements apart, or null
+  __nv_bfloat16* out;      // [Tq][n_q][dv]
+  int q_scale_n, gate_ld, dk, dv, q_ld;
   int n_q, n_kv, max_blocks, max_q_tiles, window;
   float scale, softcap;
   int* status;
 };
 
-template <int HD>
+template <int DK, int DV>
 struct FaCfg {
-  static constexpr int BKV = HD <= 128 ? 128 : 64;            // keys per tile
+  static constexpr int BKV = (DK <= 128 && DV <= 128) ? 128 : 64;   // keys per tile
   static constexpr int NS = 2;                                 // S buffers in TMEM
   static constexpr int CTAS = 1;                               // one CTA per SM: its softmax threads keep a whole S row in registers
   static constexpr uint32_t TMEM_COLS = 512;
-  static constexpr int ATOMS = HD / 64;                        // 64-column (128-byte) swizzle atoms per row of Q / K / V
-  static constexpr int Q_BYTES = FA_BQ * HD * 2;
-  static constexpr int KV_BYTES = BKV * HD * 2;
+  static constexpr int KATOMS = DK / 64, VATOMS = DV / 64;     // 64-column (128-byte) swizzle atoms per row of Q / K and of V
+  static constexpr int Q_BYTES = FA_BQ * DK * 2;
+  static constexpr int K_BYTES = BKV * DK * 2, V_BYTES = BKV * DV * 2;
   static constexpr int KS = 2, VS = 2;                         // tiles in flight
   static constexpr int P_BYTES = FA_BQ * BKV * 2;
   static constexpr int Q_OFF = 0;
   static constexpr int K_OFF = Q_OFF + Q_BYTES;
-  static constexpr int V_OFF = K_OFF + KS * KV_BYTES;
-  static constexpr int P_OFF = V_OFF + VS * KV_BYTES;
+  static constexpr int V_OFF = K_OFF + KS * K_BYTES;
+  static constexpr int P_OFF = V_OFF + VS * V_BYTES;
   static constexpr int BAR_OFF = P_OFF + P_BYTES;
   static constexpr int TOTAL = BAR_OFF + 256 + 1024;
   static_assert(TOTAL <= 232448, "shared memory plan exceeds 227 KB");
-  static_assert(NS * BKV + HD <= (int)TMEM_COLS, "TMEM plan");
+  static_assert(NS * BKV + DV <= (int)TMEM_COLS, "TMEM plan");
 };
 
 __device__ __forceinline__ void tmem_st_32x32(uint32_t taddr, const uint32_t (&r)[32]) {
@@ -79,11 +85,11 @@ __device__ __forceinline__ float ex2_fast(float x) {
   return y;
 }
 
-template <int HD, bool CAP>
-__global__ void __launch_bounds__(192, FaCfg<HD>::CTAS)
+template <int DK, int DV, bool CAP>
+__global__ void __launch_bounds__(192, FaCfg<DK, DV>::CTAS)
 fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                   const __grid_constant__ CUtensorMap tmap_v, const FaParams p) {
-  using L = FaCfg<HD>;
+  using L = FaCfg<DK, DV>;
   constexpr int BKV = L::BKV, NS = L::NS, KS = L::KS, VS = L::VS;
   constexpr float LOG2E = 1.4426950408889634f;
   constexpr float RESCALE_STEP = 8.f;            // in log2 units: O is rescaled when the maximum has grown by a factor of 256
@@ -134,7 +140,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       prefetch_tmap(&tmap_q); prefetch_tmap(&tmap_k); prefetch_tmap(&tmap_v);
       mbar_expect_tx(b_qfull, L::Q_BYTES);
 #pragma unroll
-      for (int a = 0; a < L::ATOMS; ++a)
+      for (int a = 0; a < L::KATOMS; ++a)
         tma_load_3d(sbase + L::Q_OFF + a * (FA_BQ * 128), &tmap_q, b_qfull, a * 64, head, q_begin + t0);
       bool ok = true;
       for (int j = 0; j < n_tiles && ok; ++j) {
@@ -143,21 +149,21 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         const int blk = p.block_table[(size_t)b * p.max_blocks + key0 / FA_PAGE];
         const int krow = key0 % FA_PAGE;
         if (!(ok = mbar_wait(b_kempty + 8 * sk, phk ^ 1, p.status, ERR_MBAR_TIMEOUT_PRODUCER, abort_flag))) break;
-        mbar_expect_tx(b_kfull + 8 * sk, L::KV_BYTES);
+        mbar_expect_tx(b_kfull + 8 * sk, L::K_BYTES);
 #pragma unroll
-        for (int a = 0; a < L::ATOMS; ++a)
-          tma_load_4d(sbase + L::K_OFF + sk * L::KV_BYTES + a * (BKV * 128), &tmap_k, b_kfull + 8 * sk, a * 64, krow, kvh, blk);
+        for (int a = 0; a < L::KATOMS; ++a)
+          tma_load_4d(sbase + L::K_OFF + sk * L::K_BYTES + a * (BKV * 128), &tmap_k, b_kfull + 8 * sk, a * 64, krow, kvh, blk);
         if (!(ok = mbar_wait(b_vempty + 8 * sv, phv ^ 1, p.status, ERR_MBAR_TIMEOUT_PRODUCER, abort_flag))) break;
-        mbar_expect_tx(b_vfull + 8 * sv, L::KV_BYTES);
+        mbar_expect_tx(b_vfull + 8 * sv, L::V_BYTES);
 #pragma unroll
-        for (int a = 0; a < L::ATOMS; ++a)
-          tma_load_4d(sbase + L::V_OFF + sv * L::KV_BYTES + a * (BKV * 128), &tmap_v, b_vfull + 8 * sv, a * 64, krow, kvh, blk);
+        for (int a = 0; a < L::VATOMS; ++a)
+          tma_load_4d(sbase + L::V_OFF + sv * L::V_BYTES + a * (BKV * 128), &tmap_v, b_vfull + 8 * sv, a * 64, krow, kvh, blk);
       }
     }
   } else if (warp == 1) {
     if (lane == 0) {
       constexpr uint32_t idesc_s = umma_idesc_bf16(FA_BQ, BKV, 0, 0);
-      constexpr uint32_t idesc_o = umma_idesc_bf16(FA_BQ, HD, 0, 1);      // B = V is MN-major (head_dim contiguous)
+      constexpr uint32_t idesc_o = umma_idesc_bf16(FA_BQ, DV, 0, 1);      // B = V is MN-major (head_dim contiguous)
       bool ok = mbar_wait(b_qfull, 0, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag);
       // S(j) = Q K_j^T into S buffer j % NS (waits for K_j and for the softmax threads to have released that buffer)
       auto issue_s = [&](int j) -> bool {
@@ -165,9 +171,9 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         if (!mbar_wait(b_kfull + 8 * sk, phk, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag)) return false;
         if (!mbar_wait(b_sempty + 8 * sb, phs ^ 1, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag)) return false;
         tc_fence_after();
-        const uint32_t qa = sbase + L::Q_OFF, ka = sbase + L::K_OFF + sk * L::KV_BYTES;
+        const uint32_t qa = sbase + L::Q_OFF, ka = sbase + L::K_OFF + sk * L::K_BYTES;
 #pragma unroll
-        for (int kk = 0; kk < HD / 16; ++kk) {
+        for (int kk = 0; kk < DK / 16; ++kk) {
           const uint64_t ad = umma_desc_k_sw128(qa + (kk >> 2) * (FA_BQ * 128) + (kk & 3) * 32);
           const uint64_t bd = umma_desc_k_sw128(ka + (kk >> 2) * (BKV * 128) + (kk & 3) * 32);
           umma_bf16(tmem_base + sb * BKV, ad, bd, idesc_s, kk != 0);
@@ -183,7 +189,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         if (!(ok = mbar_wait(b_pfull, j & 1, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag))) break;
         if (!(ok = mbar_wait(b_vfull + 8 * sv, phv, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag))) break;
         tc_fence_after();
-        const uint32_t pa = sbase + L::P_OFF, va = sbase + L::V_OFF + sv * L::KV_BYTES;
+        const uint32_t pa = sbase + L::P_OFF, va = sbase + L::V_OFF + sv * L::V_BYTES;
 #pragma unroll
         for (int kk = 0; kk < BKV / 16; ++kk) {
           const uint64_t ad = umma_desc_k_sw128(pa + (kk >> 2) * (FA_BQ * 128) + (kk & 3) * 32);
@@ -203,8 +209,12 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     const int r = q4 * 32 + lane;                  // row inside the tile == TMEM lane
     const int qpos = pos0 + r;
     const bool row_ok = r < rows;
-    const float c = CAP ? 1.f : p.scale * LOG2E;   // factor from the stored score to log2 units
-    const float cap_c = p.softcap * LOG2E, inv_cap = CAP ? p.scale / p.softcap : 0.f;
+    const float qs = p.scale * (p.q_scale ? p.q_scale[min(qpos, p.q_scale_n - 1)] : 1.f);
+    // c: factor from the stored score to log2 units, applied after the maximum.  That needs c > 0: a row whose factor is not (a
+    // temperature law may change sign) multiplies its scores first and goes on with 1.
+    const bool early = !CAP && !(qs > 0.f);
+    const float c = (CAP || early) ? 1.f : qs * LOG2E;
+    const float cap_c = p.softcap * LOG2E, inv_cap = CAP ? qs / p.softcap : 0.f;
     float m = -1e30f, l = 0.f;                     // reference maximum (log2 units) and running denominator
     const uint32_t lane_addr = (uint32_t)(q4 * 32) << 16;
     bool ok = true;
@@ -224,6 +234,9 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       if (CAP) {
 #pragma unroll
         for (int i = 0; i < BKV; ++i) sv[i] = cap_c * tanh_fast(sv[i] * inv_cap);
+      } else if (early) {
+#pragma unroll
+        for (int i = 0; i < BKV; ++i) sv[i] *= qs * LOG2E;
       }
       // a tile needs per-key masking only at the diagonal, at the window edge and at the sequence end
       if ((key0 + BKV - 1 > pos0) || (p.window > 0 && key0 <= pos0 + FA_BQ - 1 - p.window) || (key0 + BKV > seq_len)) {
@@ -249,7 +262,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         l *= alpha;
         tc_fence_after();
 #pragma unroll 1
-        for (int cb = 0; cb < HD; cb += 32) {
+        for (int cb = 0; cb < DV; cb += 32) {
           uint32_t ov[32];
           tmem_ld_32x32(tmem_o + lane_addr + cb, ov);
           tmem_ld_wait();
@@ -289,9 +302,11 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       tc_fence_after();
       if (p.sinks) l += ex2_fast(p.sinks[head] * LOG2E - m);
       const float inv = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* orow = p.out + ((size_t)(q_begin + t0 + r) * p.n_q + head) * HD;
+      const int dv = p.dv;
+      __nv_bfloat16* orow = p.out + ((size_t)(q_begin + t0 + r) * p.n_q + head) * dv;
+      const __nv_bfloat16* grow = p.gate ? p.gate + (size_t)(q_begin + t0 + r) * p.gate_ld + (size_t)head * dv : nullptr;
 #pragma unroll 1
-      for (int cb = 0; cb < HD; cb += 32) {
+      for (int cb = 0; cb < DV; cb += 32) {
         uint32_t ov[32];
         if (n_tiles > 0) {
           tmem_ld_32x32(tmem_o + lane_addr + cb, ov);
@@ -302,10 +317,22 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         }
         if (row_ok) {
 #pragma unroll
-          for (int i = 0; i < 32; i += 8)
-            *reinterpret_cast<uint4*>(orow + cb + i) =
-                make_uint4(pack_bf16(__uint_as_float(ov[i]) * inv, __uint_as_float(ov[i + 1]) * inv), pack_bf16(__uint_as_float(ov[i + 2]) * inv, __uint_as_float(ov[i + 3]) * inv),
-                           pack_bf16(__uint_as_float(ov[i + 4]) * inv, __uint_as_float(ov[i + 5]) * inv), pack_bf16(__uint_as_float(ov[i + 6]) * inv, __uint_as_float(ov[i + 7]) * inv));
+          for (int i = 0; i < 32; i += 8) {
+            if (cb + i >= dv) break;
+            float o[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) o[e] = __uint_as_float(ov[i + e]) * inv;
+            if (grow) {
+              const uint4 g4 = *reinterpret_cast<const uint4*>(grow + cb + i);
+              const uint32_t gw[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                o[2 * e] *= sigmoid_f<false>(bf16_lo(gw[e]));
+                o[2 * e + 1] *= sigmoid_f<false>(bf16_hi(gw[e]));
+              }
+            }
+            *reinterpret_cast<uint4*>(orow + cb + i) = make_uint4(pack_bf16(o[0], o[1]), pack_bf16(o[2], o[3]), pack_bf16(o[4], o[5]), pack_bf16(o[6], o[7]));
+          }
         }
       }
     }
@@ -319,27 +346,30 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
   if (warp == 1) tmem_dealloc(tmem_base, L::TMEM_COLS);
 }
 
-template <int HD, bool CAP>
+template <int DK, int DV, bool CAP>
 static int launch_fa(const void* q, const void* k_cache, const void* v_cache, const FaParams& p, int B, int Tq, int n_blocks, cudaStream_t st) {
-  using L = FaCfg<HD>;
+  using L = FaCfg<DK, DV>;
   CUtensorMap tq, tk, tv;
   {
-    uint64_t dims[3] = {(uint64_t)HD, (uint64_t)p.n_q, (uint64_t)Tq};
-    uint64_t strides[2] = {(uint64_t)HD * 2, (uint64_t)HD * 2 * p.n_q};
+    uint64_t dims[3] = {(uint64_t)p.dk, (uint64_t)p.n_q, (uint64_t)Tq};
+    uint64_t strides[2] = {(uint64_t)p.dk * 2, (uint64_t)p.q_ld * 2};
     uint32_t box[3] = {64, 1, FA_BQ};
     int r = make_tmap_bf16(&tq, q, 3, dims, strides, box, 1);
     if (r) return r;
   }
   {
-    uint64_t dims[4] = {(uint64_t)HD, (uint64_t)FA_PAGE, (uint64_t)p.n_kv, (uint64_t)n_blocks};
-    uint64_t strides[3] = {(uint64_t)HD * 2, (uint64_t)HD * 2 * FA_PAGE, (uint64_t)HD * 2 * FA_PAGE * p.n_kv};
-    uint32_t box[4] = {64, (uint32_t)L::BKV, 1, 1};
-    int r = make_tmap_bf16(&tk, k_cache, 4, dims, strides, box, 1);
+    auto page_map = [&](CUtensorMap* m, const void* base, uint64_t d) {
+      uint64_t dims[4] = {d, (uint64_t)FA_PAGE, (uint64_t)p.n_kv, (uint64_t)n_blocks};
+      uint64_t strides[3] = {d * 2, d * 2 * FA_PAGE, d * 2 * FA_PAGE * p.n_kv};
+      uint32_t box[4] = {64, (uint32_t)L::BKV, 1, 1};
+      return make_tmap_bf16(m, base, 4, dims, strides, box, 1);
+    };
+    int r = page_map(&tk, k_cache, (uint64_t)p.dk);
     if (r) return r;
-    r = make_tmap_bf16(&tv, v_cache, 4, dims, strides, box, 1);
+    r = page_map(&tv, v_cache, (uint64_t)p.dv);
     if (r) return r;
   }
-  auto kern = fa_prefill_kernel<HD, CAP>;
+  auto kern = fa_prefill_kernel<DK, DV, CAP>;
   static DeviceOnce configured;
   if (configured.pending()) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
@@ -351,27 +381,61 @@ static int launch_fa(const void* q, const void* k_cache, const void* v_cache, co
   return (int)cudaGetLastError();
 }
 
+// the instance whose tiles are the key / value widths rounded up to 64, 128 or 256 columns
+static int dispatch_fa(const void* q, const void* k_cache, const void* v_cache, const FaParams& p, int B, int Tq, int n_blocks, cudaStream_t st) {
+  if (p.dk < 8 || p.dv < 8 || p.dk > 256 || p.dv > 256 || p.dk % 8 || p.dv % 8 || p.q_ld % 8 || p.gate_ld % 8) return -112;
+  if (p.gate && ((uintptr_t)p.gate & 15)) return -112;
+  const int a = p.dk <= 64 ? 64 : p.dk <= 128 ? 128 : 256, b = p.dv <= 64 ? 64 : p.dv <= 128 ? 128 : 256;
+#define MX_FA(DK_, DV_, CAP_) launch_fa<DK_, DV_, CAP_>(q, k_cache, v_cache, p, B, Tq, n_blocks, st)
+  if (p.softcap > 0.f) {
+    if (a != b) return -112;
+    return a == 64 ? MX_FA(64, 64, true) : a == 128 ? MX_FA(128, 128, true) : MX_FA(256, 256, true);
+  }
+  switch (a * 1000 + b) {
+    case 64064: return MX_FA(64, 64, false);
+    case 64128: return MX_FA(64, 128, false);
+    case 64256: return MX_FA(64, 256, false);
+    case 128064: return MX_FA(128, 64, false);
+    case 128128: return MX_FA(128, 128, false);
+    case 128256: return MX_FA(128, 256, false);
+    case 256064: return MX_FA(256, 64, false);
+    case 256128: return MX_FA(256, 128, false);
+    default: return MX_FA(256, 256, false);
+  }
+#undef MX_FA
+}
+
 }  // namespace mx
 
 using namespace mx;
 
-// Tensor-core prefill attention.  Requirements: head_dim 64, 128 or 256, KV page size 128.  softcap > 0 applies
-// cap * tanh(score / cap) to the scaled scores.  n_blocks is the number of pages in the cache tensors (their leading dimension).
-MX_HOST_API int mx_attention_prefill_tc(const void* q, const void* k_cache, const void* v_cache, const int* block_table, const int* seq_lens,
-                                        const int* cu_q, const float* sinks, void* out, int B, int Tq, int max_q_len, int n_q, int n_kv,
-                                        int hd, int max_blocks, int n_blocks, int block_size, int window, float scale, float softcap,
-                                        cudaStream_t st) {
+// Tensor-core prefill attention over pages of 128 tokens.  Queries: [Tq] rows of [n_q][dk], q_ld elements apart; out [Tq][n_q][dv];
+// optional gate (rows of [n_q][dv], gate_ld apart; out *= sigmoid(gate)) and per-position score factors q_scale [q_scale_n].  softcap > 0
+// applies cap * tanh(score / cap) to the scaled scores.  n_blocks is the number of pages in the cache tensors (their leading dimension).
+MX_HOST_API int mx_attention_prefill_tc_ext(const void* q, int q_ld, const void* k_cache, const void* v_cache, const int* block_table,
+                                            const int* seq_lens, const int* cu_q, const float* sinks, const void* gate, int gate_ld,
+                                            const float* q_scale, int q_scale_n, void* out, int B, int Tq, int max_q_len, int n_q, int n_kv, int dk,
+                                            int dv, int max_blocks, int n_blocks, int block_size, int window, float scale, float softcap,
+                                            cudaStream_t st) {
   if (B <= 0 || Tq <= 0) return 0;
   if (block_size != FA_PAGE) return -110;
   if (n_q % n_kv) return -111;
   FaParams p;
   p.block_table = block_table; p.seq_lens = seq_lens; p.cu_q = cu_q; p.sinks = sinks; p.out = (__nv_bfloat16*)out;
+  p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate ? gate_ld : 0; p.q_scale = q_scale; p.q_scale_n = q_scale_n;
+  p.dk = dk; p.dv = dv; p.q_ld = q_ld;
   p.n_q = n_q; p.n_kv = n_kv; p.max_blocks = max_blocks; p.window = window; p.scale = scale; p.softcap = softcap;
   p.max_q_tiles = (max_q_len + FA_BQ - 1) / FA_BQ;
   p.status = status_word();
-  const bool cap = softcap > 0.f;
-  if (hd == 64) return cap ? launch_fa<64, true>(q, k_cache, v_cache, p, B, Tq, n_blocks, st) : launch_fa<64, false>(q, k_cache, v_cache, p, B, Tq, n_blocks, st);
-  if (hd == 128) return cap ? launch_fa<128, true>(q, k_cache, v_cache, p, B, Tq, n_blocks, st) : launch_fa<128, false>(q, k_cache, v_cache, p, B, Tq, n_blocks, st);
-  if (hd == 256) return cap ? launch_fa<256, true>(q, k_cache, v_cache, p, B, Tq, n_blocks, st) : launch_fa<256, false>(q, k_cache, v_cache, p, B, Tq, n_blocks, st);
-  return -112;
+  return dispatch_fa(q, k_cache, v_cache, p, B, Tq, n_blocks, st);
+}
+
+// The plain form: dense queries, head_dim 64, 128 or 256 for keys and values.
+MX_HOST_API int mx_attention_prefill_tc(const void* q, const void* k_cache, const void* v_cache, const int* block_table, const int* seq_lens,
+                                        const int* cu_q, const float* sinks, void* out, int B, int Tq, int max_q_len, int n_q, int n_kv,
+                                        int hd, int max_blocks, int n_blocks, int block_size, int window, float scale, float softcap,
+                                        cudaStream_t st) {
+  if (hd != 64 && hd != 128 && hd != 256) return -112;
+  return mx_attention_prefill_tc_ext(q, n_q * hd, k_cache, v_cache, block_table, seq_lens, cu_q, sinks, nullptr, 0, nullptr, 0, out, B, Tq, max_q_len,
+                                     n_q, n_kv, hd, hd, max_blocks, n_blocks, block_size, window, scale, softcap, st);
 }

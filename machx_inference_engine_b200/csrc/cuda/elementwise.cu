@@ -4,10 +4,14 @@
 //   qkv_post        : bias + per-head QK RMSNorm + NEOX RoPE (table driven: llama3 factors and
 //                     YaRN are baked into the cos/sin tables) + Q|gate split + paged KV write
 //   glu             : SwiGLU / clamped OAI SwiGLU / GeGLU over 16-column interleaved gate|up
+//   group_norm      : RMSNorm over equal groups of a row; one pass norms a branch output, adds it to the residual and norms the
+//                     sum for the next branch (norms on both sides of a sublayer)
+//   kv_store        : K / V columns of a projection (own widths, no rotation) into the paged cache
 //   gated_rmsnorm   : y = w * x / rms(x) * silu(z) per head (DeltaNet output norm)
 //   misc            : sigmoid gate multiply, scaled add, casts
 // Reference parity: src/ops/elementwise.cpp:29-786, src/ops/embedding.cpp:45-206,
 // src/core/kv_cache.cpp:107-133, src/ops/deltanet.cpp:41-81.
+#include "act.cuh"
 #include "common.cuh"
 #include "dequant.cuh"
 #include "host_util.h"
@@ -145,6 +149,183 @@ __global__ void __launch_bounds__(256) rmsnorm_combine_kernel(float* __restrict_
     if (one_plus_w) { g.x += 1.f; g.y += 1.f; g.z += 1.f; g.w += 1.f; }
     *reinterpret_cast<uint2*>(out + (size_t)t * H + i) = make_uint2(pack_bf16(v.x * inv * g.x, v.y * inv * g.y), pack_bf16(v.z * inv * g.z, v.w * inv * g.w));
   }
+}
+
+// ------------------------------------------------------------------ group_norm
+// A row of H elements is `groups` equal parts, each normalised by its own root mean square.  In one pass over a row:
+//   x  (fp32 residual) = (FRESH ? 0 : x) + norm(delta) * delta_w      (delta null: x is only read)
+//   out               = norm(x) * w                                   (out null: skipped)
+// Rows have ld elements (ld >= H, multiple of 4); columns H.. are padding: written as zeros in out (and in x when it starts fresh).
+// A team of `wpg` warps owns a group; with more groups than warps the teams (one warp each) walk over them.
+struct GroupNormParams {
+  float* x;
+  const void* delta;
+  const float* delta_w;
+  const float* w;
+  void* out;
+  float eps;
+  int H, ld, groups, gs, wpg, fresh;      // gs = H / groups
+};
+constexpr int GN_WARPS = 8;
+
+// sum over the warps of a team; every warp of the block calls it (barrier) when a team has more than one warp
+__device__ __forceinline__ float team_sum(float v, float* red, int warp, int wpg) {
+  v = warp_sum(v);
+  if (wpg == 1) return v;
+  __syncthreads();                        // readers of the previous use are done
+  if ((threadIdx.x & 31) == 0) red[warp] = v;
+  __syncthreads();
+  const int first = warp - warp % wpg;
+  float t = 0.f;
+  for (int i = 0; i < wpg && first + i < GN_WARPS; ++i) t += red[first + i];
+  return t;
+}
+
+// V elements per access; NV > 0: a lane keeps its NV pieces of x in registers; NV == 0: any size, x is re-read
+template <typename DT, typename OT, int V, int NV>
+__global__ void __launch_bounds__(GN_WARPS * 32) group_norm_kernel(const GroupNormParams p) {
+  pdl_prologue();
+  __shared__ float red[GN_WARPS];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const size_t row = (size_t)blockIdx.x * p.ld;
+  float* xr = p.x + row;
+  const DT* dr = reinterpret_cast<const DT*>(p.delta) + row;
+  OT* orow = reinterpret_cast<OT*>(p.out) + row;
+  const int wpg = p.wpg, teams = GN_WARPS / wpg, team = warp / wpg;
+  const int first = (warp % wpg) * 32 + lane, step = wpg * 32, pieces = p.gs / V;
+  const float inv_n = 1.f / (float)p.gs;
+  for (int g0 = 0; g0 < p.groups; g0 += teams) {
+    const int g = g0 + team;
+    const bool live = team < teams && g < p.groups;        // idle warps still reach the team barriers
+    const int base = g * p.gs, n = live ? pieces : 0;
+    if constexpr (NV > 0) {
+      float xv[NV][V];
+      float ss = 0.f;
+      if (p.delta) {
+        float dv[NV][V];
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+          const int i = first + j * step;
+          if (i < n) {
+            loadv<V>(dr + base + i * V, dv[j]);
+            if (!p.fresh) loadv<V>(xr + base + i * V, xv[j]);
+#pragma unroll
+            for (int e = 0; e < V; ++e) ss = fmaf(dv[j][e], dv[j][e], ss);
+          }
+        }
+        const float dinv = rsqrtf(team_sum(ss, red, warp, wpg) * inv_n + p.eps);
+        ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+          const int i = first + j * step;
+          if (i < n) {
+            float wv[V];
+            loadv<V>(p.delta_w + base + i * V, wv);
+#pragma unroll
+            for (int e = 0; e < V; ++e) {
+              const float add = dv[j][e] * dinv * wv[e];
+              xv[j][e] = p.fresh ? add : xv[j][e] + add;
+              ss = fmaf(xv[j][e], xv[j][e], ss);
+            }
+            storev<V>(xr + base + i * V, xv[j]);
+          }
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+          const int i = first + j * step;
+          if (i < n) {
+            loadv<V>(xr + base + i * V, xv[j]);
+#pragma unroll
+            for (int e = 0; e < V; ++e) ss = fmaf(xv[j][e], xv[j][e], ss);
+          }
+        }
+      }
+      if (p.out) {
+        const float inv = rsqrtf(team_sum(ss, red, warp, wpg) * inv_n + p.eps);
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+          const int i = first + j * step;
+          if (i < n) {
+            float wv[V];
+            loadv<V>(p.w + base + i * V, wv);
+#pragma unroll
+            for (int e = 0; e < V; ++e) wv[e] *= xv[j][e] * inv;
+            storev<V>(orow + base + i * V, wv);
+          }
+        }
+      }
+    } else {
+      float ss = 0.f;
+      if (p.delta) {
+        for (int i = first; i < n; i += step) {
+          float dv[V];
+          loadv<V>(dr + base + i * V, dv);
+#pragma unroll
+          for (int e = 0; e < V; ++e) ss = fmaf(dv[e], dv[e], ss);
+        }
+        const float dinv = rsqrtf(team_sum(ss, red, warp, wpg) * inv_n + p.eps);
+        ss = 0.f;
+        for (int i = first; i < n; i += step) {
+          float dv[V], wv[V], xv[V];
+          loadv<V>(dr + base + i * V, dv);
+          loadv<V>(p.delta_w + base + i * V, wv);
+          if (!p.fresh) loadv<V>(xr + base + i * V, xv);
+#pragma unroll
+          for (int e = 0; e < V; ++e) {
+            const float add = dv[e] * dinv * wv[e];
+            xv[e] = p.fresh ? add : xv[e] + add;
+            ss = fmaf(xv[e], xv[e], ss);
+          }
+          storev<V>(xr + base + i * V, xv);
+        }
+      } else {
+        for (int i = first; i < n; i += step) {
+          float xv[V];
+          loadv<V>(xr + base + i * V, xv);
+#pragma unroll
+          for (int e = 0; e < V; ++e) ss = fmaf(xv[e], xv[e], ss);
+        }
+      }
+      if (p.out) {
+        const float inv = rsqrtf(team_sum(ss, red, warp, wpg) * inv_n + p.eps);
+        for (int i = first; i < n; i += step) {           // a lane reads back the elements it wrote itself
+          float xv[V], wv[V];
+          loadv<V>(xr + base + i * V, xv);
+          loadv<V>(p.w + base + i * V, wv);
+#pragma unroll
+          for (int e = 0; e < V; ++e) wv[e] *= xv[e] * inv;
+          storev<V>(orow + base + i * V, wv);
+        }
+      }
+    }
+  }
+  for (int i = p.H + threadIdx.x; i < p.ld; i += blockDim.x) {
+    if (p.out) orow[i] = from_f32<OT>(0.f);
+    if (p.fresh) xr[i] = 0.f;
+  }
+}
+
+// ------------------------------------------------------------------ kv_store
+// Columns of a projection row ([n_kv][dk] keys, [n_kv][dv] values; any row stride) -> paged cache rows, 16 bytes per thread.
+__global__ void __launch_bounds__(256) kv_store_kernel(const uint4* __restrict__ k, const uint4* __restrict__ v, int k_ld, int v_ld,
+                                                       const long long* __restrict__ slot_map, uint4* __restrict__ k_cache, uint4* __restrict__ v_cache,
+                                                       int T, int n_kv, int pk, int pv, int block_size) {   // pk, pv: 16-byte pieces per row of a head
+  pdl_prologue();
+  const int per_tok = n_kv * (pk + pv);
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= (long long)T * per_tok) return;
+  const int t = (int)(i / per_tok);
+  int c = (int)(i - (long long)t * per_tok);
+  const long long slot = slot_map[t];
+  if (slot < 0) return;
+  const long long blk = slot / block_size, off = slot % block_size;
+  const bool is_v = c >= n_kv * pk;
+  if (is_v) c -= n_kv * pk;
+  const int per = is_v ? pv : pk, h = c / per, e = c - h * per;
+  const size_t dst = ((size_t)(blk * n_kv + h) * block_size + off) * per + e;
+  if (is_v) v_cache[dst] = v[(size_t)t * v_ld + c];
+  else k_cache[dst] = k[(size_t)t * k_ld + c];
 }
 
 // ------------------------------------------------------------------ qkv_post
@@ -480,6 +661,48 @@ MX_HOST_API int mx_rmsnorm_combine(float* x, const void* yp, const int* pair_to_
   if (H % 4 || K > 32 || K < 1) return -107;
   launch_pdl(rmsnorm_combine_kernel, dim3(T), dim3(256), 0, st, x, (const __nv_bfloat16*)yp, pair_to_packed, cw, K, w, (__nv_bfloat16*)out_bf16, eps, H,
              one_plus_w, delta_scale);
+  return (int)cudaGetLastError();
+}
+
+namespace mx {
+template <typename DT, typename OT>
+static int launch_group_norm(const GroupNormParams& p, int T, cudaStream_t st) {
+  const int lanes = 32 * p.wpg;
+  const bool v4 = p.gs % 4 == 0;
+  const int per_lane = v4 ? (p.gs / 4 + lanes - 1) / lanes : 0;
+  if (v4 && per_lane <= 2) launch_pdl(group_norm_kernel<DT, OT, 4, 2>, dim3(T), dim3(GN_WARPS * 32), 0, st, p);
+  else if (v4 && per_lane <= 4) launch_pdl(group_norm_kernel<DT, OT, 4, 4>, dim3(T), dim3(GN_WARPS * 32), 0, st, p);
+  else if (v4 && per_lane <= 8) launch_pdl(group_norm_kernel<DT, OT, 4, 8>, dim3(T), dim3(GN_WARPS * 32), 0, st, p);
+  else if (v4) launch_pdl(group_norm_kernel<DT, OT, 4, 0>, dim3(T), dim3(GN_WARPS * 32), 0, st, p);
+  else launch_pdl(group_norm_kernel<DT, OT, 1, 0>, dim3(T), dim3(GN_WARPS * 32), 0, st, p);
+  return (int)cudaGetLastError();
+}
+}  // namespace mx
+
+// See group_norm_kernel.  x [T][ld] fp32; delta [T][ld] bf16 / fp32 or null; out [T][ld] bf16 / fp32 or null; delta_w, w fp32 [H].
+MX_HOST_API int mx_group_norm(float* x, const void* delta, int delta_is_f32, const float* delta_w, const float* w, void* out, int out_is_f32,
+                              float eps, int T, int H, int ld, int groups, int fresh, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (groups < 1 || H < groups || H % groups || ld < H || ld % 4) return -107;
+  if ((delta && !delta_w) || (out && !w) || (fresh && !delta)) return -109;
+  GroupNormParams p;
+  p.x = x; p.delta = delta; p.delta_w = delta_w; p.w = w; p.out = out; p.eps = eps; p.H = H; p.ld = ld; p.groups = groups; p.gs = H / groups;
+  p.wpg = groups >= GN_WARPS ? 1 : GN_WARPS / groups;
+  p.fresh = fresh;
+  if (delta_is_f32) return out_is_f32 ? launch_group_norm<float, float>(p, T, st) : launch_group_norm<float, __nv_bfloat16>(p, T, st);
+  return out_is_f32 ? launch_group_norm<__nv_bfloat16, float>(p, T, st) : launch_group_norm<__nv_bfloat16, __nv_bfloat16>(p, T, st);
+}
+
+// k / v: rows of n_kv * dk / n_kv * dv elements, k_ld / v_ld elements apart; elem_bytes 2 or 4; every row, head and stride a multiple of 16 bytes.
+MX_HOST_API int mx_kv_store(const void* k, const void* v, int k_ld, int v_ld, const long long* slot_map, void* k_cache, void* v_cache, int T, int n_kv,
+                            int dk, int dv, int block_size, int elem_bytes, cudaStream_t st) {
+  if (T <= 0 || n_kv <= 0) return 0;
+  const int pe = 16 / elem_bytes;
+  if ((elem_bytes != 2 && elem_bytes != 4) || dk % pe || dv % pe || k_ld % pe || v_ld % pe) return -108;
+  if (((uintptr_t)k | (uintptr_t)v | (uintptr_t)k_cache | (uintptr_t)v_cache) & 15) return -108;
+  const long long n = (long long)T * n_kv * (dk / pe + dv / pe);
+  launch_pdl(kv_store_kernel, dim3((unsigned)((n + 255) / 256)), dim3(256), 0, st, (const uint4*)k, (const uint4*)v, k_ld / pe, v_ld / pe, slot_map,
+             (uint4*)k_cache, (uint4*)v_cache, T, n_kv, dk / pe, dv / pe, block_size);
   return (int)cudaGetLastError();
 }
 

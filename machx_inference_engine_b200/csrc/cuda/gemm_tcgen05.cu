@@ -15,6 +15,7 @@
 // (src/ops/gemm_fp16.cpp:64, gemm_onednn.cpp:76-111, gemm_q4k_xmx.cpp:129-432,
 // dequant_kernels.cpp) and the dispatcher in src/model/dense_dispatch.hpp:562-754, and the MoE
 // prefill GEMMs of src/ops/moe_fused.cpp:568-1961.  Ragged K and N are handled natively.
+#include "act.cuh"
 #include "common.cuh"
 #include "comm.cuh"
 #include "dequant.cuh"
@@ -27,7 +28,7 @@ constexpr int BK = 64;
 constexpr int kNumEpilogueWarps = 4;
 constexpr int kNumDequantWarps = 8;
 
-enum Act : int { ACT_NONE = 0, ACT_SWIGLU = 1, ACT_SWIGLU_OAI = 2, ACT_GEGLU = 3 };
+enum Act : int { ACT_NONE = 0, ACT_SWIGLU = 1, ACT_SWIGLU_OAI = 2, ACT_GEGLU = 3, ACT_XIELU = ACT_CODE_XIELU };
 
 struct GemmParams {
   int M, N, K;
@@ -319,7 +320,11 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
           v[j] = __uint_as_float(r[j]);
           if (bias && col0 + j < p.N) v[j] += bias[col0 + j];
         }
-        if (p.act == ACT_NONE) {
+        if (!act_gated(p.act)) {
+          if (p.act != ACT_NONE) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) v[j] = act_unary<false>(p.act, v[j], p.act_alpha, p.act_limit);
+          }
 #pragma unroll
           for (int j = 0; j < 32; ++j) v[j] *= rs;
           const int n_dst = p.peer.world ? peer_count(p.peer) : 1;
@@ -564,7 +569,7 @@ static int gemm_impl(const void* a, int wfmt, const void* w0, const void* w1, co
   if (K % 8) return -101;
   if (wfmt != WF_BF16 && (K % 32)) return -102;
   if ((wfmt == WF_Q4K || wfmt == WF_Q6K) && (K % 256)) return -103;
-  if (act != ACT_NONE && (N % 32)) return -104;
+  if (act_gated(act) && (N % 32)) return -104;
   GemmParams p;
   p.M = M; p.N = N; p.K = K;
   p.num_m_tiles = (M + BM - 1) / BM;

@@ -12,6 +12,7 @@
 // Reference parity: src/ops/gemv_q4k.cpp:72, gemv_q8dot.cpp:276-680, gemv_q6k.cpp:76-670,
 // gemv_mxfp4.cpp:94-323, gemv_fp16.cpp:64 and the batched-T verify kernels gemv_q8dot.cpp:391,499;
 // MoE decode pair moe_fused.cpp:101-541.
+#include "act.cuh"
 #include "common.cuh"
 #include "comm.cuh"
 #include "dequant.cuh"
@@ -34,7 +35,7 @@ struct GemvParams {
   int e_lo, e_hi;           // expert mode: experts owned by this rank (weights hold [e_lo, e_hi)); other slots yield zeros
   int M, N, K;
   int out_f32;
-  int act;                  // 0 none, 1 swiglu, 2 swiglu_oai, 3 geglu (16-row interleaved gate/up)
+  int act;                  // 0 none, 1 swiglu, 2 swiglu_oai, 3 geglu (16-row interleaved gate/up), 4 xIELU (unary, act.cuh)
   float act_alpha, act_limit;
   PeerOut peer;             // world > 0: fp32 partials go to every rank's inbox instead of y (fused all-reduce)
 };
@@ -149,9 +150,9 @@ __global__ void __launch_bounds__(GEMV_WARPS * 32) gemv_kernel(const GemvParams 
   for (int m = 0; m < MM; ++m) {
     if (m >= rows_out) break;
     const size_t orow = p.slot_expert ? (size_t)slot : (size_t)m;
-    if (p.act == 0) {
+    if (!act_gated(p.act)) {
       for (int r = 0; r < GEMV_ROWS && n0 + r < p.N; ++r) {
-        const float v = owned ? (acc[r][m] + (bias ? bias[n0 + r] : 0.f)) * oscale : 0.f;
+        const float v = owned ? act_unary<false>(p.act, acc[r][m] + (bias ? bias[n0 + r] : 0.f), p.act_alpha, p.act_limit) * oscale : 0.f;
         if (p.peer.world) {
           // fused all-reduce: the partial goes to slot [my_rank] of every rank's inbox
           for (int d = 0; d < p.peer.world; ++d) reinterpret_cast<float*>(peer_slot(p.peer, d, next_seq))[orow * p.N + n0 + r] = v;
@@ -350,7 +351,7 @@ __global__ void __launch_bounds__(GEMV_WARPS * 32) gemv_group_kernel(const Group
 
 template <int FMT>
 static int launch_group(const GroupParams& p, int n_experts, cudaStream_t st) {
-  if (p.act != 0) {
+  if (act_gated(p.act)) {
     const int units = (p.N / 2 + 1) / 2;
     launch_pdl(gemv_group_kernel<FMT, true>, dim3(dim3((units + GEMV_WARPS - 1) / GEMV_WARPS, n_experts)), dim3(GEMV_WARPS * 32), 0, st, p);
   } else {
@@ -362,7 +363,7 @@ static int launch_group(const GroupParams& p, int n_experts, cudaStream_t st) {
 
 template <int FMT>
 static int launch_gemv(const GemvParams& p, int slots, cudaStream_t st) {
-  if (p.act != 0) {
+  if (act_gated(p.act)) {
     const int F = p.N / 2;
     dim3 grid((F + GEMV_WARPS * GEMV_ROWS - 1) / (GEMV_WARPS * GEMV_ROWS), slots);
     launch_pdl(gemv_gated_kernel<FMT>, dim3(grid), dim3(GEMV_WARPS * 32), 0, st, p);
@@ -419,7 +420,7 @@ MX_HOST_API int mx_dequant_bf16(int wfmt, const void* w0, const void* w1, const 
 }
 
 // Dense: y[M][N] from x[M][K], M <= 8.   Expert: y[slots][N] with slot_expert != null.
-// With act != 0 the weight holds interleaved gate/up rows (N = 2F) and y is [rows][F]; in that
+// With a gated act the weight holds interleaved gate/up rows (N = 2F) and y is [rows][F]; in that
 // mode every activation row is a "slot" (dense callers pass slots = M and slot_expert = null).
 static int gemv_impl(int wfmt, const void* w0, const void* w1, const void* w2, const void* w3, const void* x, void* y,
                      const float* bias, int M, int N, int K, int out_f32, int act, float act_alpha, float act_limit,
@@ -439,7 +440,7 @@ MX_HOST_API int mx_gemv_group(int wfmt, const void* w0, const void* w1, const vo
   if (N <= 0 || K <= 0 || n_experts <= 0) return 0;
   if (K % 32) return -102;
   if ((wfmt == WF_Q4K || wfmt == WF_Q6K) && (K % 256)) return -103;
-  if (act != 0 && (N % 32)) return -104;
+  if (act != 0 && (N % 32 || !act_gated(act))) return -104;
   GroupParams p;
   p.w = WeightRef{w0, w1, w2, w3}; p.x = (const __nv_bfloat16*)x; p.x_index = x_index; p.y = (__nv_bfloat16*)y; p.bias = bias;
   p.counts = counts; p.seg_start = seg_start; p.e_lo = e_lo; p.N = N; p.K = K; p.act = act; p.act_alpha = act_alpha; p.act_limit = act_limit;
@@ -491,11 +492,11 @@ static int gemv_impl(int wfmt, const void* w0, const void* w1, const void* w2, c
                      const int* slot_expert, const float* slot_scale, int slots, int x_div, const mx::PeerOut* peer, cudaStream_t stream) {
   using namespace mx;
   if (N <= 0 || K <= 0) return 0;
-  if (K % 32 && !(wfmt == WF_BF16 && K % 8 == 0 && act == 0)) return -102;
+  if (K % 32 && !(wfmt == WF_BF16 && K % 8 == 0 && !act_gated(act))) return -102;
   if ((wfmt == WF_Q4K || wfmt == WF_Q6K) && (K % 256)) return -103;
-  if (!slot_expert && act == 0 && (M < 1 || M > GEMV_MAX_M)) return -106;
+  if (!slot_expert && !act_gated(act) && (M < 1 || M > GEMV_MAX_M)) return -106;
   if (g_gemv_path == 2 || (g_gemv_path == 0 && (wfmt == WF_BF16 || wfmt == WF_Q8 || (wfmt == WF_Q4K && K >= g_kq_stream_min_k) ||
-                                                (wfmt == WF_Q6K && act == 0 && K >= g_kq_stream_min_k) || (wfmt == WF_MXFP4 && act != 0)))) {
+                                                (wfmt == WF_Q6K && !act_gated(act) && K >= g_kq_stream_min_k) || (wfmt == WF_MXFP4 && act_gated(act))))) {
     const int rc = gemv_stream_try(wfmt, WeightRef{w0, w1, w2, w3}, x, y, bias, M, N, K, out_f32, act, act_alpha, act_limit, slot_expert,
                                    slot_scale, slots, x_div, g_e_lo, g_e_hi, peer, stream);
     if (rc != 1) return rc;
@@ -508,7 +509,7 @@ static int gemv_impl(int wfmt, const void* w0, const void* w1, const void* w2, c
   p.M = M; p.N = N; p.K = K; p.out_f32 = out_f32;
   p.act = act; p.act_alpha = act_alpha; p.act_limit = act_limit;
   if (peer) p.peer = *peer; else p.peer.world = 0;
-  const int ns = (slot_expert || act != 0) ? (slots > 0 ? slots : M) : 1;
+  const int ns = (slot_expert || act_gated(act)) ? (slots > 0 ? slots : M) : 1;
   switch (wfmt) {
     case WF_BF16: return launch_gemv<WF_BF16>(p, ns, stream);
     case WF_Q8: return launch_gemv<WF_Q8>(p, ns, stream);

@@ -25,6 +25,7 @@
 //
 // Reference parity: src/ops/gemv_fp16.cpp:64, gemv_q8dot.cpp:276-680, gemv_mxfp4.cpp:94-323, moe_fused.cpp:101-541.
 #include <cstring>
+#include "act.cuh"
 #include "common.cuh"
 #include "comm.cuh"
 #include "dequant.cuh"
@@ -829,7 +830,7 @@ gemv_stream_kernel(const GsParams p, const __grid_constant__ CUtensorMap tm0, co
             for (int m = 0; m < MM; ++m) {
               if (!p.slot_mode && m >= p.M) break;
               const size_t orow = p.slot_mode ? (size_t)slot : (size_t)m;
-              const float v = owned ? (acc[r][m] + (bias ? bias[n] : 0.f)) * oscale : 0.f;
+              const float v = owned ? act_unary<false>(p.act, acc[r][m] + (bias ? bias[n] : 0.f), p.act_alpha, p.act_limit) * oscale : 0.f;
               if (p.peer.world) {
                 for (int d = 0; d < p.peer.world; ++d) reinterpret_cast<float*>(peer_slot(p.peer, d, next_seq))[orow * p.N + n] = v;
               } else if (p.out_f32) ((float*)p.y)[orow * p.N + n] = v;
@@ -953,7 +954,7 @@ static int gs_dispatch_ng(GsParams& p, int smem, bool gated, cudaStream_t st) {
 template <int FMT>
 static int gs_dispatch(GsParams& p, cudaStream_t st) {
   constexpr int WARPS = GsCfg<FMT>::WARPS, RPW = GsCfg<FMT>::RPW, RB = WARPS * RPW;
-  const bool gated = p.act != 0;
+  const bool gated = act_gated(p.act);
   p.KC = p.K; p.nkc = 1;
   if (gs_is_bf16(FMT) && p.K > 4096) {
     int n = (p.K + 4095) / 4096;
@@ -1007,13 +1008,13 @@ static int gemv_stream_fused(int wfmt, const WeightRef& w, const void* x, void* 
   if (wfmt != WF_BF16 && wfmt != WF_Q8 && wfmt != WF_MXFP4 && wfmt != WF_Q4K && wfmt != WF_Q6K) return 1;
   if (K % 32 && !(wfmt == WF_BF16 && K % 8 == 0)) return 1;
   if ((wfmt == WF_Q4K || wfmt == WF_Q6K) && K % 256) return 1;
-  if (act != 0 && wfmt != WF_MXFP4 && wfmt != WF_Q4K && !(wfmt == WF_Q8 && !norm && !route)) return 1;      // gated epilogue: one feature per warp needs RPW == 2
-  if (act != 0 && (N % 32)) return 1;
+  if (act_gated(act) && wfmt != WF_MXFP4 && wfmt != WF_Q4K && !(wfmt == WF_Q8 && !norm && !route)) return 1;      // gated epilogue: one feature per warp needs RPW == 2
+  if (act_gated(act) && (N % 32)) return 1;
   GsParams p;
   p.w = w; p.x = (const __nv_bfloat16*)x; p.y = y; p.bias = bias; p.slot_expert = slot_expert; p.slot_scale = slot_scale;
   p.x_div = x_div > 0 ? x_div : 1; p.e_lo = e_lo; p.e_hi = e_hi; p.M = M; p.N = N; p.K = K; p.out_f32 = out_f32; p.act = act;
   p.act_alpha = act_alpha; p.act_limit = act_limit; p.status = status_word();
-  p.slot_mode = (slot_expert != nullptr || act != 0) ? 1 : 0;
+  p.slot_mode = (slot_expert != nullptr || act_gated(act)) ? 1 : 0;
   p.slots = p.slot_mode ? (slots > 0 ? slots : M) : 1;
   p.n_xrows = p.slot_mode ? (p.slots + p.x_div - 1) / p.x_div : M;
   if (p.n_xrows < 1 || p.n_xrows > GS_MAX_XROWS) return 1;

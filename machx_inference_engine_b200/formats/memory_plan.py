@@ -9,6 +9,7 @@ models is counted, and ``describe()`` prints the per-GPU share.
 """
 from __future__ import annotations
 
+import os
 from dataclasses import dataclass
 from typing import Optional
 
@@ -72,6 +73,15 @@ def estimate_state_bytes(kv: dict, n_seqs: int = 1) -> int:
     return n_seqs * n_lin * (n_v * d * d * 4 + conv)
 
 
+def _folder_bytes(path: str, ctx: int, n_seqs: int) -> tuple:
+    """(weights, kv, state) bytes of a checkpoint folder whose config lists its layers."""
+    from .model_config import read_json_config
+    c = read_json_config(path)
+    weights = sum(os.path.getsize(os.path.join(path, f)) for f in os.listdir(path) if f.endswith(".safetensors"))
+    kv = sum(s.kv_heads * (s.key_dim + s.value_dim) for s in c.layer_specs) * ctx * 2 * n_seqs
+    return weights, kv, sum(s.width for s in c.layer_specs) * 4 * n_seqs
+
+
 def visible_gpus() -> tuple:
     """(count, usable bytes per GPU)."""
     try:
@@ -88,11 +98,16 @@ def visible_gpus() -> tuple:
 def plan_placement(path_or_reader, n_gpus: int = 0, ctx: int = 8192, n_seqs: int = 1, avail: Optional[int] = None,
                    per_gpu_bytes: Optional[int] = None) -> PlacementPlan:
     """``n_gpus`` 0 = decide; otherwise the request is respected (clamped to the visible GPUs)."""
-    r = path_or_reader if isinstance(path_or_reader, GGUFReader) else GGUFReader(path_or_reader)
     p = PlacementPlan()
-    p.weights_bytes = r.total_tensor_bytes
-    p.kv_bytes = estimate_kv_bytes(r.kv, ctx, n_seqs)
-    p.state_bytes = estimate_state_bytes(r.kv, n_seqs)
+    one_gpu = isinstance(path_or_reader, str) and os.path.isdir(path_or_reader)
+    if one_gpu:
+        p.weights_bytes, p.kv_bytes, p.state_bytes = _folder_bytes(path_or_reader, ctx, n_seqs)
+        n_gpus = 1                        # the graphs of these checkpoints are not sharded
+    else:
+        r = path_or_reader if isinstance(path_or_reader, GGUFReader) else GGUFReader(path_or_reader)
+        p.weights_bytes = r.total_tensor_bytes
+        p.kv_bytes = estimate_kv_bytes(r.kv, ctx, n_seqs)
+        p.state_bytes = estimate_state_bytes(r.kv, n_seqs)
     n_vis, usable = visible_gpus()
     p.avail_gpus = avail if avail is not None else n_vis
     p.per_gpu_bytes = per_gpu_bytes if per_gpu_bytes is not None else usable
@@ -100,7 +115,7 @@ def plan_placement(path_or_reader, n_gpus: int = 0, ctx: int = 8192, n_seqs: int
         p.forced = True
         p.n_gpus = min(n_gpus, max(p.avail_gpus, 1))
         p.fits = (p.weights_bytes + p.kv_bytes + p.state_bytes) / p.n_gpus + p.ws_bytes <= p.per_gpu_bytes
-        p.note = f"forced --gpus {n_gpus} (using {p.n_gpus})" + ("" if p.fits else " -- does not fit, expect an out-of-memory error")
+        p.note = ("this design runs on one GPU" if one_gpu else f"forced --gpus {n_gpus} (using {p.n_gpus})") + ("" if p.fits else " -- does not fit, expect an out-of-memory error")
         return p
     if p.need_bytes <= p.per_gpu_bytes:
         p.n_gpus, p.note = 1, "fits one GPU"

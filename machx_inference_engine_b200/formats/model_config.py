@@ -7,6 +7,8 @@ keeps one struct per family; here one dataclass serves all graphs.
 """
 from __future__ import annotations
 
+import json
+import os
 from dataclasses import dataclass, field, asdict
 from typing import Any, Mapping
 
@@ -15,10 +17,29 @@ MOE_ARCHS = ("qwen3moe", "gpt-oss")
 HYBRID_ARCHS = ("qwen3next", "qwen35", "qwen35moe")
 GEMMA_ARCHS = ("gemma4",)
 SUPPORTED_ARCHS = DENSE_ARCHS + MOE_ARCHS + HYBRID_ARCHS + GEMMA_ARCHS
+# checkpoints that are a folder with config.json + safetensors and list their layers one by one: "architecture" value -> arch
+LAYER_LIST_ARCHS = {"Tikarax": "tikarax"}
 
 
 class ConfigError(ValueError):
     pass
+
+
+@dataclass
+class LayerSpec:
+    """One layer of a design whose configuration lists its layers: a mixer with its sizes and constants, and a feed-forward (0 = none)."""
+    mixer: str                     # "attention" | "mingru"
+    ffn: int = 0
+    # attention without rotation, with its own value width, query temperature and output gate
+    heads: int = 0
+    kv_heads: int = 0
+    key_dim: int = 0
+    value_dim: int = 0
+    scale: float = 0.0
+    q_temp_coef: float = 0.0       # queries at position p are multiplied by 1 + coef * ln(floor((p + 1) / every) + 1)
+    q_temp_every: float = 1.0
+    # minGRU
+    width: int = 0
 
 
 @dataclass
@@ -62,6 +83,9 @@ class ModelConfig:
     rope_theta_swa: float = 10000.0
     layer_swa: list = field(default_factory=list)        # per layer: True = sliding-window layer
     layer_n_kv: list = field(default_factory=list)       # per layer: KV head count
+    # designs that list their layers (LAYER_LIST_ARCHS): head_dim / n_heads / n_kv_heads / ffn above are the largest of any layer
+    layer_specs: list = field(default_factory=list)      # LayerSpec per layer
+    norm_groups: int = 1                                  # RMS norms run over this many equal parts of the row
     # Granite scalars
     embedding_scale: float = 1.0
     residual_scale: float = 1.0
@@ -83,6 +107,8 @@ class ModelConfig:
         return self.arch in HYBRID_ARCHS
 
     def layer_is_full_attention(self, layer: int) -> bool:
+        if self.layer_specs:
+            return self.layer_specs[layer].mixer == "attention"
         if not self.is_hybrid:
             return True
         return (layer + 1) % self.full_attn_interval == 0
@@ -232,6 +258,74 @@ def read_config(kv: Mapping[str, Any], tensor_names=()) -> ModelConfig:
     return c
 
 
+def _tikarax_config(d: Mapping[str, Any]) -> ModelConfig:
+    c = ModelConfig(arch="tikarax", hidden=int(d["width"]), vocab=int(d["vocab"]), rms_eps=float(d["norm"]["eps"]), norm_groups=int(d["norm"]["groups"]),
+                    name=str(d.get("name", "")))
+    for i, e in enumerate(d["layers"]):
+        m, mlp = e["mixer"], e.get("mlp")
+        if mlp is not None and mlp.get("kind", "dense") != "dense":
+            raise ConfigError(f"layer {i}: unknown feed-forward kind {mlp['kind']!r}")
+        s = LayerSpec(e["type"], ffn=0 if mlp is None else int(mlp["ff"]))
+        if s.mixer == "attention":
+            s.heads, s.kv_heads, s.key_dim, s.value_dim, s.scale = int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"])
+            t = m.get("q_temp")
+            if t is not None:
+                s.q_temp_coef, s.q_temp_every = float(t["coef"]), float(t["every"])
+                if s.q_temp_every <= 0:
+                    raise ConfigError(f"layer {i}: q_temp.every must be positive")
+            if s.kv_heads < 1 or s.heads % s.kv_heads:
+                raise ConfigError(f"layer {i}: {s.heads} query heads do not divide over {s.kv_heads} key/value heads")
+        elif s.mixer == "mingru":
+            s.width = int(m["width"])
+        else:
+            raise ConfigError(f"layer {i}: unknown mixer {s.mixer!r}")
+        c.layer_specs.append(s)
+    if c.hidden < 1 or c.vocab < 1 or not c.layer_specs or c.norm_groups < 1 or c.hidden % c.norm_groups:
+        raise ConfigError("the width must be positive and a multiple of norm.groups, with at least one layer")
+    return _finish_layer_list(c)
+
+
+def _finish_layer_list(c: ModelConfig) -> ModelConfig:
+    """Derived fields of a layer-list config: the largest sizes of any layer (pool sizing, reports)."""
+    big = lambda f, lo=0: max([lo] + [getattr(s, f) for s in c.layer_specs])
+    c.n_layers = len(c.layer_specs)
+    c.n_heads, c.n_kv_heads, c.ffn = big("heads", 1), big("kv_heads", 1), big("ffn")
+    c.head_dim = max(big("key_dim", 1), big("value_dim"))
+    c.n_rot, c.ctx_train = 0, 1 << 20                      # no rotation: positions have no trained limit of their own
+    return c
+
+
+def read_json_config(path_or_dict) -> ModelConfig:
+    """config.json of a checkpoint folder (or the parsed dict) of a layer-list design."""
+    d = path_or_dict
+    if not isinstance(d, Mapping):
+        p = os.path.join(d, "config.json") if os.path.isdir(d) else d
+        with open(p) as f:
+            d = json.load(f)
+    a = d.get("architecture")
+    readers = {"tikarax": _tikarax_config}
+    if a not in LAYER_LIST_ARCHS:
+        raise ConfigError(f"unsupported architecture {a!r} in config.json (supported: {', '.join(LAYER_LIST_ARCHS)})")
+    try:
+        return readers[LAYER_LIST_ARCHS[a]](d)
+    except (KeyError, TypeError) as e:
+        raise ConfigError(f"config.json of a {a} model: missing or malformed {e}") from e
+
+
+def config_to_json(c: ModelConfig) -> dict:
+    """Inverse of :func:`read_json_config`."""
+    layers = []
+    for s in c.layer_specs:
+        if s.mixer == "attention":
+            m = {"heads": s.heads, "kv_heads": s.kv_heads, "dim": s.key_dim, "vdim": s.value_dim, "scale": s.scale,
+                 "q_temp": {"coef": s.q_temp_coef, "every": int(s.q_temp_every) if float(s.q_temp_every).is_integer() else s.q_temp_every}}
+        else:
+            m = {"width": s.width}
+        layers.append({"type": s.mixer, "mixer": m, "mlp": {"kind": "dense", "ff": s.ffn} if s.ffn else None})
+    arch = {v: k for k, v in LAYER_LIST_ARCHS.items()}[c.arch]
+    return {"architecture": arch, "layers": layers, "norm": {"eps": c.rms_eps, "groups": c.norm_groups}, "vocab": c.vocab, "width": c.hidden}
+
+
 def config_to_kv(c: ModelConfig) -> dict:
     """Inverse of :func:`read_config` for the synthetic-checkpoint generator."""
     a = c.arch
@@ -277,6 +371,18 @@ def config_to_kv(c: ModelConfig) -> dict:
         kv[f"{a}.attention.scale"] = float(c.attention_scale)
         kv[f"{a}.logit_scale"] = float(1.0 / c.logit_scale) if c.logit_scale else 1.0
     return kv
+
+
+def _tikarax_preset(hidden, n_layers, heads, kv_heads, dim, vdim, ffn, width, vocab, attn_every=4, groups=2, every=8192) -> ModelConfig:
+    """Every ``attn_every``-th layer attention, the others minGRU."""
+    c = ModelConfig(arch="tikarax", hidden=hidden, vocab=vocab, rms_eps=1e-6, norm_groups=groups)
+    for l in range(n_layers):
+        if (l + 1) % attn_every == 0:
+            c.layer_specs.append(LayerSpec("attention", ffn=ffn, heads=heads, kv_heads=kv_heads, key_dim=dim, value_dim=vdim, scale=dim ** -0.5,
+                                           q_temp_coef=0.1, q_temp_every=every))
+        else:
+            c.layer_specs.append(LayerSpec("mingru", ffn=ffn, width=width))
+    return _finish_layer_list(c)
 
 
 # ---- named architectures used by the benches and tests (random-init; see formats/synth.py)
@@ -334,6 +440,10 @@ def preset(name: str) -> ModelConfig:
                                          rms_eps=1e-6, rope_theta=1e6, n_rot=128, ctx_train=4096, sliding_window=128, head_dim_swa=64,
                                          n_rot_swa=64, rope_theta_swa=10000.0, layer_swa=[True, True, False], layer_n_kv=[2, 2, 1],
                                          final_logit_softcap=30.0, embedding_scale=16.0, attention_scale=1.0, tie_embeddings=True),
+        "tiny-tikarax": _tikarax_preset(160, 4, 6, 2, 40, 56, 224, 288, 384, attn_every=2, groups=5, every=48),
+        # layers of common model sizes: 1 B class and 8 B class (un-gated feed-forward with the parameters of a gated one of 2/3 its width)
+        "tikarax-1b": _tikarax_preset(2048, 16, 32, 8, 64, 64, 12288, 4096, 128256),
+        "tikarax-8b": _tikarax_preset(4096, 32, 32, 8, 128, 128, 21504, 6144, 128256),
         "tiny-qwen2": ModelConfig(arch="qwen2", n_layers=2, hidden=256, n_heads=4, n_kv_heads=2, head_dim=64, ffn=512, vocab=2048,
                                   rms_eps=1e-6, rope_theta=1e6, n_rot=64, ctx_train=4096),
         "tiny-phi3": ModelConfig(arch="phi3", n_layers=2, hidden=256, n_heads=4, n_kv_heads=4, head_dim=64, ffn=512, vocab=2048,

@@ -15,7 +15,7 @@ from typing import Callable, Iterable
 import numpy as np
 
 from .gguf import GGMLType, GGUFWriter, block_elems
-from .model_config import ModelConfig, config_to_kv
+from .model_config import ModelConfig, config_to_json, config_to_kv
 from .quant import quantize
 
 _CHATML_TEMPLATE = "{% for m in messages %}<|im_start|>{{ m.role }}\n{{ m.content }}<|im_end|>\n{% endfor %}<|im_start|>assistant\n"
@@ -289,6 +289,52 @@ def write_synthetic_gguf(cfg: ModelConfig, path: str, quant: str = "q8_0", seed:
     w.write(path)
     import os
     return {"tensors": n, "bytes": os.path.getsize(path)}
+
+
+def folder_tensor_plan(cfg: ModelConfig) -> list:
+    """(name, kind, shape) of every tensor of a layer-list checkpoint folder (``LAYER_LIST_ARCHS``); matrices are [out, in]."""
+    H = cfg.hidden
+    out = [("embed", "matrix", (cfg.vocab, H)), ("embed.norm", "norm", (H,)), ("final.norm", "norm", (H,)), ("head", "matrix", (cfg.vocab, H))]
+    for i, s in enumerate(cfg.layer_specs):
+        p = f"l{i}"
+        out += [(f"{p}.norm1", "norm", (H,)), (f"{p}.norm1b", "norm", (H,))]
+        if s.mixer == "attention":
+            biased = {"q": s.heads * s.key_dim, "k": s.kv_heads * s.key_dim, "v": s.kv_heads * s.value_dim}
+            plain, width = {"g": s.heads * s.value_dim}, s.heads * s.value_dim
+        else:
+            biased, plain, width = {"z": s.width, "x": s.width}, {"g": s.width}, s.width
+        for n, rows in biased.items():
+            out += [(f"{p}.mix.{n}", "matrix", (rows, H)), (f"{p}.mix.{n}.b", "vector", (rows,))]
+        out += [(f"{p}.mix.{n}", "matrix", (rows, H)) for n, rows in plain.items()] + [(f"{p}.mix.o", "matrix", (H, width))]
+        if s.ffn:
+            out += [(f"{p}.norm2", "norm", (H,)), (f"{p}.norm2b", "norm", (H,)), (f"{p}.mlp.up", "matrix", (s.ffn, H)),
+                    (f"{p}.mlp.down", "matrix", (H, s.ffn)), (f"{p}.mlp.act", "vector", (2,))]
+    return out
+
+
+def write_synthetic_folder(cfg: ModelConfig, path: str, seed: int = 0) -> dict:
+    """Random-init checkpoint folder (config.json + bf16 model.safetensors) of a layer-list design."""
+    import json
+    import os
+
+    from .safetensors import write_safetensors
+    os.makedirs(path, exist_ok=True)
+    with open(os.path.join(path, "config.json"), "w") as f:
+        json.dump(config_to_json(cfg), f, indent=1)
+    tensors = {}
+    for name, kind, shape in folder_tensor_plan(cfg):
+        g = np.random.default_rng([seed, zlib.crc32(name.encode())])
+        v = g.standard_normal(shape, dtype=np.float32)
+        v = {"matrix": lambda: v / np.sqrt(np.float32(shape[-1])), "norm": lambda: 1.0 + 0.1 * v, "vector": lambda: 0.1 * v}[kind]()
+        bits = np.ascontiguousarray(v, dtype=np.float32).view(np.uint32)
+        tensors[name] = ("BF16", ((bits + 0x7FFF + ((bits >> 16) & 1)) >> 16).astype(np.uint16))
+    write_safetensors(os.path.join(path, "model.safetensors"), tensors)
+    return {"tensors": len(tensors), "bytes": os.path.getsize(os.path.join(path, "model.safetensors"))}
+
+
+def write_synthetic(cfg: ModelConfig, path: str, quant: str = "q8_0", seed: int = 0) -> dict:
+    """The checkpoint form of the architecture: a GGUF file, or a folder for designs that list their layers."""
+    return write_synthetic_folder(cfg, path, seed) if cfg.layer_specs else write_synthetic_gguf(cfg, path, quant=quant, seed=seed)
 
 
 def assistant_tensor_plan(a) -> list:

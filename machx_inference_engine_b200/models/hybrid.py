@@ -23,43 +23,55 @@ from .. import ops
 from ..formats.model_config import ModelConfig
 from ..ops import ACT_SWIGLU, QuantWeight
 from ..parallel.comm import ParallelCtx
-from .transformer import AttentionBlock, DenseFFN, ForwardBatch, KVCache, Linear, MoEFFN, TransformerModel, _fuse_rows
+from .transformer import AttentionBlock, DenseFFN, ForwardBatch, KVCache, Linear, MoEFFN, TransformerModel, _fuse_rows, round_up
 
 D_HEAD = 128      # DeltaNet key / value head width (the only geometry the families use)
 
 
-class DeltaNetState:
-    """Recurrent state of every DeltaNet layer for ``n_slots`` concurrent sequences (include/ie/deltanet_state.hpp:28-75):
-    ``S[l]`` fp32 [slots, n_v, 128 (v), 128 (k)] and ``conv[l]`` bf16 [slots, kernel-1, channels]."""
+class RecurrentState:
+    """Recurrent state of ``n_slots`` concurrent sequences: ``tensors[name][layer]`` has the slot as its first dimension.  What the engine
+    needs of a state -- reset, copy, snapshot and restore of a slot -- does not depend on what a layer keeps in it."""
 
-    def __init__(self, layers: list, n_slots: int, n_v: int, channels: int, kernel: int, device):
-        self.layers, self.n_slots, self.n_v, self.channels, self.kernel, self.device = layers, n_slots, n_v, channels, kernel, device
-        self.S = {l: torch.zeros(n_slots, n_v, D_HEAD, D_HEAD, dtype=torch.float32, device=device) for l in layers}
-        self.conv = {l: torch.zeros(n_slots, kernel - 1, channels, dtype=torch.bfloat16, device=device) for l in layers}
-        self.ckpt_S: dict = {}
-        self.ckpt_conv: dict = {}
-        self.ckpt_rows = 0
+    def __init__(self, n_slots: int, tensors: dict, device):
+        self.n_slots, self.tensors, self.device = n_slots, tensors, device
 
     def reset(self, slots) -> None:
         idx = torch.as_tensor(list(slots), dtype=torch.long, device=self.device)
         if idx.numel() == 0:
             return
-        for l in self.layers:
-            self.S[l].index_fill_(0, idx, 0.0)
-            self.conv[l].index_fill_(0, idx, 0.0)
+        for per_layer in self.tensors.values():
+            for t in per_layer.values():
+                t.index_fill_(0, idx, 0.0)
 
     def copy_slot(self, src: int, dst: int) -> None:
-        for l in self.layers:
-            self.S[l][dst].copy_(self.S[l][src])
-            self.conv[l][dst].copy_(self.conv[l][src])
+        for per_layer in self.tensors.values():
+            for t in per_layer.values():
+                t[dst].copy_(t[src])
 
     def snapshot(self, slot: int) -> dict:
-        return {"S": {l: self.S[l][slot].clone() for l in self.layers}, "conv": {l: self.conv[l][slot].clone() for l in self.layers}}
+        return {name: {l: t[slot].clone() for l, t in per_layer.items()} for name, per_layer in self.tensors.items()}
 
     def restore(self, slot: int, snap: dict) -> None:
-        for l in self.layers:
-            self.S[l][slot].copy_(snap["S"][l])
-            self.conv[l][slot].copy_(snap["conv"][l])
+        for name, per_layer in self.tensors.items():
+            for l, t in per_layer.items():
+                t[slot].copy_(snap[name][l])
+
+    def nbytes(self) -> int:
+        return sum(t.numel() * t.element_size() for d in self.tensors.values() for t in d.values())
+
+
+class DeltaNetState(RecurrentState):
+    """Recurrent state of every DeltaNet layer for ``n_slots`` concurrent sequences (include/ie/deltanet_state.hpp:28-75):
+    ``S[l]`` fp32 [slots, n_v, 128 (v), 128 (k)] and ``conv[l]`` bf16 [slots, kernel-1, channels]."""
+
+    def __init__(self, layers: list, n_slots: int, n_v: int, channels: int, kernel: int, device):
+        self.layers, self.n_v, self.channels, self.kernel = layers, n_v, channels, kernel
+        self.S = {l: torch.zeros(n_slots, n_v, D_HEAD, D_HEAD, dtype=torch.float32, device=device) for l in layers}
+        self.conv = {l: torch.zeros(n_slots, kernel - 1, channels, dtype=torch.bfloat16, device=device) for l in layers}
+        super().__init__(n_slots, {"S": self.S, "conv": self.conv}, device)
+        self.ckpt_S: dict = {}
+        self.ckpt_conv: dict = {}
+        self.ckpt_rows = 0
 
     # ---- per-position checkpoints of one verify step (Qwen35SpecCheckpoint, src/model/qwen35_dense.cpp:892-937)
     def enable_checkpoints(self, rows: int) -> None:
@@ -73,9 +85,6 @@ class DeltaNetState:
         for l in self.layers:
             self.S[l][slot].copy_(self.ckpt_S[l][row])
             self.conv[l][slot].copy_(self.ckpt_conv[l][row])
-
-    def nbytes(self) -> int:
-        return sum(t.numel() * t.element_size() for d in (self.S, self.conv) for t in d.values())
 
 
 class LinearAttentionBlock:
@@ -157,6 +166,31 @@ class LinearAttentionBlock:
                               state.S[l], fb.state_slots, fb.cu_q, self.n_v, eps=1e-6, ckpt=state.ckpt_S[l] if checkpoint else None)
         g = ops.gated_rmsnorm_heads(o, y[:, self.z_off:self.z_off + self.n_v * D_HEAD], self.norm_w, self.eps, D_HEAD)
         return self.out(g, par if self.sharded else None)
+
+
+class MinGRUBlock:
+    """minGRU layer: one projection [z | candidate | gate], the element-wise recurrence with its activations and its SiLU output gate in
+    one kernel (state fp32), output projection.  The biases of z and of the candidate are added inside the recurrence, in fp32."""
+
+    def __init__(self, src, prefix: str, layer: int, hidden: int, row: int, width: int):
+        self.layer = layer
+        W = self.width = round_up(width, 32)
+        ws = [src.matrix(f"{prefix}.{n}", width, hidden).pad_groups(rows=(1, W), cols=(1, row)) for n in ("z", "x", "g")]
+        self.proj = _fuse_rows(ws, [None] * 3)
+
+        def bias(name):
+            b = torch.zeros(W, dtype=torch.float32, device=ws[0].device)
+            b[:width] = src.vector(f"{prefix}.{name}.b", width)
+            return b
+
+        self.zb, self.xb = bias("z"), bias("x")
+        self.out = Linear(src.matrix(f"{prefix}.o", hidden, width).pad_groups(rows=(1, row), cols=(1, W)))
+
+    def __call__(self, h: torch.Tensor, fb: ForwardBatch, state: RecurrentState) -> torch.Tensor:
+        y, W = self.proj(h), self.width
+        s = ops.mingru_scan(y[:, :W], y[:, W:2 * W], y[:, 2 * W:], self.zb, self.xb, state.tensors["S"][self.layer], fb.state_slots, fb.cu_q, fb.seq_lens,
+                            fb.max_q_len)
+        return self.out(s)
 
 
 class SharedExpert:

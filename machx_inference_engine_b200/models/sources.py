@@ -59,6 +59,44 @@ class GGUFSource:
         return v.to(self.device)
 
 
+class SafetensorsSource:
+    """A checkpoint folder's safetensors under the names the graphs ask for; ``names`` maps graph names to file names where they differ.
+    Matrices are stored [out, in] and become bf16 weights (exact for bf16 payloads), vectors fp32."""
+
+    def __init__(self, model, device, names: Optional[dict] = None):
+        self.m, self.device, self.names = model, torch.device(device), names or {}
+
+    def _name(self, name: str) -> str:
+        return self.names.get(name, name)
+
+    def has(self, name: str) -> bool:
+        return self.m.has(self._name(name))
+
+    def _checked(self, name: str, shape: tuple) -> str:
+        n = self._name(name)
+        if not self.m.has(n):
+            raise ValueError(f"the checkpoint has no tensor {n!r}")
+        if tuple(self.m.shape(n)) != tuple(shape):
+            raise ValueError(f"{n}: expected shape {tuple(shape)}, file has {tuple(self.m.shape(n))}")
+        return n
+
+    def matrix(self, name: str, N: int, K: int, E: int = 1, experts: Optional[tuple[int, int]] = None) -> QuantWeight:
+        if E != 1 or experts is not None:
+            raise ValueError("expert stacks are not read from safetensors folders")
+        n = self._checked(name, (N, K))
+        if self.m.dtype(n) == "BF16":
+            t = torch.from_numpy(np.array(self.m.numpy(n), copy=True).view(np.int16)).view(torch.bfloat16)
+        else:
+            t = torch.from_numpy(np.array(self.m.float32(n), copy=True)).to(torch.bfloat16)
+        return QuantWeight(WFormat.BF16, N, K, 1, t.reshape(1, N, K).to(self.device).contiguous())
+
+    def vector(self, name: str, n: int) -> torch.Tensor:
+        return self.table(name, (n,))
+
+    def table(self, name: str, shape: tuple[int, ...]) -> torch.Tensor:
+        return torch.from_numpy(np.array(self.m.float32(self._checked(name, shape)), copy=True)).to(self.device)
+
+
 def default_policy(arch: str, quant: str) -> Callable[[str], WFormat]:
     """Weight format per tensor name for a named quantisation recipe.
 
@@ -165,6 +203,8 @@ class SynthSource:
 
     def vector(self, name: str, n: int) -> torch.Tensor:
         g = self._gen(name)
+        if name.endswith(".norm") or name.rsplit(".", 1)[-1] in ("norm1", "norm1b", "norm2", "norm2b"):
+            return (1.0 + 0.05 * torch.randn(n, generator=g, device=self.gen_device)).to(self.device)
         if name.endswith("norm.weight") or "_norm" in name or name.endswith(".scale") or name.endswith("layer_output_scale.weight"):
             return (1.0 + 0.05 * torch.randn(n, generator=g, device=self.gen_device)).to(self.device)
         if name.endswith("ssm_a"):

@@ -60,26 +60,29 @@ class ForwardBatch:
 
 
 class KVCache:
-    """Paged KV: per attention layer ``k, v [num_blocks, n_kv_local, KV_BLOCK, head_dim]`` bf16, or int8 with one fp32 scale
+    """Paged KV: per attention layer ``k, v [num_blocks, n_kv_local, KV_BLOCK, head_dim]`` bf16 or fp32, or int8 with one fp32 scale
     per (block, kv head, token) row in ``ks, vs [num_blocks, n_kv_local, KV_BLOCK]`` (value = q * scale, scale = max|x| / 127).
+    ``geometry`` gives layers their own (n_kv, head_dim) or (n_kv, key width, value width).
 
     The reference cache is contiguous per sequence (include/ie/kv_cache.hpp:27-114) and keeps int8 rows beside it when
     ``--int8-kv`` is given (src/core/kv_cache.cpp:182-240, src/ops/attention.cpp:145-229); pages make continuous batching
     and block-level prefix sharing possible, and here the int8 rows replace the bf16 ones instead of shadowing them.
     """
 
+    BLOCK = KV_BLOCK
+
     def __init__(self, n_layers: int, num_blocks: int, n_kv: int, head_dim: int, device, attn_layers: Optional[list[int]] = None,
                  dtype: str = "bf16", geometry: Optional[dict] = None):
-        if dtype not in ("bf16", "int8"):
+        if dtype not in ("bf16", "fp32", "int8"):
             raise ValueError(f"unknown KV cache dtype {dtype!r}")
         self.num_blocks = num_blocks
         self.block_size = KV_BLOCK
         self.dtype = dtype
         layers = attn_layers if attn_layers is not None else list(range(n_layers))
-        td = torch.bfloat16 if dtype == "bf16" else torch.int8
-        geo = {l: ((geometry or {}).get(l) or (n_kv, head_dim)) for l in layers}       # per layer (n_kv, head_dim): Gemma-4 mixes two
+        td = {"bf16": torch.bfloat16, "fp32": torch.float32, "int8": torch.int8}[dtype]
+        geo = {l: ((geometry or {}).get(l) or (n_kv, head_dim)) for l in layers}       # per layer: Gemma-4 mixes two, Tikarax lists them
         self.k = {l: torch.zeros(num_blocks, geo[l][0], KV_BLOCK, geo[l][1], dtype=td, device=device) for l in layers}
-        self.v = {l: torch.zeros(num_blocks, geo[l][0], KV_BLOCK, geo[l][1], dtype=td, device=device) for l in layers}
+        self.v = {l: torch.zeros(num_blocks, geo[l][0], KV_BLOCK, geo[l][-1], dtype=td, device=device) for l in layers}
         self.ks = {l: torch.ones(num_blocks, geo[l][0], KV_BLOCK, dtype=torch.float32, device=device) for l in layers} if dtype == "int8" else None
         self.vs = {l: torch.ones(num_blocks, geo[l][0], KV_BLOCK, dtype=torch.float32, device=device) for l in layers} if dtype == "int8" else None
 
@@ -129,7 +132,7 @@ class MultiLinear:
 
     def __init__(self, parts: list[Linear]):
         self.parts = parts
-        self.widths = [p.w.N // 2 if p.act != ACT_NONE else p.w.N for p in parts]
+        self.widths = [p.w.N // 2 if ops.act_gated(p.act) else p.w.N for p in parts]
 
     def __call__(self, x, par=None, out_f32=False):
         # every part writes its own column slice of one output (no concatenation pass)
@@ -267,6 +270,61 @@ def _attn_gathered(self, sc, T: int, gbuf: int, fb: ForwardBatch, kv: KVCache, r
 
 
 AttentionBlock.forward_gathered = _attn_gathered
+
+
+def round_up(n: int, m: int) -> int:
+    return (n + m - 1) // m * m
+
+
+class NoRopeAttentionBlock:
+    """Attention without rotation: separate key and value widths, biased q / k / v, a query temperature given as a table over positions
+    (folded into the fp32 scores) and a sigmoid output gate that reads the block's own input.
+
+    One projection produces the columns [q | k | v | gate]; the queries and the gate are read in place by the attention kernel (which
+    applies the gate as it writes), only K and V are moved, into the cache pages.  Head widths are padded to multiples of 8 at load."""
+
+    def __init__(self, src, prefix: str, layer: int, hidden: int, row: int, heads: int, kv_heads: int, key_dim: int, value_dim: int, scale: float,
+                 q_scale: Optional[torch.Tensor] = None):
+        self.layer, self.n_q, self.n_kv, self.scale, self.q_scale = layer, heads, kv_heads, scale, q_scale
+        self.dk, self.dv = round_up(key_dim, 8), round_up(value_dim, 8)
+        H = hidden
+
+        def rows(name, n, d, dp, biased=True):
+            w = src.matrix(f"{prefix}.{name}", n * d, H).pad_groups(rows=(n, dp), cols=(1, row))
+            b = torch.zeros(n, dp, dtype=torch.float32, device=w.device)
+            if biased:
+                b[:, :d] = src.vector(f"{prefix}.{name}.b", n * d).reshape(n, d)
+            return w, b.reshape(-1)
+
+        parts = [rows("q", heads, key_dim, self.dk), rows("k", kv_heads, key_dim, self.dk), rows("v", kv_heads, value_dim, self.dv),
+                 rows("g", heads, value_dim, self.dv, biased=False)]
+        self.proj = _fuse_rows([w for w, _ in parts], [b for _, b in parts])
+        ends = [0]
+        for w, _ in parts:
+            ends.append(ends[-1] + w.N)
+        self.cols = ends
+        wo = src.matrix(f"{prefix}.o", H, heads * value_dim).pad_groups(rows=(1, row), cols=(heads, self.dv))
+        self.o = Linear(wo)
+
+    def __call__(self, h: torch.Tensor, fb: ForwardBatch, kv: KVCache) -> torch.Tensor:
+        y = self.proj(h)
+        T, c, l = y.shape[0], self.cols, self.layer
+        ops.kv_store(y[:, c[1]:c[2]], y[:, c[2]:c[3]], fb.slot_map, kv.k[l], kv.v[l])
+        a = ops.attention(y[:, :c[1]].view(T, self.n_q, self.dk), kv.k[l], kv.v[l], fb.block_table, fb.seq_lens, fb.cu_q, fb.max_q_len, scale=self.scale,
+                          max_kv_len=fb.max_kv_len, q_scale=self.q_scale, gate=y[:, c[3]:])
+        return self.o(a.reshape(T, self.n_q * self.dv))
+
+
+class UnaryFFN:
+    """down(act(up h)): a feed-forward without a gate branch; the activation runs in the up projection's epilogue."""
+
+    def __init__(self, src, prefix: str, hidden: int, row: int, ffn: int, act: int, act_a: float = 0.0, act_b: float = 0.0):
+        f = round_up(ffn, 32)
+        self.up = Linear(src.matrix(f"{prefix}.up", ffn, hidden).pad_groups(rows=(1, f), cols=(1, row)), act=act, act_alpha=act_a, act_limit=act_b)
+        self.down = Linear(src.matrix(f"{prefix}.down", hidden, ffn).pad_groups(rows=(1, row), cols=(1, f)))
+
+    def __call__(self, h):
+        return self.down(self.up(h))
 
 
 class DenseFFN:
@@ -589,10 +647,10 @@ class TransformerModel:
         self.layer_lo, self.layer_hi = ((par.rank * c.n_layers) // par.world, ((par.rank + 1) * c.n_layers) // par.world) if self.pp else (0, c.n_layers)
         self.first_stage, self.last_stage = (not self.pp or par.rank == 0), (not self.pp or par.rank == par.world - 1)
         self.tied = not src.has("output.weight") or c.tie_embeddings
-        self.embed_w = src.matrix("token_embd.weight", c.vocab, c.hidden) if (self.first_stage or (self.last_stage and self.tied)) else None
+        self.embed_w = self._vocab_matrix(src, "token_embd.weight") if (self.first_stage or (self.last_stage and self.tied)) else None
         head = None
         if self.last_stage:
-            head = self.embed_w if self.tied else src.matrix("output.weight", c.vocab, c.hidden)
+            head = self.embed_w if self.tied else self._vocab_matrix(src, "output.weight")
         self.vocab_lo, self.vocab_hi = 0, c.vocab
         if tp > 1:
             lo, hi = _even_chunks(c.vocab, tp, 16)[par.rank] if c.vocab % (16 * tp) == 0 else (0, c.vocab)
@@ -611,6 +669,9 @@ class TransformerModel:
         self.n_kv_local = next((L["attn"].n_kv for L in self.layers if "attn" in L), 0)
 
     # ---- construction
+    def _vocab_matrix(self, src, name: str) -> QuantWeight:
+        return src.matrix(name, self.cfg.vocab, self.cfg.hidden)
+
     def _build_layer(self, l: int, src) -> dict:
         c, par = self.cfg, self.par
         p = f"blk.{l}"
@@ -628,6 +689,9 @@ class TransformerModel:
 
     def new_kv_cache(self, num_blocks: int, dtype: str = "bf16") -> KVCache:
         return KVCache(self.cfg.n_layers, num_blocks, self.n_kv_local, self.cfg.head_dim, self.device, self.attn_layers, dtype=dtype)
+
+    def kv_bytes_per_block(self, dtype: str = "bf16") -> int:
+        return KVCache.bytes_per_block(len(self.attn_layers), self.n_kv_local, self.cfg.head_dim, dtype)
 
     def weight_bytes(self) -> int:
         n = (self.embed_w.nbytes if self.embed_w is not None else 0) + (0 if (self.tied or self.lm_head is None) else self.lm_head.w.nbytes)

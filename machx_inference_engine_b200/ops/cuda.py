@@ -12,7 +12,7 @@ from typing import Optional
 import torch
 
 from .. import _lib
-from .ref import ACT_GEGLU, ACT_NONE, ACT_SWIGLU, ACT_SWIGLU_OAI, MOE_TILE, MoePacking, moe_max_rows
+from .ref import ACT_GEGLU, ACT_NONE, ACT_SWIGLU, ACT_SWIGLU_OAI, MOE_TILE, MoePacking, act_gated, moe_max_rows
 from .weights import QuantWeight, WFormat
 
 _vp = C.c_void_p
@@ -130,6 +130,37 @@ def rmsnorm(x, w, eps, delta=None, dbias=None, one_plus_w=False, delta_scale=1.0
                                   C.c_float(delta_scale), int(write_x), _stream()), "rmsnorm")
     _count()
     return out
+
+
+def group_norm(x, w, eps, groups=1, delta=None, delta_w=None, fresh=False, width=None, out_dtype=torch.bfloat16, want_out=True):
+    T, ld = x.shape
+    H = ld if width is None else width
+    assert x.dtype == torch.float32 and x.is_contiguous() and (delta is None or (delta.is_contiguous() and delta.shape == x.shape))
+    out = torch.empty(T, ld, dtype=out_dtype, device=x.device) if want_out else None
+    _check(_lib.cuda().mx_group_norm(_p(x), _p(delta), int(delta is not None and delta.dtype == torch.float32), _p(delta_w), _p(w), _p(out),
+                                     int(out_dtype == torch.float32), C.c_float(eps), T, H, ld, int(groups), int(fresh), _stream()), "group_norm")
+    _count()
+    return out
+
+
+def kv_store(k, v, slot_map, k_cache, v_cache):
+    T, n_kv, bs, dk = k.shape[0], k_cache.shape[1], k_cache.shape[2], k_cache.shape[3]
+    dv = v_cache.shape[3]
+    assert k.dtype == v.dtype == k_cache.dtype == v_cache.dtype and k.stride(1) == 1 and v.stride(1) == 1
+    assert k.shape[1] == n_kv * dk and v.shape[1] == n_kv * dv
+    _check(_lib.cuda().mx_kv_store(_p(k), _p(v), k.stride(0), v.stride(0), _p(slot_map), _p(k_cache), _p(v_cache), T, n_kv, dk, dv, bs,
+                                   k.element_size(), _stream()), "kv_store")
+    _count()
+
+
+def mingru_scan(z, u, g, zb, ub, state, state_slots, cu_q, seq_lens, max_q_len):
+    T, W = z.shape
+    assert z.dtype == u.dtype == g.dtype and z.stride() == u.stride() == g.stride() and z.stride(1) == 1 and state.dtype == torch.float32
+    y = torch.empty(T, W, dtype=z.dtype, device=z.device)
+    _check(_lib.cuda().mx_mingru_scan(_p(z), _p(u), _p(g), z.stride(0), _p(zb), _p(ub), _p(state), _p(state_slots), _p(cu_q), _p(seq_lens), _p(y),
+                                      cu_q.numel() - 1, W, int(max_q_len), int(z.dtype == torch.float32), _stream()), "mingru_scan")
+    _count()
+    return y
 
 
 class CombineDelta:
@@ -297,12 +328,14 @@ def _out_kind(dtype) -> int:
 def linear(x, w: QuantWeight, bias=None, act=ACT_NONE, act_alpha=1.702, act_limit=7.0, out_f32=False, row_scale=None, out=None):
     """``out``: write into this [M, n_out] view (unit column stride; a column slice of a wider matrix is fine), so that projections
     whose weights differ in format can share one output without a concatenation."""
+    if x.dtype == torch.float32:
+        return _linear_f32(x, w, bias, act, act_alpha, act_limit, row_scale, out)
     assert x.dtype == torch.bfloat16 and x.is_contiguous() and x.shape[-1] == w.K and w.E == 1
     M = x.shape[0]
     if w.fmt == WFormat.EXL3:
         assert act == ACT_NONE and row_scale is None, "EXL3 layers have no fused activation or row scale"
         return _exl3_linear(x, w, bias, out_f32, out)
-    n_out = w.N // 2 if act != ACT_NONE else w.N
+    n_out = w.N // 2 if act_gated(act) else w.N
     odt = torch.float32 if out_f32 else torch.bfloat16
     if out is None:
         out = torch.empty(M, n_out, dtype=odt, device=x.device)
@@ -330,6 +363,22 @@ def linear(x, w: QuantWeight, bias=None, act=ACT_NONE, act_alpha=1.702, act_limi
         _check(lib.mx_gemm(_p(xa), fmt, p0, p1, p2, p3, 1, _p(out), out.stride(0), int(out_f32), _p(bias), _p(row_scale), act,
                            C.c_float(act_alpha), C.c_float(act_limit), M, w.N, w.K, _vp(0), _vp(0), _pick_bn(M, w.N), _stream()), "gemm")
     _count()
+    return out
+
+
+def _linear_f32(x, w: QuantWeight, bias, act, act_alpha, act_limit, row_scale, out):
+    """fp32 activations: the layer runs in full 32-bit on the CUDA cores (``csrc/cuda/linear_f32.cu``); dense bf16 weights only."""
+    if w.fmt != WFormat.BF16 or w.E != 1 or row_scale is not None or act_gated(act):
+        raise KernelError("32-bit linear layers take dense bf16 weights and no gated activation")
+    assert x.is_contiguous() and x.shape[-1] == w.K
+    M = x.shape[0]
+    if out is None:
+        out = torch.empty(M, w.N, dtype=torch.float32, device=x.device)
+    assert out.shape == (M, w.N) and out.dtype == torch.float32 and (M == 0 or out.stride(1) == 1)
+    if M:
+        _check(_lib.cuda().mx_linear_f32(_p(x), _p(w.p0), _p(bias), _p(out), M, w.N, w.K, out.stride(0), act, C.c_float(act_alpha), C.c_float(act_limit),
+                                         _stream()), "linear_f32")
+        _count()
     return out
 
 
@@ -395,7 +444,7 @@ def _exl3_linear(x, w: QuantWeight, bias, out_f32, out):
 def gemm(x, w: QuantWeight, bias=None, act=ACT_NONE, act_alpha=1.702, act_limit=7.0, out_f32=False, row_scale=None, bn=None):
     """Always the tcgen05 path (tests and benches)."""
     M = x.shape[0]
-    n_out = w.N // 2 if act != ACT_NONE else w.N
+    n_out = w.N // 2 if act_gated(act) else w.N
     out = torch.empty(M, n_out, dtype=torch.float32 if out_f32 else torch.bfloat16, device=x.device)
     fmt, p0, p1, p2, p3 = _planes(w)
     xa = _gemm_a(x, w)
@@ -441,15 +490,24 @@ _attn_scratch: dict = {}
 TC_PREFILL_MIN_Q = 64      # query segments at least this long take the tensor-core kernel
 
 
-def attention_prefill_tc(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks=None, window=0, scale=None, softcap=0.0):
-    """tcgen05 FlashAttention (head_dim 64 / 128 / 256, page size 128, optional logit soft-cap)."""
+def _q_rows(q):
+    """Elements between query rows: q is [Tq, n_q, dk] with dense heads, possibly a column range of a wider projection."""
+    assert q.stride(2) == 1 and (q.shape[1] == 1 or q.stride(1) == q.shape[2])
+    return q.stride(0)
+
+
+def attention_prefill_tc(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks=None, window=0, scale=None, softcap=0.0, q_scale=None,
+                         gate=None):
+    """tcgen05 FlashAttention (key / value widths that are multiples of 8 up to 256, page size 128, optional logit soft-cap)."""
     Tq, n_q, hd = q.shape
-    n_kv, bs = k_cache.shape[1], k_cache.shape[2]
+    n_kv, bs, dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
     scale = scale if scale is not None else 1.0 / math.sqrt(hd)
-    out = torch.empty(Tq, n_q, hd, dtype=torch.bfloat16, device=q.device)
-    _check(_lib.cuda().mx_attention_prefill_tc(_p(q), _p(k_cache), _p(v_cache), _p(block_table), _p(seq_lens), _p(cu_q), _p(sinks), _p(out),
-                                               seq_lens.numel(), Tq, int(max_q_len), n_q, n_kv, hd, block_table.shape[1], k_cache.shape[0], bs,
-                                               int(window), C.c_float(scale), C.c_float(softcap or 0.0), _stream()), "attention_prefill_tc")
+    out = torch.empty(Tq, n_q, dv, dtype=torch.bfloat16, device=q.device)
+    _check(_lib.cuda().mx_attention_prefill_tc_ext(_p(q), _q_rows(q), _p(k_cache), _p(v_cache), _p(block_table), _p(seq_lens), _p(cu_q), _p(sinks),
+                                                   _p(gate), 0 if gate is None else gate.stride(0), _p(q_scale), 0 if q_scale is None else q_scale.numel(),
+                                                   _p(out), seq_lens.numel(), Tq, int(max_q_len), n_q, n_kv, hd, dv, block_table.shape[1],
+                                                   k_cache.shape[0], bs, int(window), C.c_float(scale), C.c_float(softcap or 0.0), _stream()),
+           "attention_prefill_tc")
     _count()
     return out
 
@@ -483,19 +541,30 @@ def _dequant_pages(k_cache, v_cache, kv_scales, block_table, seq_lens, max_kv_le
 ATTN_MAX_SPLITS = 32
 
 
+def _tc_prefill_takes(q, dk, dv, softcap, kv_scales) -> bool:
+    if q.dtype != torch.bfloat16:
+        return False
+    if dk == dv and dk in (64, 128, 256):
+        return True
+    return kv_scales is None and not softcap and 8 <= dk <= 256 and 8 <= dv <= 256 and dk % 8 == 0 and dv % 8 == 0
+
+
 def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks=None, window=0, scale=None, softcap=0.0, n_splits=None,
-              kv_scales=None, max_kv_len=0):
+              kv_scales=None, max_kv_len=0, q_scale=None, gate=None):
     Tq, n_q, hd = q.shape
-    n_kv, bs = k_cache.shape[1], k_cache.shape[2]
+    n_kv, bs, dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
+    assert k_cache.dtype == torch.int8 or k_cache.dtype == v_cache.dtype == q.dtype
+    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape == (Tq, n_q * dv))
     B = seq_lens.numel()
     scale = scale if scale is not None else 1.0 / math.sqrt(hd)
     assert (k_cache.dtype == torch.int8) == (kv_scales is not None)
-    if max_q_len >= TC_PREFILL_MIN_Q and hd in (64, 128, 256) and bs == 128 and n_splits is None:
+    if max_q_len >= TC_PREFILL_MIN_Q and bs == 128 and n_splits is None and _tc_prefill_takes(q, hd, dv, softcap, kv_scales):
         if kv_scales is not None:       # the tensor-core kernel reads bf16 pages: expand this batch's pages first
             dk, dv, table = _dequant_pages(k_cache, v_cache, kv_scales, block_table, seq_lens, max_kv_len)
-            return attention_prefill_tc(q, dk, dv, table, seq_lens, cu_q, max_q_len, sinks=sinks, window=window, scale=scale, softcap=softcap)
+            return attention_prefill_tc(q, dk, dv, table, seq_lens, cu_q, max_q_len, sinks=sinks, window=window, scale=scale, softcap=softcap,
+                                        q_scale=q_scale, gate=gate)
         return attention_prefill_tc(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks=sinks, window=window, scale=scale,
-                                    softcap=softcap)
+                                    softcap=softcap, q_scale=q_scale, gate=gate)
     if n_splits is None:
         # decode-sized problems: split the KV range so that ~2 CTAs per SM exist
         ctas = B * n_kv * max(1, (max_q_len * (n_q // n_kv) + 31) // 32)
@@ -503,7 +572,7 @@ def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks
         # (the cap: with two KV heads of 256 and one sequence, 128 ranges instead of 32 took a 16k context from 119 to 103 us but a 4k
         # context from 48 to 54 us -- the last CTA's merge grows with the ranges; the kernel itself takes any number)
         n_splits = max(1, min(max_kv_tiles, ATTN_MAX_SPLITS, (2 * sm_count()) // max(ctas, 1)))
-    need = n_splits * Tq * n_q * (hd + 2)
+    need = n_splits * Tq * n_q * (dv + 2)
     if torch.cuda.is_current_stream_capturing():
         # a captured kernel keeps the raw address: the scratch must live exactly as long as the graph, so it comes from the
         # graph's own pool.  (The shared buffer below is re-allocated when a larger request arrives; a graph that had
@@ -514,18 +583,20 @@ def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks
         if buf is None or buf.numel() < need:
             buf = torch.empty(max(need, 1 << 20), dtype=torch.float32, device=q.device)
             _attn_scratch[q.device] = buf
-    o_part = buf[: n_splits * Tq * n_q * hd]
-    ml_part = buf[n_splits * Tq * n_q * hd: need]
-    out = torch.empty(Tq, n_q, hd, dtype=torch.bfloat16, device=q.device)
+    o_part = buf[: n_splits * Tq * n_q * dv]
+    ml_part = buf[n_splits * Tq * n_q * dv: need]
+    out = torch.empty(Tq, n_q, dv, dtype=q.dtype, device=q.device)
     if kv_scales is not None:
+        assert q_scale is None and gate is None and q.is_contiguous(), "the int8 cache has no gated / position-scaled form"
         _check(_lib.cuda().mx_attention_kv8(_p(q), _p(k_cache), _p(v_cache), _p(kv_scales[0]), _p(kv_scales[1]), _p(block_table), _p(seq_lens),
                                             _p(cu_q), _p(sinks), _p(out), _p(o_part), _p(ml_part), B, Tq, int(max_q_len), n_q, n_kv, hd,
                                             block_table.shape[1], bs, int(window), C.c_float(scale), C.c_float(softcap), int(n_splits),
                                             _stream()), "attention_kv8")
     else:
-        _check(_lib.cuda().mx_attention(_p(q), _p(k_cache), _p(v_cache), _p(block_table), _p(seq_lens), _p(cu_q), _p(sinks), _p(out),
-                                        _p(o_part), _p(ml_part), B, Tq, int(max_q_len), n_q, n_kv, hd, block_table.shape[1], bs, int(window),
-                                        C.c_float(scale), C.c_float(softcap), int(n_splits), _stream()), "attention")
+        _check(_lib.cuda().mx_attention_ext(_p(q), _q_rows(q), _p(k_cache), _p(v_cache), _p(block_table), _p(seq_lens), _p(cu_q), _p(sinks), _p(gate),
+                                            0 if gate is None else gate.stride(0), _p(q_scale), 0 if q_scale is None else q_scale.numel(), _p(out),
+                                            _p(o_part), _p(ml_part), B, Tq, int(max_q_len), n_q, n_kv, hd, dv, block_table.shape[1], bs, int(window),
+                                            C.c_float(scale), C.c_float(softcap), int(n_splits), int(q.dtype == torch.float32), _stream()), "attention")
     _count(_lib.cuda().mx_attention_launches(B, int(max_q_len), n_q, n_kv))
     return out
 

@@ -14,7 +14,14 @@ import torch
 
 from .weights import QuantWeight
 
-ACT_NONE, ACT_SWIGLU, ACT_SWIGLU_OAI, ACT_GEGLU = 0, 1, 2, 3
+ACT_NONE, ACT_SWIGLU, ACT_SWIGLU_OAI, ACT_GEGLU, ACT_XIELU = 0, 1, 2, 3, 4
+
+
+def act_gated(act: int) -> bool:
+    """Gated activations combine 16-row interleaved gate / up columns (N columns become N / 2); the others are element-wise."""
+    return act in (ACT_SWIGLU, ACT_SWIGLU_OAI, ACT_GEGLU)
+
+
 MOE_TILE = 128
 
 
@@ -90,6 +97,14 @@ def rmsnorm(x, w, eps, delta=None, dbias=None, one_plus_w=False, delta_scale=1.0
     return (xs * inv * g).to(torch.bfloat16)
 
 
+def act_unary(act, z, a, b):
+    """xIELU: a z^2 + z / 2 above zero, b (e^z - 1 - z) + z / 2 below (a = softplus(p), b = 1/2 + softplus(q))."""
+    if act != ACT_XIELU:
+        return z
+    neg = z.clamp(max=0.0)
+    return torch.where(z > 0, a * z * z, b * (torch.expm1(neg) - neg)) + 0.5 * z
+
+
 def _act(act, g, u, alpha, limit):
     if act == ACT_SWIGLU:
         return torch.nn.functional.silu(g) * u
@@ -118,12 +133,14 @@ def linear(x, w: QuantWeight, bias=None, act=ACT_NONE, act_alpha=1.702, act_limi
     y = _mm(x, _dense(w)[0])
     if bias is not None:
         y = y + bias
-    if act != ACT_NONE:
+    if act_gated(act):
         g, u = _deinterleave16(y)
         y = _act(act, g, u, act_alpha, act_limit)
+    elif act != ACT_NONE:
+        y = act_unary(act, y, act_alpha, act_limit)
     if row_scale is not None:
         y = y * row_scale.unsqueeze(-1)
-    return y if out_f32 else y.to(torch.bfloat16)
+    return y if (out_f32 or x.dtype == torch.float32) else y.to(torch.bfloat16)      # fp32 activations: the layer runs in fp32 throughout
 
 
 def hadamard128(x, pre=None, post=None, bias=None, out_f32=False, out=None):
@@ -237,14 +254,71 @@ def qkv_post(qkv, bias, q_norm_w, k_norm_w, positions, rope_cos, rope_sin, slot_
     return qpart.to(torch.bfloat16).contiguous(), gate
 
 
+def group_norm(x, w, eps, groups=1, delta=None, delta_w=None, fresh=False, width=None, out_dtype=torch.bfloat16, want_out=True):
+    """RMSNorm over ``groups`` equal parts of a row.  With ``delta``: x <- (0 if fresh else x) + norm(delta) * delta_w, in place; returns
+    norm(x) * w.  Rows are padded to x.shape[1] columns; the first ``width`` (default: all) are the row, the padding stays zero."""
+    H = x.shape[1] if width is None else width
+
+    def norm(t, g):
+        p = t[:, :H].to(torch.float32).reshape(t.shape[0], groups, H // groups)
+        return (p * torch.rsqrt(p.pow(2).mean(-1, keepdim=True) + eps)).reshape(-1, H) * g
+
+    if delta is not None:
+        d = norm(delta, delta_w)
+        if fresh:
+            x.zero_()
+        x[:, :H] += d
+    if not want_out:
+        return None
+    out = torch.zeros(x.shape, dtype=out_dtype, device=x.device)
+    out[:, :H] = norm(x, w).to(out_dtype)
+    return out
+
+
+def kv_store(k, v, slot_map, k_cache, v_cache):
+    """k [T, n_kv * dk], v [T, n_kv * dv] (any row stride) -> rows of the paged caches [blocks, n_kv, bs, dk / dv]; slots < 0 are skipped."""
+    T, n_kv, bs = k.shape[0], k_cache.shape[1], k_cache.shape[2]
+    ok = slot_map >= 0
+    blk, off = (slot_map[ok] // bs).long(), (slot_map[ok] % bs).long()
+    k_cache[blk, :, off] = k.reshape(T, n_kv, -1)[ok].to(k_cache.dtype)
+    v_cache[blk, :, off] = v.reshape(T, n_kv, -1)[ok].to(v_cache.dtype)
+
+
+def mingru_scan(z, u, g, zb, ub, state, state_slots, cu_q, seq_lens, max_q_len):
+    """Element-wise gated recurrence over packed sequences: S_t = (1 - s(z)) S_(t-1) + s(z) c(u), y = S_t * silu(g) with s the sigmoid and
+    c(u) = u + 1/2 above zero, s(u) below; z and u get their biases here.  z, u, g [T, W] (any row stride); state fp32 [slots, W] is
+    advanced in place and starts from zeros for a sequence whose step begins at position 0."""
+    T, W = z.shape
+    y = torch.empty(T, W, dtype=z.dtype, device=z.device)
+    zz = torch.sigmoid(z.to(torch.float32) + zb)
+    uu = u.to(torch.float32) + ub
+    c = torch.where(uu >= 0, uu + 0.5, torch.sigmoid(uu))
+    gate = torch.nn.functional.silu(g.to(torch.float32))
+    cu = cu_q.tolist()
+    for b in range(len(cu) - 1):
+        t0, t1 = cu[b], cu[b + 1]
+        if t1 <= t0:
+            continue
+        slot = int(state_slots[b])
+        S = torch.zeros(W, dtype=torch.float32, device=z.device) if int(seq_lens[b]) == t1 - t0 else state[slot].clone()
+        for t in range(t0, t1):
+            S = (1.0 - zz[t]) * S + zz[t] * c[t]
+            y[t] = (S * gate[t]).to(y.dtype)
+        state[slot] = S
+    return y
+
+
 def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks=None, window=0, scale=None, softcap=0.0, n_splits=1,
-              kv_scales=None, max_kv_len=0):
-    """q [Tq,n_q,hd]; caches [blocks,n_kv,bs,hd] (bf16, or int8 with kv_scales = (k_scale, v_scale) [blocks,n_kv,bs]); returns bf16 [Tq,n_q,hd]."""
+              kv_scales=None, max_kv_len=0, q_scale=None, gate=None):
+    """q [Tq,n_q,hd]; caches [blocks,n_kv,bs,hd] (bf16 / fp32, or int8 with kv_scales = (k_scale, v_scale) [blocks,n_kv,bs]); values may be
+    wider or narrower than keys; returns [Tq,n_q,value width] (bf16; fp32 for fp32 queries).  ``q_scale`` [positions]: factor on the scores
+    of a query at that position; ``gate`` [Tq, n_q * value width]: the result is multiplied by its sigmoid."""
     Tq, n_q, hd = q.shape
+    dv = v_cache.shape[3]
     n_kv, bs = k_cache.shape[1], k_cache.shape[2]
     gqa = n_q // n_kv
     scale = scale if scale is not None else 1.0 / math.sqrt(hd)
-    out = torch.zeros(Tq, n_q, hd, dtype=torch.float32, device=q.device)
+    out = torch.zeros(Tq, n_q, dv, dtype=torch.float32, device=q.device)
     cu = cu_q.tolist()
     for b in range(len(cu) - 1):
         q0, q1 = cu[b], cu[b + 1]
@@ -257,8 +331,10 @@ def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks
         if kv_scales is not None:
             Kp, Vp = Kp * kv_scales[0][blocks].unsqueeze(-1), Vp * kv_scales[1][blocks].unsqueeze(-1)
         K = Kp.permute(1, 0, 2, 3).reshape(n_kv, nblk * bs, hd)[:, :L]
-        V = Vp.permute(1, 0, 2, 3).reshape(n_kv, nblk * bs, hd)[:, :L]
+        V = Vp.permute(1, 0, 2, 3).reshape(n_kv, nblk * bs, dv)[:, :L]
         qq = q[q0:q1].to(torch.float32) * scale                                 # [t, n_q, hd]
+        if q_scale is not None:
+            qq = qq * q_scale[L - (q1 - q0):L].reshape(-1, 1, 1)
         Kh = K.repeat_interleave(gqa, dim=0)
         Vh = V.repeat_interleave(gqa, dim=0)
         s = torch.einsum("thd,hkd->htk", qq.to(_MM_DTYPE), Kh.to(_MM_DTYPE)).to(torch.float32)
@@ -276,7 +352,9 @@ def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks
         else:
             p = torch.softmax(s, dim=-1)
         out[q0:q1] = torch.einsum("htk,hkd->thd", p.to(_MM_DTYPE), Vh.to(_MM_DTYPE)).to(torch.float32)
-    return out.to(torch.bfloat16)
+    if gate is not None:
+        out = out * torch.sigmoid(gate.to(torch.float32)).reshape(Tq, n_q, dv)
+    return out if q.dtype == torch.float32 else out.to(torch.bfloat16)
 
 
 def sigmoid_mul(x, g):

@@ -126,6 +126,24 @@ class QuantWeight:
         w.N = hi - lo
         return w
 
+    def pad_groups(self, rows: Optional[tuple] = None, cols: Optional[tuple] = None) -> "QuantWeight":
+        """bf16 only: (groups, size) on the rows / columns -- each of ``groups`` equal runs is padded with zeros to ``size`` elements, so that
+        head or feature ranges start where the kernels' vector accesses want them.  A padded row gives a zero output, a padded column
+        meets a zero activation: the product is unchanged."""
+        if self.fmt != WFormat.BF16:
+            raise ValueError(f"only bf16 weights can be padded, not {self.fmt.name}")
+        t = self.p0
+        for dim, spec in ((1, rows), (2, cols)):
+            if spec is None or t.shape[dim] == spec[0] * spec[1]:
+                continue
+            n, size = spec
+            per = t.shape[dim] // n
+            v = t.reshape(*t.shape[:dim], n, per, *t.shape[dim + 1:])
+            out = torch.zeros(*v.shape[:dim + 1], size, *v.shape[dim + 2:], dtype=t.dtype, device=t.device)
+            out.narrow(dim + 1, 0, per).copy_(v)
+            t = out.reshape(*t.shape[:dim], n * size, *t.shape[dim + 1:])
+        return QuantWeight(WFormat.BF16, t.shape[1], t.shape[2], self.E, t.contiguous())
+
     def slice_experts(self, lo: int, hi: int) -> "QuantWeight":
         w = self._map_planes(lambda t: t[lo:hi].contiguous())
         w.E = hi - lo

@@ -65,17 +65,19 @@ class Engine:
 
     # ------------------------------------------------------------------ loading
     @classmethod
-    def load(cls, path: str, device="cuda", opts: Optional[EngineOptions] = None, par=None, spec_head: Optional[str] = None) -> "Engine":
-        """``spec_head``: a separate draft-head checkpoint (Gemma-4's ``gemma4-assistant`` GGUF); heads stored inside the model file
+    def load(cls, path: str, device="cuda", opts: Optional[EngineOptions] = None, par=None, spec_head: Optional[str] = None,
+             dtype: str = "bf16") -> "Engine":
+        """``path``: a GGUF file, or a folder with config.json + safetensors (no tokenizer: prompts are token ids).  ``dtype``: "bf16", or
+        "fp32" for graphs that also run in 32-bit.  ``spec_head``: a separate draft-head checkpoint (Gemma-4's ``gemma4-assistant`` GGUF); heads stored inside the model file
         (Qwen3-Next's MTP layer) need none."""
         from ..models import load_model
         opts = opts or EngineOptions()
-        model, reader = load_model(path, device, par, max_ctx=opts.max_ctx)
+        model, reader = load_model(path, device, par, max_ctx=opts.max_ctx, dtype=dtype)
         if spec_head:
             from ..models.gemma4_assistant import load_assistant_head
             load_assistant_head(model, spec_head)
         opts.max_ctx = min(opts.max_ctx, model.max_ctx)
-        tok = Tokenizer.from_gguf_kv(reader.kv)
+        tok = Tokenizer.from_gguf_kv(reader.kv) if any(k.startswith("tokenizer.") for k in reader.kv) else None
         return cls(model, tok, opts, model_id=str(reader.kv.get("general.name", "")) or path.rsplit("/", 1)[-1])
 
     def _find(self, s: str) -> int:
@@ -95,11 +97,18 @@ class Engine:
 
     # ------------------------------------------------------------------ text API (blocking, single request)
     def encode_chat(self, turns: Sequence[ChatTurn], enable_thinking=True, tools_json: str = "") -> list:
+        if self.tok is None:
+            raise ValueError("this checkpoint has no tokenizer: send token ids")
         text = templates.render(self.family, turns, True, enable_thinking, tools_json, self.model_has_think, self.cfg.mistral_sysprompt)
         return self.tok.encode(text, allow_special=True)
 
     def generate(self, prompt: str | list, sp: Optional[SamplingParams] = None, on_text: Optional[Callable[[str], None]] = None) -> GenerateResult:
-        ids = self.tok.encode(prompt, allow_special=True) if isinstance(prompt, str) else list(prompt)
+        if isinstance(prompt, str):
+            if self.tok is None:
+                return GenerateResult(finish_reason="error", error="this checkpoint has no tokenizer: send token ids")
+            ids = self.tok.encode(prompt, allow_special=True)
+        else:
+            ids = list(prompt)
         with self._lock:
             return self._run_blocking(ids, sp or SamplingParams(), on_text)
 

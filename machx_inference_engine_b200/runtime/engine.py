@@ -257,6 +257,20 @@ class Scheduler:
             budget -= n
         return plan
 
+    def admit(self, entries: list) -> list:
+        """Plan of a step whose tokens the caller chose: ``entries`` = [(seq, n tokens past what is computed)].  Blocks and state slots are
+        taken here; nothing is queued or preempted, a pool that cannot hold the step raises before anything has run."""
+        for seq, n in entries:
+            if seq not in self.running:
+                if len(self.running) >= self.opts.max_seqs or (self.uses_state and not self.free_state):
+                    raise OutOfBlocks("no free sequence slot")
+                if self.uses_state:
+                    seq.state_slot = self.free_state.popleft()
+                self.running.append(seq)
+            if not self._ensure_blocks(seq, seq.n_computed + n):
+                raise OutOfBlocks("KV block pool exhausted")
+        return list(entries)
+
     def _preempt(self, seq: Sequence) -> None:
         """Out of blocks: push the sequence back to the queue; its KV is recomputed later."""
         self.running.remove(seq)
@@ -285,14 +299,12 @@ class LLMEngine:
         self.model = model
         self.opts = opts or EngineOptions()
         self.device = model.device
-        cfg = model.cfg
         o = self.opts
         blocks_per_seq = (o.max_ctx + KV_BLOCK - 1) // KV_BLOCK
         nb = o.num_blocks or (o.max_seqs * blocks_per_seq + 1)
         if o.kv_memory_fraction > 0 and self.device.type == "cuda":
             free, _ = torch.cuda.mem_get_info(self.device)
-            from ..models.transformer import KVCache
-            per = max(1, KVCache.bytes_per_block(len(model.attn_layers), model.n_kv_local, cfg.head_dim, o.kv_dtype))
+            per = max(1, model.kv_bytes_per_block(o.kv_dtype))
             nb = max(blocks_per_seq + 1, int(free * o.kv_memory_fraction) // per)
         self.max_blocks_per_seq = blocks_per_seq
         self.kv = model.new_kv_cache(nb, o.kv_dtype) if o.kv_dtype != "bf16" else model.new_kv_cache(nb)
@@ -364,6 +376,35 @@ class LLMEngine:
     def has_work(self) -> bool:
         return self.sched.has_work()
 
+    # ------------------------------------------------------------------ steps whose tokens the caller gives
+    def open_sequence(self) -> Sequence:
+        """A sequence that is fed through :meth:`feed` instead of being scheduled and sampled; :meth:`abort` gives back what it holds."""
+        return Sequence(next(self._ids), [], SamplingParams(), t_arrival=time.perf_counter())
+
+    def feed(self, entries: list) -> Optional[torch.Tensor]:
+        """One forward over [(seq, its next tokens, places among them whose logits are wanted)]: the batch assembly, cache, state slots and
+        execution paths (graphs included) of :meth:`step`, without its sampling.  Returns fp32 logits [wanted, vocab] in the order of the
+        entries and of their places, or None when nothing is wanted."""
+        for seq, toks, _ in entries:
+            if not toks or len(seq.tokens) + len(toks) > self.opts.max_ctx:
+                raise ContextLengthExceeded(f"{len(seq.tokens)} + {len(toks)} tokens do not fit the context of {self.opts.max_ctx}")
+        plan = self.sched.admit([(seq, len(toks)) for seq, toks, _ in entries])
+        rows, base = [], 0
+        for seq, toks, want in entries:
+            if any(not 0 <= w < len(toks) for w in want):
+                raise ValueError("a wanted place lies outside its tokens")
+            seq.tokens.extend(toks)
+            rows.extend(base + w for w in want)
+            base += len(toks)
+        if self.state is not None:
+            self._restore_states(plan)
+        logits = self._logits(plan, rows)
+        for seq, n in plan:
+            seq.n_computed += n
+            self.stats["prefill_tokens" if n > 1 else "decode_tokens"] += n
+        self.stats["steps"] += 1
+        return logits.clone() if rows else None           # (a graph's output buffer is written again by its next replay)
+
     # ------------------------------------------------------------------ one step
     def step(self) -> list:
         """Runs one forward over the scheduled batch; returns [(seq, token, finished)] for sequences that produced a token."""
@@ -418,8 +459,10 @@ class LLMEngine:
             seq.finished, seq.finish_reason = True, "length"
 
     # ------------------------------------------------------------------ batch assembly + execution
-    def _build_batch(self, plan: list, sampled_rows: list, pad_to: int = 0):
-        ids, pos, slots, cu, lens, tables, logit_rows = [], [], [], [0], [], [], []
+    def _build_batch(self, plan: list, logit_rows: list, pad_to: int = 0):
+        """``logit_rows``: rows of the flattened batch whose logits are computed."""
+        logit_rows = list(logit_rows)
+        ids, pos, slots, cu, lens, tables = [], [], [], [0], [], []
         for i, (seq, n) in enumerate(plan):
             s0 = seq.n_computed
             ids.extend(seq.tokens[s0:s0 + n])
@@ -429,8 +472,6 @@ class LLMEngine:
             cu.append(cu[-1] + n)
             lens.append(s0 + n)
             tables.append(seq.blocks)
-        for i in sampled_rows:
-            logit_rows.append(cu[i + 1] - 1)
         B = len(plan)
         for _ in range(max(0, pad_to - B)):                # graph padding: null sequences of one token in block 0
             ids.append(0); pos.append(0); slots.append(-1); cu.append(cu[-1] + 1); lens.append(1); tables.append([0])
@@ -469,48 +510,66 @@ class LLMEngine:
             t[i], k[i], p[i], m[i] = s.params.temperature, s.params.top_k, s.params.top_p, s.params.min_p
         return t, k, p, m
 
+    def _graphs_ok(self) -> bool:
+        # graphs hold only this library's kernels: the NCCL baseline path (no fused collectives) and the layer split (NCCL
+        # point-to-point hand-offs between the stages) run eagerly
+        par = getattr(self.model, "par", None)
+        nccl_path = par is not None and par.enabled and (par.fused is None or par.mode == "pp")
+        return self.opts.cuda_graphs and self.device.type == "cuda" and not nccl_path and not self.spec_k
+
+    def _decode_graph_ok(self, plan: list) -> bool:
+        return (self._graphs_ok() and all(n == 1 for _, n in plan) and len(plan) <= max(self.opts.graph_batch_sizes)
+                and (self.state is None or all(s.n_computed > 0 for s, _ in plan)))
+
+    def _prefill_graph_ok(self, plan: list) -> bool:
+        if not (self._graphs_ok() and self.opts.prefill_graphs and self.opts.kv_dtype == "bf16" and len(plan) == 1):
+            return False
+        n = plan[0][1]
+        return n in (512, 1024, 2048, 4096, 8192) or (n == self.opts.max_batch_tokens and n % KV_BLOCK == 0 and n >= 256)
+
     def _run(self, plan: list, sampled_rows: list) -> list:
         if self.state is not None:
             self._restore_states(plan)
-        decode_only = all(n == 1 for _, n in plan) and len(sampled_rows) == len(plan)
         seqs = [plan[i][0] for i in sampled_rows]
         greedy = all(s.params.temperature <= 0 and s.params.repetition_penalty == 1.0 for s in seqs)
-        par = getattr(self.model, "par", None)
-        # graphs hold only this library's kernels: the NCCL baseline path (no fused collectives) and the layer split (NCCL
-        # point-to-point hand-offs between the stages) run eagerly
-        nccl_path = par is not None and par.enabled and (par.fused is None or par.mode == "pp")
-        use_graph = (decode_only and greedy and self.opts.cuda_graphs and self.device.type == "cuda"
-                     and (self.state is None or all(s.n_computed > 0 for s, _ in plan))
-                     and len(plan) <= max(self.opts.graph_batch_sizes) and not nccl_path and not self.spec_k)
-        if use_graph:
-            return self._run_graph(plan)
-        if (self.opts.cuda_graphs and self.opts.prefill_graphs and self.opts.kv_dtype == "bf16" and self.device.type == "cuda" and not nccl_path
-                and len(plan) == 1
-                and (plan[0][1] in (512, 1024, 2048, 4096, 8192) or (plan[0][1] == self.opts.max_batch_tokens and plan[0][1] % KV_BLOCK == 0
-                                                                      and plan[0][1] >= 256)) and not self.spec_k):
-            return self._run_prefill_graph(plan, sampled_rows, seqs)
-        host, max_q = self._build_batch(plan, sampled_rows)
+        if greedy and len(sampled_rows) == len(plan) and self._decode_graph_ok(plan):
+            out = self._replay_decode(plan)["out"].cpu()
+            self.stats["d2h_bytes"] += out.numel() * 4
+            return out[:len(plan)].tolist()
+        ends = list(itertools.accumulate(n for _, n in plan))
+        logits = self._logits(plan, [ends[i] - 1 for i in sampled_rows], greedy=greedy)
+        if self.spec_k and sampled_rows:
+            logits, hidden = logits
+            for r, s in enumerate(seqs):
+                s.h_last = hidden[r:r + 1]
+        if not sampled_rows:
+            return []
+        out = self._sample(logits, seqs).cpu()
+        self.stats["d2h_bytes"] += out.numel() * 4
+        return out.tolist()
+
+    def _logits(self, plan: list, rows: list, greedy: bool = True) -> torch.Tensor:
+        """Runs the step and returns the fp32 logits of ``rows`` (places in the flattened batch): the decode graph for a batch of single
+        tokens, the prefill graph for a single-sequence chunk of a graphed size whose only wanted row is its last, eager otherwise."""
+        T = sum(n for _, n in plan)
+        if greedy and self._decode_graph_ok(plan):
+            logits = self._replay_decode(plan)["logits"]
+            return logits[:T] if rows == list(range(T)) else logits[torch.tensor(rows, dtype=torch.long, device=self.device)]
+        if self._prefill_graph_ok(plan) and all(r == T - 1 for r in rows):
+            logits = self._replay_prefill(plan)["logits"]
+            return logits if len(rows) <= 1 else logits.expand(len(rows), -1)
+        host, max_q = self._build_batch(plan, rows)
         dev = self._to_device(host)
         fb = ForwardBatch(dev["ids"], dev["positions"], dev["slot_map"], dev["block_table"], dev["seq_lens"], dev["cu_q"], max_q,
-                          logit_rows=dev["logit_rows"] if sampled_rows else dev["cu_q"][1:2].long() - 1)
+                          logit_rows=dev["logit_rows"] if rows else dev["cu_q"][1:2].long() - 1)
         fb.max_kv_len = max(s.n_computed + n for s, n in plan)
         if self.state is not None:
             fb.state_slots_host = [s.state_slot for s, _ in plan]
             fb.state_slots = dev["state_slots"]
             fb.q_lens_host = [n for _, n in plan]
             fb.start_host = [s.n_computed for s, _ in plan]
-        fb.want_hidden = bool(self.spec_k) and bool(sampled_rows)
-        logits = self.model.forward(fb, self.kv, self.state) if self.state is not None else self.model.forward(fb, self.kv)
-        if fb.want_hidden:
-            logits, hidden = logits
-            for r, s in enumerate(seqs):
-                s.h_last = hidden[r:r + 1]
-        if not sampled_rows:
-            return []
-        toks = self._sample(logits, seqs)
-        out = toks.cpu()
-        self.stats["d2h_bytes"] += out.numel() * 4
-        return out.tolist()
+        fb.want_hidden = bool(self.spec_k) and bool(rows)
+        return self.model.forward(fb, self.kv, self.state) if self.state is not None else self.model.forward(fb, self.kv)
 
     def _sample(self, logits: torch.Tensor, seqs: list) -> torch.Tensor:
         if all(s.params.temperature <= 0 and s.params.repetition_penalty == 1.0 for s in seqs):
@@ -594,7 +653,8 @@ class LLMEngine:
         return out
 
     # ------------------------------------------------------------------ CUDA-graphed greedy decode
-    def _run_graph(self, plan: list) -> list:
+    def _replay_decode(self, plan: list) -> dict:
+        """One token per sequence; the graph's "out" holds the arg-max tokens and "logits" the logits, one row per sequence."""
         B = len(plan)
         gb = next(b for b in self.opts.graph_batch_sizes if b >= B)
         host, _ = self._build_batch(plan, list(range(B)), pad_to=gb)
@@ -609,17 +669,15 @@ class LLMEngine:
         from ..ops import cuda as kernels
         kernels._count(g["kernels"])
         self.stats["graph_replays"] += 1
-        out = g["out"].cpu()
-        self.stats["d2h_bytes"] += out.numel() * 4
-        return out[:B].tolist()
+        return g
 
     # ------------------------------------------------------------------ CUDA-graphed prefill chunks
-    def _run_prefill_graph(self, plan: list, sampled_rows: list, seqs: list) -> list:
+    def _replay_prefill(self, plan: list) -> dict:
         """A single-sequence prefill chunk of n tokens (n a multiple of the KV block) has fixed shapes: its whole forward is one
         graph replay.  With tensor parallelism the per-kernel GPU time shrinks with the rank count while the host cost of
         ~500 launches does not, so an eager prefill becomes launch-bound; the graph removes that floor."""
         seq, n = plan[0]
-        host, max_q = self._build_batch(plan, [0])            # always one logit row: the chunk's last token
+        host, max_q = self._build_batch(plan, [n - 1])        # always one logit row: the chunk's last token
         key = ("prefill", n)
         g = self._graphs.get(key)
         if self.state is not None and seq.n_computed == 0:
@@ -634,11 +692,7 @@ class LLMEngine:
         from ..ops import cuda as kernels
         kernels._count(g["kernels"])
         self.stats["graph_replays"] += 1
-        if not sampled_rows:
-            return []
-        toks = self._sample(g["logits"], seqs).cpu()
-        self.stats["d2h_bytes"] += toks.numel() * 4
-        return toks.tolist()
+        return g
 
     def _capture(self, gb: int, host: dict, prefill_tokens: int = 0) -> dict:
         dev = {k: v.to(self.device) for k, v in host.items()}
@@ -668,14 +722,15 @@ class LLMEngine:
         from ..ops import cuda as kernels
         n0 = kernels.launches()
         with torch.cuda.graph(graph, pool=self._graph_pool):
-            out = post(fwd())
+            logits = fwd()
+            out = post(logits)
         n_kernels = kernels.launches() - n0          # kernels recorded in the graph: every replay launches them again
         if snap is not None:
             for sl, sn in snap.items():
                 self.state.restore(sl, sn)
         if self._graph_pool is None:
             self._graph_pool = graph.pool()
-        return {"graph": graph, "in": dev, "out": out, "logits": out, "kernels": n_kernels}
+        return {"graph": graph, "in": dev, "out": out, "logits": logits, "kernels": n_kernels}
 
     # ------------------------------------------------------------------ convenience
     def generate(self, prompts: list, params: Optional[SamplingParams] = None) -> list:

@@ -15,6 +15,13 @@ def _yarn_corr_dim(n_dims: int, n_ctx_orig: int, n_rot: float, base: float) -> f
     return n_dims * math.log(n_ctx_orig / (n_rot * 2 * math.pi)) / (2 * math.log(base))
 
 
+def query_temperature_table(max_pos: int, coef: float, every: float, device="cpu") -> torch.Tensor:
+    """fp32 [max_pos]: the factor 1 + coef * ln(floor((p + 1) / every) + 1) of a query at position p (attention that sharpens with the
+    length of what it looks back on), formed in fp64."""
+    p = torch.arange(1, max_pos + 1, dtype=torch.float64)
+    return (1.0 + coef * torch.log(torch.floor(p / every) + 1.0)).to(torch.float32).to(device).contiguous()
+
+
 def rope_tables(max_pos: int, n_rot: int, theta: float, freq_factors: Optional[torch.Tensor] = None, scaling_type: str = "none",
                 scaling_factor: float = 1.0, orig_ctx: int = 0, beta_fast: float = 32.0, beta_slow: float = 1.0,
                 device="cpu") -> tuple[torch.Tensor, torch.Tensor]:
