@@ -381,7 +381,7 @@ static __device__ int g_attn_tickets[ATT_TICKET_SLOTS * ATT_TICKETS_PER_SLOT];
 template <typename T, int HD, int PPW, bool EXACT>
 static int launch_partial(const AttnParams& p, cudaStream_t st) {
   constexpr int PAIRS = ATT_WARPS * PPW;
-  constexpr size_t SMEM_MAX = 227 * 1024;
+  constexpr size_t SMEM_MAX = 226 * 1024;             // (the kernel also has a few static bytes)
   const size_t smem = (size_t)PAIRS * p.dk * 4 + (size_t)ATT_TILE * (p.dk + att_kpad<T>()) * sizeof(T) + (size_t)ATT_TILE * p.dv * sizeof(T);
   if (smem > SMEM_MAX) return -112;
   auto kern = attn_partial_kernel<T, HD, PPW, EXACT>;
