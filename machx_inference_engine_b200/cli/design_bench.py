@@ -1,0 +1,222 @@
+"""Throughput of a layer-list design beside the framework's closest models at equal size, and its kernels beside the like kernels.
+
+    python bench.py --design tikarax [--design-part models|kernels|all]
+
+Models (random-init bf16 weights, random tokens): prefill of one 4096-token prompt and decode at a 2048-token context for 1, 8 and 32
+sequences, through ``LLMEngine`` (CUDA graphs as in serving), for
+  * the design as its preset orders it (one attention layer in four, minGRU otherwise),
+  * the design with attention in every layer,
+  * a llama of the same width, heads and parameters per layer (gated feed-forward of 2/3 the width),
+  * a DeltaNet hybrid (qwen35) of the same width, with full attention in every fourth layer.
+Weights are larger than L2 (126 MB), so every pass streams them.
+
+Kernels: device time inside a CUDA graph over buffers that together exceed L2, as a fraction of the roofline (bytes over the measured copy
+rate or FLOPs over the measured bf16 rate, whichever is longer), each beside the kernel that does the like work in the closest models.
+"""
+from __future__ import annotations
+
+import gc
+import json
+import sys
+import time
+
+import torch
+
+from ..formats.model_config import ModelConfig, _tikarax_preset
+
+LAYERS = 8
+SIZES = {  # hidden, heads, kv_heads, head width, un-gated feed-forward, minGRU width
+    "1b-layers": dict(hidden=2048, heads=32, kv_heads=8, dim=64, ffn=12288, width=4096),
+    "8b-layers": dict(hidden=4096, heads=32, kv_heads=8, dim=128, ffn=21504, width=6144),
+}
+VOCAB = 32768
+PREFILL, CONTEXT, DECODE = 4096, 2048, 64
+
+
+def _configs(s: dict) -> dict:
+    tk = lambda every: _tikarax_preset(s["hidden"], LAYERS, s["heads"], s["kv_heads"], s["dim"], s["dim"], s["ffn"], s["width"], VOCAB, attn_every=every)
+    common = dict(n_layers=LAYERS, hidden=s["hidden"], n_heads=s["heads"], n_kv_heads=s["kv_heads"], ffn=s["ffn"] * 2 // 3, vocab=VOCAB, ctx_train=16384)
+    return {"tikarax": tk(4), "tikarax, attention only": tk(1),
+            "llama": ModelConfig(arch="llama", head_dim=s["dim"], n_rot=s["dim"], **common),
+            "qwen35 hybrid": ModelConfig(arch="qwen35", head_dim=s["dim"], n_rot=s["dim"] // 2, full_attn_interval=4, ssm_inner=32 * 128, ssm_state=128,
+                                         ssm_n_k_heads=16, ssm_n_v_heads=32, ssm_conv_kernel=4, **common)}
+
+
+def _timed(fn) -> float:
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    e0.record()
+    fn()
+    e1.record()
+    torch.cuda.synchronize()
+    return e0.elapsed_time(e1)
+
+
+def bench_models(dev, emit) -> None:
+    from ..models import build_model
+    from ..ops import cuda as K
+    from ..runtime.engine import EngineOptions, LLMEngine, SamplingParams
+    for size, s in SIZES.items():
+        for name, cfg in _configs(s).items():
+            model = build_model(cfg, dev, quant="bf16", max_ctx=PREFILL + 256)
+            row = {"size": size, "model": name, "layers": LAYERS, "weight_gb": round(model.weight_bytes() / 1e9, 2)}
+            g = torch.Generator().manual_seed(0)
+            prompt = lambda n: torch.randint(0, VOCAB, (n,), generator=g).tolist()
+            eng = LLMEngine(model, EngineOptions(max_ctx=PREFILL + 256, max_batch_tokens=PREFILL, max_seqs=1, enable_prefix_cache=False))
+
+            def prefill():
+                eng.add_request(prompt(PREFILL), SamplingParams(max_tokens=1))
+                eng.step()
+            for _ in range(3):
+                prefill()
+            ms = sorted(_timed(prefill) for _ in range(5))[2]
+            row["prefill_tok_s"] = round(PREFILL / ms * 1e3)
+            row["prefill_ms"] = round(ms, 3)
+            del eng
+            for B in (1, 8, 32):
+                eng = LLMEngine(model, EngineOptions(max_ctx=CONTEXT + 256, max_batch_tokens=CONTEXT, max_seqs=B, enable_prefix_cache=False))
+                for _ in range(B):
+                    eng.add_request(prompt(CONTEXT), SamplingParams(max_tokens=DECODE + 32, ignore_eos=True))
+                while any(q.n_computed < len(q.prompt) for q in eng.sched.running) or eng.sched.waiting:
+                    eng.step()
+                for _ in range(4):
+                    eng.step()
+                n0, n = eng.stats["decode_tokens"], 0
+
+                def decode():
+                    for _ in range(DECODE // 2):
+                        eng.step()
+                ms = _timed(decode)
+                n = eng.stats["decode_tokens"] - n0
+                row[f"decode_b{B}_tok_s"] = round(n / ms * 1e3)
+                row[f"decode_b{B}_ms"] = round(ms / (DECODE // 2), 3)
+                del eng
+            K.check_status()
+            emit(row)
+            del model
+            gc.collect()
+            torch.cuda.empty_cache()
+
+
+def _per_call(fns: list, reps: int = 40) -> float:
+    """Microseconds per call of the functions (same work on different buffers), cycled inside one CUDA graph."""
+    n = max(reps, len(fns))
+    side = torch.cuda.Stream()
+    side.wait_stream(torch.cuda.current_stream())
+    with torch.cuda.stream(side):
+        for f in fns:
+            f()
+    torch.cuda.current_stream().wait_stream(side)
+    g = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(g):
+        for i in range(n):
+            fns[i % len(fns)]()
+    for _ in range(3):
+        g.replay()
+    return sorted(_timed(g.replay) for _ in range(7))[3] * 1e3 / n
+
+
+def bench_kernels(dev, emit) -> None:
+    from ..ops import cuda as K
+    from ..ops import ref
+    from ..ops.weights import QuantWeight, WFormat
+    from ..utils.rope import query_temperature_table, rope_tables
+    from .kernel_bench import peaks
+    pk = peaks()
+    bf = lambda *sh: (torch.randn(*sh, device=dev) * 0.5).to(torch.bfloat16)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    bufs = lambda nbytes: max(2, int(3e8 // nbytes) + 1) if nbytes < 3e8 else 1
+
+    def row(kernel, role, fns, bytes_=0.0, flops=0.0):
+        us = _per_call(fns)
+        roof = max(bytes_ / pk["hbm_gbs"] / 1e3, flops / pk["bf16_tflops"] / 1e6)
+        emit({"kernel": kernel, "role": role, "us": round(us, 2), "gbs": round(bytes_ / us / 1e3) if bytes_ else None,
+              "tflops": round(flops / us / 1e6, 1) if flops else None, f"fraction_of_{pk['src']}_roofline": round(roof / us, 3)})
+
+    for size, s in SIZES.items():
+        H, W, F, nq, nkv, d = s["hidden"], s["width"], s["ffn"], s["heads"], s["kv_heads"], s["dim"]
+        for T in (1, 32, PREFILL):
+            # ---- norms: both sides of a sublayer in one pass, against residual add + norm
+            nb = bufs(T * H * 12) if T > 64 else 8
+            xs, ds, w = [torch.randn(T, H, device=dev) for _ in range(nb)], [bf(T, H) for _ in range(nb)], torch.ones(H, device=dev)
+            by = T * H * (4 + 4 + 2 + 2)
+            row(f"group_norm (branch norm + add + norm) T={T} H={H}", "new", [lambda x=x, q=q: K.group_norm(x, w, 1e-6, 2, delta=q, delta_w=w) for x, q in zip(xs, ds)], by)
+            row(f"rmsnorm (add + norm) T={T} H={H}", "like", [lambda x=x, q=q: K.rmsnorm(x, w, 1e-6, delta=q) for x, q in zip(xs, ds)], by)
+            # ---- up projection with its activation
+            ws = [QuantWeight(WFormat.BF16, F, H, 1, bf(1, F, H)) for _ in range(bufs(F * H * 2))]
+            gs = [QuantWeight(WFormat.BF16, F // 3 * 4 // 32 * 32, H, 1, bf(1, F // 3 * 4 // 32 * 32, H)) for _ in range(bufs(F * H * 2))]
+            h = bf(T, H)
+            fl = 2.0 * T * F * H
+            row(f"up + xIELU T={T} {F}x{H}", "new", [lambda m=m: K.linear(h, m, act=ref.ACT_XIELU, act_alpha=0.8, act_limit=1.2) for m in ws], F * H * 2 + T * (H + F) * 2, fl)
+            row(f"plain projection T={T} {F}x{H}", "like", [lambda m=m: K.linear(h, m) for m in ws], F * H * 2 + T * (H + F) * 2, fl)
+            N = gs[0].N
+            row(f"gate|up + SwiGLU T={T} {N}x{H}", "like", [lambda m=m: K.linear(h, m, act=ref.ACT_SWIGLU) for m in gs], N * H * 2 + T * (H + N // 2) * 2, 2.0 * T * N * H)
+            del ws, gs
+        # ---- recurrence
+        for B, n in ((1, PREFILL), (8, 512), (1, 1), (32, 1)):
+            T = B * n
+            nb = bufs(T * W * 8) if T > 64 else 8
+            ys, st = [bf(T, 3 * W) for _ in range(nb)], torch.zeros(B, W, device=dev)
+            zb, slots, cu, sl = torch.zeros(W, device=dev), i32(list(range(B))), i32([i * n for i in range(B + 1)]), i32([n + 64] * B)
+            row(f"mingru_scan B={B} n={n} W={W}", "new",
+                [lambda y=y: K.mingru_scan(y[:, :W], y[:, W:2 * W], y[:, 2 * W:], zb, zb, st, slots, cu, sl, n) for y in ys], T * W * 8 + B * W * 8)
+            C = 8192
+            xs, cw, cs = [bf(T, C) for _ in range(bufs(T * C * 4) if T > 64 else 8)], torch.randn(C, 4, device=dev), torch.zeros(B, 3, C, dtype=torch.bfloat16, device=dev)
+            row(f"conv1d_silu B={B} n={n} C={C}", "like", [lambda x=x: K.conv1d_silu(x, cw, cs, slots, cu, n) for x in xs], T * C * 4 + B * 3 * C * 4)
+            nv, nk = 32, 16
+            ab, ai, S = bf(T, 2 * nv), i32(list(range(nv))), torch.zeros(B, nv, 128, 128, device=dev)
+            kv, sa = (ai // 2).to(torch.int32), -torch.rand(nv, device=dev)
+            row(f"deltanet_scan B={B} n={n} heads={nk}/{nv}", "like",
+                [lambda x=x: K.deltanet_scan(x, nk, ab, ai, ai + nv, kv, sa, sa, S, slots, cu, nv) for x in xs], T * C * 2 + T * nv * 128 * 4 + 2 * S.numel() * 4)
+        # ---- attention, epilogue
+        temp = query_temperature_table(2 * PREFILL, 0.1, 512, device=dev)
+        cos, sin = rope_tables(2 * PREFILL, d, 1e4, device=dev)
+        for B, n, ctx in ((1, PREFILL, PREFILL), (1, 1, 8192), (1, 1, 2048), (32, 1, 2048)):
+            T, nblk = B * n, (ctx + 127) // 128
+            pages = B * nblk + 1
+            nb = min(16, bufs(pages * nkv * 128 * d * 4)) if n == 1 else 2
+            kc, vc = [bf(pages, nkv, 128, d) for _ in range(nb)], [bf(pages, nkv, 128, d) for _ in range(nb)]
+            bt = torch.arange(1, pages, dtype=torch.int32, device=dev).reshape(B, nblk)
+            sl, cu = i32([ctx] * B), i32([i * n for i in range(B + 1)])
+            y, q = bf(T, (2 * nq + 2 * nkv) * d), bf(T, nq, d)
+            keys = n * ctx - n * (n - 1) // 2
+            by, fl = B * ctx * nkv * d * 4 + T * nq * d * 4, 4.0 * B * keys * nq * d
+            row(f"attention + gate + temperature B={B} n={n} ctx={ctx} {nq}/{nkv}x{d}", "new",
+                [lambda k=k, v=v: K.attention(y[:, :nq * d].view(T, nq, d), k, v, bt, sl, cu, n, scale=d ** -0.5, q_scale=temp, gate=y[:, -nq * d:]) for k, v in zip(kc, vc)],
+                by + T * nq * d * 2, fl)
+            row(f"attention B={B} n={n} ctx={ctx} {nq}/{nkv}x{d}", "like", [lambda k=k, v=v: K.attention(q, k, v, bt, sl, cu, n, scale=d ** -0.5) for k, v in zip(kc, vc)], by, fl)
+            if d == 128 and ctx != 8192:      # widths that differ and fill no tile: 96-wide keys, 128-wide values
+                k96 = [bf(pages, nkv, 128, 96) for _ in range(nb)]
+                q96 = bf(T, nq, 96)
+                row(f"attention + gate, 96-wide keys B={B} n={n} ctx={ctx}", "new",
+                    [lambda k=k, v=v: K.attention(q96, k, v, bt, sl, cu, n, scale=0.1, q_scale=temp, gate=y[:, -nq * d:]) for k, v in zip(k96, vc)],
+                    B * ctx * nkv * (96 + d) * 2 + T * nq * (96 + 2 * d) * 2, 2.0 * B * keys * nq * (96 + d))
+                del k96
+            slots = torch.arange(128, 128 + T, dtype=torch.int64, device=dev)
+            pos = torch.arange(T, dtype=torch.int32, device=dev)
+            if ctx != 8192:
+                nb2 = bufs(T * nkv * d * 8) if T > 64 else 8
+                yk = [bf(T, (2 * nq + 2 * nkv) * d) for _ in range(min(nb2, 8))]
+                row(f"kv_store T={T}", "new", [lambda t=t: K.kv_store(t[:, nq * d:(nq + nkv) * d], t[:, (nq + nkv) * d:(nq + 2 * nkv) * d], slots, kc[0], vc[0]) for t in yk], T * nkv * d * 8)
+                yp = [t[:, :(nq + 2 * nkv) * d].contiguous() for t in yk]
+                row(f"qkv_post T={T}", "like", [lambda t=t: K.qkv_post(t, None, None, None, pos, cos, sin, slots, kc[0], vc[0], nq, nkv, d, d) for t in yp],
+                    T * (nq * d * 4 + nkv * d * 8))
+            del kc, vc
+            torch.cuda.empty_cache()
+    K.check_status()
+
+
+def main(part: str = "all") -> int:
+    dev = torch.device("cuda:0")
+    torch.cuda.set_device(dev)
+    t0 = time.time()
+
+    def emit(obj):
+        print(json.dumps(obj))
+        sys.stdout.flush()
+    if part in ("all", "models"):
+        bench_models(dev, emit)
+    if part in ("all", "kernels"):
+        bench_kernels(dev, emit)
+    emit({"design_bench": "done", "seconds": round(time.time() - t0, 1)})
+    return 0

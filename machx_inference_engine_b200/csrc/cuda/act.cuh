@@ -23,9 +23,16 @@ __device__ __forceinline__ float act_unary(int act, float z, float a, float b) {
   return act == ACT_CODE_XIELU ? xielu<PRECISE>(z, a, b) : z;
 }
 
-// sigmoid with the fast or the full-precision exponential
+// sigmoid with the full-precision exponential and division, or with the hardware's base-2 exponential and reciprocal (a few units in
+// the last place of fp32; the exponential overflows to infinity below about -88 and the result is 0)
 template <bool PRECISE>
-__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + (PRECISE ? expf(-x) : __expf(-x))); }
+__device__ __forceinline__ float sigmoid_f(float x) {
+  if constexpr (PRECISE) return 1.f / (1.f + expf(-x));
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * -1.4426950408889634f));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+  return r;
+}
 
 // ---------------------------------------------------------------- element types of activations (bf16 or fp32)
 template <typename T> __device__ __forceinline__ float to_f32(T v);

@@ -215,6 +215,10 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     const bool early = !CAP && !(qs > 0.f);
     const float c = (CAP || early) ? 1.f : qs * LOG2E;
     const float cap_c = p.softcap * LOG2E, inv_cap = CAP ? qs / p.softcap : 0.f;
+    if (p.gate && row_ok) {                        // bring the row's gate into L2 while the keys are walked
+      const __nv_bfloat16* g0 = p.gate + (size_t)(q_begin + t0 + r) * p.gate_ld + (size_t)head * p.dv;
+      for (int i = 0; i < p.dv; i += 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(g0 + i));
+    }
     float m = -1e30f, l = 0.f;                     // reference maximum (log2 units) and running denominator
     const uint32_t lane_addr = (uint32_t)(q4 * 32) << 16;
     bool ok = true;
@@ -297,16 +301,25 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       __syncwarp();
       if (lane == 0) mbar_arrive(b_pfull);
     }
+    const int dv = p.dv;
+    const __nv_bfloat16* grow = p.gate && row_ok ? p.gate + (size_t)(q_begin + t0 + r) * p.gate_ld + (size_t)head * dv : nullptr;
+    // the first GPRE columns of the row's gate travel while the last PV runs (the score registers are free here)
+    constexpr int GPRE = DV < 128 ? DV : 128;
+    uint4 gpre[GPRE / 8];
+    if (grow) {
+#pragma unroll
+      for (int i = 0; i < GPRE / 8; ++i)
+        if (8 * i < dv) gpre[i] = __ldg(reinterpret_cast<const uint4*>(grow + 8 * i));
+    }
     if (ok && n_tiles > 0) ok = mbar_wait(b_pvdone, (n_tiles - 1) & 1, p.status, ERR_MBAR_TIMEOUT_SOFTMAX, abort_flag);
     if (ok) {
       tc_fence_after();
       if (p.sinks) l += ex2_fast(p.sinks[head] * LOG2E - m);
       const float inv = l > 0.f ? 1.f / l : 0.f;
-      const int dv = p.dv;
       __nv_bfloat16* orow = p.out + ((size_t)(q_begin + t0 + r) * p.n_q + head) * dv;
-      const __nv_bfloat16* grow = p.gate ? p.gate + (size_t)(q_begin + t0 + r) * p.gate_ld + (size_t)head * dv : nullptr;
-#pragma unroll 1
+#pragma unroll
       for (int cb = 0; cb < DV; cb += 32) {
+        if (cb >= dv) break;
         uint32_t ov[32];
         if (n_tiles > 0) {
           tmem_ld_32x32(tmem_o + lane_addr + cb, ov);
@@ -323,7 +336,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
 #pragma unroll
             for (int e = 0; e < 8; ++e) o[e] = __uint_as_float(ov[i + e]) * inv;
             if (grow) {
-              const uint4 g4 = *reinterpret_cast<const uint4*>(grow + cb + i);
+              const uint4 g4 = cb + i < GPRE ? gpre[(cb + i) < GPRE ? (cb + i) / 8 : 0] : __ldg(reinterpret_cast<const uint4*>(grow + cb + i));
               const uint32_t gw[4] = {g4.x, g4.y, g4.z, g4.w};
 #pragma unroll
               for (int e = 0; e < 4; ++e) {

@@ -156,7 +156,7 @@ __global__ void __launch_bounds__(256) rmsnorm_combine_kernel(float* __restrict_
 //   x  (fp32 residual) = (FRESH ? 0 : x) + norm(delta) * delta_w      (delta null: x is only read)
 //   out               = norm(x) * w                                   (out null: skipped)
 // Rows have ld elements (ld >= H, multiple of 4); columns H.. are padding: written as zeros in out (and in x when it starts fresh).
-// A team of `wpg` warps owns a group; with more groups than warps the teams (one warp each) walk over them.
+// A team of `wpg` warps owns one (row, group); a CTA holds 8 / wpg teams, which work on consecutive groups and never wait for each other.
 struct GroupNormParams {
   float* x;
   const void* delta;
@@ -164,20 +164,21 @@ struct GroupNormParams {
   const float* w;
   void* out;
   float eps;
-  int H, ld, groups, gs, wpg, fresh;      // gs = H / groups
+  int T, H, ld, groups, gs, wpg, fresh;   // gs = H / groups
 };
 constexpr int GN_WARPS = 8;
+constexpr int GN_LANE_MAX = 16;          // elements of a group that a lane holds, before the team gets more warps
 
-// sum over the warps of a team; every warp of the block calls it (barrier) when a team has more than one warp
+// sum over the warps of a team (a team of several warps meets at its own named barrier)
 __device__ __forceinline__ float team_sum(float v, float* red, int warp, int wpg) {
   v = warp_sum(v);
   if (wpg == 1) return v;
-  __syncthreads();                        // readers of the previous use are done
+  const int team = warp / wpg, first = team * wpg;
+  asm volatile("bar.sync %0, %1;" ::"r"(1 + team), "r"(wpg * 32) : "memory");     // readers of the previous use are done
   if ((threadIdx.x & 31) == 0) red[warp] = v;
-  __syncthreads();
-  const int first = warp - warp % wpg;
+  asm volatile("bar.sync %0, %1;" ::"r"(1 + team), "r"(wpg * 32) : "memory");
   float t = 0.f;
-  for (int i = 0; i < wpg && first + i < GN_WARPS; ++i) t += red[first + i];
+  for (int i = 0; i < wpg; ++i) t += red[first + i];
   return t;
 }
 
@@ -187,17 +188,18 @@ __global__ void __launch_bounds__(GN_WARPS * 32) group_norm_kernel(const GroupNo
   pdl_prologue();
   __shared__ float red[GN_WARPS];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const size_t row = (size_t)blockIdx.x * p.ld;
+  const int wpg = p.wpg;
+  const unsigned unit = blockIdx.x * (GN_WARPS / wpg) + warp / wpg;      // (T * groups fits 32 bits: checked by the host)
+  if (unit >= (unsigned)p.T * p.groups) return;            // a whole team leaves
+  const unsigned t = unit / (unsigned)p.groups;
+  const int g = (int)(unit - t * p.groups);
+  const size_t row = (size_t)t * p.ld;
   float* xr = p.x + row;
   const DT* dr = reinterpret_cast<const DT*>(p.delta) + row;
   OT* orow = reinterpret_cast<OT*>(p.out) + row;
-  const int wpg = p.wpg, teams = GN_WARPS / wpg, team = warp / wpg;
-  const int first = (warp % wpg) * 32 + lane, step = wpg * 32, pieces = p.gs / V;
+  const int first = (warp % wpg) * 32 + lane, step = wpg * 32, n = p.gs / V, base = g * p.gs;
   const float inv_n = 1.f / (float)p.gs;
-  for (int g0 = 0; g0 < p.groups; g0 += teams) {
-    const int g = g0 + team;
-    const bool live = team < teams && g < p.groups;        // idle warps still reach the team barriers
-    const int base = g * p.gs, n = live ? pieces : 0;
+  {
     if constexpr (NV > 0) {
       float xv[NV][V];
       float ss = 0.f;
@@ -300,10 +302,11 @@ __global__ void __launch_bounds__(GN_WARPS * 32) group_norm_kernel(const GroupNo
       }
     }
   }
-  for (int i = p.H + threadIdx.x; i < p.ld; i += blockDim.x) {
-    if (p.out) orow[i] = from_f32<OT>(0.f);
-    if (p.fresh) xr[i] = 0.f;
-  }
+  if (g == p.groups - 1)
+    for (int i = p.H + first; i < p.ld; i += step) {
+      if (p.out) orow[i] = from_f32<OT>(0.f);
+      if (p.fresh) xr[i] = 0.f;
+    }
 }
 
 // ------------------------------------------------------------------ kv_store
@@ -666,15 +669,20 @@ MX_HOST_API int mx_rmsnorm_combine(float* x, const void* yp, const int* pair_to_
 
 namespace mx {
 template <typename DT, typename OT>
-static int launch_group_norm(const GroupNormParams& p, int T, cudaStream_t st) {
-  const int lanes = 32 * p.wpg;
+static int launch_group_norm(GroupNormParams p, cudaStream_t st) {
   const bool v4 = p.gs % 4 == 0;
-  const int per_lane = v4 ? (p.gs / 4 + lanes - 1) / lanes : 0;
-  if (v4 && per_lane <= 2) launch_pdl(group_norm_kernel<DT, OT, 4, 2>, dim3(T), dim3(GN_WARPS * 32), 0, st, p);
-  else if (v4 && per_lane <= 4) launch_pdl(group_norm_kernel<DT, OT, 4, 4>, dim3(T), dim3(GN_WARPS * 32), 0, st, p);
-  else if (v4 && per_lane <= 8) launch_pdl(group_norm_kernel<DT, OT, 4, 8>, dim3(T), dim3(GN_WARPS * 32), 0, st, p);
-  else if (v4) launch_pdl(group_norm_kernel<DT, OT, 4, 0>, dim3(T), dim3(GN_WARPS * 32), 0, st, p);
-  else launch_pdl(group_norm_kernel<DT, OT, 1, 0>, dim3(T), dim3(GN_WARPS * 32), 0, st, p);
+  const long long units = (long long)p.T * p.groups;
+  // warps per group: enough that a lane holds at most 16 elements, then more while the chip has room for them (4096 rows of 2 x 2048:
+  // 37 us with 16 elements per lane, 49 with 8, 58 with 32)
+  p.wpg = 1;
+  while (p.wpg < GN_WARPS && (p.gs > 32 * p.wpg * GN_LANE_MAX || (units * p.wpg < 16ll * sm_count() && p.gs > 32 * p.wpg * 4))) p.wpg *= 2;
+  const dim3 grid((unsigned)((units + GN_WARPS / p.wpg - 1) / (GN_WARPS / p.wpg))), block(GN_WARPS * 32);
+  const int lanes = 32 * p.wpg, per_lane = v4 ? (p.gs / 4 + lanes - 1) / lanes : 0;
+  if (v4 && per_lane <= 2) launch_pdl(group_norm_kernel<DT, OT, 4, 2>, grid, block, 0, st, p);
+  else if (v4 && per_lane <= 4) launch_pdl(group_norm_kernel<DT, OT, 4, 4>, grid, block, 0, st, p);
+  else if (v4 && per_lane <= 8) launch_pdl(group_norm_kernel<DT, OT, 4, 8>, grid, block, 0, st, p);
+  else if (v4) launch_pdl(group_norm_kernel<DT, OT, 4, 0>, grid, block, 0, st, p);
+  else launch_pdl(group_norm_kernel<DT, OT, 1, 0>, grid, block, 0, st, p);
   return (int)cudaGetLastError();
 }
 }  // namespace mx
@@ -683,14 +691,13 @@ static int launch_group_norm(const GroupNormParams& p, int T, cudaStream_t st) {
 MX_HOST_API int mx_group_norm(float* x, const void* delta, int delta_is_f32, const float* delta_w, const float* w, void* out, int out_is_f32,
                               float eps, int T, int H, int ld, int groups, int fresh, cudaStream_t st) {
   if (T <= 0) return 0;
-  if (groups < 1 || H < groups || H % groups || ld < H || ld % 4) return -107;
+  if (groups < 1 || H < groups || H % groups || ld < H || ld % 4 || (long long)T * groups > 0x7fffffffll) return -107;
   if ((delta && !delta_w) || (out && !w) || (fresh && !delta)) return -109;
   GroupNormParams p;
   p.x = x; p.delta = delta; p.delta_w = delta_w; p.w = w; p.out = out; p.eps = eps; p.H = H; p.ld = ld; p.groups = groups; p.gs = H / groups;
-  p.wpg = groups >= GN_WARPS ? 1 : GN_WARPS / groups;
-  p.fresh = fresh;
-  if (delta_is_f32) return out_is_f32 ? launch_group_norm<float, float>(p, T, st) : launch_group_norm<float, __nv_bfloat16>(p, T, st);
-  return out_is_f32 ? launch_group_norm<__nv_bfloat16, float>(p, T, st) : launch_group_norm<__nv_bfloat16, __nv_bfloat16>(p, T, st);
+  p.T = T; p.fresh = fresh;
+  if (delta_is_f32) return out_is_f32 ? launch_group_norm<float, float>(p, st) : launch_group_norm<float, __nv_bfloat16>(p, st);
+  return out_is_f32 ? launch_group_norm<__nv_bfloat16, float>(p, st) : launch_group_norm<__nv_bfloat16, __nv_bfloat16>(p, st);
 }
 
 // k / v: rows of n_kv * dk / n_kv * dv elements, k_ld / v_ld elements apart; elem_bytes 2 or 4; every row, head and stride a multiple of 16 bytes.

@@ -11,6 +11,7 @@ but works at KV-block granularity so hits are shared between live requests witho
 """
 from __future__ import annotations
 
+import gc
 import hashlib
 import itertools
 import time
@@ -721,9 +722,17 @@ class LLMEngine:
         graph = torch.cuda.CUDAGraph()
         from ..ops import cuda as kernels
         n0 = kernels.launches()
-        with torch.cuda.graph(graph, pool=self._graph_pool):
-            logits = fwd()
-            out = post(logits)
+        # a dropped engine is cyclic garbage, and destroying its graphs while this stream captures would invalidate the capture
+        gc.collect()
+        gc_on = gc.isenabled()
+        gc.disable()
+        try:
+            with torch.cuda.graph(graph, pool=self._graph_pool):
+                logits = fwd()
+                out = post(logits)
+        finally:
+            if gc_on:
+                gc.enable()
         n_kernels = kernels.launches() - n0          # kernels recorded in the graph: every replay launches them again
         if snap is not None:
             for sl, sn in snap.items():
