@@ -127,9 +127,11 @@ class QuantWeight:
         return w
 
     def pad_groups(self, rows: Optional[tuple] = None, cols: Optional[tuple] = None) -> "QuantWeight":
-        """bf16 only: (groups, size) on the rows / columns -- each of ``groups`` equal runs is padded with zeros to ``size`` elements, so that
+        """(groups, size) on the rows / columns (bf16 unless nothing has to be padded) -- each of ``groups`` equal runs is padded with zeros to ``size`` elements, so that
         head or feature ranges start where the kernels' vector accesses want them.  A padded row gives a zero output, a padded column
         meets a zero activation: the product is unchanged."""
+        if all(spec is None or n == spec[0] * spec[1] for spec, n in ((rows, self.N), (cols, self.K))):
+            return self
         if self.fmt != WFormat.BF16:
             raise ValueError(f"only bf16 weights can be padded, not {self.fmt.name}")
         t = self.p0

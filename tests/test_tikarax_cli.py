@@ -132,6 +132,31 @@ def test_pool_is_made_for_the_tokens_of_live_requests(tmp_path):
         assert eng.bm.num_blocks * 128 <= limit + 4 * 64 + 256
 
 
+def test_quantised_weights_need_widths_that_are_not_padded():
+    from machx_inference_engine_b200.runtime.engine import EngineOptions, LLMEngine
+    aligned = read_json_config(oracle.random_config([A(4, 2, 32, 64, 128), M(96, 64)], vocab=96, width=64))
+    toks, out = tokens_of(50, 96), {}
+    for quant in ("bf16", "q8_0"):
+        eng = LLMEngine(build_model(aligned, "cpu", quant=quant, max_ctx=128), EngineOptions(max_ctx=128, max_seqs=1))
+        out[quant] = eng.feed([(eng.open_sequence(), toks, list(range(50)))]).numpy()
+    assert 1e-4 < logit_error(out["q8_0"], out["bf16"]) < 0.1
+    with pytest.raises(ValueError, match="padded"):
+        build_model(preset("tiny-tikarax"), "cpu", quant="q8_0")
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("quant", ["bf16", "q8_0"])
+def test_quantised_weights_on_the_gpu(quant):
+    from machx_inference_engine_b200.runtime.engine import EngineOptions, LLMEngine
+    aligned = read_json_config(oracle.random_config([A(4, 2, 32, 64, 128), M(96, 64)], vocab=96, width=64))
+    toks, out = tokens_of(90, 96), {}
+    for dev in ("cpu", "cuda:0"):
+        eng = LLMEngine(build_model(aligned, torch.device(dev), quant=quant, max_ctx=128, gen_device="cpu"), EngineOptions(max_ctx=128, max_seqs=1))
+        seq = eng.open_sequence()
+        out[dev] = torch.cat([eng.feed([(seq, toks[:80], list(range(80)))])] + [eng.feed([(seq, [t], [0])]) for t in toks[80:]]).cpu().numpy()
+    assert logit_error(out["cuda:0"], out["cpu"]) < TOL["bf16"]
+
+
 def test_component_names_existing_sources():
     have = {p.stem for p in (_build.CSRC / "cuda").glob("*.cu")}
     assert all(set(v) <= have for v in _build.COMPONENTS.values())
