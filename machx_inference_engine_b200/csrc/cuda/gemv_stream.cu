@@ -903,6 +903,9 @@ gemv_stream_kernel(const GsParams p, const __grid_constant__ CUtensorMap tm0, co
 
 template <int FMT, int MM, bool GATED, int NG>
 static int gs_launch(const GsParams& p, int smem, cudaStream_t st) {
+  // the consumers read MM activation rows; the rows past M hold nothing that is stored, but they must lie inside the shared window (with
+  // 5 rows of 12288 elements, for one, the eighth would end past it)
+  if ((long long)MM * gs_xrow_bytes<FMT>(p.K) + 128 > smem) return 1;
   constexpr int THREADS = (GsCfg<FMT>::WARPS + 1) * 32;
   static DeviceOnce attr_done;
   if (attr_done.pending()) {

@@ -325,6 +325,15 @@ def _out_kind(dtype) -> int:
     return {torch.bfloat16: 0, torch.float32: 1, torch.float16: 2}[dtype]
 
 
+def _few_rows_take_gemm(M: int, w: QuantWeight, act: int) -> bool:
+    """A few rows against a bf16 matrix that the streaming GEMV serves badly: rows too long to sit in its shared memory beside two stages
+    (the register GEMV would run: 8 x 21504 against 4096 rows 392 us, the tensor-core kernel 74), or so much weight that five and more rows
+    are bound by its arithmetic (8 x 4096 against 21504 rows: 121 us against 55)."""
+    if w.fmt != WFormat.BF16 or act_gated(act) or w.K % 8:
+        return False
+    return (M >= 3 and 2 * M * w.K + 16 * min(w.K, 4096) > 190 * 1024) or (M >= 5 and w.N * w.K >= 48 << 20)
+
+
 def linear(x, w: QuantWeight, bias=None, act=ACT_NONE, act_alpha=1.702, act_limit=7.0, out_f32=False, row_scale=None, out=None):
     """``out``: write into this [M, n_out] view (unit column stride; a column slice of a wider matrix is fine), so that projections
     whose weights differ in format can share one output without a concatenation."""
@@ -344,7 +353,7 @@ def linear(x, w: QuantWeight, bias=None, act=ACT_NONE, act_alpha=1.702, act_limi
         return out
     fmt, p0, p1, p2, p3 = _planes(w)
     lib = _lib.cuda()
-    if M <= GEMV_MAX_M and row_scale is None:
+    if M <= GEMV_MAX_M and row_scale is None and not _few_rows_take_gemm(M, w, act):
         # the GEMV kernels write dense rows: a strided view of more than one row goes through a dense buffer
         dst = out if (M == 1 or out.stride(0) == n_out) else torch.empty(M, n_out, dtype=odt, device=x.device)
         _check(lib.mx_gemv(fmt, p0, p1, p2, p3, _p(x), _p(dst), _p(bias), M, w.N, w.K, int(out_f32), act, C.c_float(act_alpha),

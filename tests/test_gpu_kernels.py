@@ -10,7 +10,7 @@ import pytest
 import torch
 
 from machx_inference_engine_b200.ops import ref
-from machx_inference_engine_b200.ops.weights import WFormat, from_dense
+from machx_inference_engine_b200.ops.weights import QuantWeight, WFormat, from_dense
 
 pytestmark = pytest.mark.gpu
 
@@ -636,3 +636,19 @@ def test_run_twice_is_bit_identical():
     x = torch.randn(300, 1024, device=dev()).to(torch.bfloat16)
     a, b = K().gemm(x, qw, out_f32=True), K().gemm(x, qw, out_f32=True)
     assert torch.equal(a, b)
+
+
+@pytest.mark.parametrize("M", [3, 5, 6, 7])
+@pytest.mark.parametrize("K_", [12288, 14336])
+def test_gemv_of_a_few_long_rows(M, K_):
+    """Row counts between the kernel's instances (1, 2, 4, 8) with rows so long that the instance's last row would not fit shared memory."""
+    w = QuantWeight(WFormat.BF16, 64, K_, 1, (torch.randn(1, 64, K_, device=dev()) * 0.02).to(torch.bfloat16))
+    x = torch.randn(M, K_, device=dev()).to(torch.bfloat16)
+    want = ref.linear(x, w)
+    assert rel_err(K().linear(x, w), want) < 1e-2            # (some of these go to the tensor-core kernel)
+    keep = K()._few_rows_take_gemm
+    K()._few_rows_take_gemm = lambda *a: False
+    try:
+        assert rel_err(K().linear(x, w), want) < 1e-2
+    finally:
+        K()._few_rows_take_gemm = keep
