@@ -30,7 +30,8 @@ def _inspect_folder(path: str, tensors: bool, out) -> int:
         return 0
     mixers = Counter(s.mixer for s in c.layer_specs)
     print(f"config: arch={c.arch} layers={c.n_layers} ({', '.join(f'{n} {k}' for k, n in mixers.items())}) hidden={c.hidden} norm_groups={c.norm_groups} "
-          f"ffn={c.ffn} vocab={c.vocab}", file=out)
+          f"ffn={c.ffn} vocab={c.vocab}" + (f" experts={c.n_experts} (top {c.n_experts_used})" if c.n_experts else "")
+          + (f" loop={c.loop_start}..{c.loop_stop - 1} x {c.loop_times}" if c.loop_times else ""), file=out)
     return 0
 
 

@@ -78,7 +78,7 @@ def _folder_bytes(path: str, ctx: int, n_seqs: int) -> tuple:
     from .model_config import read_json_config
     c = read_json_config(path)
     weights = sum(os.path.getsize(os.path.join(path, f)) for f in os.listdir(path) if f.endswith(".safetensors"))
-    kv = sum(s.kv_heads * (s.key_dim + s.value_dim) for s in c.layer_specs) * ctx * 2 * n_seqs
+    kv = sum(c.layer_specs[l].kv_width() for l, _ in c.layer_runs()) * ctx * 2 * n_seqs
     return weights, kv, sum(s.width for s in c.layer_specs) * 4 * n_seqs
 
 

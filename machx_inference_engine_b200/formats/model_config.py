@@ -10,7 +10,7 @@ from __future__ import annotations
 import json
 import os
 from dataclasses import dataclass, field, asdict
-from typing import Any, Mapping
+from typing import Any, Mapping, Optional
 
 DENSE_ARCHS = ("llama", "qwen2", "qwen3", "phi3", "granite", "mistral")
 MOE_ARCHS = ("qwen3moe", "gpt-oss")
@@ -18,7 +18,7 @@ HYBRID_ARCHS = ("qwen3next", "qwen35", "qwen35moe")
 GEMMA_ARCHS = ("gemma4",)
 SUPPORTED_ARCHS = DENSE_ARCHS + MOE_ARCHS + HYBRID_ARCHS + GEMMA_ARCHS
 # checkpoints that are a folder with config.json + safetensors and list their layers one by one: "architecture" value -> arch
-LAYER_LIST_ARCHS = {"Tikarax": "tikarax"}
+LAYER_LIST_ARCHS = {"Tikarax": "tikarax", "Pubodra": "pubodra"}
 
 
 class ConfigError(ValueError):
@@ -27,9 +27,13 @@ class ConfigError(ValueError):
 
 @dataclass
 class LayerSpec:
-    """One layer of a design whose configuration lists its layers: a mixer with its sizes and constants, and a feed-forward (0 = none)."""
-    mixer: str                     # "attention" | "mingru"
+    """One layer of a design whose configuration lists its layers: a mixer with its sizes and constants, and a feed-forward (``ffn`` wide, or
+    ``experts`` of ``expert_ffn`` each with ``experts_used`` per token; none when both are 0)."""
+    mixer: str                     # "attention" | "mingru" | "latent_attention"
     ffn: int = 0
+    experts: int = 0
+    experts_used: int = 0
+    expert_ffn: int = 0
     # attention without rotation, with its own value width, query temperature and output gate
     heads: int = 0
     kv_heads: int = 0
@@ -38,8 +42,18 @@ class LayerSpec:
     scale: float = 0.0
     q_temp_coef: float = 0.0       # queries at position p are multiplied by 1 + coef * ln(floor((p + 1) / every) + 1)
     q_temp_every: float = 1.0
+    # latent attention: key_dim above is the unrotated part of a head, kv_heads stays 0 (one latent row per token serves all heads)
+    kv_rank: int = 0
+    rot_dim: int = 0
+    window: int = 0                # keys a query sees, itself included (0 = all before it)
+    rope_theta: float = 10000.0
+    yarn: Optional[tuple] = None   # (factor, original context, fast turns, slow turns)
     # minGRU
     width: int = 0
+
+    def kv_width(self) -> int:
+        """Cached elements per token."""
+        return self.kv_heads * (self.key_dim + self.value_dim) + self.kv_rank + self.rot_dim
 
 
 @dataclass
@@ -86,6 +100,9 @@ class ModelConfig:
     # designs that list their layers (LAYER_LIST_ARCHS): head_dim / n_heads / n_kv_heads / ffn above are the largest of any layer
     layer_specs: list = field(default_factory=list)      # LayerSpec per layer
     norm_groups: int = 1                                  # RMS norms run over this many equal parts of the row
+    loop_start: int = 0                                   # layers loop_start .. loop_stop - 1 run loop_times times in a row (0: no loop); every
+    loop_stop: int = 0                                    # pass has its own cache and adds a learned vector to the residual first
+    loop_times: int = 0
     # Granite scalars
     embedding_scale: float = 1.0
     residual_scale: float = 1.0
@@ -108,10 +125,18 @@ class ModelConfig:
 
     def layer_is_full_attention(self, layer: int) -> bool:
         if self.layer_specs:
-            return self.layer_specs[layer].mixer == "attention"
+            return self.layer_specs[layer].mixer in ("attention", "latent_attention")
         if not self.is_hybrid:
             return True
         return (layer + 1) % self.full_attn_interval == 0
+
+    def layer_runs(self) -> list:
+        """(layer, number of the pass that begins with it or None) in the order of execution."""
+        if not self.loop_times:
+            return [(l, None) for l in range(self.n_layers)]
+        a, b = self.loop_start, self.loop_stop
+        return ([(l, None) for l in range(a)] + [(l, t if l == a else None) for t in range(self.loop_times) for l in range(a, b)]
+                + [(l, None) for l in range(b, self.n_layers)])
 
     def layer_window(self, layer: int) -> int:
         """Sliding window of a layer (0 = full).  gpt-oss windows the even layers (src/model/gptoss.cpp:133), Gemma-4 the
@@ -120,6 +145,8 @@ class ModelConfig:
             return self.sliding_window if layer % 2 == 0 else 0
         if self.arch == "gemma4":
             return self.sliding_window if self.layer_swa[layer] else 0
+        if self.layer_specs:
+            return self.layer_specs[layer].window
         return self.sliding_window
 
     def layer_geometry(self, layer: int) -> tuple:
@@ -285,13 +312,54 @@ def _tikarax_config(d: Mapping[str, Any]) -> ModelConfig:
     return _finish_layer_list(c)
 
 
+def _pubodra_config(d: Mapping[str, Any]) -> ModelConfig:
+    c = ModelConfig(arch="pubodra", hidden=int(d["width"]), vocab=int(d["vocab"]), rms_eps=float(d["norm"]["eps"]), tie_embeddings=True,
+                    name=str(d.get("name", "")))
+    for i, e in enumerate(d["layers"]):
+        m, mlp = e["mixer"], e.get("mlp")
+        if e["type"] != "latent_attention":
+            raise ConfigError(f"layer {i}: unknown mixer {e['type']!r}")
+        rot, mask = m["rot"], m.get("mask")
+        s = LayerSpec("latent_attention", heads=int(m["heads"]), key_dim=int(m["dim"]), value_dim=int(m["vdim"]), kv_rank=int(m["kv_rank"]),
+                      rot_dim=int(m["rot_dim"]), scale=float(m["scale"]), rope_theta=float(rot["base"]))
+        if min(s.heads, s.key_dim, s.value_dim, s.kv_rank, s.rot_dim) < 1 or s.rot_dim % 2 or int(rot["dims"]) != s.rot_dim:
+            raise ConfigError(f"layer {i}: sizes must be positive and rot.dims the even rot_dim")
+        if mask is not None:
+            s.window = int(mask["size"])
+            if s.window < 1:
+                raise ConfigError(f"layer {i}: mask.size must be positive")
+        if rot.get("scaling") is not None:
+            y = rot["scaling"]
+            s.yarn = (float(y["factor"]), float(y["original"]), float(y["fast"]), float(y["slow"]))
+            if min(s.yarn) <= 0:
+                raise ConfigError(f"layer {i}: rot.scaling values must be positive")
+        kind = None if mlp is None else mlp.get("kind", "dense")
+        if kind == "dense":
+            s.ffn = int(mlp["ff"])
+        elif kind == "moe":
+            s.experts, s.experts_used, s.expert_ffn = int(mlp["router"]["experts"]), int(mlp["router"]["top"]), int(mlp["expert"]["ff"])
+            if not 1 <= s.experts_used <= s.experts:
+                raise ConfigError(f"layer {i}: {s.experts_used} of {s.experts} experts per token")
+        elif kind is not None:
+            raise ConfigError(f"layer {i}: unknown feed-forward kind {kind!r}")
+        c.layer_specs.append(s)
+    if d.get("loop") is not None:
+        c.loop_start, c.loop_stop, c.loop_times = (int(d["loop"][k]) for k in ("start", "stop", "times"))
+        if not 0 <= c.loop_start < c.loop_stop <= len(c.layer_specs) or c.loop_times < 1:
+            raise ConfigError("loop: start .. stop must be a range of layers that runs at least once")
+    if c.hidden < 1 or c.vocab < 1 or not c.layer_specs:
+        raise ConfigError("the width must be positive, with at least one layer")
+    return _finish_layer_list(c)
+
+
 def _finish_layer_list(c: ModelConfig) -> ModelConfig:
     """Derived fields of a layer-list config: the largest sizes of any layer (pool sizing, reports)."""
     big = lambda f, lo=0: max([lo] + [getattr(s, f) for s in c.layer_specs])
     c.n_layers = len(c.layer_specs)
     c.n_heads, c.n_kv_heads, c.ffn = big("heads", 1), big("kv_heads", 1), big("ffn")
     c.head_dim = max(big("key_dim", 1), big("value_dim"))
-    c.n_rot, c.ctx_train = 0, 1 << 20                      # no rotation: positions have no trained limit of their own
+    c.n_experts, c.n_experts_used, c.expert_ffn = big("experts"), big("experts_used"), big("expert_ffn")
+    c.n_rot, c.ctx_train = 0, 1 << 20                      # rotations, where there are any, belong to the layers; positions have no limit of their own
     return c
 
 
@@ -303,7 +371,7 @@ def read_json_config(path_or_dict) -> ModelConfig:
         with open(p) as f:
             d = json.load(f)
     a = d.get("architecture")
-    readers = {"tikarax": _tikarax_config}
+    readers = {"tikarax": _tikarax_config, "pubodra": _pubodra_config}
     if a not in LAYER_LIST_ARCHS:
         raise ConfigError(f"unsupported architecture {a!r} in config.json (supported: {', '.join(LAYER_LIST_ARCHS)})")
     try:
@@ -314,16 +382,31 @@ def read_json_config(path_or_dict) -> ModelConfig:
 
 def config_to_json(c: ModelConfig) -> dict:
     """Inverse of :func:`read_json_config`."""
+    whole = lambda v: int(v) if float(v).is_integer() else v
     layers = []
     for s in c.layer_specs:
         if s.mixer == "attention":
             m = {"heads": s.heads, "kv_heads": s.kv_heads, "dim": s.key_dim, "vdim": s.value_dim, "scale": s.scale,
-                 "q_temp": {"coef": s.q_temp_coef, "every": int(s.q_temp_every) if float(s.q_temp_every).is_integer() else s.q_temp_every}}
+                 "q_temp": {"coef": s.q_temp_coef, "every": whole(s.q_temp_every)}}
+        elif s.mixer == "latent_attention":
+            rot = {"base": s.rope_theta, "dims": s.rot_dim}
+            if s.yarn is not None:
+                rot["scaling"] = dict(zip(("factor", "original", "fast", "slow"), (s.yarn[0], whole(s.yarn[1]), s.yarn[2], s.yarn[3])))
+            m = {"heads": s.heads, "dim": s.key_dim, "rot_dim": s.rot_dim, "vdim": s.value_dim, "kv_rank": s.kv_rank, "scale": s.scale, "rot": rot}
+            if s.window:
+                m["mask"] = {"size": s.window}
         else:
             m = {"width": s.width}
-        layers.append({"type": s.mixer, "mixer": m, "mlp": {"kind": "dense", "ff": s.ffn} if s.ffn else None})
+        mlp = {"kind": "dense", "ff": s.ffn} if s.ffn else None
+        if s.experts:
+            mlp = {"kind": "moe", "expert": {"ff": s.expert_ffn}, "router": {"experts": s.experts, "top": s.experts_used}}
+        layers.append({"type": s.mixer, "mixer": m, "mlp": mlp})
     arch = {v: k for k, v in LAYER_LIST_ARCHS.items()}[c.arch]
-    return {"architecture": arch, "layers": layers, "norm": {"eps": c.rms_eps, "groups": c.norm_groups}, "vocab": c.vocab, "width": c.hidden}
+    norm = {"eps": c.rms_eps, "groups": c.norm_groups} if c.arch == "tikarax" else {"eps": c.rms_eps}
+    out = {"architecture": arch, "layers": layers, "norm": norm, "vocab": c.vocab, "width": c.hidden}
+    if c.loop_times:
+        out["loop"] = {"start": c.loop_start, "stop": c.loop_stop, "times": c.loop_times}
+    return out
 
 
 def config_to_kv(c: ModelConfig) -> dict:
@@ -382,6 +465,23 @@ def _tikarax_preset(hidden, n_layers, heads, kv_heads, dim, vdim, ffn, width, vo
                                            q_temp_coef=0.1, q_temp_every=every))
         else:
             c.layer_specs.append(LayerSpec("mingru", ffn=ffn, width=width))
+    return _finish_layer_list(c)
+
+
+def _pubodra_preset(hidden, n_layers, heads, dim, rot_dim, vdim, kv_rank, window, ffn, vocab, experts=0, used=0, expert_ffn=0, moe_every=2, loop=None,
+                    theta=1e5, yarn=(8.0, 4096.0, 32.0, 1.0)) -> ModelConfig:
+    """Every ``moe_every``-th layer has experts (when there are any), the others a dense feed-forward."""
+    c = ModelConfig(arch="pubodra", hidden=hidden, vocab=vocab, rms_eps=1e-6, tie_embeddings=True)
+    for l in range(n_layers):
+        s = LayerSpec("latent_attention", heads=heads, key_dim=dim, rot_dim=rot_dim, value_dim=vdim, kv_rank=kv_rank, window=window,
+                      scale=(dim + rot_dim) ** -0.5, rope_theta=theta, yarn=yarn)
+        if experts and (l + 1) % moe_every == 0:
+            s.experts, s.experts_used, s.expert_ffn = experts, used, expert_ffn
+        else:
+            s.ffn = ffn
+        c.layer_specs.append(s)
+    if loop is not None:
+        c.loop_start, c.loop_stop, c.loop_times = loop
     return _finish_layer_list(c)
 
 
@@ -444,6 +544,10 @@ def preset(name: str) -> ModelConfig:
         # layers of common model sizes: 1 B class and 8 B class (un-gated feed-forward with the parameters of a gated one of 2/3 its width)
         "tikarax-1b": _tikarax_preset(2048, 16, 32, 8, 64, 64, 12288, 4096, 128256),
         "tikarax-8b": _tikarax_preset(4096, 32, 32, 8, 128, 128, 21504, 6144, 128256),
+        "tiny-pubodra": _pubodra_preset(160, 3, 5, 24, 8, 40, 48, 70, 224, 384, experts=6, used=2, expert_ffn=96, loop=(1, 3, 2), yarn=(4.0, 64.0, 32.0, 1.0)),
+        # layers of common model sizes: 1 B class and 8 B class, the latter with 64 small experts in every other layer
+        "pubodra-1b": _pubodra_preset(2048, 16, 16, 128, 64, 128, 512, 1024, 12288, 128256),
+        "pubodra-8b": _pubodra_preset(4096, 32, 32, 128, 64, 128, 512, 4096, 21504, 128256, experts=64, used=6, expert_ffn=1536),
         "tiny-qwen2": ModelConfig(arch="qwen2", n_layers=2, hidden=256, n_heads=4, n_kv_heads=2, head_dim=64, ffn=512, vocab=2048,
                                   rms_eps=1e-6, rope_theta=1e6, n_rot=64, ctx_train=4096),
         "tiny-phi3": ModelConfig(arch="phi3", n_layers=2, hidden=256, n_heads=4, n_kv_heads=4, head_dim=64, ffn=512, vocab=2048,

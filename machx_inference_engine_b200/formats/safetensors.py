@@ -134,7 +134,7 @@ def write_safetensors(path: str, tensors: dict, metadata: dict | None = None) ->
         dt = None
         if isinstance(a, tuple):
             dt, a = a
-        a = np.ascontiguousarray(a)
+        a = np.asarray(a, order="C")               # (ascontiguousarray would turn a scalar into a vector)
         dt = dt or rev[a.dtype]
         b = a.tobytes()
         header[name] = {"dtype": dt, "shape": list(a.shape), "data_offsets": [off, off + len(b)]}

@@ -291,8 +291,7 @@ def write_synthetic_gguf(cfg: ModelConfig, path: str, quant: str = "q8_0", seed:
     return {"tensors": n, "bytes": os.path.getsize(path)}
 
 
-def folder_tensor_plan(cfg: ModelConfig) -> list:
-    """(name, kind, shape) of every tensor of a layer-list checkpoint folder (``LAYER_LIST_ARCHS``); matrices are [out, in]."""
+def _tikarax_tensors(cfg: ModelConfig) -> list:
     H = cfg.hidden
     out = [("embed", "matrix", (cfg.vocab, H)), ("embed.norm", "norm", (H,)), ("final.norm", "norm", (H,)), ("head", "matrix", (cfg.vocab, H))]
     for i, s in enumerate(cfg.layer_specs):
@@ -312,6 +311,35 @@ def folder_tensor_plan(cfg: ModelConfig) -> list:
     return out
 
 
+def _pubodra_tensors(cfg: ModelConfig) -> list:
+    H = cfg.hidden
+    norm = lambda n: [(n, "norm", (H,)), (f"{n}.b", "vector", (H,)), (f"{n}.alpha", "alpha", ())]
+    out = [("embed", "matrix", (cfg.vocab, H))] + norm("final.norm")
+    if cfg.loop_times:
+        out.append(("loop.step", "vector", (cfg.loop_times, H)))
+    for i, s in enumerate(cfg.layer_specs):
+        p = f"l{i}"
+        out += norm(f"{p}.norm1")
+        out += [(f"{p}.mix.q", "matrix", (s.heads * (s.key_dim + s.rot_dim), H)), (f"{p}.mix.dkv", "matrix", (s.kv_rank + s.rot_dim, H)),
+                (f"{p}.mix.dkv.norm", "norm", (s.kv_rank,)), (f"{p}.mix.uk", "matrix", (s.heads * s.key_dim, s.kv_rank)),
+                (f"{p}.mix.uv", "matrix", (s.heads * s.value_dim, s.kv_rank)), (f"{p}.mix.g", "matrix", (s.heads * s.value_dim, H)),
+                (f"{p}.mix.o", "matrix", (H, s.heads * s.value_dim))]
+        if s.ffn or s.experts:
+            out += norm(f"{p}.norm2")
+        if s.ffn:
+            out += [(f"{p}.mlp.up", "matrix", (s.ffn, H)), (f"{p}.mlp.down", "matrix", (H, s.ffn))]
+        for e in range(s.experts):
+            out += [(f"{p}.mlp.e{e}.up", "matrix", (s.expert_ffn, H)), (f"{p}.mlp.e{e}.down", "matrix", (H, s.expert_ffn))]
+        if s.experts:
+            out.append((f"{p}.mlp.router", "matrix", (s.experts, H)))
+    return out
+
+
+def folder_tensor_plan(cfg: ModelConfig) -> list:
+    """(name, kind, shape) of every tensor of a layer-list checkpoint folder (``LAYER_LIST_ARCHS``); matrices are [out, in]."""
+    return {"tikarax": _tikarax_tensors, "pubodra": _pubodra_tensors}[cfg.arch](cfg)
+
+
 def write_synthetic_folder(cfg: ModelConfig, path: str, seed: int = 0) -> dict:
     """Random-init checkpoint folder (config.json + bf16 model.safetensors) of a layer-list design."""
     import json
@@ -324,9 +352,9 @@ def write_synthetic_folder(cfg: ModelConfig, path: str, seed: int = 0) -> dict:
     tensors = {}
     for name, kind, shape in folder_tensor_plan(cfg):
         g = np.random.default_rng([seed, zlib.crc32(name.encode())])
-        v = g.standard_normal(shape, dtype=np.float32)
-        v = {"matrix": lambda: v / np.sqrt(np.float32(shape[-1])), "norm": lambda: 1.0 + 0.1 * v, "vector": lambda: 0.1 * v}[kind]()
-        bits = np.ascontiguousarray(v, dtype=np.float32).view(np.uint32)
+        v = np.asarray(g.standard_normal(shape), dtype=np.float32) if shape == () else g.standard_normal(shape, dtype=np.float32)
+        v = {"alpha": lambda: 0.7 + 0.05 * v, "matrix": lambda: v / np.sqrt(np.float32(shape[-1])), "norm": lambda: 1.0 + 0.1 * v, "vector": lambda: 0.1 * v}[kind]()
+        bits = np.asarray(v, dtype=np.float32, order="C").view(np.uint32)
         tensors[name] = ("BF16", ((bits + 0x7FFF + ((bits >> 16) & 1)) >> 16).astype(np.uint16))
     write_safetensors(os.path.join(path, "model.safetensors"), tensors)
     return {"tensors": len(tensors), "bytes": os.path.getsize(os.path.join(path, "model.safetensors"))}

@@ -9,7 +9,8 @@ from ..formats.model_config import ModelConfig, read_config, read_json_config
 from ..parallel.comm import ParallelCtx
 
 # file names of the tensors that every graph asks for under its GGUF name
-_FOLDER_NAMES = {"tikarax": {"token_embd.weight": "embed", "output_norm.weight": "final.norm", "output.weight": "head"}}
+_FOLDER_NAMES = {"tikarax": {"token_embd.weight": "embed", "output_norm.weight": "final.norm", "output.weight": "head"},
+                 "pubodra": {"token_embd.weight": "embed", "output_norm.weight": "final.norm"}}
 
 
 def _graph_class(cfg: ModelConfig):
@@ -22,6 +23,9 @@ def _graph_class(cfg: ModelConfig):
     if cfg.arch == "tikarax":
         from .tikarax import TikaraxModel
         return TikaraxModel
+    if cfg.arch == "pubodra":
+        from .pubodra import PubodraModel
+        return PubodraModel
     from .transformer import TransformerModel
     return TransformerModel
 

@@ -81,8 +81,12 @@ class SafetensorsSource:
         return n
 
     def matrix(self, name: str, N: int, K: int, E: int = 1, experts: Optional[tuple[int, int]] = None) -> QuantWeight:
+        if "*" in name:                  # one tensor per expert, the number in the place of the star
+            lo, hi = experts if experts is not None else (0, E)
+            p0 = torch.cat([self.matrix(name.replace("*", str(e)), N, K).p0 for e in range(lo, hi)])
+            return QuantWeight(WFormat.BF16, N, K, hi - lo, p0.contiguous())
         if E != 1 or experts is not None:
-            raise ValueError("expert stacks are not read from safetensors folders")
+            raise ValueError(f"{name}: expert stacks are read from one tensor per expert")
         n = self._checked(name, (N, K))
         if self.m.dtype(n) == "BF16":
             t = torch.from_numpy(np.array(self.m.numpy(n), copy=True).view(np.int16)).view(torch.bfloat16)
@@ -94,7 +98,10 @@ class SafetensorsSource:
         return self.table(name, (n,))
 
     def table(self, name: str, shape: tuple[int, ...]) -> torch.Tensor:
-        return torch.from_numpy(np.array(self.m.float32(self._checked(name, shape)), copy=True)).to(self.device)
+        return torch.from_numpy(np.array(self.m.float32(self._checked(name, shape)), copy=True).reshape(shape)).to(self.device)
+
+    def scalar(self, name: str) -> float:
+        return float(self.table(name, ()))
 
 
 def default_policy(arch: str, quant: str) -> Callable[[str], WFormat]:
@@ -210,6 +217,9 @@ class SynthSource:
         if name.endswith("ssm_a"):
             return (-torch.exp(torch.randn(n, generator=g, device=self.gen_device) * 0.5)).to(self.device)
         return (0.02 * torch.randn(n, generator=g, device=self.gen_device)).to(self.device)
+
+    def scalar(self, name: str) -> float:
+        return 0.7 + 0.05 * float(torch.randn((), generator=self._gen(name), device=self.gen_device))
 
     def table(self, name: str, shape: tuple[int, ...]) -> torch.Tensor:
         g = self._gen(name)

@@ -28,47 +28,33 @@ import torch
 
 from .. import ops
 from ..formats.model_config import ModelConfig
-from ..ops import ACT_XIELU, QuantWeight
+from ..ops import ACT_XIELU
 from ..parallel.comm import ParallelCtx
 from ..utils.rope import query_temperature_table
 from .hybrid import MinGRUBlock, RecurrentState
-from .transformer import ForwardBatch, KVCache, NoRopeAttentionBlock, TransformerModel, UnaryFFN, round_up
+from .layer_list import LayerListModel
+from .transformer import ForwardBatch, KVCache, NoRopeAttentionBlock, UnaryFFN
 
 
 def _softplus(v: float) -> float:
     return max(v, 0.0) + math.log1p(math.exp(-abs(v)))
 
 
-class TikaraxModel(TransformerModel):
-    COMPUTE_DTYPES = ("bf16", "fp32")
-
+class TikaraxModel(LayerListModel):
     def __init__(self, cfg: ModelConfig, src, device, par: Optional[ParallelCtx] = None, max_ctx: int = 8192, dtype: str = "bf16"):
-        par = par or ParallelCtx()
-        if par.world > 1:
-            raise ValueError("the Tikarax graph runs on one GPU")
-        self.dtype = dtype
-        self.act_dtype = {"bf16": torch.bfloat16, "fp32": torch.float32}[dtype]
-        self.row = round_up(cfg.hidden, 32)              # columns of a residual / activation row
-        self._tables: dict = {}
-        super().__init__(cfg, src, device, par, max_ctx=max_ctx)
+        super().__init__(cfg, src, device, par, max_ctx=max_ctx, dtype=dtype)
         self.embed_norm = src.vector("embed.norm", cfg.hidden)
-        self.n_kv_local = max([L["attn"].n_kv for L in self.layers if "attn" in L], default=0)
-        self.kv_geometry = {l: (L["attn"].n_kv, L["attn"].dk, L["attn"].dv) for l, L in zip(self.layer_ids, self.layers) if "attn" in L}
 
     @property
     def needs_state(self) -> bool:
         return any("lin" in L for L in self.layers)
 
     # ---- construction
-    def _vocab_matrix(self, src, name: str) -> QuantWeight:
-        return super()._vocab_matrix(src, name).pad_groups(cols=(1, self.row))
+    def _kv_geometry(self) -> dict:
+        return {l: (L["attn"].n_kv, L["attn"].dk, L["attn"].dv) for l, L in zip(self.layer_ids, self.layers) if "attn" in L}
 
     def _q_scale(self, coef: float, every: float) -> Optional[torch.Tensor]:
-        if coef == 0.0:
-            return None
-        if (coef, every) not in self._tables:
-            self._tables[coef, every] = query_temperature_table(self.max_ctx, coef, every, device=self.device)
-        return self._tables[coef, every]
+        return None if coef == 0.0 else self._table((coef, every), lambda: query_temperature_table(self.max_ctx, coef, every, device=self.device))
 
     def _build_layer(self, l: int, src) -> dict:
         s, H, p = self.cfg.layer_specs[l], self.cfg.hidden, f"l{l}"
@@ -83,16 +69,6 @@ class TikaraxModel(TransformerModel):
             L.update(norm2=src.vector(f"{p}.norm2", H), norm2b=src.vector(f"{p}.norm2b", H),
                      ffn=UnaryFFN(src, f"{p}.mlp", H, self.row, s.ffn, ACT_XIELU, _softplus(a[0]), 0.5 + _softplus(a[1])))
         return L
-
-    def new_kv_cache(self, num_blocks: int, dtype: str = "bf16") -> KVCache:
-        if dtype == "int8":
-            raise ValueError("the int8 KV cache is not built for this design")
-        return KVCache(self.cfg.n_layers, num_blocks, self.n_kv_local, self.cfg.head_dim, self.device, self.attn_layers, dtype=self.dtype,
-                       geometry=self.kv_geometry)
-
-    def kv_bytes_per_block(self, dtype: str = "bf16") -> int:
-        per_tok = sum(n * (dk + dv) for n, dk, dv in self.kv_geometry.values())
-        return per_tok * KVCache.BLOCK * (2 if self.dtype == "bf16" else 4)
 
     def new_state(self, n_slots: int) -> RecurrentState:
         widths = {l: L["lin"].width for l, L in zip(self.layer_ids, self.layers) if "lin" in L}

@@ -49,6 +49,7 @@ class ForwardBatch:
     start_host: Optional[list] = None           # host copy of per-sequence start positions (0 = fresh state)
     want_hidden: bool = False                   # also return the pre-final-norm hidden rows (MTP)
     max_kv_len: int = 0                         # host copy of max(seq_lens); 0 = unknown (the block table's capacity is assumed)
+    short: Optional[tuple] = None               # (sequences, rows, longest query) of the leading short ones, when short and long queries meet in a batch
 
     @property
     def T(self) -> int:
@@ -58,11 +59,21 @@ class ForwardBatch:
     def B(self) -> int:
         return self.seq_lens.numel()
 
+    def query_parts(self) -> list:
+        """[(first row, end row, block table, sequence lengths, cu_q, longest query)]: the batch, or its short and its long queries (cu_q keeps
+        the rows of the whole batch)."""
+        if self.short is None:
+            return [(0, self.T, self.block_table, self.seq_lens, self.cu_q, self.max_q_len)]
+        n, rows, longest = self.short
+        return [(0, rows, self.block_table[:n], self.seq_lens[:n], self.cu_q[:n + 1], longest),
+                (rows, self.T, self.block_table[n:], self.seq_lens[n:], self.cu_q[n:], self.max_q_len)]
+
 
 class KVCache:
     """Paged KV: per attention layer ``k, v [num_blocks, n_kv_local, KV_BLOCK, head_dim]`` bf16 or fp32, or int8 with one fp32 scale
     per (block, kv head, token) row in ``ks, vs [num_blocks, n_kv_local, KV_BLOCK]`` (value = q * scale, scale = max|x| / 127).
-    ``geometry`` gives layers their own (n_kv, head_dim) or (n_kv, key width, value width).
+    ``geometry`` gives layers their own (n_kv, head_dim) or (n_kv, key width, value width); a value width of 0 is a latent cache, whose
+    values are formed from the key rows.  A layer that runs several times has one entry per run.
 
     The reference cache is contiguous per sequence (include/ie/kv_cache.hpp:27-114) and keeps int8 rows beside it when
     ``--int8-kv`` is given (src/core/kv_cache.cpp:182-240, src/ops/attention.cpp:145-229); pages make continuous batching
@@ -315,6 +326,74 @@ class NoRopeAttentionBlock:
         return self.o(a.reshape(T, self.n_q * self.dv))
 
 
+class LatentAttentionBlock:
+    """Attention over a cached latent: one row per token, [c | r], serves all heads.  A head's key is [W_uk c | r] with the rotated part r shared
+    by the heads, its value W_uv c; sliding window; sigmoid output gate that reads the block's own input.
+
+    One projection produces the columns [q: per head unrotated | rotated | c, r | gate].  Short queries (decoding, small portions) stay in the
+    latent space: q is taken through W_uk^T once, the kernel reads each cached row once for all heads and as key and value, and W_uv follows.
+    Long queries form the keys and values of the pages in reach once per step and run on the prefill kernel, which costs a head (dim + rot_dim +
+    vdim) products per key and query where the latent space costs 2 rank + rot_dim.  Widths are padded to multiples of 8 at load."""
+
+    EXPAND_MIN_Q = 64            # query segments at least this long take per-head keys and values
+    MAX_RANK = 512               # what the latent kernel's accumulators hold
+
+    def __init__(self, src, prefix: str, hidden: int, row: int, heads: int, dim: int, rot_dim: int, vdim: int, rank: int, scale: float, window: int,
+                 eps: float, rope: tuple):
+        if rank > self.MAX_RANK:
+            raise ValueError(f"{prefix}: a latent of {rank} elements is wider than the {self.MAX_RANK} the kernels take")
+        H, K = heads, hidden
+        self.n_q, self.n_kv, self.scale, self.window, self.eps, self.rank, self.rope = H, 1, scale, window, eps, rank, rope
+        self.d, self.r, self.v, self.R = (round_up(n, 8) for n in (dim, rot_dim, vdim, rank))
+
+        def padded(w: QuantWeight, parts, sizes, row_to):
+            """Rows of every group are ``parts`` runs; each run is padded to its size, the columns to ``row_to``."""
+            t = (w if w.fmt == WFormat.BF16 else QuantWeight(**_as_bf16(w))).p0[0]
+            t = t.reshape(-1, sum(parts), t.shape[-1])
+            out = torch.zeros(t.shape[0], sum(sizes), row_to, dtype=t.dtype, device=t.device)
+            lo = at = 0
+            for n, m in zip(parts, sizes):
+                out[:, at:at + n, :t.shape[2]] = t[:, lo:lo + n]
+                lo, at = lo + n, at + m
+            return out
+
+        stack = lambda t: QuantWeight(WFormat.BF16, t.shape[1], t.shape[2], t.shape[0], t.contiguous())
+        flat = lambda t: t.reshape(1, -1, t.shape[-1])
+        q = padded(src.matrix(f"{prefix}.q", H * (dim + rot_dim), K), (dim, rot_dim), (self.d, self.r), row)
+        ckv = padded(src.matrix(f"{prefix}.dkv", rank + rot_dim, K), (rank, rot_dim), (self.R, self.r), row)
+        g = padded(src.matrix(f"{prefix}.g", H * vdim, K), (vdim,), (self.v,), row)
+        self.proj = Linear(stack(torch.cat([flat(q), flat(ckv), flat(g)], dim=1)))
+        self.cols = (H * (self.d + self.r), H * (self.d + self.r) + self.R + self.r)
+        uk = padded(src.matrix(f"{prefix}.uk", H * dim, rank), (dim,), (self.d,), self.R)
+        uv = padded(src.matrix(f"{prefix}.uv", H * vdim, rank), (vdim,), (self.v,), self.R)
+        self.kv_up = stack(torch.cat([flat(uk), flat(uv)], dim=1))          # keys of all heads, then values
+        self.absorb = stack(uk.transpose(1, 2))                               # per head [R, d]
+        self.v_up = QuantWeight(WFormat.BF16, self.v, self.R, H, self.kv_up.p0[0, H * self.d:].view(H, self.v, self.R))
+        self.norm = torch.zeros(self.R, dtype=torch.float32, device=uk.device)
+        self.norm[:rank] = src.vector(f"{prefix}.dkv.norm", rank)
+        self.o = Linear(src.matrix(f"{prefix}.o", K, H * vdim).pad_groups(rows=(1, row), cols=(H, self.v)))
+
+    def __call__(self, h: torch.Tensor, fb: ForwardBatch, cache: torch.Tensor, plans: dict) -> torch.Tensor:
+        y = self.proj(h)
+        T, H, d, R = y.shape[0], self.n_q, self.d, self.R
+        q, ckv, gate = y[:, :self.cols[0]].view(T, H, d + self.r), y[:, self.cols[0]:self.cols[1]], y[:, self.cols[1]:]
+        a = torch.empty(T, H, self.v, dtype=y.dtype, device=y.device)
+        for lo, hi, table, lens, cu, longest in fb.query_parts():
+            latent = longest < self.EXPAND_MIN_Q or (y.is_cuda and y.dtype == torch.float32)
+            rows = slice(lo, hi)
+            qc = torch.empty(hi - lo, H, R + self.r, dtype=y.dtype, device=y.device) if latent else None
+            ops.latent_post(q[rows, :, d:], ckv[rows], self.norm, self.rank, self.eps, fb.positions[rows], self.rope[0], self.rope[1], fb.slot_map[rows],
+                            cache, qc[..., R:] if latent else q[rows, :, d:])
+            if latent:               # (the latent part of a batch starts at its first row)
+                ops.head_linear(q[rows, :, :d], self.absorb, out=qc[..., :R])
+                o = ops.latent_attention(qc, cache, table, lens, cu, longest, R, window=self.window, scale=self.scale)
+                ops.head_linear(o, self.v_up, gate=gate[rows], out=a[rows])
+            else:
+                ops.latent_attention_expanded(q, self.kv_up, cache, table, lens, cu, longest, d, self.v, R, window=self.window, scale=self.scale,
+                                              gate=gate, out=a, plans=plans)
+        return self.o(a.view(T, H * self.v))
+
+
 class UnaryFFN:
     """down(act(up h)): a feed-forward without a gate branch; the activation runs in the up projection's epilogue."""
 
@@ -477,6 +556,11 @@ class MoEFFN:
         self.shared = None          # optional always-on expert (hybrid families): its partial joins the sum before the reduction
         self._arange = {}
 
+    LAZY_COMBINE = False         # the graph's norm takes an expert combine that has not been formed (ops.cuda.CombineDelta)
+
+    def _lazy(self, h) -> bool:
+        return self.LAZY_COMBINE and h.is_cuda and ops.backend() != "torch" and self.shared is None and not self.reduce and self.K <= 32
+
     def _stage_banks(self) -> None:
         """Spilled layer: copy the banks from host memory into the shared staging area and point the layer at them."""
         sp, host = self._spill
@@ -534,7 +618,7 @@ class MoEFFN:
             y = ops.expert_gemv(q8(a), self.down, slot_e, x_div=1, bias=self.down_bias, e_lo=self.e_lo)
             pk = ops.ref.MoePacking(None, None, None, torch.arange(T * self.K, dtype=torch.int32, device=h.device), None, None, T * self.K, self.K)
             out = ops.moe_combine(y, pk, w)
-        elif T <= 8:
+        elif T <= 8 and h.dtype != torch.float32:
             # decode: one GEMV slot per (token, expert) pair, weights streamed once per pair; under expert
             # parallelism the slots of experts that live on other ranks contribute zero rows here
             slot_e = idx.reshape(-1)
@@ -547,6 +631,9 @@ class MoEFFN:
                 self._arange[key] = pk
             if fuse_push:
                 return par.fused.moe_combine_push(y, self._arange[key].pair_to_packed, w)
+            if self._lazy(h):
+                from ..ops.cuda import CombineDelta
+                return CombineDelta(y, self._arange[key].pair_to_packed, w)
             out = ops.moe_combine(y, self._arange[key], w)
         elif T <= self.group_gemv_max_tokens and T * self.K <= 8 * local:
             # expert-major GEMV over a compact packing: every local expert streams its weights once against all of its rows (token
@@ -566,12 +653,32 @@ class MoEFFN:
             y = ops.grouped_linear(a, self.down, te, pk.num_tiles, bias=self.down_bias)
             if fuse_push:
                 return par.fused.moe_combine_push(y, pk.pair_to_packed, w)
+            if self._lazy(h):
+                from ..ops.cuda import CombineDelta
+                return CombineDelta(y, pk.pair_to_packed, w)
             out = ops.moe_combine(y, pk, w)
         if self.shared is not None:
             out = self.shared.add_into(out, h)
         if self.reduce:
             out = par.fused.push(out) if (par.fused is not None and out.is_cuda) else par.all_reduce(out)
         return out
+
+
+class UnaryMoEFFN(MoEFFN):
+    """Experts down(act(up h)) without a gate branch and without biases, of which each token uses the best K by router score; the weights are
+    the softmax scores of the chosen ones, renormalised.  Routing, packing and execution are :class:`MoEFFN`'s; one GPU."""
+
+    LAZY_COMBINE = True
+
+    def __init__(self, src, prefix: str, hidden: int, row: int, experts: int, used: int, ffn: int, act: int):
+        f = round_up(ffn, 32)
+        self.E, self.K, self.e_lo, self.e_hi, self.expert_tp = experts, used, 0, experts, False
+        rw = src.matrix(f"{prefix}.router", experts, hidden)
+        self.router = Linear((rw if rw.fmt == WFormat.BF16 else QuantWeight(**_as_bf16(rw))).pad_groups(cols=(1, row)))
+        self.gate_up = src.matrix(f"{prefix}.e*.up", ffn, hidden, experts).pad_groups(rows=(1, f), cols=(1, row))
+        self.down = src.matrix(f"{prefix}.e*.down", hidden, ffn, experts).pad_groups(rows=(1, row), cols=(1, f))
+        self.router_bias = self.gu_bias = self.down_bias = self.expert_scale = self.shared = self.mx = self._spill = None
+        self.act, self.a8, self.reduce, self.group_gemv_max_tokens, self._arange = act, False, False, 0, {}
 
 
 def _mx_experts(self, h: torch.Tensor, idx: torch.Tensor, pre=None, ksplit: int = 1):

@@ -14,7 +14,7 @@ import torch
 
 from .weights import QuantWeight
 
-ACT_NONE, ACT_SWIGLU, ACT_SWIGLU_OAI, ACT_GEGLU, ACT_XIELU = 0, 1, 2, 3, 4
+ACT_NONE, ACT_SWIGLU, ACT_SWIGLU_OAI, ACT_GEGLU, ACT_XIELU, ACT_GELU_TANH, ACT_RELU2 = 0, 1, 2, 3, 4, 5, 6
 
 
 def act_gated(act: int) -> bool:
@@ -98,7 +98,12 @@ def rmsnorm(x, w, eps, delta=None, dbias=None, one_plus_w=False, delta_scale=1.0
 
 
 def act_unary(act, z, a, b):
-    """xIELU: a z^2 + z / 2 above zero, b (e^z - 1 - z) + z / 2 below (a = softplus(p), b = 1/2 + softplus(q))."""
+    """xIELU: a z^2 + z / 2 above zero, b (e^z - 1 - z) + z / 2 below (a = softplus(p), b = 1/2 + softplus(q)); GELU in its tanh form; the
+    square of ReLU."""
+    if act == ACT_GELU_TANH:
+        return torch.nn.functional.gelu(z, approximate="tanh")
+    if act == ACT_RELU2:
+        return z.clamp(min=0.0).square()
     if act != ACT_XIELU:
         return z
     neg = z.clamp(max=0.0)
@@ -113,6 +118,14 @@ def _act(act, g, u, alpha, limit):
         u = u.clamp(-limit, limit)
         return g * torch.sigmoid(alpha * g) * (u + 1.0)
     return torch.nn.functional.gelu(g, approximate="tanh") * u
+
+
+def _epilogue_act(y, act, alpha, limit):
+    """A projection's activation: gate and up columns combined, or element by element."""
+    if act_gated(act):
+        g, u = _deinterleave16(y)
+        return _act(act, g, u, alpha, limit)
+    return y if act == ACT_NONE else act_unary(act, y, alpha, limit)
 
 
 def _deinterleave16(y: torch.Tensor):
@@ -133,11 +146,7 @@ def linear(x, w: QuantWeight, bias=None, act=ACT_NONE, act_alpha=1.702, act_limi
     y = _mm(x, _dense(w)[0])
     if bias is not None:
         y = y + bias
-    if act_gated(act):
-        g, u = _deinterleave16(y)
-        y = _act(act, g, u, act_alpha, act_limit)
-    elif act != ACT_NONE:
-        y = act_unary(act, y, act_alpha, act_limit)
+    y = _epilogue_act(y, act, act_alpha, act_limit)
     if row_scale is not None:
         y = y * row_scale.unsqueeze(-1)
     return y if (out_f32 or x.dtype == torch.float32) else y.to(torch.bfloat16)      # fp32 activations: the layer runs in fp32 throughout
@@ -163,7 +172,7 @@ def grouped_linear(xp, w: QuantWeight, tile_expert, num_tiles, bias=None, act=AC
     """xp: packed rows [P,K]; tile t (rows 128t..128t+127) uses expert tile_expert[t] for t < num_tiles[0]."""
     W = _dense(w)
     P = xp.shape[0]
-    n_out = w.N // 2 if act != ACT_NONE else w.N
+    n_out = w.N // 2 if act_gated(act) else w.N
     out = torch.zeros(P, n_out, dtype=torch.float32, device=xp.device)
     nt = int(num_tiles[0])
     te = tile_expert[:nt].tolist()
@@ -172,11 +181,9 @@ def grouped_linear(xp, w: QuantWeight, tile_expert, num_tiles, bias=None, act=AC
         y = _mm(xp[rows], W[e])
         if bias is not None:
             y = y + bias[e]
-        if act != ACT_NONE:
-            g, u = _deinterleave16(y)
-            y = _act(act, g, u, act_alpha, act_limit)
+        y = _epilogue_act(y, act, act_alpha, act_limit)
         out[rows] = y
-    return out.to(out_dtype) if out_dtype is not None else (out if out_f32 else out.to(torch.bfloat16))
+    return out.to(out_dtype) if out_dtype is not None else (out if (out_f32 or xp.dtype == torch.float32) else out.to(torch.bfloat16))
 
 
 def expert_gemv(x, w: QuantWeight, slot_expert, x_div=1, bias=None, act=ACT_NONE, act_alpha=1.702, act_limit=7.0, slot_scale=None, out_f32=False,
@@ -192,13 +199,11 @@ def expert_gemv(x, w: QuantWeight, slot_expert, x_div=1, bias=None, act=ACT_NONE
     y = torch.einsum("sk,snk->sn", xe.to(_MM_DTYPE), W[se]).to(torch.float32)
     if bias is not None:
         y = y + bias[se]
-    if act != ACT_NONE:
-        g, u = _deinterleave16(y)
-        y = _act(act, g, u, act_alpha, act_limit)
+    y = _epilogue_act(y, act, act_alpha, act_limit)
     y = y * owned.unsqueeze(-1)
     if slot_scale is not None:
         y = y * slot_scale.unsqueeze(-1)
-    return y if out_f32 else y.to(torch.bfloat16)
+    return y if (out_f32 or x.dtype == torch.float32) else y.to(torch.bfloat16)
 
 
 def qkv_post(qkv, bias, q_norm_w, k_norm_w, positions, rope_cos, rope_sin, slot_map, k_cache, v_cache, n_q, n_kv, hd, n_rot,
@@ -273,6 +278,15 @@ def group_norm(x, w, eps, groups=1, delta=None, delta_w=None, fresh=False, width
     out = torch.zeros(x.shape, dtype=out_dtype, device=x.device)
     out[:, :H] = norm(x, w).to(out_dtype)
     return out
+
+
+def dyt_norm(x, alpha, w, b, delta=None, step=None, out_dtype=torch.bfloat16, want_out=True):
+    """x <- x + delta + step (fp32, in place; step is one vector for all rows); returns tanh(alpha x) w + b."""
+    if delta is not None:
+        x += delta.to(torch.float32)
+    if step is not None:
+        x += step
+    return (torch.tanh(alpha * x) * w + b).to(out_dtype) if want_out else None
 
 
 def kv_store(k, v, slot_map, k_cache, v_cache):
@@ -355,6 +369,70 @@ def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks
     if gate is not None:
         out = out * torch.sigmoid(gate.to(torch.float32)).reshape(Tq, n_q, dv)
     return out if q.dtype == torch.float32 else out.to(torch.bfloat16)
+
+
+# ------------------------------------------------------------------ latent attention
+def _rotate_pairs(t, cos, sin):
+    """Interleaved pairs (2i, 2i + 1) of the first 2 * cos.shape[-1] elements."""
+    n = 2 * cos.shape[-1]
+    u, v = t[..., 0:n:2], t[..., 1:n:2]
+    return torch.cat([torch.stack([u * cos - v * sin, v * cos + u * sin], dim=-1).flatten(-2), t[..., n:]], dim=-1)
+
+
+def latent_post(q_rot, ckv, norm_w, rank, eps, positions, rope_cos, rope_sin, slot_map, cache, q_out):
+    """Head epilogue of latent attention.  q_rot [T, H, r]: the rotated part of the queries -> rotated into q_out [T, H, r] (may be the same
+    memory).  ckv [T, R + r]: columns [0, rank) are RMS-normed (weight norm_w [R], zero past rank), columns R.. are the shared key part, rotated;
+    the row goes into the paged cache [blocks, 1, bs, R + r] (slots < 0 are skipped)."""
+    R, bs = norm_w.numel(), cache.shape[2]
+    pos = positions.long().clamp(0, rope_cos.shape[0] - 1)
+    c, s = rope_cos[pos], rope_sin[pos]
+    q_out.copy_(_rotate_pairs(q_rot.to(torch.float32), c.unsqueeze(1), s.unsqueeze(1)).to(q_out.dtype))
+    x = ckv.to(torch.float32)
+    lat = x[:, :R] * torch.rsqrt(x[:, :rank].pow(2).mean(-1, keepdim=True) + eps) * norm_w
+    row = torch.cat([lat, _rotate_pairs(x[:, R:], c, s)], dim=-1).to(cache.dtype)
+    ok = slot_map >= 0
+    cache[(slot_map[ok] // bs).long(), 0, (slot_map[ok] % bs).long()] = row[ok]
+
+
+def head_linear(x, w: QuantWeight, gate=None, out=None):
+    """Every head its own matrix: out[t, h] = W[h] x[t, h] (* sigmoid(gate[t, h])).  x [T, H, K] (any row / head stride), w stacks H matrices
+    [N, K]; gate [T, H * N]; out [T, H, N]."""
+    y = torch.einsum("thk,hnk->thn", x.to(_MM_DTYPE), _dense(w)).to(torch.float32)
+    if gate is not None:
+        y = y * torch.sigmoid(gate.to(torch.float32)).reshape(y.shape)
+    y = y.to(x.dtype)
+    return y if out is None else out.copy_(y)
+
+
+def latent_attention(q, cache, block_table, seq_lens, cu_q, max_q_len, rank, window=0, scale=1.0):
+    """Attention in the latent space: all heads share one cached row per token, whose first ``rank`` elements are also the value.
+    q [Tq, H, width of a cache row] -> [Tq, H, rank]."""
+    return attention(q, cache, cache[..., :rank], block_table, seq_lens, cu_q, max_q_len, window=window, scale=scale)
+
+
+def latent_attention_expanded(q, w_kv: QuantWeight, cache, block_table, seq_lens, cu_q, max_q_len, dim, vdim, rank, window=0, scale=1.0, gate=None,
+                              out=None, plans=None):
+    """Attention with per-head keys and values formed from the cached latents.  q [Tq, H, dim + r] (rotated), w_kv [H * dim + H * vdim, rank] (key
+    rows of all heads, then value rows) -> [Tq, H, vdim] (* sigmoid(gate)).  Only the rows that cu_q names are written."""
+    H, bs = q.shape[1], cache.shape[2]
+    out = torch.zeros(q.shape[0], H, vdim, dtype=q.dtype, device=q.device) if out is None else out
+    cu, W = cu_q.tolist(), _dense(w_kv)[0]
+    for b in range(len(cu) - 1):
+        q0, q1 = cu[b], cu[b + 1]
+        if q1 <= q0:
+            continue
+        L = int(seq_lens[b])
+        rows = cache[block_table[b, :(L + bs - 1) // bs].long(), 0].reshape(-1, cache.shape[3])[:L]
+        kv = _mm(rows[:, :rank], W).to(q.dtype).to(torch.float32)
+        K = torch.cat([kv[:, :H * dim].reshape(L, H, dim), rows[:, rank:].to(torch.float32).unsqueeze(1).expand(L, H, -1)], dim=-1)
+        s = torch.einsum("thd,khd->htk", q[q0:q1].to(torch.float32) * scale, K)
+        gap = torch.arange(L - (q1 - q0), L, device=q.device).unsqueeze(1) - torch.arange(L, device=q.device)
+        s = s.masked_fill((gap < 0) | ((gap >= window) if window > 0 else False), float("-inf"))
+        o = torch.einsum("htk,khd->thd", torch.softmax(s, dim=-1), kv[:, H * dim:].reshape(L, H, vdim))
+        if gate is not None:
+            o = o * torch.sigmoid(gate[q0:q1].to(torch.float32)).reshape(o.shape)
+        out[q0:q1] = o.to(q.dtype)
+    return out
 
 
 def sigmoid_mul(x, g):
@@ -594,7 +672,7 @@ def expert_group_gemv(x, w: QuantWeight, pk: MoePacking, x_index=None, bias=None
     """y[r] = W[expert of packed row r] @ x[x_index[r] or r] over a compact packing; bf16 [max_rows, N_out]."""
     W = _dense(w)
     P = pk.max_rows
-    n_out = w.N // 2 if act != ACT_NONE else w.N
+    n_out = w.N // 2 if act_gated(act) else w.N
     out = torch.zeros(P, n_out, dtype=torch.float32, device=x.device)
     xf = x.to(torch.float32)
     for el in range(w.E):
@@ -607,9 +685,7 @@ def expert_group_gemv(x, w: QuantWeight, pk: MoePacking, x_index=None, bias=None
         y = _mm(xin, W[el])
         if bias is not None:
             y = y + bias[el]
-        if act != ACT_NONE:
-            g, u = _deinterleave16(y)
-            y = _act(act, g, u, act_alpha, act_limit)
+        y = _epilogue_act(y, act, act_alpha, act_limit)
         out[rows] = y
     return out.to(torch.bfloat16)
 

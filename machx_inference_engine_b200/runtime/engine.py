@@ -389,14 +389,15 @@ class LLMEngine:
         for seq, toks, _ in entries:
             if not toks or len(seq.tokens) + len(toks) > self.opts.max_ctx:
                 raise ContextLengthExceeded(f"{len(seq.tokens)} + {len(toks)} tokens do not fit the context of {self.opts.max_ctx}")
-        plan = self.sched.admit([(seq, len(toks)) for seq, toks, _ in entries])
-        rows, base = [], 0
+        plan = self._short_first(self.sched.admit([(seq, len(toks)) for seq, toks, _ in entries]))
+        starts = itertools.accumulate([n for _, n in plan], initial=0)
+        base = {seq.seq_id: at for (seq, _), at in zip(plan, starts)}
+        rows = []
         for seq, toks, want in entries:
             if any(not 0 <= w < len(toks) for w in want):
                 raise ValueError("a wanted place lies outside its tokens")
             seq.tokens.extend(toks)
-            rows.extend(base + w for w in want)
-            base += len(toks)
+            rows.extend(base[seq.seq_id] + w for w in want)
         if self.state is not None:
             self._restore_states(plan)
         logits = self._logits(plan, rows)
@@ -406,10 +407,15 @@ class LLMEngine:
         self.stats["steps"] += 1
         return logits.clone() if rows else None           # (a graph's output buffer is written again by its next replay)
 
+    def _short_first(self, plan: list) -> list:
+        """Models that treat short and long queries differently (``split_query_len``) get the short ones of a batch first."""
+        split = getattr(self.model, "split_query_len", 0)
+        return sorted(plan, key=lambda e: e[1] >= split) if split else plan
+
     # ------------------------------------------------------------------ one step
     def step(self) -> list:
         """Runs one forward over the scheduled batch; returns [(seq, token, finished)] for sequences that produced a token."""
-        plan = self.sched.schedule()
+        plan = self._short_first(self.sched.schedule())
         if not plan:
             if self.sched.waiting and not self.sched.running:
                 raise OutOfBlocks("a waiting request cannot be scheduled: KV pool too small for its prompt")
@@ -564,6 +570,9 @@ class LLMEngine:
         fb = ForwardBatch(dev["ids"], dev["positions"], dev["slot_map"], dev["block_table"], dev["seq_lens"], dev["cu_q"], max_q,
                           logit_rows=dev["logit_rows"] if rows else dev["cu_q"][1:2].long() - 1)
         fb.max_kv_len = max(s.n_computed + n for s, n in plan)
+        few = [n for _, n in plan if n < getattr(self.model, "split_query_len", 0)]
+        if 0 < len(few) < len(plan):
+            fb.short = (len(few), sum(few), max(few))
         if self.state is not None:
             fb.state_slots_host = [s.state_slot for s, _ in plan]
             fb.state_slots = dev["state_slots"]

@@ -11,7 +11,7 @@ from typing import Optional
 import torch
 
 
-def _yarn_corr_dim(n_dims: int, n_ctx_orig: int, n_rot: float, base: float) -> float:
+def _yarn_corr_dim(n_dims: int, n_ctx_orig: float, n_rot: float, base: float) -> float:
     return n_dims * math.log(n_ctx_orig / (n_rot * 2 * math.pi)) / (2 * math.log(base))
 
 
@@ -23,7 +23,7 @@ def query_temperature_table(max_pos: int, coef: float, every: float, device="cpu
 
 
 def rope_tables(max_pos: int, n_rot: int, theta: float, freq_factors: Optional[torch.Tensor] = None, scaling_type: str = "none",
-                scaling_factor: float = 1.0, orig_ctx: int = 0, beta_fast: float = 32.0, beta_slow: float = 1.0,
+                scaling_factor: float = 1.0, orig_ctx: float = 0, beta_fast: float = 32.0, beta_slow: float = 1.0,
                 device="cpu") -> tuple[torch.Tensor, torch.Tensor]:
     """Returns fp32 (cos, sin), each [max_pos, n_rot/2]."""
     half = n_rot // 2
@@ -34,7 +34,7 @@ def rope_tables(max_pos: int, n_rot: int, theta: float, freq_factors: Optional[t
     pos = torch.arange(max_pos, dtype=torch.float64).unsqueeze(1)
     extrap = pos * inv.unsqueeze(0)
     mscale = 1.0
-    if scaling_type == "yarn" and scaling_factor > 1.0 and orig_ctx > 0:
+    if scaling_type == "yarn" and scaling_factor > 0.0 and orig_ctx > 0:
         freq_scale = 1.0 / scaling_factor
         lo = max(0.0, math.floor(_yarn_corr_dim(n_rot, orig_ctx, beta_fast, theta)))
         hi = min(n_rot - 1.0, math.ceil(_yarn_corr_dim(n_rot, orig_ctx, beta_slow, theta)))
