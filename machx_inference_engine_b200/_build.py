@@ -71,10 +71,11 @@ def build_host(force: bool = False) -> Path:
     return HOST_LIB
 
 
-# Kernel sources a dense / recurrent graph needs without experts, DeltaNet, EXL3 or sharded prefill.  A checkout without the full library
+# Kernel sources the layer-list graphs need: no DeltaNet, EXL3, MXFP4 or sharded prefill.  A checkout without the full library
 # can compile just these (``_lib.use_components("core")``); the full library, when it is there, serves every graph.
 COMPONENTS = {
-    "core": ("common", "comm", "elementwise", "gemm_tcgen05", "gemv", "gemv_stream", "linear_f32", "attention", "attention_tc", "mingru", "sampling"),
+    "core": ("common", "comm", "elementwise", "gemm_tcgen05", "gemv", "gemv_stream", "linear_f32", "attention", "attention_tc", "mingru", "latent",
+             "latent_tc", "moe", "sampling"),
 }
 
 

@@ -5,8 +5,9 @@
 
 namespace mx {
 
-// activation codes: 0 none; 1 SwiGLU, 2 clamped SwiGLU, 3 GeGLU (gated: N columns become N / 2); 4 xIELU (unary)
-constexpr int ACT_CODE_XIELU = 4;
+// activation codes: 0 none; 1 SwiGLU, 2 clamped SwiGLU, 3 GeGLU (gated: N columns become N / 2); 4 xIELU, 5 GELU (tanh form),
+// 6 the square of ReLU (unary)
+constexpr int ACT_CODE_XIELU = 4, ACT_CODE_GELU_TANH = 5, ACT_CODE_RELU2 = 6;
 __host__ __device__ constexpr bool act_gated(int act) { return act >= 1 && act <= 3; }
 
 // xIELU: a z^2 + z / 2 for z > 0, b (e^z - 1 - z) + z / 2 otherwise (a = softplus(p), b = 1/2 + softplus(q), formed by the caller).
@@ -18,11 +19,6 @@ __device__ __forceinline__ float xielu(float z, float a, float b) {
   return fmaf(0.5f, z, z > 0.f ? a * z * z : b * tail);
 }
 
-template <bool PRECISE>
-__device__ __forceinline__ float act_unary(int act, float z, float a, float b) {
-  return act == ACT_CODE_XIELU ? xielu<PRECISE>(z, a, b) : z;
-}
-
 // sigmoid with the full-precision exponential and division, or with the hardware's base-2 exponential and reciprocal (a few units in
 // the last place of fp32; the exponential overflows to infinity below about -88 and the result is 0)
 template <bool PRECISE>
@@ -32,6 +28,40 @@ __device__ __forceinline__ float sigmoid_f(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * -1.4426950408889634f));
   asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
   return r;
+}
+
+// GELU, tanh form: 0.5 z (1 + tanh u) = z sigmoid(2 u) with u = sqrt(2 / pi) (z + 0.044715 z^3)
+template <bool PRECISE>
+__device__ __forceinline__ float gelu_tanh(float z) {
+  const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+  if constexpr (PRECISE) return 0.5f * z * (1.f + tanhf(u));
+  return z * sigmoid_f<false>(2.f * u);
+}
+__device__ __forceinline__ float relu2(float z) {
+  const float m = fmaxf(z, 0.f);
+  return m * m;
+}
+
+template <bool PRECISE>
+__device__ __forceinline__ float act_unary(int act, float z, float a, float b) {
+  if (act == ACT_CODE_XIELU) return xielu<PRECISE>(z, a, b);
+  if (act == ACT_CODE_GELU_TANH) return gelu_tanh<PRECISE>(z);
+  return act == ACT_CODE_RELU2 ? relu2(z) : z;
+}
+
+// the same over a run of values: one branch for the run
+template <bool PRECISE, int N>
+__device__ __forceinline__ void act_unary_run(int act, float (&v)[N], float a, float b) {
+  if (act == ACT_CODE_XIELU) {
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] = xielu<PRECISE>(v[j], a, b);
+  } else if (act == ACT_CODE_GELU_TANH) {
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] = gelu_tanh<PRECISE>(v[j]);
+  } else if (act == ACT_CODE_RELU2) {
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] = relu2(v[j]);
+  }
 }
 
 // ---------------------------------------------------------------- element types of activations (bf16 or fp32)

@@ -15,6 +15,8 @@
 // 64 / 128 / 256 / 512 run on instances whose widths are compile-time constants; all other shapes, and caches in fp32, run on
 // instances that take the widths at run time and only round the value width up to 64 / 128 / 256 / 512 (accumulator registers).
 //
+// A latent cache has no value pages: the values are the first dv elements of the key rows (v_cache null), which are staged once.
+//
 // KV cache layout: [block][kv_head][block_size][head_dim] bf16 (or fp32), block_size a multiple of 64.  An int8 cache has the
 // same layout with one byte per element plus an fp32 scale per (block, kv head, token) row (value = q * scale); the
 // staging loop widens it to bf16, so the math below is shared.  kv_dequant_pages_kernel expands the pages of a prefill
@@ -110,10 +112,12 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
   constexpr int VE = 16 / sizeof(T);                                               // elements per 16-byte access
   const int DK = EXACT ? HD : p.dk, DV = EXACT ? HD : p.dv;
   const int KSTR = DK + att_kpad<T>();
+  const bool v_in_k = !EXACT && p.v_cache == nullptr;
+  const int VSTR = v_in_k ? KSTR : DV;
   extern __shared__ uint8_t smem_raw[];
   float* sq = reinterpret_cast<float*>(smem_raw);                                  // [PAIRS][DK]
   T* sv = reinterpret_cast<T*>(sq + PAIRS * DK);                                   // [64][DV]
-  T* sk = sv + ATT_TILE * DV;                                                      // [64][KSTR]
+  T* sk = v_in_k ? sv : sv + ATT_TILE * DV;                                        // [64][KSTR] (v_in_k: the values are its first columns)
   const T* kc = reinterpret_cast<const T*>(p.k_cache);
   const T* vc = reinterpret_cast<const T*>(p.v_cache);
 
@@ -203,7 +207,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
             uint32_t* kd = reinterpret_cast<uint32_t*>(sk + r * KSTR + c);
             kd[0] = kv4.x; kd[1] = kv4.y; kd[2] = kv4.z; kd[3] = kv4.w;
           }
-          for (int i = threadIdx.x; i < ATT_TILE * pv; i += blockDim.x)            // the tile's rows are one dense run
+          for (int i = threadIdx.x; i < (v_in_k ? 0 : ATT_TILE * pv); i += blockDim.x)            // the tile's rows are one dense run
             reinterpret_cast<uint4*>(sv)[i] = reinterpret_cast<const uint4*>(vp)[i];
         }
       }
@@ -263,7 +267,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
       // P V: a value element is read once per key and feeds all PPW pairs
 #pragma unroll 2
       for (int j = 0; j < ATT_TILE; ++j) {
-        const T* vr = sv + j * DV;
+        const T* vr = sv + j * VSTR;
         float vv[HD / 32];
 #pragma unroll
         for (int c = 0; c < HD / 32; ++c) vv[c] = (EXACT || lane + 32 * c < DV) ? to_f32(vr[lane + 32 * c]) : 0.f;
@@ -364,7 +368,8 @@ __global__ void __launch_bounds__(128) attn_combine_kernel(const float* __restri
     float a = 0.f;
     for (int s = 0; s < n_splits; ++s) {
       const size_t row = (size_t)s * Tq * n_q + r;
-      a += o_part[row * hd + d] * att_exp<PRECISE>(ml_part[row * 2] - M);
+      const float wt = att_exp<PRECISE>(ml_part[row * 2] - M);
+      if (wt != 0.f) a += o_part[row * hd + d] * wt;                   // (a split without keys leaves its rows unwritten)
     }
     a *= inv;
     if (gate) a *= sigmoid_f<PRECISE>(to_f32(gate[(size_t)(r / n_q) * gate_ld + (size_t)h * hd + d]));
@@ -382,7 +387,7 @@ template <typename T, int HD, int PPW, bool EXACT>
 static int launch_partial(const AttnParams& p, cudaStream_t st) {
   constexpr int PAIRS = ATT_WARPS * PPW;
   constexpr size_t SMEM_MAX = 226 * 1024;             // (the kernel also has a few static bytes)
-  const size_t smem = (size_t)PAIRS * p.dk * 4 + (size_t)ATT_TILE * (p.dk + att_kpad<T>()) * sizeof(T) + (size_t)ATT_TILE * p.dv * sizeof(T);
+  const size_t smem = (size_t)PAIRS * p.dk * 4 + (size_t)ATT_TILE * (p.dk + att_kpad<T>()) * sizeof(T) + (p.v_cache ? (size_t)ATT_TILE * p.dv * sizeof(T) : 0);
   if (smem > SMEM_MAX) return -112;
   auto kern = attn_partial_kernel<T, HD, PPW, EXACT>;
   static DeviceOnce configured;
@@ -462,8 +467,8 @@ static int attention_impl(const void* q, const void* k_cache, const void* v_cach
 #define MX_ATT(T_, HD_, EX_) \
   (ppw == 4 ? launch_partial<T_, HD_, 4, EX_>(p, st) : ppw == 2 ? launch_partial<T_, HD_, 2, EX_>(p, st) : launch_partial<T_, HD_, 1, EX_>(p, st))
   const int dk = sh.dk, dv = sh.dv, ve = sh.elem_f32 ? 4 : 8;
-  if (dk < 1 || dv < 1 || dk > 512 || dv > 512 || dk % ve || dv % ve) return -112;
-  if (!sh.elem_f32 && dk == dv && (dk == 64 || dk == 128 || dk == 256 || dk == 512)) {
+  if (dk < 1 || dv < 1 || dk > (v_cache ? 512 : 1024) || dv > 512 || dk % ve || dv % ve || (!v_cache && dv > dk)) return -112;
+  if (!sh.elem_f32 && v_cache && dk == dv && (dk == 64 || dk == 128 || dk == 256 || dk == 512)) {
     switch (dk) {
       case 64: rc = MX_ATT(__nv_bfloat16, 64, true); break;
       case 128: rc = MX_ATT(__nv_bfloat16, 128, true); break;
@@ -489,6 +494,16 @@ static int attention_impl(const void* q, const void* k_cache, const void* v_cach
   return (int)cudaGetLastError();
 }
 
+// Merge of split partials (o_part un-normalised, ml_part (maximum, denominator) per row): out bf16 [Tq][n_q][dv].
+MX_HOST_API int mx_attention_combine(const float* o_part, const float* ml_part, void* out, int Tq, int n_q, int dv, int n_splits, cudaStream_t st) {
+  if (Tq <= 0) return 0;
+  const float* no_sinks = nullptr;
+  const __nv_bfloat16* no_gate = nullptr;
+  launch_pdl(attn_combine_kernel<__nv_bfloat16>, dim3((Tq * n_q + 3) / 4), dim3(128), 0, st, o_part, ml_part, no_sinks, no_gate, 0, (__nv_bfloat16*)out, Tq, n_q, dv,
+             n_splits);
+  return (int)cudaGetLastError();
+}
+
 static AttnShape plain_shape(int n_q, int hd) {
   AttnShape sh;
   sh.dk = sh.dv = hd;
@@ -498,7 +513,8 @@ static AttnShape plain_shape(int n_q, int hd) {
 
 // Queries [Tq] rows of [n_q][dk] (q_ld elements apart), cache pages of dk- / dv-wide rows, out [Tq][n_q][dv]; optional gate (rows of
 // [n_q][dv], gate_ld apart; out *= sigmoid(gate)) and per-position score factors q_scale [q_scale_n].  elem_f32: everything in fp32.
-// o_part needs n_splits*Tq*n_q*dv floats.  Rows, widths and strides are multiples of 16 bytes.
+// o_part needs n_splits*Tq*n_q*dv floats.  Rows, widths and strides are multiples of 16 bytes.  v_cache null: a value is the first dv elements of
+// its key row.
 MX_HOST_API int mx_attention_ext(const void* q, int q_ld, const void* k_cache, const void* v_cache, const int* block_table, const int* seq_lens,
                                  const int* cu_q, const float* sinks, const void* gate, int gate_ld, const float* q_scale, int q_scale_n, void* out,
                                  float* o_part, float* ml_part, int B, int Tq, int max_q_len, int n_q, int n_kv, int dk, int dv, int max_blocks,

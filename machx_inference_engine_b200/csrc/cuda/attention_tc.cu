@@ -3,6 +3,10 @@
 // widths (multiples of 8 up to 256): the shared tiles are 64 / 128 / 256 columns wide and the tensor maps, whose rows end at the real
 // width, fill the rest with zeros, so the cache itself is not padded.
 //
+// Keys in two parts (ROT = 1; latent attention over expanded keys): the first DK - 64 columns of a head come from expanded pages [row][head][dim],
+// the last 64 from a part that all heads share, at its place in the latent cache; each part has its own tensor maps (and page table).  The values
+// are expanded pages too.
+//
 // One CTA owns 128 query tokens of one query head and walks the key tiles of its range (128 keys per tile, 64 for
 // head_dim 256 so that two K and two V tiles still fit in shared memory):
 //   warp 0  : TMA loads of the K and V tiles (two-stage rings) and, once, of the Q tile
@@ -29,6 +33,7 @@ constexpr int FA_PAGE = 128;   // KV page size
 
 struct FaParams {
   const int* block_table;  // [B][max_blocks]
+  const int* rot_table;    // ROT: [B][max_blocks] pages of the shared key part (block_table: the expanded pages)
   const int* seq_lens;     // [B]
   const int* cu_q;         // [B+1]
   const float* sinks;      // [n_q] or null
@@ -85,10 +90,11 @@ __device__ __forceinline__ float ex2_fast(float x) {
   return y;
 }
 
-template <int DK, int DV, bool CAP>
+template <int DK, int DV, bool CAP, int ROT>
 __global__ void __launch_bounds__(192, FaCfg<DK, DV>::CTAS)
 fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
-                  const __grid_constant__ CUtensorMap tmap_v, const FaParams p) {
+                  const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_qr,
+                  const __grid_constant__ CUtensorMap tmap_kr, const FaParams p) {
   using L = FaCfg<DK, DV>;
   constexpr int BKV = L::BKV, NS = L::NS, KS = L::KS, VS = L::VS;
   constexpr float LOG2E = 1.4426950408889634f;
@@ -141,18 +147,22 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       mbar_expect_tx(b_qfull, L::Q_BYTES);
 #pragma unroll
       for (int a = 0; a < L::KATOMS; ++a)
-        tma_load_3d(sbase + L::Q_OFF + a * (FA_BQ * 128), &tmap_q, b_qfull, a * 64, head, q_begin + t0);
+        if (a < L::KATOMS - ROT) tma_load_3d(sbase + L::Q_OFF + a * (FA_BQ * 128), &tmap_q, b_qfull, a * 64, head, q_begin + t0);
+        else tma_load_3d(sbase + L::Q_OFF + a * (FA_BQ * 128), &tmap_qr, b_qfull, 0, head, q_begin + t0);
       bool ok = true;
       for (int j = 0; j < n_tiles && ok; ++j) {
         const uint32_t sk = j % KS, phk = (j / KS) & 1, sv = j % VS, phv = (j / VS) & 1;
         const int key0 = (tile_lo + j) * BKV;
         const int blk = p.block_table[(size_t)b * p.max_blocks + key0 / FA_PAGE];
         const int krow = key0 % FA_PAGE;
+        int rblk = 0;
+        if constexpr (ROT != 0) rblk = p.rot_table[(size_t)b * p.max_blocks + key0 / FA_PAGE];
         if (!(ok = mbar_wait(b_kempty + 8 * sk, phk ^ 1, p.status, ERR_MBAR_TIMEOUT_PRODUCER, abort_flag))) break;
         mbar_expect_tx(b_kfull + 8 * sk, L::K_BYTES);
 #pragma unroll
         for (int a = 0; a < L::KATOMS; ++a)
-          tma_load_4d(sbase + L::K_OFF + sk * L::K_BYTES + a * (BKV * 128), &tmap_k, b_kfull + 8 * sk, a * 64, krow, kvh, blk);
+          if (a < L::KATOMS - ROT) tma_load_4d(sbase + L::K_OFF + sk * L::K_BYTES + a * (BKV * 128), &tmap_k, b_kfull + 8 * sk, a * 64, krow, kvh, blk);
+          else tma_load_3d(sbase + L::K_OFF + sk * L::K_BYTES + a * (BKV * 128), &tmap_kr, b_kfull + 8 * sk, 0, krow, rblk);
         if (!(ok = mbar_wait(b_vempty + 8 * sv, phv ^ 1, p.status, ERR_MBAR_TIMEOUT_PRODUCER, abort_flag))) break;
         mbar_expect_tx(b_vfull + 8 * sv, L::V_BYTES);
 #pragma unroll
@@ -382,7 +392,7 @@ static int launch_fa(const void* q, const void* k_cache, const void* v_cache, co
     r = page_map(&tv, v_cache, (uint64_t)p.dv);
     if (r) return r;
   }
-  auto kern = fa_prefill_kernel<DK, DV, CAP>;
+  auto kern = fa_prefill_kernel<DK, DV, CAP, 0>;
   static DeviceOnce configured;
   if (configured.pending()) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
@@ -390,7 +400,47 @@ static int launch_fa(const void* q, const void* k_cache, const void* v_cache, co
     configured.mark();
   }
   dim3 grid(B * p.max_q_tiles, p.n_q);
-  kern<<<grid, 192, L::TOTAL, st>>>(tq, tk, tv, p);
+  kern<<<grid, 192, L::TOTAL, st>>>(tq, tk, tv, tq, tk, p);
+  return (int)cudaGetLastError();
+}
+
+// Keys in two parts: `kv` holds expanded pages of 128 rows [n_q][dim] | [n_q][vdim] (kv_ld elements per row), `cache` the latent pages with the shared
+// key part (rot elements from column `rank`, rows cache_ld elements apart).  Queries: rows of [n_q][dim | rot].
+struct FaSplit { const void* kv; const void* cache; int dim, rot, rank, kv_ld, cache_ld, n_pages; };
+template <int DK, int DV>
+static int launch_fa_split(const void* q, const FaSplit& x, const FaParams& p, int B, int Tq, int n_blocks, cudaStream_t st) {
+  using L = FaCfg<DK, DV>;
+  using bf = __nv_bfloat16;
+  CUtensorMap tq, tqr, tk, tkr, tv;
+  int r = 0;
+  auto q_map = [&](CUtensorMap* m, const void* base, int width) {
+    uint64_t dims[3] = {(uint64_t)width, (uint64_t)p.n_q, (uint64_t)Tq};
+    uint64_t strides[2] = {(uint64_t)(x.dim + x.rot) * 2, (uint64_t)p.q_ld * 2};
+    uint32_t box[3] = {64, 1, FA_BQ};
+    return make_tmap_bf16(m, base, 3, dims, strides, box, 1);
+  };
+  auto page_map = [&](CUtensorMap* m, const void* base, int width) {
+    uint64_t dims[4] = {(uint64_t)width, (uint64_t)FA_PAGE, (uint64_t)p.n_q, (uint64_t)x.n_pages};
+    uint64_t strides[3] = {(uint64_t)x.kv_ld * 2, (uint64_t)width * 2, (uint64_t)x.kv_ld * 2 * FA_PAGE};
+    uint32_t box[4] = {64, (uint32_t)L::BKV, 1, 1};
+    return make_tmap_bf16(m, base, 4, dims, strides, box, 1);
+  };
+  if ((r = q_map(&tq, q, x.dim)) || (r = q_map(&tqr, (const bf*)q + x.dim, x.rot))) return r;
+  if ((r = page_map(&tk, x.kv, x.dim)) || (r = page_map(&tv, (const bf*)x.kv + (size_t)p.n_q * x.dim, p.dv))) return r;
+  {
+    uint64_t dims[3] = {(uint64_t)x.rot, (uint64_t)FA_PAGE, (uint64_t)n_blocks};
+    uint64_t strides[2] = {(uint64_t)x.cache_ld * 2, (uint64_t)x.cache_ld * 2 * FA_PAGE};
+    uint32_t box[3] = {64, (uint32_t)L::BKV, 1};
+    if ((r = make_tmap_bf16(&tkr, (const bf*)x.cache + x.rank, 3, dims, strides, box, 1))) return r;
+  }
+  auto kern = fa_prefill_kernel<DK, DV, false, 1>;
+  static DeviceOnce configured;
+  if (configured.pending()) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
+    if (e != cudaSuccess) return (int)e;
+    configured.mark();
+  }
+  kern<<<dim3(B * p.max_q_tiles, p.n_q), 192, L::TOTAL, st>>>(tq, tk, tv, tqr, tkr, p);
   return (int)cudaGetLastError();
 }
 
@@ -434,7 +484,7 @@ MX_HOST_API int mx_attention_prefill_tc_ext(const void* q, int q_ld, const void*
   if (block_size != FA_PAGE) return -110;
   if (n_q % n_kv) return -111;
   FaParams p;
-  p.block_table = block_table; p.seq_lens = seq_lens; p.cu_q = cu_q; p.sinks = sinks; p.out = (__nv_bfloat16*)out;
+  p.block_table = block_table; p.rot_table = nullptr; p.seq_lens = seq_lens; p.cu_q = cu_q; p.sinks = sinks; p.out = (__nv_bfloat16*)out;
   p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate ? gate_ld : 0; p.q_scale = q_scale; p.q_scale_n = q_scale_n;
   p.dk = dk; p.dv = dv; p.q_ld = q_ld;
   p.n_q = n_q; p.n_kv = n_kv; p.max_blocks = max_blocks; p.window = window; p.scale = scale; p.softcap = softcap;
@@ -451,4 +501,37 @@ MX_HOST_API int mx_attention_prefill_tc(const void* q, const void* k_cache, cons
   if (hd != 64 && hd != 128 && hd != 256) return -112;
   return mx_attention_prefill_tc_ext(q, n_q * hd, k_cache, v_cache, block_table, seq_lens, cu_q, sinks, nullptr, 0, nullptr, 0, out, B, Tq, max_q_len,
                                      n_q, n_kv, hd, hd, max_blocks, n_blocks, block_size, window, scale, softcap, st);
+}
+
+// Latent attention over expanded pages (see FaSplit).  q: [Tq] rows of [n_q][dim | rot], q_ld elements apart, rotated; kv: [n_pages * 128][n_q * (dim +
+// vdim)], its pages listed by kv_table; cache: [n_blocks][128][rank + rot], its pages listed by block_table (both tables [B][max_blocks]); gate (rows of
+// [n_q][vdim], gate_ld apart; out *= sigmoid(gate)); out [Tq][n_q][vdim].  Widths are multiples of 8: dim up to 192, rot up to 64, vdim up to 256.
+MX_HOST_API int mx_attention_prefill_latent(const void* q, int q_ld, const void* kv, int n_pages, const int* kv_table, const void* cache, int n_blocks,
+                                            const int* block_table, int max_blocks, const int* seq_lens, const int* cu_q, const void* gate, int gate_ld,
+                                            void* out, int B, int Tq, int max_q_len, int n_q, int dim, int rot, int vdim, int rank, int window, float scale,
+                                            cudaStream_t st) {
+  if (B <= 0 || Tq <= 0) return 0;
+  if (dim < 8 || dim > 192 || rot < 8 || rot > 64 || vdim < 8 || vdim > 256 || dim % 8 || rot % 8 || vdim % 8 || rank % 8 || q_ld % 8 || gate_ld % 8) return -112;
+  if (((uintptr_t)q | (uintptr_t)kv | (uintptr_t)cache | (uintptr_t)gate | (uintptr_t)out) & 15) return -112;
+  FaParams p;
+  p.block_table = kv_table; p.rot_table = block_table; p.seq_lens = seq_lens; p.cu_q = cu_q; p.sinks = nullptr; p.out = (__nv_bfloat16*)out;
+  p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate ? gate_ld : 0; p.q_scale = nullptr; p.q_scale_n = 0;
+  p.dk = dim + rot; p.dv = vdim; p.q_ld = q_ld; p.n_q = n_q; p.n_kv = n_q; p.max_blocks = max_blocks; p.window = window; p.scale = scale; p.softcap = 0.f;
+  p.max_q_tiles = (max_q_len + FA_BQ - 1) / FA_BQ;
+  p.status = status_word();
+  FaSplit x{kv, cache, dim, rot, rank, n_q * (dim + vdim), rank + rot, n_pages};
+#define MX_FAS(DK_, DV_) launch_fa_split<DK_, DV_>(q, x, p, B, Tq, n_blocks, st)
+  const int a = dim <= 64 ? 0 : dim <= 128 ? 1 : 2, b = vdim <= 64 ? 0 : vdim <= 128 ? 1 : 2;
+  switch (a * 3 + b) {
+    case 0: return MX_FAS(128, 64);
+    case 1: return MX_FAS(128, 128);
+    case 2: return MX_FAS(128, 256);
+    case 3: return MX_FAS(192, 64);
+    case 4: return MX_FAS(192, 128);
+    case 5: return MX_FAS(192, 256);
+    case 6: return MX_FAS(256, 64);
+    case 7: return MX_FAS(256, 128);
+    default: return MX_FAS(256, 256);
+  }
+#undef MX_FAS
 }

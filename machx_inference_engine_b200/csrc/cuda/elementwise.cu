@@ -6,6 +6,7 @@
 //   glu             : SwiGLU / clamped OAI SwiGLU / GeGLU over 16-column interleaved gate|up
 //   group_norm      : RMSNorm over equal groups of a row; one pass norms a branch output, adds it to the residual and norms the
 //                     sum for the next branch (norms on both sides of a sublayer)
+//   dyt_norm        : residual add (branch output or expert combine, plus a vector of the row) + tanh(alpha x) w + b, one pass
 //   kv_store        : K / V columns of a projection (own widths, no rotation) into the paged cache
 //   gated_rmsnorm   : y = w * x / rms(x) * silu(z) per head (DeltaNet output norm)
 //   misc            : sigmoid gate multiply, scaled add, casts
@@ -307,6 +308,69 @@ __global__ void __launch_bounds__(GN_WARPS * 32) group_norm_kernel(const GroupNo
       if (p.out) orow[i] = from_f32<OT>(0.f);
       if (p.fresh) xr[i] = 0.f;
     }
+}
+
+// ------------------------------------------------------------------ dyt_norm
+// A norm without statistics: every element on its own, so a thread needs no other thread.
+//   x (fp32 residual) += delta + step;   out = tanh(alpha x) w + b
+// delta: rows of DT (KIND 1), the weighted sum of expert outputs (KIND 2: rows pair_to_packed[t * K + k] of delta times cw[t * K + k]), or
+// none (KIND 0).  Four columns per thread; ld is a multiple of 4; padded columns are zero in w, b, delta and step and stay zero.
+struct DytParams {
+  float* x;
+  const void* delta;
+  const int* pair_to_packed;
+  const float* cw;
+  const float* step;          // [ld] or null
+  const float* w;
+  const float* b;
+  void* out;
+  float alpha;
+  int K, ld4;                 // ld4 = ld / 4
+  long long n4;               // rows * ld4
+};
+
+template <int KIND, typename DT, typename OT>
+__global__ void __launch_bounds__(256) dyt_norm_kernel(const DytParams p) {
+  pdl_prologue();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= p.n4) return;
+  const long long t = i / p.ld4;
+  const int c = (int)(i - t * p.ld4) * 4;
+  float x[4];
+  loadv<4>(p.x + i * 4, x);
+  if constexpr (KIND == 1) {
+    float d[4];
+    loadv<4>(reinterpret_cast<const DT*>(p.delta) + i * 4, d);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[e] += d[e];
+  } else if constexpr (KIND == 2) {
+    float a[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int k = 0; k < p.K; ++k) {
+      const int pos = p.pair_to_packed[t * p.K + k];
+      if (pos < 0) continue;
+      const float cw = p.cw[t * p.K + k];
+      float d[4];
+      loadv<4>(reinterpret_cast<const DT*>(p.delta) + (size_t)pos * (p.ld4 * 4) + c, d);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) a[e] = fmaf(cw, d[e], a[e]);
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[e] += a[e];
+  }
+  if (p.step) {
+    float s[4];
+    loadv<4>(p.step + c, s);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[e] += s[e];
+  }
+  if (KIND != 0 || p.step) storev<4>(p.x + i * 4, x);
+  if (!p.out) return;
+  float w[4], b[4];
+  loadv<4>(p.w + c, w);
+  loadv<4>(p.b + c, b);
+#pragma unroll
+  for (int e = 0; e < 4; ++e) w[e] = fmaf(tanhf(p.alpha * x[e]), w[e], b[e]);
+  storev<4>(reinterpret_cast<OT*>(p.out) + i * 4, w);
 }
 
 // ------------------------------------------------------------------ kv_store
@@ -698,6 +762,27 @@ MX_HOST_API int mx_group_norm(float* x, const void* delta, int delta_is_f32, con
   p.T = T; p.fresh = fresh;
   if (delta_is_f32) return out_is_f32 ? launch_group_norm<float, float>(p, st) : launch_group_norm<float, __nv_bfloat16>(p, st);
   return out_is_f32 ? launch_group_norm<__nv_bfloat16, float>(p, st) : launch_group_norm<__nv_bfloat16, __nv_bfloat16>(p, st);
+}
+
+// See dyt_norm_kernel.  x [T][ld] fp32; delta (null: none) [T][ld], or with pair_to_packed [rows][ld] combined with cw [T][K]; step, w, b [ld];
+// out (null: skipped) [T][ld].
+MX_HOST_API int mx_dyt_norm(float* x, const void* delta, int delta_is_f32, const int* pair_to_packed, const float* cw, int K, const float* step,
+                            float alpha, const float* w, const float* b, void* out, int out_is_f32, int T, int ld, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (ld < 4 || ld % 4 || (pair_to_packed && (!delta || K < 1))) return -107;
+  if (out && (!w || !b)) return -109;
+  DytParams p;
+  p.x = x; p.delta = delta; p.pair_to_packed = pair_to_packed; p.cw = cw; p.step = step; p.w = w; p.b = b; p.out = out; p.alpha = alpha; p.K = K;
+  p.ld4 = ld / 4; p.n4 = (long long)T * p.ld4;
+  const dim3 grid((unsigned)((p.n4 + 255) / 256)), block(256);
+  using bf = __nv_bfloat16;
+#define MX_DYT(KIND_, DT_) \
+  (out_is_f32 ? launch_pdl(dyt_norm_kernel<KIND_, DT_, float>, grid, block, 0, st, p) : launch_pdl(dyt_norm_kernel<KIND_, DT_, bf>, grid, block, 0, st, p))
+  if (!delta) MX_DYT(0, float);
+  else if (pair_to_packed) { if (delta_is_f32) MX_DYT(2, float); else MX_DYT(2, bf); }
+  else { if (delta_is_f32) MX_DYT(1, float); else MX_DYT(1, bf); }
+#undef MX_DYT
+  return (int)cudaGetLastError();
 }
 
 // k / v: rows of n_kv * dk / n_kv * dv elements, k_ld / v_ld elements apart; elem_bytes 2 or 4; every row, head and stride a multiple of 16 bytes.

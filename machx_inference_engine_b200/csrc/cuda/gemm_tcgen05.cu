@@ -28,7 +28,7 @@ constexpr int BK = 64;
 constexpr int kNumEpilogueWarps = 4;
 constexpr int kNumDequantWarps = 8;
 
-enum Act : int { ACT_NONE = 0, ACT_SWIGLU = 1, ACT_SWIGLU_OAI = 2, ACT_GEGLU = 3, ACT_XIELU = ACT_CODE_XIELU };
+enum Act : int { ACT_NONE = 0, ACT_SWIGLU = 1, ACT_SWIGLU_OAI = 2, ACT_GEGLU = 3 };      // unary codes: act.cuh
 
 struct GemmParams {
   int M, N, K;
@@ -52,6 +52,13 @@ struct GemmParams {
   const int* a_flags;           // [world] flags of the gather buffer (this rank's copy), null = plain A
   const int* a_seq;             // device word: the sequence number the flags have to reach
   int a_rows_per_src, a_world, m_rot;
+  // per-head products: batch_tiles > 0 m-tiles per head, head h uses weight slab h, activations a 3-D tensor (K, rows, heads), output at
+  // h * c_batch; gate (non-null): the output is multiplied by sigmoid(gate[row * gate_ld + h * N + n])
+  int batch_tiles;
+  long long c_batch;
+  const __nv_bfloat16* gate;
+  int gate_ld;
+  const int* a_pages;           // paged activations: m-tile i reads page a_pages[i] (BM rows each), null = row i * BM
 };
 
 constexpr int kRawDepth = 10;   // k-iterations of packed weight bytes kept in flight per producer thread
@@ -175,7 +182,8 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
       for (int t = blockIdx.x; t < total_tiles && ok; t += gridDim.x) {
         int mt, nt;
         tile_coords(t, m_tiles, p.num_n_tiles, p.group_m, mt, nt, p.m_rot);
-        const int e = p.tile_expert ? p.tile_expert[mt] : 0;
+        const int e = p.batch_tiles ? mt / p.batch_tiles : (p.tile_expert ? p.tile_expert[mt] : 0);
+        const int a_row = (p.batch_tiles ? mt - e * p.batch_tiles : (p.a_pages ? p.a_pages[mt] : mt)) * BM;
         if (p.a_flags) {
           // the rows of this m-tile come from one owner rank: wait (bounded) until that rank's stores have been published
           const int src = min((mt * BM) / p.a_rows_per_src, p.a_world - 1);
@@ -199,7 +207,8 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
             // a k-block past the end of K is fetched all the same: the out-of-range box arrives as zeros
             const int k = kl * KS + j;
             const uint32_t ps = s * KS + j;
-            tma_load_2d(smem_base + L::A_OFFSET + ps * L::A_BYTES, &tmap_a, bar_full + 8 * s, k * BK, mt * BM);
+            if (p.batch_tiles) tma_load_3d(smem_base + L::A_OFFSET + ps * L::A_BYTES, &tmap_a, bar_full + 8 * s, k * BK, a_row, e);
+            else tma_load_2d(smem_base + L::A_OFFSET + ps * L::A_BYTES, &tmap_a, bar_full + 8 * s, k * BK, a_row);
             if (!kDequant) tma_load_3d(smem_base + L::B_OFFSET + ps * L::B_BYTES, &tmap_b, bar_full + 8 * s, k * BK, nt * BN, e);
           }
         }
@@ -244,11 +253,12 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
     for (int t = blockIdx.x; t < total_tiles && ok; t += gridDim.x, ++tile_n) {
       int mt, nt;
       tile_coords(t, m_tiles, p.num_n_tiles, p.group_m, mt, nt, p.m_rot);
-      const int e = p.tile_expert ? p.tile_expert[mt] : 0;
+      const int e = p.batch_tiles ? mt / p.batch_tiles : (p.tile_expert ? p.tile_expert[mt] : 0);
       const uint32_t acc = tile_n & 1, acc_ph = (tile_n >> 1) & 1;
       if (!(ok = mbar_wait(bar_tfull + 8 * acc, acc_ph, p.status, ERR_MBAR_TIMEOUT_EPILOGUE, abort_flag))) break;
       tc_fence_after();
-      const int row = mt * BM + q * 32 + lane;
+      const int row = (p.batch_tiles ? mt - e * p.batch_tiles : mt) * BM + q * 32 + lane;
+      const size_t c_off = p.batch_tiles ? (size_t)e * p.c_batch : 0;
       const bool row_ok = row < p.M;
       const float rs = (p.row_scale && row_ok) ? p.row_scale[row] : 1.f;
       const float* bias = p.bias ? p.bias + (size_t)e * p.N : nullptr;
@@ -321,9 +331,20 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
           if (bias && col0 + j < p.N) v[j] += bias[col0 + j];
         }
         if (!act_gated(p.act)) {
-          if (p.act != ACT_NONE) {
+          if (p.act != ACT_NONE) act_unary_run<false>(p.act, v, p.act_alpha, p.act_limit);
+          if (p.gate) {
+            const __nv_bfloat16* g = p.gate + (size_t)row * p.gate_ld + (size_t)e * p.N + col0;
 #pragma unroll
-            for (int j = 0; j < 32; ++j) v[j] = act_unary<false>(p.act, v[j], p.act_alpha, p.act_limit);
+            for (int j = 0; j < 32; j += 8) {
+              if (col0 + j >= p.N) break;                          // (N is a multiple of 8)
+              const uint4 g4 = __ldg(reinterpret_cast<const uint4*>(g + j));
+              const uint32_t gw[4] = {g4.x, g4.y, g4.z, g4.w};
+#pragma unroll
+              for (int i = 0; i < 4; ++i) {
+                v[j + 2 * i] *= sigmoid_f<false>(bf16_lo(gw[i]));
+                v[j + 2 * i + 1] *= sigmoid_f<false>(bf16_hi(gw[i]));
+              }
+            }
           }
 #pragma unroll
           for (int j = 0; j < 32; ++j) v[j] *= rs;
@@ -332,7 +353,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
           for (int dst = dst0; dst < dst0 + n_dst; ++dst) {
           void* cbase = p.peer.world ? (void*)peer_slot(p.peer, dst, next_seq) : p.C;
           if (p.out_f32 == 1) {
-            float* out = (float*)cbase + (size_t)row * p.ldc + col0;
+            float* out = (float*)cbase + c_off + (size_t)row * p.ldc + col0;
             if (col0 + 32 <= p.N && (p.ldc & 3) == 0) {
 #pragma unroll
               for (int j = 0; j < 32; j += 4) *reinterpret_cast<float4*>(out + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
@@ -341,7 +362,7 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
             }
           } else {
             const bool h = p.out_f32 == 2;
-            __nv_bfloat16* out = (__nv_bfloat16*)cbase + (size_t)row * p.ldc + col0;
+            __nv_bfloat16* out = (__nv_bfloat16*)cbase + c_off + (size_t)row * p.ldc + col0;
             if (col0 + 32 <= p.N && (p.ldc & 7) == 0) {
 #pragma unroll
               for (int j = 0; j < 32; j += 8)
@@ -522,10 +543,18 @@ static int dispatch_fmt(int fmt, const CUtensorMap& ta, const CUtensorMap& tb, c
 //   bn         32, 64 or 128 (tile width); the caller picks small tiles for small M
 // Returns 0 or a CUDA / driver error code.
 struct GatherIn { const int* flags; const int* seq; int rows_per_src, world, m_rot; };
+// Activations that are not one dense matrix: per head (heads > 0: row t of head h at a + t * lda + h * a_head, output at c + h * c_head) or pages
+// of 128 rows (pages: page number per m-tile, a_rows rows in all, lda elements apart).
+struct StridedIn {
+  int heads = 0, lda = 0, gate_ld = 0;
+  long long a_head = 0, c_head = 0, a_rows = 0;
+  const void* gate = nullptr;
+  const int* pages = nullptr;
+};
 static int gemm_impl(const void* a, int wfmt, const void* w0, const void* w1, const void* w2, const void* w3, int n_experts,
                      void* c, int ldc, int out_f32, const float* bias, const float* row_scale, int act, float act_alpha,
                      float act_limit, int M, int N, int K, const int* tile_expert, const int* num_m_tiles_dev, int bn,
-                     const mx::PeerOut* peer, cudaStream_t stream, const GatherIn* gin = nullptr);
+                     const mx::PeerOut* peer, cudaStream_t stream, const GatherIn* gin = nullptr, const StridedIn* sin = nullptr);
 
 MX_HOST_API int mx_gemm(const void* a, int wfmt, const void* w0, const void* w1, const void* w2, const void* w3, int n_experts,
                         void* c, int ldc, int out_f32, const float* bias, const float* row_scale, int act, float act_alpha,
@@ -563,7 +592,7 @@ MX_HOST_API int mx_gemm_allreduce(const void* a, int wfmt, const void* w0, const
 static int gemm_impl(const void* a, int wfmt, const void* w0, const void* w1, const void* w2, const void* w3, int n_experts,
                      void* c, int ldc, int out_f32, const float* bias, const float* row_scale, int act, float act_alpha,
                      float act_limit, int M, int N, int K, const int* tile_expert, const int* num_m_tiles_dev, int bn,
-                     const mx::PeerOut* peer, cudaStream_t stream, const GatherIn* gin) {
+                     const mx::PeerOut* peer, cudaStream_t stream, const GatherIn* gin, const StridedIn* sin) {
   using namespace mx;
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   if (K % 8) return -101;
@@ -591,8 +620,26 @@ static int gemm_impl(const void* a, int wfmt, const void* w0, const void* w1, co
     p.group_m = 1;                                      // m-major walk: all n-tiles of a row chunk before the next chunk is needed
   }
 
+  p.batch_tiles = 0; p.c_batch = 0; p.gate = nullptr; p.gate_ld = 0; p.a_pages = nullptr;
+
   CUtensorMap ta, tb;
-  {
+  if (sin && sin->heads) {
+    p.batch_tiles = p.num_m_tiles;
+    p.num_m_tiles *= sin->heads;
+    p.c_batch = sin->c_head; p.gate = (const __nv_bfloat16*)sin->gate; p.gate_ld = sin->gate_ld; p.group_m = 1;
+    uint64_t dims[3] = {(uint64_t)K, (uint64_t)M, (uint64_t)sin->heads};
+    uint64_t strides[2] = {(uint64_t)sin->lda * 2, (uint64_t)sin->a_head * 2};
+    uint32_t box[3] = {BK, BM, 1};
+    int r = make_tmap_bf16(&ta, a, 3, dims, strides, box, 1);
+    if (r) return r;
+  } else if (sin) {
+    p.a_pages = sin->pages;
+    uint64_t dims[2] = {(uint64_t)K, (uint64_t)sin->a_rows};
+    uint64_t strides[1] = {(uint64_t)sin->lda * 2};
+    uint32_t box[2] = {BK, BM};
+    int r = make_tmap_bf16(&ta, a, 2, dims, strides, box, 1);
+    if (r) return r;
+  } else {
     uint64_t dims[2] = {(uint64_t)K, (uint64_t)M};
     uint64_t strides[1] = {(uint64_t)K * 2};
     uint32_t box[2] = {BK, BM};
@@ -614,4 +661,30 @@ static int gemm_impl(const void* a, int wfmt, const void* w0, const void* w1, co
     case 32: return dispatch_fmt<32, 8, 6, 4>(wfmt, ta, tb, p, stream);
     default: return -105;
   }
+}
+
+// Every head its own matrix: c[t][h][:] = a[t][h][:] W[h]^T (* sigmoid(gate[t][h][:])).  a: row t of head h at t * lda + h * a_head, K elements; w bf16
+// [heads][N][K]; c: bf16, row t of head h at t * ldc + h * c_head; gate (or null): rows of heads * N, gate_ld apart.  Widths, strides and bases are
+// multiples of 8 elements.
+MX_HOST_API int mx_gemm_heads(const void* a, int lda, long long a_head, const void* w, void* c, int ldc, long long c_head, const void* gate, int gate_ld,
+                              int T, int heads, int N, int K, int bn, cudaStream_t stream) {
+  if (T <= 0 || heads <= 0) return 0;
+  if (N % 8 || K % 8 || lda % 8 || a_head % 8 || ldc % 8 || c_head % 8 || (gate && gate_ld % 8)) return -101;
+  if (((uintptr_t)a | (uintptr_t)w | (uintptr_t)c | (uintptr_t)gate) & 15) return -101;
+  StridedIn s;
+  s.heads = heads; s.lda = lda; s.a_head = a_head; s.c_head = c_head; s.gate = gate; s.gate_ld = gate_ld;
+  return gemm_impl(a, mx::WF_BF16, w, nullptr, nullptr, nullptr, heads, c, ldc, 0, nullptr, nullptr, 0, 0.f, 0.f, T, N, K, nullptr, nullptr, bn, nullptr, stream,
+                   nullptr, &s);
+}
+
+// c[i * 128 + r][:] = (row r of page pages[i]) W^T for the first num_tiles[0] of max_tiles pages.  a: pages of 128 rows, lda elements apart, K of them
+// used (a_rows rows in all); w bf16 [N][K]; c bf16 [max_tiles * 128][N].
+MX_HOST_API int mx_gemm_paged(const void* a, int lda, long long a_rows, const int* pages, const int* num_tiles, const void* w, void* c, int max_tiles, int N,
+                              int K, int bn, cudaStream_t stream) {
+  if (max_tiles <= 0) return 0;
+  if (lda % 8 || a_rows % 128 || !pages || !num_tiles || (((uintptr_t)a | (uintptr_t)w | (uintptr_t)c) & 15)) return -101;
+  StridedIn s;
+  s.lda = lda; s.a_rows = a_rows; s.pages = pages;
+  return gemm_impl(a, mx::WF_BF16, w, nullptr, nullptr, nullptr, 1, c, N, 0, nullptr, nullptr, 0, 0.f, 0.f, max_tiles * 128, N, K, nullptr, num_tiles, bn, nullptr,
+                   stream, nullptr, &s);
 }

@@ -7,6 +7,7 @@
 //   combine  : y[t] (+)= sum_k w[t,k] * packed_out[pos(t,k)]  (fixed order: deterministic)
 // Reference parity: src/ops/moe.cpp:30-80,268-291,371-429, host router src/model/gptoss.cpp:23-47,
 // host packer src/model/qwen3moe_pack.cpp:5-31, reduce src/ops/moe_fused.cpp:1937-1961.
+#include "act.cuh"
 #include "common.cuh"
 #include "comm.cuh"
 #include "host_util.h"
@@ -17,12 +18,13 @@ namespace mx {
 constexpr int MOE_TILE = 128;
 
 // one warp per token; E <= 1024
+template <bool PRECISE>
 __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int T, int E, int K,
                                                         int renorm, int* __restrict__ topk_idx, float* __restrict__ topk_w) {
   pdl_prologue();
   const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
   if (t >= T) return;
-  route_token_warp(logits, bias, t, E, K, renorm, topk_idx, topk_w);
+  route_token_warp<PRECISE>(logits, bias, t, E, K, renorm, topk_idx, topk_w);
 }
 
 // Single-CTA packer.  n = T*K pairs.  Outputs:
@@ -183,8 +185,8 @@ __global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ x, const int
 }
 
 // out[t][:] = (accumulate ? out : 0) + sum_k w[t,k] * yp[pair_to_packed[t,k]][:]
-template <typename OT>
-__global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ yp, const int* __restrict__ pair_to_packed, const float* __restrict__ w,
+template <typename YT, typename OT>
+__global__ void moe_combine_kernel(const YT* __restrict__ yp, const int* __restrict__ pair_to_packed, const float* __restrict__ w,
                                    OT* __restrict__ out, int H, int K, int accumulate) {
   pdl_prologue();
   const int t = blockIdx.x;
@@ -193,10 +195,10 @@ __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ yp, const i
     for (int k = 0; k < K; ++k) {
       const int pos = pair_to_packed[(size_t)t * K + k];
       if (pos < 0) continue;
-      const uint32_t v = *reinterpret_cast<const uint32_t*>(yp + (size_t)pos * H + i);
+      const float2 v = load2(yp + (size_t)pos * H + i);
       const float ww = w[(size_t)t * K + k];
-      a0 = fmaf(ww, bf16_lo(v), a0);
-      a1 = fmaf(ww, bf16_hi(v), a1);
+      a0 = fmaf(ww, v.x, a0);
+      a1 = fmaf(ww, v.y, a1);
     }
     if constexpr (sizeof(OT) == 4) {
       float* o = (float*)out + (size_t)t * H + i;
@@ -282,11 +284,13 @@ MX_HOST_API int mx_moe_combine_push(const void* yp, const int* pair_to_packed, c
   return (int)cudaGetLastError();
 }
 
-MX_HOST_API int mx_moe_route(const float* logits, const float* bias, int T, int E, int K, int renorm, int* topk_idx, float* topk_w,
+// precise: the softmax uses the full-precision exponential
+MX_HOST_API int mx_moe_route(const float* logits, const float* bias, int T, int E, int K, int renorm, int precise, int* topk_idx, float* topk_w,
                              cudaStream_t st) {
   if (T <= 0) return 0;
   if (E > 1024 || K > 32 || K > E) return -120;
-  launch_pdl(moe_route_kernel, dim3((T + 3) / 4), dim3(128), 0, st, logits, bias, T, E, K, renorm, topk_idx, topk_w);
+  if (precise) launch_pdl(moe_route_kernel<true>, dim3((T + 3) / 4), dim3(128), 0, st, logits, bias, T, E, K, renorm, topk_idx, topk_w);
+  else launch_pdl(moe_route_kernel<false>, dim3((T + 3) / 4), dim3(128), 0, st, logits, bias, T, E, K, renorm, topk_idx, topk_w);
   return (int)cudaGetLastError();
 }
 
@@ -316,11 +320,14 @@ MX_HOST_API int mx_moe_gather(const void* x, const int* packed_token, const int*
   return (int)cudaGetLastError();
 }
 
-MX_HOST_API int mx_moe_combine(const void* yp, const int* pair_to_packed, const float* w, void* out, int out_f32, int T, int H, int K,
+// yp: bf16 rows, or fp32 ones (y_f32; out is fp32 then too)
+MX_HOST_API int mx_moe_combine(const void* yp, int y_f32, const int* pair_to_packed, const float* w, void* out, int out_f32, int T, int H, int K,
                                int accumulate, cudaStream_t st) {
   if (T <= 0) return 0;
-  if (H % 2) return -101;
-  if (out_f32) launch_pdl(moe_combine_kernel<float>, dim3(T), dim3(256), 0, st, (const __nv_bfloat16*)yp, pair_to_packed, w, (float*)out, H, K, accumulate);
-  else launch_pdl(moe_combine_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, st, (const __nv_bfloat16*)yp, pair_to_packed, w, (__nv_bfloat16*)out, H, K, accumulate);
+  if (H % 2 || (y_f32 && !out_f32)) return -101;
+  using bf = __nv_bfloat16;
+  if (y_f32) launch_pdl(moe_combine_kernel<float, float>, dim3(T), dim3(256), 0, st, (const float*)yp, pair_to_packed, w, (float*)out, H, K, accumulate);
+  else if (out_f32) launch_pdl(moe_combine_kernel<bf, float>, dim3(T), dim3(256), 0, st, (const bf*)yp, pair_to_packed, w, (float*)out, H, K, accumulate);
+  else launch_pdl(moe_combine_kernel<bf, bf>, dim3(T), dim3(256), 0, st, (const bf*)yp, pair_to_packed, w, (bf*)out, H, K, accumulate);
   return (int)cudaGetLastError();
 }

@@ -6,6 +6,10 @@
 
 namespace mx {
 
+template <bool PRECISE> __device__ __forceinline__ float route_exp(float x) { return PRECISE ? expf(x) : __expf(x); }
+
+// PRECISE: weights through expf (models that run in 32-bit), otherwise the fast exponential.
+template <bool PRECISE = false>
 __device__ __forceinline__ void route_token_warp(const float* __restrict__ logits, const float* __restrict__ bias, int t, int E, int K, int renorm,
                                                  int* __restrict__ topk_idx, float* __restrict__ topk_w, int w_copies = 1) {
   const int lane = threadIdx.x & 31;
@@ -21,7 +25,7 @@ __device__ __forceinline__ void route_token_warp(const float* __restrict__ logit
   mx_all = warp_max(mx_all);
   float denom_all = 0.f;
 #pragma unroll
-  for (int i = 0; i < 32; ++i) if (i < per) denom_all += __expf(v[i] - mx_all);
+  for (int i = 0; i < 32; ++i) if (i < per) denom_all += route_exp<PRECISE>(v[i] - mx_all);
   denom_all = warp_sum(denom_all);
   float sel_sum = 0.f;
   float my_w = 0.f; int my_e = 0;    // lane k keeps the k-th selection (K <= 32)
@@ -38,7 +42,7 @@ __device__ __forceinline__ void route_token_warp(const float* __restrict__ logit
       const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
       if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
     }
-    const float pw = __expf(best - mx_all);
+    const float pw = route_exp<PRECISE>(best - mx_all);
     sel_sum += pw;
     if (lane == k) { my_w = pw; my_e = bi; }
 #pragma unroll

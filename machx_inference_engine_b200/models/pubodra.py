@@ -99,4 +99,5 @@ class PubodraModel(LayerListModel):
 
     def _head(self, x, delta, fb: ForwardBatch):
         rows = fb.logit_rows if fb.logit_rows is not None else (fb.cu_q[1:].long() - 1)
-        return self.lm_head(self._dyt(x.index_select(0, rows), self.final_norm, delta.index_select(0, rows)), out_f32=True)
+        delta = delta.index_select(0, rows) if isinstance(delta, torch.Tensor) else delta.rows(rows)
+        return self.lm_head(self._dyt(x.index_select(0, rows), self.final_norm, delta), out_f32=True)

@@ -59,10 +59,10 @@ class ForwardBatch:
     def B(self) -> int:
         return self.seq_lens.numel()
 
-    def query_parts(self) -> list:
-        """[(first row, end row, block table, sequence lengths, cu_q, longest query)]: the batch, or its short and its long queries (cu_q keeps
-        the rows of the whole batch)."""
-        if self.short is None:
+    def query_parts(self, apart: bool = True) -> list:
+        """[(first row, end row, block table, sequence lengths, cu_q, longest query)]: the batch, or (``apart``) its short and its long queries
+        (cu_q keeps the rows of the whole batch)."""
+        if self.short is None or not apart:
             return [(0, self.T, self.block_table, self.seq_lens, self.cu_q, self.max_q_len)]
         n, rows, longest = self.short
         return [(0, rows, self.block_table[:n], self.seq_lens[:n], self.cu_q[:n + 1], longest),
@@ -378,8 +378,9 @@ class LatentAttentionBlock:
         T, H, d, R = y.shape[0], self.n_q, self.d, self.R
         q, ckv, gate = y[:, :self.cols[0]].view(T, H, d + self.r), y[:, self.cols[0]:self.cols[1]], y[:, self.cols[1]:]
         a = torch.empty(T, H, self.v, dtype=y.dtype, device=y.device)
-        for lo, hi, table, lens, cu, longest in fb.query_parts():
-            latent = longest < self.EXPAND_MIN_Q or (y.is_cuda and y.dtype == torch.float32)
+        expand = not (y.is_cuda and y.dtype == torch.float32)          # 32-bit kernels: latent space only
+        for lo, hi, table, lens, cu, longest in fb.query_parts(apart=expand):
+            latent = longest < self.EXPAND_MIN_Q or not expand
             rows = slice(lo, hi)
             qc = torch.empty(hi - lo, H, R + self.r, dtype=y.dtype, device=y.device) if latent else None
             ops.latent_post(q[rows, :, d:], ckv[rows], self.norm, self.rank, self.eps, fb.positions[rows], self.rope[0], self.rope[1], fb.slot_map[rows],
@@ -595,7 +596,7 @@ class MoEFFN:
             idx, w, xq, sfx = moe_route_quant(logits, self.router_bias, self.K, h, w_copies=ksplit)
             pre = (xq, sfx)
         else:
-            idx, w = ops.moe_route(logits, self.router_bias, self.K, True)
+            idx, w = ops.moe_route(logits, self.router_bias, self.K, True, precise=h.dtype == torch.float32)
         if self.expert_scale is not None:
             w = w * self.expert_scale[idx.long()]
         local = self.e_hi - self.e_lo

@@ -143,6 +143,20 @@ def group_norm(x, w, eps, groups=1, delta=None, delta_w=None, fresh=False, width
     return out
 
 
+def dyt_norm(x, alpha, w, b, delta=None, step=None, out_dtype=torch.bfloat16, want_out=True):
+    T, ld = x.shape
+    comb = delta if isinstance(delta, CombineDelta) else None
+    rows = comb.y if comb is not None else delta
+    assert x.dtype == torch.float32 and x.is_contiguous() and w.numel() == b.numel() == ld and (step is None or step.numel() == ld)
+    assert rows is None or (rows.is_contiguous() and rows.shape[1] == ld and (comb is not None or rows.shape[0] == T))
+    out = torch.empty(T, ld, dtype=out_dtype, device=x.device) if want_out else None
+    _check(_lib.cuda().mx_dyt_norm(_p(x), _p(rows), int(rows is not None and rows.dtype == torch.float32), _p(comb.pair_to_packed if comb else None),
+                                   _p(comb.w if comb else None), comb.w.shape[1] if comb else 0, _p(step), C.c_float(alpha), _p(w), _p(b), _p(out),
+                                   int(out_dtype == torch.float32), T, ld, _stream()), "dyt_norm")
+    _count()
+    return out
+
+
 def kv_store(k, v, slot_map, k_cache, v_cache):
     T, n_kv, bs, dk = k.shape[0], k_cache.shape[1], k_cache.shape[2], k_cache.shape[3]
     dv = v_cache.shape[3]
@@ -178,6 +192,11 @@ class CombineDelta:
     def index_select(self, dim, rows):
         assert dim == 0
         return self.materialize().index_select(0, rows)
+
+    def rows(self, rows):
+        """The combine of some tokens only, still not formed."""
+        K = self.w.shape[1]
+        return CombineDelta(self.y, self.pair_to_packed.view(-1, K).index_select(0, rows).reshape(-1), self.w.index_select(0, rows))
 
 
 @_profiled("rmsnorm_combine")
@@ -467,7 +486,15 @@ def grouped_linear(xp, w: QuantWeight, tile_expert, num_tiles, bias=None, act=AC
                    out_dtype=None):
     """``out_dtype`` (bf16 / fp16 / fp32) overrides ``out_f32``; fp16 feeds a following MXFP4 GEMM without a cast."""
     P = xp.shape[0]
-    n_out = w.N // 2 if act != ACT_NONE else w.N
+    if xp.dtype == torch.float32:            # 32-bit models: every row in fp32 on the CUDA cores
+        if w.fmt != WFormat.BF16 or bias is not None or act_gated(act) or out_dtype not in (None, torch.float32):
+            raise KernelError("32-bit grouped layers take bf16 weights without biases and no gated activation")
+        out = torch.empty(P, w.N, dtype=torch.float32, device=xp.device)
+        _check(_lib.cuda().mx_grouped_linear_f32(_p(xp), _p(w.p0), _p(out), P, w.N, w.K, _p(tile_expert), _p(num_tiles), act, C.c_float(act_alpha),
+                                                 C.c_float(act_limit), _stream()), "grouped linear_f32")
+        _count()
+        return out
+    n_out = w.N // 2 if act_gated(act) else w.N
     odt = out_dtype or (torch.float32 if out_f32 else torch.bfloat16)
     out = torch.empty(P, n_out, dtype=odt, device=xp.device)
     fmt, p0, p1, p2, p3 = _planes(w)
@@ -482,7 +509,7 @@ def expert_gemv(x, w: QuantWeight, slot_expert, x_div=1, bias=None, act=ACT_NONE
                 e_lo=0):
     """``w`` holds experts [e_lo, e_lo + w.E); slots routed to other experts produce zero rows (expert parallelism)."""
     S = slot_expert.numel()
-    n_out = w.N // 2 if act != ACT_NONE else w.N
+    n_out = w.N // 2 if act_gated(act) else w.N
     out = torch.empty(S, n_out, dtype=torch.float32 if out_f32 else torch.bfloat16, device=x.device)
     fmt, p0, p1, p2, p3 = _planes(w)
     _check(_lib.cuda().mx_gemv_experts(fmt, p0, p1, p2, p3, _p(x), _p(out), _p(bias), w.N, w.K, int(out_f32), act, C.c_float(act_alpha),
@@ -559,15 +586,16 @@ def _tc_prefill_takes(q, dk, dv, softcap, kv_scales) -> bool:
 
 
 def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks=None, window=0, scale=None, softcap=0.0, n_splits=None,
-              kv_scales=None, max_kv_len=0, q_scale=None, gate=None):
+              kv_scales=None, max_kv_len=0, q_scale=None, gate=None, v_width=0):
+    """``v_cache`` None: a value is the first ``v_width`` elements of its key row (latent cache)."""
     Tq, n_q, hd = q.shape
-    n_kv, bs, dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
-    assert k_cache.dtype == torch.int8 or k_cache.dtype == v_cache.dtype == q.dtype
+    n_kv, bs, dv = k_cache.shape[1], k_cache.shape[2], v_width if v_cache is None else v_cache.shape[3]
+    assert k_cache.dtype == torch.int8 or (k_cache.dtype == q.dtype and (v_cache is None or v_cache.dtype == q.dtype))
     assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape == (Tq, n_q * dv))
     B = seq_lens.numel()
     scale = scale if scale is not None else 1.0 / math.sqrt(hd)
     assert (k_cache.dtype == torch.int8) == (kv_scales is not None)
-    if max_q_len >= TC_PREFILL_MIN_Q and bs == 128 and n_splits is None and _tc_prefill_takes(q, hd, dv, softcap, kv_scales):
+    if max_q_len >= TC_PREFILL_MIN_Q and bs == 128 and n_splits is None and v_cache is not None and _tc_prefill_takes(q, hd, dv, softcap, kv_scales):
         if kv_scales is not None:       # the tensor-core kernel reads bf16 pages: expand this batch's pages first
             dk, dv, table = _dequant_pages(k_cache, v_cache, kv_scales, block_table, seq_lens, max_kv_len)
             return attention_prefill_tc(q, dk, dv, table, seq_lens, cu_q, max_q_len, sinks=sinks, window=window, scale=scale, softcap=softcap,
@@ -610,12 +638,110 @@ def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks
     return out
 
 
+# ------------------------------------------------------------------ latent attention
+def latent_post(q_rot, ckv, norm_w, rank, eps, positions, rope_cos, rope_sin, slot_map, cache, q_out):
+    T, H, r = q_rot.shape
+    R = norm_w.numel()
+    assert q_rot.dtype == ckv.dtype == cache.dtype == q_out.dtype and q_rot.stride(2) == ckv.stride(1) == q_out.stride(2) == 1
+    assert cache.is_contiguous() and cache.shape[1] == 1 and cache.shape[3] == R + r == ckv.shape[1] and q_out.shape == q_rot.shape
+    _check(_lib.cuda().mx_latent_post(_p(q_rot), q_rot.stride(0), q_rot.stride(1), _p(q_out), q_out.stride(0), q_out.stride(1), _p(ckv), ckv.stride(0),
+                                      _p(norm_w), int(rank), C.c_float(eps), _p(positions), _p(rope_cos), _p(rope_sin), rope_cos.shape[1], rope_cos.shape[0],
+                                      _p(slot_map), _p(cache), T, H, R, r, int(cache.dtype == torch.float32), _stream()), "latent_post")
+    _count()
+
+
+HEAD_GEMV_MAX_T = 8          # up to this many rows a head's matrix is streamed by the CUDA cores; more go to the tensor cores
+
+
+def head_linear(x, w: QuantWeight, gate=None, out=None):
+    T, H, K = x.shape
+    assert w.fmt == WFormat.BF16 and (w.E, w.K) == (H, K) and x.stride(2) == 1
+    if out is None:
+        out = torch.empty(T, H, w.N, dtype=x.dtype, device=x.device)
+    assert out.shape == (T, H, w.N) and out.dtype == x.dtype and out.stride(2) == 1 and (gate is None or (gate.dtype == x.dtype and gate.stride(1) == 1))
+    g_ld = 0 if gate is None else gate.stride(0)
+    if x.dtype == torch.float32 or T <= HEAD_GEMV_MAX_T:
+        _check(_lib.cuda().mx_head_linear(_p(x), C.c_longlong(x.stride(0)), x.stride(1), _p(w.p0), _p(gate), g_ld, _p(out), C.c_longlong(out.stride(0)),
+                                          out.stride(1), T, H, w.N, K, int(x.dtype == torch.float32), _stream()), "head_linear")
+    else:
+        tiles = H * ((T + 127) // 128)
+        bn = next((b for b in (128, 64, 32) if tiles * ((w.N + b - 1) // b) >= sm_count()), 32)
+        _check(_lib.cuda().mx_gemm_heads(_p(x), x.stride(0), C.c_longlong(x.stride(1)), _p(w.p0), _p(out), out.stride(0), C.c_longlong(out.stride(1)), _p(gate),
+                                         g_ld, T, H, w.N, K, bn, _stream()), "gemm_heads")
+    _count()
+    return out
+
+
+def latent_attention(q, cache, block_table, seq_lens, cu_q, max_q_len, rank, window=0, scale=1.0, n_splits=None):
+    Tq, H, width = q.shape
+    B, bs = seq_lens.numel(), cache.shape[2]
+    if q.dtype == torch.float32:
+        return attention(q, cache, None, block_table, seq_lens, cu_q, max_q_len, window=window, scale=scale, n_splits=n_splits, v_width=rank)
+    assert q.is_contiguous() and cache.is_contiguous() and q.dtype == cache.dtype == torch.bfloat16 and cache.shape[1:] == (1, 128, width)
+    out = torch.empty(Tq, H, rank, dtype=q.dtype, device=q.device)
+    if n_splits is None:
+        # ranges of whole pages, so that about one CTA per SM exists
+        pages = block_table.shape[1] if window <= 0 else min(block_table.shape[1], (window + max_q_len + bs - 3) // bs + 1)
+        rows = max_q_len * H
+        ctas = B * ((rows + 63) // 64 if rows > 32 else 1)
+        n_splits = max(1, min(pages, ATTN_MAX_SPLITS, sm_count() // ctas))
+    part = torch.empty(n_splits * Tq * H * (rank + 2), dtype=torch.float32, device=q.device) if n_splits > 1 else None
+    ml = part[n_splits * Tq * H * rank:] if part is not None else None
+    _check(_lib.cuda().mx_latent_attention(_p(q), _p(cache), cache.shape[0], _p(block_table), block_table.shape[1], _p(seq_lens), _p(cu_q), _p(out), _p(part),
+                                           _p(ml), B, Tq, int(max_q_len), H, int(rank), width - rank, int(window), C.c_float(scale), int(n_splits), _stream()),
+           "latent_attention")
+    _count()
+    if n_splits > 1:
+        _check(_lib.cuda().mx_attention_combine(_p(part), _p(ml), _p(out), Tq, H, int(rank), int(n_splits), _stream()), "attention_combine")
+        _count()
+    return out
+
+
+def _latent_plan(plans, block_table, seq_lens, cu_q, Tq, window, bs):
+    """(page list, number of live pages, table of the expanded pages) of the batch; one per window and forward."""
+    key = (window, block_table.data_ptr())
+    if plans is not None and key in plans:
+        return plans[key]
+    B, mb = block_table.shape
+    # a segment of n queries reaches n + window - 1 keys: at most n / bs + (window - 2) / bs + 2 pages
+    most = B * mb if window <= 0 else min(B * mb, Tq // bs + 1 + B * ((window + bs - 3) // bs + 2))
+    buf = torch.empty(most + B * mb + 1, dtype=torch.int32, device=block_table.device)
+    pages, table, num = buf[:most], buf[most:most + B * mb], buf[most + B * mb:]
+    _check(_lib.cuda().mx_latent_plan(_p(block_table), _p(seq_lens), _p(cu_q), B, mb, bs, int(window), most, _p(pages), _p(table), _p(num), _stream()), "latent_plan")
+    _count()
+    if plans is not None:
+        plans[key] = (pages, num, table)
+    return pages, num, table
+
+
+def latent_attention_expanded(q, w_kv: QuantWeight, cache, block_table, seq_lens, cu_q, max_q_len, dim, vdim, rank, window=0, scale=1.0, gate=None,
+                              out=None, plans=None):
+    Tq, H, dq = q.shape
+    bs, width = cache.shape[2], cache.shape[3]
+    assert q.dtype == cache.dtype == torch.bfloat16 and bs == 128 and cache.is_contiguous() and w_kv.fmt == WFormat.BF16 and block_table.is_contiguous()
+    assert (w_kv.N, w_kv.K) == (H * (dim + vdim), rank) and dq - dim == width - rank
+    if out is None:
+        out = torch.empty(Tq, H, vdim, dtype=q.dtype, device=q.device)
+    assert out.is_contiguous() and out.shape == (Tq, H, vdim)
+    pages, num, table = _latent_plan(plans, block_table, seq_lens, cu_q, Tq, window, bs)
+    n = pages.numel()
+    kv = torch.empty(n * bs, w_kv.N, dtype=torch.bfloat16, device=q.device)
+    lib = _lib.cuda()
+    _check(lib.mx_gemm_paged(_p(cache), width, C.c_longlong(cache.shape[0] * bs), _p(pages), _p(num), _p(w_kv.p0), _p(kv), n, w_kv.N, rank,
+                             _pick_bn(n * bs, w_kv.N), _stream()), "gemm_paged")
+    _check(lib.mx_attention_prefill_latent(_p(q), _q_rows(q), _p(kv), n, _p(table), _p(cache), cache.shape[0], _p(block_table), block_table.shape[1],
+                                           _p(seq_lens), _p(cu_q), _p(gate), 0 if gate is None else gate.stride(0), _p(out), seq_lens.numel(), Tq,
+                                           int(max_q_len), H, dim, dq - dim, vdim, rank, int(window), C.c_float(scale), _stream()), "attention_prefill_latent")
+    _count(2)
+    return out
+
+
 # ------------------------------------------------------------------ MoE
-def moe_route(logits, bias, k, renorm=True):
+def moe_route(logits, bias, k, renorm=True, precise=False):
     T, E = logits.shape
     idx = torch.empty(T, k, dtype=torch.int32, device=logits.device)
     w = torch.empty(T, k, dtype=torch.float32, device=logits.device)
-    _check(_lib.cuda().mx_moe_route(_p(logits), _p(bias), T, E, k, int(renorm), _p(idx), _p(w), _stream()), "moe_route")
+    _check(_lib.cuda().mx_moe_route(_p(logits), _p(bias), T, E, k, int(renorm), int(precise), _p(idx), _p(w), _stream()), "moe_route")
     _count()
     return idx, w
 
@@ -761,7 +887,7 @@ def expert_group_gemv(x, w: QuantWeight, pk: MoePacking, x_index=None, bias=None
     and multiplies them with all rows routed to it (8 rows per pass).  Row r of the output belongs to packed position r;
     its input is ``x[x_index[r]]`` (gate|up reads the token rows in place) or ``x[r]`` (down)."""
     P = pk.max_rows
-    n_out = w.N // 2 if act != ACT_NONE else w.N
+    n_out = w.N // 2 if act_gated(act) else w.N
     out = torch.empty(P, n_out, dtype=torch.bfloat16, device=x.device)
     fmt, p0, p1, p2, p3 = _planes(w)
     _check(_lib.cuda().mx_gemv_group(fmt, p0, p1, p2, p3, _p(x), _p(x_index), _p(out), _p(bias), w.N, w.K, act, C.c_float(act_alpha),
@@ -774,20 +900,20 @@ def moe_gather(x, pk: MoePacking, f16=False, zero_pad=False):
     """Rows of ``x`` in packed order.  Padding rows of the expert tiles are left unwritten unless ``zero_pad`` (no consumer reads them:
     a grouped GEMM row depends on its own input row only)."""
     H = x.shape[1]
-    xp = torch.empty(pk.max_rows, H, dtype=torch.float16 if f16 else torch.bfloat16, device=x.device)
-    _check(_lib.cuda().mx_moe_gather(_p(x), _p(pk.packed_token), _p(pk.num_tiles), _p(xp), H, pk.max_rows, int(f16), int(zero_pad), _stream()), "moe_gather")
+    assert x.is_contiguous() and (x.dtype == torch.bfloat16 or (x.dtype == torch.float32 and not f16))
+    xp = torch.empty(pk.max_rows, H, dtype=torch.float16 if f16 else x.dtype, device=x.device)
+    _check(_lib.cuda().mx_moe_gather(_p(x), _p(pk.packed_token), _p(pk.num_tiles), _p(xp), H * (x.element_size() // 2), pk.max_rows, int(f16), int(zero_pad), _stream()), "moe_gather")
     _count()
     return xp
 
 
 def moe_combine(yp, pk: MoePacking, w, out=None, accumulate=False):
-    assert yp.dtype == torch.bfloat16
     T, K = w.shape
     H = yp.shape[1]
     if out is None:
         out = torch.empty(T, H, dtype=torch.float32, device=yp.device)
         accumulate = False
-    _check(_lib.cuda().mx_moe_combine(_p(yp), _p(pk.pair_to_packed), _p(w), _p(out), int(out.dtype == torch.float32), T, H, K,
+    _check(_lib.cuda().mx_moe_combine(_p(yp), int(yp.dtype == torch.float32), _p(pk.pair_to_packed), _p(w), _p(out), int(out.dtype == torch.float32), T, H, K,
                                       int(accumulate), _stream()), "moe_combine")
     _count()
     return out

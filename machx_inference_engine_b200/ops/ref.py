@@ -581,7 +581,7 @@ def deltanet_scan_chunked(qkv, n_k, ab, a_idx, b_idx, k_of_v, ssm_a, dt_bias, st
     return out.reshape(T, n_v * D)
 
 
-def moe_route(logits, bias, k, renorm=True):
+def moe_route(logits, bias, k, renorm=True, precise=False):
     x = logits.to(torch.float32)
     if bias is not None:
         x = x + bias
