@@ -1,4 +1,4 @@
-"""Shared by the Tikarax tests: checkpoint folders from oracle weights, engines over them, the error measure."""
+"""Shared by the tests of layer-list designs: checkpoint folders from oracle weights, engines over them, the error measure."""
 import json
 import os
 
@@ -21,7 +21,7 @@ def write_folder(path, cfg, weights):
     os.makedirs(path, exist_ok=True)
     with open(os.path.join(path, "config.json"), "w") as f:
         json.dump(cfg, f)
-    bits = {n: ("BF16", (np.ascontiguousarray(a, dtype=np.float32).view(np.uint32) >> 16).astype(np.uint16)) for n, a in weights.items()}
+    bits = {n: ("BF16", (np.array(a, dtype=np.float32, order="C").view(np.uint32) >> 16).astype(np.uint16)) for n, a in weights.items()}
     write_safetensors(os.path.join(path, "model.safetensors"), bits)
     return str(path)
 

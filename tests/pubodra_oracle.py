@@ -180,8 +180,9 @@ def round_bf16(a):
     return u.view(np.float32)
 
 
-def random_weights(cfg, seed=0):
-    """Every tensor the configuration asks for, as float32 arrays that hold bfloat16 values."""
+def random_weights(cfg, seed=0, clear_routing=False):
+    """Every tensor the configuration asks for, as float32 arrays that hold bfloat16 values.  ``clear_routing``: the routers read a few columns
+    that hold a code of the token and that no layer writes to, so that no choice of experts is within rounding of another."""
     g = np.random.default_rng(seed)
     H, W = cfg["width"], {}
 
@@ -217,4 +218,33 @@ def random_weights(cfg, seed=0):
             for e in range(f["router"]["experts"]):
                 mat(f"{l}.mlp.e{e}.up", f["expert"]["ff"], H)
                 mat(f"{l}.mlp.e{e}.down", H, f["expert"]["ff"])
+    if clear_routing:
+        _settle_routing(cfg, W, g)
     return W
+
+
+def _settle_routing(cfg, W, g, codes=8, gap=0.3):
+    for n in list(W):
+        if n.endswith(".mix.o") or n.endswith(".down"):
+            W[n][:codes] = 0.0
+        elif n == "loop.step":
+            W[n][:, :codes] = 0.0
+    layers = [i for i, layer in enumerate(cfg["layers"]) if layer["mlp"] is not None and layer["mlp"]["kind"] == "moe"]
+    for i in layers:
+        W[f"l{i}.mlp.router"] = round_bf16(np.pad(g.standard_normal((cfg["layers"][i]["mlp"]["router"]["experts"], codes)), ((0, 0), (0, cfg["width"] - codes))))
+    for t in range(cfg["vocab"]):
+        for _ in range(2000):
+            x = np.zeros(cfg["width"])
+            x[:codes] = 2.0 * g.choice([-1.0, 1.0], codes)
+            gaps = [np.inf]
+            for i in layers:
+                l, top = f"l{i}", cfg["layers"][i]["mlp"]["router"]["top"]
+                h = dynamic_tanh(x, *(np.float64(W[f"{l}.norm2{s}"]) for s in (".alpha", "", ".b")))
+                z = np.sort(np.float64(W[f"{l}.mlp.router"])[:, :codes] @ h[:codes])[::-1]
+                if top < len(z):
+                    gaps.append(z[top - 1] - z[top])
+            if min(gaps) > gap:
+                break
+        else:
+            raise ValueError("no code of this token settles its routing")
+        W["embed"][t, :codes] = x[:codes]

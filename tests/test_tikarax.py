@@ -5,7 +5,7 @@ import pytest
 import torch
 
 import tikarax_oracle as oracle
-from tikarax_util import ARMS, TOL, engine, logit_error, run_portions, tokens_of, write_folder
+from design_util import ARMS, TOL, engine, logit_error, run_portions, tokens_of, write_folder
 from machx_inference_engine_b200.models import load_model
 from machx_inference_engine_b200.runtime.engine import EngineOptions, LLMEngine, OutOfBlocks, SamplingParams
 

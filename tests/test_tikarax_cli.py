@@ -8,7 +8,7 @@ import pytest
 import torch
 
 import tikarax_oracle as oracle
-from tikarax_util import ARMS, TOL, logit_error, tokens_of, write_folder
+from design_util import ARMS, TOL, logit_error, tokens_of, write_folder
 from machx_inference_engine_b200 import _build
 from machx_inference_engine_b200.cli import trace_run
 from machx_inference_engine_b200.cli.inspect_gguf import inspect

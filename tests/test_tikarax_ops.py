@@ -5,7 +5,7 @@ import pytest
 import torch
 
 import tikarax_oracle as oracle
-from tikarax_util import DEVICES
+from design_util import DEVICES
 from machx_inference_engine_b200 import ops
 from machx_inference_engine_b200.ops import QuantWeight, WFormat
 from machx_inference_engine_b200.utils.rope import query_temperature_table
