@@ -1,13 +1,13 @@
 """Throughput of a layer-list design beside the framework's closest models at equal size, and its kernels beside the like kernels.
 
-    python bench.py --design tikarax [--design-part models|kernels|all]
+    python bench.py --design tikarax|pubodra [--design-part models|kernels|all]
 
 Models (random-init bf16 weights, random tokens): prefill of one 4096-token prompt and decode at a 2048-token context for 1, 8 and 32
 sequences, through ``LLMEngine`` (CUDA graphs as in serving), for
-  * the design as its preset orders it (one attention layer in four, minGRU otherwise),
-  * the design with attention in every layer,
-  * a llama of the same width, heads and parameters per layer (gated feed-forward of 2/3 the width),
-  * a DeltaNet hybrid (qwen35) of the same width, with full attention in every fourth layer.
+  tikarax:  the design as its preset orders it (one attention layer in four, minGRU otherwise), with attention in every layer; a llama of the same
+            width, heads and parameters per layer (gated feed-forward of 2/3 the width); a DeltaNet hybrid (qwen35) of the same width
+  pubodra:  the design with dense feed-forwards, with experts in every other layer, and with experts in every layer; a llama of the same width,
+            heads, sliding window and parameters per layer; a qwen3moe with the same experts (gated, 2/3 the width) in every layer
 Weights are larger than L2 (126 MB), so every pass streams them.
 
 Kernels: device time inside a CUDA graph over buffers that together exceed L2, as a fraction of the roofline (bytes over the measured copy
@@ -22,24 +22,37 @@ import time
 
 import torch
 
-from ..formats.model_config import ModelConfig, _tikarax_preset
+from ..formats.model_config import ModelConfig, _pubodra_preset, _tikarax_preset
 
 LAYERS = 8
-SIZES = {  # hidden, heads, kv_heads, head width, un-gated feed-forward, minGRU width
+SIZES = {"tikarax": {  # hidden, heads, kv_heads, head width, un-gated feed-forward, minGRU width
     "1b-layers": dict(hidden=2048, heads=32, kv_heads=8, dim=64, ffn=12288, width=4096),
     "8b-layers": dict(hidden=4096, heads=32, kv_heads=8, dim=128, ffn=21504, width=6144),
-}
+}, "pubodra": {       # hidden, heads, unrotated / rotated / value widths, latent, window, un-gated feed-forward; experts, per token, their width
+    "1b-layers": dict(hidden=2048, heads=16, dim=128, rot=64, vdim=128, rank=512, window=1024, ffn=12288, experts=64, used=6, eff=1536),
+    "8b-layers": dict(hidden=4096, heads=32, dim=128, rot=64, vdim=128, rank=512, window=4096, ffn=21504, experts=64, used=6, eff=2304),
+}}
 VOCAB = 32768
 PREFILL, CONTEXT, DECODE = 4096, 2048, 64
 
 
-def _configs(s: dict) -> dict:
+def _tikarax_configs(s: dict) -> dict:
     tk = lambda every: _tikarax_preset(s["hidden"], LAYERS, s["heads"], s["kv_heads"], s["dim"], s["dim"], s["ffn"], s["width"], VOCAB, attn_every=every)
     common = dict(n_layers=LAYERS, hidden=s["hidden"], n_heads=s["heads"], n_kv_heads=s["kv_heads"], ffn=s["ffn"] * 2 // 3, vocab=VOCAB, ctx_train=16384)
     return {"tikarax": tk(4), "tikarax, attention only": tk(1),
             "llama": ModelConfig(arch="llama", head_dim=s["dim"], n_rot=s["dim"], **common),
             "qwen35 hybrid": ModelConfig(arch="qwen35", head_dim=s["dim"], n_rot=s["dim"] // 2, full_attn_interval=4, ssm_inner=32 * 128, ssm_state=128,
                                          ssm_n_k_heads=16, ssm_n_v_heads=32, ssm_conv_kernel=4, **common)}
+
+
+def _pubodra_configs(s: dict) -> dict:
+    pb = lambda moe_every: _pubodra_preset(s["hidden"], LAYERS, s["heads"], s["dim"], s["rot"], s["vdim"], s["rank"], s["window"], s["ffn"], VOCAB,
+                                           *((s["experts"], s["used"], s["eff"], moe_every) if moe_every else ()))
+    common = dict(n_layers=LAYERS, hidden=s["hidden"], n_heads=s["heads"], n_kv_heads=s["heads"] // 4, head_dim=128, n_rot=128, vocab=VOCAB, ctx_train=16384,
+                  sliding_window=s["window"])
+    return {"pubodra, dense": pb(0), "pubodra, experts in every other layer": pb(2), "pubodra, experts": pb(1),
+            "llama": ModelConfig(arch="llama", ffn=s["ffn"] * 2 // 3, **common),
+            "qwen3moe": ModelConfig(arch="qwen3moe", ffn=s["ffn"] * 2 // 3, n_experts=s["experts"], n_experts_used=s["used"], expert_ffn=s["eff"] * 2 // 3, **common)}
 
 
 def _timed(fn) -> float:
@@ -52,12 +65,12 @@ def _timed(fn) -> float:
     return e0.elapsed_time(e1)
 
 
-def bench_models(dev, emit) -> None:
+def bench_models(design, dev, emit) -> None:
     from ..models import build_model
     from ..ops import cuda as K
     from ..runtime.engine import EngineOptions, LLMEngine, SamplingParams
-    for size, s in SIZES.items():
-        for name, cfg in _configs(s).items():
+    for size, s in SIZES[design].items():
+        for name, cfg in {"tikarax": _tikarax_configs, "pubodra": _pubodra_configs}[design](s).items():
             model = build_model(cfg, dev, quant="bf16", max_ctx=PREFILL + 256)
             row = {"size": size, "model": name, "layers": LAYERS, "weight_gb": round(model.weight_bytes() / 1e9, 2)}
             g = torch.Generator().manual_seed(0)
@@ -116,24 +129,39 @@ def _per_call(fns: list, reps: int = 40) -> float:
     return sorted(_timed(g.replay) for _ in range(7))[3] * 1e3 / n
 
 
-def bench_kernels(dev, emit) -> None:
+class _Rows:
+    """Helpers of a kernel table: buffers, and one timed row per kernel."""
+
+    def __init__(self, dev, emit):
+        from .kernel_bench import peaks
+        self.dev, self.emit, self.pk = dev, emit, peaks()
+
+    def bf(self, *sh):
+        return (torch.randn(*sh, device=self.dev) * 0.5).to(torch.bfloat16)
+
+    def i32(self, v):
+        return torch.tensor(v, dtype=torch.int32, device=self.dev)
+
+    @staticmethod
+    def bufs(nbytes):
+        return max(2, int(3e8 // nbytes) + 1) if nbytes < 3e8 else 1
+
+    def row(self, kernel, role, fns, bytes_=0.0, flops=0.0):
+        us = _per_call(fns)
+        pk = self.pk
+        roof = max(bytes_ / pk["hbm_gbs"] / 1e3, flops / pk["bf16_tflops"] / 1e6)
+        self.emit({"kernel": kernel, "role": role, "us": round(us, 2), "gbs": round(bytes_ / us / 1e3) if bytes_ else None,
+                   "tflops": round(flops / us / 1e6, 1) if flops else None, f"fraction_of_{pk['src']}_roofline": round(roof / us, 3)})
+
+
+def bench_kernels_tikarax(dev, emit) -> None:
     from ..ops import cuda as K
     from ..ops import ref
     from ..ops.weights import QuantWeight, WFormat
     from ..utils.rope import query_temperature_table, rope_tables
-    from .kernel_bench import peaks
-    pk = peaks()
-    bf = lambda *sh: (torch.randn(*sh, device=dev) * 0.5).to(torch.bfloat16)
-    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
-    bufs = lambda nbytes: max(2, int(3e8 // nbytes) + 1) if nbytes < 3e8 else 1
-
-    def row(kernel, role, fns, bytes_=0.0, flops=0.0):
-        us = _per_call(fns)
-        roof = max(bytes_ / pk["hbm_gbs"] / 1e3, flops / pk["bf16_tflops"] / 1e6)
-        emit({"kernel": kernel, "role": role, "us": round(us, 2), "gbs": round(bytes_ / us / 1e3) if bytes_ else None,
-              "tflops": round(flops / us / 1e6, 1) if flops else None, f"fraction_of_{pk['src']}_roofline": round(roof / us, 3)})
-
-    for size, s in SIZES.items():
+    t = _Rows(dev, emit)
+    bf, i32, bufs, row = t.bf, t.i32, t.bufs, t.row
+    for size, s in SIZES["tikarax"].items():
         H, W, F, nq, nkv, d = s["hidden"], s["width"], s["ffn"], s["heads"], s["kv_heads"], s["dim"]
         for T in (1, 32, PREFILL):
             # ---- norms: both sides of a sublayer in one pass, against residual add + norm
@@ -206,7 +234,135 @@ def bench_kernels(dev, emit) -> None:
     K.check_status()
 
 
-def main(part: str = "all") -> int:
+def bench_kernels_pubodra(dev, emit) -> None:
+    from ..ops import cuda as K
+    from ..ops import ref
+    from ..ops.weights import QuantWeight, WFormat
+    from ..utils.rope import rope_tables
+    t = _Rows(dev, emit)
+    bf, i32, bufs, row = t.bf, t.i32, t.bufs, t.row
+    mats = lambda n, k, e=1, least=1: [QuantWeight(WFormat.BF16, n, k, e, (torch.randn(e, n, k, device=dev) * k ** -0.5).to(torch.bfloat16))
+                                       for _ in range(max(least, bufs(e * n * k * 2)))]
+    for size, s in SIZES["pubodra"].items():
+        H, F, nh, d, r, v, R, win = s["hidden"], s["ffn"], s["heads"], s["dim"], s["rot"], s["vdim"], s["rank"], s["window"]
+        E, top, ef = s["experts"], s["used"], s["eff"]
+        for T in (1, 32, PREFILL):
+            # ---- norms
+            nb = bufs(T * H * 12) if T > 64 else 8
+            xs, ds, w = [torch.randn(T, H, device=dev) for _ in range(nb)], [bf(T, H) for _ in range(nb)], torch.ones(H, device=dev)
+            by = T * H * (4 + 4 + 2 + 2)
+            row(f"dyt_norm (add + tanh) T={T} H={H}", "new", [lambda x=x, q=q: K.dyt_norm(x, 0.7, w, w, delta=q) for x, q in zip(xs, ds)], by)
+            row(f"rmsnorm (add + norm) T={T} H={H}", "like", [lambda x=x, q=q: K.rmsnorm(x, w, 1e-6, delta=q) for x, q in zip(xs, ds)], by)
+            # ---- ... that form the experts' weighted sum
+            ys, pos, cw = [bf(T * top, H) for _ in range(nb)], torch.randperm(T * top, device=dev).to(torch.int32), torch.rand(T, top, device=dev)
+            by = T * H * (4 + 4 + 2 + 2 * top)
+            comb = [K.CombineDelta(y, pos, cw) for y in ys]
+            row(f"dyt_norm + combine of {top} T={T} H={H}", "new", [lambda x=x, q=q: K.dyt_norm(x, 0.7, w, w, delta=q) for x, q in zip(xs, comb)], by)
+            row(f"rmsnorm_combine of {top} T={T} H={H}", "like", [lambda x=x, q=q: K.rmsnorm_combine(x, w, 1e-6, q) for x, q in zip(xs, comb)], by)
+            del xs, ds, ys, comb
+            # ---- up projections with their activations
+            h = bf(T, H)
+            ws = mats(F, H)
+            row(f"up + GELU T={T} {F}x{H}", "new", [lambda m=m: K.linear(h, m, act=ref.ACT_GELU_TANH) for m in ws], F * H * 2 + T * (H + F) * 2, 2.0 * T * F * H)
+            N = F // 3 * 4 // 32 * 32
+            ws = mats(N, H)
+            row(f"gate|up + SwiGLU T={T} {N}x{H}", "like", [lambda m=m: K.linear(h, m, act=ref.ACT_SWIGLU) for m in ws], N * H * 2 + T * (H + N // 2) * 2, 2.0 * T * N * H)
+            del ws
+            # ---- experts
+            idx = torch.stack([torch.randperm(E, device=dev)[:top] for _ in range(T)]).to(torch.int32)
+            live = len(set(idx.reshape(-1).tolist()))
+            gf = ef * 2 // 3
+            for name, role, n_up, k_dn, act in (("relu^2", "new", ef, ef, ref.ACT_RELU2), ("SwiGLU", "like", 2 * gf, gf, ref.ACT_SWIGLU)):
+                ups, dns = mats(n_up, H, E), mats(H, k_dn, E)
+                if T <= 8:
+                    se = idx.reshape(-1)
+                    a = bf(T * top, k_dn)
+                    row(f"expert up + {name} T={T} {E}x{n_up}x{H}", role, [lambda m=m: K.expert_gemv(h, m, se, x_div=top, act=act) for m in ups], live * n_up * H * 2)
+                    row(f"expert down T={T} {E}x{H}x{k_dn}", role, [lambda m=m: K.expert_gemv(a, m, se) for m in dns], live * k_dn * H * 2)
+                else:
+                    pk = K.moe_pack(idx, E)
+                    xp, a = K.moe_gather(h, pk), bf(pk.max_rows, k_dn)
+                    row(f"expert up + {name} T={T} {E}x{n_up}x{H}", role, [lambda m=m: K.grouped_linear(xp, m, pk.tile_expert, pk.num_tiles, act=act) for m in ups],
+                        live * n_up * H * 2 + T * top * (H + k_dn) * 2, 2.0 * T * top * n_up * H)
+                    row(f"expert down T={T} {E}x{H}x{k_dn}", role, [lambda m=m: K.grouped_linear(a, m, pk.tile_expert, pk.num_tiles) for m in dns],
+                        live * k_dn * H * 2 + T * top * (H + k_dn) * 2, 2.0 * T * top * k_dn * H)
+                del ups, dns
+            # ---- head epilogue
+            cos, sin = rope_tables(2 * PREFILL, r, 1e4, device=dev)
+            cosl, sinl = rope_tables(2 * PREFILL, 128, 1e4, device=dev)
+            pages = T // 128 + 2
+            slots, pos = torch.arange(128, 128 + T, dtype=torch.int64, device=dev), torch.arange(T, dtype=torch.int32, device=dev)
+            cache = torch.zeros(pages, 1, 128, R + r, dtype=torch.bfloat16, device=dev)
+            nw, cq, nkv = torch.ones(R, device=dev), nh * (d + r), nh // 4
+            yk = [bf(T, cq + R + r + nh * v) for _ in range(bufs(T * cq * 2) if T > 64 else 8)][:8]
+            row(f"latent_post T={T}", "new", [lambda y=y: K.latent_post(y[:, :cq].view(T, nh, d + r)[..., d:], y[:, cq:cq + R + r], nw, R, 1e-6, pos, cos, sin, slots,
+                cache, y[:, :cq].view(T, nh, d + r)[..., d:]) for y in yk], T * (nh * r * 4 + (R + r) * 4))
+            kc, vc = torch.zeros(pages, nkv, 128, 128, dtype=torch.bfloat16, device=dev), torch.zeros(pages, nkv, 128, 128, dtype=torch.bfloat16, device=dev)
+            yk = [bf(T, (nh + 2 * nkv) * 128) for _ in range(8)]
+            row(f"qkv_post T={T}", "like", [lambda y=y: K.qkv_post(y, None, None, None, pos, cosl, sinl, slots, kc, vc, nh, nkv, 128, 128) for y in yk],
+                T * (nh * 128 * 4 + nkv * 128 * 8))
+            del yk, kc, vc
+        # ---- per-head products of the latent space, against a plain projection of the same weight
+        for T in (1, 8, 32):
+            y, o, g = bf(T, nh, d + r), bf(T, nh, R), bf(T, nh * v)
+            qc = torch.empty(T, nh, R + r, dtype=torch.bfloat16, device=dev)
+            ab, vu, pl = mats(R, d, nh), mats(v, R, nh), mats(nh * R // 4, 4 * d)
+            row(f"queries into the latent space T={T} {nh}x{R}x{d}", "new", [lambda m=m: K.head_linear(y[..., :d], m, out=qc[..., :R]) for m in ab],
+                nh * R * d * 2 + T * nh * (d + R) * 2, 2.0 * T * nh * R * d)
+            row(f"latent outputs to values + gate T={T} {nh}x{v}x{R}", "new", [lambda m=m: K.head_linear(o, m, gate=g) for m in vu],
+                nh * R * v * 2 + T * nh * (2 * v + R) * 2, 2.0 * T * nh * R * v)
+            h = bf(T, 4 * d)
+            row(f"plain projection T={T} {nh * R // 4}x{4 * d}", "like", [lambda m=m: K.linear(h, m) for m in pl], nh * R * d * 2 + T * (4 * d + nh * R // 4) * 2, 2.0 * T * nh * R * d)
+            del ab, vu, pl
+        # ---- attention: decoding
+        nkv = nh // 4
+        for B, ctx, w_ in ((1, 8192, 0), (1, 2048, 0), (8, 2048, win), (32, 2048, win), (32, 8192, 0)):
+            nblk = (ctx + 127) // 128
+            pages = B * nblk + 1
+            keys = min(ctx, w_) if w_ else ctx
+            caches = [bf(pages, 1, 128, R + r) for _ in range(min(16, bufs(B * keys * (R + r) * 2)))]
+            bt = torch.arange(1, pages, dtype=torch.int32, device=dev).reshape(B, nblk)
+            sl, cu = i32([ctx] * B), i32(list(range(B + 1)))
+            q = bf(B, nh, R + r)
+            row(f"latent attention B={B} ctx={ctx} window={w_} {nh}x({R}+{r})", "new",
+                [lambda c=c: K.latent_attention(q, c, bt, sl, cu, 1, R, window=w_, scale=0.07) for c in caches],
+                B * keys * (R + r) * 2 + B * nh * (2 * R + r) * 2, 2.0 * B * keys * nh * (2 * R + r))
+            del caches
+            kv = [(bf(pages, nkv, 128, 128), bf(pages, nkv, 128, 128)) for _ in range(min(16, bufs(B * keys * nkv * 512)))]
+            q = bf(B, nh, 128)
+            row(f"attention B={B} ctx={ctx} window={w_} {nh}/{nkv}x128", "like", [lambda k=k, x=x: K.attention(q, k, x, bt, sl, cu, 1, window=w_, scale=0.09) for k, x in kv],
+                B * keys * nkv * 512 + B * nh * 512, 4.0 * B * keys * nh * 128)
+            del kv
+            torch.cuda.empty_cache()
+        # ---- attention: prompts
+        for n, ctx in ((PREFILL, PREFILL), (512, PREFILL)):
+            nblk = ctx // 128
+            bt, sl, cu = torch.arange(1, nblk + 1, dtype=torch.int32, device=dev).reshape(1, nblk), i32([ctx]), i32([0, n])
+            first = max(0, ctx - n - win + 1)
+            pairs = float(sum(min(p + 1, win) for p in range(ctx - n, ctx)))
+            q, g, out = bf(n, nh, d + r), bf(n, nh * v), torch.empty(n, nh, v, dtype=torch.bfloat16, device=dev)
+            caches, wk = [bf(nblk + 1, 1, 128, R + r) for _ in range(4)], mats(nh * (d + v), R)
+            rows_ = ctx - first // 128 * 128
+            fl_up, fl_at = 2.0 * rows_ * R * nh * (d + v), 2.0 * pairs * nh * (d + r + v)
+            plan = K._latent_plan(None, bt, sl, cu, n, win, 128)
+            kvb = torch.empty(plan[0].numel() * 128, nh * (d + v), dtype=torch.bfloat16, device=dev)
+            row(f"keys and values of {rows_} rows {nh * (d + v)}x{R}", "new",
+                [lambda m=m, c=c: K.gemm_paged(c, plan, m, kvb) for m, c in zip(wk, caches * 8)], rows_ * (R + nh * (d + v)) * 2 + R * nh * (d + v) * 2, fl_up)
+            hp, pm = bf(rows_, R), mats(nh * (d + v), R)
+            row(f"plain projection T={rows_} {nh * (d + v)}x{R}", "like", [lambda m=m: K.linear(hp, m) for m in pm], rows_ * (R + nh * (d + v)) * 2 + R * nh * (d + v) * 2, fl_up)
+            row(f"expanded attention n={n} ctx={ctx} window={win} {nh}x({d}+{r}/{v}) + gate, without forming keys", "new",
+                [lambda c=c: K.expanded_attention(q, kvb, plan, c, bt, sl, cu, n, d, v, R, win, 0.07, g, out) for c in caches],
+                rows_ * nh * (d + v) * 2 + n * nh * (d + r + 2 * v) * 2, fl_at)
+            kc, vc = bf(nblk + 1, nkv, 128, 128), bf(nblk + 1, nkv, 128, 128)
+            q1 = bf(n, nh, 128)
+            row(f"attention n={n} ctx={ctx} window={win} {nh}/{nkv}x128", "like", [lambda: K.attention(q1, kc, vc, bt, sl, cu, n, window=win, scale=0.09)],
+                rows_ * nkv * 512 + n * nh * 512, 4.0 * pairs * nh * 128)
+            del caches, wk, kvb, kc, vc, pm
+            torch.cuda.empty_cache()
+    K.check_status()
+
+
+def main(design: str, part: str = "all") -> int:
     dev = torch.device("cuda:0")
     torch.cuda.set_device(dev)
     t0 = time.time()
@@ -215,8 +371,8 @@ def main(part: str = "all") -> int:
         print(json.dumps(obj))
         sys.stdout.flush()
     if part in ("all", "models"):
-        bench_models(dev, emit)
+        bench_models(design, dev, emit)
     if part in ("all", "kernels"):
-        bench_kernels(dev, emit)
+        {"tikarax": bench_kernels_tikarax, "pubodra": bench_kernels_pubodra}[design](dev, emit)
     emit({"design_bench": "done", "seconds": round(time.time() - t0, 1)})
     return 0

@@ -383,11 +383,15 @@ __global__ void __launch_bounds__(128) attn_combine_kernel(const float* __restri
 constexpr int ATT_TICKET_SLOTS = 8, ATT_TICKETS_PER_SLOT = 2048;
 static __device__ int g_attn_tickets[ATT_TICKET_SLOTS * ATT_TICKETS_PER_SLOT];
 
+constexpr size_t ATT_SMEM_MAX = 226 * 1024;           // (the kernel also has a few static bytes)
+static size_t att_smem(const AttnParams& p, int ppw, int elem, int kpad) {
+  return (size_t)ATT_WARPS * ppw * p.dk * 4 + (size_t)ATT_TILE * (p.dk + kpad) * elem + (p.v_cache ? (size_t)ATT_TILE * p.dv * elem : 0);
+}
+
 template <typename T, int HD, int PPW, bool EXACT>
 static int launch_partial(const AttnParams& p, cudaStream_t st) {
-  constexpr int PAIRS = ATT_WARPS * PPW;
-  constexpr size_t SMEM_MAX = 226 * 1024;             // (the kernel also has a few static bytes)
-  const size_t smem = (size_t)PAIRS * p.dk * 4 + (size_t)ATT_TILE * (p.dk + att_kpad<T>()) * sizeof(T) + (p.v_cache ? (size_t)ATT_TILE * p.dv * sizeof(T) : 0);
+  constexpr size_t SMEM_MAX = ATT_SMEM_MAX;
+  const size_t smem = att_smem(p, PPW, sizeof(T), att_kpad<T>());
   if (smem > SMEM_MAX) return -112;
   auto kern = attn_partial_kernel<T, HD, PPW, EXACT>;
   static DeviceOnce configured;
@@ -406,8 +410,9 @@ static int launch_partial(const AttnParams& p, cudaStream_t st) {
 using namespace mx;
 
 // pairs per warp (1 for decode-sized work, 4 when there are many query tokens), query tokens per CTA, query tiles per sequence
-static void att_tiling(int max_q_len, int gqa, int& ppw, int& q_tile, int& max_q_tiles) {
+static void att_tiling(int max_q_len, int gqa, int& ppw, int& q_tile, int& max_q_tiles, int max_ppw = 4) {
   ppw = (max_q_len * gqa > ATT_WARPS * 2) ? 4 : (max_q_len * gqa > ATT_WARPS ? 2 : 1);
+  if (ppw > max_ppw) ppw = max_ppw;
   const int pairs = ATT_WARPS * ppw;
   q_tile = pairs / gqa > 0 ? pairs / gqa : 1;
   if (q_tile > max_q_len) q_tile = max_q_len;
@@ -447,7 +452,9 @@ static int attention_impl(const void* q, const void* k_cache, const void* v_cach
   p.B = B; p.n_q = n_q; p.n_kv = n_kv; p.max_blocks = max_blocks; p.block_size = block_size;
   p.n_splits = n_splits < 1 ? 1 : n_splits; p.Tq = Tq; p.window = window; p.scale = scale; p.softcap = softcap;
   int ppw;
-  att_tiling(max_q_len, gqa, ppw, p.q_tile, p.max_q_tiles);
+  int max_ppw = 4;                                    // wide rows: fewer queries at a time, so that they fit beside the key tile
+  while (max_ppw > 1 && att_smem(p, max_ppw, sh.elem_f32 ? 4 : 2, 2) > ATT_SMEM_MAX) max_ppw /= 2;
+  att_tiling(max_q_len, gqa, ppw, p.q_tile, p.max_q_tiles, max_ppw);
   p.tickets = nullptr; p.sinks = sinks; p.out = out;
   const long long groups = (long long)B * p.max_q_tiles * n_kv;
   if (groups <= ATT_TICKETS_PER_SLOT) {

@@ -335,7 +335,8 @@ class LatentAttentionBlock:
     Long queries form the keys and values of the pages in reach once per step and run on the prefill kernel, which costs a head (dim + rot_dim +
     vdim) products per key and query where the latent space costs 2 rank + rot_dim.  Widths are padded to multiples of 8 at load."""
 
-    EXPAND_MIN_Q = 64            # query segments at least this long take per-head keys and values
+    EXPAND_MIN_Q = 64            # query segments at least this long take per-head keys and values ...
+    EXPAND_MAX = (192, 64, 256)  # ... when the widths (unrotated, rotated, value) fit that kernel; otherwise all stay in the latent space
     MAX_RANK = 512               # what the latent kernel's accumulators hold
 
     def __init__(self, src, prefix: str, hidden: int, row: int, heads: int, dim: int, rot_dim: int, vdim: int, rank: int, scale: float, window: int,
@@ -345,6 +346,7 @@ class LatentAttentionBlock:
         H, K = heads, hidden
         self.n_q, self.n_kv, self.scale, self.window, self.eps, self.rank, self.rope = H, 1, scale, window, eps, rank, rope
         self.d, self.r, self.v, self.R = (round_up(n, 8) for n in (dim, rot_dim, vdim, rank))
+        self.can_expand = all(n <= m for n, m in zip((self.d, self.r, self.v), self.EXPAND_MAX))
 
         def padded(w: QuantWeight, parts, sizes, row_to):
             """Rows of every group are ``parts`` runs; each run is padded to its size, the columns to ``row_to``."""
@@ -378,7 +380,7 @@ class LatentAttentionBlock:
         T, H, d, R = y.shape[0], self.n_q, self.d, self.R
         q, ckv, gate = y[:, :self.cols[0]].view(T, H, d + self.r), y[:, self.cols[0]:self.cols[1]], y[:, self.cols[1]:]
         a = torch.empty(T, H, self.v, dtype=y.dtype, device=y.device)
-        expand = not (y.is_cuda and y.dtype == torch.float32)          # 32-bit kernels: latent space only
+        expand = self.can_expand and not (y.is_cuda and y.dtype == torch.float32)          # (32-bit kernels: latent space only)
         for lo, hi, table, lens, cu, longest in fb.query_parts(apart=expand):
             latent = longest < self.EXPAND_MIN_Q or not expand
             rows = slice(lo, hi)

@@ -723,16 +723,30 @@ def latent_attention_expanded(q, w_kv: QuantWeight, cache, block_table, seq_lens
     if out is None:
         out = torch.empty(Tq, H, vdim, dtype=q.dtype, device=q.device)
     assert out.is_contiguous() and out.shape == (Tq, H, vdim)
-    pages, num, table = _latent_plan(plans, block_table, seq_lens, cu_q, Tq, window, bs)
-    n = pages.numel()
-    kv = torch.empty(n * bs, w_kv.N, dtype=torch.bfloat16, device=q.device)
-    lib = _lib.cuda()
-    _check(lib.mx_gemm_paged(_p(cache), width, C.c_longlong(cache.shape[0] * bs), _p(pages), _p(num), _p(w_kv.p0), _p(kv), n, w_kv.N, rank,
-                             _pick_bn(n * bs, w_kv.N), _stream()), "gemm_paged")
-    _check(lib.mx_attention_prefill_latent(_p(q), _q_rows(q), _p(kv), n, _p(table), _p(cache), cache.shape[0], _p(block_table), block_table.shape[1],
-                                           _p(seq_lens), _p(cu_q), _p(gate), 0 if gate is None else gate.stride(0), _p(out), seq_lens.numel(), Tq,
-                                           int(max_q_len), H, dim, dq - dim, vdim, rank, int(window), C.c_float(scale), _stream()), "attention_prefill_latent")
-    _count(2)
+    plan = _latent_plan(plans, block_table, seq_lens, cu_q, Tq, window, bs)
+    kv = torch.empty(plan[0].numel() * bs, w_kv.N, dtype=torch.bfloat16, device=q.device)
+    gemm_paged(cache, plan, w_kv, kv)
+    return expanded_attention(q, kv, plan, cache, block_table, seq_lens, cu_q, max_q_len, dim, vdim, rank, window, scale, gate, out)
+
+
+def gemm_paged(cache, plan, w: QuantWeight, out) -> None:
+    """Rows of ``plan``'s pages of a latent cache (their first ``w.K`` elements) times ``w``, page after page into ``out``."""
+    pages, num, _ = plan
+    bs, width = cache.shape[2], cache.shape[3]
+    _check(_lib.cuda().mx_gemm_paged(_p(cache), width, C.c_longlong(cache.shape[0] * bs), _p(pages), _p(num), _p(w.p0), _p(out), pages.numel(), w.N, w.K,
+                                     _pick_bn(pages.numel() * bs, w.N), _stream()), "gemm_paged")
+    _count()
+
+
+def expanded_attention(q, kv, plan, cache, block_table, seq_lens, cu_q, max_q_len, dim, vdim, rank, window, scale, gate, out):
+    """The attention of :func:`latent_attention_expanded` over keys and values ``kv`` that :func:`gemm_paged` has formed."""
+    pages, _, table = plan
+    Tq, H, dq = q.shape
+    _check(_lib.cuda().mx_attention_prefill_latent(_p(q), _q_rows(q), _p(kv), pages.numel(), _p(table), _p(cache), cache.shape[0], _p(block_table),
+                                                   block_table.shape[1], _p(seq_lens), _p(cu_q), _p(gate), 0 if gate is None else gate.stride(0), _p(out),
+                                                   seq_lens.numel(), Tq, int(max_q_len), H, dim, dq - dim, vdim, rank, int(window), C.c_float(scale), _stream()),
+           "attention_prefill_latent")
+    _count()
     return out
 
 

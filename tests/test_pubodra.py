@@ -18,6 +18,8 @@ CONFIGS = {
                                   vocab=131, width=84, eps=1e-3, loop=(1, 3, 2)),
     "no-loop": oracle.random_config([L(4, 32, 16, 48, 64, 128, 64, scaling=YARN), L(2, 64, 64, 64, 128, 200, (4, 4, 64))], vocab=64, width=64),
     "all-looped": oracle.random_config([L(2, 16, 8, 16, 24, 33, (5, 1, 24)), L(3, 8, 4, 20, 16, 64, 50)], vocab=90, width=50, loop=(0, 2, 3)),
+    # widths that the expanded form does not take
+    "latent-space-only": oracle.random_config([L(2, 200, 72, 264, 40, 60, 64), L(1, 24, 8, 16, 24, 100, 40)], vocab=60, width=64),
     "one-pass-loop-at-the-end": oracle.random_config([L(2, 24, 8, 32, 48, 1, 40), L(1, 100, 12, 72, 88, 140, 96)], vocab=70, width=96, loop=(1, 2, 1)),
 }
 _cache = {}

@@ -199,7 +199,7 @@ def latent_space_oracle(q, rows, lens, q_lens, rank, scale, window):
     return np.concatenate(outs)
 
 
-SHAPES = [(1, 8, 8), (5, 40, 8), (8, 64, 16), (3, 192, 72), (16, 512, 64), (40, 256, 32), (64, 128, 64), (7, 136, 24)]
+SHAPES = [(4, 512, 128), (1, 8, 8), (5, 40, 8), (8, 64, 16), (3, 192, 72), (16, 512, 64), (40, 256, 32), (64, 128, 64), (7, 136, 24)]
 BATCHES = [([1, 130, 300, 257], [1, 1, 1, 1]), ([9, 129, 260], [9, 2, 37]), ([1], [1]), ([40, 400], [40, 1])]
 
 
@@ -250,7 +250,7 @@ def test_latent_attention_scores_that_grow():
         assert rel(got, latent_space_oracle(f64(q), rows, [L], [1], rank, 1.0, 0)) < 1e-2
 
 
-EXPANDED = [(3, 24, 8, 40, 40), (2, 64, 16, 64, 64), (4, 40, 64, 128, 192), (2, 56, 8, 200, 24), (3, 100, 16, 56, 72), (2, 128, 64, 128, 512), (1, 96, 24, 232, 136),
+EXPANDED = [(3, 24, 8, 40, 40), (2, 64, 16, 64, 64), (4, 40, 64, 128, 192), (2, 56, 8, 200, 24), (3, 104, 16, 56, 72), (2, 128, 64, 128, 512), (1, 96, 24, 232, 136),
             (2, 160, 32, 48, 64), (2, 192, 64, 128, 128), (1, 136, 8, 256, 40)]
 
 
