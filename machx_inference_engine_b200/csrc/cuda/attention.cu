@@ -346,35 +346,54 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
   }
 }
 
-// out[t][h][:] = sum_s acc_s e^{m_s - M} / (sum_s l_s e^{m_s - M} + e^{sink_h - M}) [* sigmoid(gate)]
+// out[t][h][:] = sum_s acc_s e^{m_s - M} / (sum_s l_s e^{m_s - M} + e^{sink_h - M}) [* sigmoid(gate)].  blockIdx: (row, run of 256 columns);
+// every warp forms the weights of the splits, a lane per split, and a thread sums two columns over them.
+constexpr int CMB_COLS = 256;
 template <typename T>
-__global__ void __launch_bounds__(128) attn_combine_kernel(const float* __restrict__ o_part, const float* __restrict__ ml_part,
-                                                           const float* __restrict__ sinks, const T* __restrict__ gate, int gate_ld, T* __restrict__ out,
-                                                           int Tq, int n_q, int hd, int n_splits) {
+__global__ void __launch_bounds__(CMB_COLS / 2) attn_combine_kernel(const float* __restrict__ o_part, const float* __restrict__ ml_part,
+                                                                    const float* __restrict__ sinks, const T* __restrict__ gate, int gate_ld,
+                                                                    T* __restrict__ out, int Tq, int n_q, int hd, int n_splits) {
   constexpr bool PRECISE = sizeof(T) == 4;
   pdl_prologue();
-  const int r = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (r >= Tq * n_q) return;
-  const int h = r % n_q;
+  const int r = blockIdx.x, lane = threadIdx.x & 31, h = r % n_q;
+  const int d = blockIdx.y * CMB_COLS + threadIdx.x * 2;
+  const size_t rows = (size_t)Tq * n_q;
+  const float2* ml = reinterpret_cast<const float2*>(ml_part);
   float M = sinks ? sinks[h] : -1e30f;
-  for (int s = 0; s < n_splits; ++s) M = fmaxf(M, ml_part[((size_t)s * Tq * n_q + r) * 2]);
-  float L = sinks ? att_exp<PRECISE>(sinks[h] - M) : 0.f;
-  for (int s = 0; s < n_splits; ++s) {
-    const float* ml = ml_part + ((size_t)s * Tq * n_q + r) * 2;
-    L += ml[1] * att_exp<PRECISE>(ml[0] - M);
-  }
-  const float inv = L > 0.f ? 1.f / L : 0.f;
-  for (int d = lane; d < hd; d += 32) {
-    float a = 0.f;
-    for (int s = 0; s < n_splits; ++s) {
-      const size_t row = (size_t)s * Tq * n_q + r;
-      const float wt = att_exp<PRECISE>(ml_part[row * 2] - M);
-      if (wt != 0.f) a += o_part[row * hd + d] * wt;                   // (a split without keys leaves its rows unwritten)
+  for (int s = lane; s < n_splits; s += 32) M = fmaxf(M, ml[s * rows + r].x);
+  M = warp_max(M);
+  float L = 0.f;
+  float a0 = 0.f, a1 = 0.f;
+  for (int s0 = 0; s0 < n_splits; s0 += 32) {
+    float w = 0.f;
+    if (s0 + lane < n_splits) {
+      const float2 v = ml[(s0 + lane) * rows + r];
+      w = att_exp<PRECISE>(v.x - M);
+      L = fmaf(v.y, w, L);
     }
-    a *= inv;
-    if (gate) a *= sigmoid_f<PRECISE>(to_f32(gate[(size_t)(r / n_q) * gate_ld + (size_t)h * hd + d]));
-    out[(size_t)r * hd + d] = from_f32<T>(a);
+    const int cnt = min(32, n_splits - s0);
+    const float* op = o_part + ((size_t)s0 * rows + r) * hd + d;
+#pragma unroll 8
+    for (int j = 0; j < cnt; ++j) {
+      const float wj = __shfl_sync(0xffffffffu, w, j);
+      if (wj != 0.f && d < hd) {                                       // (a split without keys leaves its rows unwritten)
+        const float2 v = *reinterpret_cast<const float2*>(op + (size_t)j * rows * hd);
+        a0 = fmaf(v.x, wj, a0);
+        a1 = fmaf(v.y, wj, a1);
+      }
+    }
   }
+  L = warp_sum(L) + (sinks ? att_exp<PRECISE>(sinks[h] - M) : 0.f);
+  if (d >= hd) return;
+  const float inv = L > 0.f ? 1.f / L : 0.f;
+  a0 *= inv;
+  a1 *= inv;
+  if (gate) {
+    const float2 g = load2(gate + (size_t)(r / n_q) * gate_ld + (size_t)h * hd + d);
+    a0 *= sigmoid_f<PRECISE>(g.x);
+    a1 *= sigmoid_f<PRECISE>(g.y);
+  }
+  store2(out + (size_t)r * hd + d, a0, a1);
 }
 
 // Tickets of the fused merge: zero at load, and every launch leaves its counters at zero again.  Consecutive launches rotate
@@ -492,11 +511,11 @@ static int attention_impl(const void* q, const void* k_cache, const void* v_cach
   }
 #undef MX_ATT
   if (rc || p.tickets) return rc;
-  const dim3 cgrid((Tq * n_q + 3) / 4);
+  const dim3 cgrid(Tq * n_q, (dv + CMB_COLS - 1) / CMB_COLS);
   if (sh.elem_f32)
-    launch_pdl(attn_combine_kernel<float>, cgrid, dim3(128), 0, st, o_part, ml_part, sinks, (const float*)sh.gate, sh.gate_ld, (float*)out, Tq, n_q, dv, p.n_splits);
+    launch_pdl(attn_combine_kernel<float>, cgrid, dim3(CMB_COLS / 2), 0, st, o_part, ml_part, sinks, (const float*)sh.gate, sh.gate_ld, (float*)out, Tq, n_q, dv, p.n_splits);
   else
-    launch_pdl(attn_combine_kernel<__nv_bfloat16>, cgrid, dim3(128), 0, st, o_part, ml_part, sinks, (const __nv_bfloat16*)sh.gate, sh.gate_ld,
+    launch_pdl(attn_combine_kernel<__nv_bfloat16>, cgrid, dim3(CMB_COLS / 2), 0, st, o_part, ml_part, sinks, (const __nv_bfloat16*)sh.gate, sh.gate_ld,
                (__nv_bfloat16*)out, Tq, n_q, dv, p.n_splits);
   return (int)cudaGetLastError();
 }
@@ -506,7 +525,7 @@ MX_HOST_API int mx_attention_combine(const float* o_part, const float* ml_part, 
   if (Tq <= 0) return 0;
   const float* no_sinks = nullptr;
   const __nv_bfloat16* no_gate = nullptr;
-  launch_pdl(attn_combine_kernel<__nv_bfloat16>, dim3((Tq * n_q + 3) / 4), dim3(128), 0, st, o_part, ml_part, no_sinks, no_gate, 0, (__nv_bfloat16*)out, Tq, n_q, dv,
+  launch_pdl(attn_combine_kernel<__nv_bfloat16>, dim3(Tq * n_q, (dv + CMB_COLS - 1) / CMB_COLS), dim3(CMB_COLS / 2), 0, st, o_part, ml_part, no_sinks, no_gate, 0, (__nv_bfloat16*)out, Tq, n_q, dv,
              n_splits);
   return (int)cudaGetLastError();
 }

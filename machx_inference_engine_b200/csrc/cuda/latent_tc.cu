@@ -6,9 +6,9 @@
 //   S^T [128 keys][NR]      = tile [128][rank + rot]  Q^T            (K-major operands)
 //   O^T [rank][NR]         += tile[:, :rank]^T [rank][128]  P^T      (the tile read MN-major: no transpose is made)
 // so that 16 or 32 heads cost no padding to 128 rows, and the accumulator of a 512-wide latent takes 4 x NR TMEM columns.
-//   warp 0  : TMA.  The rotated part of a tile goes to a ring of its own and is free again after S^T; the latent part travels in pairs of
+//   warp 0  : TMA, with the next tile on its way into L2 while this one is loaded.  The rotated part of a tile goes to a ring of its own and is free again after S^T; the latent part travels in pairs of
 //             64-column atoms (128 latent rows of O^T) through a ring whose slots are held until their O^T product is done
-//   warp 1  : tcgen05.mma.  With room for two tiles S^T of the next tile runs ahead of O^T of this one
+//   warp 1  : tcgen05.mma.  As much of the next tile's S^T as there is room for runs ahead of O^T of this tile
 //   warps 2-5: one thread per key (TMEM lane).  Scores -> mask -> maximum over the keys by a transposing butterfly (lane n of every warp ends up
 //             with row n), exchanged over the four warps; P is formed against a reference maximum that moves only when a row has grown by 2^8
 //             (then O^T is rescaled in place) and stored as bf16 into the swizzled operand tile; denominators stay per thread until the end
@@ -91,6 +91,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap_qc, const __grid_con
   constexpr int G = NR / 32;                     // groups of 32 query rows
   constexpr int QATOM = NR * 128;                // bytes of a 64-column atom of the query rows
   constexpr float RESCALE_STEP = 8.f;
+  pdl_launch_dependents();
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   const uint32_t sbase = smem_u32(smem);
@@ -116,6 +117,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap_qc, const __grid_con
   const int tile_lo = all_lo + split * per, n_tiles = min(per, all_lo + all_n - tile_lo);
   const long long out_row0 = (long long)q_begin * p.heads + r0;
   if (n_tiles <= 0) {                            // (only with several ranges)
+    pdl_wait();
     if (p.o_part && threadIdx.x < rows) {
       float* ml = p.ml_part + ((long long)split * p.rows_all + out_row0 + threadIdx.x) * 2;
       ml[0] = -1e30f; ml[1] = 0.f;
@@ -142,6 +144,7 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap_qc, const __grid_con
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = tmem_slot, tmem_o = tmem_base + 2 * NR;
+  pdl_wait();                                    // queries and the newest cache rows come from the kernels before
 
   if (warp == 0) {
     if (lane == 0) {
@@ -153,6 +156,11 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap_qc, const __grid_con
       int it = 0;
       for (int j = 0; j < n_tiles && ok; ++j) {
         const int blk = p.block_table[(size_t)b * p.max_blocks + tile_lo + j];
+        if (j + 1 < n_tiles) {
+          const int nb = p.block_table[(size_t)b * p.max_blocks + tile_lo + j + 1];
+          for (int a = 0; a < ratoms; ++a) tma_prefetch_3d(&tmap_r, a * 64, 0, nb);
+          for (int a = 0; a < catoms; ++a) tma_prefetch_3d(&tmap_c, a * 64, 0, nb);
+        }
         const int rs = j % rslots, rph = (j / rslots) & 1;
         if (!(ok = mbar_wait(b_rempty + 8 * rs, rph ^ 1, p.status, ERR_MBAR_TIMEOUT_PRODUCER, abort_flag))) break;
         mbar_expect_tx(b_rfull + 8 * rs, ratoms * LA_ATOM);
@@ -170,44 +178,55 @@ latent_attn_kernel(const __grid_constant__ CUtensorMap tmap_qc, const __grid_con
       constexpr uint32_t idesc_s = umma_idesc_bf16(128, NR, 0, 0);
       constexpr uint32_t idesc_o = umma_idesc_bf16(128, NR, 1, 0);       // A = tile^T is MN-major (latent columns contiguous)
       bool ok = mbar_wait(b_qfull, 0, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag);
-      auto issue_s = [&](int j) -> bool {
-        const int rs = j % rslots, rph = (j / rslots) & 1, sb = j & 1, sph = (j >> 1) & 1;
-        if (!mbar_wait(b_sempty + 8 * sb, sph ^ 1, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag)) return false;
-        if (!mbar_wait(b_rfull + 8 * rs, rph, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag)) return false;
-        tc_fence_after();
-        const uint32_t d = tmem_base + sb * NR;
-        auto atom = [&](uint32_t tile, uint32_t q, bool first) {
+      // descriptors differ in their address field only (16-byte units): the constant part is formed once
+      const uint64_t dk = umma_desc_k_sw128(0), dm = umma_desc_mn_sw128(0, LA_ATOM, 1024);
+      const uint64_t q0 = dk + ((sbase + p.q_off) >> 4), p0 = dk + ((sbase + p.p_off) >> 4), r_0 = dk + ((sbase + p.r_off) >> 4);
+      const uint64_t ck0 = dk + ((sbase + p.c_off) >> 4), cm0 = dm + ((sbase + p.c_off) >> 4);
+      constexpr int A16 = LA_ATOM >> 4, Q16 = QATOM >> 4;
+      auto atom = [&](uint32_t d, uint64_t tile, uint64_t q, bool acc) {
+        umma_bf16(d, tile, q, idesc_s, acc);
 #pragma unroll
-          for (int kk = 0; kk < 4; ++kk)
-            umma_bf16(d, umma_desc_k_sw128(tile + kk * 32), umma_desc_k_sw128(q + kk * 32), idesc_s, !(first && kk == 0));
-        };
-        for (int a = 0; a < ratoms; ++a) atom(sbase + p.r_off + (rs * ratoms + a) * LA_ATOM, sbase + p.q_off + (catoms + a) * QATOM, a == 0);
-        umma_commit(b_rempty + 8 * rs);
-        for (int c = 0; c < cpairs; ++c) {
-          const int it = j * cpairs + c, s = it % nslots, ph = (it / nslots) & 1, na = min(2, catoms - 2 * c);
+        for (int kk = 1; kk < 4; ++kk) umma_bf16(d, tile + 2 * kk, q + 2 * kk, idesc_s, 1);
+      };
+      // latent pairs [c_lo, c_hi) of S^T(j); the first call of a tile (c_lo == 0) brings the rotated part, the last one hands S^T over
+      auto issue_s = [&](int j, int c_lo, int c_hi) -> bool {
+        const int sb = j & 1;
+        const uint32_t d = tmem_base + sb * NR;
+        if (c_lo == 0) {
+          const int rs = j % rslots, rph = (j / rslots) & 1;
+          if (!mbar_wait(b_sempty + 8 * sb, ((j >> 1) & 1) ^ 1, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag)) return false;
+          if (!mbar_wait(b_rfull + 8 * rs, rph, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag)) return false;
+          tc_fence_after();
+          for (int a = 0; a < ratoms; ++a) atom(d, r_0 + (rs * ratoms + a) * A16, q0 + (catoms + a) * Q16, a != 0);
+          umma_commit(b_rempty + 8 * rs);
+        }
+        for (int c = c_lo; c < c_hi; ++c) {
+          const int it = j * cpairs + c, s = it % nslots, ph = (it / nslots) & 1;
           if (!mbar_wait(b_cfull + 8 * s, ph, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag)) return false;
           tc_fence_after();
-          for (int a = 0; a < na; ++a) atom(sbase + p.c_off + (2 * s + a) * LA_ATOM, sbase + p.q_off + (2 * c + a) * QATOM, false);
+          atom(d, ck0 + 2 * s * A16, q0 + 2 * c * Q16, true);
+          if (2 * c + 1 < catoms) atom(d, ck0 + (2 * s + 1) * A16, q0 + (2 * c + 1) * Q16, true);
         }
-        umma_commit(b_sfull + 8 * sb);
+        if (c_hi == cpairs) umma_commit(b_sfull + 8 * sb);
         return true;
       };
-      const bool ahead = nslots >= 2 * cpairs;       // otherwise the next tile's last atoms wait for this tile's slots
-      if (ok) ok = issue_s(0);
+      const int early = min(cpairs, nslots - cpairs);      // pairs of the next tile that fit beside this tile
+      if (ok) ok = issue_s(0, 0, cpairs);
       for (int j = 0; j < n_tiles && ok; ++j) {
-        if (ahead && j + 1 < n_tiles && !(ok = issue_s(j + 1))) break;
+        if (early > 0 && j + 1 < n_tiles && !(ok = issue_s(j + 1, 0, early))) break;
         if (!(ok = mbar_wait(b_pfull, j & 1, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag))) break;
         tc_fence_after();
         for (int c = 0; c < cpairs; ++c) {
           const int s = (j * cpairs + c) % nslots;
-          const uint32_t va = sbase + p.c_off + 2 * s * LA_ATOM, pa = sbase + p.p_off, d = tmem_o + c * NR;
+          const uint64_t va = cm0 + 2 * s * A16;
+          const uint32_t d = tmem_o + c * NR;
+          umma_bf16(d, va, p0, idesc_o, j != 0);
 #pragma unroll
-          for (int kk = 0; kk < LA_PAGE / 16; ++kk)
-            umma_bf16(d, umma_desc_mn_sw128(va + kk * 2048, LA_ATOM, 1024), umma_desc_k_sw128(pa + (kk >> 2) * QATOM + (kk & 3) * 32), idesc_o, (j | kk) != 0);
+          for (int kk = 1; kk < LA_PAGE / 16; ++kk) umma_bf16(d, va + kk * 128, p0 + (kk >> 2) * Q16 + (kk & 3) * 2, idesc_o, 1);
           umma_commit(b_cempty + 8 * s);
         }
         umma_commit(b_pvdone);
-        if (!ahead && j + 1 < n_tiles && !(ok = issue_s(j + 1))) break;
+        if (early < cpairs && j + 1 < n_tiles && !(ok = issue_s(j + 1, early, cpairs))) break;
       }
     }
   } else {
@@ -414,7 +433,7 @@ static int launch_latent(const void* q, const void* cache, LaParams& p, int smem
     if (e != cudaSuccess) return (int)e;
     configured.mark();
   }
-  kern<<<dim3(B * p.row_tiles, p.n_splits), 192, smem, st>>>(qc, qr, tc, tr, p);
+  launch_pdl(kern, dim3(B * p.row_tiles, p.n_splits), dim3(192), (size_t)smem, st, qc, qr, tc, tr, p);
   return (int)cudaGetLastError();
 }
 

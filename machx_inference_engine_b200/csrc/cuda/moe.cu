@@ -165,21 +165,22 @@ __device__ __forceinline__ uint32_t bf16x2_to_f16x2(uint32_t v) {
 __global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ x, const int* __restrict__ packed_token, const int* __restrict__ total_rows,
                                   __nv_bfloat16* __restrict__ xp, int H, int to_f16, int zero_pad) {
   pdl_prologue();
-  const int r = blockIdx.x;
-  if (r >= total_rows[1]) return;
-  const int t = packed_token[r];
-  uint4* dst = reinterpret_cast<uint4*>(xp + (size_t)r * H);
-  if (t < 0) {
-    // tile padding: unless asked, the row is left as it is.  The grouped GEMM's output row depends on its own input row only and
-    // nothing refers to padding rows afterwards, and at ten experts per token the padding is as many rows as the live ones.
-    if (!zero_pad) return;
-    for (int i = threadIdx.x; i < H / 8; i += blockDim.x) dst[i] = make_uint4(0, 0, 0, 0);
-  } else {
-    const uint4* src = reinterpret_cast<const uint4*>(x + (size_t)t * H);
-    for (int i = threadIdx.x; i < H / 8; i += blockDim.x) {
-      uint4 v = src[i];
-      if (to_f16) { v.x = bf16x2_to_f16x2(v.x); v.y = bf16x2_to_f16x2(v.y); v.z = bf16x2_to_f16x2(v.z); v.w = bf16x2_to_f16x2(v.w); }
-      dst[i] = v;
+  const int rows = total_rows[1];
+  for (int r = blockIdx.x; r < rows; r += gridDim.x) {
+    const int t = packed_token[r];
+    uint4* dst = reinterpret_cast<uint4*>(xp + (size_t)r * H);
+    if (t < 0) {
+      // tile padding: unless asked, the row is left as it is.  The grouped GEMM's output row depends on its own input row only and
+      // nothing refers to padding rows afterwards, and at ten experts per token the padding is as many rows as the live ones.
+      if (!zero_pad) continue;
+      for (int i = threadIdx.x; i < H / 8; i += blockDim.x) dst[i] = make_uint4(0, 0, 0, 0);
+    } else {
+      const uint4* src = reinterpret_cast<const uint4*>(x + (size_t)t * H);
+      for (int i = threadIdx.x; i < H / 8; i += blockDim.x) {
+        uint4 v = src[i];
+        if (to_f16) { v.x = bf16x2_to_f16x2(v.x); v.y = bf16x2_to_f16x2(v.y); v.z = bf16x2_to_f16x2(v.z); v.w = bf16x2_to_f16x2(v.w); }
+        dst[i] = v;
+      }
     }
   }
 }
@@ -315,7 +316,8 @@ MX_HOST_API int mx_moe_gather(const void* x, const int* packed_token, const int*
                               int zero_pad, cudaStream_t st) {
   if (max_rows <= 0) return 0;
   if (H % 8) return -101;
-  launch_pdl(moe_gather_kernel, dim3(max_rows), dim3(128), 0, st, (const __nv_bfloat16*)x, packed_token, num_tiles, (__nv_bfloat16*)xp, H, to_f16,
+  const int ctas = 16 * sm_count();          // most of max_rows is room for padding: the live rows are walked
+  launch_pdl(moe_gather_kernel, dim3(max_rows < ctas ? max_rows : ctas), dim3(128), 0, st, (const __nv_bfloat16*)x, packed_token, num_tiles, (__nv_bfloat16*)xp, H, to_f16,
              zero_pad);
   return (int)cudaGetLastError();
 }

@@ -219,7 +219,8 @@ class SynthSource:
         return (0.02 * torch.randn(n, generator=g, device=self.gen_device)).to(self.device)
 
     def scalar(self, name: str) -> float:
-        return 0.7 + 0.05 * float(torch.randn((), generator=self._gen(name), device=self.gen_device))
+        # (tanh scale of a dynamic-tanh norm: large enough that embedding rows of this std, not the bias, decide the first layers)
+        return 0.16 / self.std * (1.0 + 0.05 * float(torch.randn((), generator=self._gen(name), device=self.gen_device)))
 
     def table(self, name: str, shape: tuple[int, ...]) -> torch.Tensor:
         g = self._gen(name)

@@ -483,6 +483,7 @@ class MoEFFN:
 
     MXF4_TENSOR_CORE = True      # class switch (tests compare against the bf16-activation path by turning it off)
     EXPERT_TP = False            # True: split every expert's FFN width over the ranks even when the expert count divides (tests)
+    PAIR_GEMV_MAX_TOKENS = 8     # up to this many tokens every (token, expert) pair streams its expert in a GEMV slot; more are packed
     MXF4_PAIR_MAX_TOKENS = 8     # up to this many tokens every (token, expert) pair is its own tile: no packing pass
     DOWN_KSPLIT = 3              # one-token decode: K ranges of the down projection (their partial rows are summed by the combine)
 
@@ -621,7 +622,7 @@ class MoEFFN:
             y = ops.expert_gemv(q8(a), self.down, slot_e, x_div=1, bias=self.down_bias, e_lo=self.e_lo)
             pk = ops.ref.MoePacking(None, None, None, torch.arange(T * self.K, dtype=torch.int32, device=h.device), None, None, T * self.K, self.K)
             out = ops.moe_combine(y, pk, w)
-        elif T <= 8 and h.dtype != torch.float32:
+        elif T <= self.PAIR_GEMV_MAX_TOKENS and h.dtype != torch.float32:
             # decode: one GEMV slot per (token, expert) pair, weights streamed once per pair; under expert
             # parallelism the slots of experts that live on other ranks contribute zero rows here
             slot_e = idx.reshape(-1)
@@ -672,6 +673,7 @@ class UnaryMoEFFN(MoEFFN):
     the softmax scores of the chosen ones, renormalised.  Routing, packing and execution are :class:`MoEFFN`'s; one GPU."""
 
     LAZY_COMBINE = True
+    PAIR_GEMV_MAX_TOKENS = 6     # 8 tokens, 6 of 64 experts of 2304 x 4096: slots 478 us, packed 301; 4 tokens: 174 against 198
 
     def __init__(self, src, prefix: str, hidden: int, row: int, experts: int, used: int, ffn: int, act: int):
         f = round_up(ffn, 32)

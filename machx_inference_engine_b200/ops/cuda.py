@@ -650,7 +650,8 @@ def latent_post(q_rot, ckv, norm_w, rank, eps, positions, rope_cos, rope_sin, sl
     _count()
 
 
-HEAD_GEMV_MAX_T = 8          # up to this many rows a head's matrix is streamed by the CUDA cores; more go to the tensor cores
+LATENT_MAX_SPLITS = 64
+HEAD_GEMV_MAX_T = 4          # up to this many rows a head's matrix is streamed by the CUDA cores; more go to the tensor cores
 
 
 def head_linear(x, w: QuantWeight, gate=None, out=None):
@@ -684,7 +685,7 @@ def latent_attention(q, cache, block_table, seq_lens, cu_q, max_q_len, rank, win
         pages = block_table.shape[1] if window <= 0 else min(block_table.shape[1], (window + max_q_len + bs - 3) // bs + 1)
         rows = max_q_len * H
         ctas = B * ((rows + 63) // 64 if rows > 32 else 1)
-        n_splits = max(1, min(pages, ATTN_MAX_SPLITS, sm_count() // ctas))
+        n_splits = max(1, min(pages, LATENT_MAX_SPLITS, sm_count() // ctas))
     part = torch.empty(n_splits * Tq * H * (rank + 2), dtype=torch.float32, device=q.device) if n_splits > 1 else None
     ml = part[n_splits * Tq * H * rank:] if part is not None else None
     _check(_lib.cuda().mx_latent_attention(_p(q), _p(cache), cache.shape[0], _p(block_table), block_table.shape[1], _p(seq_lens), _p(cu_q), _p(out), _p(part),
