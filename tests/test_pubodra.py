@@ -5,10 +5,11 @@ import pytest
 import torch
 
 import pubodra_oracle as oracle
-from design_util import ARMS, TOL, engine, logit_error, run_portions, tokens_of, write_folder
+from design_util import ARMS, engine, logit_error, run_portions, tokens_of, write_folder
 from machx_inference_engine_b200.models import load_model
 from machx_inference_engine_b200.runtime.engine import EngineOptions, LLMEngine, OutOfBlocks, SamplingParams
 
+TOL = {"fp32": 1e-5, "bf16": 1.5e-2}      # of the logits, whose size the tied table sets
 L = oracle.latent_layer
 YARN = (4.0, 100, 16.0, 1.0)
 CONFIGS = {
