@@ -122,8 +122,8 @@ gemm_kernel(const __grid_constant__ CUtensorMap tmap_a, const __grid_constant__ 
   // k-blocks per barrier handshake.  The single MMA-issuing thread pays a fixed cost per wait / commit pair, which at one
   // 64-wide k-block per handshake exceeded the tensor time of a 128x128 tile: TMA-fed (bf16) weights hand over two blocks
   // at once (measured 973 -> 1103 TFLOP/s at 8192^3).  Decoded weights are bound by the decode warps, not by the
-  // handshake (no gain measured), and keep the finer ring.
-  constexpr int KS = (!kDequant && SA % 2 == 0) ? 2 : 1;
+  // handshake (no gain measured), and keep the finer ring; a 256-column block has twice the tensor time and needs no pairing.
+  constexpr int KS = (!kDequant && SA % 2 == 0 && BN <= 128) ? 2 : 1;
   constexpr int LA = SA / KS, LB = (kDequant ? SB : SA) / KS;      // logical ring depths
   constexpr uint32_t TMEM_COLS = (2 * BN) < 32 ? 32 : (2 * BN);   // power of two for BN in {32,64,128,256}
   extern __shared__ uint8_t smem_raw[];
@@ -540,7 +540,7 @@ static int dispatch_fmt(int fmt, const CUtensorMap& ta, const CUtensorMap& tb, c
 //   out_f32    output kind: 0 bf16, 1 fp32, 2 fp16
 //   wfmt/w0..w3  weight format and plane pointers (see WFormat); n_experts >= 1
 //   tile_expert / num_m_tiles_dev: grouped mode (both null for a plain GEMM)
-//   bn         32, 64 or 128 (tile width); the caller picks small tiles for small M
+//   bn         32, 64 or 128 (tile width), with bf16 weights also 256; the caller picks small tiles for small M
 // Returns 0 or a CUDA / driver error code.
 struct GatherIn { const int* flags; const int* seq; int rows_per_src, world, m_rot; };
 // Activations that are not one dense matrix: per head (heads > 0: row t of head h at a + t * lda + h * a_head, output at c + h * c_head) or pages
@@ -656,6 +656,7 @@ static int gemm_impl(const void* a, int wfmt, const void* w0, const void* w1, co
     tb = ta;
   }
   switch (bn) {
+    case 256: return wfmt == WF_BF16 ? launch<WF_BF16, 256, 4, 1>(ta, tb, p, stream) : -105;
     case 128: return dispatch_fmt<128, 6, 4, 6>(wfmt, ta, tb, p, stream);
     case 64: return dispatch_fmt<64, 8, 6, 4>(wfmt, ta, tb, p, stream);
     case 32: return dispatch_fmt<32, 8, 6, 4>(wfmt, ta, tb, p, stream);

@@ -35,7 +35,10 @@
 
 namespace mx {
 
-static int g_gs_bf16_wide = 0;    // bf16 matrices with eight consumer warps per CTA (mx_gemv_stream_set_bf16_wide: A/B timing)
+// bf16 matrices with eight consumer warps per CTA: 0 never, 1 always, 2 for rows of up to GS_WIDE_MAX_K elements, whose stages are short (12288 x 2048:
+// 11.1 us instead of 16.7; the larger CTAs leave the next kernel's less room to start early, which costs longer rows more than it gives)
+static int g_gs_bf16_wide = 2;
+constexpr int GS_WIDE_MAX_K = 2048;
 static int g_gs_tma = 1;          // tiled TMA loads for chunked stages (mx_gemv_stream_set_tma: A/B timing)
 
 constexpr int GS_MAX_STAGES = 4;
@@ -1033,7 +1036,10 @@ static int gemv_stream_fused(int wfmt, const WeightRef& w, const void* x, void* 
   if (route) p.route = *route; else p.route.ticket = nullptr;
   if ((norm || route) && (wfmt == WF_MXFP4 || wfmt == WF_Q4K || wfmt == WF_Q6K || p.slot_mode)) return 1;
   switch (wfmt) {
-    case WF_BF16: return g_gs_bf16_wide ? gs_dispatch<WF_BF16W>(p, st) : gs_dispatch<WF_BF16>(p, st);
+    case WF_BF16: {
+      const bool wide = g_gs_bf16_wide == 1 || (g_gs_bf16_wide == 2 && K <= GS_WIDE_MAX_K && !norm && !route);
+      return wide ? gs_dispatch<WF_BF16W>(p, st) : gs_dispatch<WF_BF16>(p, st);
+    }
     case WF_Q8: return (norm || route) ? gs_dispatch<WF_Q8>(p, st) : gs_dispatch<WF_Q8I>(p, st);
     case WF_Q4K: return gs_dispatch<WF_Q4K>(p, st);
     case WF_Q6K: return gs_dispatch<WF_Q6K>(p, st);
@@ -1043,7 +1049,7 @@ static int gemv_stream_fused(int wfmt, const WeightRef& w, const void* x, void* 
 
 }  // namespace mx
 MX_HOST_API void mx_gemv_stream_set_tma(int on) { mx::g_gs_tma = on ? 1 : 0; }
-MX_HOST_API void mx_gemv_stream_set_bf16_wide(int on) { mx::g_gs_bf16_wide = on ? 1 : 0; }
+MX_HOST_API void mx_gemv_stream_set_bf16_wide(int on) { mx::g_gs_bf16_wide = on == 2 ? 2 : (on ? 1 : 0); }
 namespace mx {
 
 // One ticket word per launch of a router GEMV with the routing tail; launches rotate through the words (see attention.cu).

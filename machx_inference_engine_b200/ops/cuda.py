@@ -68,9 +68,10 @@ def set_gemv_path(path) -> None:
     _lib.cuda().mx_gemv_set_path(code)
 
 
-def set_gemv_bf16_wide(on: bool) -> None:
-    """Streaming GEMV over bf16 weights with eight consumer warps per CTA instead of four (MX_GEMV_BF16_WIDE=0/1 sets it at import)."""
-    _lib.cuda().mx_gemv_stream_set_bf16_wide(int(bool(on)))
+def set_gemv_bf16_wide(on: Optional[bool]) -> None:
+    """Streaming GEMV over bf16 weights with eight consumer warps per CTA instead of four; None: for short rows only, the default
+    (MX_GEMV_BF16_WIDE=0/1 sets it at import)."""
+    _lib.cuda().mx_gemv_stream_set_bf16_wide(2 if on is None else int(bool(on)))
 
 
 def set_gemv_tma(on: bool) -> None:
@@ -312,7 +313,8 @@ def qkv_post(qkv, bias, q_norm_w, k_norm_w, positions, rope_cos, rope_sin, slot_
 GEMV_MAX_M = 8
 
 
-def _pick_bn(M: int, N: int) -> int:
+def _pick_bn(M: int, N: int, wide: bool = False) -> int:
+    """Columns per GEMM tile.  ``wide`` (bf16 weights): 256-column tiles may be taken."""
     # small-M problems are weight-read bound: use narrow tiles so every SM streams weights
     sms = sm_count()
     if M <= 128:
@@ -320,8 +322,12 @@ def _pick_bn(M: int, N: int) -> int:
             if (N + bn - 1) // bn >= sms:
                 return bn
         return 32
-    tiles128 = ((M + 127) // 128) * ((N + 127) // 128)
-    return 128 if tiles128 >= sms else 64
+    tiles = lambda bn: ((M + 127) // 128) * ((N + bn - 1) // bn)
+    if tiles(128) < sms:
+        return 64
+    # whole waves of tiles, a 256-column tile at 1.71 times the time of a 128-column one (8192^3: 1005 against 1172 us)
+    waves = lambda bn: (tiles(bn) + sms - 1) // sms
+    return 256 if wide and 1.71 * waves(256) < waves(128) else 128
 
 
 def _gemm_a(x, w: QuantWeight):
@@ -389,7 +395,7 @@ def linear(x, w: QuantWeight, bias=None, act=ACT_NONE, act_alpha=1.702, act_limi
             _count()
             fmt, p0, p1, p2, p3 = int(WFormat.BF16), _p(wb), _vp(0), _vp(0), _vp(0)
         _check(lib.mx_gemm(_p(xa), fmt, p0, p1, p2, p3, 1, _p(out), out.stride(0), int(out_f32), _p(bias), _p(row_scale), act,
-                           C.c_float(act_alpha), C.c_float(act_limit), M, w.N, w.K, _vp(0), _vp(0), _pick_bn(M, w.N), _stream()), "gemm")
+                           C.c_float(act_alpha), C.c_float(act_limit), M, w.N, w.K, _vp(0), _vp(0), _pick_bn(M, w.N, wide=fmt == int(WFormat.BF16)), _stream()), "gemm")
     _count()
     return out
 
@@ -735,7 +741,7 @@ def gemm_paged(cache, plan, w: QuantWeight, out) -> None:
     pages, num, _ = plan
     bs, width = cache.shape[2], cache.shape[3]
     _check(_lib.cuda().mx_gemm_paged(_p(cache), width, C.c_longlong(cache.shape[0] * bs), _p(pages), _p(num), _p(w.p0), _p(out), pages.numel(), w.N, w.K,
-                                     _pick_bn(pages.numel() * bs, w.N), _stream()), "gemm_paged")
+                                     _pick_bn(pages.numel() * bs, w.N, wide=True), _stream()), "gemm_paged")
     _count()
 
 

@@ -102,7 +102,7 @@ def test_gemm_tcgen05(fmt, shape):
     qw = make_weight(fmt, N, Kd)
     x = (torch.randn(M, Kd, device=dev()) * 0.5).to(torch.bfloat16)
     bias = torch.randn(N, device=dev())
-    for bn in (128, 64, 32):
+    for bn in (128, 64, 32) + ((256,) if fmt == WFormat.BF16 else ()):
         got = K().gemm(x, qw, bias=bias, out_f32=True, bn=bn)
         K().check_status()
         want = ref.linear(x, qw, bias=bias, out_f32=True)
@@ -305,7 +305,7 @@ def test_streaming_gemv_bf16_eight_warps():
             k.check_status()
             assert torch.equal(outs[0], outs[1]), (M, N, Kd)
     finally:
-        k.set_gemv_bf16_wide(False)
+        k.set_gemv_bf16_wide(None)
 
 
 def test_streaming_gemv_chunk_copies_both_ways():
