@@ -79,7 +79,7 @@ def _folder_bytes(path: str, ctx: int, n_seqs: int) -> tuple:
     c = read_json_config(path)
     weights = sum(os.path.getsize(os.path.join(path, f)) for f in os.listdir(path) if f.endswith(".safetensors"))
     kv = sum(c.layer_specs[l].kv_width() for l, _ in c.layer_runs()) * ctx * 2 * n_seqs
-    return weights, kv, sum(s.width for s in c.layer_specs) * 4 * n_seqs
+    return weights, kv, sum(s.state_bytes(c.hidden) for s in c.layer_specs) * n_seqs
 
 
 def visible_gpus() -> tuple:

@@ -8,6 +8,7 @@ keeps one struct per family; here one dataclass serves all graphs.
 from __future__ import annotations
 
 import json
+import math
 import os
 from dataclasses import dataclass, field, asdict
 from typing import Any, Mapping, Optional
@@ -18,7 +19,7 @@ HYBRID_ARCHS = ("qwen3next", "qwen35", "qwen35moe")
 GEMMA_ARCHS = ("gemma4",)
 SUPPORTED_ARCHS = DENSE_ARCHS + MOE_ARCHS + HYBRID_ARCHS + GEMMA_ARCHS
 # checkpoints that are a folder with config.json + safetensors and list their layers one by one: "architecture" value -> arch
-LAYER_LIST_ARCHS = {"Tikarax": "tikarax", "Pubodra": "pubodra"}
+LAYER_LIST_ARCHS = {"Tikarax": "tikarax", "Pubodra": "pubodra", "Beputar": "beputar"}
 
 
 class ConfigError(ValueError):
@@ -29,7 +30,7 @@ class ConfigError(ValueError):
 class LayerSpec:
     """One layer of a design whose configuration lists its layers: a mixer with its sizes and constants, and a feed-forward (``ffn`` wide, or
     ``experts`` of ``expert_ffn`` each with ``experts_used`` per token; none when both are 0)."""
-    mixer: str                     # "attention" | "mingru" | "latent_attention"
+    mixer: str                     # "attention" | "mingru" | "latent_attention" | "rotary_attention" | "wkv" | "parallel"
     ffn: int = 0
     experts: int = 0
     experts_used: int = 0
@@ -50,10 +51,24 @@ class LayerSpec:
     yarn: Optional[tuple] = None   # (factor, original context, fast turns, slow turns)
     # minGRU
     width: int = 0
+    # rotary attention (and the left half of a parallel mixer): heads .. scale and rot_dim .. yarn above
+    keep_first: int = 0            # with a window: the first tokens of a sequence that stay visible
+    # experts whose weight scales their input
+    shared_ffn: int = 0            # width of the expert that every token uses (0: none)
+    # recurrences with a matrix per head (wkv, the right half of a parallel mixer)
+    lin_heads: int = 0
+    lin_key_dim: int = 0
+    lin_value_dim: int = 0
+    lin_decay: tuple = ()          # per head; empty where the decay comes from the data
+    decay_rank: int = 0            # wkv: inner width of the decay's projection (0: as the checkpoint's tensor has it)
 
     def kv_width(self) -> int:
         """Cached elements per token."""
-        return self.kv_heads * (self.key_dim + self.value_dim) + self.kv_rank + self.rot_dim
+        return self.kv_heads * (self.key_dim + self.value_dim) + (self.kv_rank + self.rot_dim if self.kv_rank else 0)
+
+    def state_bytes(self, hidden: int) -> int:
+        """Recurrent state per sequence (fp32): the minGRU row, or a matrix per head and, for wkv, the last row of its input."""
+        return 4 * (self.width + self.lin_heads * self.lin_key_dim * self.lin_value_dim + (hidden if self.mixer == "wkv" else 0))
 
 
 @dataclass
@@ -125,7 +140,7 @@ class ModelConfig:
 
     def layer_is_full_attention(self, layer: int) -> bool:
         if self.layer_specs:
-            return self.layer_specs[layer].mixer in ("attention", "latent_attention")
+            return self.layer_specs[layer].mixer in ("attention", "latent_attention", "rotary_attention", "parallel")
         if not self.is_hybrid:
             return True
         return (layer + 1) % self.full_attn_interval == 0
@@ -352,6 +367,70 @@ def _pubodra_config(d: Mapping[str, Any]) -> ModelConfig:
     return _finish_layer_list(c)
 
 
+def _yarn(rot: Mapping[str, Any], where: str) -> Optional[tuple]:
+    y = rot.get("scaling")
+    if y is None:
+        return None
+    out = (float(y["factor"]), float(y["original"]), float(y["fast"]), float(y["slow"]))
+    if min(out) <= 0:
+        raise ConfigError(f"{where}: rot.scaling values must be positive")
+    return out
+
+
+def _beputar_attention(s: LayerSpec, m: Mapping[str, Any], where: str) -> None:
+    rot, mask = m["rot"], m.get("mask")
+    s.heads, s.kv_heads, s.key_dim, s.value_dim, s.scale = int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"])
+    s.rot_dim, s.rope_theta, s.yarn = int(rot["dims"]), float(rot["base"]), _yarn(rot, where)
+    if min(s.heads, s.kv_heads, s.key_dim) < 1 or s.heads % s.kv_heads:
+        raise ConfigError(f"{where}: {s.heads} query heads do not divide over {s.kv_heads} key/value heads")
+    if s.value_dim != s.key_dim:
+        raise ConfigError(f"{where}: the values are the projected keys, so vdim must equal dim")
+    if not 0 <= s.rot_dim <= s.key_dim or s.rot_dim % 2:
+        raise ConfigError(f"{where}: rot.dims must be even and at most dim")
+    if mask is not None:
+        s.window, s.keep_first = int(mask["size"]), int(mask.get("keep_first", 0))
+        if s.window < 1 or s.keep_first < 0:
+            raise ConfigError(f"{where}: mask.size must be positive and keep_first not negative")
+
+
+def _beputar_config(d: Mapping[str, Any]) -> ModelConfig:
+    c = ModelConfig(arch="beputar", hidden=int(d["width"]), vocab=int(d["vocab"]), rms_eps=float(d["norm"]["eps"]), tie_embeddings=True,
+                    embedding_scale=float(d["embedding"]["scale"]), name=str(d.get("name", "")))
+    for i, e in enumerate(d["layers"]):
+        m, mlp, where = e["mixer"], e.get("mlp"), f"layer {i}"
+        if e["type"] == "attention":
+            s = LayerSpec("rotary_attention")
+            _beputar_attention(s, m, where)
+        elif e["type"] == "wkv":
+            s = LayerSpec("wkv", lin_heads=int(m["heads"]), lin_key_dim=int(m["dim"]), lin_value_dim=int(m["dim"]))
+        elif e["type"] == "parallel":
+            r = m["right"]
+            s = LayerSpec("parallel", lin_heads=int(r["heads"]), lin_key_dim=int(r["dim"]), lin_value_dim=int(r["vdim"]),
+                          lin_decay=tuple(float(v) for v in r["decay"]))
+            _beputar_attention(s, m["left"], f"{where}, left")
+            if len(s.lin_decay) != s.lin_heads:
+                raise ConfigError(f"{where}: one decay per head")
+        else:
+            raise ConfigError(f"{where}: unknown mixer {e['type']!r}")
+        if s.mixer != "rotary_attention" and min(s.lin_heads, s.lin_key_dim, s.lin_value_dim) < 1:
+            raise ConfigError(f"{where}: sizes must be positive")
+        kind = None if mlp is None else mlp.get("kind", "dense")
+        if kind == "dense":
+            s.ffn = int(mlp["ff"])
+        elif kind == "moe":
+            s.experts, s.experts_used, s.expert_ffn = int(mlp["router"]["experts"]), int(mlp["router"]["top"]), int(mlp["expert"]["ff"])
+            if mlp.get("shared") is not None:
+                s.shared_ffn = int(mlp["shared"]["ff"])
+            if not 1 <= s.experts_used <= s.experts:
+                raise ConfigError(f"{where}: {s.experts_used} of {s.experts} experts per token")
+        elif kind is not None:
+            raise ConfigError(f"{where}: unknown feed-forward kind {kind!r}")
+        c.layer_specs.append(s)
+    if c.hidden < 1 or c.vocab < 1 or not c.layer_specs:
+        raise ConfigError("the width must be positive, with at least one layer")
+    return _finish_layer_list(c)
+
+
 def _finish_layer_list(c: ModelConfig) -> ModelConfig:
     """Derived fields of a layer-list config: the largest sizes of any layer (pool sizing, reports)."""
     big = lambda f, lo=0: max([lo] + [getattr(s, f) for s in c.layer_specs])
@@ -359,6 +438,7 @@ def _finish_layer_list(c: ModelConfig) -> ModelConfig:
     c.n_heads, c.n_kv_heads, c.ffn = big("heads", 1), big("kv_heads", 1), big("ffn")
     c.head_dim = max(big("key_dim", 1), big("value_dim"))
     c.n_experts, c.n_experts_used, c.expert_ffn = big("experts"), big("experts_used"), big("expert_ffn")
+    c.shared_expert_ffn = big("shared_ffn")
     c.n_rot, c.ctx_train = 0, 1 << 20                      # rotations, where there are any, belong to the layers; positions have no limit of their own
     return c
 
@@ -371,7 +451,7 @@ def read_json_config(path_or_dict) -> ModelConfig:
         with open(p) as f:
             d = json.load(f)
     a = d.get("architecture")
-    readers = {"tikarax": _tikarax_config, "pubodra": _pubodra_config}
+    readers = {"tikarax": _tikarax_config, "pubodra": _pubodra_config, "beputar": _beputar_config}
     if a not in LAYER_LIST_ARCHS:
         raise ConfigError(f"unsupported architecture {a!r} in config.json (supported: {', '.join(LAYER_LIST_ARCHS)})")
     try:
@@ -384,15 +464,31 @@ def config_to_json(c: ModelConfig) -> dict:
     """Inverse of :func:`read_json_config`."""
     whole = lambda v: int(v) if float(v).is_integer() else v
     layers = []
+
+    def rotation(s):
+        rot = {"base": s.rope_theta, "dims": s.rot_dim}
+        if s.yarn is not None:
+            rot["scaling"] = dict(zip(("factor", "original", "fast", "slow"), (s.yarn[0], whole(s.yarn[1]), s.yarn[2], s.yarn[3])))
+        return rot
+
+    def rotary(s):
+        m = {"heads": s.heads, "kv_heads": s.kv_heads, "dim": s.key_dim, "vdim": s.value_dim, "scale": s.scale, "rot": rotation(s)}
+        if s.window:
+            m["mask"] = {"size": s.window, **({"keep_first": s.keep_first} if s.keep_first else {})}
+        return m
+
     for s in c.layer_specs:
-        if s.mixer == "attention":
+        if s.mixer == "rotary_attention":
+            m = rotary(s)
+        elif s.mixer == "wkv":
+            m = {"heads": s.lin_heads, "dim": s.lin_key_dim}
+        elif s.mixer == "parallel":
+            m = {"left": rotary(s), "right": {"heads": s.lin_heads, "dim": s.lin_key_dim, "vdim": s.lin_value_dim, "decay": list(s.lin_decay)}}
+        elif s.mixer == "attention":
             m = {"heads": s.heads, "kv_heads": s.kv_heads, "dim": s.key_dim, "vdim": s.value_dim, "scale": s.scale,
                  "q_temp": {"coef": s.q_temp_coef, "every": whole(s.q_temp_every)}}
         elif s.mixer == "latent_attention":
-            rot = {"base": s.rope_theta, "dims": s.rot_dim}
-            if s.yarn is not None:
-                rot["scaling"] = dict(zip(("factor", "original", "fast", "slow"), (s.yarn[0], whole(s.yarn[1]), s.yarn[2], s.yarn[3])))
-            m = {"heads": s.heads, "dim": s.key_dim, "rot_dim": s.rot_dim, "vdim": s.value_dim, "kv_rank": s.kv_rank, "scale": s.scale, "rot": rot}
+            m = {"heads": s.heads, "dim": s.key_dim, "rot_dim": s.rot_dim, "vdim": s.value_dim, "kv_rank": s.kv_rank, "scale": s.scale, "rot": rotation(s)}
             if s.window:
                 m["mask"] = {"size": s.window}
         else:
@@ -400,10 +496,14 @@ def config_to_json(c: ModelConfig) -> dict:
         mlp = {"kind": "dense", "ff": s.ffn} if s.ffn else None
         if s.experts:
             mlp = {"kind": "moe", "expert": {"ff": s.expert_ffn}, "router": {"experts": s.experts, "top": s.experts_used}}
-        layers.append({"type": s.mixer, "mixer": m, "mlp": mlp})
+            if s.shared_ffn:
+                mlp["shared"] = {"ff": s.shared_ffn}
+        layers.append({"type": {"rotary_attention": "attention"}.get(s.mixer, s.mixer), "mixer": m, "mlp": mlp})
     arch = {v: k for k, v in LAYER_LIST_ARCHS.items()}[c.arch]
     norm = {"eps": c.rms_eps, "groups": c.norm_groups} if c.arch == "tikarax" else {"eps": c.rms_eps}
     out = {"architecture": arch, "layers": layers, "norm": norm, "vocab": c.vocab, "width": c.hidden}
+    if c.arch == "beputar":
+        out["embedding"] = {"scale": c.embedding_scale}
     if c.loop_times:
         out["loop"] = {"start": c.loop_start, "stop": c.loop_stop, "times": c.loop_times}
     return out
@@ -485,6 +585,29 @@ def _pubodra_preset(hidden, n_layers, heads, dim, rot_dim, vdim, kv_rank, window
     return _finish_layer_list(c)
 
 
+def _beputar_preset(hidden, n_layers, heads, kv_heads, dim, window, keep_first, lin_heads, lin_dim, lin_vdim, wkv_heads, wkv_dim, decay_rank, ffn, vocab, experts=0,
+                    used=0, expert_ffn=0, shared=0, order=("parallel", "rotary_attention", "wkv"), theta=1e6, yarn=(8.0, 2048.0, 32.0, 1.0)) -> ModelConfig:
+    """The mixers of ``order`` in turn; the first layer has a dense feed-forward, the others experts (when there are any)."""
+    c = ModelConfig(arch="beputar", hidden=hidden, vocab=vocab, rms_eps=1e-6, tie_embeddings=True, embedding_scale=12.0)
+    for l in range(n_layers):
+        s = LayerSpec(order[l % len(order)])
+        if s.mixer == "wkv":
+            s.lin_heads, s.lin_key_dim, s.lin_value_dim, s.decay_rank = wkv_heads, wkv_dim, wkv_dim, decay_rank
+        else:
+            s.heads, s.kv_heads, s.key_dim, s.value_dim, s.window, s.scale = heads, kv_heads, dim, dim, window, dim ** -0.5
+            s.rot_dim, s.rope_theta = (dim // 4 * 2, theta) if s.mixer == "parallel" else (dim, 1e4)
+            s.yarn = None if s.mixer == "parallel" else yarn
+        if s.mixer == "parallel":
+            s.keep_first, s.lin_heads, s.lin_key_dim, s.lin_value_dim = keep_first, lin_heads, lin_dim, lin_vdim
+            s.lin_decay = tuple(math.exp(-2.0 ** (-8.0 * (h + 1) / lin_heads)) for h in range(lin_heads))
+        if experts and l:
+            s.experts, s.experts_used, s.expert_ffn, s.shared_ffn = experts, used, expert_ffn, shared
+        else:
+            s.ffn = ffn
+        c.layer_specs.append(s)
+    return _finish_layer_list(c)
+
+
 # ---- named architectures used by the benches and tests (random-init; see formats/synth.py)
 def preset(name: str) -> ModelConfig:
     p = {
@@ -548,6 +671,11 @@ def preset(name: str) -> ModelConfig:
         # layers of common model sizes: 1 B class and 8 B class, the latter with 64 small experts in every other layer
         "pubodra-1b": _pubodra_preset(2048, 16, 16, 128, 64, 128, 512, 1024, 12288, 128256),
         "pubodra-8b": _pubodra_preset(4096, 32, 32, 128, 64, 128, 512, 4096, 21504, 128256, experts=64, used=6, expert_ffn=1536),
+        "tiny-beputar": _beputar_preset(160, 4, 6, 2, 40, 50, 3, 5, 24, 40, 3, 40, 24, 224, 384, experts=6, used=2, expert_ffn=96, shared=64,
+                                        yarn=(4.0, 64.0, 32.0, 1.0)),
+        # layers of common model sizes: 1 B class and 8 B class
+        "beputar-1b": _beputar_preset(2048, 15, 32, 8, 64, 1024, 16, 16, 128, 128, 32, 64, 64, 8192, 128256, experts=64, used=6, expert_ffn=1024, shared=2048),
+        "beputar-8b": _beputar_preset(4096, 30, 32, 8, 128, 4096, 16, 32, 128, 128, 64, 64, 64, 16384, 128256, experts=64, used=6, expert_ffn=1536, shared=3072),
         "tiny-qwen2": ModelConfig(arch="qwen2", n_layers=2, hidden=256, n_heads=4, n_kv_heads=2, head_dim=64, ffn=512, vocab=2048,
                                   rms_eps=1e-6, rope_theta=1e6, n_rot=64, ctx_train=4096),
         "tiny-phi3": ModelConfig(arch="phi3", n_layers=2, hidden=256, n_heads=4, n_kv_heads=4, head_dim=64, ffn=512, vocab=2048,

@@ -335,9 +335,42 @@ def _pubodra_tensors(cfg: ModelConfig) -> list:
     return out
 
 
+def _beputar_tensors(cfg: ModelConfig) -> list:
+    H = cfg.hidden
+    out = [("embed", "matrix", (cfg.vocab, H)), ("final.norm", "norm", (H,))]
+    matrices = lambda p, shapes: [(f"{p}.{n}", "matrix", shape) for n, shape in shapes.items()]
+    for i, s in enumerate(cfg.layer_specs):
+        p, m, q, kv, lk, lv = f"l{i}", f"l{i}.mix", s.heads * s.key_dim, s.kv_heads * s.key_dim, s.lin_heads * s.lin_key_dim, s.lin_heads * s.lin_value_dim
+        if s.mixer == "rotary_attention":
+            out += matrices(m, {"q": (q, H), "k": (kv, H), "o": (H, q)}) + [(f"{m}.q.b", "vector", (q,)), (f"{m}.k.b", "vector", (kv,))]
+        elif s.mixer == "wkv":
+            r = s.decay_rank or 16
+            out += matrices(m, {"r": (lk, H), "k": (lk, H), "v": (lv, H), "g": (lv, H), "w1": (r, H), "w2": (lk, r), "o": (H, lv)})
+            out += [(f"{m}.mu.{n}", "vector", (H,)) for n in "rkvgw"]
+            out += [(f"{m}.w0", "vector", (lk,)), (f"{m}.u", "vector", (s.lin_heads, s.lin_key_dim)), (f"{m}.norm", "norm", (lv,))]
+        else:
+            out += matrices(f"{m}.left", {"q": (q, H), "k": (kv, H), "g": (s.heads, H), "o": (H, q)})
+            out += matrices(f"{m}.right", {"q": (lk, H), "k": (lk, H), "v": (lv, H), "g": (lv, H), "o": (H, lv)})
+            out += [(f"{m}.left.q.norm", "norm", (s.key_dim,)), (f"{m}.left.k.norm", "norm", (s.key_dim,)), (f"{m}.right.norm", "norm", (lv,)),
+                    (f"{m}.left.out", "norm", (H,)), (f"{m}.right.out", "norm", (H,))]
+        out += [(f"{p}.norm1", "norm", (H,)), (f"{p}.ls1", "norm", (H,))]
+        if s.ffn or s.experts:
+            out += [(f"{p}.norm2", "norm", (H,)), (f"{p}.ls2", "norm", (H,))]
+        if s.ffn:
+            out += matrices(f"{p}.mlp", {"up": (s.ffn, H), "down": (H, s.ffn)})
+        gated = lambda n, f: matrices(f"{p}.mlp{n}", {"gate": (f, H), "up": (f, H), "down": (H, f)})
+        for e in range(s.experts):
+            out += gated(f".e{e}", s.expert_ffn)
+        if s.experts:
+            out.append((f"{p}.mlp.router", "matrix", (s.experts, H)))
+        if s.shared_ffn:
+            out += gated(".shared", s.shared_ffn)
+    return out
+
+
 def folder_tensor_plan(cfg: ModelConfig) -> list:
     """(name, kind, shape) of every tensor of a layer-list checkpoint folder (``LAYER_LIST_ARCHS``); matrices are [out, in]."""
-    return {"tikarax": _tikarax_tensors, "pubodra": _pubodra_tensors}[cfg.arch](cfg)
+    return {"tikarax": _tikarax_tensors, "pubodra": _pubodra_tensors, "beputar": _beputar_tensors}[cfg.arch](cfg)
 
 
 def write_synthetic_folder(cfg: ModelConfig, path: str, seed: int = 0) -> dict:

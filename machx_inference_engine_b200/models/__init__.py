@@ -10,7 +10,8 @@ from ..parallel.comm import ParallelCtx
 
 # file names of the tensors that every graph asks for under its GGUF name
 _FOLDER_NAMES = {"tikarax": {"token_embd.weight": "embed", "output_norm.weight": "final.norm", "output.weight": "head"},
-                 "pubodra": {"token_embd.weight": "embed", "output_norm.weight": "final.norm"}}
+                 "pubodra": {"token_embd.weight": "embed", "output_norm.weight": "final.norm"},
+                 "beputar": {"token_embd.weight": "embed", "output_norm.weight": "final.norm"}}
 
 
 def _graph_class(cfg: ModelConfig):
@@ -26,6 +27,9 @@ def _graph_class(cfg: ModelConfig):
     if cfg.arch == "pubodra":
         from .pubodra import PubodraModel
         return PubodraModel
+    if cfg.arch == "beputar":
+        from .beputar import BeputarModel
+        return BeputarModel
     from .transformer import TransformerModel
     return TransformerModel
 

@@ -21,9 +21,9 @@ import torch
 
 from .. import ops
 from ..formats.model_config import ModelConfig
-from ..ops import ACT_SWIGLU, QuantWeight
+from ..ops import ACT_SWIGLU, ACT_TANH, QuantWeight
 from ..parallel.comm import ParallelCtx
-from .transformer import AttentionBlock, DenseFFN, ForwardBatch, KVCache, Linear, MoEFFN, TransformerModel, _fuse_rows, round_up
+from .transformer import AttentionBlock, DenseFFN, ForwardBatch, KVCache, Linear, MoEFFN, TransformerModel, _as_bf16, _fuse_rows, round_up
 
 D_HEAD = 128      # DeltaNet key / value head width (the only geometry the families use)
 
@@ -191,6 +191,87 @@ class MinGRUBlock:
         s = ops.mingru_scan(y[:, :W], y[:, W:2 * W], y[:, 2 * W:], self.zb, self.xb, state.tensors["S"][self.layer], fb.state_slots, fb.cu_q, fb.seq_lens,
                             fb.max_q_len)
         return self.out(s)
+
+
+class DecayAttentionBlock:
+    """Linear attention with a fixed decay per head (lightning attention): q, k, v = silu of their projections, S <- decay S + k v^T, o = S^T q; the heads
+    RMS-normed together, times the sigmoid of a gate, output projection.  ``parts`` are the rows [q | k | v | gate] of one projection (see
+    KeyValueAttentionBlock); head widths are padded to multiples of 8 at load."""
+
+    def __init__(self, src, prefix: str, layer: int, hidden: int, row: int, heads: int, key_dim: int, value_dim: int, decay, eps: float):
+        self.layer, self.H, self.eps, self.live = layer, heads, eps, heads * value_dim
+        dk, dv = self.dk, self.dv = round_up(key_dim, 8), round_up(value_dim, 8)
+        rows = lambda n, d, to: (src.matrix(f"{prefix}.{n}", heads * d, hidden).pad_groups(rows=(heads, to), cols=(1, row)), None)
+        self.parts = [rows("q", key_dim, dk), rows("k", key_dim, dk), rows("v", value_dim, dv), rows("g", value_dim, dv)]
+        dev = self.parts[0][0].device
+        self.decay = torch.tensor(list(decay), dtype=torch.float64).to(torch.float32).to(dev)
+        self.norm = _pad_heads(src.vector(f"{prefix}.norm", heads * value_dim), heads, dv)
+        self.out = Linear(src.matrix(f"{prefix}.o", hidden, heads * value_dim).pad_groups(rows=(1, row), cols=(heads, dv)))
+        self.state_shape = {"S": (heads, dk, dv)}
+
+    def attend(self, y: torch.Tensor, fb: ForwardBatch, state: RecurrentState) -> torch.Tensor:
+        """y: this block's columns of the projection."""
+        H, dk, dv = self.H, self.dk, self.dv
+        q, k, v, g = y.split([H * dk, H * dk, H * dv, H * dv], dim=1)
+        o = ops.decay_scan(q.unflatten(1, (H, dk)), k.unflatten(1, (H, dk)), v.unflatten(1, (H, dv)), state.tensors["S"][self.layer], fb.state_slots, fb.cu_q,
+                           fb.seq_lens, fb.max_q_len, decay=self.decay, silu=True)
+        return self.out(ops.gated_group_norm(o, g, self.norm, self.eps, width=self.live, out_dtype=y.dtype))
+
+
+class WkvBlock:
+    """RWKV-style time mixing: r, k, v, gate and the decay's input are mixes of the token's row and the one before it; a matrix state per head with a
+    decay per key channel that comes from the data, and a bonus for the current token; per-head RMS norm, SiLU gate, output projection.
+
+    Launches: the shifted mixes, the four projections of equal shape as one product over a stack, the two small ones of the decay, the recurrence, the
+    gated norm, the output projection.  Works on the fp32 residual itself."""
+
+    MIXES = ("r", "k", "v", "g", "w")
+
+    def __init__(self, src, prefix: str, layer: int, hidden: int, row: int, heads: int, dim: int, rank: int, eps: float, act_dtype: torch.dtype):
+        self.layer, self.H, self.dim, self.eps, self.act_dtype = layer, heads, dim, eps, act_dtype
+        d = self.d = round_up(dim, 8)
+        rank = src.shape(f"{prefix}.w1")[0] if hasattr(src, "shape") else rank or 16
+        rp = round_up(rank, 32)
+        self.mu = torch.stack([torch.nn.functional.pad(src.vector(f"{prefix}.mu.{n}", hidden), (0, row - hidden)) for n in self.MIXES]).contiguous()
+        ws = [src.matrix(f"{prefix}.{n}", heads * dim, hidden).pad_groups(rows=(heads, d), cols=(1, row)) for n in "rkvg"]
+        if any(w.fmt != ops.WFormat.BF16 for w in ws):
+            ws = [QuantWeight(**_as_bf16(w)) for w in ws]
+        self.rkvg = QuantWeight(ops.WFormat.BF16, heads * d, row, 4, torch.cat([w.p0 for w in ws]).contiguous())
+        self.w1 = Linear(src.matrix(f"{prefix}.w1", rank, hidden).pad_groups(rows=(1, rp), cols=(1, row)), act=ACT_TANH)
+        self.w2 = Linear(src.matrix(f"{prefix}.w2", heads * dim, rank).pad_groups(rows=(heads, d), cols=(1, rp)),
+                         _pad_heads(src.vector(f"{prefix}.w0", heads * dim), heads, d))
+        self.u = torch.nn.functional.pad(src.table(f"{prefix}.u", (heads, dim)), (0, d - dim)).contiguous()
+        self.norm = _pad_heads(src.vector(f"{prefix}.norm", heads * dim), heads, d)
+        self.out = Linear(src.matrix(f"{prefix}.o", hidden, heads * dim).pad_groups(rows=(1, row), cols=(heads, d)))
+        self.state_shape = {"S": (heads, d, d), "shift": (row,)}
+
+    def __call__(self, x: torch.Tensor, fb: ForwardBatch, state: RecurrentState) -> torch.Tensor:
+        H, d = self.H, self.d
+        mix = ops.token_shift(x, self.mu, state.tensors["shift"][self.layer], fb.state_slots, fb.cu_q, fb.seq_lens, out_dtype=self.act_dtype)
+        r, k, v, g = ops.stacked_linear(mix[:4], self.rkvg)
+        z = self.w2(self.w1(mix[4]), out_f32=True)
+        heads = lambda t: t.unflatten(1, (H, d))
+        o = ops.decay_scan(heads(r), heads(k), heads(v), state.tensors["S"][self.layer], fb.state_slots, fb.cu_q, fb.seq_lens, fb.max_q_len, z=z, u=self.u)
+        return self.out(ops.gated_group_norm(o, g, self.norm, self.eps, groups=H, width=self.dim, silu=True, out_dtype=self.act_dtype))
+
+
+def _pad_heads(v: torch.Tensor, heads: int, to: int) -> torch.Tensor:
+    return torch.nn.functional.pad(v.reshape(heads, -1), (0, to - v.numel() // heads)).reshape(-1).contiguous()
+
+
+class ParallelMixer:
+    """Two mixers that read the same input through one projection; the mean of their outputs, each RMS-normed over the model width first.  Returned
+    unformed (:class:`ops.BranchMean`): the norms run inside the residual add."""
+
+    def __init__(self, left, right, left_norm: torch.Tensor, right_norm: torch.Tensor):
+        self.left, self.right, self.norms = left, right, (left_norm, right_norm)
+        self.cut = left.columns
+        self.proj = _fuse_rows(*map(list, zip(*(left.parts + right.parts))))
+        left.parts = right.parts = None
+
+    def __call__(self, h: torch.Tensor, fb: ForwardBatch, kv: KVCache, state: RecurrentState):
+        y = self.proj(h)
+        return ops.BranchMean(self.left.attend(y[:, :self.cut], fb, kv), self.norms[0], self.right.attend(y[:, self.cut:], fb, state), self.norms[1])
 
 
 class SharedExpert:

@@ -80,6 +80,13 @@ class SafetensorsSource:
             raise ValueError(f"{n}: expected shape {tuple(shape)}, file has {tuple(self.m.shape(n))}")
         return n
 
+    def shape(self, name: str) -> tuple:
+        """Sizes that only a tensor gives."""
+        n = self._name(name)
+        if not self.m.has(n):
+            raise ValueError(f"the checkpoint has no tensor {n!r}")
+        return tuple(self.m.shape(n))
+
     def matrix(self, name: str, N: int, K: int, E: int = 1, experts: Optional[tuple[int, int]] = None) -> QuantWeight:
         if "*" in name:                  # one tensor per expert, the number in the place of the star
             lo, hi = experts if experts is not None else (0, E)
@@ -210,7 +217,7 @@ class SynthSource:
 
     def vector(self, name: str, n: int) -> torch.Tensor:
         g = self._gen(name)
-        if name.endswith(".norm") or name.rsplit(".", 1)[-1] in ("norm1", "norm1b", "norm2", "norm2b"):
+        if name.endswith(".norm") or name.rsplit(".", 1)[-1] in ("norm1", "norm1b", "norm2", "norm2b", "ls1", "ls2", "out"):
             return (1.0 + 0.05 * torch.randn(n, generator=g, device=self.gen_device)).to(self.device)
         if name.endswith("norm.weight") or "_norm" in name or name.endswith(".scale") or name.endswith("layer_output_scale.weight"):
             return (1.0 + 0.05 * torch.randn(n, generator=g, device=self.gen_device)).to(self.device)

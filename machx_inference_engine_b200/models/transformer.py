@@ -397,6 +397,73 @@ class LatentAttentionBlock:
         return self.o(a.view(T, H * self.v))
 
 
+class KeyValueAttentionBlock:
+    """Attention whose values are its keys as projected (before norm and rotation): no value projection.  Rotation of part of a head in either pairing,
+    per-head RMS norms of queries and keys with a weight before it or without one after it, sliding window that may keep the first tokens of the
+    sequence, an optional score of 0 in the softmax denominator (``zero_sink``) and an optional output gate of one number per head.
+
+    One projection gives the columns [q | k | gate]; the queries are rotated where they stand, keys and values go into the cache pages.  ``parts`` are the
+    projection's row blocks, so that a mixer that reads the same input can share it.  Head widths are padded to multiples of 8 at load."""
+
+    def __init__(self, src, prefix: str, layer: int, hidden: int, row: int, heads: int, kv_heads: int, dim: int, scale: float, window: int, keep_first: int,
+                 rot_dim: int, rope: tuple, eps: float, interleaved: bool = False, biased: bool = False, qk_norm: bool = False, norm_after: bool = False,
+                 head_gate: bool = False, zero_sink: bool = False):
+        self.layer, self.n_q, self.n_kv, self.dim, self.scale, self.eps = layer, heads, kv_heads, dim, scale, eps
+        self.window, self.keep_first = window, keep_first
+        self.rot_dim, self.rope, self.interleaved, self.norm_after = rot_dim, rope, interleaved, norm_after
+        dp = self.dp = round_up(dim, 8)
+
+        def rows(name, n, d, to):
+            w = src.matrix(f"{prefix}.{name}", n * d, hidden).pad_groups(rows=(n, to), cols=(1, row))
+            if not biased:
+                return w, None
+            b = torch.zeros(n, to, dtype=torch.float32, device=w.device)
+            b[:, :d] = src.vector(f"{prefix}.{name}.b", n * d).reshape(n, d)
+            return w, b.reshape(-1)
+
+        self.parts = [rows("q", heads, dim, dp), rows("k", kv_heads, dim, dp)]
+        self.gate_at = (heads + kv_heads) * dp if head_gate else None
+        if head_gate:
+            self.parts.append((src.matrix(f"{prefix}.g", heads, hidden).pad_groups(rows=(1, round_up(heads, 8)), cols=(1, row)), None))
+        self.columns = sum(w.N for w, _ in self.parts)
+        norm = lambda n: torch.nn.functional.pad(src.vector(f"{prefix}.{n}.norm", dim), (0, dp - dim)).contiguous()
+        self.q_norm, self.k_norm = (norm("q"), norm("k")) if qk_norm else (None, None)
+        self.sinks = torch.zeros(heads, dtype=torch.float32, device=self.parts[0][0].device) if zero_sink else None
+        self.o = Linear(src.matrix(f"{prefix}.o", hidden, heads * dim).pad_groups(rows=(1, row), cols=(heads, dp)))
+        self.proj = None
+
+    def own_projection(self) -> "KeyValueAttentionBlock":
+        self.proj, self.parts = _fuse_rows(*map(list, zip(*self.parts))), None
+        return self
+
+    def __call__(self, h: torch.Tensor, fb: ForwardBatch, kv: KVCache) -> torch.Tensor:
+        return self.attend(self.proj(h), fb, kv)
+
+    def attend(self, y: torch.Tensor, fb: ForwardBatch, kv: KVCache) -> torch.Tensor:
+        """y: this block's columns of the projection."""
+        T, nq, dp, l = y.shape[0], self.n_q * self.dp, self.dp, self.layer
+        q = ops.qk_post(y[:, :nq].unflatten(1, (self.n_q, dp)), y[:, nq:nq + self.n_kv * dp].unflatten(1, (self.n_kv, dp)), fb.positions, self.rope[0],
+                        self.rope[1], fb.slot_map, kv.k[l], kv.v[l], self.dim, self.rot_dim, interleaved=self.interleaved, q_norm=self.q_norm,
+                        k_norm=self.k_norm, norm_after=self.norm_after, eps=self.eps)
+        gate = y[:, self.gate_at:self.gate_at + self.n_q] if self.gate_at is not None else None
+        a = ops.attention(q, kv.k[l], kv.v[l], fb.block_table, fb.seq_lens, fb.cu_q, fb.max_q_len, sinks=self.sinks, window=self.window, scale=self.scale,
+                          max_kv_len=fb.max_kv_len, gate=gate, keep_first=self.keep_first)
+        return self.o(a.reshape(T, nq))
+
+
+class GatedFFN:
+    """down(act(gate h, up h)), the gate and up rows interleaved for the projection's epilogue."""
+
+    def __init__(self, src, prefix: str, hidden: int, row: int, ffn: int, act: int = ACT_SWIGLU):
+        f = round_up(ffn, 32)
+        g, u = (src.matrix(f"{prefix}.{n}", ffn, hidden).pad_groups(rows=(1, f), cols=(1, row)) for n in ("gate", "up"))
+        self.gate_up = Linear(QuantWeight.interleave_gate_up(g, u), act=act)
+        self.down = Linear(src.matrix(f"{prefix}.down", hidden, ffn).pad_groups(rows=(1, row), cols=(1, f)))
+
+    def __call__(self, h):
+        return self.down(self.gate_up(h))
+
+
 class UnaryFFN:
     """down(act(up h)): a feed-forward without a gate branch; the activation runs in the up projection's epilogue."""
 
@@ -684,6 +751,37 @@ class UnaryMoEFFN(MoEFFN):
         self.down = src.matrix(f"{prefix}.e*.down", hidden, ffn, experts).pad_groups(rows=(1, row), cols=(1, f))
         self.router_bias = self.gu_bias = self.down_bias = self.expert_scale = self.shared = self.mx = self._spill = None
         self.act, self.a8, self.reduce, self.group_gemv_max_tokens, self._arange = act, False, False, 0, {}
+
+
+class ScaledInputMoEFFN(UnaryMoEFFN):
+    """Gated experts without biases, of which each token uses the best K by router score; the weight -- the sigmoid of the chosen score, as it is --
+    multiplies what the expert reads, so the branch is a plain sum of rows, to which an always-on expert may add one.  Returns the sum unformed
+    (:class:`ops.ExpertSum`).  One GPU."""
+
+    PAIR_GEMV_MAX_TOKENS = 4
+
+    def __init__(self, src, prefix: str, hidden: int, row: int, experts: int, used: int, ffn: int, shared_ffn: int = 0, act: int = ACT_SWIGLU):
+        super().__init__(src, prefix, hidden, row, experts, used, ffn, act)          # (gate_up holds the up rows so far)
+        gate = src.matrix(f"{prefix}.e*.gate", ffn, hidden, experts).pad_groups(rows=(1, round_up(ffn, 32)), cols=(1, row))
+        self.gate_up = QuantWeight.interleave_gate_up(gate, self.gate_up)
+        self.shared = GatedFFN(src, f"{prefix}.shared", hidden, row, shared_ffn, act) if shared_ffn else None
+
+    def __call__(self, h: torch.Tensor, par: Optional[ParallelCtx] = None):
+        T, K = h.shape[0], self.K
+        idx, w = ops.moe_route(self.router(h, out_f32=True), None, K, precise=h.dtype == torch.float32, sigmoid=True)
+        if T <= self.PAIR_GEMV_MAX_TOKENS and h.dtype != torch.float32:
+            slot_e = idx.reshape(-1)
+            a = ops.expert_gemv(ops.moe_scale_rows(h, w), self.gate_up, slot_e, act=self.act)
+            y = ops.expert_gemv(a, self.down, slot_e)
+            if (T, h.device) not in self._arange:
+                self._arange[T, h.device] = torch.arange(T * K, dtype=torch.int32, device=h.device)
+            pos = self._arange[T, h.device]
+        else:
+            pk = ops.moe_pack(idx, self.E)
+            a = ops.grouped_linear(ops.moe_scale_rows(h, w, pk), self.gate_up, pk.tile_expert, pk.num_tiles, act=self.act)
+            y = ops.grouped_linear(a, self.down, pk.tile_expert, pk.num_tiles)
+            pos = pk.pair_to_packed
+        return ops.ExpertSum(y, pos, K, None if self.shared is None else self.shared(h))
 
 
 def _mx_experts(self, h: torch.Tensor, idx: torch.Tensor, pre=None, ksplit: int = 1):

@@ -14,7 +14,7 @@ import torch
 
 from .weights import QuantWeight
 
-ACT_NONE, ACT_SWIGLU, ACT_SWIGLU_OAI, ACT_GEGLU, ACT_XIELU, ACT_GELU_TANH, ACT_RELU2 = 0, 1, 2, 3, 4, 5, 6
+ACT_NONE, ACT_SWIGLU, ACT_SWIGLU_OAI, ACT_GEGLU, ACT_XIELU, ACT_GELU_TANH, ACT_RELU2, ACT_TANH = 0, 1, 2, 3, 4, 5, 6, 7
 
 
 def act_gated(act: int) -> bool:
@@ -99,7 +99,9 @@ def rmsnorm(x, w, eps, delta=None, dbias=None, one_plus_w=False, delta_scale=1.0
 
 def act_unary(act, z, a, b):
     """xIELU: a z^2 + z / 2 above zero, b (e^z - 1 - z) + z / 2 below (a = softplus(p), b = 1/2 + softplus(q)); GELU in its tanh form; the
-    square of ReLU."""
+    square of ReLU; tanh."""
+    if act == ACT_TANH:
+        return torch.tanh(z)
     if act == ACT_GELU_TANH:
         return torch.nn.functional.gelu(z, approximate="tanh")
     if act == ACT_RELU2:
@@ -137,7 +139,7 @@ def _deinterleave16(y: torch.Tensor):
 
 def glu(x, act, alpha=1.702, limit=7.0):
     g, u = _deinterleave16(x.to(torch.float32))
-    return _act(act, g, u, alpha, limit).to(torch.bfloat16)
+    return _act(act, g, u, alpha, limit).to(torch.float32 if x.dtype == torch.float32 else torch.bfloat16)
 
 
 def linear(x, w: QuantWeight, bias=None, act=ACT_NONE, act_alpha=1.702, act_limit=7.0, out_f32=False, row_scale=None, out=None):
@@ -323,10 +325,11 @@ def mingru_scan(z, u, g, zb, ub, state, state_slots, cu_q, seq_lens, max_q_len):
 
 
 def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks=None, window=0, scale=None, softcap=0.0, n_splits=1,
-              kv_scales=None, max_kv_len=0, q_scale=None, gate=None):
+              kv_scales=None, max_kv_len=0, q_scale=None, gate=None, keep_first=0):
     """q [Tq,n_q,hd]; caches [blocks,n_kv,bs,hd] (bf16 / fp32, or int8 with kv_scales = (k_scale, v_scale) [blocks,n_kv,bs]); values may be
     wider or narrower than keys; returns [Tq,n_q,value width] (bf16; fp32 for fp32 queries).  ``q_scale`` [positions]: factor on the scores
-    of a query at that position; ``gate`` [Tq, n_q * value width]: the result is multiplied by its sigmoid."""
+    of a query at that position; ``gate`` [Tq, n_q * value width] or [Tq, n_q] (one number per head): the result is multiplied by its sigmoid.
+    With a window the first ``keep_first`` keys of a sequence stay visible."""
     Tq, n_q, hd = q.shape
     dv = v_cache.shape[3]
     n_kv, bs = k_cache.shape[1], k_cache.shape[2]
@@ -358,7 +361,7 @@ def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks
         kpos = torch.arange(L, device=q.device).unsqueeze(0)
         ok = kpos <= qpos
         if window and window > 0:
-            ok = ok & (kpos > qpos - window)
+            ok = ok & ((kpos > qpos - window) | (kpos < keep_first))
         s = s.masked_fill(~ok.unsqueeze(0), float("-inf"))
         if sinks is not None:
             sk = sinks.to(torch.float32).reshape(n_q, 1, 1).expand(n_q, q1 - q0, 1)
@@ -367,8 +370,144 @@ def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks
             p = torch.softmax(s, dim=-1)
         out[q0:q1] = torch.einsum("htk,hkd->thd", p.to(_MM_DTYPE), Vh.to(_MM_DTYPE)).to(torch.float32)
     if gate is not None:
-        out = out * torch.sigmoid(gate.to(torch.float32)).reshape(Tq, n_q, dv)
+        out = out * torch.sigmoid(gate.to(torch.float32)).reshape(Tq, n_q, -1)
     return out if q.dtype == torch.float32 else out.to(torch.bfloat16)
+
+
+def qk_post(q, k, positions, rope_cos, rope_sin, slot_map, k_cache, v_cache, dim, rot_dim, interleaved=False, q_norm=None, k_norm=None, norm_after=False,
+            eps=1e-6):
+    """Head epilogue of attention whose values are its projected keys.  q [T, n_q, dp], k [T, n_kv, dp] (column ranges of one projection; the first
+    ``dim`` elements are the head, the rest zero padding): RMS norm with the weights q_norm / k_norm [dp], rotation of the first ``rot_dim``
+    elements in interleaved pairs or half splits, and with ``norm_after`` an RMS norm without a weight behind it.  Returns the queries (the kernel works
+    in place); the keys go into k_cache, and as they came into v_cache (slots < 0 are skipped)."""
+    pos = positions.long().clamp(0, rope_cos.shape[0] - 1)
+    c, s = rope_cos[pos].unsqueeze(1), rope_sin[pos].unsqueeze(1)
+    half = rot_dim // 2
+    rms = lambda t: t * torch.rsqrt(t[..., :dim].pow(2).mean(-1, keepdim=True) + eps)
+
+    def turn(t, w):
+        t = t.to(torch.float32)
+        if w is not None:
+            t = rms(t) * w
+        if interleaved:
+            t = _rotate_pairs(t, c, s)
+        else:
+            a, b = t[..., :half], t[..., half:rot_dim]
+            t = torch.cat([a * c - b * s, b * c + a * s, t[..., rot_dim:]], dim=-1)
+        return rms(t) if norm_after else t
+
+    ok = slot_map >= 0
+    bs = k_cache.shape[2]
+    blk, off = (slot_map[ok] // bs).long(), (slot_map[ok] % bs).long()
+    k_cache[blk, :, off] = turn(k, k_norm)[ok].to(k_cache.dtype)
+    v_cache[blk, :, off] = k[ok].to(v_cache.dtype)
+    return turn(q, q_norm).to(q.dtype)
+
+
+# ------------------------------------------------------------------ matrix-valued recurrences without a delta rule
+def token_shift(x, mu, state, state_slots, cu_q, seq_lens, out_dtype=torch.bfloat16):
+    """out[n] = x + (x' - x) mu[n], x' the row of the sequence's previous token (zeros before its first).  x fp32 [T, W], mu [n, W]; state fp32
+    [slots, W] holds the last row of what came before and gets the last row of this step.  Returns [n, T, W]."""
+    prev = torch.zeros_like(x)
+    prev[1:] = x[:-1]
+    cu = cu_q.tolist()
+    for b in range(len(cu) - 1):
+        if cu[b + 1] <= cu[b]:
+            continue
+        slot = int(state_slots[b])
+        prev[cu[b]] = 0.0 if int(seq_lens[b]) == cu[b + 1] - cu[b] else state[slot]
+        state[slot] = x[cu[b + 1] - 1]
+    return (x.unsqueeze(0) + (prev - x).unsqueeze(0) * mu.unsqueeze(1)).to(out_dtype)
+
+
+def decay_scan(q, k, v, state, state_slots, cu_q, seq_lens, max_q_len, decay=None, z=None, u=None, silu=False):
+    """Linear attention with a decaying state S [dk, dv] per head.  q, k [T, H, dk], v [T, H, dv] (any row stride); state fp32 [slots, H, dk, dv], advanced
+    in place, from zeros for a sequence whose step begins at position 0.  Returns o fp32 [T, H * dv].
+      decay [H]                        S <- decay S + k v^T, o = S^T q           (``silu``: q, k and v pass through it first)
+      z fp32 [T, H * dk], u [H, dk]    o = (S + (u k) v^T)^T q, then S <- diag(exp(-exp(z))) S + k v^T"""
+    T, H, dk = q.shape
+    q, k, v = (t.to(torch.float32) for t in (q, k, v))
+    if silu:
+        q, k, v = (torch.nn.functional.silu(t) for t in (q, k, v))
+    w = torch.exp(-torch.exp(z)).reshape(T, H, dk) if z is not None else None
+    out = torch.empty(T, H, v.shape[2], dtype=torch.float32, device=q.device)
+    cu = cu_q.tolist()
+    for b in range(len(cu) - 1):
+        t0, t1 = cu[b], cu[b + 1]
+        if t1 <= t0:
+            continue
+        slot = int(state_slots[b])
+        S = torch.zeros_like(state[slot]) if int(seq_lens[b]) == t1 - t0 else state[slot].clone()
+        for t in range(t0, t1):
+            kv = k[t].unsqueeze(-1) * v[t].unsqueeze(1)
+            if w is None:
+                S = decay.reshape(H, 1, 1) * S + kv
+                out[t] = torch.einsum("hk,hkv->hv", q[t], S)
+            else:
+                out[t] = torch.einsum("hk,hkv->hv", q[t], S + u.unsqueeze(-1) * kv)
+                S = w[t].unsqueeze(-1) * S + kv
+        state[slot] = S
+    return out.reshape(T, -1)
+
+
+def gated_group_norm(o, gate, w, eps, groups=1, width=None, silu=False, out_dtype=torch.bfloat16):
+    """norm(o) * w * act(gate): RMS norm over each of ``groups`` equal runs of a row whose first ``width`` elements (default: all) are live, the rest
+    zero; act is SiLU or the sigmoid.  o fp32 [T, W], gate [T, W] (any row stride), w [W]."""
+    T, W = o.shape
+    x = o.reshape(T, groups, W // groups)
+    n = x.shape[2] if width is None else width
+    x = (x * torch.rsqrt(x.pow(2).sum(-1, keepdim=True) / n + eps)).reshape(T, W)
+    g = gate.to(torch.float32)
+    return (x * w * (torch.nn.functional.silu(g) if silu else torch.sigmoid(g))).to(out_dtype)
+
+
+# ------------------------------------------------------------------ norms on a sublayer's output
+@dataclass
+class ExpertSum:
+    """A branch that has not been formed: the sum of the rows of a token's experts (``y`` [rows, H], row pair_to_packed[t * k + j] for its j-th) and,
+    when there is one, of ``shared`` [T, H]."""
+    y: torch.Tensor
+    pair_to_packed: torch.Tensor
+    k: int
+    shared: Optional[torch.Tensor] = None
+
+    def rows(self, idx):
+        return ExpertSum(self.y, self.pair_to_packed.view(-1, self.k).index_select(0, idx).reshape(-1), self.k,
+                         None if self.shared is None else self.shared.index_select(0, idx))
+
+    def materialize(self, eps=0.0, width=None):
+        d = self.y.to(torch.float32)[self.pair_to_packed.long()].view(-1, self.k, self.y.shape[1]).sum(1)
+        return d if self.shared is None else d + self.shared.to(torch.float32)
+
+
+@dataclass
+class BranchMean:
+    """A branch that has not been formed: the mean of two branches [T, H], each RMS-normed with its own weight first."""
+    a: torch.Tensor
+    a_w: torch.Tensor
+    b: torch.Tensor
+    b_w: torch.Tensor
+
+    def rows(self, idx):
+        return BranchMean(self.a.index_select(0, idx), self.a_w, self.b.index_select(0, idx), self.b_w)
+
+    def materialize(self, eps=0.0, width=None):
+        n = width or self.a.shape[1]
+        rms = lambda t: t.to(torch.float32) * torch.rsqrt(t.to(torch.float32).pow(2).sum(-1, keepdim=True) / n + eps)
+        return 0.5 * (rms(self.a) * self.a_w + rms(self.b) * self.b_w)
+
+
+def sublayer_norm(x, delta, delta_w, eps, w=None, width=None, out_dtype=torch.bfloat16, want_out=True):
+    """x <- x + norm(delta) * delta_w (fp32, in place; delta: a tensor, an :class:`ExpertSum`, a :class:`BranchMean`, or None); returns norm(x) * w, or
+    without ``w`` x itself, as ``out_dtype``.  Rows are padded to x.shape[1] columns (weights too, with zeros); the mean runs over ``width``."""
+    n = width or x.shape[1]
+    rms = lambda t: t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) / n + eps)
+    if delta is not None:
+        d = delta.to(torch.float32) if isinstance(delta, torch.Tensor) else delta.materialize(eps, n)
+        x += rms(d) * delta_w
+    if not want_out:
+        return None
+    return (x if w is None else rms(x) * w).to(out_dtype)
 
 
 # ------------------------------------------------------------------ latent attention
@@ -402,6 +541,11 @@ def head_linear(x, w: QuantWeight, gate=None, out=None):
         y = y * torch.sigmoid(gate.to(torch.float32)).reshape(y.shape)
     y = y.to(x.dtype)
     return y if out is None else out.copy_(y)
+
+
+def stacked_linear(x, w: QuantWeight):
+    """Every matrix of a stack with its own input: out[n] = x[n] W[n]^T.  x [n, T, K] (contiguous), w n matrices [N, K] -> [n, T, N]."""
+    return torch.einsum("ntk,nmk->ntm", x.to(_MM_DTYPE), _dense(w)).to(torch.float32).to(x.dtype)
 
 
 def latent_attention(q, cache, block_table, seq_lens, cu_q, max_q_len, rank, window=0, scale=1.0):
@@ -581,14 +725,17 @@ def deltanet_scan_chunked(qkv, n_k, ab, a_idx, b_idx, k_of_v, ssm_a, dt_bias, st
     return out.reshape(T, n_v * D)
 
 
-def moe_route(logits, bias, k, renorm=True, precise=False):
+def moe_route(logits, bias, k, renorm=True, precise=False, sigmoid=False):
+    """``sigmoid``: the weights are the sigmoids of the chosen logits, as they are."""
     x = logits.to(torch.float32)
     if bias is not None:
         x = x + bias
     # descending value, ties -> lowest index (stable sort on -x)
     order = torch.sort(-x, dim=-1, stable=True).indices[:, :k]
     sel = torch.gather(x, 1, order)
-    if renorm:
+    if sigmoid:
+        w = torch.sigmoid(sel)
+    elif renorm:
         w = torch.softmax(sel, dim=-1)
     else:
         w = torch.exp(sel - torch.logsumexp(x, dim=-1, keepdim=True))
@@ -653,6 +800,17 @@ def moe_gather(x, pk: MoePacking, f16=False):
     xp = torch.zeros(pk.max_rows, x.shape[1], dtype=torch.float16 if f16 else x.dtype, device=x.device)
     ok = pk.packed_token >= 0
     xp[ok] = x[pk.packed_token[ok].long()].to(xp.dtype)
+    return xp
+
+
+def moe_scale_rows(x, w, pk: Optional[MoePacking] = None):
+    """Rows for experts whose weight scales their input: row of pair (t, k) = w[t, k] x[t], at its packed place or, without a packing, at t * K + k."""
+    T, K = w.shape
+    rows = (x.to(torch.float32).unsqueeze(1) * w.unsqueeze(-1)).reshape(T * K, -1).to(x.dtype)
+    if pk is None:
+        return rows
+    xp = torch.zeros(pk.max_rows, x.shape[1], dtype=x.dtype, device=x.device)
+    xp[pk.pair_to_packed.long()] = rows
     return xp
 
 
