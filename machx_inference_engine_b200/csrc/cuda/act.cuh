@@ -6,8 +6,8 @@
 namespace mx {
 
 // activation codes: 0 none; 1 SwiGLU, 2 clamped SwiGLU, 3 GeGLU (gated: N columns become N / 2); 4 xIELU, 5 GELU (tanh form),
-// 6 the square of ReLU (unary)
-constexpr int ACT_CODE_XIELU = 4, ACT_CODE_GELU_TANH = 5, ACT_CODE_RELU2 = 6;
+// 6 the square of ReLU, 7 tanh (unary)
+constexpr int ACT_CODE_XIELU = 4, ACT_CODE_GELU_TANH = 5, ACT_CODE_RELU2 = 6, ACT_CODE_TANH = 7;
 __host__ __device__ constexpr bool act_gated(int act) { return act >= 1 && act <= 3; }
 
 // xIELU: a z^2 + z / 2 for z > 0, b (e^z - 1 - z) + z / 2 otherwise (a = softplus(p), b = 1/2 + softplus(q), formed by the caller).
@@ -46,6 +46,7 @@ template <bool PRECISE>
 __device__ __forceinline__ float act_unary(int act, float z, float a, float b) {
   if (act == ACT_CODE_XIELU) return xielu<PRECISE>(z, a, b);
   if (act == ACT_CODE_GELU_TANH) return gelu_tanh<PRECISE>(z);
+  if (act == ACT_CODE_TANH) return tanhf(z);
   return act == ACT_CODE_RELU2 ? relu2(z) : z;
 }
 
@@ -61,6 +62,9 @@ __device__ __forceinline__ void act_unary_run(int act, float (&v)[N], float a, f
   } else if (act == ACT_CODE_RELU2) {
 #pragma unroll
     for (int j = 0; j < N; ++j) v[j] = relu2(v[j]);
+  } else if (act == ACT_CODE_TANH) {
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] = tanhf(v[j]);
   }
 }
 

@@ -49,6 +49,8 @@ struct AttnParams {
   const float* q_scale;        // [q_scale_n] factor on the scores of a query at that position, or null
   const void* gate;            // out is multiplied by sigmoid(gate): [Tq] rows of [n_q][dv], gate_ld elements apart, or null
   int q_scale_n, q_ld, gate_ld, dk, dv;
+  int gate_heads;              // the gate has one number per head: rows of [n_q]
+  int keep_first;              // with a window: the first keys of the sequence that stay visible
   float* o_part;               // [splits][Tq][n_q][dv]
   float* ml_part;              // [splits][Tq][n_q][2]
   int* tickets;                // non-null: one counter per (batch entry, query tile, kv head) group; the last split merges
@@ -136,9 +138,10 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
   const int kv_hi = min(seq_len, pos0 + nt);
   const int kv_lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
   const int tile_lo = kv_lo / ATT_TILE, tile_hi = (kv_hi + ATT_TILE - 1) / ATT_TILE;
-  const int n_tiles = tile_hi - tile_lo;
+  const int n_keep = min((p.keep_first + ATT_TILE - 1) / ATT_TILE, tile_lo);       // kept tiles before the window's
+  const int n_tiles = n_keep + tile_hi - tile_lo;
   const int per = (n_tiles + p.n_splits - 1) / p.n_splits;
-  const int my_lo = tile_lo + split * per, my_hi = min(tile_hi, my_lo + per);
+  const int my_lo = split * per, my_hi = min(n_tiles, my_lo + per);
   // splits that own at least one key tile (n_tiles >= 1: a query always sees its own position's tile)
   const int eff = p.tickets ? (n_tiles + per - 1) / per : p.n_splits;
   if (split >= eff) return;
@@ -167,7 +170,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
     }
     for (int tile = my_lo; tile < my_hi; ++tile) {
       __syncthreads();
-      const int key0 = tile * ATT_TILE;
+      const int key0 = (tile < n_keep ? tile : tile_lo + tile - n_keep) * ATT_TILE;
       const int blk = p.block_table[(size_t)b * p.max_blocks + key0 / p.block_size];
       const size_t row0 = ((size_t)blk * p.n_kv + kvh) * p.block_size + key0 % p.block_size;
       if (EXACT && sizeof(T) == 2 && p.k_scale) {
@@ -246,7 +249,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
               const int kpos = key0 + lane + 32 * half;
               float dd = half ? d1[pi] : d0[pi];
               if (p.softcap > 0.f) dd = p.softcap * tanhf(dd / p.softcap);
-              const bool ok = pr < total_pairs && kpos < seq_len && kpos <= qpos && (p.window <= 0 || kpos > qpos - p.window);
+              const bool ok = pr < total_pairs && kpos < seq_len && kpos <= qpos && (p.window <= 0 || kpos > qpos - p.window || kpos < p.keep_first);
               sc[pi][half] = ok ? dd : -INFINITY;
             }
           }
@@ -340,7 +343,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
       const int d = lane + 32 * c;
       if (!EXACT && d >= DV) continue;
       float o = acc[c] * inv;
-      if (p.gate) o *= sigmoid_f<PRECISE>(to_f32(reinterpret_cast<const T*>(p.gate)[(size_t)(q_begin + t0 + tq) * p.gate_ld + (size_t)hq * DV + d]));
+      if (p.gate) o *= sigmoid_f<PRECISE>(to_f32(reinterpret_cast<const T*>(p.gate)[(size_t)(q_begin + t0 + tq) * p.gate_ld + (p.gate_heads ? hq : (size_t)hq * DV + d)]));
       reinterpret_cast<T*>(p.out)[r * DV + d] = from_f32<T>(o);
     }
   }
@@ -351,7 +354,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
 constexpr int CMB_COLS = 256;
 template <typename T>
 __global__ void __launch_bounds__(CMB_COLS / 2) attn_combine_kernel(const float* __restrict__ o_part, const float* __restrict__ ml_part,
-                                                                    const float* __restrict__ sinks, const T* __restrict__ gate, int gate_ld,
+                                                                    const float* __restrict__ sinks, const T* __restrict__ gate, int gate_ld, int gate_heads,
                                                                     T* __restrict__ out, int Tq, int n_q, int hd, int n_splits) {
   constexpr bool PRECISE = sizeof(T) == 4;
   pdl_prologue();
@@ -389,7 +392,8 @@ __global__ void __launch_bounds__(CMB_COLS / 2) attn_combine_kernel(const float*
   a0 *= inv;
   a1 *= inv;
   if (gate) {
-    const float2 g = load2(gate + (size_t)(r / n_q) * gate_ld + (size_t)h * hd + d);
+    const T* gr = gate + (size_t)(r / n_q) * gate_ld;
+    const float2 g = gate_heads ? make_float2(to_f32(gr[h]), to_f32(gr[h])) : load2(gr + (size_t)h * hd + d);
     a0 *= sigmoid_f<PRECISE>(g.x);
     a1 *= sigmoid_f<PRECISE>(g.y);
   }
@@ -454,6 +458,7 @@ struct AttnShape {            // what the plain entry points leave at its defaul
   const float* q_scale = nullptr;
   int q_scale_n = 0;
   int elem_f32 = 0;           // queries, cache, gate and output in fp32
+  int gate_heads = 0, keep_first = 0;
 };
 static int attention_impl(const void* q, const void* k_cache, const void* v_cache, const float* k_scale, const float* v_scale,
                           const int* block_table, const int* seq_lens, const int* cu_q, const float* sinks, void* out, float* o_part,
@@ -465,7 +470,7 @@ static int attention_impl(const void* q, const void* k_cache, const void* v_cach
   const int gqa = n_q / n_kv;
   AttnParams p;
   p.q = q; p.k_cache = k_cache; p.v_cache = v_cache;
-  p.dk = sh.dk; p.dv = sh.dv; p.q_ld = sh.q_ld; p.gate = sh.gate; p.gate_ld = sh.gate_ld; p.q_scale = sh.q_scale; p.q_scale_n = sh.q_scale_n;
+  p.dk = sh.dk; p.dv = sh.dv; p.q_ld = sh.q_ld; p.gate = sh.gate; p.gate_ld = sh.gate_ld; p.gate_heads = sh.gate_heads; p.keep_first = window > 0 ? sh.keep_first : 0; p.q_scale = sh.q_scale; p.q_scale_n = sh.q_scale_n;
   p.k_scale = k_scale; p.v_scale = k_scale ? v_scale : nullptr;
   p.block_table = block_table; p.seq_lens = seq_lens; p.cu_q = cu_q; p.o_part = o_part; p.ml_part = ml_part;
   p.B = B; p.n_q = n_q; p.n_kv = n_kv; p.max_blocks = max_blocks; p.block_size = block_size;
@@ -513,9 +518,9 @@ static int attention_impl(const void* q, const void* k_cache, const void* v_cach
   if (rc || p.tickets) return rc;
   const dim3 cgrid(Tq * n_q, (dv + CMB_COLS - 1) / CMB_COLS);
   if (sh.elem_f32)
-    launch_pdl(attn_combine_kernel<float>, cgrid, dim3(CMB_COLS / 2), 0, st, o_part, ml_part, sinks, (const float*)sh.gate, sh.gate_ld, (float*)out, Tq, n_q, dv, p.n_splits);
+    launch_pdl(attn_combine_kernel<float>, cgrid, dim3(CMB_COLS / 2), 0, st, o_part, ml_part, sinks, (const float*)sh.gate, sh.gate_ld, sh.gate_heads, (float*)out, Tq, n_q, dv, p.n_splits);
   else
-    launch_pdl(attn_combine_kernel<__nv_bfloat16>, cgrid, dim3(CMB_COLS / 2), 0, st, o_part, ml_part, sinks, (const __nv_bfloat16*)sh.gate, sh.gate_ld,
+    launch_pdl(attn_combine_kernel<__nv_bfloat16>, cgrid, dim3(CMB_COLS / 2), 0, st, o_part, ml_part, sinks, (const __nv_bfloat16*)sh.gate, sh.gate_ld, sh.gate_heads,
                (__nv_bfloat16*)out, Tq, n_q, dv, p.n_splits);
   return (int)cudaGetLastError();
 }
@@ -525,7 +530,7 @@ MX_HOST_API int mx_attention_combine(const float* o_part, const float* ml_part, 
   if (Tq <= 0) return 0;
   const float* no_sinks = nullptr;
   const __nv_bfloat16* no_gate = nullptr;
-  launch_pdl(attn_combine_kernel<__nv_bfloat16>, dim3(Tq * n_q, (dv + CMB_COLS - 1) / CMB_COLS), dim3(CMB_COLS / 2), 0, st, o_part, ml_part, no_sinks, no_gate, 0, (__nv_bfloat16*)out, Tq, n_q, dv,
+  launch_pdl(attn_combine_kernel<__nv_bfloat16>, dim3(Tq * n_q, (dv + CMB_COLS - 1) / CMB_COLS), dim3(CMB_COLS / 2), 0, st, o_part, ml_part, no_sinks, no_gate, 0, 0, (__nv_bfloat16*)out, Tq, n_q, dv,
              n_splits);
   return (int)cudaGetLastError();
 }
@@ -538,14 +543,16 @@ static AttnShape plain_shape(int n_q, int hd) {
 }
 
 // Queries [Tq] rows of [n_q][dk] (q_ld elements apart), cache pages of dk- / dv-wide rows, out [Tq][n_q][dv]; optional gate (rows of
-// [n_q][dv], gate_ld apart; out *= sigmoid(gate)) and per-position score factors q_scale [q_scale_n].  elem_f32: everything in fp32.
+// [n_q][dv], or with gate_heads of [n_q], gate_ld apart; out *= sigmoid(gate)) and per-position score factors q_scale [q_scale_n].  elem_f32: everything in
+// fp32.  With a window the first keep_first keys of a sequence stay visible.
 // o_part needs n_splits*Tq*n_q*dv floats.  Rows, widths and strides are multiples of 16 bytes.  v_cache null: a value is the first dv elements of
 // its key row.
 MX_HOST_API int mx_attention_ext(const void* q, int q_ld, const void* k_cache, const void* v_cache, const int* block_table, const int* seq_lens,
                                  const int* cu_q, const float* sinks, const void* gate, int gate_ld, const float* q_scale, int q_scale_n, void* out,
                                  float* o_part, float* ml_part, int B, int Tq, int max_q_len, int n_q, int n_kv, int dk, int dv, int max_blocks,
-                                 int block_size, int window, float scale, float softcap, int n_splits, int elem_f32, cudaStream_t st) {
+                                 int block_size, int window, int keep_first, int gate_heads, float scale, float softcap, int n_splits, int elem_f32, cudaStream_t st) {
   AttnShape sh;
+  sh.gate_heads = gate_heads; sh.keep_first = keep_first;
   sh.dk = dk; sh.dv = dv; sh.q_ld = q_ld; sh.gate = gate; sh.gate_ld = gate_ld; sh.q_scale = q_scale; sh.q_scale_n = q_scale_n; sh.elem_f32 = elem_f32;
   return attention_impl(q, k_cache, v_cache, nullptr, nullptr, block_table, seq_lens, cu_q, sinks, out, o_part, ml_part, B, Tq, max_q_len, n_q, n_kv,
                         sh, max_blocks, block_size, window, scale, softcap, n_splits, st);

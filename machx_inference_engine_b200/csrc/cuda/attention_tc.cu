@@ -41,6 +41,7 @@ struct FaParams {
   const __nv_bfloat16* gate;   // out *= sigmoid(gate): [Tq] rows of [n_q][dv], gate_ld elements apart, or null
   __nv_bfloat16* out;      // [Tq][n_q][dv]
   int q_scale_n, gate_ld, dk, dv, q_ld;
+  int gate_heads, keep_first;   // one gate number per head; with a window: the first keys that stay visible
   int n_q, n_kv, max_blocks, max_q_tiles, window;
   float scale, softcap;
   int* status;
@@ -122,7 +123,9 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
   const int kv_hi = min(seq_len, pos0 + rows);   // exclusive
   const int kv_lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
   const int tile_lo = kv_lo / BKV, tile_hi = (kv_hi + BKV - 1) / BKV;
-  const int n_tiles = tile_hi - tile_lo;
+  const int n_keep = min((p.keep_first + BKV - 1) / BKV, tile_lo);            // kept tiles before the window's
+  const int n_tiles = n_keep + tile_hi - tile_lo;
+  auto first_key = [&](int j) { return (j < n_keep ? j : tile_lo + j - n_keep) * BKV; };
 
   if (threadIdx.x == 0) {
     mbar_init(b_qfull, 1);
@@ -152,7 +155,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       bool ok = true;
       for (int j = 0; j < n_tiles && ok; ++j) {
         const uint32_t sk = j % KS, phk = (j / KS) & 1, sv = j % VS, phv = (j / VS) & 1;
-        const int key0 = (tile_lo + j) * BKV;
+        const int key0 = first_key(j);
         const int blk = p.block_table[(size_t)b * p.max_blocks + key0 / FA_PAGE];
         const int krow = key0 % FA_PAGE;
         int rblk = 0;
@@ -225,7 +228,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     const bool early = !CAP && !(qs > 0.f);
     const float c = (CAP || early) ? 1.f : qs * LOG2E;
     const float cap_c = p.softcap * LOG2E, inv_cap = CAP ? qs / p.softcap : 0.f;
-    if (p.gate && row_ok) {                        // bring the row's gate into L2 while the keys are walked
+    if (p.gate && !p.gate_heads && row_ok) {       // bring the row's gate into L2 while the keys are walked
       const __nv_bfloat16* g0 = p.gate + (size_t)(q_begin + t0 + r) * p.gate_ld + (size_t)head * p.dv;
       for (int i = 0; i < p.dv; i += 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(g0 + i));
     }
@@ -244,7 +247,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(b_sempty + 8 * sb);
-      const int key0 = (tile_lo + j) * BKV;
+      const int key0 = first_key(j);
       if (CAP) {
 #pragma unroll
         for (int i = 0; i < BKV; ++i) sv[i] = cap_c * tanh_fast(sv[i] * inv_cap);
@@ -257,7 +260,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
 #pragma unroll
         for (int i = 0; i < BKV; ++i) {
           const int kpos = key0 + i;
-          const bool keep = kpos <= qpos && kpos < seq_len && (p.window <= 0 || kpos > qpos - p.window);
+          const bool keep = kpos <= qpos && kpos < seq_len && (p.window <= 0 || kpos > qpos - p.window || kpos < p.keep_first);
           sv[i] = keep ? sv[i] : -INFINITY;
         }
       }
@@ -312,7 +315,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       if (lane == 0) mbar_arrive(b_pfull);
     }
     const int dv = p.dv;
-    const __nv_bfloat16* grow = p.gate && row_ok ? p.gate + (size_t)(q_begin + t0 + r) * p.gate_ld + (size_t)head * dv : nullptr;
+    const __nv_bfloat16* grow = p.gate && !p.gate_heads && row_ok ? p.gate + (size_t)(q_begin + t0 + r) * p.gate_ld + (size_t)head * dv : nullptr;
     // the first GPRE columns of the row's gate travel while the last PV runs (the score registers are free here)
     constexpr int GPRE = DV < 128 ? DV : 128;
     uint4 gpre[GPRE / 8];
@@ -325,7 +328,8 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     if (ok) {
       tc_fence_after();
       if (p.sinks) l += ex2_fast(p.sinks[head] * LOG2E - m);
-      const float inv = l > 0.f ? 1.f / l : 0.f;
+      float inv = l > 0.f ? 1.f / l : 0.f;
+      if (p.gate && p.gate_heads && row_ok) inv *= sigmoid_f<false>(__bfloat162float(p.gate[(size_t)(q_begin + t0 + r) * p.gate_ld + head]));
       __nv_bfloat16* orow = p.out + ((size_t)(q_begin + t0 + r) * p.n_q + head) * dv;
 #pragma unroll
       for (int cb = 0; cb < DV; cb += 32) {
@@ -446,8 +450,8 @@ static int launch_fa_split(const void* q, const FaSplit& x, const FaParams& p, i
 
 // the instance whose tiles are the key / value widths rounded up to 64, 128 or 256 columns
 static int dispatch_fa(const void* q, const void* k_cache, const void* v_cache, const FaParams& p, int B, int Tq, int n_blocks, cudaStream_t st) {
-  if (p.dk < 8 || p.dv < 8 || p.dk > 256 || p.dv > 256 || p.dk % 8 || p.dv % 8 || p.q_ld % 8 || p.gate_ld % 8) return -112;
-  if (p.gate && ((uintptr_t)p.gate & 15)) return -112;
+  if (p.dk < 8 || p.dv < 8 || p.dk > 256 || p.dv > 256 || p.dk % 8 || p.dv % 8 || p.q_ld % 8) return -112;
+  if (p.gate && !p.gate_heads && (p.gate_ld % 8 || ((uintptr_t)p.gate & 15))) return -112;
   const int a = p.dk <= 64 ? 64 : p.dk <= 128 ? 128 : 256, b = p.dv <= 64 ? 64 : p.dv <= 128 ? 128 : 256;
 #define MX_FA(DK_, DV_, CAP_) launch_fa<DK_, DV_, CAP_>(q, k_cache, v_cache, p, B, Tq, n_blocks, st)
   if (p.softcap > 0.f) {
@@ -473,20 +477,21 @@ static int dispatch_fa(const void* q, const void* k_cache, const void* v_cache, 
 using namespace mx;
 
 // Tensor-core prefill attention over pages of 128 tokens.  Queries: [Tq] rows of [n_q][dk], q_ld elements apart; out [Tq][n_q][dv];
-// optional gate (rows of [n_q][dv], gate_ld apart; out *= sigmoid(gate)) and per-position score factors q_scale [q_scale_n].  softcap > 0
+// optional gate (rows of [n_q][dv], or with gate_heads of [n_q], gate_ld apart; out *= sigmoid(gate)) and per-position score factors q_scale
+// [q_scale_n].  With a window the first keep_first keys of a sequence stay visible.  softcap > 0
 // applies cap * tanh(score / cap) to the scaled scores.  n_blocks is the number of pages in the cache tensors (their leading dimension).
 MX_HOST_API int mx_attention_prefill_tc_ext(const void* q, int q_ld, const void* k_cache, const void* v_cache, const int* block_table,
                                             const int* seq_lens, const int* cu_q, const float* sinks, const void* gate, int gate_ld,
                                             const float* q_scale, int q_scale_n, void* out, int B, int Tq, int max_q_len, int n_q, int n_kv, int dk,
-                                            int dv, int max_blocks, int n_blocks, int block_size, int window, float scale, float softcap,
-                                            cudaStream_t st) {
+                                            int dv, int max_blocks, int n_blocks, int block_size, int window, int keep_first, int gate_heads, float scale,
+                                            float softcap, cudaStream_t st) {
   if (B <= 0 || Tq <= 0) return 0;
   if (block_size != FA_PAGE) return -110;
   if (n_q % n_kv) return -111;
   FaParams p;
   p.block_table = block_table; p.rot_table = nullptr; p.seq_lens = seq_lens; p.cu_q = cu_q; p.sinks = sinks; p.out = (__nv_bfloat16*)out;
   p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate ? gate_ld : 0; p.q_scale = q_scale; p.q_scale_n = q_scale_n;
-  p.dk = dk; p.dv = dv; p.q_ld = q_ld;
+  p.dk = dk; p.dv = dv; p.q_ld = q_ld; p.gate_heads = gate_heads; p.keep_first = window > 0 ? keep_first : 0;
   p.n_q = n_q; p.n_kv = n_kv; p.max_blocks = max_blocks; p.window = window; p.scale = scale; p.softcap = softcap;
   p.max_q_tiles = (max_q_len + FA_BQ - 1) / FA_BQ;
   p.status = status_word();
@@ -500,7 +505,7 @@ MX_HOST_API int mx_attention_prefill_tc(const void* q, const void* k_cache, cons
                                         cudaStream_t st) {
   if (hd != 64 && hd != 128 && hd != 256) return -112;
   return mx_attention_prefill_tc_ext(q, n_q * hd, k_cache, v_cache, block_table, seq_lens, cu_q, sinks, nullptr, 0, nullptr, 0, out, B, Tq, max_q_len,
-                                     n_q, n_kv, hd, hd, max_blocks, n_blocks, block_size, window, scale, softcap, st);
+                                     n_q, n_kv, hd, hd, max_blocks, n_blocks, block_size, window, 0, 0, scale, softcap, st);
 }
 
 // Latent attention over expanded pages (see FaSplit).  q: [Tq] rows of [n_q][dim | rot], q_ld elements apart, rotated; kv: [n_pages * 128][n_q * (dim +
@@ -515,7 +520,7 @@ MX_HOST_API int mx_attention_prefill_latent(const void* q, int q_ld, const void*
   if (((uintptr_t)q | (uintptr_t)kv | (uintptr_t)cache | (uintptr_t)gate | (uintptr_t)out) & 15) return -112;
   FaParams p;
   p.block_table = kv_table; p.rot_table = block_table; p.seq_lens = seq_lens; p.cu_q = cu_q; p.sinks = nullptr; p.out = (__nv_bfloat16*)out;
-  p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate ? gate_ld : 0; p.q_scale = nullptr; p.q_scale_n = 0;
+  p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate ? gate_ld : 0; p.q_scale = nullptr; p.q_scale_n = 0; p.gate_heads = p.keep_first = 0;
   p.dk = dim + rot; p.dv = vdim; p.q_ld = q_ld; p.n_q = n_q; p.n_kv = n_q; p.max_blocks = max_blocks; p.window = window; p.scale = scale; p.softcap = 0.f;
   p.max_q_tiles = (max_q_len + FA_BQ - 1) / FA_BQ;
   p.status = status_word();

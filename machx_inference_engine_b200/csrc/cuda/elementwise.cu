@@ -310,6 +310,134 @@ __global__ void __launch_bounds__(GN_WARPS * 32) group_norm_kernel(const GroupNo
     }
 }
 
+// ------------------------------------------------------------------ sublayer_norm
+// Norms on a sublayer's output.  In one pass over a row, the branch d formed as it is read:
+//   x (fp32 residual) += norm(d) * delta_w          (KIND 0: x is only read)
+//   out                = x, or norm(x) * w when w is given   (out null: skipped)
+// d: a row (KIND 1); the sum of the rows pos[t * K + k] of a, k < K, and of row t of b when there is one (KIND 2: a token's experts and the expert that
+// every token uses); the mean of norm(a) * a_w and norm(b) * b_w (KIND 3: two mixers side by side).
+// Rows have ld elements (a multiple of 4) of which the first H count; the others are zero in a, b and the weights and stay zero.
+// A team of `wpg` warps owns a row and keeps NV pieces of four elements per lane; NV == 0: any width, memory is read again.
+struct SublayerNormParams {
+  float* x;
+  const void* a;
+  const void* b;
+  const int* pos;
+  const float* a_w;
+  const float* b_w;
+  const float* delta_w;
+  const float* w;
+  void* out;
+  float eps, inv_h;
+  int T, ld, K, wpg;
+};
+
+template <int KIND, typename DT, typename OT, int NV>
+__global__ void __launch_bounds__(GN_WARPS * 32) sublayer_norm_kernel(const SublayerNormParams p) {
+  pdl_prologue();
+  __shared__ float red[GN_WARPS], red2[GN_WARPS];
+  constexpr int N = NV > 0 ? NV : 1;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wpg = p.wpg;
+  const int t = blockIdx.x * (GN_WARPS / wpg) + warp / wpg;
+  if (t >= p.T) return;                                  // a whole team leaves
+  const size_t row = (size_t)t * p.ld;
+  float* xr = p.x + row;
+  const DT* ar = reinterpret_cast<const DT*>(p.a) + row;
+  const DT* br = reinterpret_cast<const DT*>(p.b) + row;
+  OT* orow = reinterpret_cast<OT*>(p.out) + row;
+  const int first = ((warp % wpg) * 32 + lane) * 4, step = wpg * 128;
+  float x[N][4], d[N][4], e2[KIND == 3 ? N : 1][4];
+
+  auto fetch = [&](int c, float (&dv)[4], float (&ev)[4]) {
+    if constexpr (KIND == 1) loadv<4>(ar + c, dv);
+    if constexpr (KIND == 2) {
+      if (p.b) loadv<4>(br + c, dv);
+      else dv[0] = dv[1] = dv[2] = dv[3] = 0.f;
+      for (int k = 0; k < p.K; ++k) {
+        float v[4];
+        loadv<4>(reinterpret_cast<const DT*>(p.a) + (size_t)p.pos[(size_t)t * p.K + k] * p.ld + c, v);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) dv[e] += v[e];
+      }
+    }
+    if constexpr (KIND == 3) { loadv<4>(ar + c, dv); loadv<4>(br + c, ev); }
+  };
+  auto mean = [&](int c, float (&dv)[4], const float (&ev)[4], float ia, float ib) {
+    float wa[4], wb[4];
+    loadv<4>(p.a_w + c, wa);
+    loadv<4>(p.b_w + c, wb);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) dv[e] = 0.5f * (dv[e] * ia * wa[e] + ev[e] * ib * wb[e]);
+  };
+  auto square = [](const float (&v)[4], float s) {
+#pragma unroll
+    for (int e = 0; e < 4; ++e) s = fmaf(v[e], v[e], s);
+    return s;
+  };
+  // every piece of the row that this lane owns: body(column, index of its registers)
+  auto each = [&](auto&& body) {
+    if constexpr (NV > 0) {
+#pragma unroll
+      for (int j = 0; j < NV; ++j)
+        if (first + j * step < p.ld) body(first + j * step, j);
+    } else {
+      for (int c = first; c < p.ld; c += step) body(c, 0);
+    }
+  };
+  float ia = 0.f, ib = 0.f, ss = 0.f;
+  if constexpr (KIND != 0) {
+    float sa = 0.f, sb = 0.f;
+    each([&](int c, int j) {
+      if (NV > 0) loadv<4>(xr + c, x[j]);
+      fetch(c, d[j], e2[KIND == 3 ? j : 0]);
+      sa = square(d[j], sa);
+      if (KIND == 3) sb = square(e2[KIND == 3 ? j : 0], sb);
+    });
+    if constexpr (KIND == 3) {
+      ia = rsqrtf(team_sum(sa, red, warp, wpg) * p.inv_h + p.eps);
+      ib = rsqrtf(team_sum(sb, red2, warp, wpg) * p.inv_h + p.eps);
+      sa = 0.f;
+      each([&](int c, int j) {
+        if (NV == 0) fetch(c, d[j], e2[j]);
+        mean(c, d[j], e2[j], ia, ib);
+        sa = square(d[j], sa);
+      });
+    }
+    const float dinv = rsqrtf(team_sum(sa, red, warp, wpg) * p.inv_h + p.eps);
+    each([&](int c, int j) {
+      if (NV == 0) {
+        loadv<4>(xr + c, x[j]);
+        fetch(c, d[j], e2[KIND == 3 ? j : 0]);
+        if constexpr (KIND == 3) mean(c, d[j], e2[j], ia, ib);
+      }
+      float wv[4];
+      loadv<4>(p.delta_w + c, wv);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) x[j][e] = fmaf(d[j][e] * dinv, wv[e], x[j][e]);
+      storev<4>(xr + c, x[j]);
+      ss = square(x[j], ss);
+    });
+  } else {
+    each([&](int c, int j) {
+      loadv<4>(xr + c, x[j]);
+      ss = square(x[j], ss);
+    });
+  }
+  if (!p.out) return;
+  const float inv = p.w ? rsqrtf(team_sum(ss, red2, warp, wpg) * p.inv_h + p.eps) : 1.f;
+  each([&](int c, int j) {
+    if (NV == 0) loadv<4>(xr + c, x[j]);                 // (a lane reads back what it wrote itself)
+    float o[4] = {x[j][0], x[j][1], x[j][2], x[j][3]};
+    if (p.w) {
+      float wv[4];
+      loadv<4>(p.w + c, wv);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) o[e] *= inv * wv[e];
+    }
+    storev<4>(orow + c, o);
+  });
+}
+
 // ------------------------------------------------------------------ dyt_norm
 // A norm without statistics: every element on its own, so a thread needs no other thread.
 //   x (fp32 residual) += delta + step;   out = tanh(alpha x) w + b
@@ -606,6 +734,135 @@ __global__ void __launch_bounds__(128) qkv_post_token_kernel(const QkvPostParams
   }
 }
 
+// ------------------------------------------------------------------ qk_post
+// Head epilogue of attention whose values are its projected keys: per-head RMS norm with a weight, rotation of the first `rot` elements (interleaved pairs or
+// half splits), optional RMS norm without a weight behind it; queries in place, keys and raw keys (the values) into the cache pages.  One warp per
+// (token, head); a lane holds groups of G consecutive elements, group g at g * 32 G.
+struct QkPostParams {
+  void* q;                     // row t of head h at t * q_ld + h * dp
+  const void* k;
+  const float* q_norm;         // [dp] or null
+  const float* k_norm;
+  const int* positions;        // [T]
+  const float* rope_cos;       // [max_pos][rot / 2]
+  const float* rope_sin;
+  const long long* slot_map;   // [T], < 0: no cache row
+  void* k_cache;               // [blocks][n_kv][block_size][dp]
+  void* v_cache;
+  int q_ld, k_ld, T, n_q, n_kv, dp, dim, rot, interleaved, norm_after, block_size, max_pos;
+  float eps;
+};
+constexpr int QK_WARPS = 4;
+
+template <int G, typename T> __device__ __forceinline__ void load_group(const T* p, float (&v)[G]) {
+  if constexpr (G == 2) { const float2 a = load2(p); v[0] = a.x; v[1] = a.y; }
+  else if constexpr (G == 4) loadv<4>(p, v);
+  else { loadv<4>(p, *reinterpret_cast<float(*)[4]>(&v[0])); loadv<4>(p + 4, *reinterpret_cast<float(*)[4]>(&v[4])); }
+}
+template <int G, typename T> __device__ __forceinline__ void store_group(T* p, const float (&v)[G]) {
+  if constexpr (G == 2) store2(p, v[0], v[1]);
+  else if constexpr (G == 4) storev<4>(p, v);
+  else { storev<4>(p, *reinterpret_cast<const float(*)[4]>(&v[0])); storev<4>(p + 4, *reinterpret_cast<const float(*)[4]>(&v[4])); }
+}
+
+template <typename T, int G, int NG>
+__global__ void __launch_bounds__(QK_WARPS * 32) qk_post_kernel(const QkPostParams p) {
+  pdl_prologue();
+  __shared__ float sh[QK_WARPS][32 * G * NG];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int heads = p.n_q + p.n_kv;
+  const long long unit = (long long)blockIdx.x * QK_WARPS + warp;
+  if (unit >= (long long)p.T * heads) return;
+  const int t = (int)(unit / heads), h = (int)(unit - (long long)t * heads);
+  const bool is_q = h < p.n_q;
+  const long long slot = is_q ? 0 : p.slot_map[t];
+  if (slot < 0) return;
+  const int dp = p.dp, kh = h - p.n_q;
+  T* qrow = reinterpret_cast<T*>(p.q) + (size_t)t * p.q_ld + (size_t)h * dp;
+  const T* src = is_q ? qrow : reinterpret_cast<const T*>(p.k) + (size_t)t * p.k_ld + (size_t)kh * dp;
+  const long long crow = is_q ? 0 : (((slot / p.block_size) * p.n_kv + kh) * p.block_size + slot % p.block_size) * dp;
+  const float* nw = is_q ? p.q_norm : p.k_norm;
+  int pos = p.positions[t];
+  pos = pos < 0 ? 0 : (pos >= p.max_pos ? p.max_pos - 1 : pos);
+  const int half = p.rot / 2;
+  const float* cs = p.rope_cos + (size_t)pos * half;
+  const float* sn = p.rope_sin + (size_t)pos * half;
+  float v[NG][G], ss = 0.f;
+#pragma unroll
+  for (int g = 0; g < NG; ++g) {
+    const int e0 = (g * 32 + lane) * G;
+    if (e0 < dp) {
+      load_group<G>(src + e0, v[g]);
+      if (!is_q) store_group<G>(reinterpret_cast<T*>(p.v_cache) + crow + e0, v[g]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < G; ++e) v[g][e] = 0.f;
+    }
+#pragma unroll
+    for (int e = 0; e < G; ++e) ss = fmaf(v[g][e], v[g][e], ss);
+  }
+  if (nw) {
+    const float inv = rsqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+#pragma unroll
+    for (int g = 0; g < NG; ++g) {
+      const int e0 = (g * 32 + lane) * G;
+      if (e0 < dp) {
+        float w[G];
+        load_group<G>(nw + e0, w);
+#pragma unroll
+        for (int e = 0; e < G; ++e) v[g][e] *= inv * w[e];
+      }
+    }
+  }
+  if (p.interleaved) {
+#pragma unroll
+    for (int g = 0; g < NG; ++g) {
+      const int e0 = (g * 32 + lane) * G;
+#pragma unroll
+      for (int e = 0; e < G; e += 2)
+        if (e0 + e < p.rot) {
+          const int i = (e0 + e) >> 1;
+          const float a = v[g][e], b = v[g][e + 1], c = __ldg(cs + i), s = __ldg(sn + i);
+          v[g][e] = a * c - b * s;
+          v[g][e + 1] = b * c + a * s;
+        }
+    }
+  } else {
+    float* buf = sh[warp];
+#pragma unroll
+    for (int g = 0; g < NG; ++g) store_group<G>(buf + (g * 32 + lane) * G, v[g]);
+    __syncwarp();
+#pragma unroll
+    for (int g = 0; g < NG; ++g) {
+      const int e0 = (g * 32 + lane) * G;
+#pragma unroll
+      for (int e = 0; e < G; ++e) {
+        const int i = e0 + e;
+        if (i < half) v[g][e] = v[g][e] * __ldg(cs + i) - buf[i + half] * __ldg(sn + i);
+        else if (i < p.rot) v[g][e] = v[g][e] * __ldg(cs + i - half) + buf[i - half] * __ldg(sn + i - half);
+      }
+    }
+  }
+  if (p.norm_after) {
+    ss = 0.f;
+#pragma unroll
+    for (int g = 0; g < NG; ++g)
+#pragma unroll
+      for (int e = 0; e < G; ++e) ss = fmaf(v[g][e], v[g][e], ss);
+    const float inv = rsqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+#pragma unroll
+    for (int g = 0; g < NG; ++g)
+#pragma unroll
+      for (int e = 0; e < G; ++e) v[g][e] *= inv;
+  }
+  T* dst = is_q ? qrow : reinterpret_cast<T*>(p.k_cache) + crow;
+#pragma unroll
+  for (int g = 0; g < NG; ++g) {
+    const int e0 = (g * 32 + lane) * G;
+    if (e0 < dp) store_group<G>(dst + e0, v[g]);
+  }
+}
+
 // ------------------------------------------------------------------ GLU over interleaved-16 columns
 __device__ __forceinline__ float glu_act(int act, float g, float u, float alpha, float limit) {
   if (act == 1) return g / (1.f + __expf(-g)) * u;
@@ -616,6 +873,20 @@ __device__ __forceinline__ float glu_act(int act, float g, float u, float alpha,
   }
   const float t = tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g));
   return 0.5f * g * (1.f + t) * u;
+}
+// (fp32 rows: SwiGLU through the full-precision exponential)
+__device__ __forceinline__ float glu_act_precise(int act, float g, float u, float alpha, float limit) {
+  return act == 1 ? g * sigmoid_f<true>(g) * u : glu_act(act, g, u, alpha, limit);
+}
+__global__ void glu_f32_kernel(const float* __restrict__ in, float* __restrict__ out, long long total_out, int F, int act, float alpha, float limit) {
+  pdl_prologue();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= total_out) return;
+  const long long t = i / F;
+  const int f = (int)(i % F);
+  const float* row = in + t * 2 * F;
+  const int g = 32 * (f >> 4) + (f & 15);
+  out[i] = glu_act_precise(act, row[g], row[g + 16], alpha, limit);
 }
 __global__ void glu_kernel(const __nv_bfloat16* __restrict__ in, __nv_bfloat16* __restrict__ out, long long total_out, int F, int act,
                            float alpha, float limit) {
@@ -764,6 +1035,62 @@ MX_HOST_API int mx_group_norm(float* x, const void* delta, int delta_is_f32, con
   return out_is_f32 ? launch_group_norm<__nv_bfloat16, float>(p, st) : launch_group_norm<__nv_bfloat16, __nv_bfloat16>(p, st);
 }
 
+namespace mx {
+template <int KIND, typename DT, typename OT>
+static int launch_sublayer_norm(SublayerNormParams p, cudaStream_t st) {
+  // enough warps per row that a lane holds at most 16 elements (32 with eight), then more while the chip has room for them
+  p.wpg = 1;
+  while (p.wpg < GN_WARPS && (p.ld > 512 * p.wpg || ((long long)p.T * p.wpg < 16ll * sm_count() && p.ld > 128 * p.wpg))) p.wpg *= 2;
+  const dim3 grid((unsigned)((p.T + GN_WARPS / p.wpg - 1) / (GN_WARPS / p.wpg))), block(GN_WARPS * 32);
+  const int pieces = (p.ld + 128 * p.wpg - 1) / (128 * p.wpg);
+  if (pieces <= 2) launch_pdl(sublayer_norm_kernel<KIND, DT, OT, 2>, grid, block, 0, st, p);
+  else if (pieces <= 4) launch_pdl(sublayer_norm_kernel<KIND, DT, OT, 4>, grid, block, 0, st, p);
+  else if (pieces <= 8) launch_pdl(sublayer_norm_kernel<KIND, DT, OT, 8>, grid, block, 0, st, p);
+  else launch_pdl(sublayer_norm_kernel<KIND, DT, OT, 0>, grid, block, 0, st, p);
+  return (int)cudaGetLastError();
+}
+template <typename DT, typename OT>
+static int dispatch_sublayer_norm(int kind, const SublayerNormParams& p, cudaStream_t st) {
+  switch (kind) {
+    case 0: return launch_sublayer_norm<0, DT, OT>(p, st);
+    case 1: return launch_sublayer_norm<1, DT, OT>(p, st);
+    case 2: return launch_sublayer_norm<2, DT, OT>(p, st);
+    default: return launch_sublayer_norm<3, DT, OT>(p, st);
+  }
+}
+}  // namespace mx
+
+// See sublayer_norm_kernel.  x fp32 [T][ld]; kind 0 nothing, 1 a row of a, 2 rows pos[t][K] of a (+ row t of b), 3 the mean of a and b normed; a and b are
+// bf16, or fp32 when out is (out null: elem_f32 names the dtype of a and b).
+MX_HOST_API int mx_sublayer_norm(int kind, float* x, const void* a, const void* b, const int* pos, int K, const float* a_w, const float* b_w, const float* delta_w,
+                                 const float* w, void* out, int elem_f32, float eps, int T, int H, int ld, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (H < 1 || ld < H || ld % 4 || kind < 0 || kind > 3) return -107;
+  if ((kind && (!a || !delta_w)) || (kind == 2 && (!pos || K < 1)) || (kind == 3 && (!b || !a_w || !b_w))) return -109;
+  SublayerNormParams p;
+  p.x = x; p.a = a; p.b = b; p.pos = pos; p.a_w = a_w; p.b_w = b_w; p.delta_w = delta_w; p.w = w; p.out = out; p.eps = eps; p.inv_h = 1.f / (float)H;
+  p.T = T; p.ld = ld; p.K = K;
+  return elem_f32 ? dispatch_sublayer_norm<float, float>(kind, p, st) : dispatch_sublayer_norm<__nv_bfloat16, __nv_bfloat16>(kind, p, st);
+}
+
+// See qk_post_kernel.  dp (the padded head width) a multiple of 8 up to 512, dim <= dp its live elements, rot <= dim even.
+MX_HOST_API int mx_qk_post(void* q, int q_ld, const void* k, int k_ld, const float* q_norm, const float* k_norm, const int* positions, const float* rope_cos,
+                           const float* rope_sin, int max_pos, const long long* slot_map, void* k_cache, void* v_cache, int T, int n_q, int n_kv, int dp, int dim,
+                           int rot, int interleaved, int norm_after, int block_size, float eps, int elem_f32, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (dp < 8 || dp > 512 || dp % 8 || dim < 1 || dim > dp || rot < 0 || rot > dim || rot % 2 || q_ld % 8 || k_ld % 8 || (((uintptr_t)q | (uintptr_t)k) & 15)) return -108;
+  QkPostParams p;
+  p.q = q; p.k = k; p.q_norm = q_norm; p.k_norm = k_norm; p.positions = positions; p.rope_cos = rope_cos; p.rope_sin = rope_sin; p.slot_map = slot_map;
+  p.k_cache = k_cache; p.v_cache = v_cache; p.q_ld = q_ld; p.k_ld = k_ld; p.T = T; p.n_q = n_q; p.n_kv = n_kv; p.dp = dp; p.dim = dim; p.rot = rot;
+  p.interleaved = interleaved; p.norm_after = norm_after; p.block_size = block_size; p.max_pos = max_pos; p.eps = eps;
+  const long long units = (long long)T * (n_q + n_kv);
+  const dim3 grid((unsigned)((units + QK_WARPS - 1) / QK_WARPS)), block(QK_WARPS * 32);
+#define MX_QK(T_)   (dp <= 64 ? launch_pdl(qk_post_kernel<T_, 2, 1>, grid, block, 0, st, p) : dp <= 128 ? launch_pdl(qk_post_kernel<T_, 4, 1>, grid, block, 0, st, p)    : dp <= 256 ? launch_pdl(qk_post_kernel<T_, 8, 1>, grid, block, 0, st, p) : launch_pdl(qk_post_kernel<T_, 8, 2>, grid, block, 0, st, p))
+  if (elem_f32) MX_QK(float); else MX_QK(__nv_bfloat16);
+#undef MX_QK
+  return (int)cudaGetLastError();
+}
+
 // See dyt_norm_kernel.  x [T][ld] fp32; delta (null: none) [T][ld], or with pair_to_packed [rows][ld] combined with cw [T][K]; step, w, b [ld];
 // out (null: skipped) [T][ld].
 MX_HOST_API int mx_dyt_norm(float* x, const void* delta, int delta_is_f32, const int* pair_to_packed, const float* cw, int K, const float* step,
@@ -849,6 +1176,14 @@ MX_HOST_API int mx_glu(const void* in, void* out, long long T, int F, int act, f
   if (total <= 0) return 0;
   if (F % 16) return -104;
   launch_pdl(glu_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, st, (const __nv_bfloat16*)in, (__nv_bfloat16*)out, total, F, act, alpha, limit);
+  return (int)cudaGetLastError();
+}
+
+MX_HOST_API int mx_glu_f32(const float* in, float* out, long long T, int F, int act, float alpha, float limit, cudaStream_t st) {
+  const long long total = T * F;
+  if (total <= 0) return 0;
+  if (F % 16) return -104;
+  launch_pdl(glu_f32_kernel, dim3((unsigned)((total + 255) / 256)), dim3(256), 0, st, in, out, total, F, act, alpha, limit);
   return (int)cudaGetLastError();
 }
 

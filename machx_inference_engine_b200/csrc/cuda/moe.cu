@@ -185,6 +185,26 @@ __global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ x, const int
   }
 }
 
+// Rows for experts whose weight scales their input: w[pair] * x[pair / K] at row pair_to_packed[pair] (null: row `pair`).
+template <typename T>
+__global__ void __launch_bounds__(128) moe_scale_rows_kernel(const T* __restrict__ x, const float* __restrict__ w, const int* __restrict__ pair_to_packed,
+                                                             T* __restrict__ xp, int H, int K) {
+  pdl_prologue();
+  const int pair = blockIdx.x;
+  const int r = pair_to_packed ? pair_to_packed[pair] : pair;
+  if (r < 0) return;
+  const float s = w[pair];
+  const T* src = x + (size_t)(pair / K) * H;
+  T* dst = xp + (size_t)r * H;
+  for (int i = threadIdx.x * 4; i < H; i += 512) {
+    float v[4];
+    loadv<4>(src + i, v);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[e] *= s;
+    storev<4>(dst + i, v);
+  }
+}
+
 // out[t][:] = (accumulate ? out : 0) + sum_k w[t,k] * yp[pair_to_packed[t,k]][:]
 template <typename YT, typename OT>
 __global__ void moe_combine_kernel(const YT* __restrict__ yp, const int* __restrict__ pair_to_packed, const float* __restrict__ w,
@@ -285,7 +305,7 @@ MX_HOST_API int mx_moe_combine_push(const void* yp, const int* pair_to_packed, c
   return (int)cudaGetLastError();
 }
 
-// precise: the softmax uses the full-precision exponential
+// renorm: see moe_route.cuh; precise: the softmax uses the full-precision exponential
 MX_HOST_API int mx_moe_route(const float* logits, const float* bias, int T, int E, int K, int renorm, int precise, int* topk_idx, float* topk_w,
                              cudaStream_t st) {
   if (T <= 0) return 0;
@@ -319,6 +339,16 @@ MX_HOST_API int mx_moe_gather(const void* x, const int* packed_token, const int*
   const int ctas = 16 * sm_count();          // most of max_rows is room for padding: the live rows are walked
   launch_pdl(moe_gather_kernel, dim3(max_rows < ctas ? max_rows : ctas), dim3(128), 0, st, (const __nv_bfloat16*)x, packed_token, num_tiles, (__nv_bfloat16*)xp, H, to_f16,
              zero_pad);
+  return (int)cudaGetLastError();
+}
+
+// See moe_scale_rows_kernel; H a multiple of 4.
+MX_HOST_API int mx_moe_scale_rows(const void* x, const float* w, const int* pair_to_packed, void* xp, int n_pairs, int H, int K, int elem_f32, cudaStream_t st) {
+  if (n_pairs <= 0) return 0;
+  if (H % 4 || K < 1) return -101;
+  using bf = __nv_bfloat16;
+  if (elem_f32) launch_pdl(moe_scale_rows_kernel<float>, dim3(n_pairs), dim3(128), 0, st, (const float*)x, w, pair_to_packed, (float*)xp, H, K);
+  else launch_pdl(moe_scale_rows_kernel<bf>, dim3(n_pairs), dim3(128), 0, st, (const bf*)x, w, pair_to_packed, (bf*)xp, H, K);
   return (int)cudaGetLastError();
 }
 

@@ -1,4 +1,5 @@
-// Router top-k for one token, executed by one warp: weights = softmax over the selected logits (renorm) or softmax over all.
+// Router top-k for one token, executed by one warp: weights = softmax over the selected logits (renorm 1), softmax over all (0)
+// or the sigmoids of the selected logits as they are (2).
 // Lane k < K ends up holding the k-th selection; E <= 1024, K <= 32.  The logits are read past L1: the caller may be the last CTA
 // of the kernel that produced them.
 #pragma once
@@ -28,7 +29,7 @@ __device__ __forceinline__ void route_token_warp(const float* __restrict__ logit
   for (int i = 0; i < 32; ++i) if (i < per) denom_all += route_exp<PRECISE>(v[i] - mx_all);
   denom_all = warp_sum(denom_all);
   float sel_sum = 0.f;
-  float my_w = 0.f; int my_e = 0;    // lane k keeps the k-th selection (K <= 32)
+  float my_w = 0.f, my_z = 0.f; int my_e = 0;    // lane k keeps the k-th selection (K <= 32)
   for (int k = 0; k < K; ++k) {
     float best = -INFINITY; int bi = 0x7fffffff;
 #pragma unroll
@@ -44,14 +45,14 @@ __device__ __forceinline__ void route_token_warp(const float* __restrict__ logit
     }
     const float pw = route_exp<PRECISE>(best - mx_all);
     sel_sum += pw;
-    if (lane == k) { my_w = pw; my_e = bi; }
+    if (lane == k) { my_w = pw; my_z = best; my_e = bi; }
 #pragma unroll
     for (int i = 0; i < 32; ++i) if (lane + 32 * i == bi) v[i] = -INFINITY;
   }
   if (lane < K) {
     topk_idx[(size_t)t * K + lane] = my_e;
     // w_copies > 1: the weight row is [w_copies][K] (a consumer that sums several partial rows per pair reads one weight per partial)
-    const float wv = my_w / (renorm ? sel_sum : denom_all);
+    const float wv = renorm == 2 ? 1.f / (1.f + expf(-my_z)) : my_w / (renorm ? sel_sum : denom_all);
     for (int c = 0; c < w_copies; ++c) topk_w[((size_t)t * w_copies + c) * K + lane] = wv;
   }
 }

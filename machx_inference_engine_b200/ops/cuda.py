@@ -12,7 +12,7 @@ from typing import Optional
 import torch
 
 from .. import _lib
-from .ref import ACT_GEGLU, ACT_NONE, ACT_SWIGLU, ACT_SWIGLU_OAI, MOE_TILE, MoePacking, act_gated, moe_max_rows
+from .ref import ACT_GEGLU, ACT_NONE, ACT_SWIGLU, ACT_SWIGLU_OAI, MOE_TILE, BranchMean, ExpertSum, MoePacking, act_gated, moe_max_rows
 from .weights import QuantWeight, WFormat
 
 _vp = C.c_void_p
@@ -158,6 +158,76 @@ def dyt_norm(x, alpha, w, b, delta=None, step=None, out_dtype=torch.bfloat16, wa
     return out
 
 
+def sublayer_norm(x, delta, delta_w, eps, w=None, width=None, out_dtype=torch.bfloat16, want_out=True):
+    T, ld = x.shape
+    kind, a, b, pos, k, aw, bw = 0, None, None, None, 0, None, None
+    if isinstance(delta, ExpertSum):
+        kind, a, b, pos, k = 2, delta.y, delta.shared, delta.pair_to_packed, delta.k
+        assert pos.numel() == T * k and pos.dtype == torch.int32
+    elif isinstance(delta, BranchMean):
+        kind, a, b, aw, bw = 3, delta.a, delta.b, delta.a_w, delta.b_w
+    elif delta is not None:
+        kind, a = 1, delta
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    assert all(v is None or (v.dtype == torch.float32 and v.numel() == ld) for v in (delta_w, w, aw, bw))
+    assert all(t is None or (t.is_contiguous() and t.dtype == out_dtype and t.shape[1] == ld and (kind == 2 or t.shape[0] == T)) for t in (a, b))
+    out = torch.empty(T, ld, dtype=out_dtype, device=x.device) if want_out else None
+    _check(_lib.cuda().mx_sublayer_norm(kind, _p(x), _p(a), _p(b), _p(pos), int(k), _p(aw), _p(bw), _p(delta_w), _p(w), _p(out),
+                                        int(out_dtype == torch.float32), C.c_float(eps), T, int(width or ld), ld, _stream()), "sublayer_norm")
+    _count()
+    return out
+
+
+def qk_post(q, k, positions, rope_cos, rope_sin, slot_map, k_cache, v_cache, dim, rot_dim, interleaved=False, q_norm=None, k_norm=None, norm_after=False,
+            eps=1e-6):
+    T, n_q, dp = q.shape
+    n_kv = k.shape[1]
+    assert q.dtype == k.dtype == k_cache.dtype == v_cache.dtype and k_cache.shape == v_cache.shape and k_cache.shape[1] == n_kv and k_cache.shape[3] == dp
+    for t in (q, k):
+        assert t.stride(2) == 1 and (t.shape[1] == 1 or t.stride(1) == dp)
+    assert rope_cos.shape[1] == rot_dim // 2 and all(n is None or n.numel() == dp for n in (q_norm, k_norm))
+    _check(_lib.cuda().mx_qk_post(_p(q), q.stride(0), _p(k), k.stride(0), _p(q_norm), _p(k_norm), _p(positions), _p(rope_cos), _p(rope_sin), rope_cos.shape[0],
+                                  _p(slot_map), _p(k_cache), _p(v_cache), T, n_q, n_kv, dp, int(dim), int(rot_dim), int(interleaved), int(norm_after),
+                                  k_cache.shape[2], C.c_float(eps), int(q.dtype == torch.float32), _stream()), "qk_post")
+    _count()
+    return q
+
+
+def token_shift(x, mu, state, state_slots, cu_q, seq_lens, out_dtype=torch.bfloat16):
+    T, W = x.shape
+    n = mu.shape[0]
+    assert x.dtype == mu.dtype == state.dtype == torch.float32 and x.is_contiguous() and mu.is_contiguous() and mu.shape[1] == state.shape[1] == W
+    out = torch.empty(n, T, W, dtype=out_dtype, device=x.device)
+    _check(_lib.cuda().mx_token_shift(_p(x), _p(mu), _p(state), _p(state_slots), _p(cu_q), _p(seq_lens), _p(out), int(out_dtype == torch.float32), T, W, n,
+                                      cu_q.numel() - 1, _stream()), "token_shift")
+    _count()
+    return out
+
+
+def decay_scan(q, k, v, state, state_slots, cu_q, seq_lens, max_q_len, decay=None, z=None, u=None, silu=False):
+    T, H, dk = q.shape
+    dv = v.shape[2]
+    assert q.dtype == k.dtype == v.dtype and state.dtype == torch.float32 and state.shape[1:] == (H, dk, dv) and k.shape == q.shape
+    for t in (q, k, v):
+        assert t.stride(2) == 1 and (H == 1 or t.stride(1) == t.shape[2])
+    assert z is None or (z.dtype == torch.float32 and z.is_contiguous() and z.shape == (T, H * dk) and u.shape == (H, dk))
+    out = torch.empty(T, H * dv, dtype=torch.float32, device=q.device)
+    _check(_lib.cuda().mx_decay_scan(_p(q), q.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), _p(z), _p(u), _p(decay), _p(state), _p(state_slots), _p(cu_q),
+                                     _p(seq_lens), _p(out), cu_q.numel() - 1, H, dk, dv, int(silu), int(q.dtype == torch.float32), _stream()), "decay_scan")
+    _count()
+    return out
+
+
+def gated_group_norm(o, gate, w, eps, groups=1, width=None, silu=False, out_dtype=torch.bfloat16):
+    T, W = o.shape
+    assert o.dtype == torch.float32 and o.is_contiguous() and gate.shape == o.shape and gate.stride(1) == 1 and gate.dtype == out_dtype and w.numel() == W
+    out = torch.empty(T, W, dtype=out_dtype, device=o.device)
+    _check(_lib.cuda().mx_gated_group_norm(_p(o), _p(gate), gate.stride(0), _p(w), _p(out), int(out_dtype == torch.float32), C.c_float(eps), T, int(groups),
+                                           W // groups, int(width or W // groups), int(silu), _stream()), "gated_group_norm")
+    _count()
+    return out
+
+
 def kv_store(k, v, slot_map, k_cache, v_cache):
     T, n_kv, bs, dk = k.shape[0], k_cache.shape[1], k_cache.shape[2], k_cache.shape[3]
     dv = v_cache.shape[3]
@@ -212,6 +282,11 @@ def rmsnorm_combine(x, w, eps, d: "CombineDelta", one_plus_w=False, delta_scale=
 
 def glu(x, act, alpha=1.702, limit=7.0):
     T, F2 = x.shape
+    if x.dtype == torch.float32:
+        out = torch.empty(T, F2 // 2, dtype=torch.float32, device=x.device)
+        _check(_lib.cuda().mx_glu_f32(_p(x), _p(out), C.c_longlong(T), F2 // 2, act, C.c_float(alpha), C.c_float(limit), _stream()), "glu")
+        _count()
+        return out
     out = torch.empty(T, F2 // 2, dtype=torch.bfloat16, device=x.device)
     _check(_lib.cuda().mx_glu(_p(x), _p(out), C.c_longlong(T), F2 // 2, act, C.c_float(alpha), C.c_float(limit), _stream()), "glu")
     _count()
@@ -402,8 +477,11 @@ def linear(x, w: QuantWeight, bias=None, act=ACT_NONE, act_alpha=1.702, act_limi
 
 def _linear_f32(x, w: QuantWeight, bias, act, act_alpha, act_limit, row_scale, out):
     """fp32 activations: the layer runs in full 32-bit on the CUDA cores (``csrc/cuda/linear_f32.cu``); dense bf16 weights only."""
-    if w.fmt != WFormat.BF16 or w.E != 1 or row_scale is not None or act_gated(act):
-        raise KernelError("32-bit linear layers take dense bf16 weights and no gated activation")
+    if w.fmt != WFormat.BF16 or w.E != 1 or row_scale is not None:
+        raise KernelError("32-bit linear layers take dense bf16 weights")
+    if act_gated(act):
+        y = glu(_linear_f32(x, w, bias, ACT_NONE, 0.0, 0.0, None, None), act, act_alpha, act_limit)
+        return y if out is None else out.copy_(y)
     assert x.is_contiguous() and x.shape[-1] == w.K
     M = x.shape[0]
     if out is None:
@@ -493,8 +571,10 @@ def grouped_linear(xp, w: QuantWeight, tile_expert, num_tiles, bias=None, act=AC
     """``out_dtype`` (bf16 / fp16 / fp32) overrides ``out_f32``; fp16 feeds a following MXFP4 GEMM without a cast."""
     P = xp.shape[0]
     if xp.dtype == torch.float32:            # 32-bit models: every row in fp32 on the CUDA cores
-        if w.fmt != WFormat.BF16 or bias is not None or act_gated(act) or out_dtype not in (None, torch.float32):
-            raise KernelError("32-bit grouped layers take bf16 weights without biases and no gated activation")
+        if w.fmt != WFormat.BF16 or bias is not None or out_dtype not in (None, torch.float32):
+            raise KernelError("32-bit grouped layers take bf16 weights without biases")
+        if act_gated(act):                   # (rows past the live tiles pass through unread)
+            return glu(grouped_linear(xp, w, tile_expert, num_tiles), act, act_alpha, act_limit)
         out = torch.empty(P, w.N, dtype=torch.float32, device=xp.device)
         _check(_lib.cuda().mx_grouped_linear_f32(_p(xp), _p(w.p0), _p(out), P, w.N, w.K, _p(tile_expert), _p(num_tiles), act, C.c_float(act_alpha),
                                                  C.c_float(act_limit), _stream()), "grouped linear_f32")
@@ -539,7 +619,7 @@ def _q_rows(q):
 
 
 def attention_prefill_tc(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks=None, window=0, scale=None, softcap=0.0, q_scale=None,
-                         gate=None):
+                         gate=None, keep_first=0):
     """tcgen05 FlashAttention (key / value widths that are multiples of 8 up to 256, page size 128, optional logit soft-cap)."""
     Tq, n_q, hd = q.shape
     n_kv, bs, dv = k_cache.shape[1], k_cache.shape[2], v_cache.shape[3]
@@ -548,7 +628,8 @@ def attention_prefill_tc(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q
     _check(_lib.cuda().mx_attention_prefill_tc_ext(_p(q), _q_rows(q), _p(k_cache), _p(v_cache), _p(block_table), _p(seq_lens), _p(cu_q), _p(sinks),
                                                    _p(gate), 0 if gate is None else gate.stride(0), _p(q_scale), 0 if q_scale is None else q_scale.numel(),
                                                    _p(out), seq_lens.numel(), Tq, int(max_q_len), n_q, n_kv, hd, dv, block_table.shape[1],
-                                                   k_cache.shape[0], bs, int(window), C.c_float(scale), C.c_float(softcap or 0.0), _stream()),
+                                                   k_cache.shape[0], bs, int(window), int(keep_first), int(gate is not None and gate.shape[1] == n_q), C.c_float(scale),
+                                                   C.c_float(softcap or 0.0), _stream()),
            "attention_prefill_tc")
     _count()
     return out
@@ -592,12 +673,12 @@ def _tc_prefill_takes(q, dk, dv, softcap, kv_scales) -> bool:
 
 
 def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks=None, window=0, scale=None, softcap=0.0, n_splits=None,
-              kv_scales=None, max_kv_len=0, q_scale=None, gate=None, v_width=0):
+              kv_scales=None, max_kv_len=0, q_scale=None, gate=None, v_width=0, keep_first=0):
     """``v_cache`` None: a value is the first ``v_width`` elements of its key row (latent cache)."""
     Tq, n_q, hd = q.shape
     n_kv, bs, dv = k_cache.shape[1], k_cache.shape[2], v_width if v_cache is None else v_cache.shape[3]
     assert k_cache.dtype == torch.int8 or (k_cache.dtype == q.dtype and (v_cache is None or v_cache.dtype == q.dtype))
-    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape == (Tq, n_q * dv))
+    assert gate is None or (gate.dtype == q.dtype and gate.stride(1) == 1 and gate.shape in ((Tq, n_q * dv), (Tq, n_q)))
     B = seq_lens.numel()
     scale = scale if scale is not None else 1.0 / math.sqrt(hd)
     assert (k_cache.dtype == torch.int8) == (kv_scales is not None)
@@ -607,7 +688,7 @@ def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks
             return attention_prefill_tc(q, dk, dv, table, seq_lens, cu_q, max_q_len, sinks=sinks, window=window, scale=scale, softcap=softcap,
                                         q_scale=q_scale, gate=gate)
         return attention_prefill_tc(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks=sinks, window=window, scale=scale,
-                                    softcap=softcap, q_scale=q_scale, gate=gate)
+                                    softcap=softcap, q_scale=q_scale, gate=gate, keep_first=keep_first)
     if n_splits is None:
         # decode-sized problems: split the KV range so that ~2 CTAs per SM exist
         ctas = B * n_kv * max(1, (max_q_len * (n_q // n_kv) + 31) // 32)
@@ -630,7 +711,7 @@ def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks
     ml_part = buf[n_splits * Tq * n_q * dv: need]
     out = torch.empty(Tq, n_q, dv, dtype=q.dtype, device=q.device)
     if kv_scales is not None:
-        assert q_scale is None and gate is None and q.is_contiguous(), "the int8 cache has no gated / position-scaled form"
+        assert q_scale is None and gate is None and not keep_first and q.is_contiguous(), "the int8 cache has no gated / position-scaled form"
         _check(_lib.cuda().mx_attention_kv8(_p(q), _p(k_cache), _p(v_cache), _p(kv_scales[0]), _p(kv_scales[1]), _p(block_table), _p(seq_lens),
                                             _p(cu_q), _p(sinks), _p(out), _p(o_part), _p(ml_part), B, Tq, int(max_q_len), n_q, n_kv, hd,
                                             block_table.shape[1], bs, int(window), C.c_float(scale), C.c_float(softcap), int(n_splits),
@@ -639,7 +720,8 @@ def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks
         _check(_lib.cuda().mx_attention_ext(_p(q), _q_rows(q), _p(k_cache), _p(v_cache), _p(block_table), _p(seq_lens), _p(cu_q), _p(sinks), _p(gate),
                                             0 if gate is None else gate.stride(0), _p(q_scale), 0 if q_scale is None else q_scale.numel(), _p(out),
                                             _p(o_part), _p(ml_part), B, Tq, int(max_q_len), n_q, n_kv, hd, dv, block_table.shape[1], bs, int(window),
-                                            C.c_float(scale), C.c_float(softcap), int(n_splits), int(q.dtype == torch.float32), _stream()), "attention")
+                                            int(keep_first), int(gate is not None and gate.shape[1] == n_q), C.c_float(scale), C.c_float(softcap), int(n_splits),
+                                            int(q.dtype == torch.float32), _stream()), "attention")
     _count(_lib.cuda().mx_attention_launches(B, int(max_q_len), n_q, n_kv))
     return out
 
@@ -677,6 +759,36 @@ def head_linear(x, w: QuantWeight, gate=None, out=None):
                                          g_ld, T, H, w.N, K, bn, _stream()), "gemm_heads")
     _count()
     return out
+
+
+STACK_GEMV_MAX_ROWS = 8      # up to this many rows in all matrices together stream their matrix each; more take the tensor-core kernel
+_stack_slots: dict = {}
+
+
+def stacked_linear(x, w: QuantWeight):
+    n, T, K = x.shape
+    assert x.is_contiguous() and w.fmt == WFormat.BF16 and (w.E, w.K) == (n, K)
+    if x.dtype == torch.float32:
+        out = torch.empty(n, T, w.N, dtype=x.dtype, device=x.device)
+        for i in range(n):
+            _linear_f32(x[i], QuantWeight(WFormat.BF16, w.N, K, 1, w.p0[i:i + 1]), None, ACT_NONE, 0.0, 0.0, None, out[i])
+        return out
+    if n * T <= STACK_GEMV_MAX_ROWS:
+        if (n, T, x.device) not in _stack_slots:
+            _stack_slots[n, T, x.device] = torch.arange(n, dtype=torch.int32, device=x.device).repeat_interleave(T).contiguous()
+        return expert_gemv(x.view(n * T, K), w, _stack_slots[n, T, x.device]).view(n, T, w.N)
+    out = torch.empty(n, T, w.N, dtype=x.dtype, device=x.device)
+    _check(_lib.cuda().mx_gemm_heads(_p(x), K, C.c_longlong(T * K), _p(w.p0), _p(out), w.N, C.c_longlong(T * w.N), _vp(0), 0, T, n, w.N, K,
+                                     _stack_bn(n, T, w.N), _stream()), "gemm_heads")
+    _count()
+    return out
+
+
+def _stack_bn(n: int, T: int, N: int) -> int:
+    rows = n * ((T + 127) // 128)
+    if T > 128:
+        return _pick_bn(rows * 128, N, wide=True)
+    return next((b for b in (128, 64, 32) if rows * ((N + b - 1) // b) >= sm_count()), 32)
 
 
 def latent_attention(q, cache, block_table, seq_lens, cu_q, max_q_len, rank, window=0, scale=1.0, n_splits=None):
@@ -758,11 +870,11 @@ def expanded_attention(q, kv, plan, cache, block_table, seq_lens, cu_q, max_q_le
 
 
 # ------------------------------------------------------------------ MoE
-def moe_route(logits, bias, k, renorm=True, precise=False):
+def moe_route(logits, bias, k, renorm=True, precise=False, sigmoid=False):
     T, E = logits.shape
     idx = torch.empty(T, k, dtype=torch.int32, device=logits.device)
     w = torch.empty(T, k, dtype=torch.float32, device=logits.device)
-    _check(_lib.cuda().mx_moe_route(_p(logits), _p(bias), T, E, k, int(renorm), int(precise), _p(idx), _p(w), _stream()), "moe_route")
+    _check(_lib.cuda().mx_moe_route(_p(logits), _p(bias), T, E, k, 2 if sigmoid else int(renorm), int(precise), _p(idx), _p(w), _stream()), "moe_route")
     _count()
     return idx, w
 
@@ -924,6 +1036,17 @@ def moe_gather(x, pk: MoePacking, f16=False, zero_pad=False):
     assert x.is_contiguous() and (x.dtype == torch.bfloat16 or (x.dtype == torch.float32 and not f16))
     xp = torch.empty(pk.max_rows, H, dtype=torch.float16 if f16 else x.dtype, device=x.device)
     _check(_lib.cuda().mx_moe_gather(_p(x), _p(pk.packed_token), _p(pk.num_tiles), _p(xp), H * (x.element_size() // 2), pk.max_rows, int(f16), int(zero_pad), _stream()), "moe_gather")
+    _count()
+    return xp
+
+
+def moe_scale_rows(x, w, pk: Optional[MoePacking] = None):
+    T, K = w.shape
+    H = x.shape[1]
+    assert x.is_contiguous() and x.shape[0] == T and w.dtype == torch.float32 and w.is_contiguous()
+    xp = torch.empty(T * K if pk is None else pk.max_rows, H, dtype=x.dtype, device=x.device)
+    _check(_lib.cuda().mx_moe_scale_rows(_p(x), _p(w), _p(None if pk is None else pk.pair_to_packed), _p(xp), T * K, H, K, int(x.dtype == torch.float32),
+                                         _stream()), "moe_scale_rows")
     _count()
     return xp
 
