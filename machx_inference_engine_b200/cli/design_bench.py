@@ -1,6 +1,6 @@
 """Throughput of a layer-list design beside the framework's closest models at equal size, and its kernels beside the like kernels.
 
-    python bench.py --design tikarax|pubodra [--design-part models|kernels|all]
+    python bench.py --design tikarax|pubodra|beputar [--design-part models|kernels|all]
 
 Models (random-init bf16 weights, random tokens): prefill of one 4096-token prompt and decode at a 2048-token context for 1, 8 and 32
 sequences, through ``LLMEngine`` (CUDA graphs as in serving), for
@@ -8,6 +8,8 @@ sequences, through ``LLMEngine`` (CUDA graphs as in serving), for
             width, heads and parameters per layer (gated feed-forward of 2/3 the width); a DeltaNet hybrid (qwen35) of the same width
   pubodra:  the design with dense feed-forwards, with experts in every other layer, and with experts in every layer; a llama of the same width,
             heads, sliding window and parameters per layer; a qwen3moe with the same experts (gated, 2/3 the width) in every layer
+  beputar:  the design (parallel, attention and wkv layers in turn) with dense feed-forwards, and with experts in every layer but the first; the DeltaNet
+            hybrids of the same width, heads and parameters per feed-forward (qwen35: gated, 2/3 the width; qwen35moe: the same experts and shared expert)
 Weights are larger than L2 (126 MB), so every pass streams them.
 
 Kernels: device time inside a CUDA graph over buffers that together exceed L2, as a fraction of the roofline (bytes over the measured copy
@@ -22,7 +24,7 @@ import time
 
 import torch
 
-from ..formats.model_config import ModelConfig, _pubodra_preset, _tikarax_preset
+from ..formats.model_config import ModelConfig, _beputar_preset, _pubodra_preset, _tikarax_preset
 
 LAYERS = 8
 SIZES = {"tikarax": {  # hidden, heads, kv_heads, head width, un-gated feed-forward, minGRU width
@@ -31,6 +33,9 @@ SIZES = {"tikarax": {  # hidden, heads, kv_heads, head width, un-gated feed-forw
 }, "pubodra": {       # hidden, heads, unrotated / rotated / value widths, latent, window, un-gated feed-forward; experts, per token, their width
     "1b-layers": dict(hidden=2048, heads=16, dim=128, rot=64, vdim=128, rank=512, window=1024, ffn=12288, experts=64, used=6, eff=1536),
     "8b-layers": dict(hidden=4096, heads=32, dim=128, rot=64, vdim=128, rank=512, window=4096, ffn=21504, experts=64, used=6, eff=2304),
+}, "beputar": {       # hidden, heads, kv_heads, head width, window, kept first; lightning heads of 128, wkv heads of 64; un-gated feed-forward; experts ...
+    "1b-layers": dict(layers=9, hidden=2048, heads=32, kv_heads=8, dim=64, window=1024, keep=16, lin=16, wkv=32, ffn=12288, experts=64, used=6, eff=1024, shared=2048),
+    "8b-layers": dict(layers=9, hidden=4096, heads=32, kv_heads=8, dim=128, window=4096, keep=16, lin=32, wkv=64, ffn=21504, experts=64, used=6, eff=1536, shared=3072),
 }}
 VOCAB = 32768
 PREFILL, CONTEXT, DECODE = 4096, 2048, 64
@@ -55,6 +60,17 @@ def _pubodra_configs(s: dict) -> dict:
             "qwen3moe": ModelConfig(arch="qwen3moe", ffn=s["ffn"] * 2 // 3, n_experts=s["experts"], n_experts_used=s["used"], expert_ffn=s["eff"] * 2 // 3, **common)}
 
 
+def _beputar_configs(s: dict) -> dict:
+    bp = lambda *moe: _beputar_preset(s["hidden"], s["layers"], s["heads"], s["kv_heads"], s["dim"], s["window"], s["keep"], s["lin"], 128, 128, s["wkv"], 64, 64, s["ffn"],
+                                      VOCAB, *moe)
+    common = dict(n_layers=s["layers"], hidden=s["hidden"], n_heads=s["heads"], n_kv_heads=s["kv_heads"], ffn=s["ffn"] * 2 // 3, vocab=VOCAB, ctx_train=16384,
+                  head_dim=s["dim"], n_rot=s["dim"] // 2, full_attn_interval=3, ssm_inner=s["lin"] * 128, ssm_state=128, ssm_n_k_heads=s["lin"] // 2,
+                  ssm_n_v_heads=s["lin"], ssm_conv_kernel=4)
+    return {"beputar, dense": bp(), "qwen35 hybrid": ModelConfig(arch="qwen35", **common),
+            "beputar, experts": bp(s["experts"], s["used"], s["eff"], s["shared"]),
+            "qwen35moe hybrid": ModelConfig(arch="qwen35moe", n_experts=s["experts"], n_experts_used=s["used"], expert_ffn=s["eff"], shared_expert_ffn=s["shared"], **common)}
+
+
 def _timed(fn) -> float:
     e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
     torch.cuda.synchronize()
@@ -70,9 +86,9 @@ def bench_models(design, dev, emit) -> None:
     from ..ops import cuda as K
     from ..runtime.engine import EngineOptions, LLMEngine, SamplingParams
     for size, s in SIZES[design].items():
-        for name, cfg in {"tikarax": _tikarax_configs, "pubodra": _pubodra_configs}[design](s).items():
+        for name, cfg in {"tikarax": _tikarax_configs, "pubodra": _pubodra_configs, "beputar": _beputar_configs}[design](s).items():
             model = build_model(cfg, dev, quant="bf16", max_ctx=PREFILL + 256)
-            row = {"size": size, "model": name, "layers": LAYERS, "weight_gb": round(model.weight_bytes() / 1e9, 2)}
+            row = {"size": size, "model": name, "layers": cfg.n_layers, "weight_gb": round(model.weight_bytes() / 1e9, 2)}
             g = torch.Generator().manual_seed(0)
             prompt = lambda n: torch.randint(0, VOCAB, (n,), generator=g).tolist()
             eng = LLMEngine(model, EngineOptions(max_ctx=PREFILL + 256, max_batch_tokens=PREFILL, max_seqs=1, enable_prefix_cache=False))
@@ -362,6 +378,118 @@ def bench_kernels_pubodra(dev, emit) -> None:
     K.check_status()
 
 
+def bench_kernels_beputar(dev, emit) -> None:
+    from ..ops import cuda as K
+    from ..ops import ref
+    from ..ops.weights import QuantWeight, WFormat
+    from ..utils.rope import rope_tables
+    t = _Rows(dev, emit)
+    bf, i32, bufs, row = t.bf, t.i32, t.bufs, t.row
+    mats = lambda n, k, e=1: [QuantWeight(WFormat.BF16, n, k, e, (torch.randn(e, n, k, device=dev) * k ** -0.5).to(torch.bfloat16)) for _ in range(bufs(e * n * k * 2))]
+    f32 = lambda *sh: torch.randn(*sh, device=dev)
+    for size, s in SIZES["beputar"].items():
+        H, nq, nkv, d, win, keep, lin, wkv = s["hidden"], s["heads"], s["kv_heads"], s["dim"], s["window"], s["keep"], s["lin"], s["wkv"]
+        E, top, ef = s["experts"], s["used"], s["eff"]
+        for T in (1, 32, PREFILL):
+            # ---- norms on a sublayer's output
+            nb = bufs(T * H * 12) if T > 64 else 8
+            xs, ds, w = [f32(T, H) for _ in range(nb)], [bf(T, H) for _ in range(nb)], torch.ones(H, device=dev)
+            by = T * H * (4 + 4 + 2 + 2)
+            row(f"sublayer_norm (branch norm + add) T={T} H={H}", "new", [lambda x=x, q=q: K.sublayer_norm(x, q, w, 1e-6) for x, q in zip(xs, ds)], by)
+            row(f"sublayer_norm of two normed branches T={T} H={H}", "new",
+                [lambda x=x, q=q, r=r: K.sublayer_norm(x, ref.BranchMean(q, w, r, w), w, 1e-6) for x, q, r in zip(xs, ds, ds[1:] + ds[:1])], by + T * H * 2)
+            row(f"rmsnorm (add + norm) T={T} H={H}", "like", [lambda x=x, q=q: K.rmsnorm(x, w, 1e-6, delta=q) for x, q in zip(xs, ds)], by)
+            ys, pos, cw = [bf(T * top, H) for _ in range(nb)], torch.randperm(T * top, device=dev).to(torch.int32), torch.rand(T, top, device=dev)
+            by = T * H * (4 + 4 + 2 + 2 * top)
+            row(f"sublayer_norm of {top} experts + shared T={T} H={H}", "new",
+                [lambda x=x, y=y, q=q: K.sublayer_norm(x, ref.ExpertSum(y, pos, top, q), w, 1e-6) for x, y, q in zip(xs, ys, ds)], by + T * H * 2)
+            row(f"rmsnorm_combine of {top} T={T} H={H}", "like", [lambda x=x, y=y: K.rmsnorm_combine(x, w, 1e-6, K.CombineDelta(y, pos, cw)) for x, y in zip(xs, ys)], by)
+            del ds, ys
+            # ---- expert rows
+            h, idx = bf(T, H), torch.stack([torch.randperm(E, device=dev)[:top] for _ in range(T)]).to(torch.int32)
+            pk = K.moe_pack(idx, E)
+            hs = [bf(T, H) for _ in range(nb)]
+            row(f"moe_scale_rows T={T} x {top}", "new", [lambda x=x: K.moe_scale_rows(x, cw, pk) for x in hs], T * H * 2 * (1 + top))
+            row(f"moe_gather T={T} x {top}", "like", [lambda x=x: K.moe_gather(x, pk) for x in hs], T * H * 2 * (1 + top))
+            z = f32(T, E)
+            row(f"moe_route, sigmoid T={T} {top} of {E}", "new", [lambda: K.moe_route(z, None, top, sigmoid=True)], T * (E + 2 * top) * 4)
+            row(f"moe_route, softmax T={T} {top} of {E}", "like", [lambda: K.moe_route(z, None, top)], T * (E + 2 * top) * 4)
+            # ---- projections: the four of a wkv layer over their own inputs
+            N = wkv * 64
+            st, x4 = mats(N, H, 4), bf(4, T, H)
+            row(f"four projections of four inputs T={T} {N}x{H}", "new", [lambda m=m: K.stacked_linear(x4, m) for m in st], 4 * N * H * 2 + 4 * T * (H + N) * 2, 8.0 * T * N * H)
+            del st
+            pl = mats(4 * N, H)
+            row(f"plain projection T={T} {4 * N}x{H}", "like", [lambda m=m: K.linear(h, m) for m in pl], 4 * N * H * 2 + T * (H + 4 * N) * 2, 8.0 * T * N * H)
+            del pl
+            # ---- head epilogue
+            cos, sin = rope_tables(2 * PREFILL, d, 1e4, device=dev)
+            cosh, sinh = rope_tables(2 * PREFILL, d // 2, 1e4, device=dev)
+            pages, bs = T // 128 + 2, 128
+            slots, pos1 = torch.arange(128, 128 + T, dtype=torch.int64, device=dev), torch.arange(T, dtype=torch.int32, device=dev)
+            kc, vc = torch.zeros(pages, nkv, bs, d, dtype=torch.bfloat16, device=dev), torch.zeros(pages, nkv, bs, d, dtype=torch.bfloat16, device=dev)
+            ys, nw = [bf(T, (nq + 2 * nkv) * d) for _ in range(min(8, bufs(T * nq * d * 4) if T > 64 else 8))], torch.ones(d, device=dev)
+            q_, k_ = (lambda y: y[:, :nq * d].view(T, nq, d)), (lambda y: y[:, nq * d:(nq + nkv) * d].view(T, nkv, d))
+            by = T * (nq * d * 4 + nkv * d * 6)
+            row(f"qk_post, norm then half splits T={T}", "new",
+                [lambda y=y: K.qk_post(q_(y), k_(y), pos1, cosh, sinh, slots, kc, vc, d, d // 2, q_norm=nw, k_norm=nw) for y in ys], by)
+            row(f"qk_post, pairs then norm T={T}", "new",
+                [lambda y=y: K.qk_post(q_(y), k_(y), pos1, cos, sin, slots, kc, vc, d, d, interleaved=True, norm_after=True) for y in ys], by)
+            row(f"qkv_post, norm T={T}", "like", [lambda y=y: K.qkv_post(y, None, nw, nw, pos1, cos, sin, slots, kc, vc, nq, nkv, d, d) for y in ys], by + T * nkv * d * 2)
+            del ys, kc, vc
+        # ---- recurrences and what is around them
+        for B, n in ((1, PREFILL), (8, 512), (1, 1), (32, 1)):
+            T = B * n
+            slots, cu, sl = i32(list(range(B))), i32([i * n for i in range(B + 1)]), i32([n + 64] * B)
+            nb = bufs(T * H * 8) if T > 64 else 8
+            xs, mu, sh = [f32(T, H) for _ in range(nb)], torch.rand(5, H, device=dev), torch.zeros(B, H, device=dev)
+            row(f"token_shift B={B} n={n} 5 mixes of {H}", "new", [lambda x=x: K.token_shift(x, mu, sh, slots, cu, sl) for x in xs], T * H * 14 + B * H * 8)
+            C = 2 * lin * 128
+            xc, cwt, cst = [bf(T, C) for _ in range(nb)], f32(C, 4), torch.zeros(B, 3, C, dtype=torch.bfloat16, device=dev)
+            row(f"conv1d_silu B={B} n={n} C={C}", "like", [lambda x=x: K.conv1d_silu(x, cwt, cst, slots, cu, n) for x in xc], T * C * 4 + B * 3 * C * 4)
+            W = wkv * 64
+            r4, z, u, S = [bf(4, T, W) for _ in range(nb)], -2.0 + f32(T, W), f32(wkv, 64), torch.zeros(B, wkv, 64, 64, device=dev)
+            hd = lambda y: y.view(T, wkv, 64)
+            row(f"decay_scan, wkv B={B} n={n} {wkv} heads of 64", "new",
+                [lambda y=y: K.decay_scan(hd(y[0]), hd(y[1]), hd(y[2]), S, slots, cu, sl, n, z=z, u=u) for y in r4], T * W * (6 + 4 + 4) + 2 * S.numel() * 4)
+            W2 = lin * 128
+            y4, dec, S2 = [bf(T, 4 * W2) for _ in range(nb)], torch.linspace(0.5, 0.999, lin, device=dev), torch.zeros(B, lin, 128, 128, device=dev)
+            cut = lambda y, i: y[:, i * W2:(i + 1) * W2].view(T, lin, 128)
+            row(f"decay_scan, lightning B={B} n={n} {lin} heads of 128", "new",
+                [lambda y=y: K.decay_scan(cut(y, 0), cut(y, 1), cut(y, 2), S2, slots, cu, sl, n, decay=dec, silu=True) for y in y4], T * W2 * (6 + 4) + 2 * S2.numel() * 4)
+            nv, nk = lin, lin // 2
+            ab, ai, S3 = bf(T, 2 * nv), i32(list(range(nv))), torch.zeros(B, nv, 128, 128, device=dev)
+            kv, sa = (ai // 2).to(torch.int32), -torch.rand(nv, device=dev)
+            row(f"deltanet_scan B={B} n={n} heads={nk}/{nv}", "like",
+                [lambda x=x: K.deltanet_scan(x, nk, ab, ai, ai + nv, kv, sa, sa, S3, slots, cu, nv) for x in xc], T * C * 2 + T * nv * 128 * 4 + 2 * S3.numel() * 4)
+            os_, g, w = [f32(T, W2) for _ in range(nb)], bf(T, W2), torch.ones(W2, device=dev)
+            by = T * W2 * (4 + 2 + 2)
+            row(f"gated_group_norm, one group T={T} W={W2}", "new", [lambda o=o: K.gated_group_norm(o, g, w, 1e-6) for o in os_], by)
+            row(f"gated_group_norm, groups of 64 T={T} W={W2}", "new", [lambda o=o: K.gated_group_norm(o, g, w, 1e-6, groups=W2 // 64, silu=True) for o in os_], by)
+            row(f"gated_rmsnorm_heads T={T} W={W2}", "like", [lambda o=o: K.gated_rmsnorm_heads(o, g, w[:128], 1e-6, 128) for o in os_], by)
+            del xs, xc, r4, y4, os_
+            torch.cuda.empty_cache()
+        # ---- attention
+        for B, n, ctx in ((1, PREFILL, PREFILL), (1, 512, PREFILL), (1, 1, 8192), (1, 1, 2048), (32, 1, 2048), (32, 1, 8192)):
+            T, nblk = B * n, (ctx + 127) // 128
+            pages, live = B * nblk + 1, min(ctx, win + n)
+            nb = min(16, bufs(B * live * nkv * d * 4)) if n == 1 else 2
+            kc, vc = [bf(pages, nkv, 128, d) for _ in range(nb)], [bf(pages, nkv, 128, d) for _ in range(nb)]
+            bt = torch.arange(1, pages, dtype=torch.int32, device=dev).reshape(B, nblk)
+            sl, cu = i32([ctx] * B), i32([i * n for i in range(B + 1)])
+            q, g, sink = bf(T, nq, d), bf(T, 40), torch.zeros(nq, device=dev)
+            seen = lambda kept: float(sum(min(p + 1, win + kept) for p in range(ctx - n, ctx)))
+            by, fl = B * live * nkv * d * 4 + T * nq * d * 4, 4.0 * B * nq * d
+            kw = dict(window=win, scale=d ** -0.5)
+            row(f"attention + kept {keep} + head gate + zero sink B={B} n={n} ctx={ctx} window={win} {nq}/{nkv}x{d}", "new",
+                [lambda k=k, v=v: K.attention(q, k, v, bt, sl, cu, n, sinks=sink, keep_first=keep, gate=g[:, :nq], **kw) for k, v in zip(kc, vc)], by, fl * seen(keep))
+            row(f"attention B={B} n={n} ctx={ctx} window={win} {nq}/{nkv}x{d}", "like", [lambda k=k, v=v: K.attention(q, k, v, bt, sl, cu, n, **kw) for k, v in zip(kc, vc)],
+                by, fl * seen(0))
+            del kc, vc
+            torch.cuda.empty_cache()
+    K.check_status()
+
+
 def main(design: str, part: str = "all") -> int:
     dev = torch.device("cuda:0")
     torch.cuda.set_device(dev)
@@ -373,6 +501,6 @@ def main(design: str, part: str = "all") -> int:
     if part in ("all", "models"):
         bench_models(design, dev, emit)
     if part in ("all", "kernels"):
-        {"tikarax": bench_kernels_tikarax, "pubodra": bench_kernels_pubodra}[design](dev, emit)
+        {"tikarax": bench_kernels_tikarax, "pubodra": bench_kernels_pubodra, "beputar": bench_kernels_beputar}[design](dev, emit)
     emit({"design_bench": "done", "seconds": round(time.time() - t0, 1)})
     return 0

@@ -736,8 +736,8 @@ __global__ void __launch_bounds__(128) qkv_post_token_kernel(const QkvPostParams
 
 // ------------------------------------------------------------------ qk_post
 // Head epilogue of attention whose values are its projected keys: per-head RMS norm with a weight, rotation of the first `rot` elements (interleaved pairs or
-// half splits), optional RMS norm without a weight behind it; queries in place, keys and raw keys (the values) into the cache pages.  One warp per
-// (token, head); a lane holds groups of G consecutive elements, group g at g * 32 G.
+// half splits), optional RMS norm without a weight behind it; queries in place, keys and raw keys (the values) into the cache pages.  A warp holds a head, a
+// lane groups of G consecutive elements of it, group g at g * 32 G.
 struct QkPostParams {
   void* q;                     // row t of head h at t * q_ld + h * dp
   const void* k;
@@ -749,7 +749,7 @@ struct QkPostParams {
   const long long* slot_map;   // [T], < 0: no cache row
   void* k_cache;               // [blocks][n_kv][block_size][dp]
   void* v_cache;
-  int q_ld, k_ld, T, n_q, n_kv, dp, dim, rot, interleaved, norm_after, block_size, max_pos;
+  int q_ld, k_ld, T, n_q, n_kv, dp, dim, rot, interleaved, norm_after, block_size, max_pos, hpw;
   float eps;
 };
 constexpr int QK_WARPS = 4;
@@ -765,101 +765,130 @@ template <int G, typename T> __device__ __forceinline__ void store_group(T* p, c
   else { storev<4>(p, *reinterpret_cast<const float(*)[4]>(&v[0])); storev<4>(p + 4, *reinterpret_cast<const float(*)[4]>(&v[4])); }
 }
 
+// A warp takes `hpw` heads of one token (1 for few tokens; then the rotation's factors are fetched once per warp and the next head's row travels while
+// this one is worked on).
 template <typename T, int G, int NG>
 __global__ void __launch_bounds__(QK_WARPS * 32) qk_post_kernel(const QkPostParams p) {
   pdl_prologue();
-  __shared__ float sh[QK_WARPS][32 * G * NG];
+  __shared__ float sh[QK_WARPS][NG == 1 ? 32 * G : 32 * G * NG];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int heads = p.n_q + p.n_kv;
+  const int heads = p.n_q + p.n_kv, per_tok = (heads + p.hpw - 1) / p.hpw;
   const long long unit = (long long)blockIdx.x * QK_WARPS + warp;
-  if (unit >= (long long)p.T * heads) return;
-  const int t = (int)(unit / heads), h = (int)(unit - (long long)t * heads);
-  const bool is_q = h < p.n_q;
-  const long long slot = is_q ? 0 : p.slot_map[t];
-  if (slot < 0) return;
-  const int dp = p.dp, kh = h - p.n_q;
-  T* qrow = reinterpret_cast<T*>(p.q) + (size_t)t * p.q_ld + (size_t)h * dp;
-  const T* src = is_q ? qrow : reinterpret_cast<const T*>(p.k) + (size_t)t * p.k_ld + (size_t)kh * dp;
-  const long long crow = is_q ? 0 : (((slot / p.block_size) * p.n_kv + kh) * p.block_size + slot % p.block_size) * dp;
-  const float* nw = is_q ? p.q_norm : p.k_norm;
+  if (unit >= (long long)p.T * per_tok) return;
+  const int t = (int)(unit / per_tok), h0 = (int)(unit - (long long)t * per_tok);            // heads h0, h0 + per_tok, ...
+  const int dp = p.dp, half = p.rot / 2;
+  const long long slot = p.slot_map[t];
   int pos = p.positions[t];
   pos = pos < 0 ? 0 : (pos >= p.max_pos ? p.max_pos - 1 : pos);
-  const int half = p.rot / 2;
   const float* cs = p.rope_cos + (size_t)pos * half;
   const float* sn = p.rope_sin + (size_t)pos * half;
-  float v[NG][G], ss = 0.f;
+  // element i turns into v_i c_i + v_partner s_i
+  float c[NG][G], s[NG][G];
 #pragma unroll
-  for (int g = 0; g < NG; ++g) {
-    const int e0 = (g * 32 + lane) * G;
-    if (e0 < dp) {
-      load_group<G>(src + e0, v[g]);
-      if (!is_q) store_group<G>(reinterpret_cast<T*>(p.v_cache) + crow + e0, v[g]);
-    } else {
+  for (int g = 0; g < NG; ++g)
 #pragma unroll
-      for (int e = 0; e < G; ++e) v[g][e] = 0.f;
+    for (int e = 0; e < G; ++e) {
+      const int i = (g * 32 + lane) * G + e;
+      const bool first = p.interleaved ? !(i & 1) : i < half;
+      const int f = p.interleaved ? i >> 1 : first ? i : i - half;
+      c[g][e] = i < p.rot ? __ldg(cs + f) : 1.f;
+      s[g][e] = i < p.rot ? (first ? -__ldg(sn + f) : __ldg(sn + f)) : 0.f;
     }
-#pragma unroll
-    for (int e = 0; e < G; ++e) ss = fmaf(v[g][e], v[g][e], ss);
-  }
-  if (nw) {
-    const float inv = rsqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+  const bool by_shuffle = NG == 1 && half % G == 0;                      // a lane's partners sit in one other lane
+  const int partner = lane * G < half ? lane + half / G : lane - half / G;
+  auto source = [&](int h) {
+    return h < p.n_q ? reinterpret_cast<const T*>(p.q) + (size_t)t * p.q_ld + (size_t)h * dp
+                     : reinterpret_cast<const T*>(p.k) + (size_t)t * p.k_ld + (size_t)(h - p.n_q) * dp;
+  };
+  float next[NG][G];
+  auto fetch = [&](int h) {
+    const T* src = source(h);
 #pragma unroll
     for (int g = 0; g < NG; ++g) {
       const int e0 = (g * 32 + lane) * G;
-      if (e0 < dp) {
-        float w[G];
-        load_group<G>(nw + e0, w);
+      if (e0 < dp) load_group<G>(src + e0, next[g]);
+      else {
 #pragma unroll
-        for (int e = 0; e < G; ++e) v[g][e] *= inv * w[e];
+        for (int e = 0; e < G; ++e) next[g][e] = 0.f;
       }
     }
-  }
-  if (p.interleaved) {
+  };
+  fetch(h0);
+  for (int h = h0; h < heads; h += per_tok) {
+    const bool is_q = h < p.n_q;
+    if (!is_q && slot < 0) break;                                        // (key heads come last)
+    const int kh = h - p.n_q;
+    const long long crow = is_q ? 0 : (((slot / p.block_size) * p.n_kv + kh) * p.block_size + slot % p.block_size) * dp;
+    float v[NG][G], ss = 0.f;
 #pragma unroll
     for (int g = 0; g < NG; ++g) {
       const int e0 = (g * 32 + lane) * G;
 #pragma unroll
-      for (int e = 0; e < G; e += 2)
-        if (e0 + e < p.rot) {
-          const int i = (e0 + e) >> 1;
-          const float a = v[g][e], b = v[g][e + 1], c = __ldg(cs + i), s = __ldg(sn + i);
-          v[g][e] = a * c - b * s;
-          v[g][e + 1] = b * c + a * s;
-        }
+      for (int e = 0; e < G; ++e) { v[g][e] = next[g][e]; ss = fmaf(v[g][e], v[g][e], ss); }
+      if (!is_q && e0 < dp) store_group<G>(reinterpret_cast<T*>(p.v_cache) + crow + e0, v[g]);
     }
-  } else {
-    float* buf = sh[warp];
+    if (h + per_tok < heads) fetch(h + per_tok);
+    const float* nw = is_q ? p.q_norm : p.k_norm;
+    if (nw) {
+      const float inv = rsqrtf(warp_sum(ss) / (float)p.dim + p.eps);
 #pragma unroll
-    for (int g = 0; g < NG; ++g) store_group<G>(buf + (g * 32 + lane) * G, v[g]);
-    __syncwarp();
+      for (int g = 0; g < NG; ++g) {
+        const int e0 = (g * 32 + lane) * G;
+        if (e0 < dp) {
+          float w[G];
+          load_group<G>(nw + e0, w);
 #pragma unroll
-    for (int g = 0; g < NG; ++g) {
-      const int e0 = (g * 32 + lane) * G;
+          for (int e = 0; e < G; ++e) v[g][e] *= inv * w[e];
+        }
+      }
+    }
+    if (p.interleaved) {
+#pragma unroll
+      for (int g = 0; g < NG; ++g)
+#pragma unroll
+        for (int e = 0; e < G; e += 2) {
+          const float a = v[g][e], b = v[g][e + 1];
+          v[g][e] = fmaf(b, s[g][e], a * c[g][e]);
+          v[g][e + 1] = fmaf(a, s[g][e + 1], b * c[g][e + 1]);
+        }
+    } else if (by_shuffle) {
 #pragma unroll
       for (int e = 0; e < G; ++e) {
-        const int i = e0 + e;
-        if (i < half) v[g][e] = v[g][e] * __ldg(cs + i) - buf[i + half] * __ldg(sn + i);
-        else if (i < p.rot) v[g][e] = v[g][e] * __ldg(cs + i - half) + buf[i - half] * __ldg(sn + i - half);
+        const float o = __shfl_sync(0xffffffffu, v[0][e], partner & 31);
+        v[0][e] = fmaf(o, s[0][e], v[0][e] * c[0][e]);
       }
+    } else {
+      float* buf = sh[warp];
+      __syncwarp();
+#pragma unroll
+      for (int g = 0; g < NG; ++g) store_group<G>(buf + (g * 32 + lane) * G, v[g]);
+      __syncwarp();
+#pragma unroll
+      for (int g = 0; g < NG; ++g)
+#pragma unroll
+        for (int e = 0; e < G; ++e) {
+          const int i = (g * 32 + lane) * G + e;
+          if (i < p.rot) v[g][e] = fmaf(buf[i < half ? i + half : i - half], s[g][e], v[g][e] * c[g][e]);
+        }
     }
-  }
-  if (p.norm_after) {
-    ss = 0.f;
+    if (p.norm_after) {
+      ss = 0.f;
 #pragma unroll
-    for (int g = 0; g < NG; ++g)
+      for (int g = 0; g < NG; ++g)
 #pragma unroll
-      for (int e = 0; e < G; ++e) ss = fmaf(v[g][e], v[g][e], ss);
-    const float inv = rsqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+        for (int e = 0; e < G; ++e) ss = fmaf(v[g][e], v[g][e], ss);
+      const float inv = rsqrtf(warp_sum(ss) / (float)p.dim + p.eps);
 #pragma unroll
-    for (int g = 0; g < NG; ++g)
+      for (int g = 0; g < NG; ++g)
 #pragma unroll
-      for (int e = 0; e < G; ++e) v[g][e] *= inv;
-  }
-  T* dst = is_q ? qrow : reinterpret_cast<T*>(p.k_cache) + crow;
+        for (int e = 0; e < G; ++e) v[g][e] *= inv;
+    }
+    T* dst = is_q ? reinterpret_cast<T*>(p.q) + (size_t)t * p.q_ld + (size_t)h * dp : reinterpret_cast<T*>(p.k_cache) + crow;
 #pragma unroll
-  for (int g = 0; g < NG; ++g) {
-    const int e0 = (g * 32 + lane) * G;
-    if (e0 < dp) store_group<G>(dst + e0, v[g]);
+    for (int g = 0; g < NG; ++g) {
+      const int e0 = (g * 32 + lane) * G;
+      if (e0 < dp) store_group<G>(dst + e0, v[g]);
+    }
   }
 }
 
@@ -1083,7 +1112,10 @@ MX_HOST_API int mx_qk_post(void* q, int q_ld, const void* k, int k_ld, const flo
   p.q = q; p.k = k; p.q_norm = q_norm; p.k_norm = k_norm; p.positions = positions; p.rope_cos = rope_cos; p.rope_sin = rope_sin; p.slot_map = slot_map;
   p.k_cache = k_cache; p.v_cache = v_cache; p.q_ld = q_ld; p.k_ld = k_ld; p.T = T; p.n_q = n_q; p.n_kv = n_kv; p.dp = dp; p.dim = dim; p.rot = rot;
   p.interleaved = interleaved; p.norm_after = norm_after; p.block_size = block_size; p.max_pos = max_pos; p.eps = eps;
-  const long long units = (long long)T * (n_q + n_kv);
+  const int heads = n_q + n_kv;
+  p.hpw = (long long)T * heads >= 64ll * 64 * sm_count() / 8 ? 8 : 1;    // (many tokens: the chip is full with fewer, longer warps)
+  if (p.hpw > heads) p.hpw = heads;
+  const long long units = (long long)T * ((heads + p.hpw - 1) / p.hpw);
   const dim3 grid((unsigned)((units + QK_WARPS - 1) / QK_WARPS)), block(QK_WARPS * 32);
 #define MX_QK(T_)   (dp <= 64 ? launch_pdl(qk_post_kernel<T_, 2, 1>, grid, block, 0, st, p) : dp <= 128 ? launch_pdl(qk_post_kernel<T_, 4, 1>, grid, block, 0, st, p)    : dp <= 256 ? launch_pdl(qk_post_kernel<T_, 8, 1>, grid, block, 0, st, p) : launch_pdl(qk_post_kernel<T_, 8, 2>, grid, block, 0, st, p))
   if (elem_f32) MX_QK(float); else MX_QK(__nv_bfloat16);

@@ -261,7 +261,7 @@ struct GatedNormParams {
   const float* w;              // [G * gs]
   void* out;                   // [T][G * gs]
   float eps, inv_n;            // 1 / live elements of a group
-  int T, G, gs, gate_ld, wpg, silu;
+  int T, G, gs, gate_ld, wpg, lpg, silu;       // lpg: lanes per group (32, or 16 / 8 for short groups of one warp's team)
 };
 constexpr int GG_WARPS = 8;
 
@@ -271,15 +271,17 @@ __global__ void __launch_bounds__(GG_WARPS * 32) gated_group_norm_kernel(const G
   pdl_prologue();
   __shared__ float red[GG_WARPS];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, wpg = p.wpg;
-  const long long unit = (long long)blockIdx.x * (GG_WARPS / wpg) + warp / wpg;
-  if (unit >= (long long)p.T * p.G) return;              // a whole team leaves
-  const long long t = unit / p.G;
-  const int g = (int)(unit - t * p.G), base = g * p.gs;
+  const int lpg = p.lpg, gl = lane & (lpg - 1);
+  const long long unit = ((long long)blockIdx.x * (GG_WARPS / wpg) + warp / wpg) * (32 / lpg) + lane / lpg;
+  const bool some = unit < (long long)p.T * p.G;
+  if (lpg == 32 ? !some : !__any_sync(0xffffffffu, some)) return;        // a whole team (or warp) leaves
+  const long long t = some ? unit / p.G : 0;
+  const int g = some ? (int)(unit - t * p.G) : 0, base = g * p.gs;
   const float* o = p.o + (size_t)t * p.G * p.gs + base;
   const T* gate = reinterpret_cast<const T*>(p.gate) + (size_t)t * p.gate_ld + base;
   const float* w = p.w + base;
   T* out = reinterpret_cast<T*>(p.out) + (size_t)t * p.G * p.gs + base;
-  const int first = ((warp % wpg) * 32 + lane) * 4, step = wpg * 128;
+  const int first = some ? ((warp % wpg) * 32 + gl) * 4 : p.gs, step = wpg * 128;
   float x[NV > 0 ? NV : 1][4], gv[NV > 0 ? NV : 1][4], ss = 0.f;
   if constexpr (NV > 0) {
 #pragma unroll
@@ -299,7 +301,7 @@ __global__ void __launch_bounds__(GG_WARPS * 32) gated_group_norm_kernel(const G
       for (int e = 0; e < 4; ++e) ss = fmaf(x[0][e], x[0][e], ss);
     }
   }
-  ss = warp_sum(ss);
+  for (int o = lpg >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
   if (wpg > 1) {
     const int team = warp / wpg;
     if (lane == 0) red[warp] = ss;
@@ -338,7 +340,9 @@ static int launch_gated_norm(GatedNormParams p, cudaStream_t st) {
   const long long units = (long long)p.T * p.G;
   p.wpg = 1;
   while (p.wpg < GG_WARPS && (p.gs > 512 * p.wpg || (units * p.wpg < 16ll * sm_count() && p.gs > 128 * p.wpg))) p.wpg *= 2;
-  const dim3 grid((unsigned)((units + GG_WARPS / p.wpg - 1) / (GG_WARPS / p.wpg))), block(GG_WARPS * 32);
+  p.lpg = p.gs <= 32 ? 8 : p.gs <= 64 ? 16 : 32;
+  const long long per_cta = (long long)(GG_WARPS / p.wpg) * (32 / p.lpg);
+  const dim3 grid((unsigned)((units + per_cta - 1) / per_cta)), block(GG_WARPS * 32);
   const int pieces = (p.gs + 128 * p.wpg - 1) / (128 * p.wpg);
   if (pieces <= 1) launch_pdl(gated_group_norm_kernel<T, 1>, grid, block, 0, st, p);
   else if (pieces <= 2) launch_pdl(gated_group_norm_kernel<T, 2>, grid, block, 0, st, p);

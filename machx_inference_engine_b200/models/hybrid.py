@@ -207,6 +207,7 @@ class DecayAttentionBlock:
         self.decay = torch.tensor(list(decay), dtype=torch.float64).to(torch.float32).to(dev)
         self.norm = _pad_heads(src.vector(f"{prefix}.norm", heads * value_dim), heads, dv)
         self.out = Linear(src.matrix(f"{prefix}.o", hidden, heads * value_dim).pad_groups(rows=(1, row), cols=(heads, dv)))
+        self.chunked = None if float(self.decay.min()) > 0 else False        # (the chunked form takes logarithms of the decays)
         self.state_shape = {"S": (heads, dk, dv)}
 
     def attend(self, y: torch.Tensor, fb: ForwardBatch, state: RecurrentState) -> torch.Tensor:
@@ -214,7 +215,7 @@ class DecayAttentionBlock:
         H, dk, dv = self.H, self.dk, self.dv
         q, k, v, g = y.split([H * dk, H * dk, H * dv, H * dv], dim=1)
         o = ops.decay_scan(q.unflatten(1, (H, dk)), k.unflatten(1, (H, dk)), v.unflatten(1, (H, dv)), state.tensors["S"][self.layer], fb.state_slots, fb.cu_q,
-                           fb.seq_lens, fb.max_q_len, decay=self.decay, silu=True)
+                           fb.seq_lens, fb.max_q_len, decay=self.decay, silu=True, chunked=self.chunked)
         return self.out(ops.gated_group_norm(o, g, self.norm, self.eps, width=self.live, out_dtype=y.dtype))
 
 

@@ -204,7 +204,11 @@ def token_shift(x, mu, state, state_slots, cu_q, seq_lens, out_dtype=torch.bfloa
     return out
 
 
-def decay_scan(q, k, v, state, state_slots, cu_q, seq_lens, max_q_len, decay=None, z=None, u=None, silu=False):
+DECAY_CHUNKED_MIN_Q = 64          # query segments at least this long take the chunked tensor-core form
+
+
+def decay_scan(q, k, v, state, state_slots, cu_q, seq_lens, max_q_len, decay=None, z=None, u=None, silu=False, chunked=None):
+    """``chunked``: None picks the chunked tensor-core kernels for prompts in bf16 and the sequential kernel otherwise; True / False force one."""
     T, H, dk = q.shape
     dv = v.shape[2]
     assert q.dtype == k.dtype == v.dtype and state.dtype == torch.float32 and state.shape[1:] == (H, dk, dv) and k.shape == q.shape
@@ -212,6 +216,19 @@ def decay_scan(q, k, v, state, state_slots, cu_q, seq_lens, max_q_len, decay=Non
         assert t.stride(2) == 1 and (H == 1 or t.stride(1) == t.shape[2])
     assert z is None or (z.dtype == torch.float32 and z.is_contiguous() and z.shape == (T, H * dk) and u.shape == (H, dk))
     out = torch.empty(T, H * dv, dtype=torch.float32, device=q.device)
+    if chunked is None:
+        chunked = q.dtype == torch.bfloat16 and dk <= 128 and max_q_len >= DECAY_CHUNKED_MIN_Q
+    if chunked:
+        lib, B = _lib.cuda(), cu_q.numel() - 1
+        for f in (lib.mx_decay_chunk_ws_bytes, lib.mx_decay_chunk_gl_floats):
+            f.restype = C.c_longlong
+        assert q.dtype == torch.bfloat16
+        ws = torch.empty(int(lib.mx_decay_chunk_ws_bytes(T, B, H, dk, dv)), dtype=torch.uint8, device=q.device)
+        gl = torch.empty(int(lib.mx_decay_chunk_gl_floats(T, B, H, dk)), dtype=torch.float32, device=q.device)
+        _check(lib.mx_decay_scan_chunked(_p(q), q.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), _p(z), _p(u), _p(decay), _p(state), _p(state_slots),
+                                         _p(cu_q), _p(seq_lens), _p(out), B, T, H, dk, dv, int(silu), _p(ws), _p(gl), _stream()), "decay_scan_chunked")
+        _count(2)
+        return out
     _check(_lib.cuda().mx_decay_scan(_p(q), q.stride(0), _p(k), k.stride(0), _p(v), v.stride(0), _p(z), _p(u), _p(decay), _p(state), _p(state_slots), _p(cu_q),
                                      _p(seq_lens), _p(out), cu_q.numel() - 1, H, dk, dv, int(silu), int(q.dtype == torch.float32), _stream()), "decay_scan")
     _count()

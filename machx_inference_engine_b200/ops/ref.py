@@ -420,7 +420,7 @@ def token_shift(x, mu, state, state_slots, cu_q, seq_lens, out_dtype=torch.bfloa
     return (x.unsqueeze(0) + (prev - x).unsqueeze(0) * mu.unsqueeze(1)).to(out_dtype)
 
 
-def decay_scan(q, k, v, state, state_slots, cu_q, seq_lens, max_q_len, decay=None, z=None, u=None, silu=False):
+def decay_scan(q, k, v, state, state_slots, cu_q, seq_lens, max_q_len, decay=None, z=None, u=None, silu=False, chunked=None):
     """Linear attention with a decaying state S [dk, dv] per head.  q, k [T, H, dk], v [T, H, dv] (any row stride); state fp32 [slots, H, dk, dv], advanced
     in place, from zeros for a sequence whose step begins at position 0.  Returns o fp32 [T, H * dv].
       decay [H]                        S <- decay S + k v^T, o = S^T q           (``silu``: q, k and v pass through it first)

@@ -189,3 +189,148 @@ def forward(weights, cfg, tokens):
             x = x + rms_norm(FEED_FORWARD[f["kind"]](W, f"{l}.mlp", f, x), W[f"{l}.norm2"], eps) * W[f"{l}.ls2"]
         after.append(x)
     return rms_norm(x, W["final.norm"], eps) @ W["embed"].T, np.stack(after)
+
+
+# ------------------------------------------------------------------ configurations and weights of tests
+def _rot(dims, base, scaling):
+    r = {"base": base, "dims": dims}
+    if scaling is not None:
+        r["scaling"] = dict(zip(("factor", "original", "fast", "slow"), scaling))
+    return r
+
+
+def feed_forward(mlp):
+    """None, a width (dense), or (experts, top, expert width, width of the shared expert or 0)."""
+    if not isinstance(mlp, tuple):
+        return None if mlp is None else {"kind": "dense", "ff": mlp}
+    f = {"kind": "moe", "expert": {"ff": mlp[2]}, "router": {"experts": mlp[0], "top": mlp[1]}}
+    return {**f, "shared": {"ff": mlp[3]}} if mlp[3] else f
+
+
+def attention_sizes(heads, kv_heads, dim, window, rot_dims, base=10000.0, scaling=None, keep_first=None, scale=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "rot": _rot(rot_dims, base, scaling), "scale": scale or 1.0 / math.sqrt(dim)}
+    if window:
+        m["mask"] = {"size": window} if keep_first is None else {"size": window, "keep_first": keep_first}
+    return m
+
+
+def attention_layer(mlp, *sizes, **kw):
+    return {"type": "attention", "mlp": feed_forward(mlp), "mixer": attention_sizes(*sizes, **kw)}
+
+
+def wkv_layer(mlp, heads, dim):
+    return {"type": "wkv", "mlp": feed_forward(mlp), "mixer": {"heads": heads, "dim": dim}}
+
+
+def parallel_layer(mlp, left, heads, dim, vdim, decay):
+    return {"type": "parallel", "mlp": feed_forward(mlp), "mixer": {"left": left, "right": {"heads": heads, "dim": dim, "vdim": vdim, "decay": list(decay)}}}
+
+
+def random_config(layers, vocab=96, width=64, eps=1e-6, scale=3.0):
+    return {"architecture": "Beputar", "embedding": {"scale": scale}, "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+def round_bf16(a):
+    """float array -> float32 values that bfloat16 represents (round to nearest even)."""
+    u = np.array(a, dtype=np.float32, order="C").view(np.uint32).astype(np.uint64)
+    u = ((u + 0x7FFF + ((u >> 16) & 1)) >> 16 << 16).astype(np.uint32)
+    return u.view(np.float32)
+
+
+CODES = 8            # columns that hold a code of the token and that no layer writes to, read by the routers alone
+
+
+def random_weights(cfg, seed=0, rank=12):
+    """Every tensor the configuration asks for, as float32 arrays that hold bfloat16 values.  The routers read a code of the token, so that no choice of
+    experts is within rounding of another.  ``rank``: inner width of the decay's projection."""
+    g = np.random.default_rng(seed)
+    H, W = cfg["width"], {}
+
+    def mat(name, n, k, gain=1.0):
+        W[name] = round_bf16(g.standard_normal((n, k)) * gain / math.sqrt(k))
+
+    def vec(name, n, mean=0.0, std=0.2):
+        W[name] = round_bf16(mean + std * g.standard_normal(n))
+
+    def gated(name, f):
+        for n, shape in (("gate", (f, H)), ("up", (f, H)), ("down", (H, f))):
+            mat(f"{name}.{n}", *shape)
+
+    W["embed"] = round_bf16(g.standard_normal((cfg["vocab"], H)) / cfg["embedding"]["scale"])
+    vec("final.norm", H, 1.0)
+    for i, layer in enumerate(cfg["layers"]):
+        l, p, m, f = f"l{i}", f"l{i}.mix", layer["mixer"], layer["mlp"]
+        vec(f"{l}.norm1", H, 1.0)
+        vec(f"{l}.ls1", H, 0.5, 0.1)
+        if layer["type"] == "attention":
+            for n, k in (("q", m["heads"]), ("k", m["kv_heads"])):
+                mat(f"{p}.{n}", k * m["dim"], H, 1.5)
+                vec(f"{p}.{n}.b", k * m["dim"], 0.0, 0.5)
+            mat(f"{p}.o", H, m["heads"] * m["dim"])
+        elif layer["type"] == "wkv":
+            n = m["heads"] * m["dim"]
+            for k in "rkvg":
+                mat(f"{p}.{k}", n, H)
+            for k in "rkvgw":
+                W[f"{p}.mu.{k}"] = round_bf16(g.uniform(0.0, 1.0, H))
+            mat(f"{p}.w1", rank, H)
+            mat(f"{p}.w2", n, rank)
+            W[f"{p}.w0"] = round_bf16(g.uniform(-5.0, 0.5, n))
+            W[f"{p}.u"] = round_bf16(0.5 * g.standard_normal((m["heads"], m["dim"])))
+            vec(f"{p}.norm", n, 1.0)
+            mat(f"{p}.o", H, n)
+        else:
+            a, b = m["left"], m["right"]
+            for n, k in (("q", a["heads"]), ("k", a["kv_heads"])):
+                mat(f"{p}.left.{n}", k * a["dim"], H, 1.5)
+                vec(f"{p}.left.{n}.norm", a["dim"], 1.3)
+            mat(f"{p}.left.g", a["heads"], H)
+            mat(f"{p}.left.o", H, a["heads"] * a["dim"])
+            nk, nv = b["heads"] * b["dim"], b["heads"] * b["vdim"]
+            for n, k in (("q", nk), ("k", nk), ("v", nv), ("g", nv)):
+                mat(f"{p}.right.{n}", k, H)
+            vec(f"{p}.right.norm", nv, 1.0)
+            mat(f"{p}.right.o", H, nv)
+            vec(f"{p}.left.out", H, 1.0)
+            vec(f"{p}.right.out", H, 1.0)
+        if f is None:
+            continue
+        vec(f"{l}.norm2", H, 1.0)
+        vec(f"{l}.ls2", H, 0.5, 0.1)
+        if f["kind"] == "dense":
+            mat(f"{l}.mlp.up", f["ff"], H)
+            mat(f"{l}.mlp.down", H, f["ff"])
+        else:
+            for e in range(f["router"]["experts"]):
+                gated(f"{l}.mlp.e{e}", f["expert"]["ff"])
+            if f.get("shared"):
+                gated(f"{l}.mlp.shared", f["shared"]["ff"])
+    _settle_routing(cfg, W, g)
+    return W
+
+
+def _settle_routing(cfg, W, g, gap=0.3):
+    moe = [(i, layer["mlp"]["router"]) for i, layer in enumerate(cfg["layers"]) if layer["mlp"] is not None and layer["mlp"]["kind"] == "moe"]
+    if not moe:
+        return
+    for i, _ in enumerate(cfg["layers"]):
+        for n in (f"l{i}.ls1", f"l{i}.ls2"):
+            if n in W:
+                W[n][:CODES] = 0.0
+    scale = cfg["embedding"]["scale"]
+    for i, r in moe:
+        z = g.standard_normal((r["experts"], CODES)) * 0.5
+        W[f"l{i}.mlp.router"] = round_bf16(np.pad(z, ((0, 0), (0, cfg["width"] - CODES))))
+    for t in range(cfg["vocab"]):
+        for _ in range(2000):
+            code = round_bf16(2.0 * g.choice([-1.0, 1.0], CODES) / scale)
+            gaps = [np.inf]
+            for i, r in moe:
+                z = np.sort(np.float64(W[f"l{i}.mlp.router"])[:, :CODES] @ (np.float64(code) * scale))[::-1]
+                if r["top"] < len(z):
+                    gaps.append(z[r["top"] - 1] - z[r["top"]])
+            if min(gaps) > gap:
+                break
+        else:
+            raise ValueError("no code of this token settles its routing")
+        W["embed"][t, :CODES] = code
