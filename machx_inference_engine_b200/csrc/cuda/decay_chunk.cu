@@ -9,9 +9,9 @@
 //   *_prep_kernel      one CTA per (chunk, head), all chunks in parallel: decays in fp32, M through one tcgen05.mma batch, and the operands Q'', KD, M, V as
 //       ready-made shared-memory images (rows of 128 bytes, 128-byte swizzle).  With a fixed decay M is (Q K^T) times a table.  With decays from the data
 //       the exponents are split so that no factor grows: the chunk falls into four blocks of 16 tokens, a query's factor runs from the start of its own
-//       block, and every later block has its own copy of the keys, decayed up to its start (rows K'_1 .. K'_3 of the B operand).  Inside a block the keys'
-//       factor does grow, by less than e^80 -- inside the range of bf16, whose relative precision does not depend on size; a chunk in which it would grow
-//       further forms those 16 x 16 products one by one in fp32.
+//       block (or pair of blocks), and the keys of earlier ones are decayed up to that start.  Inside a block the keys' factor does grow, by less than
+//       e^80 -- inside the range of bf16, whose relative precision does not depend on size; a chunk in which it would grow further forms those 16 x 16
+//       products one by one in fp32.
 //   decay_chunk_scan_kernel  one CTA per (sequence, head, 64 value columns), chunks in order.  The state slice stays in registers (thread = key channel);
 //       once per chunk it goes to shared memory as a bf16 high + low pair, Q'' S0 + M V and KD^T V run as one MMA batch, and the next chunk's images
 //       arrive by bulk copies meanwhile.
@@ -178,115 +178,158 @@ __global__ void __launch_bounds__(256) decay_fixed_prep_kernel(const DecayChunkP
 }
 
 // ------------------------------------------------------------------------------------------------ prep, decays from the data
-// B operand rows: K'' (0 .. 63: keys against the start of their own block), U (64 .. 127: u k against the query's factor, for the diagonal), K'_1 (128 ..),
-// K'_2 (144 ..), K'_3 (176 .. 223).
-constexpr int WB_ROWS = 224;
+// Blocks of 16 tokens 0 .. 3.  A: queries against the start of their own block; A2: block 3 against the start of block 2 instead (block 2 as in A).
+// B operand rows: K'' (0 .. 63: keys against the start of their own block, a growing factor), K_1 (64 .. 79: block 0 decayed to its end, for block 1),
+// K_3 (80 .. 95: block 2 decayed to its end, for block 3), K_H (96 .. 127: blocks 0 and 1 decayed to the end of block 1, for A2's blocks 2 and 3).
+constexpr int WB_ROWS = 128, WB_K1 = 64, WB_K3 = 80, WB_KH = 96;
 constexpr float WKV_MAX_GROWTH = -80.f;
 template <int KA>
 struct DataSmem {
-  static constexpr int A = 0, B = KA * CA, BA = WB_ROWS * 128;          // BA: bytes of a B atom
+  static constexpr int A = 0, A2 = KA * CA, B = 2 * KA * CA, BA = WB_ROWS * 128;      // BA: bytes of a B atom
   static constexpr int LOGS = B + KA * BA;                               // cumulative logs inside the blocks, fp32 [64][64 KA + 1] (slow path only)
   static constexpr int DIAG = LOGS + CC * (64 * KA + 1) * 4;             // [64][16] fp32 (slow path only)
-  static constexpr int TOT = DIAG + CC * 16 * 4;                         // block totals [4][64 KA]
-  static constexpr int MISC = TOT + 4 * 64 * KA * 4;
+  static constexpr int MISC = DIAG + CC * 16 * 4;
   static constexpr int TOTAL = MISC + 64 + 1024;
-  static_assert(KA * CA + CA <= LOGS, "A over-read stays inside the images");
 };
-__device__ __forceinline__ int kprime_row(int I) { return I == 1 ? 128 : I == 2 ? 144 : 176; }
+__device__ __forceinline__ void sts32(uint32_t addr, uint32_t v) { asm volatile("st.shared.b32 [%0], %1;" ::"r"(addr), "r"(v) : "memory"); }
+__device__ __forceinline__ void sts128(uint32_t addr, uint32_t a, uint32_t b, uint32_t c, uint32_t d) {
+  asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(addr), "r"(a), "r"(b), "r"(c), "r"(d) : "memory");
+}
+__device__ __forceinline__ float4 lds128(uint32_t addr) {
+  float4 v;
+  asm volatile("ld.shared.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(addr));
+  return v;
+}
 
 template <int KA>
-__global__ void __launch_bounds__(256 * KA, 2 / KA) decay_data_prep_kernel(const DecayChunkParams p) {
+__global__ void __launch_bounds__(128 * KA, 4 / KA) decay_data_prep_kernel(const DecayChunkParams p) {
   using L = DataSmem<KA>;
-  constexpr int W = 64 * KA, LS = W + 1, THREADS = 256 * KA;
+  constexpr int W = 64 * KA, LS = W + 1, THREADS = 128 * KA;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   const uint32_t sbase = smem_u32(smem);
+  __shared__ __align__(8) float tot[4][W];               // sums of the logs of the blocks
+  __shared__ float bonus[KA][CC];                        // r . (u k) of the tokens, one part per warp of a block
   uint64_t* bar = reinterpret_cast<uint64_t*>(smem + L::MISC);
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bar + 1);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  float* tot = reinterpret_cast<float*>(smem + L::TOT);
   float* logs = reinterpret_cast<float*>(smem + L::LOGS);
   float* diag = reinterpret_cast<float*>(smem + L::DIAG);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y;
-  const int c = tid % W, J = tid / W;                    // key channel, block of 16 tokens
+  const int c = (tid % (32 * KA)) * 2, J = tid / (32 * KA);              // two key channels, a block
   pdl_prologue();
   int t0, n;
   if (!chunk_locate(p.cu_q, p.B, blockIdx.x, t0, n)) return;            // whole CTA, before any barrier / TMEM use
   if (tid == 0) { mbar_init(smem_u32(bar), 1); *abort_flag = 0; fence_mbar_init(); }
-  if (warp == 0) { tmem_alloc(smem_u32(tmem_slot), 256); tmem_relinquish(); }
-  float lg[16], r[16], k[16];                            // cumulative log decays inside the block
+  if (warp == 0) { tmem_alloc(smem_u32(tmem_slot), 128); tmem_relinquish(); }
   const bool live = c < p.dk;
-  const float uc = live ? p.u[(size_t)h * p.dk + c] : 0.f;
-  {
-    float z[16];
+  uint32_t r2[16], k2[16];                               // bf16 pairs
+  float lg[16][2];                                       // cumulative log decays inside the block
 #pragma unroll
-    for (int t = 0; t < 16; ++t) {
-      const int row = 16 * J + t;
-      const size_t tt = (size_t)(t0 + row);
-      r[t] = k[t] = 0.f;
-      z[t] = -INFINITY;                                  // (rows past the end: log decay 0)
-      if (live && row < n) {
-        r[t] = __bfloat162float(p.q[tt * p.q_ld + (size_t)h * p.dk + c]);
-        k[t] = __bfloat162float(p.k[tt * p.k_ld + (size_t)h * p.dk + c]);
-        z[t] = p.z[(tt * p.H + h) * p.dk + c];
-      }
-    }
-    float s = 0.f;
-#pragma unroll
-    for (int t = 0; t < 16; ++t) {
-      s -= fminf(expf(z[t]), 110.f);                     // (a decay of e^-104 and less is zero in fp32; larger sums would cost the others their digits)
-      lg[t] = s;
+  for (int t = 0; t < 16; ++t) {
+    const int row = 16 * J + t;
+    const size_t tt = (size_t)(t0 + row);
+    r2[t] = k2[t] = 0u;
+    lg[t][0] = lg[t][1] = -INFINITY;                     // (rows past the end: log decay 0)
+    if (live && row < n) {
+      r2[t] = *reinterpret_cast<const uint32_t*>(p.q + tt * p.q_ld + (size_t)h * p.dk + c);
+      k2[t] = *reinterpret_cast<const uint32_t*>(p.k + tt * p.k_ld + (size_t)h * p.dk + c);
+      const float2 z = *reinterpret_cast<const float2*>(p.z + (tt * p.H + h) * p.dk + c);
+      lg[t][0] = z.x;
+      lg[t][1] = z.y;
     }
   }
-  tot[J * W + c] = lg[15];
+  float2 u = make_float2(0.f, 0.f);
+  if (live) u = *reinterpret_cast<const float2*>(p.u + (size_t)h * p.dk + c);
+  {
+    float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+    for (int t = 0; t < 16; ++t) {                       // (a decay of e^-104 and less is zero in fp32; larger sums would cost the others their digits)
+      s0 -= fminf(expf(lg[t][0]), 110.f);
+      s1 -= fminf(expf(lg[t][1]), 110.f);
+      lg[t][0] = s0;
+      lg[t][1] = s1;
+    }
+  }
+  *reinterpret_cast<float2*>(&tot[J][c]) = make_float2(lg[15][0], lg[15][1]);
+  {
+    float v[16];
+#pragma unroll
+    for (int t = 0; t < 16; ++t) v[t] = bf16_lo(r2[t]) * u.x * bf16_lo(k2[t]) + bf16_hi(r2[t]) * u.y * bf16_hi(k2[t]);
+    // sum over the lanes, halving the values that a lane keeps: lane l ends with token l / 2
+#pragma unroll
+    for (int m = 8; m > 0; m >>= 1) {
+      const bool up = lane & (2 * m);
+#pragma unroll
+      for (int i = 0; i < m; ++i) {
+        const float give = up ? v[i] : v[i + m], keep = up ? v[i + m] : v[i];
+        v[i] = keep + __shfl_xor_sync(0xffffffffu, give, 2 * m);
+      }
+    }
+    v[0] += __shfl_xor_sync(0xffffffffu, v[0], 1);
+    if (!(lane & 1)) bonus[KA == 1 ? 0 : warp & 1][16 * J + (lane >> 1)] = v[0];
+  }
   tc_fence_before();
-  const bool slow = __syncthreads_or(lg[15] < WKV_MAX_GROWTH);
+  const bool slow = __syncthreads_or(fminf(lg[15][0], lg[15][1]) < WKV_MAX_GROWTH);
   tc_fence_after();
   const uint32_t tmem = *tmem_slot;
   uint8_t* ws = p.ws + ((size_t)blockIdx.x * p.H + h) * ws_bytes(KA, p.va);
-  float before = 0.f, after = 0.f, step[3] = {0.f, 0.f, 0.f};            // logs of the blocks before and after; of those between J and block J + 1 + i
+  float eb[2], ea[2], eh[2], e2[2], after[2] = {0.f, 0.f};              // e^{logs of the blocks before; after; to the end of block 1; of block 2}
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const float x = tot[i * W + c];
-    if (i < J) before += x;
-    if (i > J) { after += x; }
+  for (int x = 0; x < 2; ++x) {
+    float before = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float v = tot[i][c + x];
+      if (i < J) before += v;
+      if (i > J) after[x] += v;
+    }
+    eb[x] = __expf(before);
+    ea[x] = __expf(after[x]);
+    eh[x] = J == 0 ? __expf(tot[1][c + x]) : 1.f;
+    e2[x] = J == 3 ? __expf(tot[2][c + x]) : 1.f;
   }
-  step[1] = J + 1 < 4 ? tot[(J + 1) * W + c] : 0.f;
-  step[2] = J + 2 < 4 ? step[1] + tot[(J + 2) * W + c] : 0.f;
-  const float e_before = __expf(before), e_after = __expf(after), e_step[3] = {1.f, __expf(step[1]), __expf(step[2])};
   {
+    // the low bits of 16 J + t and of every image's first row come from t alone
     const uint32_t piece = (c & 63) >> 3, sub = (c & 7) * 2, atom = c >> 6;
-    auto put = [&](uint8_t* base, int stride, int row, float x) {
-      *reinterpret_cast<bf16*>(base + atom * stride + sw128_offset(row, piece) + sub) = __float2bfloat16(x);
-    };
-    float e_prev = 1.f, l_prev = 0.f;                    // e^{sum of the block's logs before t}
+    const uint32_t sa = sbase + L::A + atom * CA + J * 2048 + sub, sa2 = sa + (L::A2 - L::A);
+    const uint32_t sb = sbase + L::B + atom * L::BA + J * 2048 + sub;
+    const uint32_t side = J == 0 ? (WB_K1 >> 3) * 1024 : J == 2 ? ((WB_K3 >> 3) - 4) * 1024 : 0;       // from the K'' row of the block to its K_1 / K_3 row
+    uint8_t* gq = ws + atom * CA + J * 2048 + sub;
+    float ep[2] = {1.f, 1.f};                            // e^{sum of the block's logs before t}
 #pragma unroll
     for (int t = 0; t < 16; ++t) {
-      const int row = 16 * J + t;
-      const float e_t = __expf(lg[t]), to_end = __expf(lg[15] - lg[t]);
-      put(smem + L::A, CA, row, r[t] * e_prev);
-      put(smem + L::B, L::BA, row, k[t] * __expf(-lg[t]));
-      put(smem + L::B, L::BA, 64 + row, uc * k[t] * __expf(-l_prev));
-#pragma unroll
-      for (int i = 0; i < 3; ++i)
-        if (J + 1 + i < 4) put(smem + L::B, L::BA, kprime_row(J + 1 + i) + row, k[t] * to_end * e_step[i]);
-      put(ws, CA, row, r[t] * e_prev * e_before);
-      put(ws + KA * CA, CA, row, k[t] * to_end * e_after);
-      if (slow) logs[row * LS + c] = lg[t];
-      e_prev = e_t;
-      l_prev = lg[t];
+      const uint32_t at = (t >> 3) * 1024 + (t & 7) * 128 + ((piece ^ (t & 7)) << 4);
+      const float r0 = bf16_lo(r2[t]) * ep[0], r1 = bf16_hi(r2[t]) * ep[1], k0 = bf16_lo(k2[t]), k1 = bf16_hi(k2[t]);
+      const float d0 = k0 * __expf(lg[15][0] - lg[t][0]), d1 = k1 * __expf(lg[15][1] - lg[t][1]);      // decayed to the block's end
+      sts32(sa + at, pack_bf16(r0, r1));
+      if (J >= 2) sts32(sa2 + at, pack_bf16(r0 * e2[0], r1 * e2[1]));
+      sts32(sb + at, pack_bf16(k0 * __expf(-lg[t][0]), k1 * __expf(-lg[t][1])));
+      if (side) sts32(sb + side + at, pack_bf16(d0, d1));
+      if (J < 2) sts32(sb + (WB_KH >> 3) * 1024 + at, pack_bf16(d0 * eh[0], d1 * eh[1]));
+      *reinterpret_cast<uint32_t*>(gq + at) = pack_bf16(r0 * eb[0], r1 * eb[1]);
+      *reinterpret_cast<uint32_t*>(gq + KA * CA + at) = pack_bf16(d0 * ea[0], d1 * ea[1]);
+      if (slow) {
+        logs[(16 * J + t) * LS + c] = lg[t][0];
+        logs[(16 * J + t) * LS + c + 1] = lg[t][1];
+      }
+      ep[0] = __expf(lg[t][0]);
+      ep[1] = __expf(lg[t][1]);
     }
   }
-  if (J == 0) p.gl[((size_t)blockIdx.x * p.H + h) * W + c] = __expf(lg[15] + after);
+  if (J == 0)
+    *reinterpret_cast<float2*>(p.gl + ((size_t)blockIdx.x * p.H + h) * W + c) = make_float2(__expf(lg[15][0] + after[0]), __expf(lg[15][1] + after[1]));
   fence_proxy_async();
   __syncthreads();
   const uint32_t mbar = smem_u32(bar);
   if (tid == 0) {
-    constexpr uint32_t idesc = umma_idesc_bf16(128, WB_ROWS, 0, 0);
+    constexpr uint32_t idesc = umma_idesc_bf16(128, WB_KH, 0, 0), idesc_h = umma_idesc_bf16(128, WB_ROWS - WB_KH, 0, 0);
 #pragma unroll
-    for (int kk = 0; kk < KA * 4; ++kk)
-      umma_bf16(tmem, umma_desc_k_sw128(sbase + L::A + (kk >> 2) * CA + (kk & 3) * 32), umma_desc_k_sw128(sbase + L::B + (kk >> 2) * L::BA + (kk & 3) * 32), idesc,
-                kk != 0);
+    for (int kk = 0; kk < KA * 4; ++kk) {
+      const uint32_t ao = (kk >> 2) * CA + (kk & 3) * 32, bo = sbase + L::B + (kk >> 2) * L::BA + (kk & 3) * 32;
+      umma_bf16(tmem, umma_desc_k_sw128(sbase + L::A + ao), umma_desc_k_sw128(bo), idesc, kk != 0);
+      umma_bf16(tmem + WB_KH, umma_desc_k_sw128(sbase + L::A2 + ao), umma_desc_k_sw128(bo + WB_KH * 128), idesc_h, kk != 0);
+    }
     umma_commit(mbar);
   }
   value_image(p, ws + (2 * KA + 1) * CA, h, t0, n, tid, THREADS);
@@ -294,13 +337,11 @@ __global__ void __launch_bounds__(256 * KA, 2 / KA) decay_data_prep_kernel(const
     for (int e = tid; e < CC * 16; e += THREADS) {
       const int i = e >> 4, j = (i & ~15) + (e & 15);
       float s = 0.f;
-      if (j <= i && i < n) {
+      if (j < i && i < n) {
         const bf16* ri = p.q + (size_t)(t0 + i) * p.q_ld + (size_t)h * p.dk;
         const bf16* kj = p.k + (size_t)(t0 + j) * p.k_ld + (size_t)h * p.dk;
-        for (int x = 0; x < p.dk; ++x) {
-          const float d = j == i ? p.u[(size_t)h * p.dk + x] : __expf(logs[(i - 1) * LS + x] - logs[j * LS + x]);
-          s = fmaf(__bfloat162float(ri[x]) * d, __bfloat162float(kj[x]), s);
-        }
+        for (int x = 0; x < p.dk; ++x)
+          s = fmaf(__bfloat162float(ri[x]) * __expf(logs[(i - 1) * LS + x] - logs[j * LS + x]), __bfloat162float(kj[x]), s);
       }
       diag[e] = s;
     }
@@ -309,71 +350,60 @@ __global__ void __launch_bounds__(256 * KA, 2 / KA) decay_data_prep_kernel(const
   const bool ok = mbar_wait(mbar, 0, p.status, ERR_MBAR_TIMEOUT_EPILOGUE, abort_flag, 32);
   tc_fence_after();
   if (ok && warp < 2) {                                  // rows 32 warp + lane: blocks 2 warp and 2 warp + 1
-    const int i = warp * 32 + lane;
+    const int i = warp * 32 + lane, at = lane & 15;
     const bool lo = lane < 16;                           // the warp's first block
     const uint32_t ta = tmem + ((uint32_t)(warp * 32) << 16);
-    float own[16];                                       // the block's own 16 columns, diagonal included
-    {
-      uint32_t d[32], g[32];
-      tmem_ld_32x32(ta + warp * 32, d);
-      tmem_ld_32x32(ta + 64 + warp * 32, g);
-      tmem_ld_wait();
-      uint32_t bonus = 0;
+    uint32_t d[32], x[32], y[32];
+    tmem_ld_32x32(ta + warp * 32, d);                    // own columns of both blocks
+    tmem_ld_32x32(ta + WB_K1, x);                        // K_1 | K_3
+    if (warp) tmem_ld_32x32(ta + WB_KH, y);
+    tmem_ld_wait();
+    const float b = KA == 1 ? bonus[0][i] : bonus[0][i] + bonus[KA - 1][i];
+    float own[16];
 #pragma unroll
-      for (int x = 0; x < 32; ++x) bonus = lane == x ? g[x] : bonus;
-#pragma unroll
-      for (int j = 0; j < 16; ++j) {
-        const int at = lane & 15;
-        own[j] = j < at ? __uint_as_float(lo ? d[j] : d[16 + j]) : j == at ? __uint_as_float(bonus) : 0.f;
-        if (slow) own[j] = diag[i * 16 + j];
-      }
+    for (int j = 0; j < 16; ++j) {
+      own[j] = j < at ? __uint_as_float(lo ? d[j] : d[16 + j]) : j == at ? b : 0.f;
+      if (slow && j < at) own[j] = diag[i * 16 + j];
     }
-    auto store16 = [&](int Jc, const float (&x)[16]) {
+    uint8_t* wm = ws + 2 * KA * CA;
+    auto store16 = [&](int Jc, const float (&v)[16]) {
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         float m[8];
 #pragma unroll
-        for (int e = 0; e < 8; ++e) m[e] = x[8 * half + e];
-        *reinterpret_cast<uint4*>(ws + 2 * KA * CA + sw128_offset(i, 2 * Jc + half)) = pack8(m);
+        for (int e = 0; e < 8; ++e) m[e] = v[8 * half + e];
+        *reinterpret_cast<uint4*>(wm + sw128_offset(i, 2 * Jc + half)) = pack8(m);
       }
     };
-    float x0[16], x1[16], x2[16], x3[16];
-    if (warp == 0) {
-      uint32_t a[32];
-      tmem_ld_32x32(ta + 128, a);                        // K'_1 in its first 16 columns
-      tmem_ld_wait();
+    float a[16], e[16];                                  // columns of the warp's first and second block
 #pragma unroll
-      for (int j = 0; j < 16; ++j) {
-        x0[j] = lo ? own[j] : __uint_as_float(a[j]);
-        x1[j] = lo ? 0.f : own[j];
-        x2[j] = x3[j] = 0.f;
-      }
-    } else {
-      uint32_t a[32], b[32], e[32];
-      tmem_ld_32x32(ta + 144, a);                        // K'_2
-      tmem_ld_32x32(ta + 176, b);                        // K'_3, columns 0 .. 31
-      tmem_ld_32x32(ta + 192, e);                        // ... 16 .. 47
-      tmem_ld_wait();
-#pragma unroll
-      for (int j = 0; j < 16; ++j) {
-        x0[j] = __uint_as_float(lo ? a[j] : b[j]);
-        x1[j] = __uint_as_float(lo ? a[16 + j] : b[16 + j]);
-        x2[j] = lo ? own[j] : __uint_as_float(e[16 + j]);
-        x3[j] = lo ? 0.f : own[j];
-      }
+    for (int j = 0; j < 16; ++j) {
+      a[j] = lo ? own[j] : __uint_as_float(warp ? x[16 + j] : x[j]);
+      e[j] = lo ? 0.f : own[j];
     }
-    store16(0, x0); store16(1, x1); store16(2, x2); store16(3, x3);
+    store16(2 * warp, a);
+    store16(2 * warp + 1, e);
+#pragma unroll
+    for (int j = 0; j < 16; ++j) {                       // the other half of the columns
+      a[j] = warp ? __uint_as_float(y[j]) : 0.f;
+      e[j] = warp ? __uint_as_float(y[16 + j]) : 0.f;
+    }
+    store16(2 - 2 * warp, a);
+    store16(3 - 2 * warp, e);
   }
   tc_fence_before();
   __syncthreads();
-  if (warp == 0) tmem_dealloc(tmem, 256);
+  if (warp == 0) tmem_dealloc(tmem, 128);
 }
 
 // ------------------------------------------------------------------------------------------------ scan
 template <int KA>
 struct ChunkScanSmem {
+  static constexpr int NS = 3;                                           // stages: images of this chunk and the next two
   static constexpr int Q = 0, KD = KA * CA, M = 2 * KA * CA, V = M + CA, STAGE = V + CA;
-  static constexpr int SHI = 2 * STAGE, SLO = SHI + 2 * CA, BARS = SLO + 2 * CA;      // state slice: [128 keys][64 values] high and low part
+  static constexpr int SHI = NS * STAGE, SLO = SHI + KA * CA;            // state slice: [64 KA keys][64 values] high and low part
+  static constexpr int OUT = SLO + KA * CA, OUT_ROW = CV * 4 + 16;       // two output tiles [64 tokens][64 values] fp32
+  static constexpr int BARS = OUT + 2 * CC * OUT_ROW;
   static constexpr int TOTAL = BARS + 64 + 1024;
   static_assert(TOTAL <= 232448, "shared memory plan exceeds 227 KB");
 };
@@ -384,12 +414,13 @@ __device__ __forceinline__ void chunk_bulk(uint32_t dst, const void* src, uint32
 template <int KA>
 __global__ void __launch_bounds__(128) decay_chunk_scan_kernel(const DecayChunkParams p) {
   using L = ChunkScanSmem<KA>;
+  constexpr int NS = L::NS;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   const uint32_t sbase = smem_u32(smem);
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + L::BARS);
-  const uint32_t bar_load = smem_u32(bars), bar_inc = bar_load + 16, bar_o = bar_load + 24;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 4);
+  const uint32_t bar_load = smem_u32(bars), bar_inc = bar_load + 8 * NS, bar_o = bar_inc + 8;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + NS + 2);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   const int tid = threadIdx.x, warp = tid >> 5, h = blockIdx.y, vs = blockIdx.x, b = blockIdx.z;
   pdl_prologue();
@@ -399,7 +430,7 @@ __global__ void __launch_bounds__(128) decay_chunk_scan_kernel(const DecayChunkP
   int cb = 0;                                            // index of this sequence's first chunk
   for (int i = 0; i < b; ++i) cb += (p.cu_q[i + 1] - p.cu_q[i] + CC - 1) / CC;
   if (tid == 0) {
-    mbar_init(bar_load, 1); mbar_init(bar_load + 8, 1); mbar_init(bar_inc, 1); mbar_init(bar_o, 1);
+    for (int s = 0; s < NS + 2; ++s) mbar_init(bar_load + 8 * s, 1);
     *abort_flag = 0;
     fence_mbar_init();
   }
@@ -408,10 +439,19 @@ __global__ void __launch_bounds__(128) decay_chunk_scan_kernel(const DecayChunkP
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = *tmem_slot, tm_lane = (uint32_t)(warp * 32) << 16;
+  auto issue_load = [&](int c) {
+    const uint8_t* ws = p.ws + ((size_t)(cb + c) * p.H + h) * ws_bytes(KA, p.va);
+    const uint32_t dst = sbase + (c % NS) * L::STAGE, bar = bar_load + 8 * (c % NS);
+    mbar_expect_tx(bar, L::STAGE);
+    chunk_bulk(dst, ws, L::V, bar);
+    chunk_bulk(dst + L::V, ws + L::V + vs * CA, CA, bar);
+  };
+  if (tid == 0)
+    for (int c = 0; c < NS - 1 && c < nc; ++c) issue_load(c);
 
   // thread = key channel; S[j] = its state against value column 64 vs + j
   const int dv = p.dv, v0 = vs * CV, nv = min(CV, dv - v0);              // (nv is a multiple of 8)
-  const bool live = tid < p.dk;
+  const bool live = tid < p.dk, own = tid < 64 * KA;
   float S[CV];
   float* sp = p.state + (((size_t)p.slots[b] * p.H + h) * p.dk + tid) * dv + v0;
   const bool fresh = p.seq_lens[b] == len;
@@ -421,21 +461,25 @@ __global__ void __launch_bounds__(128) decay_chunk_scan_kernel(const DecayChunkP
     if (live && !fresh && j < nv) s = *reinterpret_cast<const float4*>(sp + j);
     S[j] = s.x; S[j + 1] = s.y; S[j + 2] = s.z; S[j + 3] = s.w;
   }
-  auto issue_load = [&](int c) {
-    const int stg = c & 1;
-    const uint8_t* ws = p.ws + ((size_t)(cb + c) * p.H + h) * ws_bytes(KA, p.va);
-    const uint32_t dst = sbase + stg * L::STAGE, bar = bar_load + 8 * stg;
-    mbar_expect_tx(bar, L::STAGE);
-    chunk_bulk(dst, ws, L::V, bar);
-    chunk_bulk(dst + L::V, ws + L::V + vs * CA, CA, bar);
+  const float* gl = p.gl + ((size_t)cb * p.H + h) * 64 * KA + tid;
+  const size_t gl_step = (size_t)p.H * 64 * KA;
+  float decay = own ? gl[0] : 0.f;
+  // rows of a finished output tile leave coalesced, one chunk later (after the barrier that every chunk has anyway)
+  auto flush = [&](int c) {
+    const int rows = min(CC, len - c * CC);
+    const uint32_t tile = sbase + L::OUT + (c & 1) * (CC * L::OUT_ROW);
+    float* o = p.out + ((size_t)(t_begin + c * CC) * p.H + h) * dv + v0;
+    const int col = (tid & 15) * 4;
+    if (col < nv) {
+#pragma unroll 4
+      for (int r = tid >> 4; r < rows; r += 8) *reinterpret_cast<float4*>(o + (size_t)r * p.H * dv + col) = lds128(tile + r * L::OUT_ROW + col * 4);
+    }
   };
-  if (tid == 0) issue_load(0);
   constexpr uint32_t idesc = umma_idesc_bf16(128, CV, 0, 1), idesc_t = umma_idesc_bf16(128, CV, 1, 1);
   bool ok = true;
   for (int c = 0; c < nc && ok; ++c) {
-    const uint32_t st = sbase + (c & 1) * L::STAGE;
-    const float decay = tid < 64 * KA ? p.gl[((size_t)(cb + c) * p.H + h) * 64 * KA + tid] : 0.f;
-    if (tid < 64 * KA) {
+    const uint32_t st = sbase + (c % NS) * L::STAGE;
+    if (own) {
 #pragma unroll
       for (int ch = 0; ch < 8; ++ch) {
         uint32_t hi[4], lo[4];
@@ -445,16 +489,15 @@ __global__ void __launch_bounds__(128) decay_chunk_scan_kernel(const DecayChunkP
           hi[e] = pack_bf16(x, y);
           lo[e] = pack_bf16(x - bf16_lo(hi[e]), y - bf16_hi(hi[e]));
         }
-        *reinterpret_cast<uint4*>(smem + L::SHI + sw128_offset(tid, ch)) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
-        *reinterpret_cast<uint4*>(smem + L::SLO + sw128_offset(tid, ch)) = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+        sts128(sbase + L::SHI + sw128_offset(tid, ch), hi[0], hi[1], hi[2], hi[3]);
+        sts128(sbase + L::SLO + sw128_offset(tid, ch), lo[0], lo[1], lo[2], lo[3]);
       }
     }
     fence_proxy_async();
     tc_fence_before();
     __syncthreads();
     if (tid == 0) {
-      if (c + 1 < nc) issue_load(c + 1);                 // that stage's readers (the MMAs of chunk c - 1) have completed
-      if (mbar_wait(bar_load + 8 * (c & 1), (c >> 1) & 1, p.status, ERR_MBAR_TIMEOUT_PRODUCER, abort_flag)) {
+      if (mbar_wait(bar_load + 8 * (c % NS), (c / NS) & 1, p.status, ERR_MBAR_TIMEOUT_PRODUCER, abort_flag)) {
         tc_fence_after();
 #pragma unroll
         for (int kk = 0; kk < CC / 16; ++kk)             // state increment [key][value]
@@ -467,14 +510,17 @@ __global__ void __launch_bounds__(128) decay_chunk_scan_kernel(const DecayChunkP
         for (int part = 0; part < 2; ++part)
 #pragma unroll
           for (int kk = 0; kk < KA * 4; ++kk)
-            umma_bf16(tmem, umma_desc_k_sw128(st + L::Q + (kk >> 2) * CA + (kk & 3) * 32), umma_desc_mn_sw128(sbase + (part ? L::SLO : L::SHI) + kk * 2048, 2 * CA, 1024),
+            umma_bf16(tmem, umma_desc_k_sw128(st + L::Q + (kk >> 2) * CA + (kk & 3) * 32), umma_desc_mn_sw128(sbase + (part ? L::SLO : L::SHI) + kk * 2048, KA * CA, 1024),
                       idesc, 1);
         umma_commit(bar_o);
+        if (c + NS - 1 < nc) issue_load(c + NS - 1);     // the stage of chunk c - 1, whose readers have completed
       }
     }
+    const float decay_next = own && c + 1 < nc ? gl[(c + 1) * gl_step] : 0.f;
+    if (c) flush(c - 1);
     if (!(ok = mbar_wait(bar_inc, c & 1, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag))) break;
     tc_fence_after();
-    if (warp < 2 * KA) {
+    if (own) {                                           // (whole warps)
       uint32_t d0[32], d1[32];
       tmem_ld_32x32(tmem + tm_lane + CV, d0);
       tmem_ld_32x32(tmem + tm_lane + CV + 32, d1);
@@ -485,6 +531,7 @@ __global__ void __launch_bounds__(128) decay_chunk_scan_kernel(const DecayChunkP
         S[32 + j] = fmaf(decay, S[32 + j], __uint_as_float(d1[j]));
       }
     }
+    decay = decay_next;
     if (!(ok = mbar_wait(bar_o, c & 1, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag))) break;
     tc_fence_after();
     if (warp < 2) {
@@ -492,27 +539,24 @@ __global__ void __launch_bounds__(128) decay_chunk_scan_kernel(const DecayChunkP
       tmem_ld_32x32(tmem + tm_lane, d0);
       tmem_ld_32x32(tmem + tm_lane + 32, d1);
       tmem_ld_wait();
-      if (tid < min(CC, len - c * CC)) {
-        float* o = p.out + ((size_t)(t_begin + c * CC + tid) * p.H + h) * dv + v0;
+      const uint32_t row = sbase + L::OUT + (c & 1) * (CC * L::OUT_ROW) + tid * L::OUT_ROW;
 #pragma unroll
-        for (int j = 0; j < CV; j += 4) {
-          const uint32_t* s = j < 32 ? d0 : d1;
-          if (j < nv)
-            *reinterpret_cast<float4*>(o + j) = make_float4(__uint_as_float(s[j & 31]), __uint_as_float(s[(j & 31) + 1]), __uint_as_float(s[(j & 31) + 2]),
-                                                            __uint_as_float(s[(j & 31) + 3]));
-        }
+      for (int j = 0; j < 32; j += 4) {
+        sts128(row + 4 * j, d0[j], d0[j + 1], d0[j + 2], d0[j + 3]);
+        sts128(row + 128 + 4 * j, d1[j], d1[j + 1], d1[j + 2], d1[j + 3]);
       }
     }
   }
+  if (!ok)
+    for (int i = 0; i < 200; ++i) __nanosleep(1000);     // a wait ran out: let copies in flight land before shared memory is released
+  tc_fence_before();
+  __syncthreads();
   if (ok) {
+    flush(nc - 1);
 #pragma unroll
     for (int j = 0; j < CV; j += 4)
       if (live && j < nv) *reinterpret_cast<float4*>(sp + j) = make_float4(S[j], S[j + 1], S[j + 2], S[j + 3]);
-  } else {
-    for (int i = 0; i < 200; ++i) __nanosleep(1000);     // a wait ran out: let copies in flight land before shared memory is released
   }
-  tc_fence_before();
-  __syncthreads();
   if (warp == 0) tmem_dealloc(tmem, 128);
 }
 
@@ -527,7 +571,7 @@ static int launch_decay_chunk(const DecayChunkParams& p, int T, cudaStream_t st)
     configured.mark();
   }
   const dim3 grid((unsigned)(T / CC + p.B), (unsigned)p.H);
-  if (p.z) launch_pdl(decay_data_prep_kernel<KA>, grid, dim3(256 * KA), (size_t)DataSmem<KA>::TOTAL, st, p);
+  if (p.z) launch_pdl(decay_data_prep_kernel<KA>, grid, dim3(128 * KA), (size_t)DataSmem<KA>::TOTAL, st, p);
   else launch_pdl(decay_fixed_prep_kernel<KA>, grid, dim3(256), (size_t)FixedSmem<KA>::TOTAL, st, p);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
