@@ -13,8 +13,8 @@
 //       e^80 -- inside the range of bf16, whose relative precision does not depend on size; a chunk in which it would grow further forms those 16 x 16
 //       products one by one in fp32.
 //   decay_chunk_scan_kernel  one CTA per (sequence, head, 64 value columns), chunks in order.  The state slice stays in registers (thread = key channel);
-//       once per chunk it goes to shared memory as a bf16 high + low pair, Q'' S0 + M V and KD^T V run as one MMA batch, and the next chunk's images
-//       arrive by bulk copies meanwhile.
+//       once per chunk it goes to shared memory as a bf16 high + low pair for Q'' S0.  KD is a high + low pair too, so that what a state gathers over
+//       thousands of tokens is not rounded to 16 bits on its way in.
 //
 // Rows past a sequence's end are zero in every image and leave the state as it is.  A operands have 64 rows: the MMA's other 64 rows read whatever image
 // follows in shared memory, and their results are never read.  Every wait is bounded (status word).
@@ -38,7 +38,7 @@ struct DecayChunkParams {
   const int* cu_q; const int* seq_lens; const int* slots;
   float* state;                                    // [slots][H][dk][dv]
   float* out;                                      // [T][H * dv]
-  uint8_t* ws;                                     // per (chunk, head): Q'' | KD | M | V
+  uint8_t* ws;                                     // per (chunk, head): Q'' | KD high, low | M | V
   float* gl;                                       // [chunk][head][64 KA]: e^{G_last}
   int q_ld, k_ld, v_ld, B, H, dk, dv, silu, va;    // va: 64-column slices of V
   int* status;
@@ -57,7 +57,7 @@ __device__ __forceinline__ bool chunk_locate(const int* __restrict__ cu_q, int B
   }
   return false;
 }
-__host__ __device__ constexpr int ws_bytes(int ka, int va) { return (2 * ka + 1 + va) * CA; }
+__host__ __device__ constexpr int ws_bytes(int ka, int va) { return (3 * ka + 1 + va) * CA; }
 
 __device__ __forceinline__ void unpack8(uint4 r, float (&v)[8]) {
   v[0] = bf16_lo(r.x); v[1] = bf16_hi(r.x); v[2] = bf16_lo(r.y); v[3] = bf16_hi(r.y); v[4] = bf16_lo(r.z); v[5] = bf16_hi(r.z); v[6] = bf16_lo(r.w); v[7] = bf16_hi(r.w);
@@ -120,7 +120,7 @@ __global__ void __launch_bounds__(256) decay_fixed_prep_kernel(const DecayChunkP
   uint8_t* ws = p.ws + ((size_t)blockIdx.x * p.H + h) * ws_bytes(KA, p.va);
   for (int i = tid; i < CC * KA * 8; i += 256) {
     const int r = i / (KA * 8), c = i % (KA * 8);
-    uint4 xq = make_uint4(0, 0, 0, 0), xk = xq, xq2 = xq, xk2 = xq;
+    uint4 xq = make_uint4(0, 0, 0, 0), xk = xq, xq2 = xq, xk2 = xq, xk3 = xq;
     if (r < n && 8 * c < p.dk) {
       xq = *reinterpret_cast<const uint4*>(p.q + (size_t)(t0 + r) * p.q_ld + (size_t)h * p.dk + 8 * c);
       xk = *reinterpret_cast<const uint4*>(p.k + (size_t)(t0 + r) * p.k_ld + (size_t)h * p.dk + 8 * c);
@@ -133,12 +133,18 @@ __global__ void __launch_bounds__(256) decay_fixed_prep_kernel(const DecayChunkP
       for (int e = 0; e < 8; ++e) { q[e] *= eq; k[e] *= ek; }
       xq2 = pack8(q);
       xk2 = pack8(k);
+      float hi[8];
+      unpack8(xk2, hi);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) k[e] -= hi[e];
+      xk3 = pack8(k);
     }
     const uint32_t at = atom_offset(r, c);
     *reinterpret_cast<uint4*>(smem + L::Q + at) = xq;
     *reinterpret_cast<uint4*>(smem + L::K + at) = xk;
     *reinterpret_cast<uint4*>(ws + at) = xq2;
     *reinterpret_cast<uint4*>(ws + KA * CA + at) = xk2;
+    *reinterpret_cast<uint4*>(ws + 2 * KA * CA + at) = xk3;
   }
   fence_proxy_async();
   __syncthreads();
@@ -152,7 +158,7 @@ __global__ void __launch_bounds__(256) decay_fixed_prep_kernel(const DecayChunkP
     }
     umma_commit(mbar);
   }
-  value_image(p, ws + (2 * KA + 1) * CA, h, t0, n, tid, 256);
+  value_image(p, ws + (3 * KA + 1) * CA, h, t0, n, tid, 256);
   if (tid < 64 * KA) p.gl[((size_t)blockIdx.x * p.H + h) * 64 * KA + tid] = pw[n];
   const bool ok = mbar_wait(mbar, 0, p.status, ERR_MBAR_TIMEOUT_EPILOGUE, abort_flag, 32);
   tc_fence_after();
@@ -169,7 +175,7 @@ __global__ void __launch_bounds__(256) decay_fixed_prep_kernel(const DecayChunkP
         const int j = col0 + 8 * ch + e;
         m[e] = j <= i ? pw[i - j < 0 ? 0 : i - j] * __uint_as_float(c[8 * ch + e]) : 0.f;
       }
-      *reinterpret_cast<uint4*>(ws + 2 * KA * CA + sw128_offset(i, (col0 >> 3) + ch)) = pack8(m);
+      *reinterpret_cast<uint4*>(ws + 3 * KA * CA + sw128_offset(i, (col0 >> 3) + ch)) = pack8(m);
     }
   }
   tc_fence_before();
@@ -194,11 +200,6 @@ struct DataSmem {
 __device__ __forceinline__ void sts32(uint32_t addr, uint32_t v) { asm volatile("st.shared.b32 [%0], %1;" ::"r"(addr), "r"(v) : "memory"); }
 __device__ __forceinline__ void sts128(uint32_t addr, uint32_t a, uint32_t b, uint32_t c, uint32_t d) {
   asm volatile("st.shared.v4.b32 [%0], {%1, %2, %3, %4};" ::"r"(addr), "r"(a), "r"(b), "r"(c), "r"(d) : "memory");
-}
-__device__ __forceinline__ float4 lds128(uint32_t addr) {
-  float4 v;
-  asm volatile("ld.shared.v4.f32 {%0, %1, %2, %3}, [%4];" : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w) : "r"(addr));
-  return v;
 }
 
 template <int KA>
@@ -308,7 +309,9 @@ __global__ void __launch_bounds__(128 * KA, 4 / KA) decay_data_prep_kernel(const
       if (side) sts32(sb + side + at, pack_bf16(d0, d1));
       if (J < 2) sts32(sb + (WB_KH >> 3) * 1024 + at, pack_bf16(d0 * eh[0], d1 * eh[1]));
       *reinterpret_cast<uint32_t*>(gq + at) = pack_bf16(r0 * eb[0], r1 * eb[1]);
-      *reinterpret_cast<uint32_t*>(gq + KA * CA + at) = pack_bf16(d0 * ea[0], d1 * ea[1]);
+      const uint32_t kd = pack_bf16(d0 * ea[0], d1 * ea[1]);
+      *reinterpret_cast<uint32_t*>(gq + KA * CA + at) = kd;
+      *reinterpret_cast<uint32_t*>(gq + 2 * KA * CA + at) = pack_bf16(d0 * ea[0] - bf16_lo(kd), d1 * ea[1] - bf16_hi(kd));
       if (slow) {
         logs[(16 * J + t) * LS + c] = lg[t][0];
         logs[(16 * J + t) * LS + c + 1] = lg[t][1];
@@ -332,7 +335,7 @@ __global__ void __launch_bounds__(128 * KA, 4 / KA) decay_data_prep_kernel(const
     }
     umma_commit(mbar);
   }
-  value_image(p, ws + (2 * KA + 1) * CA, h, t0, n, tid, THREADS);
+  value_image(p, ws + (3 * KA + 1) * CA, h, t0, n, tid, THREADS);
   if (slow) {                                            // products inside the blocks one by one: no factor is formed that could leave fp32's range
     for (int e = tid; e < CC * 16; e += THREADS) {
       const int i = e >> 4, j = (i & ~15) + (e & 15);
@@ -365,7 +368,7 @@ __global__ void __launch_bounds__(128 * KA, 4 / KA) decay_data_prep_kernel(const
       own[j] = j < at ? __uint_as_float(lo ? d[j] : d[16 + j]) : j == at ? b : 0.f;
       if (slow && j < at) own[j] = diag[i * 16 + j];
     }
-    uint8_t* wm = ws + 2 * KA * CA;
+    uint8_t* wm = ws + 3 * KA * CA;
     auto store16 = [&](int Jc, const float (&v)[16]) {
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
@@ -397,32 +400,42 @@ __global__ void __launch_bounds__(128 * KA, 4 / KA) decay_data_prep_kernel(const
 }
 
 // ------------------------------------------------------------------------------------------------ scan
+// Eight warps:  0 - 3  state (thread = key channel): S as a bf16 pair to shared memory, increment from TMEM, S <- decay S + increment
+//               4, 5   output rows from TMEM to memory (row = token)
+//               6      MMAs:  KD^T V (high and low part of KD) into one of two increments; M V + Q'' [S_high | S_low] into one of two outputs
+//               7      bulk copies of the images, three chunks in flight
+// The increment of a chunk does not depend on the state, so it is issued behind the previous chunk's output product and is there when the state warps
+// want it; their conversion of the next state overlaps it.
 template <int KA>
 struct ChunkScanSmem {
-  static constexpr int NS = 3;                                           // stages: images of this chunk and the next two
-  static constexpr int Q = 0, KD = KA * CA, M = 2 * KA * CA, V = M + CA, STAGE = V + CA;
+  static constexpr int NS = 3;
+  static constexpr int Q = 0, KD = KA * CA, KL = 2 * KA * CA, M = 3 * KA * CA, V = M + CA, STAGE = V + CA;
   static constexpr int SHI = NS * STAGE, SLO = SHI + KA * CA;            // state slice: [64 KA keys][64 values] high and low part
-  static constexpr int OUT = SLO + KA * CA, OUT_ROW = CV * 4 + 16;       // two output tiles [64 tokens][64 values] fp32
-  static constexpr int BARS = OUT + 2 * CC * OUT_ROW;
-  static constexpr int TOTAL = BARS + 64 + 1024;
+  static constexpr int BARS = SLO + KA * CA;
+  static constexpr int TOTAL = BARS + 128 + 1024;
   static_assert(TOTAL <= 232448, "shared memory plan exceeds 227 KB");
 };
+constexpr int SCAN_THREADS = 256, TM_INC = 256;          // TMEM: outputs at 0 and 128 (high | low), increments at 256 and 320
 __device__ __forceinline__ void chunk_bulk(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
   asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
 }
+__device__ __forceinline__ void stg256(float* p, const float (&v)[8]) {
+  asm volatile("st.global.v8.f32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(p), "f"(v[0]), "f"(v[1]), "f"(v[2]), "f"(v[3]), "f"(v[4]), "f"(v[5]), "f"(v[6]),
+               "f"(v[7]) : "memory");
+}
 
 template <int KA>
-__global__ void __launch_bounds__(128) decay_chunk_scan_kernel(const DecayChunkParams p) {
+__global__ void __launch_bounds__(SCAN_THREADS) decay_chunk_scan_kernel(const DecayChunkParams p) {
   using L = ChunkScanSmem<KA>;
   constexpr int NS = L::NS;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
   const uint32_t sbase = smem_u32(smem);
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + L::BARS);
-  const uint32_t bar_load = smem_u32(bars), bar_inc = bar_load + 8 * NS, bar_o = bar_inc + 8;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + NS + 2);
+  const uint32_t b_load = smem_u32(bars), b_free = b_load + 8 * NS, b_inc = b_free + 8 * NS, b_out = b_inc + 16, b_ofree = b_out + 16, b_state = b_ofree + 16;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 2 * NS + 7);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  const int tid = threadIdx.x, warp = tid >> 5, h = blockIdx.y, vs = blockIdx.x, b = blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = blockIdx.y, vs = blockIdx.x, b = blockIdx.z;
   pdl_prologue();
   const int t_begin = p.cu_q[b], len = p.cu_q[b + 1] - t_begin;
   if (len <= 0) return;                                  // whole CTA, before any barrier / TMEM use
@@ -430,56 +443,110 @@ __global__ void __launch_bounds__(128) decay_chunk_scan_kernel(const DecayChunkP
   int cb = 0;                                            // index of this sequence's first chunk
   for (int i = 0; i < b; ++i) cb += (p.cu_q[i + 1] - p.cu_q[i] + CC - 1) / CC;
   if (tid == 0) {
-    for (int s = 0; s < NS + 2; ++s) mbar_init(bar_load + 8 * s, 1);
+    for (int s = 0; s < 2 * NS + 4; ++s) mbar_init(b_load + 8 * s, 1);   // load, free, inc, out
+    mbar_init(b_ofree, 2); mbar_init(b_ofree + 8, 2);
+    mbar_init(b_state, 2 * KA);
     *abort_flag = 0;
     fence_mbar_init();
   }
-  if (warp == 0) { tmem_alloc(smem_u32(tmem_slot), 128); tmem_relinquish(); }
+  if (warp == 0) { tmem_alloc(smem_u32(tmem_slot), 512); tmem_relinquish(); }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem = *tmem_slot, tm_lane = (uint32_t)(warp * 32) << 16;
-  auto issue_load = [&](int c) {
-    const uint8_t* ws = p.ws + ((size_t)(cb + c) * p.H + h) * ws_bytes(KA, p.va);
-    const uint32_t dst = sbase + (c % NS) * L::STAGE, bar = bar_load + 8 * (c % NS);
-    mbar_expect_tx(bar, L::STAGE);
-    chunk_bulk(dst, ws, L::V, bar);
-    chunk_bulk(dst + L::V, ws + L::V + vs * CA, CA, bar);
-  };
-  if (tid == 0)
-    for (int c = 0; c < NS - 1 && c < nc; ++c) issue_load(c);
-
-  // thread = key channel; S[j] = its state against value column 64 vs + j
+  const uint32_t tmem = *tmem_slot, tm_lane = (uint32_t)((warp & 3) * 32) << 16;
   const int dv = p.dv, v0 = vs * CV, nv = min(CV, dv - v0);              // (nv is a multiple of 8)
-  const bool live = tid < p.dk, own = tid < 64 * KA;
-  float S[CV];
-  float* sp = p.state + (((size_t)p.slots[b] * p.H + h) * p.dk + tid) * dv + v0;
-  const bool fresh = p.seq_lens[b] == len;
-#pragma unroll
-  for (int j = 0; j < CV; j += 4) {
-    float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (live && !fresh && j < nv) s = *reinterpret_cast<const float4*>(sp + j);
-    S[j] = s.x; S[j + 1] = s.y; S[j + 2] = s.z; S[j + 3] = s.w;
-  }
-  const float* gl = p.gl + ((size_t)cb * p.H + h) * 64 * KA + tid;
-  const size_t gl_step = (size_t)p.H * 64 * KA;
-  float decay = own ? gl[0] : 0.f;
-  // rows of a finished output tile leave coalesced, one chunk later (after the barrier that every chunk has anyway)
-  auto flush = [&](int c) {
-    const int rows = min(CC, len - c * CC);
-    const uint32_t tile = sbase + L::OUT + (c & 1) * (CC * L::OUT_ROW);
-    float* o = p.out + ((size_t)(t_begin + c * CC) * p.H + h) * dv + v0;
-    const int col = (tid & 15) * 4;
-    if (col < nv) {
-#pragma unroll 4
-      for (int r = tid >> 4; r < rows; r += 8) *reinterpret_cast<float4*>(o + (size_t)r * p.H * dv + col) = lds128(tile + r * L::OUT_ROW + col * 4);
-    }
-  };
-  constexpr uint32_t idesc = umma_idesc_bf16(128, CV, 0, 1), idesc_t = umma_idesc_bf16(128, CV, 1, 1);
   bool ok = true;
-  for (int c = 0; c < nc && ok; ++c) {
-    const uint32_t st = sbase + (c % NS) * L::STAGE;
-    if (own) {
+
+  if (warp == 7) {
+    if (lane == 0) {
+      for (int c = 0; c < nc && ok; ++c) {
+        const int s = c % NS;
+        if (c >= NS && !(ok = mbar_wait(b_free + 8 * s, (c / NS - 1) & 1, p.status, ERR_MBAR_TIMEOUT_PRODUCER, abort_flag, 32))) break;
+        const uint8_t* ws = p.ws + ((size_t)(cb + c) * p.H + h) * ws_bytes(KA, p.va);
+        const uint32_t dst = sbase + s * L::STAGE, bar = b_load + 8 * s;
+        mbar_expect_tx(bar, L::STAGE);
+        chunk_bulk(dst, ws, L::V, bar);
+        chunk_bulk(dst + L::V, ws + L::V + vs * CA, CA, bar);
+      }
+    }
+  } else if (warp == 6) {
+    if (lane == 0) {
+      constexpr uint32_t idesc = umma_idesc_bf16(128, CV, 0, 1), idesc2 = umma_idesc_bf16(128, 2 * CV, 0, 1), idesc_t = umma_idesc_bf16(128, CV, 1, 1);
+      auto increment = [&](int c) -> bool {
+        if (!mbar_wait(b_load + 8 * (c % NS), (c / NS) & 1, p.status, ERR_MBAR_TIMEOUT_PRODUCER, abort_flag)) return false;
+        tc_fence_after();
+        const uint32_t st = sbase + (c % NS) * L::STAGE;
+#pragma unroll
+        for (int part = 0; part < 2; ++part)
+#pragma unroll
+          for (int kk = 0; kk < CC / 16; ++kk)
+            umma_bf16(tmem + TM_INC + (c & 1) * CV, umma_desc_mn_sw128(st + (part ? L::KL : L::KD) + kk * 2048, CA, 1024),
+                      umma_desc_mn_sw128(st + L::V + kk * 2048, CA, 1024), idesc_t, (part | kk) != 0);
+        umma_commit(b_inc + 8 * (c & 1));
+        return true;
+      };
+      ok = increment(0);
+      for (int c = 0; c < nc && ok; ++c) {
+        const uint32_t st = sbase + (c % NS) * L::STAGE, out = tmem + (c & 1) * 128;
+        if (!(ok = mbar_wait(b_state, c & 1, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag))) break;
+        if (c >= 2 && !(ok = mbar_wait(b_ofree + 8 * (c & 1), (c / 2 - 1) & 1, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag))) break;
+        tc_fence_after();
+#pragma unroll
+        for (int kk = 0; kk < KA * 4; ++kk)              // (the stage has been waited for by its increment)
+          umma_bf16(out, umma_desc_k_sw128(st + L::Q + (kk >> 2) * CA + (kk & 3) * 32), umma_desc_mn_sw128(sbase + L::SHI + kk * 2048, KA * CA, 1024), idesc2, kk != 0);
+#pragma unroll
+        for (int kk = 0; kk < CC / 16; ++kk)
+          umma_bf16(out, umma_desc_k_sw128(st + L::M + kk * 32), umma_desc_mn_sw128(st + L::V + kk * 2048, CA, 1024), idesc, 1);
+        umma_commit(b_out + 8 * (c & 1));
+        umma_commit(b_free + 8 * (c % NS));
+        // (the state warps have read the increment of chunk c - 1: they have delivered the state of chunk c)
+        if (c + 1 < nc) ok = increment(c + 1);
+      }
+    }
+  } else if (warp >= 4) {
+    const int row = (warp - 4) * 32 + lane;              // token of the chunk == TMEM lane
+    for (int c = 0; c < nc && ok; ++c) {
+      if (!(ok = mbar_wait(b_out + 8 * (c & 1), (c >> 1) & 1, p.status, ERR_MBAR_TIMEOUT_EPILOGUE, abort_flag, 32))) break;
+      tc_fence_after();
+      const uint32_t ta = tmem + tm_lane + (c & 1) * 128;
+      uint32_t d0[32], d1[32], e0[32], e1[32];
+      tmem_ld_32x32(ta, d0);
+      tmem_ld_32x32(ta + 32, d1);
+      tmem_ld_32x32(ta + 64, e0);
+      tmem_ld_32x32(ta + 96, e1);
+      tmem_ld_wait();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(b_ofree + 8 * (c & 1));
+      if (row < min(CC, len - c * CC)) {
+        float* o = p.out + ((size_t)(t_begin + c * CC + row) * p.H + h) * dv + v0;
+#pragma unroll
+        for (int j = 0; j < CV; j += 8) {
+          float v[8];
+#pragma unroll
+          for (int e = 0; e < 8; ++e)
+            v[e] = j < 32 ? __uint_as_float(d0[(j & 31) + e]) + __uint_as_float(e0[(j & 31) + e]) : __uint_as_float(d1[(j & 31) + e]) + __uint_as_float(e1[(j & 31) + e]);
+          if (j < nv) stg256(o + j, v);
+        }
+      }
+    }
+  } else if (warp < 2 * KA) {
+    // thread = key channel; S[j] = its state against value column 64 vs + j
+    const bool live = tid < p.dk;
+    float S[CV];
+    float* sp = p.state + (((size_t)p.slots[b] * p.H + h) * p.dk + tid) * dv + v0;
+    const bool fresh = p.seq_lens[b] == len;
+#pragma unroll
+    for (int j = 0; j < CV; j += 4) {
+      float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (live && !fresh && j < nv) s = *reinterpret_cast<const float4*>(sp + j);
+      S[j] = s.x; S[j + 1] = s.y; S[j + 2] = s.z; S[j + 3] = s.w;
+    }
+    const float* gl = p.gl + ((size_t)cb * p.H + h) * 64 * KA + tid;
+    const size_t gl_step = (size_t)p.H * 64 * KA;
+    float decay = gl[0];
+    for (int c = 0; c < nc && ok; ++c) {
+      if (c && !(ok = mbar_wait(b_out + 8 * ((c - 1) & 1), ((c - 1) >> 1) & 1, p.status, ERR_MBAR_TIMEOUT_SOFTMAX, abort_flag))) break;      // its reader is done
 #pragma unroll
       for (int ch = 0; ch < 8; ++ch) {
         uint32_t hi[4], lo[4];
@@ -492,72 +559,36 @@ __global__ void __launch_bounds__(128) decay_chunk_scan_kernel(const DecayChunkP
         sts128(sbase + L::SHI + sw128_offset(tid, ch), hi[0], hi[1], hi[2], hi[3]);
         sts128(sbase + L::SLO + sw128_offset(tid, ch), lo[0], lo[1], lo[2], lo[3]);
       }
-    }
-    fence_proxy_async();
-    tc_fence_before();
-    __syncthreads();
-    if (tid == 0) {
-      if (mbar_wait(bar_load + 8 * (c % NS), (c / NS) & 1, p.status, ERR_MBAR_TIMEOUT_PRODUCER, abort_flag)) {
-        tc_fence_after();
-#pragma unroll
-        for (int kk = 0; kk < CC / 16; ++kk)             // state increment [key][value]
-          umma_bf16(tmem + CV, umma_desc_mn_sw128(st + L::KD + kk * 2048, CA, 1024), umma_desc_mn_sw128(st + L::V + kk * 2048, CA, 1024), idesc_t, kk != 0);
-        umma_commit(bar_inc);
-#pragma unroll
-        for (int kk = 0; kk < CC / 16; ++kk)
-          umma_bf16(tmem, umma_desc_k_sw128(st + L::M + kk * 32), umma_desc_mn_sw128(st + L::V + kk * 2048, CA, 1024), idesc, kk != 0);
-#pragma unroll
-        for (int part = 0; part < 2; ++part)
-#pragma unroll
-          for (int kk = 0; kk < KA * 4; ++kk)
-            umma_bf16(tmem, umma_desc_k_sw128(st + L::Q + (kk >> 2) * CA + (kk & 3) * 32), umma_desc_mn_sw128(sbase + (part ? L::SLO : L::SHI) + kk * 2048, KA * CA, 1024),
-                      idesc, 1);
-        umma_commit(bar_o);
-        if (c + NS - 1 < nc) issue_load(c + NS - 1);     // the stage of chunk c - 1, whose readers have completed
-      }
-    }
-    const float decay_next = own && c + 1 < nc ? gl[(c + 1) * gl_step] : 0.f;
-    if (c) flush(c - 1);
-    if (!(ok = mbar_wait(bar_inc, c & 1, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag))) break;
-    tc_fence_after();
-    if (own) {                                           // (whole warps)
+      fence_proxy_async();
+      tc_fence_before();                                 // (the previous increment's TMEM reads too)
+      __syncwarp();
+      if (lane == 0) mbar_arrive(b_state);
+      const float decay_next = c + 1 < nc ? gl[(c + 1) * gl_step] : 0.f;
+      if (!(ok = mbar_wait(b_inc + 8 * (c & 1), (c >> 1) & 1, p.status, ERR_MBAR_TIMEOUT_SOFTMAX, abort_flag))) break;
+      tc_fence_after();
       uint32_t d0[32], d1[32];
-      tmem_ld_32x32(tmem + tm_lane + CV, d0);
-      tmem_ld_32x32(tmem + tm_lane + CV + 32, d1);
+      const uint32_t ta = tmem + tm_lane + TM_INC + (c & 1) * CV;
+      tmem_ld_32x32(ta, d0);
+      tmem_ld_32x32(ta + 32, d1);
       tmem_ld_wait();
 #pragma unroll
       for (int j = 0; j < 32; ++j) {
         S[j] = fmaf(decay, S[j], __uint_as_float(d0[j]));
         S[32 + j] = fmaf(decay, S[32 + j], __uint_as_float(d1[j]));
       }
+      decay = decay_next;
     }
-    decay = decay_next;
-    if (!(ok = mbar_wait(bar_o, c & 1, p.status, ERR_MBAR_TIMEOUT_MMA, abort_flag))) break;
-    tc_fence_after();
-    if (warp < 2) {
-      uint32_t d0[32], d1[32];
-      tmem_ld_32x32(tmem + tm_lane, d0);
-      tmem_ld_32x32(tmem + tm_lane + 32, d1);
-      tmem_ld_wait();
-      const uint32_t row = sbase + L::OUT + (c & 1) * (CC * L::OUT_ROW) + tid * L::OUT_ROW;
+    if (ok) {
 #pragma unroll
-      for (int j = 0; j < 32; j += 4) {
-        sts128(row + 4 * j, d0[j], d0[j + 1], d0[j + 2], d0[j + 3]);
-        sts128(row + 128 + 4 * j, d1[j], d1[j + 1], d1[j + 2], d1[j + 3]);
-      }
+      for (int j = 0; j < CV; j += 4)
+        if (live && j < nv) *reinterpret_cast<float4*>(sp + j) = make_float4(S[j], S[j + 1], S[j + 2], S[j + 3]);
     }
   }
-  if (!ok)
+  if (*abort_flag)
     for (int i = 0; i < 200; ++i) __nanosleep(1000);     // a wait ran out: let copies in flight land before shared memory is released
   tc_fence_before();
   __syncthreads();
-  if (ok) {
-    flush(nc - 1);
-#pragma unroll
-    for (int j = 0; j < CV; j += 4)
-      if (live && j < nv) *reinterpret_cast<float4*>(sp + j) = make_float4(S[j], S[j + 1], S[j + 2], S[j + 3]);
-  }
-  if (warp == 0) tmem_dealloc(tmem, 128);
+  if (warp == 0) tmem_dealloc(tmem, 512);
 }
 
 template <int KA>
@@ -575,7 +606,7 @@ static int launch_decay_chunk(const DecayChunkParams& p, int T, cudaStream_t st)
   else launch_pdl(decay_fixed_prep_kernel<KA>, grid, dim3(256), (size_t)FixedSmem<KA>::TOTAL, st, p);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return (int)e;
-  launch_pdl(decay_chunk_scan_kernel<KA>, dim3((unsigned)p.va, (unsigned)p.H, (unsigned)p.B), dim3(128), (size_t)ChunkScanSmem<KA>::TOTAL, st, p);
+  launch_pdl(decay_chunk_scan_kernel<KA>, dim3((unsigned)p.va, (unsigned)p.H, (unsigned)p.B), dim3(SCAN_THREADS), (size_t)ChunkScanSmem<KA>::TOTAL, st, p);
   return (int)cudaGetLastError();
 }
 
@@ -596,7 +627,8 @@ MX_HOST_API int mx_decay_scan_chunked(const void* q, int q_ld, const void* k, in
   if (B <= 0 || H <= 0 || T <= 0) return 0;
   if (dk < 8 || dk > 128 || dk % 8 || dv < 8 || dv % 8 || q_ld % 8 || k_ld % 8 || v_ld % 8 || H > 65535 || B > 65535) return -112;
   if ((z != nullptr) == (decay != nullptr) || (z && (!u || silu))) return -109;
-  if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)ws | (uintptr_t)state | (uintptr_t)out) & 15) return -112;
+  if (((uintptr_t)q | (uintptr_t)k | (uintptr_t)v | (uintptr_t)ws | (uintptr_t)state) & 15) return -112;
+  if ((uintptr_t)out & 31) return -112;
   DecayChunkParams p;
   p.q = (const bf16*)q; p.k = (const bf16*)k; p.v = (const bf16*)v; p.z = z; p.u = u; p.decay = decay; p.cu_q = cu_q; p.seq_lens = seq_lens; p.slots = slots;
   p.state = state; p.out = out; p.ws = (uint8_t*)ws; p.gl = gl; p.q_ld = q_ld; p.k_ld = k_ld; p.v_ld = v_ld; p.B = B; p.H = H; p.dk = dk; p.dv = dv;
