@@ -257,11 +257,20 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       }
       // a tile needs per-key masking only at the diagonal, at the window edge and at the sequence end
       if ((key0 + BKV - 1 > pos0) || (p.window > 0 && key0 <= pos0 + FA_BQ - 1 - p.window) || (key0 + BKV > seq_len)) {
+        if (key0 < p.keep_first) {
 #pragma unroll
-        for (int i = 0; i < BKV; ++i) {
-          const int kpos = key0 + i;
-          const bool keep = kpos <= qpos && kpos < seq_len && (p.window <= 0 || kpos > qpos - p.window || kpos < p.keep_first);
-          sv[i] = keep ? sv[i] : -INFINITY;
+          for (int i = 0; i < BKV; ++i) {
+            const int kpos = key0 + i;
+            const bool keep = kpos <= qpos && kpos < seq_len && (kpos > qpos - p.window || kpos < p.keep_first);
+            sv[i] = keep ? sv[i] : -INFINITY;
+          }
+        } else {
+#pragma unroll
+          for (int i = 0; i < BKV; ++i) {
+            const int kpos = key0 + i;
+            const bool keep = kpos <= qpos && kpos < seq_len && (p.window <= 0 || kpos > qpos - p.window);
+            sv[i] = keep ? sv[i] : -INFINITY;
+          }
         }
       }
       float tmax = sv[0];

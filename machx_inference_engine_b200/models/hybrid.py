@@ -193,12 +193,21 @@ class MinGRUBlock:
         return self.out(s)
 
 
+MAX_DECAY_KEY = 256      # key channels per head that the decaying-state kernels take
+
+
+def _check_key_width(prefix: str, dim: int) -> None:
+    if round_up(dim, 8) > MAX_DECAY_KEY:
+        raise ValueError(f"{prefix}: {dim} key channels per head are more than the {MAX_DECAY_KEY} the kernels take")
+
+
 class DecayAttentionBlock:
     """Linear attention with a fixed decay per head (lightning attention): q, k, v = silu of their projections, S <- decay S + k v^T, o = S^T q; the heads
     RMS-normed together, times the sigmoid of a gate, output projection.  ``parts`` are the rows [q | k | v | gate] of one projection (see
     KeyValueAttentionBlock); head widths are padded to multiples of 8 at load."""
 
     def __init__(self, src, prefix: str, layer: int, hidden: int, row: int, heads: int, key_dim: int, value_dim: int, decay, eps: float):
+        _check_key_width(prefix, key_dim)
         self.layer, self.H, self.eps, self.live = layer, heads, eps, heads * value_dim
         dk, dv = self.dk, self.dv = round_up(key_dim, 8), round_up(value_dim, 8)
         rows = lambda n, d, to: (src.matrix(f"{prefix}.{n}", heads * d, hidden).pad_groups(rows=(heads, to), cols=(1, row)), None)
@@ -229,6 +238,7 @@ class WkvBlock:
     MIXES = ("r", "k", "v", "g", "w")
 
     def __init__(self, src, prefix: str, layer: int, hidden: int, row: int, heads: int, dim: int, rank: int, eps: float, act_dtype: torch.dtype):
+        _check_key_width(prefix, dim)
         self.layer, self.H, self.dim, self.eps, self.act_dtype = layer, heads, dim, eps, act_dtype
         d = self.d = round_up(dim, 8)
         rank = src.shape(f"{prefix}.w1")[0] if hasattr(src, "shape") else rank or 16

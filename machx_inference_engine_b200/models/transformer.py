@@ -405,6 +405,8 @@ class KeyValueAttentionBlock:
     One projection gives the columns [q | k | gate]; the queries are rotated where they stand, keys and values go into the cache pages.  ``parts`` are the
     projection's row blocks, so that a mixer that reads the same input can share it.  Head widths are padded to multiples of 8 at load."""
 
+    MAX_DIM = 512
+
     def __init__(self, src, prefix: str, layer: int, hidden: int, row: int, heads: int, kv_heads: int, dim: int, scale: float, window: int, keep_first: int,
                  rot_dim: int, rope: tuple, eps: float, interleaved: bool = False, biased: bool = False, qk_norm: bool = False, norm_after: bool = False,
                  head_gate: bool = False, zero_sink: bool = False):
@@ -412,6 +414,8 @@ class KeyValueAttentionBlock:
         self.window, self.keep_first = window, keep_first
         self.rot_dim, self.rope, self.interleaved, self.norm_after = rot_dim, rope, interleaved, norm_after
         dp = self.dp = round_up(dim, 8)
+        if dp > self.MAX_DIM:
+            raise ValueError(f"{prefix}: heads of {dim} elements are wider than the {self.MAX_DIM} the kernels take")
 
         def rows(name, n, d, to):
             w = src.matrix(f"{prefix}.{name}", n * d, hidden).pad_groups(rows=(n, to), cols=(1, row))

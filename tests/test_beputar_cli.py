@@ -69,6 +69,13 @@ def test_loader_checks_tensors(tmp_path):
         model.new_kv_cache(2, "int8")
 
 
+def test_widths_past_the_kernels_are_refused_at_load():
+    for layer in (oracle.attention_layer(None, 1, 1, 520, 8, 8), oracle.wkv_layer(None, 1, 264),
+                  oracle.parallel_layer(None, oracle.attention_sizes(1, 1, 8, 8, 8), 1, 264, 8, (0.5,))):
+        with pytest.raises(ValueError, match="kernels take"):
+            build_model(read_json_config(oracle.random_config([layer])), "cpu", quant="bf16")
+
+
 @pytest.mark.parametrize("rank", [1, 8, 33])
 def test_inner_width_of_the_decay_comes_from_its_tensors(tmp_path, rank):
     w = oracle.random_weights(CFG, rank=rank)
