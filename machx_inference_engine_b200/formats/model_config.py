@@ -586,16 +586,16 @@ def _pubodra_preset(hidden, n_layers, heads, dim, rot_dim, vdim, kv_rank, window
 
 
 def _beputar_preset(hidden, n_layers, heads, kv_heads, dim, window, keep_first, lin_heads, lin_dim, lin_vdim, wkv_heads, wkv_dim, decay_rank, ffn, vocab, experts=0,
-                    used=0, expert_ffn=0, shared=0, order=("parallel", "rotary_attention", "wkv"), theta=1e6, yarn=(8.0, 2048.0, 32.0, 1.0)) -> ModelConfig:
+                    used=0, expert_ffn=0, shared=0, order=("parallel", "rotary_attention", "wkv"), theta=5e5, yarn=(4.0, 4096.0, 32.0, 1.0)) -> ModelConfig:
     """The mixers of ``order`` in turn; the first layer has a dense feed-forward, the others experts (when there are any)."""
-    c = ModelConfig(arch="beputar", hidden=hidden, vocab=vocab, rms_eps=1e-6, tie_embeddings=True, embedding_scale=12.0)
+    c = ModelConfig(arch="beputar", hidden=hidden, vocab=vocab, rms_eps=1e-6, tie_embeddings=True, embedding_scale=16.0)
     for l in range(n_layers):
         s = LayerSpec(order[l % len(order)])
         if s.mixer == "wkv":
             s.lin_heads, s.lin_key_dim, s.lin_value_dim, s.decay_rank = wkv_heads, wkv_dim, wkv_dim, decay_rank
         else:
             s.heads, s.kv_heads, s.key_dim, s.value_dim, s.window, s.scale = heads, kv_heads, dim, dim, window, dim ** -0.5
-            s.rot_dim, s.rope_theta = (dim // 4 * 2, theta) if s.mixer == "parallel" else (dim, 1e4)
+            s.rot_dim, s.rope_theta = (dim // 4 * 2, theta) if s.mixer == "parallel" else (dim, 2e4)
             s.yarn = None if s.mixer == "parallel" else yarn
         if s.mixer == "parallel":
             s.keep_first, s.lin_heads, s.lin_key_dim, s.lin_value_dim = keep_first, lin_heads, lin_dim, lin_vdim
