@@ -78,8 +78,8 @@ def _folder_bytes(path: str, ctx: int, n_seqs: int) -> tuple:
     from .model_config import read_json_config
     c = read_json_config(path)
     weights = sum(os.path.getsize(os.path.join(path, f)) for f in os.listdir(path) if f.endswith(".safetensors"))
-    kv = sum(c.layer_specs[l].kv_width() for l, _ in c.layer_runs()) * ctx * 2 * n_seqs
-    return weights, kv, sum(s.state_bytes(c.hidden) for s in c.layer_specs) * n_seqs
+    runs = [c.layer_specs[l] for l, _ in c.layer_runs()]
+    return weights, int(sum(s.kv_width() for s in runs) * ctx * 2 * n_seqs), sum(s.state_bytes(c.hidden) for s in runs) * n_seqs
 
 
 def visible_gpus() -> tuple:

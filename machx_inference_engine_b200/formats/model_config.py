@@ -19,7 +19,7 @@ HYBRID_ARCHS = ("qwen3next", "qwen35", "qwen35moe")
 GEMMA_ARCHS = ("gemma4",)
 SUPPORTED_ARCHS = DENSE_ARCHS + MOE_ARCHS + HYBRID_ARCHS + GEMMA_ARCHS
 # checkpoints that are a folder with config.json + safetensors and list their layers one by one: "architecture" value -> arch
-LAYER_LIST_ARCHS = {"Tikarax": "tikarax", "Pubodra": "pubodra", "Beputar": "beputar"}
+LAYER_LIST_ARCHS = {"Tikarax": "tikarax", "Pubodra": "pubodra", "Beputar": "beputar", "Zegelix": "zegelix"}
 
 
 class ConfigError(ValueError):
@@ -30,7 +30,7 @@ class ConfigError(ValueError):
 class LayerSpec:
     """One layer of a design whose configuration lists its layers: a mixer with its sizes and constants, and a feed-forward (``ffn`` wide, or
     ``experts`` of ``expert_ffn`` each with ``experts_used`` per token; none when both are 0)."""
-    mixer: str                     # "attention" | "mingru" | "latent_attention" | "rotary_attention" | "wkv" | "parallel"
+    mixer: str                     # "attention" | "mingru" | "latent_attention" | "rotary_attention" | "wkv" | "parallel" | "pooled_attention" | "rglru"
     ffn: int = 0
     experts: int = 0
     experts_used: int = 0
@@ -49,8 +49,17 @@ class LayerSpec:
     window: int = 0                # keys a query sees, itself included (0 = all before it)
     rope_theta: float = 10000.0
     yarn: Optional[tuple] = None   # (factor, original context, fast turns, slow turns)
-    # minGRU
+    # minGRU, RG-LRU
     width: int = 0
+    # attention over a window and pooled blocks before it: heads .. scale, rot_dim .. rope_theta and window above
+    pool: int = 0                  # tokens of a pooled block (0: what left the window is gone)
+    softcap: float = 0.0           # scores are softcap * tanh(score / softcap) (0: as they are)
+    # RG-LRU: width channels in gate_blocks equal parts behind a causal convolution
+    gate_blocks: int = 0
+    conv_taps: int = 0
+    # clamped gated experts
+    act_limit: float = 0.0
+    shared_limit: float = 0.0
     # rotary attention (and the left half of a parallel mixer): heads .. scale and rot_dim .. yarn above
     keep_first: int = 0            # with a window: the first tokens of a sequence that stay visible
     # experts whose weight scales their input
@@ -62,13 +71,14 @@ class LayerSpec:
     lin_decay: tuple = ()          # per head; empty where the decay comes from the data
     decay_rank: int = 0            # wkv: inner width of the decay's projection (0: as the checkpoint's tensor has it)
 
-    def kv_width(self) -> int:
-        """Cached elements per token."""
-        return self.kv_heads * (self.key_dim + self.value_dim) + (self.kv_rank + self.rot_dim if self.kv_rank else 0)
+    def kv_width(self) -> float:
+        """Cached elements per token (a pooled block's rows count for its tokens)."""
+        return self.kv_heads * (self.key_dim + self.value_dim) * (1 + (1 / self.pool if self.pool else 0)) + (self.kv_rank + self.rot_dim if self.kv_rank else 0)
 
     def state_bytes(self, hidden: int) -> int:
-        """Recurrent state per sequence (fp32): the minGRU row, or a matrix per head and, for wkv, the last row of its input."""
-        return 4 * (self.width + self.lin_heads * self.lin_key_dim * self.lin_value_dim + (hidden if self.mixer == "wkv" else 0))
+        """Recurrent state per sequence (fp32): the minGRU / RG-LRU row with the convolution's last inputs, or a matrix per head and, for wkv, the last
+        row of its input."""
+        return 4 * (self.width * max(self.conv_taps, 1) + self.lin_heads * self.lin_key_dim * self.lin_value_dim + (hidden if self.mixer == "wkv" else 0))
 
 
 @dataclass
@@ -116,8 +126,8 @@ class ModelConfig:
     layer_specs: list = field(default_factory=list)      # LayerSpec per layer
     norm_groups: int = 1                                  # RMS norms run over this many equal parts of the row
     loop_start: int = 0                                   # layers loop_start .. loop_stop - 1 run loop_times times in a row (0: no loop); every
-    loop_stop: int = 0                                    # pass has its own cache and adds a learned vector to the residual first
-    loop_times: int = 0
+    loop_stop: int = 0                                    # pass has its own cache or state and first adds a learned vector to the residual or mixes it
+    loop_times: int = 0                                   # with the embedding output
     # Granite scalars
     embedding_scale: float = 1.0
     residual_scale: float = 1.0
@@ -140,7 +150,7 @@ class ModelConfig:
 
     def layer_is_full_attention(self, layer: int) -> bool:
         if self.layer_specs:
-            return self.layer_specs[layer].mixer in ("attention", "latent_attention", "rotary_attention", "parallel")
+            return self.layer_specs[layer].mixer in ("attention", "latent_attention", "rotary_attention", "parallel", "pooled_attention")
         if not self.is_hybrid:
             return True
         return (layer + 1) % self.full_attn_interval == 0
@@ -358,13 +368,18 @@ def _pubodra_config(d: Mapping[str, Any]) -> ModelConfig:
         elif kind is not None:
             raise ConfigError(f"layer {i}: unknown feed-forward kind {kind!r}")
         c.layer_specs.append(s)
-    if d.get("loop") is not None:
-        c.loop_start, c.loop_stop, c.loop_times = (int(d["loop"][k]) for k in ("start", "stop", "times"))
-        if not 0 <= c.loop_start < c.loop_stop <= len(c.layer_specs) or c.loop_times < 1:
-            raise ConfigError("loop: start .. stop must be a range of layers that runs at least once")
+    _read_loop(c, d)
     if c.hidden < 1 or c.vocab < 1 or not c.layer_specs:
         raise ConfigError("the width must be positive, with at least one layer")
     return _finish_layer_list(c)
+
+
+def _read_loop(c: ModelConfig, d: Mapping[str, Any]) -> None:
+    if d.get("loop") is None:
+        return
+    c.loop_start, c.loop_stop, c.loop_times = (int(d["loop"][k]) for k in ("start", "stop", "times"))
+    if not 0 <= c.loop_start < c.loop_stop <= len(c.layer_specs) or c.loop_times < 1:
+        raise ConfigError("loop: start .. stop must be a range of layers that runs at least once")
 
 
 def _yarn(rot: Mapping[str, Any], where: str) -> Optional[tuple]:
@@ -431,6 +446,47 @@ def _beputar_config(d: Mapping[str, Any]) -> ModelConfig:
     return _finish_layer_list(c)
 
 
+def _zegelix_config(d: Mapping[str, Any]) -> ModelConfig:
+    c = ModelConfig(arch="zegelix", hidden=int(d["width"]), vocab=int(d["vocab"]), rms_eps=float(d["norm"]["eps"]), tie_embeddings=True,
+                    embedding_scale=float(d["embedding"]["scale"]), logit_scale=float(d["logit_scale"]), name=str(d.get("name", "")))
+    for i, e in enumerate(d["layers"]):
+        m, mlp, where = e["mixer"], e.get("mlp"), f"layer {i}"
+        if e["type"] == "attention":
+            rot, mask = m["rot"], m.get("mask")
+            s = LayerSpec("pooled_attention", heads=int(m["heads"]), kv_heads=int(m["kv_heads"]), key_dim=int(m["dim"]), value_dim=int(m["vdim"]),
+                          scale=float(m["scale"]), softcap=float(m.get("softcap") or 0.0), rot_dim=int(rot["dims"]), rope_theta=float(rot["base"]))
+            if min(s.heads, s.kv_heads, s.key_dim, s.value_dim) < 1 or s.heads % s.kv_heads:
+                raise ConfigError(f"{where}: {s.heads} query heads do not divide over {s.kv_heads} key/value heads")
+            if not 0 <= s.rot_dim <= s.key_dim or s.rot_dim % 2 or s.value_dim % 2:
+                raise ConfigError(f"{where}: rot.dims must be even and at most dim, and vdim even")
+            if s.softcap < 0:
+                raise ConfigError(f"{where}: softcap must not be negative")
+            if mask is not None:
+                s.window, s.pool = int(mask["size"]), int(mask.get("pool") or 0)
+                if s.window < 1 or s.pool < 0:
+                    raise ConfigError(f"{where}: mask.size must be positive and mask.pool not negative")
+        elif e["type"] == "rglru":
+            s = LayerSpec("rglru", width=int(m["width"]), gate_blocks=int(m["blocks"]), conv_taps=int(m["conv"]))
+            if min(s.width, s.gate_blocks, s.conv_taps) < 1 or s.width % s.gate_blocks:
+                raise ConfigError(f"{where}: the width must be a multiple of the blocks, with at least one tap")
+        else:
+            raise ConfigError(f"{where}: unknown mixer {e['type']!r}")
+        if mlp is not None:
+            if mlp.get("kind") != "moe":
+                raise ConfigError(f"{where}: unknown feed-forward kind {mlp.get('kind')!r}")
+            s.experts, s.experts_used, s.expert_ffn = int(mlp["router"]["experts"]), int(mlp["router"]["top"]), int(mlp["expert"]["ff"])
+            s.act_limit = float(mlp["expert"]["limit"])
+            if mlp.get("shared") is not None:
+                s.shared_ffn, s.shared_limit = int(mlp["shared"]["ff"]), float(mlp["shared"]["limit"])
+            if not 1 <= s.experts_used <= s.experts:
+                raise ConfigError(f"{where}: {s.experts_used} of {s.experts} experts per token")
+        c.layer_specs.append(s)
+    _read_loop(c, d)
+    if c.hidden < 1 or c.vocab < 1 or not c.layer_specs:
+        raise ConfigError("the width must be positive, with at least one layer")
+    return _finish_layer_list(c)
+
+
 def _finish_layer_list(c: ModelConfig) -> ModelConfig:
     """Derived fields of a layer-list config: the largest sizes of any layer (pool sizing, reports)."""
     big = lambda f, lo=0: max([lo] + [getattr(s, f) for s in c.layer_specs])
@@ -451,7 +507,7 @@ def read_json_config(path_or_dict) -> ModelConfig:
         with open(p) as f:
             d = json.load(f)
     a = d.get("architecture")
-    readers = {"tikarax": _tikarax_config, "pubodra": _pubodra_config, "beputar": _beputar_config}
+    readers = {"tikarax": _tikarax_config, "pubodra": _pubodra_config, "beputar": _beputar_config, "zegelix": _zegelix_config}
     if a not in LAYER_LIST_ARCHS:
         raise ConfigError(f"unsupported architecture {a!r} in config.json (supported: {', '.join(LAYER_LIST_ARCHS)})")
     try:
@@ -484,6 +540,12 @@ def config_to_json(c: ModelConfig) -> dict:
             m = {"heads": s.lin_heads, "dim": s.lin_key_dim}
         elif s.mixer == "parallel":
             m = {"left": rotary(s), "right": {"heads": s.lin_heads, "dim": s.lin_key_dim, "vdim": s.lin_value_dim, "decay": list(s.lin_decay)}}
+        elif s.mixer == "pooled_attention":
+            m = {**rotary(s), **({"softcap": s.softcap} if s.softcap else {})}
+            if s.pool:
+                m["mask"]["pool"] = s.pool
+        elif s.mixer == "rglru":
+            m = {"width": s.width, "blocks": s.gate_blocks, "conv": s.conv_taps}
         elif s.mixer == "attention":
             m = {"heads": s.heads, "kv_heads": s.kv_heads, "dim": s.key_dim, "vdim": s.value_dim, "scale": s.scale,
                  "q_temp": {"coef": s.q_temp_coef, "every": whole(s.q_temp_every)}}
@@ -498,12 +560,18 @@ def config_to_json(c: ModelConfig) -> dict:
             mlp = {"kind": "moe", "expert": {"ff": s.expert_ffn}, "router": {"experts": s.experts, "top": s.experts_used}}
             if s.shared_ffn:
                 mlp["shared"] = {"ff": s.shared_ffn}
-        layers.append({"type": {"rotary_attention": "attention"}.get(s.mixer, s.mixer), "mixer": m, "mlp": mlp})
+            if c.arch == "zegelix":
+                mlp["expert"]["limit"] = s.act_limit
+                if s.shared_ffn:
+                    mlp["shared"]["limit"] = s.shared_limit
+        layers.append({"type": {"rotary_attention": "attention", "pooled_attention": "attention"}.get(s.mixer, s.mixer), "mixer": m, "mlp": mlp})
     arch = {v: k for k, v in LAYER_LIST_ARCHS.items()}[c.arch]
     norm = {"eps": c.rms_eps, "groups": c.norm_groups} if c.arch == "tikarax" else {"eps": c.rms_eps}
     out = {"architecture": arch, "layers": layers, "norm": norm, "vocab": c.vocab, "width": c.hidden}
-    if c.arch == "beputar":
+    if c.arch in ("beputar", "zegelix"):
         out["embedding"] = {"scale": c.embedding_scale}
+    if c.arch == "zegelix":
+        out["logit_scale"] = c.logit_scale
     if c.loop_times:
         out["loop"] = {"start": c.loop_start, "stop": c.loop_stop, "times": c.loop_times}
     return out
@@ -608,6 +676,24 @@ def _beputar_preset(hidden, n_layers, heads, kv_heads, dim, window, keep_first, 
     return _finish_layer_list(c)
 
 
+def _zegelix_preset(hidden, n_layers, heads, kv_heads, dim, vdim, rot_dim, window, pool, softcap, width, blocks, conv, experts, used, expert_ffn, shared, vocab,
+                    attn_every=3, limit=7.0, shared_limit=7.0, loop=None, theta=5e5, embedding_scale=0.0, logit_scale=1.0) -> ModelConfig:
+    """Every ``attn_every``-th layer attention, the others RG-LRU; experts in every layer."""
+    c = ModelConfig(arch="zegelix", hidden=hidden, vocab=vocab, rms_eps=1e-5, tie_embeddings=True, embedding_scale=embedding_scale or math.sqrt(hidden),
+                    logit_scale=logit_scale)
+    for l in range(n_layers):
+        if (l + 1) % attn_every == 0:
+            s = LayerSpec("pooled_attention", heads=heads, kv_heads=kv_heads, key_dim=dim, value_dim=vdim, rot_dim=rot_dim, scale=dim ** -0.5, window=window,
+                          pool=pool, softcap=softcap, rope_theta=theta)
+        else:
+            s = LayerSpec("rglru", width=width, gate_blocks=blocks, conv_taps=conv)
+        s.experts, s.experts_used, s.expert_ffn, s.shared_ffn, s.act_limit, s.shared_limit = experts, used, expert_ffn, shared, limit, shared_limit
+        c.layer_specs.append(s)
+    if loop is not None:
+        c.loop_start, c.loop_stop, c.loop_times = loop
+    return _finish_layer_list(c)
+
+
 # ---- named architectures used by the benches and tests (random-init; see formats/synth.py)
 def preset(name: str) -> ModelConfig:
     p = {
@@ -676,6 +762,11 @@ def preset(name: str) -> ModelConfig:
         # layers of common model sizes: 1 B class and 8 B class
         "beputar-1b": _beputar_preset(2048, 15, 32, 8, 64, 1024, 16, 16, 128, 128, 32, 64, 64, 8192, 128256, experts=64, used=6, expert_ffn=1024, shared=2048),
         "beputar-8b": _beputar_preset(4096, 30, 32, 8, 128, 4096, 16, 32, 128, 128, 64, 64, 64, 16384, 128256, experts=64, used=6, expert_ffn=1536, shared=3072),
+        "tiny-zegelix": _zegelix_preset(160, 3, 6, 2, 40, 56, 24, 50, 5, 30.0, 192, 3, 4, 6, 2, 96, 64, 384, attn_every=2, limit=1.5, shared_limit=2.5,
+                                        loop=(1, 3, 2), theta=2e4, logit_scale=0.75),
+        # layers of common model sizes: 1 B class and 8 B class
+        "zegelix-1b": _zegelix_preset(2048, 15, 32, 8, 64, 64, 32, 1024, 16, 50.0, 2560, 10, 4, 64, 6, 1024, 2048, 128256),
+        "zegelix-8b": _zegelix_preset(4096, 30, 32, 8, 128, 128, 64, 4096, 16, 50.0, 4096, 16, 4, 64, 6, 1536, 3072, 128256),
         "tiny-qwen2": ModelConfig(arch="qwen2", n_layers=2, hidden=256, n_heads=4, n_kv_heads=2, head_dim=64, ffn=512, vocab=2048,
                                   rms_eps=1e-6, rope_theta=1e6, n_rot=64, ctx_train=4096),
         "tiny-phi3": ModelConfig(arch="phi3", n_layers=2, hidden=256, n_heads=4, n_kv_heads=4, head_dim=64, ffn=512, vocab=2048,

@@ -368,9 +368,37 @@ def _beputar_tensors(cfg: ModelConfig) -> list:
     return out
 
 
+def _zegelix_tensors(cfg: ModelConfig) -> list:
+    H = cfg.hidden
+    out = [("embed", "matrix", (cfg.vocab, H)), ("final.norm", "norm", (H,))]
+    if cfg.loop_times:
+        out.append(("loop.in", "matrix", (H, 2 * H)))
+    matrices = lambda p, shapes: [(f"{p}.{n}", "matrix", shape) for n, shape in shapes.items()]
+    vectors = lambda p, shapes: [(f"{p}.{n}", "vector", shape) for n, shape in shapes.items()]
+    for i, s in enumerate(cfg.layer_specs):
+        p, m, q, kv, W = f"l{i}", f"l{i}.mix", s.heads * s.key_dim, s.kv_heads * s.key_dim, s.width
+        out.append((f"{p}.norm1", "norm", (H,)))
+        if s.mixer == "pooled_attention":
+            v, o = s.kv_heads * s.value_dim, s.heads * s.value_dim
+            out += matrices(m, {"q": (q, H), "k": (kv, H), "v": (v, H), "g": (o, H), "o": (H, o)})
+            out += vectors(m, {"q.b": (q,), "k.b": (kv,), "v.b": (v,), "sink": (s.heads,)}) + [(f"{m}.temp", "norm", (s.heads,))]
+        else:
+            b, n = s.gate_blocks, W // s.gate_blocks
+            out += matrices(m, {"y": (W, H), "x": (W, H), "conv": (W, s.conv_taps), "ra": (b, n, n), "ri": (b, n, n), "o": (H, W)})
+            out += vectors(m, {"y.b": (W,), "x.b": (W,), "conv.b": (W,), "ra.b": (b, n), "ri.b": (b, n), "lam": (W,)})
+        gated = lambda n, f: matrices(f"{p}.mlp{n}", {"gate": (f, H), "up": (f, H), "down": (H, f)})
+        for e in range(s.experts):
+            out += gated(f".e{e}", s.expert_ffn)
+        if s.experts:
+            out += [(f"{p}.norm2", "norm", (H,)), (f"{p}.mlp.router", "matrix", (s.experts, H)), (f"{p}.mlp.router.b", "vector", (s.experts,))]
+        if s.shared_ffn:
+            out += gated(".shared", s.shared_ffn) + [(f"{p}.mlp.shared.sg", "matrix", (1, H))]
+    return out
+
+
 def folder_tensor_plan(cfg: ModelConfig) -> list:
     """(name, kind, shape) of every tensor of a layer-list checkpoint folder (``LAYER_LIST_ARCHS``); matrices are [out, in]."""
-    return {"tikarax": _tikarax_tensors, "pubodra": _pubodra_tensors, "beputar": _beputar_tensors}[cfg.arch](cfg)
+    return {"tikarax": _tikarax_tensors, "pubodra": _pubodra_tensors, "beputar": _beputar_tensors, "zegelix": _zegelix_tensors}[cfg.arch](cfg)
 
 
 def write_synthetic_folder(cfg: ModelConfig, path: str, seed: int = 0) -> dict:

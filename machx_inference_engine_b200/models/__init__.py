@@ -11,7 +11,8 @@ from ..parallel.comm import ParallelCtx
 # file names of the tensors that every graph asks for under its GGUF name
 _FOLDER_NAMES = {"tikarax": {"token_embd.weight": "embed", "output_norm.weight": "final.norm", "output.weight": "head"},
                  "pubodra": {"token_embd.weight": "embed", "output_norm.weight": "final.norm"},
-                 "beputar": {"token_embd.weight": "embed", "output_norm.weight": "final.norm"}}
+                 "beputar": {"token_embd.weight": "embed", "output_norm.weight": "final.norm"},
+                 "zegelix": {"token_embd.weight": "embed", "output_norm.weight": "final.norm"}}
 
 
 def _graph_class(cfg: ModelConfig):
@@ -30,6 +31,9 @@ def _graph_class(cfg: ModelConfig):
     if cfg.arch == "beputar":
         from .beputar import BeputarModel
         return BeputarModel
+    if cfg.arch == "zegelix":
+        from .zegelix import ZegelixModel
+        return ZegelixModel
     from .transformer import TransformerModel
     return TransformerModel
 

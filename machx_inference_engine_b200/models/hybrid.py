@@ -15,6 +15,7 @@ snapshots after every position) so a partially accepted draft rolls the recurren
 """
 from __future__ import annotations
 
+import math
 from typing import Optional
 
 import torch
@@ -191,6 +192,45 @@ class MinGRUBlock:
         s = ops.mingru_scan(y[:, :W], y[:, W:2 * W], y[:, 2 * W:], self.zb, self.xb, state.tensors["S"][self.layer], fb.state_slots, fb.cu_q, fb.seq_lens,
                             fb.max_q_len)
         return self.out(s)
+
+
+class RglruBlock:
+    """Real-gated linear recurrent unit behind a causal convolution: one projection [u's input | y], u = conv(.), per block of channels the two gates
+    r, i = sigmoid(W u + b), S <- a S + sqrt(1 - a^2) i u with log a = -8 r softplus(lam), and S gelu(y) through the output projection.
+
+    The matrices of a block's two gates are one stack entry, so a prompt is convolution, per-block GEMM (fp32 results), recurrence with its gates and its
+    output factor; a step of single tokens is one kernel.  Blocks are padded so that each starts on a vector and all together fill rows of 32."""
+
+    def __init__(self, src, prefix: str, hidden: int, row: int, width: int, blocks: int, taps: int):
+        n = width // blocks
+        to = self.n = round_up(n, max(8, 32 // math.gcd(blocks, 32)))
+        self.blocks, self.width = blocks, blocks * to
+        ws = [src.matrix(f"{prefix}.{m}", width, hidden).pad_groups(rows=(blocks, to), cols=(1, row)) for m in ("x", "y")]
+        pad = lambda v: _pad_heads(v, blocks, to)
+        self.proj = _fuse_rows(ws, [pad(src.vector(f"{prefix}.{m}.b", width)) for m in ("x", "y")])
+        self.conv_w = torch.nn.functional.pad(src.table(f"{prefix}.conv", (width, taps)).reshape(blocks, n, taps), (0, 0, 0, to - n)).reshape(-1, taps).contiguous()
+        self.conv_b = pad(src.vector(f"{prefix}.conv.b", width))
+        gate = lambda m: torch.nn.functional.pad(src.table(f"{prefix}.{m}", (blocks, n, n)), (0, to - n, 0, to - n))
+        self.gates = QuantWeight(ops.WFormat.BF16, 2 * to, to, blocks, torch.cat([gate("ra"), gate("ri")], dim=1).to(torch.bfloat16).contiguous())
+        gb = lambda m: torch.nn.functional.pad(src.table(f"{prefix}.{m}.b", (blocks, n)), (0, to - n))
+        self.gate_b = torch.cat([gb("ra"), gb("ri")], dim=1).contiguous()
+        lam = src.vector(f"{prefix}.lam", width).to(torch.float64)
+        self.coef = pad((-8.0 * torch.nn.functional.softplus(lam)).to(torch.float32))
+        self.out = Linear(src.matrix(f"{prefix}.o", hidden, width).pad_groups(rows=(1, row), cols=(blocks, to)))
+
+    def state_tensors(self, n_slots: int, act_dtype: torch.dtype, device) -> dict:
+        return {"S": torch.zeros(n_slots, self.width, dtype=torch.float32, device=device),
+                "conv": torch.zeros(n_slots, self.conv_w.shape[1] - 1, self.width, dtype=act_dtype, device=device)}
+
+    def __call__(self, h: torch.Tensor, fb: ForwardBatch, state: RecurrentState, run: int) -> torch.Tensor:
+        """``run``: which of the state's entries (a layer that runs several times has one per run)."""
+        p, W = self.proj(h), self.width
+        x, y, S, conv = p[:, :W], p[:, W:], state.tensors["S"][run], state.tensors["conv"][run]
+        if fb.max_q_len == 1:
+            return self.out(ops.rglru_step(x, y, self.conv_w, self.conv_b, self.gates, self.gate_b, self.coef, conv, S, fb.state_slots, fb.cu_q, fb.seq_lens))
+        u = ops.causal_conv(x, self.conv_w, self.conv_b, conv, fb.state_slots, fb.cu_q, fb.seq_lens, fb.max_q_len)
+        g = ops.head_linear(u.unflatten(1, (self.blocks, self.n)), self.gates, out_f32=True)
+        return self.out(ops.rglru_scan(g, u, y, self.gate_b, self.coef, S, fb.state_slots, fb.cu_q, fb.seq_lens, fb.max_q_len))
 
 
 MAX_DECAY_KEY = 256      # key channels per head that the decaying-state kernels take

@@ -7,7 +7,7 @@ from typing import Optional
 import torch
 
 from ..formats.model_config import ModelConfig
-from ..ops import QuantWeight
+from ..ops import PoolPages, QuantWeight
 from ..parallel.comm import ParallelCtx
 from .transformer import KVCache, TransformerModel, round_up
 
@@ -42,12 +42,17 @@ class LayerListModel(TransformerModel):
             self._tables[key] = build()
         return self._tables[key]
 
+    def _kv_pools(self) -> dict:
+        """Per layer run with pooled blocks: (tokens per block, window)."""
+        return {}
+
     def new_kv_cache(self, num_blocks: int, dtype: str = "bf16") -> KVCache:
         if dtype == "int8":
             raise ValueError("the int8 KV cache is not built for this design")
         return KVCache(self.cfg.n_layers, num_blocks, self.n_kv_local, self.cfg.head_dim, self.device, list(self.kv_geometry), dtype=self.dtype,
-                       geometry=self.kv_geometry)
+                       geometry=self.kv_geometry, pools=self._kv_pools())
 
     def kv_bytes_per_block(self, dtype: str = "bf16") -> int:
-        per_tok = sum(n * (dk + dv) for n, dk, dv in self.kv_geometry.values())
-        return per_tok * KVCache.BLOCK * (2 if self.dtype == "bf16" else 4)
+        pools = self._kv_pools()
+        rows = lambda l: KVCache.BLOCK + (PoolPages.rows_per_page(KVCache.BLOCK, pools[l][0]) if l in pools else 0)
+        return sum(n * (dk + dv) * rows(l) for l, (n, dk, dv) in self.kv_geometry.items()) * (2 if self.dtype == "bf16" else 4)

@@ -73,7 +73,9 @@ class KVCache:
     """Paged KV: per attention layer ``k, v [num_blocks, n_kv_local, KV_BLOCK, head_dim]`` bf16 or fp32, or int8 with one fp32 scale
     per (block, kv head, token) row in ``ks, vs [num_blocks, n_kv_local, KV_BLOCK]`` (value = q * scale, scale = max|x| / 127).
     ``geometry`` gives layers their own (n_kv, head_dim) or (n_kv, key width, value width); a value width of 0 is a latent cache, whose
-    values are formed from the key rows.  A layer that runs several times has one entry per run.
+    values are formed from the key rows.  A layer that runs several times has one entry per run.  ``pools`` {layer: (tokens per block, window)} gives
+    layers rows for pooled blocks in every page (``pools[layer]``, :class:`ops.PoolPages`): they live and die with the page, so sharing and reuse of
+    pages cover them.
 
     The reference cache is contiguous per sequence (include/ie/kv_cache.hpp:27-114) and keeps int8 rows beside it when
     ``--int8-kv`` is given (src/core/kv_cache.cpp:182-240, src/ops/attention.cpp:145-229); pages make continuous batching
@@ -83,7 +85,7 @@ class KVCache:
     BLOCK = KV_BLOCK
 
     def __init__(self, n_layers: int, num_blocks: int, n_kv: int, head_dim: int, device, attn_layers: Optional[list[int]] = None,
-                 dtype: str = "bf16", geometry: Optional[dict] = None):
+                 dtype: str = "bf16", geometry: Optional[dict] = None, pools: Optional[dict] = None):
         if dtype not in ("bf16", "fp32", "int8"):
             raise ValueError(f"unknown KV cache dtype {dtype!r}")
         self.num_blocks = num_blocks
@@ -94,6 +96,8 @@ class KVCache:
         geo = {l: ((geometry or {}).get(l) or (n_kv, head_dim)) for l in layers}       # per layer: Gemma-4 mixes two, Tikarax lists them
         self.k = {l: torch.zeros(num_blocks, geo[l][0], KV_BLOCK, geo[l][1], dtype=td, device=device) for l in layers}
         self.v = {l: torch.zeros(num_blocks, geo[l][0], KV_BLOCK, geo[l][-1], dtype=td, device=device) for l in layers}
+        rows = lambda l, width: torch.zeros(num_blocks, geo[l][0], ops.PoolPages.rows_per_page(KV_BLOCK, pools[l][0]), width, dtype=td, device=device)
+        self.pools = {l: ops.PoolPages(rows(l, geo[l][1]), rows(l, geo[l][-1]), *pools[l]) for l in (pools or {})}
         self.ks = {l: torch.ones(num_blocks, geo[l][0], KV_BLOCK, dtype=torch.float32, device=device) for l in layers} if dtype == "int8" else None
         self.vs = {l: torch.ones(num_blocks, geo[l][0], KV_BLOCK, dtype=torch.float32, device=device) for l in layers} if dtype == "int8" else None
 
@@ -113,6 +117,8 @@ class KVCache:
         for l in self.k:
             self.k[l][d] = self.k[l][s]
             self.v[l][d] = self.v[l][s]
+            for t in (self.pools[l].k, self.pools[l].v) if l in self.pools else ():
+                t[d] = t[s]
             if self.ks is not None:
                 self.ks[l][d] = self.ks[l][s]
                 self.vs[l][d] = self.vs[l][s]
@@ -455,13 +461,78 @@ class KeyValueAttentionBlock:
         return self.o(a.reshape(T, nq))
 
 
+def pair_order(n: int, rot: int) -> torch.Tensor:
+    """Order of a head's n elements in which the planes (i, i + rot / 2) of a half-split rotation stand side by side; elements past ``rot`` stay."""
+    half = torch.arange(rot // 2)
+    return torch.cat([torch.stack([half, half + rot // 2], dim=1).reshape(-1), torch.arange(rot, n)])
+
+
+class PooledAttentionBlock:
+    """Attention over a sliding window of tokens and, before it, over pooled blocks (one key and value for ``pool`` tokens), all in one softmax.  Keys of
+    width ``dim`` rotated over ``rot_dim`` elements, values rotated over their whole width and cached so, each head's output turned back by its own position;
+    a factor per head on the scores (folded into the queries behind the rotation), soft-capped scores, a learned sink per head, sigmoid output gate that
+    reads the block's own input.
+
+    One projection gives the columns [q | k | v | gate]; queries and gate are read in place by the attention kernel (which turns the output back and gates
+    it as it writes).  Scores do not depend on the order of a head's elements, nor the output on that of its value elements when the output projection's
+    columns follow: both are reordered at load so that the half-split planes become neighbouring pairs.  Head widths are padded to multiples of 8."""
+
+    MAX_DIM = 512
+
+    def __init__(self, src, prefix: str, hidden: int, row: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, window: int, softcap: float,
+                 rot_dim: int, rope: tuple, v_rope: tuple):
+        if max(dim, vdim) > self.MAX_DIM:
+            raise ValueError(f"{prefix}: heads of {max(dim, vdim)} elements are wider than the {self.MAX_DIM} the kernels take")
+        self.n_q, self.n_kv, self.dim, self.scale, self.window, self.softcap = heads, kv_heads, dim, scale, window, softcap
+        self.rot_dim, self.rope, self.v_rope = rot_dim, rope, v_rope
+        self.dk, self.dv = round_up(dim, 8), round_up(vdim, 8)
+        index = lambda n, d, rot: (torch.arange(n).unsqueeze(1) * d + pair_order(d, rot)).reshape(-1)
+
+        def rows(name, n, d, rot, to, biased=True):
+            at = index(n, d, rot)
+            w = src.matrix(f"{prefix}.{name}", n * d, hidden)
+            w = w.select_rows(at.to(w.device)).pad_groups(rows=(n, to), cols=(1, row))
+            b = torch.zeros(n, to, dtype=torch.float32, device=w.device)
+            if biased:
+                b[:, :d] = src.vector(f"{prefix}.{name}.b", n * d)[at.to(w.device)].reshape(n, d)
+            return w, b.reshape(-1)
+
+        parts = [rows("q", heads, dim, rot_dim, self.dk), rows("k", kv_heads, dim, rot_dim, self.dk), rows("v", kv_heads, vdim, vdim, self.dv),
+                 rows("g", heads, vdim, vdim, self.dv, biased=False)]
+        self.proj = _fuse_rows(*map(list, zip(*parts)))
+        ends = [0]
+        for w, _ in parts:
+            ends.append(ends[-1] + w.N)
+        self.cols = ends
+        self.temp, self.sinks = src.vector(f"{prefix}.temp", heads), src.vector(f"{prefix}.sink", heads)
+        wo = src.matrix(f"{prefix}.o", hidden, heads * vdim)
+        if wo.fmt != WFormat.BF16:
+            wo = QuantWeight(**_as_bf16(wo))
+        wo = QuantWeight(WFormat.BF16, wo.N, wo.K, 1, wo.p0[..., index(heads, vdim, vdim).to(wo.device)].contiguous())
+        self.o = Linear(wo.pad_groups(rows=(1, row), cols=(heads, self.dv)))
+
+    def __call__(self, h: torch.Tensor, fb: ForwardBatch, kv: KVCache, run: int) -> torch.Tensor:
+        """``run``: which of the cache's entries (a layer that runs several times has one per run)."""
+        y = self.proj(h)
+        T, c, k, v, pools, dense = y.shape[0], self.cols, kv.k[run], kv.v[run], kv.pools.get(run), None
+        one_each = fb.max_q_len == 1             # a block that a single token sees first is formed beside its head epilogue
+        q = ops.qk_post(y[:, :c[1]].unflatten(1, (self.n_q, self.dk)), y[:, c[1]:c[2]].unflatten(1, (self.n_kv, self.dk)), fb.positions, self.rope[0],
+                        self.rope[1], fb.slot_map, k, v, self.dim, self.rot_dim, interleaved=True, v=y[:, c[2]:c[3]].unflatten(1, (self.n_kv, self.dv)),
+                        v_rope=self.v_rope, q_scale=self.temp, pools=pools if one_each else None, block_table=fb.block_table)
+        if pools is not None and not one_each:
+            dense = ops.pool_blocks(k, v, pools, fb.block_table, fb.seq_lens, fb.cu_q, fb.max_q_len, max_kv_len=fb.max_kv_len)
+        a = ops.attention(q, k, v, fb.block_table, fb.seq_lens, fb.cu_q, fb.max_q_len, sinks=self.sinks, window=self.window, scale=self.scale,
+                          softcap=self.softcap, max_kv_len=fb.max_kv_len, gate=y[:, c[3]:], pools=pools, pool_dense=dense, out_rope=self.v_rope)
+        return self.o(a.reshape(T, self.n_q * self.dv))
+
+
 class GatedFFN:
     """down(act(gate h, up h)), the gate and up rows interleaved for the projection's epilogue."""
 
-    def __init__(self, src, prefix: str, hidden: int, row: int, ffn: int, act: int = ACT_SWIGLU):
+    def __init__(self, src, prefix: str, hidden: int, row: int, ffn: int, act: int = ACT_SWIGLU, act_alpha: float = 1.702, act_limit: float = 7.0):
         f = round_up(ffn, 32)
         g, u = (src.matrix(f"{prefix}.{n}", ffn, hidden).pad_groups(rows=(1, f), cols=(1, row)) for n in ("gate", "up"))
-        self.gate_up = Linear(QuantWeight.interleave_gate_up(g, u), act=act)
+        self.gate_up = Linear(QuantWeight.interleave_gate_up(g, u), act=act, act_alpha=act_alpha, act_limit=act_limit)
         self.down = Linear(src.matrix(f"{prefix}.down", hidden, ffn).pad_groups(rows=(1, row), cols=(1, f)))
 
     def __call__(self, h):
@@ -786,6 +857,50 @@ class ScaledInputMoEFFN(UnaryMoEFFN):
             y = ops.grouped_linear(a, self.down, pk.tile_expert, pk.num_tiles)
             pos = pk.pair_to_packed
         return ops.ExpertSum(y, pos, K, None if self.shared is None else self.shared(h))
+
+
+class ClampedMoEFFN(UnaryMoEFFN):
+    """Experts down(clamped SwiGLU(gate h, up h)) without biases, of which each token uses the best K by biased router logit, weighted with the softmax of
+    the chosen ones; an always-on expert of the same form joins times the sigmoid of one number per token.  That number is one more row of the router's
+    matrix.  Returns the sum unformed (:class:`ops.ExpertSum`).  One GPU."""
+
+    PAIR_GEMV_MAX_TOKENS = 4
+
+    def __init__(self, src, prefix: str, hidden: int, row: int, experts: int, used: int, ffn: int, limit: float, shared_ffn: int = 0, shared_limit: float = 0.0,
+                 act: int = ACT_SWIGLU_OAI, alpha: float = 1.702):
+        super().__init__(src, prefix, hidden, row, experts, used, ffn, act)          # (gate_up holds the up rows so far)
+        gate = src.matrix(f"{prefix}.e*.gate", ffn, hidden, experts).pad_groups(rows=(1, round_up(ffn, 32)), cols=(1, row))
+        self.gate_up = QuantWeight.interleave_gate_up(gate, self.gate_up)
+        self.act_kw = dict(act=act, act_alpha=alpha, act_limit=limit)
+        self.shared = GatedFFN(src, f"{prefix}.shared", hidden, row, shared_ffn, **{**self.act_kw, "act_limit": shared_limit}) if shared_ffn else None
+        rows = [self.router.w]
+        if shared_ffn:
+            sg = src.matrix(f"{prefix}.shared.sg", 1, hidden)
+            rows.append((sg if sg.fmt == WFormat.BF16 else QuantWeight(**_as_bf16(sg))).pad_groups(cols=(1, row)))
+        w = QuantWeight.cat_rows(rows)
+        n = round_up(w.N, 8)
+        bias = torch.nn.functional.pad(src.vector(f"{prefix}.router.b", experts), (0, n - experts)).contiguous()
+        self.router = Linear(w.pad_groups(rows=(1, n)), bias)
+
+    def __call__(self, h: torch.Tensor, par: Optional[ParallelCtx] = None):
+        T, K = h.shape[0], self.K
+        z = self.router(h, out_f32=True)
+        idx, w = ops.moe_route(z, None, K, precise=h.dtype == torch.float32, experts=self.E)
+        if T <= self.PAIR_GEMV_MAX_TOKENS and h.dtype != torch.float32:
+            slot_e = idx.reshape(-1)
+            a = ops.expert_gemv(h, self.gate_up, slot_e, x_div=K, **self.act_kw)
+            y = ops.expert_gemv(a, self.down, slot_e)
+            if (T, h.device) not in self._arange:
+                self._arange[T, h.device] = torch.arange(T * K, dtype=torch.int32, device=h.device)
+            pos = self._arange[T, h.device]
+        else:
+            pk = ops.moe_pack(idx, self.E)
+            a = ops.grouped_linear(ops.moe_gather(h, pk), self.gate_up, pk.tile_expert, pk.num_tiles, **self.act_kw)
+            y = ops.grouped_linear(a, self.down, pk.tile_expert, pk.num_tiles)
+            pos = pk.pair_to_packed
+        if self.shared is None:
+            return ops.ExpertSum(y, pos, K, w=w)
+        return ops.ExpertSum(y, pos, K, self.shared(h), w, z[:, self.E])
 
 
 def _mx_experts(self, h: torch.Tensor, idx: torch.Tensor, pre=None, ksplit: int = 1):

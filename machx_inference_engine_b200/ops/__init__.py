@@ -9,7 +9,7 @@ from __future__ import annotations
 import functools
 
 from . import ref
-from .ref import ACT_GEGLU, ACT_GELU_TANH, ACT_NONE, ACT_RELU2, ACT_SWIGLU, ACT_SWIGLU_OAI, ACT_TANH, ACT_XIELU, MOE_TILE, BranchMean, ExpertSum, MoePacking, act_gated, moe_max_rows
+from .ref import ACT_GEGLU, ACT_GELU_TANH, ACT_NONE, ACT_RELU2, ACT_SWIGLU, ACT_SWIGLU_OAI, ACT_TANH, ACT_XIELU, MOE_TILE, BranchMean, ExpertSum, MoePacking, PoolPages, act_gated, moe_max_rows
 from .weights import QuantWeight, WFormat, from_dense, from_exl3, from_ggml
 from ..utils.profiler import profiler as _prof
 
@@ -18,6 +18,7 @@ _NAMES = [
     "attention", "gated_rmsnorm_heads", "conv1d_silu", "deltanet_scan", "moe_route", "moe_pack", "moe_gather", "moe_combine", "argmax", "rep_penalty", "sample",
     "hadamard128", "group_norm", "kv_store", "mingru_scan", "dyt_norm", "latent_post", "head_linear", "latent_attention", "latent_attention_expanded",
     "qk_post", "token_shift", "stacked_linear", "decay_scan", "gated_group_norm", "sublayer_norm", "moe_scale_rows",
+    "pool_blocks", "causal_conv", "rglru_scan", "rglru_step",
 ]
 
 
@@ -73,5 +74,5 @@ def _make(name):
 for _n in _NAMES:
     globals()[_n] = _make(_n)
 
-__all__ = _NAMES + ["set_backend", "QuantWeight", "WFormat", "from_dense", "from_exl3", "from_ggml", "BranchMean", "ExpertSum", "MoePacking", "moe_max_rows", "ACT_NONE", "ACT_SWIGLU",
+__all__ = _NAMES + ["set_backend", "QuantWeight", "WFormat", "from_dense", "from_exl3", "from_ggml", "BranchMean", "ExpertSum", "MoePacking", "PoolPages", "moe_max_rows", "ACT_NONE", "ACT_SWIGLU",
                     "ACT_SWIGLU_OAI", "ACT_GEGLU", "ACT_XIELU", "ACT_GELU_TANH", "ACT_RELU2", "ACT_TANH", "act_gated", "MOE_TILE"]

@@ -324,12 +324,72 @@ def mingru_scan(z, u, g, zb, ub, state, state_slots, cu_q, seq_lens, max_q_len):
     return y
 
 
+def causal_conv(x, w, b, state, state_slots, cu_q, seq_lens, max_q_len):
+    """Causal convolution per channel over packed sequences, no activation: y_t = sum_j w[:, j] x_(t - taps + 1 + j) + b, zeros before a sequence's start.
+    x [T, C] (any row stride), w fp32 [C, taps], b fp32 [C]; state [slots, taps - 1, C] of x's dtype holds the inputs before the next token and is
+    advanced in place."""
+    T, C = x.shape
+    taps = w.shape[1]
+    y = torch.empty(T, C, dtype=x.dtype, device=x.device)
+    cu = cu_q.tolist()
+    for i in range(len(cu) - 1):
+        t0, t1 = cu[i], cu[i + 1]
+        if t1 <= t0:
+            continue
+        slot = int(state_slots[i])
+        before = torch.zeros_like(state[slot]) if int(seq_lens[i]) == t1 - t0 else state[slot]
+        full = torch.cat([before, x[t0:t1]]).to(torch.float32)
+        y[t0:t1] = ((full.unfold(0, taps, 1) * w).sum(-1) + b).to(x.dtype)
+        state[slot] = full[full.shape[0] - (taps - 1):].to(state.dtype)
+    return y
+
+
+def _rglru(r, i, u, y, coef, S):
+    """One token: S <- a S + sqrt(1 - a^2) sigmoid(i) u with log a = coef sigmoid(r); (S, S gelu(y))."""
+    la = coef * torch.sigmoid(r)
+    S = torch.exp(la) * S + torch.sqrt(-torch.expm1(2.0 * la)) * torch.sigmoid(i) * u
+    return S, S * torch.nn.functional.gelu(y, approximate="tanh")
+
+
+def rglru_scan(gates, u, y, bias, coef, state, state_slots, cu_q, seq_lens, max_q_len):
+    """Real-gated linear recurrence over packed sequences (see _rglru).  gates fp32 [T, blocks, 2 n] = the pre-activations of r and of i of a block's n
+    channels, bias fp32 [blocks, 2 n] joins them; u, y [T, blocks * n] (any row stride); coef fp32 [blocks * n]; state fp32 [slots, blocks * n], advanced
+    in place, from zeros for a sequence whose step begins at position 0."""
+    T, W = u.shape
+    n = gates.shape[2] // 2
+    g = gates + bias
+    r, i = g[..., :n].reshape(T, W), g[..., n:].reshape(T, W)
+    out = torch.empty(T, W, dtype=u.dtype, device=u.device)
+    uf, yf = u.to(torch.float32), y.to(torch.float32)
+    cu = cu_q.tolist()
+    for b in range(len(cu) - 1):
+        t0, t1 = cu[b], cu[b + 1]
+        if t1 <= t0:
+            continue
+        slot = int(state_slots[b])
+        S = torch.zeros(W, dtype=torch.float32, device=u.device) if int(seq_lens[b]) == t1 - t0 else state[slot].clone()
+        for t in range(t0, t1):
+            S, o = _rglru(r[t], i[t], uf[t], yf[t], coef, S)
+            out[t] = o.to(out.dtype)
+        state[slot] = S
+    return out
+
+
+def rglru_step(x, y, conv_w, conv_b, w: QuantWeight, bias, coef, conv_state, state, state_slots, cu_q, seq_lens):
+    """One token per sequence: convolution, gates and recurrence together.  x, y [T, W] (any row stride); w stacks per block the 2 n rows of the two gates."""
+    u = causal_conv(x, conv_w, conv_b, conv_state, state_slots, cu_q, seq_lens, 1)
+    gates = head_linear(u.view(u.shape[0], w.E, w.K), w, out_f32=True)
+    return rglru_scan(gates, u, y, bias, coef, state, state_slots, cu_q, seq_lens, 1)
+
+
 def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks=None, window=0, scale=None, softcap=0.0, n_splits=1,
-              kv_scales=None, max_kv_len=0, q_scale=None, gate=None, keep_first=0):
+              kv_scales=None, max_kv_len=0, q_scale=None, gate=None, keep_first=0, pools=None, pool_dense=None, out_rope=None):
     """q [Tq,n_q,hd]; caches [blocks,n_kv,bs,hd] (bf16 / fp32, or int8 with kv_scales = (k_scale, v_scale) [blocks,n_kv,bs]); values may be
     wider or narrower than keys; returns [Tq,n_q,value width] (bf16; fp32 for fp32 queries).  ``q_scale`` [positions]: factor on the scores
     of a query at that position; ``gate`` [Tq, n_q * value width] or [Tq, n_q] (one number per head): the result is multiplied by its sigmoid.
-    With a window the first ``keep_first`` keys of a sequence stay visible."""
+    With a window the first ``keep_first`` keys of a sequence stay visible.  ``pools`` (:class:`PoolPages`): pooled blocks before the window are seen
+    beside its keys (``pool_dense`` is what :func:`pool_blocks` returned).  ``out_rope`` = (cos, sin): the result at position p is turned by -p in
+    interleaved pairs, before the gate."""
     Tq, n_q, hd = q.shape
     dv = v_cache.shape[3]
     n_kv, bs = k_cache.shape[1], k_cache.shape[2]
@@ -352,6 +412,14 @@ def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks
         qq = q[q0:q1].to(torch.float32) * scale                                 # [t, n_q, hd]
         if q_scale is not None:
             qq = qq * q_scale[L - (q1 - q0):L].reshape(-1, 1, 1)
+        n_pool = 0
+        if pools is not None:
+            n_pool = max(L - pools.window, 0) // pools.pool
+            if n_pool:
+                page, row = pools.place(torch.arange(n_pool, device=q.device), bs)
+                at = block_table[b].long()[page]
+                K = torch.cat([K, pools.k[at, :, row].to(torch.float32).transpose(0, 1)], dim=1)
+                V = torch.cat([V, pools.v[at, :, row].to(torch.float32).transpose(0, 1)], dim=1)
         Kh = K.repeat_interleave(gqa, dim=0)
         Vh = V.repeat_interleave(gqa, dim=0)
         s = torch.einsum("thd,hkd->htk", qq.to(_MM_DTYPE), Kh.to(_MM_DTYPE)).to(torch.float32)
@@ -362,6 +430,8 @@ def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks
         ok = kpos <= qpos
         if window and window > 0:
             ok = ok & ((kpos > qpos - window) | (kpos < keep_first))
+        if n_pool:
+            ok = torch.cat([ok, torch.arange(1, n_pool + 1, device=q.device).unsqueeze(0) * pools.pool - 1 <= qpos - pools.window], dim=1)
         s = s.masked_fill(~ok.unsqueeze(0), float("-inf"))
         if sinks is not None:
             sk = sinks.to(torch.float32).reshape(n_q, 1, 1).expand(n_q, q1 - q0, 1)
@@ -369,17 +439,64 @@ def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks
         else:
             p = torch.softmax(s, dim=-1)
         out[q0:q1] = torch.einsum("htk,hkd->thd", p.to(_MM_DTYPE), Vh.to(_MM_DTYPE)).to(torch.float32)
+        if out_rope is not None:
+            at = qpos.squeeze(-1).clamp(max=out_rope[0].shape[0] - 1)
+            out[q0:q1] = _rotate_pairs(out[q0:q1], out_rope[0][at].unsqueeze(1), -out_rope[1][at].unsqueeze(1))
     if gate is not None:
         out = out * torch.sigmoid(gate.to(torch.float32)).reshape(Tq, n_q, -1)
     return out if q.dtype == torch.float32 else out.to(torch.bfloat16)
 
 
+@dataclass
+class PoolPages:
+    """Pooled rows of one layer's cache: block b is the mean of the keys / values at positions b * pool .. b * pool + pool - 1.  ``k``, ``v`` [pages,
+    n_kv, rows, width]: a page of bs tokens holds, from row 0 on, the blocks whose last token lies in it.  A query sees the blocks whose last token lies
+    ``window`` or more positions before it, so a step forms the blocks that its own queries are the first to see."""
+    k: torch.Tensor
+    v: torch.Tensor
+    pool: int
+    window: int
+
+    @staticmethod
+    def rows_per_page(bs: int, pool: int) -> int:
+        return (bs + pool - 1) // pool
+
+    def place(self, block, bs: int):
+        """(page of the sequence, row in it) of a block."""
+        page = (block * self.pool + self.pool - 1) // bs
+        return page, block - page * bs // self.pool
+
+
+def _form_pools(k_cache, v_cache, pools: PoolPages, table, start: int, end: int) -> None:
+    """The blocks that a step over positions start .. end - 1 of one sequence sees first."""
+    bs, P = k_cache.shape[2], pools.pool
+    for b in range(max(start - pools.window, 0) // P, max(end - pools.window, 0) // P):
+        at = torch.arange(b * P, b * P + P, device=k_cache.device)
+        page, row = pools.place(b, bs)
+        for cache, out in ((k_cache, pools.k), (v_cache, pools.v)):
+            out[table[page], :, row] = cache[table[at // bs], :, at % bs].to(torch.float32).mean(0).to(out.dtype)
+
+
+def pool_blocks(k_cache, v_cache, pools: PoolPages, block_table, seq_lens, cu_q, max_q_len, max_kv_len=0):
+    """Forms the pooled blocks that the queries of this step are the first to see (their tokens lie in the cache).  Returns what the attention of the step
+    wants as ``pool_dense`` (here: nothing)."""
+    cu = cu_q.tolist()
+    for i in range(len(cu) - 1):
+        L = int(seq_lens[i])
+        if cu[i + 1] > cu[i]:
+            _form_pools(k_cache, v_cache, pools, block_table[i].long(), L - (cu[i + 1] - cu[i]), L)
+    return None
+
+
 def qk_post(q, k, positions, rope_cos, rope_sin, slot_map, k_cache, v_cache, dim, rot_dim, interleaved=False, q_norm=None, k_norm=None, norm_after=False,
-            eps=1e-6):
+            eps=1e-6, v=None, v_rope=None, q_scale=None, pools=None, block_table=None):
     """Head epilogue of attention whose values are its projected keys.  q [T, n_q, dp], k [T, n_kv, dp] (column ranges of one projection; the first
     ``dim`` elements are the head, the rest zero padding): RMS norm with the weights q_norm / k_norm [dp], rotation of the first ``rot_dim``
     elements in interleaved pairs or half splits, and with ``norm_after`` an RMS norm without a weight behind it.  Returns the queries (the kernel works
-    in place); the keys go into k_cache, and as they came into v_cache (slots < 0 are skipped)."""
+    in place); the keys go into k_cache, and as they came into v_cache (slots < 0 are skipped).
+    ``v`` [T, n_kv, dv]: values of their own, turned like keys, in interleaved pairs by the tables ``v_rope`` = (cos, sin) over their first 2 * columns
+    elements.  ``q_scale`` [n_q]: factor on the finished queries of a head.  ``pools``: every sequence has one token, and the pooled block that it sees
+    first, if there is one, is formed (from tokens of earlier steps)."""
     pos = positions.long().clamp(0, rope_cos.shape[0] - 1)
     c, s = rope_cos[pos].unsqueeze(1), rope_sin[pos].unsqueeze(1)
     half = rot_dim // 2
@@ -400,8 +517,18 @@ def qk_post(q, k, positions, rope_cos, rope_sin, slot_map, k_cache, v_cache, dim
     bs = k_cache.shape[2]
     blk, off = (slot_map[ok] // bs).long(), (slot_map[ok] % bs).long()
     k_cache[blk, :, off] = turn(k, k_norm)[ok].to(k_cache.dtype)
-    v_cache[blk, :, off] = k[ok].to(v_cache.dtype)
-    return turn(q, q_norm).to(q.dtype)
+    if v is None:
+        v_cache[blk, :, off] = k[ok].to(v_cache.dtype)
+    else:
+        at = positions.long().clamp(0, v_rope[0].shape[0] - 1)
+        v_cache[blk, :, off] = _rotate_pairs(v.to(torch.float32), v_rope[0][at].unsqueeze(1), v_rope[1][at].unsqueeze(1))[ok].to(v_cache.dtype)
+    if pools is not None:
+        for t in range(q.shape[0]):
+            if bool(ok[t]):
+                p = int(positions[t])
+                _form_pools(k_cache, v_cache, pools, block_table[t].long(), p, p + 1)
+    q = turn(q, q_norm)
+    return (q if q_scale is None else q * q_scale.reshape(1, -1, 1)).to(k.dtype)
 
 
 # ------------------------------------------------------------------ matrix-valued recurrences without a delta rule
@@ -464,20 +591,28 @@ def gated_group_norm(o, gate, w, eps, groups=1, width=None, silu=False, out_dtyp
 # ------------------------------------------------------------------ norms on a sublayer's output
 @dataclass
 class ExpertSum:
-    """A branch that has not been formed: the sum of the rows of a token's experts (``y`` [rows, H], row pair_to_packed[t * k + j] for its j-th) and,
-    when there is one, of ``shared`` [T, H]."""
+    """A branch that has not been formed: the sum of the rows of a token's experts (``y`` [rows, H], row pair_to_packed[t * k + j] for its j-th), each
+    times its weight when there are weights ``w`` [T, k], and, when there is one, of ``shared`` [T, H], times the sigmoid of ``shared_gate`` [T] (a
+    column of a wider matrix: any stride) when there is one."""
     y: torch.Tensor
     pair_to_packed: torch.Tensor
     k: int
     shared: Optional[torch.Tensor] = None
+    w: Optional[torch.Tensor] = None
+    shared_gate: Optional[torch.Tensor] = None
 
     def rows(self, idx):
-        return ExpertSum(self.y, self.pair_to_packed.view(-1, self.k).index_select(0, idx).reshape(-1), self.k,
-                         None if self.shared is None else self.shared.index_select(0, idx))
+        pick = lambda t: None if t is None else t.index_select(0, idx)
+        return ExpertSum(self.y, self.pair_to_packed.view(-1, self.k).index_select(0, idx).reshape(-1), self.k, pick(self.shared), pick(self.w),
+                         pick(self.shared_gate))
 
     def materialize(self, eps=0.0, width=None):
-        d = self.y.to(torch.float32)[self.pair_to_packed.long()].view(-1, self.k, self.y.shape[1]).sum(1)
-        return d if self.shared is None else d + self.shared.to(torch.float32)
+        d = self.y.to(torch.float32)[self.pair_to_packed.long()].view(-1, self.k, self.y.shape[1])
+        d = (d if self.w is None else d * self.w.unsqueeze(-1)).sum(1)
+        if self.shared is None:
+            return d
+        s = self.shared.to(torch.float32)
+        return d + (s if self.shared_gate is None else s * torch.sigmoid(self.shared_gate).unsqueeze(-1))
 
 
 @dataclass
@@ -497,17 +632,19 @@ class BranchMean:
         return 0.5 * (rms(self.a) * self.a_w + rms(self.b) * self.b_w)
 
 
-def sublayer_norm(x, delta, delta_w, eps, w=None, width=None, out_dtype=torch.bfloat16, want_out=True):
-    """x <- x + norm(delta) * delta_w (fp32, in place; delta: a tensor, an :class:`ExpertSum`, a :class:`BranchMean`, or None); returns norm(x) * w, or
-    without ``w`` x itself, as ``out_dtype``.  Rows are padded to x.shape[1] columns (weights too, with zeros); the mean runs over ``width``."""
+def sublayer_norm(x, delta, delta_w, eps, w=None, width=None, out_dtype=torch.bfloat16, want_out=True, out=None):
+    """x <- x + norm(delta) * delta_w, without ``delta_w`` x <- x + delta (fp32, in place; delta: a tensor, an :class:`ExpertSum`, a :class:`BranchMean`,
+    or None); returns norm(x) * w, or without ``w`` x itself, as ``out_dtype``.  Rows are padded to x.shape[1] columns (weights too, with zeros); the mean
+    runs over ``width``.  ``out``: where the result goes (unit column stride, any row stride)."""
     n = width or x.shape[1]
     rms = lambda t: t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) / n + eps)
     if delta is not None:
         d = delta.to(torch.float32) if isinstance(delta, torch.Tensor) else delta.materialize(eps, n)
-        x += rms(d) * delta_w
+        x += d if delta_w is None else rms(d) * delta_w
     if not want_out:
         return None
-    return (x if w is None else rms(x) * w).to(out_dtype)
+    y = (x if w is None else rms(x) * w).to(out_dtype)
+    return y if out is None else out.copy_(y)
 
 
 # ------------------------------------------------------------------ latent attention
@@ -533,13 +670,13 @@ def latent_post(q_rot, ckv, norm_w, rank, eps, positions, rope_cos, rope_sin, sl
     cache[(slot_map[ok] // bs).long(), 0, (slot_map[ok] % bs).long()] = row[ok]
 
 
-def head_linear(x, w: QuantWeight, gate=None, out=None):
+def head_linear(x, w: QuantWeight, gate=None, out=None, out_f32=False):
     """Every head its own matrix: out[t, h] = W[h] x[t, h] (* sigmoid(gate[t, h])).  x [T, H, K] (any row / head stride), w stacks H matrices
-    [N, K]; gate [T, H * N]; out [T, H, N]."""
+    [N, K]; gate [T, H * N]; out [T, H, N], in fp32 with ``out_f32``."""
     y = torch.einsum("thk,hnk->thn", x.to(_MM_DTYPE), _dense(w)).to(torch.float32)
     if gate is not None:
         y = y * torch.sigmoid(gate.to(torch.float32)).reshape(y.shape)
-    y = y.to(x.dtype)
+    y = y if out_f32 else y.to(x.dtype)
     return y if out is None else out.copy_(y)
 
 
@@ -725,9 +862,9 @@ def deltanet_scan_chunked(qkv, n_k, ab, a_idx, b_idx, k_of_v, ssm_a, dt_bias, st
     return out.reshape(T, n_v * D)
 
 
-def moe_route(logits, bias, k, renorm=True, precise=False, sigmoid=False):
-    """``sigmoid``: the weights are the sigmoids of the chosen logits, as they are."""
-    x = logits.to(torch.float32)
+def moe_route(logits, bias, k, renorm=True, precise=False, sigmoid=False, experts=None):
+    """``sigmoid``: the weights are the sigmoids of the chosen logits, as they are.  ``experts``: only the first so many columns are experts."""
+    x = logits[:, :experts].to(torch.float32)
     if bias is not None:
         x = x + bias
     # descending value, ties -> lowest index (stable sort on -x)
