@@ -75,7 +75,7 @@ def build_host(force: bool = False) -> Path:
 # can compile just these (``_lib.use_components("core")``); the full library, when it is there, serves every graph.
 COMPONENTS = {
     "core": ("common", "comm", "elementwise", "gemm_tcgen05", "gemv", "gemv_stream", "linear_f32", "attention", "attention_tc", "mingru", "latent",
-             "latent_tc", "linear_scan", "decay_chunk", "moe", "sampling"),
+             "latent_tc", "linear_scan", "decay_chunk", "pooled", "rglru", "moe", "sampling"),
 }
 
 

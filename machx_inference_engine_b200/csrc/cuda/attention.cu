@@ -15,6 +15,10 @@
 // 64 / 128 / 256 / 512 run on instances whose widths are compile-time constants; all other shapes, and caches in fp32, run on
 // instances that take the widths at run time and only round the value width up to 64 / 128 / 256 / 512 (accumulator registers).
 //
+// Pooled blocks: with a window, means of whole runs of `pool` tokens before it are keys and values too; they lie in pool pages beside the cache pages (row
+// layout: pool_row below) and are walked as tiles of their own in front of the window's.  The output may be turned back by the query's position (a rotation
+// of neighbouring pairs, before the gate), which undoes a rotation of the cached values.
+//
 // A latent cache has no value pages: the values are the first dv elements of the key rows (v_cache null), which are staged once.
 //
 // KV cache layout: [block][kv_head][block_size][head_dim] bf16 (or fp32), block_size a multiple of 64.  An int8 cache has the
@@ -51,6 +55,12 @@ struct AttnParams {
   int q_scale_n, q_ld, gate_ld, dk, dv;
   int gate_heads;              // the gate has one number per head: rows of [n_q]
   int keep_first;              // with a window: the first keys of the sequence that stay visible
+  const void* pk;              // pool pages [block][kv_head][pool_rows][dk], or null
+  const void* pv;
+  int pool, pool_rows;
+  const float* out_cos;        // [out_n][out_half] or null: the output is turned by minus its position
+  const float* out_sin;
+  int out_n, out_half;
   float* o_part;               // [splits][Tq][n_q][dv]
   float* ml_part;              // [splits][Tq][n_q][2]
   int* tickets;                // non-null: one counter per (batch entry, query tile, kv head) group; the last split merges
@@ -64,6 +74,14 @@ struct AttnParams {
   int window;                  // 0 = full causal
   float scale, softcap;
 };
+
+// blocks of `pool` tokens that a query at `pos` sees: those whose last token lies `window` or more before it
+__device__ __forceinline__ int pool_visible(int pos, int window, int pool) { return pos >= window ? (pos - window + 1) / pool : 0; }
+// row of a pool page that holds block b; the page is that of the block's last token
+__device__ __forceinline__ int pool_row(int b, int pool, int page, int block_size) { return b - page * block_size / pool; }
+
+// element d of the pair (2m, 2m + 1) turned by minus the angle; other: its neighbour
+__device__ __forceinline__ float turn_back(float own, float other, int d, float c, float s) { return d & 1 ? own * c - other * s : own * c + other * s; }
 
 // bytes `first`, `first + 1` of w as signed 8-bit integers, times scale, packed as two bf16
 __device__ __forceinline__ uint32_t s8x2_to_bf16x2(uint32_t w, int first, float scale) {
@@ -139,13 +157,16 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
   const int kv_lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
   const int tile_lo = kv_lo / ATT_TILE, tile_hi = (kv_hi + ATT_TILE - 1) / ATT_TILE;
   const int n_keep = min((p.keep_first + ATT_TILE - 1) / ATT_TILE, tile_lo);       // kept tiles before the window's
-  const int n_tiles = n_keep + tile_hi - tile_lo;
+  const int n_pooled = p.pk ? pool_visible(pos0 + nt - 1, p.window, p.pool) : 0;
+  const int n_pool = (n_pooled + ATT_TILE - 1) / ATT_TILE;                         // tiles of pooled blocks, the first ones
+  const int n_tiles = n_pool + n_keep + tile_hi - tile_lo;
   const int per = (n_tiles + p.n_splits - 1) / p.n_splits;
   const int my_lo = split * per, my_hi = min(n_tiles, my_lo + per);
   // splits that own at least one key tile (n_tiles >= 1: a query always sees its own position's tile)
   const int eff = p.tickets ? (n_tiles + per - 1) / per : p.n_splits;
   if (split >= eff) return;
 
+  __shared__ long long s_prow[ATT_TILE];
   const int total_pairs = nt * gqa;
   for (int round0 = 0; round0 < total_pairs; round0 += PAIRS) {
     __syncthreads();
@@ -170,10 +191,37 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
     }
     for (int tile = my_lo; tile < my_hi; ++tile) {
       __syncthreads();
-      const int key0 = (tile < n_keep ? tile : tile_lo + tile - n_keep) * ATT_TILE;
-      const int blk = p.block_table[(size_t)b * p.max_blocks + key0 / p.block_size];
+      const bool pooled = tile < n_pool;
+      const int tl = tile - n_pool;
+      const int key0 = (pooled ? tile : tl < n_keep ? tl : tile_lo + tl - n_keep) * ATT_TILE;           // (of a pooled tile: its first block)
+      const int blk = pooled ? 0 : p.block_table[(size_t)b * p.max_blocks + key0 / p.block_size];
       const size_t row0 = ((size_t)blk * p.n_kv + kvh) * p.block_size + key0 % p.block_size;
-      if (EXACT && sizeof(T) == 2 && p.k_scale) {
+      if (pooled) {
+        if (threadIdx.x < ATT_TILE) {
+          const int pb = key0 + threadIdx.x;
+          long long at = -1;
+          if (pb < n_pooled) {
+            const int page = (pb * p.pool + p.pool - 1) / p.block_size;
+            at = ((long long)p.block_table[(size_t)b * p.max_blocks + page] * p.n_kv + kvh) * p.pool_rows + pool_row(pb, p.pool, page, p.block_size);
+          }
+          s_prow[threadIdx.x] = at;
+        }
+        __syncthreads();
+        const int pk = DK / VE, pv = DV / VE;
+        const uint4 zero = make_uint4(0, 0, 0, 0);
+        for (int i = threadIdx.x; i < ATT_TILE * pk; i += blockDim.x) {
+          const int r = i / pk, c = (i % pk) * VE;
+          const long long at = s_prow[r];
+          const uint4 kv4 = at >= 0 ? *reinterpret_cast<const uint4*>(reinterpret_cast<const T*>(p.pk) + at * DK + c) : zero;
+          uint32_t* kd = reinterpret_cast<uint32_t*>(sk + r * KSTR + c);
+          kd[0] = kv4.x; kd[1] = kv4.y; kd[2] = kv4.z; kd[3] = kv4.w;
+        }
+        for (int i = threadIdx.x; i < ATT_TILE * pv; i += blockDim.x) {
+          const int r = i / pv, c = (i % pv) * VE;
+          const long long at = s_prow[r];
+          *reinterpret_cast<uint4*>(sv + r * DV + c) = at >= 0 ? *reinterpret_cast<const uint4*>(reinterpret_cast<const T*>(p.pv) + at * DV + c) : zero;
+        }
+      } else if (EXACT && sizeof(T) == 2 && p.k_scale) {
         const size_t base = row0 * HD;
         const int8_t* k8 = reinterpret_cast<const int8_t*>(p.k_cache);
         const int8_t* v8 = reinterpret_cast<const int8_t*>(p.v_cache);
@@ -249,7 +297,8 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
               const int kpos = key0 + lane + 32 * half;
               float dd = half ? d1[pi] : d0[pi];
               if (p.softcap > 0.f) dd = p.softcap * tanhf(dd / p.softcap);
-              const bool ok = pr < total_pairs && kpos < seq_len && kpos <= qpos && (p.window <= 0 || kpos > qpos - p.window || kpos < p.keep_first);
+              const bool ok = pr < total_pairs && (pooled ? kpos < pool_visible(qpos, p.window, p.pool)
+                                                          : kpos < seq_len && kpos <= qpos && (p.window <= 0 || kpos > qpos - p.window || kpos < p.keep_first));
               sc[pi][half] = ok ? dd : -INFINITY;
             }
           }
@@ -341,8 +390,15 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
 #pragma unroll
     for (int c = 0; c < HD / 32; ++c) {
       const int d = lane + 32 * c;
-      if (!EXACT && d >= DV) continue;
       float o = acc[c] * inv;
+      if (p.out_cos) {
+        const float other = __shfl_xor_sync(0xffffffffu, o, 1);
+        if ((d >> 1) < p.out_half) {
+          const size_t at = (size_t)min(pos0 + tq, p.out_n - 1) * p.out_half + (d >> 1);
+          o = turn_back(o, other, d, __ldg(p.out_cos + at), __ldg(p.out_sin + at));
+        }
+      }
+      if (!EXACT && d >= DV) continue;
       if (p.gate) o *= sigmoid_f<PRECISE>(to_f32(reinterpret_cast<const T*>(p.gate)[(size_t)(q_begin + t0 + tq) * p.gate_ld + (p.gate_heads ? hq : (size_t)hq * DV + d)]));
       reinterpret_cast<T*>(p.out)[r * DV + d] = from_f32<T>(o);
     }
@@ -352,10 +408,17 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
 // out[t][h][:] = sum_s acc_s e^{m_s - M} / (sum_s l_s e^{m_s - M} + e^{sink_h - M}) [* sigmoid(gate)].  blockIdx: (row, run of 256 columns);
 // every warp forms the weights of the splits, a lane per split, and a thread sums two columns over them.
 constexpr int CMB_COLS = 256;
+struct AttnTurn {              // out_cos .. of AttnParams and what gives a row its position
+  const float* cos;
+  const float* sin;
+  const int* seq_lens;
+  const int* cu_q;
+  int n, half, B;
+};
 template <typename T>
 __global__ void __launch_bounds__(CMB_COLS / 2) attn_combine_kernel(const float* __restrict__ o_part, const float* __restrict__ ml_part,
                                                                     const float* __restrict__ sinks, const T* __restrict__ gate, int gate_ld, int gate_heads,
-                                                                    T* __restrict__ out, int Tq, int n_q, int hd, int n_splits) {
+                                                                    T* __restrict__ out, int Tq, int n_q, int hd, int n_splits, const AttnTurn turn) {
   constexpr bool PRECISE = sizeof(T) == 4;
   pdl_prologue();
   const int r = blockIdx.x, lane = threadIdx.x & 31, h = r % n_q;
@@ -391,6 +454,16 @@ __global__ void __launch_bounds__(CMB_COLS / 2) attn_combine_kernel(const float*
   const float inv = L > 0.f ? 1.f / L : 0.f;
   a0 *= inv;
   a1 *= inv;
+  if (turn.cos && d / 2 < turn.half) {
+    const int t = r / n_q;
+    int b = 0;
+    while (b + 1 < turn.B && turn.cu_q[b + 1] <= t) ++b;
+    const int pos = turn.seq_lens[b] - (turn.cu_q[b + 1] - t);
+    const size_t at = (size_t)min(pos, turn.n - 1) * turn.half + d / 2;
+    const float u = a0, v = a1, c = __ldg(turn.cos + at), s = __ldg(turn.sin + at);
+    a0 = turn_back(u, v, 0, c, s);
+    a1 = turn_back(v, u, 1, c, s);
+  }
   if (gate) {
     const T* gr = gate + (size_t)(r / n_q) * gate_ld;
     const float2 g = gate_heads ? make_float2(to_f32(gr[h]), to_f32(gr[h])) : load2(gr + (size_t)h * hd + d);
@@ -459,6 +532,12 @@ struct AttnShape {            // what the plain entry points leave at its defaul
   int q_scale_n = 0;
   int elem_f32 = 0;           // queries, cache, gate and output in fp32
   int gate_heads = 0, keep_first = 0;
+  const void* pk = nullptr;
+  const void* pv = nullptr;
+  int pool = 0, pool_rows = 0;
+  const float* out_cos = nullptr;
+  const float* out_sin = nullptr;
+  int out_n = 0, out_half = 0;
 };
 static int attention_impl(const void* q, const void* k_cache, const void* v_cache, const float* k_scale, const float* v_scale,
                           const int* block_table, const int* seq_lens, const int* cu_q, const float* sinks, void* out, float* o_part,
@@ -471,6 +550,9 @@ static int attention_impl(const void* q, const void* k_cache, const void* v_cach
   AttnParams p;
   p.q = q; p.k_cache = k_cache; p.v_cache = v_cache;
   p.dk = sh.dk; p.dv = sh.dv; p.q_ld = sh.q_ld; p.gate = sh.gate; p.gate_ld = sh.gate_ld; p.gate_heads = sh.gate_heads; p.keep_first = window > 0 ? sh.keep_first : 0; p.q_scale = sh.q_scale; p.q_scale_n = sh.q_scale_n;
+  p.pk = window > 0 && sh.pool > 0 ? sh.pk : nullptr; p.pv = sh.pv; p.pool = sh.pool; p.pool_rows = sh.pool_rows;
+  p.out_cos = sh.out_cos; p.out_sin = sh.out_sin; p.out_n = sh.out_n; p.out_half = sh.out_half;
+  if (p.pk && (k_scale || !v_cache)) return -112;
   p.k_scale = k_scale; p.v_scale = k_scale ? v_scale : nullptr;
   p.block_table = block_table; p.seq_lens = seq_lens; p.cu_q = cu_q; p.o_part = o_part; p.ml_part = ml_part;
   p.B = B; p.n_q = n_q; p.n_kv = n_kv; p.max_blocks = max_blocks; p.block_size = block_size;
@@ -517,11 +599,12 @@ static int attention_impl(const void* q, const void* k_cache, const void* v_cach
 #undef MX_ATT
   if (rc || p.tickets) return rc;
   const dim3 cgrid(Tq * n_q, (dv + CMB_COLS - 1) / CMB_COLS);
+  const AttnTurn turn{p.out_cos, p.out_sin, seq_lens, cu_q, p.out_n, p.out_half, B};
   if (sh.elem_f32)
-    launch_pdl(attn_combine_kernel<float>, cgrid, dim3(CMB_COLS / 2), 0, st, o_part, ml_part, sinks, (const float*)sh.gate, sh.gate_ld, sh.gate_heads, (float*)out, Tq, n_q, dv, p.n_splits);
+    launch_pdl(attn_combine_kernel<float>, cgrid, dim3(CMB_COLS / 2), 0, st, o_part, ml_part, sinks, (const float*)sh.gate, sh.gate_ld, sh.gate_heads, (float*)out, Tq, n_q, dv, p.n_splits, turn);
   else
     launch_pdl(attn_combine_kernel<__nv_bfloat16>, cgrid, dim3(CMB_COLS / 2), 0, st, o_part, ml_part, sinks, (const __nv_bfloat16*)sh.gate, sh.gate_ld, sh.gate_heads,
-               (__nv_bfloat16*)out, Tq, n_q, dv, p.n_splits);
+               (__nv_bfloat16*)out, Tq, n_q, dv, p.n_splits, turn);
   return (int)cudaGetLastError();
 }
 
@@ -531,7 +614,7 @@ MX_HOST_API int mx_attention_combine(const float* o_part, const float* ml_part, 
   const float* no_sinks = nullptr;
   const __nv_bfloat16* no_gate = nullptr;
   launch_pdl(attn_combine_kernel<__nv_bfloat16>, dim3(Tq * n_q, (dv + CMB_COLS - 1) / CMB_COLS), dim3(CMB_COLS / 2), 0, st, o_part, ml_part, no_sinks, no_gate, 0, 0, (__nv_bfloat16*)out, Tq, n_q, dv,
-             n_splits);
+             n_splits, AttnTurn{});
   return (int)cudaGetLastError();
 }
 
@@ -546,12 +629,16 @@ static AttnShape plain_shape(int n_q, int hd) {
 // [n_q][dv], or with gate_heads of [n_q], gate_ld apart; out *= sigmoid(gate)) and per-position score factors q_scale [q_scale_n].  elem_f32: everything in
 // fp32.  With a window the first keep_first keys of a sequence stay visible.
 // o_part needs n_splits*Tq*n_q*dv floats.  Rows, widths and strides are multiples of 16 bytes.  v_cache null: a value is the first dv elements of
-// its key row.
+// its key row.  pk / pv: pool pages of `pool` tokens per block and pool_rows rows per page (window > 0); out_cos / out_sin [out_n][out_half]: the output turned
+// by minus its position in neighbouring pairs.
 MX_HOST_API int mx_attention_ext(const void* q, int q_ld, const void* k_cache, const void* v_cache, const int* block_table, const int* seq_lens,
                                  const int* cu_q, const float* sinks, const void* gate, int gate_ld, const float* q_scale, int q_scale_n, void* out,
                                  float* o_part, float* ml_part, int B, int Tq, int max_q_len, int n_q, int n_kv, int dk, int dv, int max_blocks,
-                                 int block_size, int window, int keep_first, int gate_heads, float scale, float softcap, int n_splits, int elem_f32, cudaStream_t st) {
+                                 int block_size, int window, int keep_first, int gate_heads, float scale, float softcap, int n_splits, int elem_f32,
+                                 const void* pk, const void* pv, int pool, int pool_rows, const float* out_cos, const float* out_sin, int out_n, int out_half,
+                                 cudaStream_t st) {
   AttnShape sh;
+  sh.pk = pk; sh.pv = pv; sh.pool = pool; sh.pool_rows = pool_rows; sh.out_cos = out_cos; sh.out_sin = out_sin; sh.out_n = out_n; sh.out_half = out_half;
   sh.gate_heads = gate_heads; sh.keep_first = keep_first;
   sh.dk = dk; sh.dv = dv; sh.q_ld = q_ld; sh.gate = gate; sh.gate_ld = gate_ld; sh.q_scale = q_scale; sh.q_scale_n = q_scale_n; sh.elem_f32 = elem_f32;
   return attention_impl(q, k_cache, v_cache, nullptr, nullptr, block_table, seq_lens, cu_q, sinks, out, o_part, ml_part, B, Tq, max_q_len, n_q, n_kv,

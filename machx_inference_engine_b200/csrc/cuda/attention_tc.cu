@@ -7,6 +7,10 @@
 // the last 64 from a part that all heads share, at its place in the latent cache; each part has its own tensor maps (and page table).  The values
 // are expanded pages too.
 //
+// Pooled blocks (MODE 2): means of whole runs of `pool` tokens before the window are keys and values too, read from dense pages [sequence][page][kv head]
+// [128] that pool_blocks (pooled.cu) has written for the step, as tiles in front of the window's.  This mode also takes the soft-cap as a parameter, through
+// an accurate tanh, and may turn the output back by the query's position (a rotation of neighbouring pairs, before the gate).
+//
 // One CTA owns 128 query tokens of one query head and walks the key tiles of its range (128 keys per tile, 64 for
 // head_dim 256 so that two K and two V tiles still fit in shared memory):
 //   warp 0  : TMA loads of the K and V tiles (two-stage rings) and, once, of the Q tile
@@ -42,6 +46,10 @@ struct FaParams {
   __nv_bfloat16* out;      // [Tq][n_q][dv]
   int q_scale_n, gate_ld, dk, dv, q_ld;
   int gate_heads, keep_first;   // one gate number per head; with a window: the first keys that stay visible
+  int pool, pool_pages;         // MODE 2: tokens per pooled block (0: none), dense pages per sequence
+  const float* out_cos;         // MODE 2: [out_n][out_half] or null: the output is turned by minus its position
+  const float* out_sin;
+  int out_n, out_half;
   int n_q, n_kv, max_blocks, max_q_tiles, window;
   float scale, softcap;
   int* status;
@@ -91,12 +99,45 @@ __device__ __forceinline__ float ex2_fast(float x) {
   return y;
 }
 
-template <int DK, int DV, bool CAP, int ROT>
+// cap * tanh(x / cap) over a run of raw scores, without the hardware's 11-bit tanh: its power series where all of the run is small (error below 1e-6 of
+// the argument for |y| <= 1/2), otherwise 1 - 2 / (1 + e^2y).  in: factor to y = x / cap; out_c: factor on the result.
+template <int N>
+__device__ __forceinline__ void softcap_run(float (&v)[N], float in, float out_c) {
+  float big = 0.f;
+#pragma unroll
+  for (int i = 0; i < N; ++i) big = fmaxf(big, fabsf(v[i]));
+  if (__any_sync(0xffffffffu, big * fabsf(in) > 0.5f)) {
+    const float in2 = in * 2.8853900817779268f;        // 2 / ln 2
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      float r;
+      asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + ex2_fast(v[i] * in2)));
+      v[i] = fmaf(-2.f * out_c, r, out_c);
+    }
+  } else {
+    // tanh y = y (1 - z / 3 + 2 z^2 / 15 - 17 z^3 / 315 + 62 z^4 / 2835 - 1382 z^5 / 155925 + 21844 z^6 / 6081075 - ...), z = y^2
+    const float in_sq = in * in, lin = in * out_c;
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      const float z = v[i] * v[i] * in_sq;
+      float t = fmaf(z, 3.5921280e-3f, -8.8632355e-3f);
+      t = fmaf(z, t, 2.1869489e-2f);
+      t = fmaf(z, t, -5.3968254e-2f);
+      t = fmaf(z, t, 1.3333333e-1f);
+      t = fmaf(z, t, -3.3333333e-1f);
+      v[i] *= fmaf(z * lin, t, lin);
+    }
+  }
+}
+
+// MODE: 0 plain, 1 keys in two parts, 2 pooled blocks
+template <int DK, int DV, bool CAP, int MODE>
 __global__ void __launch_bounds__(192, FaCfg<DK, DV>::CTAS)
 fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                   const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_qr,
                   const __grid_constant__ CUtensorMap tmap_kr, const FaParams p) {
   using L = FaCfg<DK, DV>;
+  constexpr int ROT = MODE == 1 ? 1 : 0;         // key atoms of the shared part
   constexpr int BKV = L::BKV, NS = L::NS, KS = L::KS, VS = L::VS;
   constexpr float LOG2E = 1.4426950408889634f;
   constexpr float RESCALE_STEP = 8.f;            // in log2 units: O is rescaled when the maximum has grown by a factor of 256
@@ -124,8 +165,16 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
   const int kv_lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
   const int tile_lo = kv_lo / BKV, tile_hi = (kv_hi + BKV - 1) / BKV;
   const int n_keep = min((p.keep_first + BKV - 1) / BKV, tile_lo);            // kept tiles before the window's
-  const int n_tiles = n_keep + tile_hi - tile_lo;
-  auto first_key = [&](int j) { return (j < n_keep ? j : tile_lo + j - n_keep) * BKV; };
+  auto blocks_seen = [&](int pos) { return pos >= p.window ? (pos - p.window + 1) / p.pool : 0; };
+  const int n_pool = MODE == 2 && p.pool ? (blocks_seen(pos0 + rows - 1) + BKV - 1) / BKV : 0;          // tiles of pooled blocks, the first ones
+  const int n_tiles = n_pool + n_keep + tile_hi - tile_lo;
+  auto first_key = [&](int j) {                  // (of a pooled tile: its first block)
+    if (MODE == 2) {
+      if (j < n_pool) return j * BKV;
+      j -= n_pool;
+    }
+    return (j < n_keep ? j : tile_lo + j - n_keep) * BKV;
+  };
 
   if (threadIdx.x == 0) {
     mbar_init(b_qfull, 1);
@@ -156,7 +205,8 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       for (int j = 0; j < n_tiles && ok; ++j) {
         const uint32_t sk = j % KS, phk = (j / KS) & 1, sv = j % VS, phv = (j / VS) & 1;
         const int key0 = first_key(j);
-        const int blk = p.block_table[(size_t)b * p.max_blocks + key0 / FA_PAGE];
+        const bool pooled = MODE == 2 && j < n_pool;
+        const int blk = pooled ? b * p.pool_pages + key0 / FA_PAGE : p.block_table[(size_t)b * p.max_blocks + key0 / FA_PAGE];
         const int krow = key0 % FA_PAGE;
         int rblk = 0;
         if constexpr (ROT != 0) rblk = p.rot_table[(size_t)b * p.max_blocks + key0 / FA_PAGE];
@@ -164,13 +214,13 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         mbar_expect_tx(b_kfull + 8 * sk, L::K_BYTES);
 #pragma unroll
         for (int a = 0; a < L::KATOMS; ++a)
-          if (a < L::KATOMS - ROT) tma_load_4d(sbase + L::K_OFF + sk * L::K_BYTES + a * (BKV * 128), &tmap_k, b_kfull + 8 * sk, a * 64, krow, kvh, blk);
+          if (a < L::KATOMS - ROT) tma_load_4d(sbase + L::K_OFF + sk * L::K_BYTES + a * (BKV * 128), pooled ? &tmap_qr : &tmap_k, b_kfull + 8 * sk, a * 64, krow, kvh, blk);
           else tma_load_3d(sbase + L::K_OFF + sk * L::K_BYTES + a * (BKV * 128), &tmap_kr, b_kfull + 8 * sk, 0, krow, rblk);
         if (!(ok = mbar_wait(b_vempty + 8 * sv, phv ^ 1, p.status, ERR_MBAR_TIMEOUT_PRODUCER, abort_flag))) break;
         mbar_expect_tx(b_vfull + 8 * sv, L::V_BYTES);
 #pragma unroll
         for (int a = 0; a < L::VATOMS; ++a)
-          tma_load_4d(sbase + L::V_OFF + sv * L::V_BYTES + a * (BKV * 128), &tmap_v, b_vfull + 8 * sv, a * 64, krow, kvh, blk);
+          tma_load_4d(sbase + L::V_OFF + sv * L::V_BYTES + a * (BKV * 128), pooled ? &tmap_kr : &tmap_v, b_vfull + 8 * sv, a * 64, krow, kvh, blk);
       }
     }
   } else if (warp == 1) {
@@ -225,9 +275,11 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     const float qs = p.scale * (p.q_scale ? p.q_scale[min(qpos, p.q_scale_n - 1)] : 1.f);
     // c: factor from the stored score to log2 units, applied after the maximum.  That needs c > 0: a row whose factor is not (a
     // temperature law may change sign) multiplies its scores first and goes on with 1.
-    const bool early = !CAP && !(qs > 0.f);
-    const float c = (CAP || early) ? 1.f : qs * LOG2E;
-    const float cap_c = p.softcap * LOG2E, inv_cap = CAP ? qs / p.softcap : 0.f;
+    const bool cap = CAP || (MODE == 2 && p.softcap > 0.f);
+    const bool early = !cap && !(qs > 0.f);
+    const float c = (cap || early) ? 1.f : qs * LOG2E;
+    const float cap_c = p.softcap * LOG2E, inv_cap = cap ? qs / p.softcap : 0.f;
+    const int seen = MODE == 2 && p.pool ? blocks_seen(qpos) : 0;
     if (p.gate && !p.gate_heads && row_ok) {       // bring the row's gate into L2 while the keys are walked
       const __nv_bfloat16* g0 = p.gate + (size_t)(q_begin + t0 + r) * p.gate_ld + (size_t)head * p.dv;
       for (int i = 0; i < p.dv; i += 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(g0 + i));
@@ -248,7 +300,9 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       __syncwarp();
       if (lane == 0) mbar_arrive(b_sempty + 8 * sb);
       const int key0 = first_key(j);
-      if (CAP) {
+      if (MODE == 2 && cap) {
+        softcap_run(sv, inv_cap, cap_c);
+      } else if (CAP) {
 #pragma unroll
         for (int i = 0; i < BKV; ++i) sv[i] = cap_c * tanh_fast(sv[i] * inv_cap);
       } else if (early) {
@@ -256,7 +310,12 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         for (int i = 0; i < BKV; ++i) sv[i] *= qs * LOG2E;
       }
       // a tile needs per-key masking only at the diagonal, at the window edge and at the sequence end
-      if ((key0 + BKV - 1 > pos0) || (p.window > 0 && key0 <= pos0 + FA_BQ - 1 - p.window) || (key0 + BKV > seq_len)) {
+      if (MODE == 2 && j < n_pool) {
+        if (key0 + BKV > blocks_seen(pos0)) {
+#pragma unroll
+          for (int i = 0; i < BKV; ++i) sv[i] = key0 + i < seen ? sv[i] : -INFINITY;
+        }
+      } else if ((key0 + BKV - 1 > pos0) || (p.window > 0 && key0 <= pos0 + FA_BQ - 1 - p.window) || (key0 + BKV > seq_len)) {
         if (key0 < p.keep_first) {
 #pragma unroll
           for (int i = 0; i < BKV; ++i) {
@@ -358,6 +417,18 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
             float o[8];
 #pragma unroll
             for (int e = 0; e < 8; ++e) o[e] = __uint_as_float(ov[i + e]) * inv;
+            if (MODE == 2 && p.out_cos) {
+              const size_t at = (size_t)min(qpos, p.out_n - 1) * p.out_half;
+#pragma unroll
+              for (int e = 0; e < 4; ++e) {
+                const int m = (cb + i) / 2 + e;
+                if (m < p.out_half) {
+                  const float co = __ldg(p.out_cos + at + m), si = __ldg(p.out_sin + at + m), u = o[2 * e], v = o[2 * e + 1];
+                  o[2 * e] = u * co + v * si;
+                  o[2 * e + 1] = v * co - u * si;
+                }
+              }
+            }
             if (grow) {
               const uint4 g4 = cb + i < GPRE ? gpre[(cb + i) < GPRE ? (cb + i) / 8 : 0] : __ldg(reinterpret_cast<const uint4*>(grow + cb + i));
               const uint32_t gw[4] = {g4.x, g4.y, g4.z, g4.w};
@@ -457,6 +528,38 @@ static int launch_fa_split(const void* q, const FaSplit& x, const FaParams& p, i
   return (int)cudaGetLastError();
 }
 
+// MODE 2: the plain pages and, for the pooled blocks, dense pages [n_dense][n_kv][128][dk / dv].
+struct FaPooled { const void* pk; const void* pv; int n_dense; };
+template <int DK, int DV>
+static int launch_fa_pooled(const void* q, const void* k_cache, const void* v_cache, const FaPooled& x, const FaParams& p, int B, int Tq, int n_blocks,
+                            cudaStream_t st) {
+  using L = FaCfg<DK, DV>;
+  CUtensorMap tq, tk, tv, tpk, tpv;
+  uint64_t qd[3] = {(uint64_t)p.dk, (uint64_t)p.n_q, (uint64_t)Tq};
+  uint64_t qs[2] = {(uint64_t)p.dk * 2, (uint64_t)p.q_ld * 2};
+  uint32_t qb[3] = {64, 1, FA_BQ};
+  auto page_map = [&](CUtensorMap* m, const void* base, uint64_t d, int pages) {
+    uint64_t dims[4] = {d, (uint64_t)FA_PAGE, (uint64_t)p.n_kv, (uint64_t)pages};
+    uint64_t strides[3] = {d * 2, d * 2 * FA_PAGE, d * 2 * FA_PAGE * p.n_kv};
+    uint32_t box[4] = {64, (uint32_t)L::BKV, 1, 1};
+    return make_tmap_bf16(m, base, 4, dims, strides, box, 1);
+  };
+  int r = 0;
+  if ((r = make_tmap_bf16(&tq, q, 3, qd, qs, qb, 1)) || (r = page_map(&tk, k_cache, p.dk, n_blocks)) || (r = page_map(&tv, v_cache, p.dv, n_blocks))) return r;
+  tpk = tk;
+  tpv = tv;
+  if (p.pool && ((r = page_map(&tpk, x.pk, p.dk, x.n_dense)) || (r = page_map(&tpv, x.pv, p.dv, x.n_dense)))) return r;
+  auto kern = fa_prefill_kernel<DK, DV, false, 2>;
+  static DeviceOnce configured;
+  if (configured.pending()) {
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, L::TOTAL);
+    if (e != cudaSuccess) return (int)e;
+    configured.mark();
+  }
+  kern<<<dim3(B * p.max_q_tiles, p.n_q), 192, L::TOTAL, st>>>(tq, tk, tv, tpk, tpv, p);
+  return (int)cudaGetLastError();
+}
+
 // the instance whose tiles are the key / value widths rounded up to 64, 128 or 256 columns
 static int dispatch_fa(const void* q, const void* k_cache, const void* v_cache, const FaParams& p, int B, int Tq, int n_blocks, cudaStream_t st) {
   if (p.dk < 8 || p.dv < 8 || p.dk > 256 || p.dv > 256 || p.dk % 8 || p.dv % 8 || p.q_ld % 8) return -112;
@@ -501,6 +604,7 @@ MX_HOST_API int mx_attention_prefill_tc_ext(const void* q, int q_ld, const void*
   p.block_table = block_table; p.rot_table = nullptr; p.seq_lens = seq_lens; p.cu_q = cu_q; p.sinks = sinks; p.out = (__nv_bfloat16*)out;
   p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate ? gate_ld : 0; p.q_scale = q_scale; p.q_scale_n = q_scale_n;
   p.dk = dk; p.dv = dv; p.q_ld = q_ld; p.gate_heads = gate_heads; p.keep_first = window > 0 ? keep_first : 0;
+  p.pool = p.pool_pages = p.out_n = p.out_half = 0; p.out_cos = p.out_sin = nullptr;
   p.n_q = n_q; p.n_kv = n_kv; p.max_blocks = max_blocks; p.window = window; p.scale = scale; p.softcap = softcap;
   p.max_q_tiles = (max_q_len + FA_BQ - 1) / FA_BQ;
   p.status = status_word();
@@ -517,6 +621,38 @@ MX_HOST_API int mx_attention_prefill_tc(const void* q, const void* k_cache, cons
                                      n_q, n_kv, hd, hd, max_blocks, n_blocks, block_size, window, 0, 0, scale, softcap, st);
 }
 
+// Attention over a window and pooled blocks before it (MODE 2).  pk / pv: dense pages [B * pool_pages][n_kv][128][dk / dv] of the blocks of `pool` tokens
+// that each sequence's last query sees, rows past them zero up to a whole page (pool 0: none); out_cos / out_sin [out_n][out_half] (or null): the output is
+// turned by minus its position in neighbouring pairs, before the gate (rows of [n_q][dv]).  softcap 0: none.
+MX_HOST_API int mx_attention_prefill_pooled(const void* q, int q_ld, const void* k_cache, const void* v_cache, const int* block_table, const int* seq_lens,
+                                            const int* cu_q, const float* sinks, const void* gate, int gate_ld, void* out, int B, int Tq, int max_q_len, int n_q,
+                                            int n_kv, int dk, int dv, int max_blocks, int n_blocks, int block_size, int window, float scale, float softcap,
+                                            const void* pk, const void* pv, int pool, int pool_pages, const float* out_cos, const float* out_sin, int out_n,
+                                            int out_half, cudaStream_t st) {
+  if (B <= 0 || Tq <= 0) return 0;
+  if (block_size != FA_PAGE) return -110;
+  if (n_kv < 1 || n_q % n_kv) return -111;
+  if (dk < 8 || dv < 8 || dk > 256 || dv > 256 || dk % 8 || dv % 8 || q_ld % 8 || out_half > dv / 2 || pool < 0) return -112;
+  if (pool && (window < 1 || !pk || !pv || pool_pages < 1)) return -112;
+  if ((gate && (gate_ld % 8 || ((uintptr_t)gate & 15))) || (((uintptr_t)q | (uintptr_t)pk | (uintptr_t)pv) & 15)) return -112;
+  FaParams p;
+  p.block_table = block_table; p.rot_table = nullptr; p.seq_lens = seq_lens; p.cu_q = cu_q; p.sinks = sinks; p.out = (__nv_bfloat16*)out;
+  p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate ? gate_ld : 0; p.q_scale = nullptr; p.q_scale_n = 0; p.gate_heads = p.keep_first = 0;
+  p.dk = dk; p.dv = dv; p.q_ld = q_ld; p.n_q = n_q; p.n_kv = n_kv; p.max_blocks = max_blocks; p.window = window; p.scale = scale; p.softcap = softcap;
+  p.pool = pool; p.pool_pages = pool_pages; p.out_cos = out_cos; p.out_sin = out_sin; p.out_n = out_n; p.out_half = out_half;
+  p.max_q_tiles = (max_q_len + FA_BQ - 1) / FA_BQ;
+  p.status = status_word();
+  const FaPooled x{pk, pv, B * pool_pages};
+  const int a = dk <= 64 ? 64 : dk <= 128 ? 128 : 256, b = dv <= 64 ? 64 : dv <= 128 ? 128 : 256;
+#define MX_FAP(DK_, DV_) launch_fa_pooled<DK_, DV_>(q, k_cache, v_cache, x, p, B, Tq, n_blocks, st)
+  if (a == 64 && b == 64) return MX_FAP(64, 64);
+  if (a == 64 && b == 128) return MX_FAP(64, 128);
+  if (a == 128 && b == 64) return MX_FAP(128, 64);
+  if (a == 128 && b == 128) return MX_FAP(128, 128);
+  return MX_FAP(256, 256);
+#undef MX_FAP
+}
+
 // Latent attention over expanded pages (see FaSplit).  q: [Tq] rows of [n_q][dim | rot], q_ld elements apart, rotated; kv: [n_pages * 128][n_q * (dim +
 // vdim)], its pages listed by kv_table; cache: [n_blocks][128][rank + rot], its pages listed by block_table (both tables [B][max_blocks]); gate (rows of
 // [n_q][vdim], gate_ld apart; out *= sigmoid(gate)); out [Tq][n_q][vdim].  Widths are multiples of 8: dim up to 192, rot up to 64, vdim up to 256.
@@ -530,6 +666,7 @@ MX_HOST_API int mx_attention_prefill_latent(const void* q, int q_ld, const void*
   FaParams p;
   p.block_table = kv_table; p.rot_table = block_table; p.seq_lens = seq_lens; p.cu_q = cu_q; p.sinks = nullptr; p.out = (__nv_bfloat16*)out;
   p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate ? gate_ld : 0; p.q_scale = nullptr; p.q_scale_n = 0; p.gate_heads = p.keep_first = 0;
+  p.pool = p.pool_pages = p.out_n = p.out_half = 0; p.out_cos = p.out_sin = nullptr;
   p.dk = dim + rot; p.dv = vdim; p.q_ld = q_ld; p.n_q = n_q; p.n_kv = n_q; p.max_blocks = max_blocks; p.window = window; p.scale = scale; p.softcap = 0.f;
   p.max_q_tiles = (max_q_len + FA_BQ - 1) / FA_BQ;
   p.status = status_word();

@@ -312,10 +312,10 @@ __global__ void __launch_bounds__(GN_WARPS * 32) group_norm_kernel(const GroupNo
 
 // ------------------------------------------------------------------ sublayer_norm
 // Norms on a sublayer's output.  In one pass over a row, the branch d formed as it is read:
-//   x (fp32 residual) += norm(d) * delta_w          (KIND 0: x is only read)
+//   x (fp32 residual) += norm(d) * delta_w          (delta_w null: += d; KIND 0: x is only read)
 //   out                = x, or norm(x) * w when w is given   (out null: skipped)
-// d: a row (KIND 1); the sum of the rows pos[t * K + k] of a, k < K, and of row t of b when there is one (KIND 2: a token's experts and the expert that
-// every token uses); the mean of norm(a) * a_w and norm(b) * b_w (KIND 3: two mixers side by side).
+// d: a row (KIND 1); the sum of the rows pos[t * K + k] of a, k < K, each times pw[t * K + k] when there are weights, and of row t of b when there is one,
+// times the sigmoid of b_gate[t * b_gate_ld] when there is a gate (KIND 2: a token's experts and the expert that every token uses); the mean of norm(a) * a_w and norm(b) * b_w (KIND 3: two mixers side by side).
 // Rows have ld elements (a multiple of 4) of which the first H count; the others are zero in a, b and the weights and stay zero.
 // A team of `wpg` warps owns a row and keeps NV pieces of four elements per lane; NV == 0: any width, memory is read again.
 struct SublayerNormParams {
@@ -323,13 +323,16 @@ struct SublayerNormParams {
   const void* a;
   const void* b;
   const int* pos;
+  const float* pw;
+  const float* b_gate;
   const float* a_w;
   const float* b_w;
   const float* delta_w;
   const float* w;
   void* out;
   float eps, inv_h;
-  int T, ld, K, wpg;
+  int T, ld, K, wpg, b_gate_ld;
+  long long out_ld;
 };
 
 template <int KIND, typename DT, typename OT, int NV>
@@ -344,8 +347,9 @@ __global__ void __launch_bounds__(GN_WARPS * 32) sublayer_norm_kernel(const Subl
   float* xr = p.x + row;
   const DT* ar = reinterpret_cast<const DT*>(p.a) + row;
   const DT* br = reinterpret_cast<const DT*>(p.b) + row;
-  OT* orow = reinterpret_cast<OT*>(p.out) + row;
+  OT* orow = reinterpret_cast<OT*>(p.out) + t * p.out_ld;
   const int first = ((warp % wpg) * 32 + lane) * 4, step = wpg * 128;
+  const float b_factor = KIND == 2 && p.b && p.b_gate ? sigmoid_f<sizeof(DT) == 4>(p.b_gate[(size_t)t * p.b_gate_ld]) : 1.f;
   float x[N][4], d[N][4], e2[KIND == 3 ? N : 1][4];
 
   auto fetch = [&](int c, float (&dv)[4], float (&ev)[4]) {
@@ -353,11 +357,16 @@ __global__ void __launch_bounds__(GN_WARPS * 32) sublayer_norm_kernel(const Subl
     if constexpr (KIND == 2) {
       if (p.b) loadv<4>(br + c, dv);
       else dv[0] = dv[1] = dv[2] = dv[3] = 0.f;
+      if (p.b_gate) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) dv[e] *= b_factor;
+      }
       for (int k = 0; k < p.K; ++k) {
         float v[4];
         loadv<4>(reinterpret_cast<const DT*>(p.a) + (size_t)p.pos[(size_t)t * p.K + k] * p.ld + c, v);
+        const float w = p.pw ? p.pw[(size_t)t * p.K + k] : 1.f;
 #pragma unroll
-        for (int e = 0; e < 4; ++e) dv[e] += v[e];
+        for (int e = 0; e < 4; ++e) dv[e] = fmaf(w, v[e], dv[e]);
       }
     }
     if constexpr (KIND == 3) { loadv<4>(ar + c, dv); loadv<4>(br + c, ev); }
@@ -403,15 +412,16 @@ __global__ void __launch_bounds__(GN_WARPS * 32) sublayer_norm_kernel(const Subl
         sa = square(d[j], sa);
       });
     }
-    const float dinv = rsqrtf(team_sum(sa, red, warp, wpg) * p.inv_h + p.eps);
+    const bool plain = p.delta_w == nullptr;
+    const float dinv = plain ? 1.f : rsqrtf(team_sum(sa, red, warp, wpg) * p.inv_h + p.eps);
     each([&](int c, int j) {
       if (NV == 0) {
         loadv<4>(xr + c, x[j]);
         fetch(c, d[j], e2[KIND == 3 ? j : 0]);
         if constexpr (KIND == 3) mean(c, d[j], e2[j], ia, ib);
       }
-      float wv[4];
-      loadv<4>(p.delta_w + c, wv);
+      float wv[4] = {1.f, 1.f, 1.f, 1.f};
+      if (!plain) loadv<4>(p.delta_w + c, wv);
 #pragma unroll
       for (int e = 0; e < 4; ++e) x[j][e] = fmaf(d[j][e] * dinv, wv[e], x[j][e]);
       storev<4>(xr + c, x[j]);
@@ -751,6 +761,17 @@ struct QkPostParams {
   void* v_cache;
   int q_ld, k_ld, T, n_q, n_kv, dp, dim, rot, interleaved, norm_after, block_size, max_pos, hpw;
   float eps;
+  const float* q_scale;        // [n_q] factor on the finished queries of a head, or null
+  // values of their own (null: the keys as they came are the values): row t of head h at t * v_ld + h * dv, turned in neighbouring pairs
+  const void* v;
+  const float* v_cos;          // [v_max_pos][v_half]
+  const float* v_sin;
+  int v_ld, dv, v_half, v_max_pos;
+  // pooled blocks of a step with one token per sequence (null: none): layout as in pooled.cu
+  void* pk;                    // [blocks][n_kv][pool_rows][dp]
+  void* pv;
+  const int* block_table;      // [T][max_blocks]
+  int pool, pool_rows, window, max_blocks;
 };
 constexpr int QK_WARPS = 4;
 
@@ -772,16 +793,50 @@ __global__ void __launch_bounds__(QK_WARPS * 32) qk_post_kernel(const QkPostPara
   pdl_prologue();
   __shared__ float sh[QK_WARPS][NG == 1 ? 32 * G : 32 * G * NG];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int heads = p.n_q + p.n_kv, per_tok = (heads + p.hpw - 1) / p.hpw;
+  // units of a token: query and key heads, then value heads, then pooled rows
+  const int qk_heads = p.n_q + p.n_kv, qk_units = (qk_heads + p.hpw - 1) / p.hpw, v_units = p.v ? (p.n_kv + p.hpw - 1) / p.hpw : 0;
+  const int all = qk_units + v_units + (p.pk ? p.n_kv : 0);
   const long long unit = (long long)blockIdx.x * QK_WARPS + warp;
-  if (unit >= (long long)p.T * per_tok) return;
-  const int t = (int)(unit / per_tok), h0 = (int)(unit - (long long)t * per_tok);            // heads h0, h0 + per_tok, ...
-  const int dp = p.dp, half = p.rot / 2;
+  if (unit >= (long long)p.T * all) return;
+  const int t = (int)(unit / all);
+  int h0 = (int)(unit - (long long)t * all);
   const long long slot = p.slot_map[t];
+  if (h0 >= qk_units + v_units) {                                          // the block that this token is the first to see, if there is one
+    const int h = h0 - qk_units - v_units, end = p.positions[t] + 1 - p.window, b = end / p.pool - 1;
+    if (slot < 0 || end < p.pool || end % p.pool) return;
+    const int* table = p.block_table + (size_t)t * p.max_blocks;
+    const int page = (end - 1) / p.block_size;
+    const size_t at = ((size_t)table[page] * p.n_kv + h) * p.pool_rows + (b - page * p.block_size / p.pool);
+    for (int which = 0; which < 2; ++which) {
+      const int width = which ? p.dv : p.dp;
+      const T* cache = reinterpret_cast<const T*>(which ? p.v_cache : p.k_cache);
+      T* out = reinterpret_cast<T*>(which ? p.pv : p.pk) + at * width;
+      for (int c = lane * 4; c < width; c += 128) {
+        float a[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 8
+        for (int j = 0; j < p.pool; ++j) {
+          const int i = b * p.pool + j;
+          float v[4];
+          loadv<4>(cache + (((size_t)table[i / p.block_size] * p.n_kv + h) * p.block_size + i % p.block_size) * width + c, v);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) a[e] += v[e];
+        }
+#pragma unroll
+        for (int e = 0; e < 4; ++e) a[e] /= (float)p.pool;
+        storev<4>(out + c, a);
+      }
+    }
+    return;
+  }
+  const bool vals = h0 >= qk_units;
+  if (vals) h0 -= qk_units;
+  const int heads = vals ? p.n_kv : qk_heads, per_tok = vals ? v_units : qk_units;           // heads h0, h0 + per_tok, ...
+  const int dp = vals ? p.dv : p.dp, half = vals ? p.v_half : p.rot / 2, rot = 2 * half, max_pos = vals ? p.v_max_pos : p.max_pos;
+  const bool interleaved = vals || p.interleaved;
   int pos = p.positions[t];
-  pos = pos < 0 ? 0 : (pos >= p.max_pos ? p.max_pos - 1 : pos);
-  const float* cs = p.rope_cos + (size_t)pos * half;
-  const float* sn = p.rope_sin + (size_t)pos * half;
+  pos = pos < 0 ? 0 : (pos >= max_pos ? max_pos - 1 : pos);
+  const float* cs = (vals ? p.v_cos : p.rope_cos) + (size_t)pos * half;
+  const float* sn = (vals ? p.v_sin : p.rope_sin) + (size_t)pos * half;
   // element i turns into v_i c_i + v_partner s_i
   float c[NG][G], s[NG][G];
 #pragma unroll
@@ -789,15 +844,16 @@ __global__ void __launch_bounds__(QK_WARPS * 32) qk_post_kernel(const QkPostPara
 #pragma unroll
     for (int e = 0; e < G; ++e) {
       const int i = (g * 32 + lane) * G + e;
-      const bool first = p.interleaved ? !(i & 1) : i < half;
-      const int f = p.interleaved ? i >> 1 : first ? i : i - half;
-      c[g][e] = i < p.rot ? __ldg(cs + f) : 1.f;
-      s[g][e] = i < p.rot ? (first ? -__ldg(sn + f) : __ldg(sn + f)) : 0.f;
+      const bool first = interleaved ? !(i & 1) : i < half;
+      const int f = interleaved ? i >> 1 : first ? i : i - half;
+      c[g][e] = i < rot ? __ldg(cs + f) : 1.f;
+      s[g][e] = i < rot ? (first ? -__ldg(sn + f) : __ldg(sn + f)) : 0.f;
     }
   const bool by_shuffle = NG == 1 && half % G == 0;                      // a lane's partners sit in one other lane
   const int partner = lane * G < half ? lane + half / G : lane - half / G;
   auto source = [&](int h) {
-    return h < p.n_q ? reinterpret_cast<const T*>(p.q) + (size_t)t * p.q_ld + (size_t)h * dp
+    return vals ? reinterpret_cast<const T*>(p.v) + (size_t)t * p.v_ld + (size_t)h * dp
+           : h < p.n_q ? reinterpret_cast<const T*>(p.q) + (size_t)t * p.q_ld + (size_t)h * dp
                      : reinterpret_cast<const T*>(p.k) + (size_t)t * p.k_ld + (size_t)(h - p.n_q) * dp;
   };
   float next[NG][G];
@@ -815,9 +871,9 @@ __global__ void __launch_bounds__(QK_WARPS * 32) qk_post_kernel(const QkPostPara
   };
   fetch(h0);
   for (int h = h0; h < heads; h += per_tok) {
-    const bool is_q = h < p.n_q;
+    const bool is_q = !vals && h < p.n_q;
     if (!is_q && slot < 0) break;                                        // (key heads come last)
-    const int kh = h - p.n_q;
+    const int kh = vals ? h : h - p.n_q;
     const long long crow = is_q ? 0 : (((slot / p.block_size) * p.n_kv + kh) * p.block_size + slot % p.block_size) * dp;
     float v[NG][G], ss = 0.f;
 #pragma unroll
@@ -825,10 +881,10 @@ __global__ void __launch_bounds__(QK_WARPS * 32) qk_post_kernel(const QkPostPara
       const int e0 = (g * 32 + lane) * G;
 #pragma unroll
       for (int e = 0; e < G; ++e) { v[g][e] = next[g][e]; ss = fmaf(v[g][e], v[g][e], ss); }
-      if (!is_q && e0 < dp) store_group<G>(reinterpret_cast<T*>(p.v_cache) + crow + e0, v[g]);
+      if (!is_q && !p.v && e0 < dp) store_group<G>(reinterpret_cast<T*>(p.v_cache) + crow + e0, v[g]);
     }
     if (h + per_tok < heads) fetch(h + per_tok);
-    const float* nw = is_q ? p.q_norm : p.k_norm;
+    const float* nw = vals ? nullptr : is_q ? p.q_norm : p.k_norm;
     if (nw) {
       const float inv = rsqrtf(warp_sum(ss) / (float)p.dim + p.eps);
 #pragma unroll
@@ -842,7 +898,7 @@ __global__ void __launch_bounds__(QK_WARPS * 32) qk_post_kernel(const QkPostPara
         }
       }
     }
-    if (p.interleaved) {
+    if (interleaved) {
 #pragma unroll
       for (int g = 0; g < NG; ++g)
 #pragma unroll
@@ -868,10 +924,10 @@ __global__ void __launch_bounds__(QK_WARPS * 32) qk_post_kernel(const QkPostPara
 #pragma unroll
         for (int e = 0; e < G; ++e) {
           const int i = (g * 32 + lane) * G + e;
-          if (i < p.rot) v[g][e] = fmaf(buf[i < half ? i + half : i - half], s[g][e], v[g][e] * c[g][e]);
+          if (i < rot) v[g][e] = fmaf(buf[i < half ? i + half : i - half], s[g][e], v[g][e] * c[g][e]);
         }
     }
-    if (p.norm_after) {
+    if (p.norm_after && !vals) {
       ss = 0.f;
 #pragma unroll
       for (int g = 0; g < NG; ++g)
@@ -883,7 +939,14 @@ __global__ void __launch_bounds__(QK_WARPS * 32) qk_post_kernel(const QkPostPara
 #pragma unroll
         for (int e = 0; e < G; ++e) v[g][e] *= inv;
     }
-    T* dst = is_q ? reinterpret_cast<T*>(p.q) + (size_t)t * p.q_ld + (size_t)h * dp : reinterpret_cast<T*>(p.k_cache) + crow;
+    if (is_q && p.q_scale) {
+      const float f = p.q_scale[h];
+#pragma unroll
+      for (int g = 0; g < NG; ++g)
+#pragma unroll
+        for (int e = 0; e < G; ++e) v[g][e] *= f;
+    }
+    T* dst = is_q ? reinterpret_cast<T*>(p.q) + (size_t)t * p.q_ld + (size_t)h * dp : reinterpret_cast<T*>(vals ? p.v_cache : p.k_cache) + crow;
 #pragma unroll
     for (int g = 0; g < NG; ++g) {
       const int e0 = (g * 32 + lane) * G;
@@ -903,8 +966,13 @@ __device__ __forceinline__ float glu_act(int act, float g, float u, float alpha,
   const float t = tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g));
   return 0.5f * g * (1.f + t) * u;
 }
-// (fp32 rows: SwiGLU through the full-precision exponential)
+// (fp32 rows: SwiGLU and its clamped form through the full-precision exponential)
 __device__ __forceinline__ float glu_act_precise(int act, float g, float u, float alpha, float limit) {
+  if (act == 2) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g * sigmoid_f<true>(alpha * g) * (u + 1.f);
+  }
   return act == 1 ? g * sigmoid_f<true>(g) * u : glu_act(act, g, u, alpha, limit);
 }
 __global__ void glu_f32_kernel(const float* __restrict__ in, float* __restrict__ out, long long total_out, int F, int act, float alpha, float limit) {
@@ -1090,34 +1158,43 @@ static int dispatch_sublayer_norm(int kind, const SublayerNormParams& p, cudaStr
 }  // namespace mx
 
 // See sublayer_norm_kernel.  x fp32 [T][ld]; kind 0 nothing, 1 a row of a, 2 rows pos[t][K] of a (+ row t of b), 3 the mean of a and b normed; a and b are
-// bf16, or fp32 when out is (out null: elem_f32 names the dtype of a and b).
-MX_HOST_API int mx_sublayer_norm(int kind, float* x, const void* a, const void* b, const int* pos, int K, const float* a_w, const float* b_w, const float* delta_w,
-                                 const float* w, void* out, int elem_f32, float eps, int T, int H, int ld, cudaStream_t st) {
+// bf16, or fp32 when out is (out null: elem_f32 names the dtype of a and b).  pw [T][K], b_gate (stride b_gate_ld): factors of kind 2, or null.  out: rows
+// out_ld elements apart (a multiple of 4).
+MX_HOST_API int mx_sublayer_norm(int kind, float* x, const void* a, const void* b, const int* pos, int K, const float* pw, const float* b_gate, int b_gate_ld,
+                                 const float* a_w, const float* b_w, const float* delta_w, const float* w, void* out, long long out_ld, int elem_f32, float eps,
+                                 int T, int H, int ld, cudaStream_t st) {
   if (T <= 0) return 0;
-  if (H < 1 || ld < H || ld % 4 || kind < 0 || kind > 3) return -107;
-  if ((kind && (!a || !delta_w)) || (kind == 2 && (!pos || K < 1)) || (kind == 3 && (!b || !a_w || !b_w))) return -109;
+  if (H < 1 || ld < H || ld % 4 || kind < 0 || kind > 3 || out_ld % 4 || (out && out_ld < ld)) return -107;
+  if ((kind && !a) || (kind == 3 && !delta_w) || (kind == 2 && (!pos || K < 1)) || (kind == 3 && (!b || !a_w || !b_w))) return -109;
   SublayerNormParams p;
   p.x = x; p.a = a; p.b = b; p.pos = pos; p.a_w = a_w; p.b_w = b_w; p.delta_w = delta_w; p.w = w; p.out = out; p.eps = eps; p.inv_h = 1.f / (float)H;
-  p.T = T; p.ld = ld; p.K = K;
+  p.T = T; p.ld = ld; p.K = K; p.pw = pw; p.b_gate = b_gate; p.b_gate_ld = b_gate_ld; p.out_ld = out_ld;
   return elem_f32 ? dispatch_sublayer_norm<float, float>(kind, p, st) : dispatch_sublayer_norm<__nv_bfloat16, __nv_bfloat16>(kind, p, st);
 }
 
-// See qk_post_kernel.  dp (the padded head width) a multiple of 8 up to 512, dim <= dp its live elements, rot <= dim even.
+// See qk_post_kernel.  dp (the padded head width) a multiple of 8 up to 512, dim <= dp its live elements, rot <= dim even; the same of dv and 2 v_half.
 MX_HOST_API int mx_qk_post(void* q, int q_ld, const void* k, int k_ld, const float* q_norm, const float* k_norm, const int* positions, const float* rope_cos,
                            const float* rope_sin, int max_pos, const long long* slot_map, void* k_cache, void* v_cache, int T, int n_q, int n_kv, int dp, int dim,
-                           int rot, int interleaved, int norm_after, int block_size, float eps, int elem_f32, cudaStream_t st) {
+                           int rot, int interleaved, int norm_after, int block_size, float eps, int elem_f32, const float* q_scale, const void* v, int v_ld, int dv,
+                           const float* v_cos, const float* v_sin, int v_half, int v_max_pos, void* pk, void* pv, const int* block_table, int max_blocks, int pool,
+                           int pool_rows, int window, cudaStream_t st) {
   if (T <= 0) return 0;
+  if (v && (dv < 8 || dv > 512 || dv % 8 || v_half < 0 || 2 * v_half > dv || v_ld % 8 || ((uintptr_t)v & 15))) return -108;
+  if (pk && (!pv || !v || !block_table || pool < 1 || window < 1 || pool_rows < (block_size + pool - 1) / pool)) return -108;
   if (dp < 8 || dp > 512 || dp % 8 || dim < 1 || dim > dp || rot < 0 || rot > dim || rot % 2 || q_ld % 8 || k_ld % 8 || (((uintptr_t)q | (uintptr_t)k) & 15)) return -108;
   QkPostParams p;
   p.q = q; p.k = k; p.q_norm = q_norm; p.k_norm = k_norm; p.positions = positions; p.rope_cos = rope_cos; p.rope_sin = rope_sin; p.slot_map = slot_map;
   p.k_cache = k_cache; p.v_cache = v_cache; p.q_ld = q_ld; p.k_ld = k_ld; p.T = T; p.n_q = n_q; p.n_kv = n_kv; p.dp = dp; p.dim = dim; p.rot = rot;
   p.interleaved = interleaved; p.norm_after = norm_after; p.block_size = block_size; p.max_pos = max_pos; p.eps = eps;
+  p.q_scale = q_scale; p.v = v; p.v_ld = v_ld; p.dv = v ? dv : dp; p.v_cos = v_cos; p.v_sin = v_sin; p.v_half = v_half; p.v_max_pos = v_max_pos;
+  p.pk = pk; p.pv = pv; p.block_table = block_table; p.max_blocks = max_blocks; p.pool = pool; p.pool_rows = pool_rows; p.window = window;
   const int heads = n_q + n_kv;
   p.hpw = (long long)T * heads >= 64ll * 64 * sm_count() / 8 ? 8 : 1;    // (many tokens: the chip is full with fewer, longer warps)
   if (p.hpw > heads) p.hpw = heads;
-  const long long units = (long long)T * ((heads + p.hpw - 1) / p.hpw);
+  const long long units = (long long)T * ((heads + p.hpw - 1) / p.hpw + (v ? (n_kv + p.hpw - 1) / p.hpw : 0) + (pk ? n_kv : 0));
+  const int wide = v && dv > dp ? dv : dp;
   const dim3 grid((unsigned)((units + QK_WARPS - 1) / QK_WARPS)), block(QK_WARPS * 32);
-#define MX_QK(T_)   (dp <= 64 ? launch_pdl(qk_post_kernel<T_, 2, 1>, grid, block, 0, st, p) : dp <= 128 ? launch_pdl(qk_post_kernel<T_, 4, 1>, grid, block, 0, st, p)    : dp <= 256 ? launch_pdl(qk_post_kernel<T_, 8, 1>, grid, block, 0, st, p) : launch_pdl(qk_post_kernel<T_, 8, 2>, grid, block, 0, st, p))
+#define MX_QK(T_)   (wide <= 64 ? launch_pdl(qk_post_kernel<T_, 2, 1>, grid, block, 0, st, p) : wide <= 128 ? launch_pdl(qk_post_kernel<T_, 4, 1>, grid, block, 0, st, p)    : wide <= 256 ? launch_pdl(qk_post_kernel<T_, 8, 1>, grid, block, 0, st, p) : launch_pdl(qk_post_kernel<T_, 8, 2>, grid, block, 0, st, p))
   if (elem_f32) MX_QK(float); else MX_QK(__nv_bfloat16);
 #undef MX_QK
   return (int)cudaGetLastError();

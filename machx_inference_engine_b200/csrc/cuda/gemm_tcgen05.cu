@@ -665,16 +665,16 @@ static int gemm_impl(const void* a, int wfmt, const void* w0, const void* w1, co
 }
 
 // Every head its own matrix: c[t][h][:] = a[t][h][:] W[h]^T (* sigmoid(gate[t][h][:])).  a: row t of head h at t * lda + h * a_head, K elements; w bf16
-// [heads][N][K]; c: bf16, row t of head h at t * ldc + h * c_head; gate (or null): rows of heads * N, gate_ld apart.  Widths, strides and bases are
+// [heads][N][K]; c: bf16 or (out_f32) fp32, row t of head h at t * ldc + h * c_head; gate (or null): rows of heads * N, gate_ld apart.  Widths, strides and bases are
 // multiples of 8 elements.
 MX_HOST_API int mx_gemm_heads(const void* a, int lda, long long a_head, const void* w, void* c, int ldc, long long c_head, const void* gate, int gate_ld,
-                              int T, int heads, int N, int K, int bn, cudaStream_t stream) {
+                              int T, int heads, int N, int K, int bn, int out_f32, cudaStream_t stream) {
   if (T <= 0 || heads <= 0) return 0;
   if (N % 8 || K % 8 || lda % 8 || a_head % 8 || ldc % 8 || c_head % 8 || (gate && gate_ld % 8)) return -101;
   if (((uintptr_t)a | (uintptr_t)w | (uintptr_t)c | (uintptr_t)gate) & 15) return -101;
   StridedIn s;
   s.heads = heads; s.lda = lda; s.a_head = a_head; s.c_head = c_head; s.gate = gate; s.gate_ld = gate_ld;
-  return gemm_impl(a, mx::WF_BF16, w, nullptr, nullptr, nullptr, heads, c, ldc, 0, nullptr, nullptr, 0, 0.f, 0.f, T, N, K, nullptr, nullptr, bn, nullptr, stream,
+  return gemm_impl(a, mx::WF_BF16, w, nullptr, nullptr, nullptr, heads, c, ldc, out_f32 ? 1 : 0, nullptr, nullptr, 0, 0.f, 0.f, T, N, K, nullptr, nullptr, bn, nullptr, stream,
                    nullptr, &s);
 }
 

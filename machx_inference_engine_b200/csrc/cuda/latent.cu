@@ -120,6 +120,7 @@ struct HeadLinearParams {
   long long x_ld, o_ld;
   int x_hs, o_hs, gate_ld;
   int T, N, K, lpr;            // lpr: lanes per weight row (a power of two)
+  int out_f32;                 // out is fp32 whatever x is
 };
 constexpr int HL_WARPS = 4, HL_ROWS = 2;           // weight rows in flight per lane group
 
@@ -195,7 +196,9 @@ __global__ void __launch_bounds__(HL_WARPS * 32) head_linear_kernel(const HeadLi
       if (n >= p.N) break;
       float v = acc[r][t];
       if (p.gate) v *= sigmoid_f<sizeof(T) == 4>(to_f32(reinterpret_cast<const T*>(p.gate)[(size_t)(t0 + t) * p.gate_ld + (size_t)h * p.N + n]));
-      reinterpret_cast<T*>(p.out)[(size_t)(t0 + t) * p.o_ld + (size_t)h * p.o_hs + n] = from_f32<T>(v);
+      const size_t at = (size_t)(t0 + t) * p.o_ld + (size_t)h * p.o_hs + n;
+      if (p.out_f32) reinterpret_cast<float*>(p.out)[at] = v;
+      else reinterpret_cast<T*>(p.out)[at] = from_f32<T>(v);
     }
   }
 }
@@ -262,14 +265,14 @@ MX_HOST_API int mx_latent_post(const void* q, int q_ld, int q_hs, void* q_out, i
   return (int)cudaGetLastError();
 }
 
-// out[t][h][:] = W[h] x[t][h][:] (* sigmoid(gate)); see HeadLinearParams.  K a multiple of 8, at most 1536; w on a 16-byte boundary.
+// out[t][h][:] = W[h] x[t][h][:] (* sigmoid(gate)), fp32 with out_f32; see HeadLinearParams.  K a multiple of 8, at most 1536; w on a 16-byte boundary.
 MX_HOST_API int mx_head_linear(const void* x, long long x_ld, int x_hs, const void* w, const void* gate, int gate_ld, void* out, long long o_ld, int o_hs, int T,
-                               int H, int N, int K, int elem_f32, cudaStream_t st) {
+                               int H, int N, int K, int elem_f32, int out_f32, cudaStream_t st) {
   if (T <= 0 || H <= 0 || N <= 0) return 0;
   if (K % 8 || K < 8 || K > 1536 || x_ld % 2 || x_hs % 2 || ((uintptr_t)w & 15) || ((uintptr_t)x & 7)) return -101;
   HeadLinearParams p;
   p.x = x; p.w = (const __nv_bfloat16*)w; p.gate = gate; p.out = out; p.x_ld = x_ld; p.o_ld = o_ld; p.x_hs = x_hs; p.o_hs = o_hs; p.gate_ld = gate_ld;
-  p.T = T; p.N = N; p.K = K;
+  p.T = T; p.N = N; p.K = K; p.out_f32 = out_f32 || elem_f32;
   p.lpr = 1;
   while (p.lpr < 32 && p.lpr * 8 < K) p.lpr *= 2;
   return elem_f32 ? launch_head_linear<float>(p, H, st) : launch_head_linear<__nv_bfloat16>(p, H, st);

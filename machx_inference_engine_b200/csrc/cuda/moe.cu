@@ -20,11 +20,11 @@ constexpr int MOE_TILE = 128;
 // one warp per token; E <= 1024
 template <bool PRECISE>
 __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int T, int E, int K,
-                                                        int renorm, int* __restrict__ topk_idx, float* __restrict__ topk_w) {
+                                                        int renorm, int ld, int* __restrict__ topk_idx, float* __restrict__ topk_w) {
   pdl_prologue();
   const int t = blockIdx.x * 4 + (threadIdx.x >> 5);
   if (t >= T) return;
-  route_token_warp<PRECISE>(logits, bias, t, E, K, renorm, topk_idx, topk_w);
+  route_token_warp<PRECISE>(logits, bias, t, E, K, renorm, topk_idx, topk_w, 1, ld);
 }
 
 // Single-CTA packer.  n = T*K pairs.  Outputs:
@@ -305,13 +305,13 @@ MX_HOST_API int mx_moe_combine_push(const void* yp, const int* pair_to_packed, c
   return (int)cudaGetLastError();
 }
 
-// renorm: see moe_route.cuh; precise: the softmax uses the full-precision exponential
-MX_HOST_API int mx_moe_route(const float* logits, const float* bias, int T, int E, int K, int renorm, int precise, int* topk_idx, float* topk_w,
+// renorm: see moe_route.cuh; precise: the softmax uses the full-precision exponential; ld: elements between the logits of two tokens
+MX_HOST_API int mx_moe_route(const float* logits, const float* bias, int T, int E, int K, int renorm, int precise, int ld, int* topk_idx, float* topk_w,
                              cudaStream_t st) {
   if (T <= 0) return 0;
-  if (E > 1024 || K > 32 || K > E) return -120;
-  if (precise) launch_pdl(moe_route_kernel<true>, dim3((T + 3) / 4), dim3(128), 0, st, logits, bias, T, E, K, renorm, topk_idx, topk_w);
-  else launch_pdl(moe_route_kernel<false>, dim3((T + 3) / 4), dim3(128), 0, st, logits, bias, T, E, K, renorm, topk_idx, topk_w);
+  if (ld < E || E > 1024 || K > 32 || K > E) return -120;
+  if (precise) launch_pdl(moe_route_kernel<true>, dim3((T + 3) / 4), dim3(128), 0, st, logits, bias, T, E, K, renorm, ld, topk_idx, topk_w);
+  else launch_pdl(moe_route_kernel<false>, dim3((T + 3) / 4), dim3(128), 0, st, logits, bias, T, E, K, renorm, ld, topk_idx, topk_w);
   return (int)cudaGetLastError();
 }
 

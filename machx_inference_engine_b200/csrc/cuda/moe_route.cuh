@@ -1,6 +1,6 @@
 // Router top-k for one token, executed by one warp: weights = softmax over the selected logits (renorm 1), softmax over all (0)
 // or the sigmoids of the selected logits as they are (2).
-// Lane k < K ends up holding the k-th selection; E <= 1024, K <= 32.  The logits are read past L1: the caller may be the last CTA
+// ld: elements between the logits of two tokens (0: E).  Lane k < K ends up holding the k-th selection; E <= 1024, K <= 32.  The logits are read past L1: the caller may be the last CTA
 // of the kernel that produced them.
 #pragma once
 #include "common.cuh"
@@ -12,7 +12,8 @@ template <bool PRECISE> __device__ __forceinline__ float route_exp(float x) { re
 // PRECISE: weights through expf (models that run in 32-bit), otherwise the fast exponential.
 template <bool PRECISE = false>
 __device__ __forceinline__ void route_token_warp(const float* __restrict__ logits, const float* __restrict__ bias, int t, int E, int K, int renorm,
-                                                 int* __restrict__ topk_idx, float* __restrict__ topk_w, int w_copies = 1) {
+                                                 int* __restrict__ topk_idx, float* __restrict__ topk_w, int w_copies = 1, int ld = 0) {
+  if (!ld) ld = E;
   const int lane = threadIdx.x & 31;
   float v[32];
   const int per = (E + 31) / 32;
@@ -20,7 +21,7 @@ __device__ __forceinline__ void route_token_warp(const float* __restrict__ logit
 #pragma unroll
   for (int i = 0; i < 32; ++i) {
     const int e = lane + 32 * i;
-    v[i] = (i < per && e < E) ? __ldcg(logits + (size_t)t * E + e) + (bias ? bias[e] : 0.f) : -INFINITY;
+    v[i] = (i < per && e < E) ? __ldcg(logits + (size_t)t * ld + e) + (bias ? bias[e] : 0.f) : -INFINITY;
     mx_all = fmaxf(mx_all, v[i]);
   }
   mx_all = warp_max(mx_all);

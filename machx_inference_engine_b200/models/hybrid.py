@@ -201,10 +201,14 @@ class RglruBlock:
     The matrices of a block's two gates are one stack entry, so a prompt is convolution, per-block GEMM (fp32 results), recurrence with its gates and its
     output factor; a step of single tokens is one kernel.  Blocks are padded so that each starts on a vector and all together fill rows of 32."""
 
+    MAX_BLOCK, MAX_TAPS = 1536, 8    # what the kernels take
+
     def __init__(self, src, prefix: str, hidden: int, row: int, width: int, blocks: int, taps: int):
         n = width // blocks
         to = self.n = round_up(n, max(8, 32 // math.gcd(blocks, 32)))
         self.blocks, self.width = blocks, blocks * to
+        if to > self.MAX_BLOCK or taps > self.MAX_TAPS:
+            raise ValueError(f"{prefix}: blocks of {n} channels with {taps} taps are more than the {self.MAX_BLOCK} and {self.MAX_TAPS} the kernels take")
         ws = [src.matrix(f"{prefix}.{m}", width, hidden).pad_groups(rows=(blocks, to), cols=(1, row)) for m in ("x", "y")]
         pad = lambda v: _pad_heads(v, blocks, to)
         self.proj = _fuse_rows(ws, [pad(src.vector(f"{prefix}.{m}.b", width)) for m in ("x", "y")])

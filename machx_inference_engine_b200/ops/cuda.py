@@ -12,7 +12,7 @@ from typing import Optional
 import torch
 
 from .. import _lib
-from .ref import ACT_GEGLU, ACT_NONE, ACT_SWIGLU, ACT_SWIGLU_OAI, MOE_TILE, BranchMean, ExpertSum, MoePacking, act_gated, moe_max_rows
+from .ref import ACT_GEGLU, ACT_NONE, ACT_SWIGLU, ACT_SWIGLU_OAI, MOE_TILE, BranchMean, ExpertSum, MoePacking, PoolPages, act_gated, moe_max_rows
 from .weights import QuantWeight, WFormat
 
 _vp = C.c_void_p
@@ -158,12 +158,13 @@ def dyt_norm(x, alpha, w, b, delta=None, step=None, out_dtype=torch.bfloat16, wa
     return out
 
 
-def sublayer_norm(x, delta, delta_w, eps, w=None, width=None, out_dtype=torch.bfloat16, want_out=True):
+def sublayer_norm(x, delta, delta_w, eps, w=None, width=None, out_dtype=torch.bfloat16, want_out=True, out=None):
     T, ld = x.shape
-    kind, a, b, pos, k, aw, bw = 0, None, None, None, 0, None, None
+    kind, a, b, pos, k, aw, bw, pw, bg = 0, None, None, None, 0, None, None, None, None
     if isinstance(delta, ExpertSum):
-        kind, a, b, pos, k = 2, delta.y, delta.shared, delta.pair_to_packed, delta.k
-        assert pos.numel() == T * k and pos.dtype == torch.int32
+        kind, a, b, pos, k, pw, bg = 2, delta.y, delta.shared, delta.pair_to_packed, delta.k, delta.w, delta.shared_gate
+        assert pos.numel() == T * k and pos.dtype == torch.int32 and (pw is None or (pw.is_contiguous() and pw.numel() == T * k and pw.dtype == torch.float32))
+        assert bg is None or (bg.dtype == torch.float32 and bg.shape == (T,))
     elif isinstance(delta, BranchMean):
         kind, a, b, aw, bw = 3, delta.a, delta.b, delta.a_w, delta.b_w
     elif delta is not None:
@@ -171,26 +172,94 @@ def sublayer_norm(x, delta, delta_w, eps, w=None, width=None, out_dtype=torch.bf
     assert x.dtype == torch.float32 and x.is_contiguous()
     assert all(v is None or (v.dtype == torch.float32 and v.numel() == ld) for v in (delta_w, w, aw, bw))
     assert all(t is None or (t.is_contiguous() and t.dtype == out_dtype and t.shape[1] == ld and (kind == 2 or t.shape[0] == T)) for t in (a, b))
-    out = torch.empty(T, ld, dtype=out_dtype, device=x.device) if want_out else None
-    _check(_lib.cuda().mx_sublayer_norm(kind, _p(x), _p(a), _p(b), _p(pos), int(k), _p(aw), _p(bw), _p(delta_w), _p(w), _p(out),
-                                        int(out_dtype == torch.float32), C.c_float(eps), T, int(width or ld), ld, _stream()), "sublayer_norm")
+    if out is None and want_out:
+        out = torch.empty(T, ld, dtype=out_dtype, device=x.device)
+    assert out is None or (out.shape == (T, ld) and out.dtype == out_dtype and out.stride(1) == 1)
+    _check(_lib.cuda().mx_sublayer_norm(kind, _p(x), _p(a), _p(b), _p(pos), int(k), _p(pw), _p(bg), 0 if bg is None else bg.stride(0), _p(aw), _p(bw), _p(delta_w),
+                                        _p(w), _p(out), C.c_longlong(ld if out is None else out.stride(0)), int(out_dtype == torch.float32), C.c_float(eps), T,
+                                        int(width or ld), ld, _stream()), "sublayer_norm")
     _count()
     return out
 
 
 def qk_post(q, k, positions, rope_cos, rope_sin, slot_map, k_cache, v_cache, dim, rot_dim, interleaved=False, q_norm=None, k_norm=None, norm_after=False,
-            eps=1e-6):
+            eps=1e-6, v=None, v_rope=None, q_scale=None, pools=None, block_table=None):
     T, n_q, dp = q.shape
     n_kv = k.shape[1]
-    assert q.dtype == k.dtype == k_cache.dtype == v_cache.dtype and k_cache.shape == v_cache.shape and k_cache.shape[1] == n_kv and k_cache.shape[3] == dp
-    for t in (q, k):
-        assert t.stride(2) == 1 and (t.shape[1] == 1 or t.stride(1) == dp)
+    dv = dp if v is None else v.shape[2]
+    assert q.dtype == k.dtype == k_cache.dtype == v_cache.dtype and k_cache.shape[1] == n_kv and k_cache.shape[3] == dp
+    assert v_cache.shape == (*k_cache.shape[:3], dv) and k_cache.is_contiguous() and v_cache.is_contiguous()
+    for t in (q, k) if v is None else (q, k, v):
+        assert t.dtype == q.dtype and t.stride(2) == 1 and (t.shape[1] == 1 or t.stride(1) == t.shape[2])
+    assert v is None or v.shape[:2] == (T, n_kv)
+    assert q_scale is None or (q_scale.dtype == torch.float32 and q_scale.numel() == n_q)
+    assert pools is None or (block_table.shape[0] == T and block_table.is_contiguous())
+    v_cos, v_sin = v_rope if v_rope is not None else (None, None)
     assert rope_cos.shape[1] == rot_dim // 2 and all(n is None or n.numel() == dp for n in (q_norm, k_norm))
     _check(_lib.cuda().mx_qk_post(_p(q), q.stride(0), _p(k), k.stride(0), _p(q_norm), _p(k_norm), _p(positions), _p(rope_cos), _p(rope_sin), rope_cos.shape[0],
                                   _p(slot_map), _p(k_cache), _p(v_cache), T, n_q, n_kv, dp, int(dim), int(rot_dim), int(interleaved), int(norm_after),
-                                  k_cache.shape[2], C.c_float(eps), int(q.dtype == torch.float32), _stream()), "qk_post")
+                                  k_cache.shape[2], C.c_float(eps), int(q.dtype == torch.float32), _p(q_scale), _p(v), 0 if v is None else v.stride(0), dv,
+                                  _p(v_cos), _p(v_sin), 0 if v_cos is None else v_cos.shape[1], 1 if v_cos is None else v_cos.shape[0],
+                                  *((_vp(0), _vp(0), _vp(0), 0, 0, 0, 0) if pools is None else
+                                    (_p(pools.k), _p(pools.v), _p(block_table), block_table.shape[1], pools.pool, pools.k.shape[2], pools.window)), _stream()),
+           "qk_post")
     _count()
     return q
+
+
+def pool_blocks(k_cache, v_cache, pools: PoolPages, block_table, seq_lens, cu_q, max_q_len, max_kv_len=0):
+    """For queries that take the tensor-core kernel: dense pages (K, V) [B * pages, n_kv, 128, width] of the blocks that every sequence's last query sees."""
+    n_pages, n_kv, bs, dk = k_cache.shape
+    dv, B, P = v_cache.shape[3], seq_lens.numel(), pools.pool
+    assert pools.k.dtype == k_cache.dtype and pools.k.shape[:2] == (n_pages, n_kv) and block_table.is_contiguous()
+    longest = max_kv_len if max_kv_len > 0 else block_table.shape[1] * bs
+    seen = max(longest - pools.window, 0) // P
+    if seen == 0:
+        return None
+    dense, pages, most = None, 0, min(seen, max_q_len // P + 1)
+    if _takes_tc(max_q_len, bs, k_cache.dtype, dk, dv):
+        pages, most = (seen + 127) // 128, seen
+        dense = tuple(torch.empty(B * pages, n_kv, 128, w, dtype=k_cache.dtype, device=k_cache.device) for w in (dk, dv))
+    _check(_lib.cuda().mx_pool_blocks(_p(k_cache), _p(v_cache), _p(pools.k), _p(pools.v), _p(dense[0] if dense else None), _p(dense[1] if dense else None),
+                                      _p(block_table), _p(seq_lens), _p(cu_q), B, n_kv, bs, dk, dv, P, pools.k.shape[2], pools.window, block_table.shape[1],
+                                      pages, most, int(k_cache.dtype == torch.float32), _stream()), "pool_blocks")
+    _count()
+    return dense
+
+
+def causal_conv(x, w, b, state, state_slots, cu_q, seq_lens, max_q_len):
+    T, W = x.shape
+    assert x.stride(1) == 1 and state.dtype == x.dtype and state.shape[1:] == (w.shape[1] - 1, W) and w.is_contiguous() and w.dtype == b.dtype == torch.float32
+    y = torch.empty(T, W, dtype=x.dtype, device=x.device)
+    _check(_lib.cuda().mx_causal_conv(_p(x), x.stride(0), _p(w), _p(b), _p(state), _p(state_slots), _p(cu_q), _p(seq_lens), _p(y), cu_q.numel() - 1, T, W,
+                                      w.shape[1], int(x.dtype == torch.float32), _stream()), "causal_conv")
+    _count(2 if w.shape[1] > 1 else 1)
+    return y
+
+
+def rglru_scan(gates, u, y, bias, coef, state, state_slots, cu_q, seq_lens, max_q_len):
+    T, W = u.shape
+    n = gates.shape[2] // 2
+    assert gates.dtype == state.dtype == torch.float32 and gates.is_contiguous() and gates.shape == (T, W // n, 2 * n) and bias.numel() == 2 * W
+    assert u.dtype == y.dtype and u.stride(1) == y.stride(1) == 1 and state.shape[1] == W == coef.numel()
+    out = torch.empty(T, W, dtype=u.dtype, device=u.device)
+    _check(_lib.cuda().mx_rglru_scan(_p(gates), _p(bias), _p(coef), _p(u), u.stride(0), _p(y), y.stride(0), _p(state), _p(state_slots), _p(cu_q), _p(seq_lens),
+                                     _p(out), cu_q.numel() - 1, W, n, int(max_q_len), int(u.dtype == torch.float32), _stream()), "rglru_scan")
+    _count()
+    return out
+
+
+def rglru_step(x, y, conv_w, conv_b, w: QuantWeight, bias, coef, conv_state, state, state_slots, cu_q, seq_lens):
+    T, W = x.shape
+    n = w.K
+    assert w.fmt == WFormat.BF16 and (w.N, w.E) == (2 * n, W // n) and x.dtype == y.dtype == conv_state.dtype and x.stride(1) == y.stride(1) == 1
+    assert cu_q.numel() - 1 == T and state.dtype == torch.float32 and state.shape[1] == W and conv_state.shape[1:] == (conv_w.shape[1] - 1, W)
+    out = torch.empty(T, W, dtype=x.dtype, device=x.device)
+    _check(_lib.cuda().mx_rglru_step(_p(x), x.stride(0), _p(y), y.stride(0), _p(conv_w), _p(conv_b), _p(w.p0), _p(bias), _p(coef), _p(conv_state), _p(state),
+                                     _p(state_slots), _p(cu_q), _p(seq_lens), _p(out), T, W, n, conv_w.shape[1], int(x.dtype == torch.float32), _stream()),
+           "rglru_step")
+    _count()
+    return out
 
 
 def token_shift(x, mu, state, state_slots, cu_q, seq_lens, out_dtype=torch.bfloat16):
@@ -689,8 +758,29 @@ def _tc_prefill_takes(q, dk, dv, softcap, kv_scales) -> bool:
     return kv_scales is None and not softcap and 8 <= dk <= 256 and 8 <= dv <= 256 and dk % 8 == 0 and dv % 8 == 0
 
 
+def _takes_tc(max_q_len: int, bs: int, dtype, dk: int, dv: int) -> bool:
+    """Whether attention over pooled blocks runs on the tensor-core kernel."""
+    return max_q_len >= TC_PREFILL_MIN_Q and bs == 128 and dtype == torch.bfloat16 and 8 <= dk <= 256 and 8 <= dv <= 256
+
+
+def attention_prefill_pooled(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks, window, scale, softcap, gate, pools, dense, out_rope):
+    """tcgen05 FlashAttention over a window and the dense pages of pooled blocks that :func:`pool_blocks` has written (None: no query sees one)."""
+    Tq, n_q, dk = q.shape
+    n_pages, n_kv, bs, dv = v_cache.shape
+    cos, sin = out_rope if out_rope is not None else (None, None)
+    pk, pv = dense if dense is not None else (None, None)
+    out = torch.empty(Tq, n_q, dv, dtype=torch.bfloat16, device=q.device)
+    _check(_lib.cuda().mx_attention_prefill_pooled(_p(q), _q_rows(q), _p(k_cache), _p(v_cache), _p(block_table), _p(seq_lens), _p(cu_q), _p(sinks), _p(gate),
+                                                   0 if gate is None else gate.stride(0), _p(out), seq_lens.numel(), Tq, int(max_q_len), n_q, n_kv, dk, dv,
+                                                   block_table.shape[1], n_pages, bs, int(window), C.c_float(scale), C.c_float(softcap or 0.0), _p(pk), _p(pv),
+                                                   pools.pool if dense is not None else 0, 0 if pk is None else pk.shape[0] // seq_lens.numel(), _p(cos), _p(sin),
+                                                   0 if cos is None else cos.shape[0], 0 if cos is None else cos.shape[1], _stream()), "attention_prefill_pooled")
+    _count()
+    return out
+
+
 def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks=None, window=0, scale=None, softcap=0.0, n_splits=None,
-              kv_scales=None, max_kv_len=0, q_scale=None, gate=None, v_width=0, keep_first=0):
+              kv_scales=None, max_kv_len=0, q_scale=None, gate=None, v_width=0, keep_first=0, pools=None, pool_dense=None, out_rope=None):
     """``v_cache`` None: a value is the first ``v_width`` elements of its key row (latent cache)."""
     Tq, n_q, hd = q.shape
     n_kv, bs, dv = k_cache.shape[1], k_cache.shape[2], v_width if v_cache is None else v_cache.shape[3]
@@ -699,7 +789,13 @@ def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks
     B = seq_lens.numel()
     scale = scale if scale is not None else 1.0 / math.sqrt(hd)
     assert (k_cache.dtype == torch.int8) == (kv_scales is not None)
-    if max_q_len >= TC_PREFILL_MIN_Q and bs == 128 and n_splits is None and v_cache is not None and _tc_prefill_takes(q, hd, dv, softcap, kv_scales):
+    extended = pools is not None or out_rope is not None
+    if extended:
+        assert kv_scales is None and v_cache is not None and not keep_first and (gate is None or gate.shape[1] == n_q * dv)
+        if n_splits is None and q_scale is None and _takes_tc(max_q_len, bs, q.dtype, hd, dv):
+            return attention_prefill_pooled(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks, window, scale, softcap, gate, pools, pool_dense,
+                                            out_rope)
+    if not extended and max_q_len >= TC_PREFILL_MIN_Q and bs == 128 and n_splits is None and v_cache is not None and _tc_prefill_takes(q, hd, dv, softcap, kv_scales):
         if kv_scales is not None:       # the tensor-core kernel reads bf16 pages: expand this batch's pages first
             dk, dv, table = _dequant_pages(k_cache, v_cache, kv_scales, block_table, seq_lens, max_kv_len)
             return attention_prefill_tc(q, dk, dv, table, seq_lens, cu_q, max_q_len, sinks=sinks, window=window, scale=scale, softcap=softcap,
@@ -738,7 +834,10 @@ def attention(q, k_cache, v_cache, block_table, seq_lens, cu_q, max_q_len, sinks
                                             0 if gate is None else gate.stride(0), _p(q_scale), 0 if q_scale is None else q_scale.numel(), _p(out),
                                             _p(o_part), _p(ml_part), B, Tq, int(max_q_len), n_q, n_kv, hd, dv, block_table.shape[1], bs, int(window),
                                             int(keep_first), int(gate is not None and gate.shape[1] == n_q), C.c_float(scale), C.c_float(softcap), int(n_splits),
-                                            int(q.dtype == torch.float32), _stream()), "attention")
+                                            int(q.dtype == torch.float32), *((_vp(0), _vp(0), 0, 0) if pools is None else
+                                                                             (_p(pools.k), _p(pools.v), pools.pool, pools.k.shape[2])),
+                                            *((_vp(0), _vp(0), 0, 0) if out_rope is None else (_p(out_rope[0]), _p(out_rope[1]), *out_rope[0].shape)),
+                                            _stream()), "attention")
     _count(_lib.cuda().mx_attention_launches(B, int(max_q_len), n_q, n_kv))
     return out
 
@@ -759,21 +858,22 @@ LATENT_MAX_SPLITS = 64
 HEAD_GEMV_MAX_T = 4          # up to this many rows a head's matrix is streamed by the CUDA cores; more go to the tensor cores
 
 
-def head_linear(x, w: QuantWeight, gate=None, out=None):
+def head_linear(x, w: QuantWeight, gate=None, out=None, out_f32=False):
     T, H, K = x.shape
     assert w.fmt == WFormat.BF16 and (w.E, w.K) == (H, K) and x.stride(2) == 1
+    odt = torch.float32 if out_f32 else x.dtype
     if out is None:
-        out = torch.empty(T, H, w.N, dtype=x.dtype, device=x.device)
-    assert out.shape == (T, H, w.N) and out.dtype == x.dtype and out.stride(2) == 1 and (gate is None or (gate.dtype == x.dtype and gate.stride(1) == 1))
+        out = torch.empty(T, H, w.N, dtype=odt, device=x.device)
+    assert out.shape == (T, H, w.N) and out.dtype == odt and out.stride(2) == 1 and (gate is None or (gate.dtype == x.dtype and gate.stride(1) == 1))
     g_ld = 0 if gate is None else gate.stride(0)
     if x.dtype == torch.float32 or T <= HEAD_GEMV_MAX_T:
         _check(_lib.cuda().mx_head_linear(_p(x), C.c_longlong(x.stride(0)), x.stride(1), _p(w.p0), _p(gate), g_ld, _p(out), C.c_longlong(out.stride(0)),
-                                          out.stride(1), T, H, w.N, K, int(x.dtype == torch.float32), _stream()), "head_linear")
+                                          out.stride(1), T, H, w.N, K, int(x.dtype == torch.float32), int(odt == torch.float32), _stream()), "head_linear")
     else:
         tiles = H * ((T + 127) // 128)
         bn = next((b for b in (128, 64, 32) if tiles * ((w.N + b - 1) // b) >= sm_count()), 32)
         _check(_lib.cuda().mx_gemm_heads(_p(x), x.stride(0), C.c_longlong(x.stride(1)), _p(w.p0), _p(out), out.stride(0), C.c_longlong(out.stride(1)), _p(gate),
-                                         g_ld, T, H, w.N, K, bn, _stream()), "gemm_heads")
+                                         g_ld, T, H, w.N, K, bn, int(out_f32), _stream()), "gemm_heads")
     _count()
     return out
 
@@ -796,7 +896,7 @@ def stacked_linear(x, w: QuantWeight):
         return expert_gemv(x.view(n * T, K), w, _stack_slots[n, T, x.device]).view(n, T, w.N)
     out = torch.empty(n, T, w.N, dtype=x.dtype, device=x.device)
     _check(_lib.cuda().mx_gemm_heads(_p(x), K, C.c_longlong(T * K), _p(w.p0), _p(out), w.N, C.c_longlong(T * w.N), _vp(0), 0, T, n, w.N, K,
-                                     _stack_bn(n, T, w.N), _stream()), "gemm_heads")
+                                     _stack_bn(n, T, w.N), 0, _stream()), "gemm_heads")
     _count()
     return out
 
@@ -887,11 +987,13 @@ def expanded_attention(q, kv, plan, cache, block_table, seq_lens, cu_q, max_q_le
 
 
 # ------------------------------------------------------------------ MoE
-def moe_route(logits, bias, k, renorm=True, precise=False, sigmoid=False):
-    T, E = logits.shape
+def moe_route(logits, bias, k, renorm=True, precise=False, sigmoid=False, experts=None):
+    T, ld = logits.shape
+    E = experts or ld
+    assert logits.is_contiguous() and logits.dtype == torch.float32
     idx = torch.empty(T, k, dtype=torch.int32, device=logits.device)
     w = torch.empty(T, k, dtype=torch.float32, device=logits.device)
-    _check(_lib.cuda().mx_moe_route(_p(logits), _p(bias), T, E, k, 2 if sigmoid else int(renorm), int(precise), _p(idx), _p(w), _stream()), "moe_route")
+    _check(_lib.cuda().mx_moe_route(_p(logits), _p(bias), T, E, k, 2 if sigmoid else int(renorm), int(precise), ld, _p(idx), _p(w), _stream()), "moe_route")
     _count()
     return idx, w
 

@@ -190,3 +190,132 @@ def greedy(cfg, weights, prompt, n):
     for _ in range(n):
         toks.append(int(np.argmax(forward(cfg, weights, toks)[-1])))
     return toks[len(prompt):]
+
+
+# ------------------------------------------------------------------ small configurations with random weights
+def feed_forward(mlp):
+    """None, or (experts, top, expert width, limit, width of the shared expert or 0, its limit)."""
+    if mlp is None:
+        return None
+    experts, top, ff, limit, shared, shared_limit = mlp
+    f = {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "router": {"experts": experts, "top": top}}
+    return {**f, "shared": {"ff": shared, "limit": shared_limit}} if shared else f
+
+
+def attention_layer(mlp, heads, kv_heads, dim, vdim, window, pool, rot_dims, base=10000.0, cap=30.0, scale=None):
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "rot": {"base": base, "dims": rot_dims}, "scale": scale or 1.0 / math.sqrt(dim)}
+    if cap:
+        m["softcap"] = cap
+    if window:
+        m["mask"] = {"size": window, "pool": pool} if pool else {"size": window}
+    return {"type": "attention", "mlp": feed_forward(mlp), "mixer": m}
+
+
+def rglru_layer(mlp, width, blocks, taps):
+    return {"type": "rglru", "mlp": feed_forward(mlp), "mixer": {"width": width, "blocks": blocks, "conv": taps}}
+
+
+def random_config(layers, vocab=96, width=64, eps=1e-6, scale=3.0, logit_scale=1.0, loop=None):
+    c = {"architecture": "Zegelix", "embedding": {"scale": scale}, "layers": layers, "logit_scale": logit_scale, "norm": {"eps": eps}, "vocab": vocab, "width": width}
+    if loop:
+        c["loop"] = dict(zip(("start", "stop", "times"), loop))
+    return c
+
+
+def round_bf16(a):
+    """float array -> float32 values that bfloat16 represents (round to nearest even)."""
+    u = np.array(a, dtype=np.float32, order="C").view(np.uint32).astype(np.uint64)
+    u = ((u + 0x7FFF + ((u >> 16) & 1)) >> 16 << 16).astype(np.uint32)
+    return u.view(np.float32)
+
+
+CODES = 8            # columns that hold a code of the token and that no layer writes to, read by the routers alone
+
+
+def random_weights(cfg, seed=0):
+    """Every tensor the configuration asks for, as float32 arrays that hold bfloat16 values.  The routers read a code of the token, so that no choice of
+    experts is within rounding of another."""
+    g = np.random.default_rng(seed)
+    H, W = cfg["width"], {}
+
+    def mat(name, n, k, gain=1.0):
+        W[name] = round_bf16(g.standard_normal((n, k)) * gain / math.sqrt(k))
+
+    def vec(name, n, mean=0.0, std=0.2):
+        W[name] = round_bf16(mean + std * g.standard_normal(n))
+
+    def gated(name, f):
+        for n, shape in (("gate", (f, H)), ("up", (f, H)), ("down", (H, f))):
+            mat(f"{name}.{n}", *shape)
+
+    W["embed"] = round_bf16(g.standard_normal((cfg["vocab"], H)) / cfg["embedding"]["scale"])
+    vec("final.norm", H, 1.0)
+    if cfg.get("loop"):
+        mat("loop.in", H, 2 * H)
+    for i, layer in enumerate(cfg["layers"]):
+        l, p, m, f = f"l{i}", f"l{i}.mix", layer["mixer"], layer["mlp"]
+        vec(f"{l}.norm1", H, 1.0)
+        if layer["type"] == "attention":
+            for n, rows in (("q", m["heads"] * m["dim"]), ("k", m["kv_heads"] * m["dim"]), ("v", m["kv_heads"] * m["vdim"])):
+                mat(f"{p}.{n}", rows, H, 1.5)
+                vec(f"{p}.{n}.b", rows, 0.0, 0.5)
+            vec(f"{p}.temp", m["heads"], 1.2, 0.4)
+            vec(f"{p}.sink", m["heads"], 0.5, 1.0)
+            mat(f"{p}.g", m["heads"] * m["vdim"], H)
+            mat(f"{p}.o", H, m["heads"] * m["vdim"], 2.0)
+        else:
+            w, b = m["width"], m["blocks"]
+            for n in "yx":
+                mat(f"{p}.{n}", w, H, 1.3)
+                vec(f"{p}.{n}.b", w, 0.0, 0.4)
+            W[f"{p}.conv"] = round_bf16(g.standard_normal((w, m["conv"])) / math.sqrt(m["conv"]))
+            vec(f"{p}.conv.b", w)
+            for n in ("ra", "ri"):
+                W[f"{p}.{n}"] = round_bf16(g.standard_normal((b, w // b, w // b)) / math.sqrt(w // b))
+                W[f"{p}.{n}.b"] = round_bf16(0.5 * g.standard_normal((b, w // b)))
+            W[f"{p}.lam"] = round_bf16(g.uniform(-7.0, 1.0, w))          # from memories of hundreds of tokens to almost none
+            mat(f"{p}.o", H, w, 1.5)
+        if f is None:
+            continue
+        vec(f"{l}.norm2", H, 1.0)
+        mat(f"{l}.mlp.router", f["router"]["experts"], H)
+        vec(f"{l}.mlp.router.b", f["router"]["experts"], 0.0, 0.1)
+        for e in range(f["router"]["experts"]):
+            gated(f"{l}.mlp.e{e}", f["expert"]["ff"])
+        if f.get("shared"):
+            gated(f"{l}.mlp.shared", f["shared"]["ff"])
+            mat(f"{l}.mlp.shared.sg", 1, H)
+    _settle_routing(cfg, W, g)
+    return W
+
+
+def _settle_routing(cfg, W, g, gap=0.1):
+    moe = [(i, layer["mlp"]["router"]) for i, layer in enumerate(cfg["layers"]) if layer["mlp"] is not None]
+    if not moe:
+        return
+    for n in W:                                          # no branch writes to the code's columns, a pass of the loop hands them on
+        if n.endswith(".mix.o") or n.endswith(".down"):
+            W[n][:CODES] = 0.0
+    if cfg.get("loop"):
+        W["loop.in"][:CODES] = 0.0
+        W["loop.in"][:CODES, :CODES] = np.eye(CODES)
+    scale = cfg["embedding"]["scale"]
+    for i, r in moe:
+        z = g.standard_normal((r["experts"], CODES)) * 0.5
+        W[f"l{i}.mlp.router"] = round_bf16(np.pad(z, ((0, 0), (0, cfg["width"] - CODES))))
+        W[f"l{i}.norm2"][:CODES] = 1.0
+    for t in range(cfg["vocab"]):
+        for _ in range(3000):
+            code = round_bf16(2.0 * g.choice([-1.0, 1.0], CODES) / scale)
+            gaps = [np.inf]
+            for i, r in moe:
+                for rms in (0.7, 1.0, 1.5, 2.5, 4.0):            # what the norm in front of the router may divide by
+                    z = np.float64(W[f"l{i}.mlp.router"])[:, :CODES] @ (np.float64(code) * scale) / rms + W[f"l{i}.mlp.router.b"]
+                    z = np.sort(z)[::-1]
+                    if r["top"] < len(z):
+                        gaps.append(z[r["top"] - 1] - z[r["top"]])
+            if min(gaps) > gap:
+                break
+        else:
+            raise ValueError("no code of this token settles its routing")
+        W["embed"][t, :CODES] = code
