@@ -257,12 +257,12 @@ def random_weights(cfg, seed=0):
         vec(f"{l}.norm1", H, 1.0)
         if layer["type"] == "attention":
             for n, rows in (("q", m["heads"] * m["dim"]), ("k", m["kv_heads"] * m["dim"]), ("v", m["kv_heads"] * m["vdim"])):
-                mat(f"{p}.{n}", rows, H, 1.5)
+                mat(f"{p}.{n}", rows, H)
                 vec(f"{p}.{n}.b", rows, 0.0, 0.5)
             vec(f"{p}.temp", m["heads"], 1.2, 0.4)
             vec(f"{p}.sink", m["heads"], 0.5, 1.0)
             mat(f"{p}.g", m["heads"] * m["vdim"], H)
-            mat(f"{p}.o", H, m["heads"] * m["vdim"], 2.0)
+            mat(f"{p}.o", H, m["heads"] * m["vdim"], 1.2)
         else:
             w, b = m["width"], m["blocks"]
             for n in "yx":
