@@ -109,7 +109,7 @@ def main():
                     help="library baseline arm: the same model graph with plain PyTorch ops (cuBLAS bf16 GEMMs on decoded weights, ATen kernels) "
                          "and NCCL all-reduce; no kernel of this engine runs")
     ap.add_argument("--replicated", action="store_true", help="keep the activations replicated on every rank (fused all-reduce) instead of the row-sharded prefill")
-    ap.add_argument("--design", default=None, choices=["tikarax", "pubodra", "beputar"], help="instead of the headline: throughput of this design beside the closest models, and its kernels")
+    ap.add_argument("--design", default=None, choices=["tikarax", "pubodra", "beputar", "zegelix"], help="instead of the headline: throughput of this design beside the closest models, and its kernels")
     ap.add_argument("--design-part", default="all", choices=["all", "models", "kernels"])
     args = ap.parse_args()
     if args.impl == "reference":

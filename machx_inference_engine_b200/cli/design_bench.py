@@ -1,6 +1,6 @@
 """Throughput of a layer-list design beside the framework's closest models at equal size, and its kernels beside the like kernels.
 
-    python bench.py --design tikarax|pubodra|beputar [--design-part models|kernels|all]
+    python bench.py --design tikarax|pubodra|beputar|zegelix [--design-part models|kernels|all]
 
 Models (random-init bf16 weights, random tokens): prefill of one 4096-token prompt and decode at a 2048-token context for 1, 8 and 32
 sequences, through ``LLMEngine`` (CUDA graphs as in serving), for
@@ -10,6 +10,8 @@ sequences, through ``LLMEngine`` (CUDA graphs as in serving), for
             heads, sliding window and parameters per layer; a qwen3moe with the same experts (gated, 2/3 the width) in every layer
   beputar:  the design (parallel, attention and wkv layers in turn) with dense feed-forwards, and with experts in every layer but the first; the DeltaNet
             hybrids of the same width, heads and parameters per feed-forward (qwen35: gated, 2/3 the width; qwen35moe: the same experts and shared expert)
+  zegelix:  the design (one attention layer in three, RG-LRU otherwise, experts and a shared one in every layer), and with its middle third run twice; the
+            DeltaNet hybrid of the same width, heads, experts and shared expert (qwen35moe); Beputar with the same experts
 Weights are larger than L2 (126 MB), so every pass streams them.
 
 Kernels: device time inside a CUDA graph over buffers that together exceed L2, as a fraction of the roofline (bytes over the measured copy
@@ -24,7 +26,7 @@ import time
 
 import torch
 
-from ..formats.model_config import ModelConfig, _beputar_preset, _pubodra_preset, _tikarax_preset
+from ..formats.model_config import ModelConfig, _beputar_preset, _pubodra_preset, _tikarax_preset, _zegelix_preset
 
 LAYERS = 8
 SIZES = {"tikarax": {  # hidden, heads, kv_heads, head width, un-gated feed-forward, minGRU width
@@ -36,6 +38,11 @@ SIZES = {"tikarax": {  # hidden, heads, kv_heads, head width, un-gated feed-forw
 }, "beputar": {       # hidden, heads, kv_heads, head width, window, kept first; lightning heads of 128, wkv heads of 64; un-gated feed-forward; experts ...
     "1b-layers": dict(layers=9, hidden=2048, heads=32, kv_heads=8, dim=64, window=1024, keep=16, lin=16, wkv=32, ffn=12288, experts=64, used=6, eff=1024, shared=2048),
     "8b-layers": dict(layers=9, hidden=4096, heads=32, kv_heads=8, dim=128, window=4096, keep=16, lin=32, wkv=64, ffn=21504, experts=64, used=6, eff=1536, shared=3072),
+}, "zegelix": {       # hidden, heads, kv_heads, head width, rotated, window, tokens per pooled block; RG-LRU width, blocks, taps; experts, per token, widths
+    "1b-layers": dict(layers=9, hidden=2048, heads=32, kv_heads=8, dim=64, rot=32, window=1024, pool=16, width=2560, blocks=10, conv=4, experts=64, used=6, eff=1024,
+                      shared=2048),
+    "8b-layers": dict(layers=9, hidden=4096, heads=32, kv_heads=8, dim=128, rot=64, window=2048, pool=16, width=4096, blocks=16, conv=4, experts=64, used=6, eff=1536,
+                      shared=3072),
 }}
 VOCAB = 32768
 PREFILL, CONTEXT, DECODE = 4096, 2048, 64
@@ -71,6 +78,20 @@ def _beputar_configs(s: dict) -> dict:
             "qwen35moe hybrid": ModelConfig(arch="qwen35moe", n_experts=s["experts"], n_experts_used=s["used"], expert_ffn=s["eff"], shared_expert_ffn=s["shared"], **common)}
 
 
+def _zegelix_configs(s: dict) -> dict:
+    zx = lambda loop: _zegelix_preset(s["hidden"], s["layers"], s["heads"], s["kv_heads"], s["dim"], s["dim"], s["rot"], s["window"], s["pool"], 50.0, s["width"],
+                                      s["blocks"], s["conv"], s["experts"], s["used"], s["eff"], s["shared"], VOCAB, loop=loop)
+    moe = dict(n_experts=s["experts"], n_experts_used=s["used"], expert_ffn=s["eff"], shared_expert_ffn=s["shared"])
+    lin = s["hidden"] // 128
+    third = s["layers"] // 3
+    return {"zegelix": zx(None), "zegelix, middle third twice": zx((third, 2 * third, 2)),
+            "qwen35moe hybrid": ModelConfig(arch="qwen35moe", n_layers=s["layers"], hidden=s["hidden"], n_heads=s["heads"], n_kv_heads=s["kv_heads"], ffn=s["eff"],
+                                            vocab=VOCAB, ctx_train=16384, head_dim=s["dim"], n_rot=s["rot"], full_attn_interval=3, ssm_inner=lin * 128, ssm_state=128,
+                                            ssm_n_k_heads=lin // 2, ssm_n_v_heads=lin, ssm_conv_kernel=4, **moe),
+            "beputar, experts": _beputar_preset(s["hidden"], s["layers"], s["heads"], s["kv_heads"], s["dim"], s["window"], 16, lin, 128, 128, s["hidden"] // 64, 64, 64,
+                                                6 * s["eff"], VOCAB, s["experts"], s["used"], s["eff"], s["shared"])}
+
+
 def _timed(fn) -> float:
     e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
     torch.cuda.synchronize()
@@ -86,7 +107,7 @@ def bench_models(design, dev, emit) -> None:
     from ..ops import cuda as K
     from ..runtime.engine import EngineOptions, LLMEngine, SamplingParams
     for size, s in SIZES[design].items():
-        for name, cfg in {"tikarax": _tikarax_configs, "pubodra": _pubodra_configs, "beputar": _beputar_configs}[design](s).items():
+        for name, cfg in {"tikarax": _tikarax_configs, "pubodra": _pubodra_configs, "beputar": _beputar_configs, "zegelix": _zegelix_configs}[design](s).items():
             model = build_model(cfg, dev, quant="bf16", max_ctx=PREFILL + 256)
             row = {"size": size, "model": name, "layers": cfg.n_layers, "weight_gb": round(model.weight_bytes() / 1e9, 2)}
             g = torch.Generator().manual_seed(0)
@@ -490,6 +511,137 @@ def bench_kernels_beputar(dev, emit) -> None:
     K.check_status()
 
 
+def bench_kernels_zegelix(dev, emit) -> None:
+    from ..models.transformer import KVCache
+    from ..ops import cuda as K
+    from ..ops import ref
+    from ..ops.weights import QuantWeight, WFormat
+    from ..utils.rope import rope_tables
+    t = _Rows(dev, emit)
+    bf, i32, bufs, row = t.bf, t.i32, t.bufs, t.row
+    mats = lambda n, k, e=1: [QuantWeight(WFormat.BF16, n, k, e, (torch.randn(e, n, k, device=dev) * k ** -0.5).to(torch.bfloat16)) for _ in range(bufs(e * n * k * 2))]
+    f32 = lambda *sh: torch.randn(*sh, device=dev)
+    for size, s in SIZES["zegelix"].items():
+        H, nq, nkv, d, rot, win, pool, W, blocks = (s[k] for k in ("hidden", "heads", "kv_heads", "dim", "rot", "window", "pool", "width", "blocks"))
+        E, top, ef, n_blk = s["experts"], s["used"], s["eff"], s["width"] // s["blocks"]
+        for T in (1, 32, PREFILL):
+            # ---- residual add + norm
+            nb = bufs(T * H * 12) if T > 64 else 8
+            xs, ds, w = [f32(T, H) for _ in range(nb)], [bf(T, H) for _ in range(nb)], torch.ones(H, device=dev)
+            by = T * H * (4 + 4 + 2 + 2)
+            row(f"sublayer_norm (add + norm) T={T} H={H}", "new", [lambda x=x, q=q: K.sublayer_norm(x, q, None, 1e-6, w=w) for x, q in zip(xs, ds)], by)
+            row(f"rmsnorm (add + norm) T={T} H={H}", "like", [lambda x=x, q=q: K.rmsnorm(x, w, 1e-6, delta=q) for x, q in zip(xs, ds)], by)
+            ys, pos, cw, z = [bf(T * top, H) for _ in range(nb)], torch.randperm(T * top, device=dev).to(torch.int32), torch.rand(T, top, device=dev), f32(T, E + 8)
+            by = T * H * (4 + 4 + 2 + 2 * top)
+            row(f"sublayer_norm of {top} weighted experts + gated shared T={T} H={H}", "new",
+                [lambda x=x, y=y, q=q: K.sublayer_norm(x, ref.ExpertSum(y, pos, top, q, cw, z[:, E]), None, 1e-6, w=w) for x, y, q in zip(xs, ys, ds)], by + T * H * 2)
+            row(f"rmsnorm_combine of {top} T={T} H={H}", "like", [lambda x=x, y=y: K.rmsnorm_combine(x, w, 1e-6, K.CombineDelta(y, pos, cw)) for x, y in zip(xs, ys)], by)
+            del ds, ys
+            # ---- experts
+            h, idx = bf(T, H), torch.stack([torch.randperm(E, device=dev)[:top] for _ in range(T)]).to(torch.int32)
+            row(f"moe_route over {E} of {E + 8} columns T={T}", "new", [lambda: K.moe_route(z, None, top, experts=E)], T * (E + 2 * top) * 4)
+            z2 = f32(T, E)
+            row(f"moe_route T={T} {top} of {E}", "like", [lambda: K.moe_route(z2, None, top)], T * (E + 2 * top) * 4)
+            gu = mats(2 * ef, H, E)
+            live = min(E, T * top)
+            by, fl = live * 2 * ef * H * 2 + T * top * (H + ef) * 2, 4.0 * T * top * ef * H
+            for name, role, act in (("clamped SwiGLU", "new", ref.ACT_SWIGLU_OAI), ("SwiGLU", "like", ref.ACT_SWIGLU)):
+                if T <= 4:
+                    row(f"expert slots + {name} T={T}", role, [lambda m=m: K.expert_gemv(h, m, idx.reshape(-1), x_div=top, act=act, act_limit=5.0) for m in gu], by, fl)
+                else:
+                    pk = K.moe_pack(idx, E)
+                    xp = K.moe_gather(h, pk)
+                    row(f"grouped experts + {name} T={T}", role, [lambda m=m: K.grouped_linear(xp, m, pk.tile_expert, pk.num_tiles, act=act, act_limit=5.0) for m in gu], by, fl)
+            del gu
+            # ---- head epilogue
+            kr, vr, full = rope_tables(2 * PREFILL, rot, 1e4, device=dev), rope_tables(2 * PREFILL, d, 1e4, device=dev), rope_tables(2 * PREFILL, d, 1e4, device=dev)
+            pages, bs = T // 128 + 2, 128
+            slots, pos1, temp = torch.arange(128, 128 + T, dtype=torch.int64, device=dev), torch.arange(T, dtype=torch.int32, device=dev), torch.ones(nq, device=dev)
+            kc, vc = torch.zeros(pages, nkv, bs, d, dtype=torch.bfloat16, device=dev), torch.zeros(pages, nkv, bs, d, dtype=torch.bfloat16, device=dev)
+            C = (nq + 2 * nkv) * d
+            ys = [bf(T, C) for _ in range(min(8, bufs(T * nq * d * 4) if T > 64 else 8))]
+            cut = lambda y, a, n: y[:, a * d:(a + n) * d].view(T, n, d)
+            by = T * (nq * d * 4 + nkv * d * 8)
+            row(f"qk_post with rotated values T={T}", "new",
+                [lambda y=y: K.qk_post(cut(y, 0, nq), cut(y, nq, nkv), pos1, *kr, slots, kc, vc, d, rot, interleaved=True, v=cut(y, nq + nkv, nkv), v_rope=vr, q_scale=temp)
+                 for y in ys], by)
+            row(f"qkv_post T={T}", "like", [lambda y=y: K.qkv_post(y, None, None, None, pos1, *full, slots, kc, vc, nq, nkv, d, d) for y in ys], by)
+            del ys, kc, vc
+        # ---- recurrence and what is around it
+        for B, n in ((1, PREFILL), (8, 512), (1, 1), (8, 1), (32, 1)):
+            T = B * n
+            slots, cu, sl = i32(list(range(B))), i32([i * n for i in range(B + 1)]), i32([n + 64] * B)
+            nb = bufs(T * W * 8) if T > 64 else 8
+            ps, cwt, cb = [bf(T, 2 * W) for _ in range(nb)], f32(W, 4), f32(W)
+            cst, S, gb, coef = torch.zeros(B, 3, W, dtype=torch.bfloat16, device=dev), torch.zeros(B, W, device=dev), f32(blocks, 2 * n_blk), -torch.rand(W, device=dev)
+            gm = mats(2 * n_blk, n_blk, blocks)
+            if n > 1:
+                row(f"causal_conv B={B} n={n} C={W}", "new", [lambda p=p: K.causal_conv(p[:, :W], cwt, cb, cst, slots, cu, sl, n) for p in ps], T * W * 4 + B * W * 12)
+                row(f"conv1d_silu B={B} n={n} C={W}", "like", [lambda p=p: K.conv1d_silu(p[:, :W], cwt, cst, slots, cu, n) for p in ps], T * W * 4 + B * W * 12)
+                us = [bf(T, W) for _ in range(nb)]
+                row(f"gate products per block T={T} {blocks} x {2 * n_blk}x{n_blk}, fp32 results", "new",
+                    [lambda u=u: K.head_linear(u.view(T, blocks, n_blk), gm[0], out_f32=True) for u in us], T * W * (2 + 8) + gm[0].nbytes, 4.0 * T * W * n_blk)
+                row(f"gate products per block T={T}, 16-bit results", "like",
+                    [lambda u=u: K.head_linear(u.view(T, blocks, n_blk), gm[0]) for u in us], T * W * (2 + 4) + gm[0].nbytes, 4.0 * T * W * n_blk)
+                gs = [f32(T, blocks, 2 * n_blk) for _ in range(nb)]
+                row(f"rglru_scan B={B} n={n} W={W}", "new",
+                    [lambda g=g, u=u, p=p: K.rglru_scan(g, u, p[:, W:], gb, coef, S, slots, cu, sl, n) for g, u, p in zip(gs, us, ps)], T * W * (8 + 6) + B * W * 8)
+                del gs, us
+            else:
+                row(f"rglru_step (conv, gates, recurrence) B={B} W={W}", "new",
+                    [lambda p=p, m=m: K.rglru_step(p[:, :W], p[:, W:], cwt, cb, m, gb, coef, cst, S, slots, cu, sl) for p, m in zip(ps * (len(gm) // len(ps) + 1), gm)],
+                    gm[0].nbytes + B * W * (6 + 8 + 12))
+                pl = mats(2 * n_blk * blocks // 8, n_blk * 8)
+                h = bf(T, n_blk * 8)
+                row(f"plain projection with as many weights T={T}", "like", [lambda m=m: K.linear(h, m) for m in pl], pl[0].nbytes)
+                row(f"conv1d_silu B={B} n={n} C={W}", "like", [lambda p=p: K.conv1d_silu(p[:, :W], cwt, cst, slots, cu, n) for p in ps], T * W * 4 + B * W * 12)
+                del pl
+            y3, zb = [bf(T, 3 * W) for _ in range(nb)], torch.zeros(W, device=dev)
+            row(f"mingru_scan B={B} n={n} W={W}", "like",
+                [lambda y=y: K.mingru_scan(y[:, :W], y[:, W:2 * W], y[:, 2 * W:], zb, zb, S, slots, cu, sl, n) for y in y3], T * W * 8 + B * W * 8)
+            del ps, y3, gm
+            torch.cuda.empty_cache()
+        # ---- attention
+        for B, n, ctx in ((1, PREFILL, PREFILL), (1, 512, PREFILL), (1, PREFILL, 4 * PREFILL), (1, 1, 8192), (1, 1, 2048), (32, 1, 2048), (32, 1, 8192)):
+            T, nblk = B * n, (ctx + 127) // 128
+            pages, blk_seen = B * nblk + 1, max(ctx - win, 0) // pool
+            live = min(ctx, win + n) + blk_seen
+            nb = min(16, bufs(B * live * nkv * d * 4)) if n == 1 else 2
+            kvs = [KVCache(1, pages, nkv, d, dev, [0], pools={0: (pool, win)}) for _ in range(nb)]
+            for kv in kvs:
+                for x in (kv.k[0], kv.v[0], kv.pools[0].k, kv.pools[0].v):
+                    x.normal_(0.0, 0.5)
+            bt = torch.arange(1, pages, dtype=torch.int32, device=dev).reshape(B, nblk)
+            sl, cu = i32([ctx] * B), i32([i * n for i in range(B + 1)])
+            q, g, sink, turn = bf(T, nq, d), bf(T, nq * d), torch.zeros(nq, device=dev), rope_tables(ctx, d, 1e4, device=dev)
+            pairs = float(sum(min(p + 1, win) + max(p + 1 - win, 0) // pool for p in range(ctx - n, ctx)))
+            plain = float(sum(min(p + 1, win) for p in range(ctx - n, ctx)))
+            by = lambda keys, gated: B * keys * nkv * d * 4 + T * nq * d * (6 if gated else 4)
+            kw = dict(window=win, scale=d ** -0.5, max_kv_len=ctx)
+            name = f"B={B} n={n} ctx={ctx} window={win} {nq}/{nkv}x{d}"
+            if n > 1:
+                form = lambda kv: K.pool_blocks(kv.k[0], kv.v[0], kv.pools[0], bt, sl, cu, n, max_kv_len=ctx)
+                row(f"pool_blocks {name}", "new", [lambda kv=kv: form(kv) for kv in kvs], (min(ctx, win + n) - win + 2 * blk_seen) * nkv * d * 4)
+                src = bf(T, 2 * nkv * d)
+                at = torch.arange(128, 128 + T, dtype=torch.int64, device=dev)
+                row(f"kv_store T={T}", "like", [lambda kv=kv: K.kv_store(src[:, :nkv * d], src[:, nkv * d:], at, kv.k[0], kv.v[0]) for kv in kvs], T * nkv * d * 8)
+                dense = [form(kv) for kv in kvs]
+            else:
+                dense = [None] * nb
+            for cap in (50.0, 0.0):
+                row(f"attention + pooled blocks + cap {cap:g} + sink + gate + turn {name}", "new",
+                    [lambda kv=kv, x=x: K.attention(q, kv.k[0], kv.v[0], bt, sl, cu, n, sinks=sink, softcap=cap, gate=g, pools=kv.pools[0], pool_dense=x, out_rope=turn, **kw)
+                     for kv, x in zip(kvs, dense)], by(live, True), 4.0 * B * nq * d * pairs)
+            if d in (64, 128, 256):
+                row(f"attention + cap 50 {name}", "like", [lambda kv=kv: K.attention(q, kv.k[0], kv.v[0], bt, sl, cu, n, softcap=50.0, **kw) for kv in kvs],
+                    by(min(ctx, win + n), False), 4.0 * B * nq * d * plain)
+            row(f"attention {name}", "like", [lambda kv=kv: K.attention(q, kv.k[0], kv.v[0], bt, sl, cu, n, **kw) for kv in kvs], by(min(ctx, win + n), False),
+                4.0 * B * nq * d * plain)
+            del kvs, dense
+            torch.cuda.empty_cache()
+    K.check_status()
+
+
 def main(design: str, part: str = "all") -> int:
     dev = torch.device("cuda:0")
     torch.cuda.set_device(dev)
@@ -501,6 +653,6 @@ def main(design: str, part: str = "all") -> int:
     if part in ("all", "models"):
         bench_models(design, dev, emit)
     if part in ("all", "kernels"):
-        {"tikarax": bench_kernels_tikarax, "pubodra": bench_kernels_pubodra, "beputar": bench_kernels_beputar}[design](dev, emit)
+        {"tikarax": bench_kernels_tikarax, "pubodra": bench_kernels_pubodra, "beputar": bench_kernels_beputar, "zegelix": bench_kernels_zegelix}[design](dev, emit)
     emit({"design_bench": "done", "seconds": round(time.time() - t0, 1)})
     return 0

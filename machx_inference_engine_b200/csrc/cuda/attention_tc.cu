@@ -99,33 +99,66 @@ __device__ __forceinline__ float ex2_fast(float x) {
   return y;
 }
 
-// cap * tanh(x / cap) over a run of raw scores, without the hardware's 11-bit tanh: its power series where all of the run is small (error below 1e-6 of
-// the argument for |y| <= 1/2), otherwise 1 - 2 / (1 + e^2y).  in: factor to y = x / cap; out_c: factor on the result.
+// two fp32 operations in one instruction
+__device__ __forceinline__ uint64_t pack2(float a, float b) {
+  uint64_t d;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(a), "f"(b));
+  return d;
+}
+__device__ __forceinline__ void unpack2(uint64_t d, float& a, float& b) { asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(d)); }
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t d;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
+  return d;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t d;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
+  return d;
+}
+
+// v x P(v^2) over a run, P of degree D with the coefficients c (of rising powers)
+template <int D, int N>
+__device__ __forceinline__ void odd_series_run(float (&v)[N], const float (&c)[D + 1]) {
+  uint64_t k[D + 1];
+#pragma unroll
+  for (int d = 0; d <= D; ++d) k[d] = pack2(c[d], c[d]);
+#pragma unroll
+  for (int i = 0; i < N; i += 2) {
+    const uint64_t x = pack2(v[i], v[i + 1]), w = mul2(x, x);
+    uint64_t t = k[D];
+#pragma unroll
+    for (int d = D - 1; d >= 0; --d) t = fma2(w, t, k[d]);
+    unpack2(mul2(x, t), v[i], v[i + 1]);
+  }
+}
+
+// cap * tanh(x / cap) over a run of raw scores, without the hardware's 11-bit tanh: the power series of tanh y where all of the run is small
+//     y (1 - z / 3 + 2 z^2 / 15 - 17 z^3 / 315 + 62 z^4 / 2835 - 1382 z^5 / 155925 + 21844 z^6 / 6081075 - ...), z = y^2
+// (three terms up to |y| = 1/8, seven up to 1/2: relative error below 1e-6), otherwise 1 - 2 / (1 + e^2y).  in: factor to y = x / cap; out_c: factor on the
+// result.
 template <int N>
 __device__ __forceinline__ void softcap_run(float (&v)[N], float in, float out_c) {
   float big = 0.f;
 #pragma unroll
-  for (int i = 0; i < N; ++i) big = fmaxf(big, fabsf(v[i]));
-  if (__any_sync(0xffffffffu, big * fabsf(in) > 0.5f)) {
+  for (int i = 0; i < N; i += 2) big = fmaxf(fmaxf(big, fabsf(v[i])), fabsf(v[i + 1]));
+  big *= fabsf(in);
+  const float s = in * in, lin = in * out_c;
+  if (!__any_sync(0xffffffffu, big > 0.125f)) {
+    const float c[3] = {lin, lin * s * -3.3333333e-1f, lin * s * s * 1.3333333e-1f};
+    odd_series_run<2>(v, c);
+  } else if (!__any_sync(0xffffffffu, big > 0.5f)) {
+    const float s2 = s * s, s3 = s2 * s;
+    const float c[7] = {lin, lin * s * -3.3333333e-1f, lin * s2 * 1.3333333e-1f, lin * s3 * -5.3968254e-2f, lin * s2 * s2 * 2.1869489e-2f,
+                        lin * s2 * s3 * -8.8632355e-3f, lin * s3 * s3 * 3.5921280e-3f};
+    odd_series_run<6>(v, c);
+  } else {
     const float in2 = in * 2.8853900817779268f;        // 2 / ln 2
 #pragma unroll
     for (int i = 0; i < N; ++i) {
       float r;
       asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + ex2_fast(v[i] * in2)));
       v[i] = fmaf(-2.f * out_c, r, out_c);
-    }
-  } else {
-    // tanh y = y (1 - z / 3 + 2 z^2 / 15 - 17 z^3 / 315 + 62 z^4 / 2835 - 1382 z^5 / 155925 + 21844 z^6 / 6081075 - ...), z = y^2
-    const float in_sq = in * in, lin = in * out_c;
-#pragma unroll
-    for (int i = 0; i < N; ++i) {
-      const float z = v[i] * v[i] * in_sq;
-      float t = fmaf(z, 3.5921280e-3f, -8.8632355e-3f);
-      t = fmaf(z, t, 2.1869489e-2f);
-      t = fmaf(z, t, -5.3968254e-2f);
-      t = fmaf(z, t, 1.3333333e-1f);
-      t = fmaf(z, t, -3.3333333e-1f);
-      v[i] *= fmaf(z * lin, t, lin);
     }
   }
 }
@@ -419,14 +452,23 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
             for (int e = 0; e < 8; ++e) o[e] = __uint_as_float(ov[i + e]) * inv;
             if (MODE == 2 && p.out_cos) {
               const size_t at = (size_t)min(qpos, p.out_n - 1) * p.out_half;
+              const int m = (cb + i) / 2;
+              float co[4], si[4];
+              if ((p.out_half & 3) == 0 && m < p.out_half) {             // (rows of whole vectors)
+                loadv<4>(p.out_cos + at + m, co);
+                loadv<4>(p.out_sin + at + m, si);
+              } else {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                  co[e] = m + e < p.out_half ? __ldg(p.out_cos + at + m + e) : 1.f;
+                  si[e] = m + e < p.out_half ? __ldg(p.out_sin + at + m + e) : 0.f;
+                }
+              }
 #pragma unroll
               for (int e = 0; e < 4; ++e) {
-                const int m = (cb + i) / 2 + e;
-                if (m < p.out_half) {
-                  const float co = __ldg(p.out_cos + at + m), si = __ldg(p.out_sin + at + m), u = o[2 * e], v = o[2 * e + 1];
-                  o[2 * e] = u * co + v * si;
-                  o[2 * e + 1] = v * co - u * si;
-                }
+                const float u = o[2 * e], v = o[2 * e + 1];
+                o[2 * e] = u * co[e] + v * si[e];
+                o[2 * e + 1] = v * co[e] - u * si[e];
               }
             }
             if (grow) {
@@ -632,7 +674,7 @@ MX_HOST_API int mx_attention_prefill_pooled(const void* q, int q_ld, const void*
   if (B <= 0 || Tq <= 0) return 0;
   if (block_size != FA_PAGE) return -110;
   if (n_kv < 1 || n_q % n_kv) return -111;
-  if (dk < 8 || dv < 8 || dk > 256 || dv > 256 || dk % 8 || dv % 8 || q_ld % 8 || out_half > dv / 2 || pool < 0) return -112;
+  if (dk < 8 || dv < 8 || dk > 256 || dv > 256 || dk % 8 || dv % 8 || q_ld % 8 || out_half > dv / 2 || pool < 0 || (((uintptr_t)out_cos | (uintptr_t)out_sin) & 15)) return -112;
   if (pool && (window < 1 || !pk || !pv || pool_pages < 1)) return -112;
   if ((gate && (gate_ld % 8 || ((uintptr_t)gate & 15))) || (((uintptr_t)q | (uintptr_t)pk | (uintptr_t)pv) & 15)) return -112;
   FaParams p;

@@ -955,6 +955,51 @@ __global__ void __launch_bounds__(QK_WARPS * 32) qk_post_kernel(const QkPostPara
   }
 }
 
+// The same for many tokens where nothing is normed and all rotations are of neighbouring pairs: a CTA per token, eight elements per thread and pass.
+template <typename T>
+__global__ void __launch_bounds__(256) qk_pairs_kernel(const QkPostParams p) {
+  pdl_prologue();
+  const int t = blockIdx.x, dp = p.dp, dv = p.dv;
+  const int cq = p.n_q * dp / 8, ck = cq + p.n_kv * dp / 8, all = ck + p.n_kv * dv / 8;
+  const long long slot = p.slot_map[t];
+  const int pos = max(p.positions[t], 0);
+  const size_t page = slot < 0 ? 0 : (size_t)(slot / p.block_size) * p.n_kv, off = slot < 0 ? 0 : (size_t)(slot % p.block_size);
+  const size_t at = (size_t)min(pos, p.max_pos - 1) * (p.rot / 2), vat = (size_t)min(pos, p.v_max_pos - 1) * p.v_half;
+#pragma unroll 2
+  for (int i = threadIdx.x; i < all; i += 256) {
+    const bool is_q = i < cq, is_v = i >= ck;
+    if (!is_q && slot < 0) break;
+    const int j = is_q ? i : is_v ? i - ck : i - cq, width = is_v ? dv : dp, h = j / (width / 8), c = (j - h * (width / 8)) * 8;
+    const int half = is_v ? p.v_half : p.rot / 2, m = c / 2;
+    const T* src = is_q ? reinterpret_cast<const T*>(p.q) + (size_t)t * p.q_ld : is_v ? reinterpret_cast<const T*>(p.v) + (size_t)t * p.v_ld
+                                                                                      : reinterpret_cast<const T*>(p.k) + (size_t)t * p.k_ld;
+    float v[8], co[4] = {1.f, 1.f, 1.f, 1.f}, si[4] = {0.f, 0.f, 0.f, 0.f};
+    load_group<8>(src + (size_t)j * 8, v);
+    if (m < half) {
+      const float* cs = is_v ? p.v_cos + vat + m : p.rope_cos + at + m;
+      const float* sn = is_v ? p.v_sin + vat + m : p.rope_sin + at + m;
+      if ((half & 3) == 0) {
+        loadv<4>(cs, co);
+        loadv<4>(sn, si);
+      } else {
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+          if (m + e < half) { co[e] = __ldg(cs + e); si[e] = __ldg(sn + e); }
+      }
+    }
+    const float f = is_q && p.q_scale ? p.q_scale[h] : 1.f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float a = v[2 * e], b = v[2 * e + 1];
+      v[2 * e] = fmaf(-b, si[e], a * co[e]) * f;
+      v[2 * e + 1] = fmaf(a, si[e], b * co[e]) * f;
+    }
+    T* dst = is_q ? reinterpret_cast<T*>(p.q) + (size_t)t * p.q_ld + (size_t)j * 8
+                  : reinterpret_cast<T*>(is_v ? p.v_cache : p.k_cache) + ((page + h) * p.block_size + off) * width + c;
+    store_group<8>(dst, v);
+  }
+}
+
 // ------------------------------------------------------------------ GLU over interleaved-16 columns
 __device__ __forceinline__ float glu_act(int act, float g, float u, float alpha, float limit) {
   if (act == 1) return g / (1.f + __expf(-g)) * u;
@@ -1193,6 +1238,12 @@ MX_HOST_API int mx_qk_post(void* q, int q_ld, const void* k, int k_ld, const flo
   if (p.hpw > heads) p.hpw = heads;
   const long long units = (long long)T * ((heads + p.hpw - 1) / p.hpw + (v ? (n_kv + p.hpw - 1) / p.hpw : 0) + (pk ? n_kv : 0));
   const int wide = v && dv > dp ? dv : dp;
+  if (v && T >= 128 && interleaved && !norm_after && !q_norm && !k_norm && !pk &&
+      (((uintptr_t)rope_cos | (uintptr_t)rope_sin | (uintptr_t)v_cos | (uintptr_t)v_sin) & 15) == 0) {
+    if (elem_f32) launch_pdl(qk_pairs_kernel<float>, dim3(T), dim3(256), 0, st, p);
+    else launch_pdl(qk_pairs_kernel<__nv_bfloat16>, dim3(T), dim3(256), 0, st, p);
+    return (int)cudaGetLastError();
+  }
   const dim3 grid((unsigned)((units + QK_WARPS - 1) / QK_WARPS)), block(QK_WARPS * 32);
 #define MX_QK(T_)   (wide <= 64 ? launch_pdl(qk_post_kernel<T_, 2, 1>, grid, block, 0, st, p) : wide <= 128 ? launch_pdl(qk_post_kernel<T_, 4, 1>, grid, block, 0, st, p)    : wide <= 256 ? launch_pdl(qk_post_kernel<T_, 8, 1>, grid, block, 0, st, p) : launch_pdl(qk_post_kernel<T_, 8, 2>, grid, block, 0, st, p))
   if (elem_f32) MX_QK(float); else MX_QK(__nv_bfloat16);

@@ -26,29 +26,49 @@ struct PoolParams {
 };
 constexpr int POOL_WARPS = 4;
 
-// four columns per lane and pass; T bf16 or fp32
+// A warp forms the mean of `pool` rows: groups of lanes take rows in turn, 16 bytes per lane.
 template <typename T>
 __device__ __forceinline__ void pool_row_mean(const PoolParams& p, const T* cache, T* out, T* dense, int b, int seq, int kvh, int width, int lane) {
   const int* table = p.block_table + (size_t)seq * p.max_blocks;
-  for (int c = lane * 4; c < width; c += 128) {
-    float a[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 8
-    for (int j = 0; j < p.pool; ++j) {
-      const int at = b * p.pool + j;
-      float v[4];
-      loadv<4>(cache + (((size_t)table[at / p.bs] * p.n_kv + kvh) * p.bs + at % p.bs) * width + c, v);
+  constexpr int VE = 16 / sizeof(T);
+  for (int p0 = 0; p0 < width / VE; p0 += 32) {
+    const int per = min(32, width / VE - p0), groups = 32 / per, g = lane / per, c = (p0 + lane % per) * VE;
+    float a[VE];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) a[e] += v[e];
+    for (int e = 0; e < VE; ++e) a[e] = 0.f;
+    if (g < groups) {
+#pragma unroll 8
+      for (int j = g; j < p.pool; j += groups) {
+        const int at = b * p.pool + j;
+        const T* row = cache + (((size_t)table[at / p.bs] * p.n_kv + kvh) * p.bs + at % p.bs) * width + c;
+#pragma unroll
+        for (int i = 0; i < VE; i += 4) {
+          float v[4];
+          loadv<4>(row + i, v);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) a[i + e] += v[e];
+        }
+      }
     }
     const float n = (float)p.pool;
 #pragma unroll
-    for (int e = 0; e < 4; ++e) a[e] /= n;
-    storev<4>(out + c, a);
-    if (dense) storev<4>(dense + c, a);
+    for (int e = 0; e < VE; ++e) {
+      const float mine = a[e];
+      for (int k = 1; k < groups; ++k) a[e] += __shfl_sync(0xffffffffu, mine, (lane + k * per) & 31);
+      a[e] /= n;
+    }
+    if (g == 0) {
+#pragma unroll
+      for (int i = 0; i < VE; i += 4) {
+        const float v[4] = {a[i], a[i + 1], a[i + 2], a[i + 3]};
+        storev<4>(out + c + i, v);
+        if (dense) storev<4>(dense + c + i, v);
+      }
+    }
   }
 }
 
-// blockIdx: (four blocks, sequence, kv head), a warp per block
+// blockIdx: (two blocks, sequence, kv head), a warp per block for its key and one for its value
 template <typename T>
 __global__ void __launch_bounds__(POOL_WARPS * 32) pool_blocks_kernel(const PoolParams p) {
   pdl_prologue();
@@ -58,18 +78,18 @@ __global__ void __launch_bounds__(POOL_WARPS * 32) pool_blocks_kernel(const Pool
   const int end = p.seq_lens[seq], start = end - n;
   const int seen = end > p.window ? (end - p.window) / p.pool : 0;                // blocks that the last query sees
   const int first = start > p.window ? (start - p.window) / p.pool : 0;           // ... that earlier steps saw
-  int b = blockIdx.x * POOL_WARPS + (threadIdx.x >> 5);
+  const bool vals = threadIdx.x & 32;
+  const int width = vals ? p.dv : p.dk;
+  int b = blockIdx.x * (POOL_WARPS / 2) + (threadIdx.x >> 6);
   if (!p.dense_k) b += first;
-  T *dk = nullptr, *dv = nullptr;
+  T* dense = nullptr;
   if (p.dense_k) {
     if (b >= (seen + 127) / 128 * 128) return;
     const size_t row = (((size_t)seq * p.dense_pages + b / 128) * p.n_kv + kvh) * 128 + b % 128;
-    dk = reinterpret_cast<T*>(p.dense_k) + row * p.dk;
-    dv = reinterpret_cast<T*>(p.dense_v) + row * p.dv;
+    dense = reinterpret_cast<T*>(vals ? p.dense_v : p.dense_k) + row * width;
     if (b >= seen) {
       const float zero[4] = {0.f, 0.f, 0.f, 0.f};
-      for (int c = lane * 4; c < p.dk; c += 128) storev<4>(dk + c, zero);
-      for (int c = lane * 4; c < p.dv; c += 128) storev<4>(dv + c, zero);
+      for (int c = lane * 4; c < width; c += 128) storev<4>(dense + c, zero);
       return;
     }
   } else if (b >= seen) {
@@ -77,15 +97,12 @@ __global__ void __launch_bounds__(POOL_WARPS * 32) pool_blocks_kernel(const Pool
   }
   const int page = (b * p.pool + p.pool - 1) / p.bs;
   const size_t at = ((size_t)p.block_table[(size_t)seq * p.max_blocks + page] * p.n_kv + kvh) * p.rows + (b - page * p.bs / p.pool);
-  T* pk = reinterpret_cast<T*>(p.pk) + at * p.dk;
-  T* pv = reinterpret_cast<T*>(p.pv) + at * p.dv;
+  T* out = reinterpret_cast<T*>(vals ? p.pv : p.pk) + at * width;
   if (b >= first) {
-    pool_row_mean(p, reinterpret_cast<const T*>(p.k_cache), pk, dk, b, seq, kvh, p.dk, lane);
-    pool_row_mean(p, reinterpret_cast<const T*>(p.v_cache), pv, dv, b, seq, kvh, p.dv, lane);
+    pool_row_mean(p, reinterpret_cast<const T*>(vals ? p.v_cache : p.k_cache), out, dense, b, seq, kvh, width, lane);
   } else {                                                                        // (dense only)
     float v[4];
-    for (int c = lane * 4; c < p.dk; c += 128) { loadv<4>(pk + c, v); storev<4>(dk + c, v); }
-    for (int c = lane * 4; c < p.dv; c += 128) { loadv<4>(pv + c, v); storev<4>(dv + c, v); }
+    for (int c = lane * 4; c < width; c += 128) { loadv<4>(out + c, v); storev<4>(dense + c, v); }
   }
 }
 
@@ -102,7 +119,7 @@ MX_HOST_API int mx_pool_blocks(const void* k_cache, const void* v_cache, void* p
   if (pool < 1 || window < 1 || dk % 8 || dv % 8 || rows < (bs + pool - 1) / pool || (dense_k && (!dense_v || dense_pages * 128 < max_blocks_seen))) return -116;
   PoolParams p{k_cache, v_cache, pk, pv, dense_k, dense_v, block_table, seq_lens, cu_q, n_kv, bs, dk, dv, pool, rows, window, max_blocks, dense_pages};
   const int units = dense_k ? dense_pages * 128 : max_blocks_seen;
-  const dim3 grid((unsigned)((units + POOL_WARPS - 1) / POOL_WARPS), B, n_kv), block(POOL_WARPS * 32);
+  const dim3 grid((unsigned)((units + POOL_WARPS / 2 - 1) / (POOL_WARPS / 2)), B, n_kv), block(POOL_WARPS * 32);
   if (elem_f32) launch_pdl(pool_blocks_kernel<float>, grid, block, 0, st, p);
   else launch_pdl(pool_blocks_kernel<__nv_bfloat16>, grid, block, 0, st, p);
   return (int)cudaGetLastError();

@@ -8,9 +8,10 @@
 // linear in S, so a run of tokens acts as S -> A S + B.  A cluster of CTAs owns 32 channels of one sequence and walks its tokens in rounds: every CTA takes
 // the next tile, every thread eight consecutive tokens of two channels, one warp chains the runs of the CTA, the cluster exchanges the CTAs' totals through
 // distributed shared memory, and the threads replay their runs from the right start.
-// Decode: rglru_step is one kernel from the projection to the recurrence's output.  A cluster owns a block of channels, a CTA of it a slice: every CTA forms
-// u of the whole block, streams its rows of the two gate matrices against it and advances its channels; the convolution's inputs move on behind a cluster
-// barrier, since all CTAs of the block read them.
+// Decode, a few sequences: rglru_step is one kernel from the projection to the recurrence's output.  A cluster owns a block of channels, a CTA of it a slice:
+// every CTA forms u of the whole block, multiplies its rows of the two gate matrices -- the first ones fetched before the preceding kernel has ended -- with it
+// and advances its channels; the convolution's inputs move on behind a cluster barrier, since all CTAs of the block read them.  With more sequences the
+// products go to the tensor cores and convolution and recurrence are step kernels, a thread per channel pair and sequence.
 #include "act.cuh"
 #include "cluster.cuh"
 #include "common.cuh"
@@ -131,8 +132,42 @@ __global__ void __launch_bounds__(128) causal_conv_state_kernel(const ConvParams
   }
 }
 
+// one token per sequence: the thread that owns two channels of a sequence also moves its inputs on
 template <typename T>
-static int launch_conv(const ConvParams& p, cudaStream_t st) {
+__global__ void __launch_bounds__(128) causal_conv_step_kernel(const ConvParams p) {
+  pdl_prologue();
+  const int b = blockIdx.y, c = (blockIdx.x * 128 + threadIdx.x) * 2, n1 = p.taps - 1;
+  if (c >= p.C) return;
+  const int t = p.cu_q[b];
+  if (p.cu_q[b + 1] == t) return;
+  const bool fresh = p.seq_lens[b] == 1;
+  T* st = reinterpret_cast<T*>(p.state) + (size_t)p.slots[b] * n1 * p.C + c;
+  const float2 x = load2(reinterpret_cast<const T*>(p.x) + (size_t)t * p.ld + c), bias = load2(p.b + c);
+  const float* w0 = p.w + (size_t)c * p.taps;
+  const float* w1 = w0 + p.taps;
+  float2 v[RC_MAX_TAPS - 1];
+#pragma unroll
+  for (int j = 0; j < RC_MAX_TAPS - 1; ++j) v[j] = j < n1 && !fresh ? load2(st + (size_t)j * p.C) : make_float2(0.f, 0.f);
+  float a0 = 0.f, a1 = 0.f;
+#pragma unroll
+  for (int j = 0; j < RC_MAX_TAPS - 1; ++j) {
+    if (j >= n1) break;
+    a0 = fmaf(w0[j], v[j].x, a0);
+    a1 = fmaf(w1[j], v[j].y, a1);
+    const float2 next = j + 1 < n1 ? v[(j + 1) % (RC_MAX_TAPS - 1)] : x;
+    store2(st + (size_t)j * p.C, next.x, next.y);
+  }
+  a0 = fmaf(w0[n1], x.x, a0) + bias.x;
+  a1 = fmaf(w1[n1], x.y, a1) + bias.y;
+  store2(reinterpret_cast<T*>(p.y) + (size_t)t * p.C + c, a0, a1);
+}
+
+template <typename T>
+static int launch_conv(const ConvParams& p, int max_q_len, cudaStream_t st) {
+  if (max_q_len == 1) {
+    launch_pdl(causal_conv_step_kernel<T>, dim3((p.C / 2 + 127) / 128, p.B), dim3(128), 0, st, p);
+    return (int)cudaGetLastError();
+  }
   const dim3 grid((p.C / 4 + 127) / 128, (p.T + RC_STRIP - 1) / RC_STRIP), block(128);
   switch (p.taps) {
     case 1: launch_pdl(causal_conv_kernel<T, 1>, grid, block, 0, st, p); return (int)cudaGetLastError();
@@ -279,10 +314,38 @@ __global__ void __launch_bounds__(RG_THREADS, 2) rglru_scan_kernel(const RglruPa
   cluster_sync_all();                                    // no CTA leaves while another still reads its totals
 }
 
+// one token per sequence
+template <typename T>
+__global__ void __launch_bounds__(128) rglru_scan_step_kernel(const RglruParams p) {
+  constexpr bool PRECISE = sizeof(T) == 4;
+  pdl_prologue();
+  const int b = blockIdx.y, ch = 2 * (blockIdx.x * blockDim.x + threadIdx.x);
+  const int t = p.cu_q[b];
+  if (ch >= p.W || p.cu_q[b + 1] == t) return;
+  const int blk = ch / p.n;
+  const size_t gc = (size_t)blk * 2 * p.n + (ch - blk * p.n);
+  const float* gr = p.gates + (size_t)t * 2 * p.W + gc;
+  const float2 r = load2(gr), i = load2(gr + p.n), rb = load2(p.bias + gc), ib = load2(p.bias + gc + p.n), co = load2(p.coef + ch);
+  const float2 u = load2(reinterpret_cast<const T*>(p.u) + (size_t)t * p.u_ld + ch), g = load2(reinterpret_cast<const T*>(p.g) + (size_t)t * p.g_ld + ch);
+  float* st = p.state + (size_t)p.state_slots[b] * p.W + ch;
+  float2 S = p.seq_lens[b] == 1 ? make_float2(0.f, 0.f) : load2(st);
+  float a0, b0, a1, b1;
+  rglru_gates<PRECISE>(r.x + rb.x, i.x + ib.x, u.x, co.x, a0, b0);
+  rglru_gates<PRECISE>(r.y + rb.y, i.y + ib.y, u.y, co.y, a1, b1);
+  S.x = fmaf(a0, S.x, b0);
+  S.y = fmaf(a1, S.y, b1);
+  store2(st, S.x, S.y);
+  store2(reinterpret_cast<T*>(p.y) + (size_t)t * p.W + ch, S.x * gelu_tanh<PRECISE>(g.x), S.y * gelu_tanh<PRECISE>(g.y));
+}
+
 static int g_rglru_cluster = 0;      // 0: by the length of the longest sequence; otherwise the cluster size (A/B timing)
 
 template <typename T>
 static int launch_rglru_scan(const RglruParams& p, int max_q_len, cudaStream_t st) {
+  if (max_q_len == 1) {
+    launch_pdl(rglru_scan_step_kernel<T>, dim3((p.W / 2 + 127) / 128, p.B), dim3(128), 0, st, p);
+    return (int)cudaGetLastError();
+  }
   constexpr int CP = 16, TPS = 8, CH = 2 * CP, TILE = RG_THREADS / CP * TPS;
   int c = 1;                         // CTAs along the tokens: no more than the longest sequence fills, and no more than fit the chip at once
   const long long base = (long long)p.B * ((p.W + CH - 1) / CH);
@@ -335,84 +398,127 @@ __device__ __forceinline__ float warp_sums(float (&v)[V], int lane) {
   return v[0];
 }
 
-// TT: sequences per pass.  Grid (slices per block as one cluster, blocks).
+// TT: sequences per pass.  Grid (slices per block as one cluster, blocks).  A warp owns every eighth channel of the slice and takes RS_GROUP of them at a time.
+constexpr int RS_GROUP = 4;
 template <typename T, int TT>
 __global__ void __launch_bounds__(RS_THREADS) rglru_step_kernel(const RglruStepParams p) {
   constexpr bool PRECISE = sizeof(T) == 4;
+  constexpr int WARPS = RS_THREADS / 32;
   extern __shared__ float rs_smem[];
   float* su = rs_smem;                                   // [TT][n]
   float* sg = su + TT * p.n;                             // [2][TT][slice]
   pdl_launch_dependents();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = p.n;
-  const int blk = blockIdx.y, c0 = blockIdx.x * p.slice, c1 = min(n, c0 + p.slice), base = blk * n;
-  const __nv_bfloat16* w = p.w + (size_t)blk * 2 * n * n;
-  for (int i = threadIdx.x * 64; i < (c1 - c0) * n; i += RS_THREADS * 64) {              // 128 bytes each, before the inputs exist
-    asm volatile("prefetch.global.L2 [%0];" ::"l"(w + (size_t)c0 * n + i));
-    asm volatile("prefetch.global.L2 [%0];" ::"l"(w + (size_t)(n + c0) * n + i));
-  }
-  pdl_wait();
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = p.n, n8 = n / 8;
+  const int blk = blockIdx.y, c0 = blockIdx.x * p.slice, c1 = min(n, c0 + p.slice), width = c1 - c0, base = blk * n;
+  const uint4* w = reinterpret_cast<const uint4*>(p.w + (size_t)blk * 2 * n * n);
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  uint4 wr[RS_GROUP], wi[RS_GROUP];                      // rows of r and of i of a group, one piece per lane; the first ones before the inputs exist
+  auto fetch = [&](int first, int e) {
+#pragma unroll
+    for (int q = 0; q < RS_GROUP; ++q) {
+      const int c = first + q * WARPS;
+      const bool ok = c < c1 && e < n8;
+      wr[q] = ok ? __ldg(w + (size_t)c * n8 + e) : zero;
+      wi[q] = ok ? __ldg(w + (size_t)(n + c) * n8 + e) : zero;
+    }
+  };
+  fetch(c0 + warp, lane);
   const int n1 = p.taps - 1;
+  float cw[RC_MAX_TAPS], cb = 0.f;                       // the thread's first channel
+#pragma unroll
+  for (int j = 0; j < RC_MAX_TAPS; ++j) cw[j] = j <= n1 && (int)threadIdx.x < n ? __ldg(p.conv_w + (size_t)(base + threadIdx.x) * p.taps + j) : 0.f;
+  if ((int)threadIdx.x < n) cb = __ldg(p.conv_b + base + threadIdx.x);
+  pdl_wait();
   for (int b0 = 0; b0 < p.B; b0 += TT) {
     const int nb = min(TT, p.B - b0);
-    for (int i = threadIdx.x; i < TT * n; i += RS_THREADS) {
-      const int k = i / n, c = i - k * n, b = b0 + k;
-      float u = 0.f;
-      if (k < nb) {
-        const float* cw = p.conv_w + (size_t)(base + c) * p.taps;
-        const T* st = reinterpret_cast<const T*>(p.conv_state) + (size_t)p.slots[b] * n1 * p.W + base + c;
-        const bool fresh = p.seq_lens[b] == 1;
-        for (int j = 0; j < n1; ++j) u = fmaf(cw[j], fresh ? 0.f : to_f32(st[(size_t)j * p.W]), u);
-        u = fmaf(cw[n1], to_f32(reinterpret_cast<const T*>(p.x)[(size_t)p.cu_q[b] * p.x_ld + base + c]), u) + p.conv_b[base + c];
-        u = to_f32(from_f32<T>(u));
+    for (int c = threadIdx.x; c < n; c += RS_THREADS) {
+      if (c >= RS_THREADS) {
+#pragma unroll
+        for (int j = 0; j < RC_MAX_TAPS; ++j) cw[j] = j <= n1 ? __ldg(p.conv_w + (size_t)(base + c) * p.taps + j) : 0.f;
+        cb = __ldg(p.conv_b + base + c);
       }
-      su[i] = u;
+#pragma unroll
+      for (int k = 0; k < TT; ++k) {
+        float u = 0.f;
+        if (k < nb) {
+          const int b = b0 + k;
+          const T* st = reinterpret_cast<const T*>(p.conv_state) + (size_t)p.slots[b] * n1 * p.W + base + c;
+          const bool fresh = p.seq_lens[b] == 1;
+          const float x = to_f32(reinterpret_cast<const T*>(p.x)[(size_t)p.cu_q[b] * p.x_ld + base + c]);
+#pragma unroll
+          for (int j = 0; j < RC_MAX_TAPS; ++j) {
+            if (j > n1) break;
+            u = fmaf(cw[j], j == n1 ? x : fresh ? 0.f : to_f32(st[(size_t)j * p.W]), u);
+          }
+          u = to_f32(from_f32<T>(u + cb));
+        }
+        su[k * n + c] = u;
+      }
     }
+    // what the recurrence wants, for the thread's first channel
+    float S0 = 0.f, g0 = 0.f, co = 0.f, rb = 0.f, ib = 0.f;
+    auto operands = [&](int i) {
+      const int k = i / width, c = c0 + i - k * width, b = b0 + k;
+      S0 = p.seq_lens[b] == 1 ? 0.f : p.state[(size_t)p.slots[b] * p.W + base + c];
+      g0 = to_f32(reinterpret_cast<const T*>(p.g)[(size_t)p.cu_q[b] * p.g_ld + base + c]);
+      co = p.coef[base + c];
+      rb = p.bias[(size_t)blk * 2 * n + c];
+      ib = p.bias[(size_t)blk * 2 * n + n + c];
+    };
+    if ((int)threadIdx.x < nb * width) operands(threadIdx.x);
     cluster_sync_all();                                  // all of the block's CTAs have read the convolution's inputs (and su is written)
-    for (int i = threadIdx.x; i < nb * (c1 - c0); i += RS_THREADS) {
-      const int k = i / (c1 - c0), c = base + c0 + i - k * (c1 - c0), b = b0 + k;
+    for (int i = threadIdx.x; i < nb * width; i += RS_THREADS) {
+      const int k = i / width, c = base + c0 + i - k * width, b = b0 + k;
       T* st = reinterpret_cast<T*>(p.conv_state) + (size_t)p.slots[b] * n1 * p.W + c;
       const bool fresh = p.seq_lens[b] == 1;
       for (int j = 0; j < n1; ++j)
         st[(size_t)j * p.W] = j + 1 < n1 ? (fresh ? from_f32<T>(0.f) : st[(size_t)(j + 1) * p.W]) : reinterpret_cast<const T*>(p.x)[(size_t)p.cu_q[b] * p.x_ld + c];
     }
-    for (int c = c0 + warp; c < c1; c += RS_THREADS / 32) {
-      const uint4* w0 = reinterpret_cast<const uint4*>(w + (size_t)c * n);
-      const uint4* w1 = reinterpret_cast<const uint4*>(w + (size_t)(n + c) * n);
-      float acc[2 * TT];
+    for (int first = c0 + warp; first < c1; first += RS_GROUP * WARPS) {
+      float acc[RS_GROUP][2 * TT];
 #pragma unroll
-      for (int i = 0; i < 2 * TT; ++i) acc[i] = 0.f;
-      for (int e = lane; e < n / 8; e += 32) {
-        const uint4 a = __ldg(w0 + e), q = __ldg(w1 + e);
-        const uint32_t aw[4] = {a.x, a.y, a.z, a.w}, qw[4] = {q.x, q.y, q.z, q.w};
+      for (int q = 0; q < RS_GROUP; ++q)
 #pragma unroll
-        for (int k = 0; k < TT; ++k) {
-          const float4 v0 = *reinterpret_cast<const float4*>(su + k * n + e * 8), v1 = *reinterpret_cast<const float4*>(su + k * n + e * 8 + 4);
-          const float uv[8] = {v0.x, v0.y, v0.z, v0.w, v1.x, v1.y, v1.z, v1.w};
+        for (int i = 0; i < 2 * TT; ++i) acc[q][i] = 0.f;
+      for (int e0 = 0; e0 < n8; e0 += 32) {
+        const int e = e0 + lane;
+        if (b0 || e0 || first != c0 + warp) fetch(first, e);
+        if (e < n8) {
 #pragma unroll
-          for (int j = 0; j < 4; ++j) {
-            acc[k] = fmaf(bf16_lo(aw[j]), uv[2 * j], acc[k]);
-            acc[k] = fmaf(bf16_hi(aw[j]), uv[2 * j + 1], acc[k]);
-            acc[TT + k] = fmaf(bf16_lo(qw[j]), uv[2 * j], acc[TT + k]);
-            acc[TT + k] = fmaf(bf16_hi(qw[j]), uv[2 * j + 1], acc[TT + k]);
+          for (int k = 0; k < TT; ++k) {
+            const float4 v0 = *reinterpret_cast<const float4*>(su + k * n + e * 8), v1 = *reinterpret_cast<const float4*>(su + k * n + e * 8 + 4);
+            const float uv[8] = {v0.x, v0.y, v0.z, v0.w, v1.x, v1.y, v1.z, v1.w};
+#pragma unroll
+            for (int q = 0; q < RS_GROUP; ++q) {
+              const uint32_t a[4] = {wr[q].x, wr[q].y, wr[q].z, wr[q].w}, d[4] = {wi[q].x, wi[q].y, wi[q].z, wi[q].w};
+#pragma unroll
+              for (int j = 0; j < 4; ++j) {
+                acc[q][k] = fmaf(bf16_lo(a[j]), uv[2 * j], acc[q][k]);
+                acc[q][k] = fmaf(bf16_hi(a[j]), uv[2 * j + 1], acc[q][k]);
+                acc[q][TT + k] = fmaf(bf16_lo(d[j]), uv[2 * j], acc[q][TT + k]);
+                acc[q][TT + k] = fmaf(bf16_hi(d[j]), uv[2 * j + 1], acc[q][TT + k]);
+              }
+            }
           }
         }
       }
-      const float v = warp_sums<2 * TT>(acc, lane);
       constexpr int PER = 32 / (2 * TT);
-      if (lane % PER == 0) sg[(lane / PER) * p.slice + c - c0] = v;
+#pragma unroll
+      for (int q = 0; q < RS_GROUP; ++q) {
+        const int c = first + q * WARPS;
+        const float v = warp_sums<2 * TT>(acc[q], lane);
+        if (c < c1 && lane % PER == 0) sg[(lane / PER) * p.slice + c - c0] = v;
+      }
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < nb * (c1 - c0); i += RS_THREADS) {
-      const int k = i / (c1 - c0), c = c0 + i - k * (c1 - c0), b = b0 + k;
-      float* st = p.state + (size_t)p.slots[b] * p.W + base + c;
-      const float* bias = p.bias + (size_t)blk * 2 * n + c;
+    for (int i = threadIdx.x; i < nb * width; i += RS_THREADS) {
+      const int k = i / width, c = i - k * width, b = b0 + k;
+      if (i >= RS_THREADS) operands(i);
       float a, bb;
-      rglru_gates<PRECISE>(sg[k * p.slice + c - c0] + bias[0], sg[(TT + k) * p.slice + c - c0] + bias[n], su[k * n + c], p.coef[base + c], a, bb);
-      const float S = fmaf(a, p.seq_lens[b] == 1 ? 0.f : *st, bb);
-      *st = S;
-      const size_t t = p.cu_q[b];
-      reinterpret_cast<T*>(p.y)[t * p.W + base + c] =
-          from_f32<T>(S * gelu_tanh<PRECISE>(to_f32(reinterpret_cast<const T*>(p.g)[t * p.g_ld + base + c])));
+      rglru_gates<PRECISE>(sg[k * p.slice + c] + rb, sg[(TT + k) * p.slice + c] + ib, su[k * n + c0 + c], co, a, bb);
+      const float S = fmaf(a, S0, bb);
+      p.state[(size_t)p.slots[b] * p.W + base + c0 + c] = S;
+      reinterpret_cast<T*>(p.y)[(size_t)p.cu_q[b] * p.W + base + c0 + c] = from_f32<T>(S * gelu_tanh<PRECISE>(g0));
     }
     __syncthreads();                                     // su and sg are written again
   }
@@ -438,8 +544,7 @@ template <typename T>
 static int dispatch_rglru_step(const RglruStepParams& p, int blocks, cudaStream_t st) {
   if (p.B == 1) return launch_rglru_step<T, 1>(p, blocks, st);
   if (p.B == 2) return launch_rglru_step<T, 2>(p, blocks, st);
-  if (p.B <= 4 || p.n > 1024) return launch_rglru_step<T, 4>(p, blocks, st);
-  return launch_rglru_step<T, 8>(p, blocks, st);
+  return launch_rglru_step<T, 4>(p, blocks, st);
 }
 
 }  // namespace mx
@@ -449,14 +554,15 @@ using namespace mx;
 // cluster size of the prompt kernel: 1, 2, 4 or 8; 0 = chosen per call (the default)
 MX_HOST_API void mx_rglru_set_cluster(int c) { mx::g_rglru_cluster = (c == 1 || c == 2 || c == 4 || c == 8) ? c : 0; }
 
-// elem_f32: x, y and the state are fp32 instead of bf16.  C and ld multiples of 4; taps 1 .. 8.  With more than one tap the state is advanced (second launch).
+// elem_f32: x, y and the state are fp32 instead of bf16.  C and ld multiples of 4; taps 1 .. 8.  With more than one tap the state is advanced (in steps of more
+// than one token by a second launch).
 MX_HOST_API int mx_causal_conv(const void* x, int ld, const float* w, const float* b, void* state, const int* slots, const int* cu_q, const int* seq_lens, void* y,
-                               int B, int T, int C, int taps, int elem_f32, cudaStream_t st) {
+                               int B, int T, int C, int taps, int max_q_len, int elem_f32, cudaStream_t st) {
   if (B <= 0 || T <= 0) return 0;
   const uintptr_t al = elem_f32 ? 15 : 7;
   if (C % 4 || ld % 4 || taps < 1 || taps > RC_MAX_TAPS || (((uintptr_t)x | (uintptr_t)y | (uintptr_t)state) & al) || ((uintptr_t)b & 15)) return -161;
   ConvParams p{x, w, b, state, slots, cu_q, seq_lens, y, ld, C, B, T, taps};
-  return elem_f32 ? launch_conv<float>(p, st) : launch_conv<__nv_bfloat16>(p, st);
+  return elem_f32 ? launch_conv<float>(p, max_q_len, st) : launch_conv<__nv_bfloat16>(p, max_q_len, st);
 }
 
 // elem_f32: u / g / y are fp32 instead of bf16.  W a multiple of n, n even; pointers and strides aligned to element pairs.

@@ -232,8 +232,8 @@ def causal_conv(x, w, b, state, state_slots, cu_q, seq_lens, max_q_len):
     assert x.stride(1) == 1 and state.dtype == x.dtype and state.shape[1:] == (w.shape[1] - 1, W) and w.is_contiguous() and w.dtype == b.dtype == torch.float32
     y = torch.empty(T, W, dtype=x.dtype, device=x.device)
     _check(_lib.cuda().mx_causal_conv(_p(x), x.stride(0), _p(w), _p(b), _p(state), _p(state_slots), _p(cu_q), _p(seq_lens), _p(y), cu_q.numel() - 1, T, W,
-                                      w.shape[1], int(x.dtype == torch.float32), _stream()), "causal_conv")
-    _count(2 if w.shape[1] > 1 else 1)
+                                      w.shape[1], int(max_q_len), int(x.dtype == torch.float32), _stream()), "causal_conv")
+    _count(2 if w.shape[1] > 1 and max_q_len > 1 else 1)
     return y
 
 
@@ -249,11 +249,18 @@ def rglru_scan(gates, u, y, bias, coef, state, state_slots, cu_q, seq_lens, max_
     return out
 
 
+RGLRU_FUSED_MAX_B = 4        # up to this many sequences a step is one kernel; more have enough rows for the tensor cores
+
+
 def rglru_step(x, y, conv_w, conv_b, w: QuantWeight, bias, coef, conv_state, state, state_slots, cu_q, seq_lens):
     T, W = x.shape
     n = w.K
     assert w.fmt == WFormat.BF16 and (w.N, w.E) == (2 * n, W // n) and x.dtype == y.dtype == conv_state.dtype and x.stride(1) == y.stride(1) == 1
     assert cu_q.numel() - 1 == T and state.dtype == torch.float32 and state.shape[1] == W and conv_state.shape[1:] == (conv_w.shape[1] - 1, W)
+    if T > RGLRU_FUSED_MAX_B and x.dtype == torch.bfloat16:
+        u = causal_conv(x, conv_w, conv_b, conv_state, state_slots, cu_q, seq_lens, 1)
+        gates = head_linear(u.view(T, w.E, n), w, out_f32=True)
+        return rglru_scan(gates, u, y, bias, coef, state, state_slots, cu_q, seq_lens, 1)
     out = torch.empty(T, W, dtype=x.dtype, device=x.device)
     _check(_lib.cuda().mx_rglru_step(_p(x), x.stride(0), _p(y), y.stride(0), _p(conv_w), _p(conv_b), _p(w.p0), _p(bias), _p(coef), _p(conv_state), _p(state),
                                      _p(state_slots), _p(cu_q), _p(seq_lens), _p(out), T, W, n, conv_w.shape[1], int(x.dtype == torch.float32), _stream()),
