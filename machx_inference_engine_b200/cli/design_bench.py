@@ -628,7 +628,7 @@ def bench_kernels_zegelix(dev, emit) -> None:
                 dense = [form(kv) for kv in kvs]
             else:
                 dense = [None] * nb
-            for cap in (50.0, 0.0):
+            for cap in (50.0, 1.0, 0.0):                   # scores far below the cap, around it, and no cap
                 row(f"attention + pooled blocks + cap {cap:g} + sink + gate + turn {name}", "new",
                     [lambda kv=kv, x=x: K.attention(q, kv.k[0], kv.v[0], bt, sl, cu, n, sinks=sink, softcap=cap, gate=g, pools=kv.pools[0], pool_dense=x, out_rope=turn, **kw)
                      for kv, x in zip(kvs, dense)], by(live, True), 4.0 * B * nq * d * pairs)
