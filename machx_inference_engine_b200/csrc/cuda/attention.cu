@@ -55,12 +55,6 @@ struct AttnParams {
   int q_scale_n, q_ld, gate_ld, dk, dv;
   int gate_heads;              // the gate has one number per head: rows of [n_q]
   int keep_first;              // with a window: the first keys of the sequence that stay visible
-  const void* pk;              // pool pages [block][kv_head][pool_rows][dk], or null
-  const void* pv;
-  int pool, pool_rows;
-  const float* out_cos;        // [out_n][out_half] or null: the output is turned by minus its position
-  const float* out_sin;
-  int out_n, out_half;
   float* o_part;               // [splits][Tq][n_q][dv]
   float* ml_part;              // [splits][Tq][n_q][2]
   int* tickets;                // non-null: one counter per (batch entry, query tile, kv head) group; the last split merges
@@ -74,6 +68,17 @@ struct AttnParams {
   int window;                  // 0 = full causal
   float scale, softcap;
 };
+// what only the extended instances take: pooled blocks and the turned output
+struct AttnExtParams : AttnParams {
+  const void* pk;              // pool pages [block][kv_head][pool_rows][dk], or null
+  const void* pv;
+  int pool, pool_rows;
+  const float* out_cos;        // [out_n][out_half] or null: the output is turned by minus its position
+  const float* out_sin;
+  int out_n, out_half;
+};
+template <bool EXT> struct AttnArgs { using T = AttnParams; };
+template <> struct AttnArgs<true> { using T = AttnExtParams; };
 
 // blocks of `pool` tokens that a query at `pos` sees: those whose last token lies `window` or more before it
 __device__ __forceinline__ int pool_visible(int pos, int window, int pool) { return pos >= window ? (pos - window + 1) / pool : 0; }
@@ -123,9 +128,9 @@ __device__ __forceinline__ float2 k_pair(const __nv_bfloat16* r, int c) { return
 __device__ __forceinline__ float2 k_pair(const float* r, int c) { return make_float2(r[2 * c], r[2 * c + 1]); }
 template <bool PRECISE> __device__ __forceinline__ float att_exp(float x) { return PRECISE ? expf(x) : __expf(x); }
 
-// EXACT: keys and values are both HD wide; otherwise the widths come from the parameters (dv <= HD)
-template <typename T, int HD, int PPW, bool EXACT>
-__global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 : (PPW == 2 || HD <= 128) ? 3 : 2) attn_partial_kernel(const AttnParams p) {
+// EXACT: keys and values are both HD wide; otherwise the widths come from the parameters (dv <= HD).  EXT: pooled blocks, turned output.
+template <typename T, int HD, int PPW, bool EXACT, bool EXT>
+__global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 : (PPW == 2 || HD <= 128) ? 3 : 2) attn_partial_kernel(const typename AttnArgs<EXT>::T p) {
   pdl_prologue();
   constexpr int PAIRS = ATT_WARPS * PPW;
   constexpr bool PRECISE = sizeof(T) == 4;
@@ -157,7 +162,10 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
   const int kv_lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
   const int tile_lo = kv_lo / ATT_TILE, tile_hi = (kv_hi + ATT_TILE - 1) / ATT_TILE;
   const int n_keep = min((p.keep_first + ATT_TILE - 1) / ATT_TILE, tile_lo);       // kept tiles before the window's
-  const int n_pooled = p.pk ? pool_visible(pos0 + nt - 1, p.window, p.pool) : 0;
+  int n_pooled = 0;
+  if constexpr (EXT) {
+    if (p.pk) n_pooled = pool_visible(pos0 + nt - 1, p.window, p.pool);
+  }
   const int n_pool = (n_pooled + ATT_TILE - 1) / ATT_TILE;                         // tiles of pooled blocks, the first ones
   const int n_tiles = n_pool + n_keep + tile_hi - tile_lo;
   const int per = (n_tiles + p.n_splits - 1) / p.n_splits;
@@ -166,7 +174,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
   const int eff = p.tickets ? (n_tiles + per - 1) / per : p.n_splits;
   if (split >= eff) return;
 
-  __shared__ long long s_prow[ATT_TILE];
+  __shared__ long long s_prow[EXT ? ATT_TILE : 1];
   const int total_pairs = nt * gqa;
   for (int round0 = 0; round0 < total_pairs; round0 += PAIRS) {
     __syncthreads();
@@ -191,12 +199,12 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
     }
     for (int tile = my_lo; tile < my_hi; ++tile) {
       __syncthreads();
-      const bool pooled = tile < n_pool;
+      const bool pooled = EXT && tile < n_pool;
       const int tl = tile - n_pool;
       const int key0 = (pooled ? tile : tl < n_keep ? tl : tile_lo + tl - n_keep) * ATT_TILE;           // (of a pooled tile: its first block)
       const int blk = pooled ? 0 : p.block_table[(size_t)b * p.max_blocks + key0 / p.block_size];
       const size_t row0 = ((size_t)blk * p.n_kv + kvh) * p.block_size + key0 % p.block_size;
-      if (pooled) {
+      if constexpr (EXT) if (pooled) {
         if (threadIdx.x < ATT_TILE) {
           const int pb = key0 + threadIdx.x;
           long long at = -1;
@@ -221,6 +229,8 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
           const long long at = s_prow[r];
           *reinterpret_cast<uint4*>(sv + r * DV + c) = at >= 0 ? *reinterpret_cast<const uint4*>(reinterpret_cast<const T*>(p.pv) + at * DV + c) : zero;
         }
+      }
+      if (pooled) {
       } else if (EXACT && sizeof(T) == 2 && p.k_scale) {
         const size_t base = row0 * HD;
         const int8_t* k8 = reinterpret_cast<const int8_t*>(p.k_cache);
@@ -297,8 +307,11 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
               const int kpos = key0 + lane + 32 * half;
               float dd = half ? d1[pi] : d0[pi];
               if (p.softcap > 0.f) dd = p.softcap * tanhf(dd / p.softcap);
-              const bool ok = pr < total_pairs && (pooled ? kpos < pool_visible(qpos, p.window, p.pool)
-                                                          : kpos < seq_len && kpos <= qpos && (p.window <= 0 || kpos > qpos - p.window || kpos < p.keep_first));
+              bool ok = pr < total_pairs;
+              if constexpr (EXT) {
+                if (pooled) ok = ok && kpos < pool_visible(qpos, p.window, p.pool);
+              }
+              if (!pooled) ok = ok && kpos < seq_len && kpos <= qpos && (p.window <= 0 || kpos > qpos - p.window || kpos < p.keep_first);
               sc[pi][half] = ok ? dd : -INFINITY;
             }
           }
@@ -391,7 +404,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32, HD == 512 ? 2 : PPW == 1 ? 4 :
     for (int c = 0; c < HD / 32; ++c) {
       const int d = lane + 32 * c;
       float o = acc[c] * inv;
-      if (p.out_cos) {
+      if constexpr (EXT) if (p.out_cos) {
         const float other = __shfl_xor_sync(0xffffffffu, o, 1);
         if ((d >> 1) < p.out_half) {
           const size_t at = (size_t)min(pos0 + tq, p.out_n - 1) * p.out_half + (d >> 1);
@@ -484,12 +497,12 @@ static size_t att_smem(const AttnParams& p, int ppw, int elem, int kpad) {
   return (size_t)ATT_WARPS * ppw * p.dk * 4 + (size_t)ATT_TILE * (p.dk + kpad) * elem + (p.v_cache ? (size_t)ATT_TILE * p.dv * elem : 0);
 }
 
-template <typename T, int HD, int PPW, bool EXACT>
-static int launch_partial(const AttnParams& p, cudaStream_t st) {
+template <typename T, int HD, int PPW, bool EXACT, bool EXT>
+static int launch_partial(const AttnExtParams& p, cudaStream_t st) {
   constexpr size_t SMEM_MAX = ATT_SMEM_MAX;
   const size_t smem = att_smem(p, PPW, sizeof(T), att_kpad<T>());
   if (smem > SMEM_MAX) return -112;
-  auto kern = attn_partial_kernel<T, HD, PPW, EXACT>;
+  auto kern = attn_partial_kernel<T, HD, PPW, EXACT, EXT>;
   static DeviceOnce configured;
   if (configured.pending()) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, EXACT ? (int)smem : (int)SMEM_MAX);
@@ -497,7 +510,8 @@ static int launch_partial(const AttnParams& p, cudaStream_t st) {
     configured.mark();
   }
   dim3 grid(p.B * p.max_q_tiles, p.n_kv, p.n_splits);
-  launch_pdl(kern, dim3(grid), dim3(ATT_WARPS * 32), smem, st, p);
+  const typename AttnArgs<EXT>::T args = p;
+  launch_pdl(kern, dim3(grid), dim3(ATT_WARPS * 32), smem, st, args);
   return (int)cudaGetLastError();
 }
 
@@ -547,7 +561,7 @@ static int attention_impl(const void* q, const void* k_cache, const void* v_cach
   if (block_size % ATT_TILE) return -110;
   if (n_q % n_kv) return -111;
   const int gqa = n_q / n_kv;
-  AttnParams p;
+  AttnExtParams p;
   p.q = q; p.k_cache = k_cache; p.v_cache = v_cache;
   p.dk = sh.dk; p.dv = sh.dv; p.q_ld = sh.q_ld; p.gate = sh.gate; p.gate_ld = sh.gate_ld; p.gate_heads = sh.gate_heads; p.keep_first = window > 0 ? sh.keep_first : 0; p.q_scale = sh.q_scale; p.q_scale_n = sh.q_scale_n;
   p.pk = window > 0 && sh.pool > 0 ? sh.pk : nullptr; p.pv = sh.pv; p.pool = sh.pool; p.pool_rows = sh.pool_rows;
@@ -577,8 +591,10 @@ static int attention_impl(const void* q, const void* k_cache, const void* v_cach
     p.tickets = base[dev] + (size_t)(turn[dev]++ % ATT_TICKET_SLOTS) * ATT_TICKETS_PER_SLOT;
   }
   int rc;
-#define MX_ATT(T_, HD_, EX_) \
-  (ppw == 4 ? launch_partial<T_, HD_, 4, EX_>(p, st) : ppw == 2 ? launch_partial<T_, HD_, 2, EX_>(p, st) : launch_partial<T_, HD_, 1, EX_>(p, st))
+  const bool ext = p.pk || p.out_cos;
+#define MX_ATT_E(T_, HD_, EX_, XT_) \
+  (ppw == 4 ? launch_partial<T_, HD_, 4, EX_, XT_>(p, st) : ppw == 2 ? launch_partial<T_, HD_, 2, EX_, XT_>(p, st) : launch_partial<T_, HD_, 1, EX_, XT_>(p, st))
+#define MX_ATT(T_, HD_, EX_) (ext ? MX_ATT_E(T_, HD_, EX_, true) : MX_ATT_E(T_, HD_, EX_, false))
   const int dk = sh.dk, dv = sh.dv, ve = sh.elem_f32 ? 4 : 8;
   if (dk < 1 || dv < 1 || dk > (v_cache ? 512 : 1024) || dv > 512 || dk % ve || dv % ve || (!v_cache && dv > dk)) return -112;
   if (!sh.elem_f32 && v_cache && dk == dv && (dk == 64 || dk == 128 || dk == 256 || dk == 512)) {
@@ -597,6 +613,7 @@ static int attention_impl(const void* q, const void* k_cache, const void* v_cach
          : dv <= 256 ? MX_ATT(__nv_bfloat16, 256, false) : MX_ATT(__nv_bfloat16, 512, false);
   }
 #undef MX_ATT
+#undef MX_ATT_E
   if (rc || p.tickets) return rc;
   const dim3 cgrid(Tq * n_q, (dv + CMB_COLS - 1) / CMB_COLS);
   const AttnTurn turn{p.out_cos, p.out_sin, seq_lens, cu_q, p.out_n, p.out_half, B};

@@ -46,14 +46,20 @@ struct FaParams {
   __nv_bfloat16* out;      // [Tq][n_q][dv]
   int q_scale_n, gate_ld, dk, dv, q_ld;
   int gate_heads, keep_first;   // one gate number per head; with a window: the first keys that stay visible
-  int pool, pool_pages;         // MODE 2: tokens per pooled block (0: none), dense pages per sequence
-  const float* out_cos;         // MODE 2: [out_n][out_half] or null: the output is turned by minus its position
-  const float* out_sin;
-  int out_n, out_half;
   int n_q, n_kv, max_blocks, max_q_tiles, window;
   float scale, softcap;
   int* status;
 };
+
+// MODE 2 alone carries these (a longer argument block alone made the other modes spill registers)
+struct FaPoolParams : FaParams {
+  int pool, pool_pages;    // tokens per pooled block (0: none), dense pages per sequence
+  const float* out_cos;    // [out_n][out_half] or null: the output is turned by minus its position
+  const float* out_sin;
+  int out_n, out_half;
+};
+template <int MODE> struct FaArgs { using T = FaParams; };
+template <> struct FaArgs<2> { using T = FaPoolParams; };
 
 template <int DK, int DV>
 struct FaCfg {
@@ -168,7 +174,7 @@ template <int DK, int DV, bool CAP, int MODE>
 __global__ void __launch_bounds__(192, FaCfg<DK, DV>::CTAS)
 fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                   const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_qr,
-                  const __grid_constant__ CUtensorMap tmap_kr, const FaParams p) {
+                  const __grid_constant__ CUtensorMap tmap_kr, const typename FaArgs<MODE>::T p) {
   using L = FaCfg<DK, DV>;
   constexpr int ROT = MODE == 1 ? 1 : 0;         // key atoms of the shared part
   constexpr int BKV = L::BKV, NS = L::NS, KS = L::KS, VS = L::VS;
@@ -198,11 +204,17 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
   const int kv_lo = p.window > 0 ? max(0, pos0 - p.window + 1) : 0;
   const int tile_lo = kv_lo / BKV, tile_hi = (kv_hi + BKV - 1) / BKV;
   const int n_keep = min((p.keep_first + BKV - 1) / BKV, tile_lo);            // kept tiles before the window's
-  auto blocks_seen = [&](int pos) { return pos >= p.window ? (pos - p.window + 1) / p.pool : 0; };
-  const int n_pool = MODE == 2 && p.pool ? (blocks_seen(pos0 + rows - 1) + BKV - 1) / BKV : 0;          // tiles of pooled blocks, the first ones
+  auto blocks_seen = [&](int pos) {
+    if constexpr (MODE == 2) return pos >= p.window ? (pos - p.window + 1) / p.pool : 0;
+    return 0;
+  };
+  int n_pool = 0;                                                             // tiles of pooled blocks, the first ones
+  if constexpr (MODE == 2) {
+    if (p.pool) n_pool = (blocks_seen(pos0 + rows - 1) + BKV - 1) / BKV;
+  }
   const int n_tiles = n_pool + n_keep + tile_hi - tile_lo;
   auto first_key = [&](int j) {                  // (of a pooled tile: its first block)
-    if (MODE == 2) {
+    if constexpr (MODE == 2) {
       if (j < n_pool) return j * BKV;
       j -= n_pool;
     }
@@ -238,8 +250,13 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       for (int j = 0; j < n_tiles && ok; ++j) {
         const uint32_t sk = j % KS, phk = (j / KS) & 1, sv = j % VS, phv = (j / VS) & 1;
         const int key0 = first_key(j);
-        const bool pooled = MODE == 2 && j < n_pool;
-        const int blk = pooled ? b * p.pool_pages + key0 / FA_PAGE : p.block_table[(size_t)b * p.max_blocks + key0 / FA_PAGE];
+        bool pooled = false;
+        int blk = 0;
+        if constexpr (MODE == 2) pooled = j < n_pool;
+        if constexpr (MODE == 2) {
+          if (pooled) blk = b * p.pool_pages + key0 / FA_PAGE;
+        }
+        if (!pooled) blk = p.block_table[(size_t)b * p.max_blocks + key0 / FA_PAGE];
         const int krow = key0 % FA_PAGE;
         int rblk = 0;
         if constexpr (ROT != 0) rblk = p.rot_table[(size_t)b * p.max_blocks + key0 / FA_PAGE];
@@ -308,11 +325,15 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
     const float qs = p.scale * (p.q_scale ? p.q_scale[min(qpos, p.q_scale_n - 1)] : 1.f);
     // c: factor from the stored score to log2 units, applied after the maximum.  That needs c > 0: a row whose factor is not (a
     // temperature law may change sign) multiplies its scores first and goes on with 1.
-    const bool cap = CAP || (MODE == 2 && p.softcap > 0.f);
+    bool cap = CAP;
+    if constexpr (MODE == 2) cap = p.softcap > 0.f;
     const bool early = !cap && !(qs > 0.f);
     const float c = (cap || early) ? 1.f : qs * LOG2E;
     const float cap_c = p.softcap * LOG2E, inv_cap = cap ? qs / p.softcap : 0.f;
-    const int seen = MODE == 2 && p.pool ? blocks_seen(qpos) : 0;
+    int seen = 0;
+    if constexpr (MODE == 2) {
+      if (p.pool) seen = blocks_seen(qpos);
+    }
     if (p.gate && !p.gate_heads && row_ok) {       // bring the row's gate into L2 while the keys are walked
       const __nv_bfloat16* g0 = p.gate + (size_t)(q_begin + t0 + r) * p.gate_ld + (size_t)head * p.dv;
       for (int i = 0; i < p.dv; i += 64) asm volatile("prefetch.global.L2 [%0];" ::"l"(g0 + i));
@@ -333,8 +354,12 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
       __syncwarp();
       if (lane == 0) mbar_arrive(b_sempty + 8 * sb);
       const int key0 = first_key(j);
-      if (MODE == 2 && cap) {
-        softcap_run(sv, inv_cap, cap_c);
+      bool capped = false;
+      if constexpr (MODE == 2) {
+        if (cap) softcap_run(sv, inv_cap, cap_c);
+        capped = cap;
+      }
+      if (capped) {
       } else if (CAP) {
 #pragma unroll
         for (int i = 0; i < BKV; ++i) sv[i] = cap_c * tanh_fast(sv[i] * inv_cap);
@@ -343,11 +368,15 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
         for (int i = 0; i < BKV; ++i) sv[i] *= qs * LOG2E;
       }
       // a tile needs per-key masking only at the diagonal, at the window edge and at the sequence end
-      if (MODE == 2 && j < n_pool) {
-        if (key0 + BKV > blocks_seen(pos0)) {
+      bool pooled = false;
+      if constexpr (MODE == 2) {
+        pooled = j < n_pool;
+        if (pooled && key0 + BKV > blocks_seen(pos0)) {
 #pragma unroll
           for (int i = 0; i < BKV; ++i) sv[i] = key0 + i < seen ? sv[i] : -INFINITY;
         }
+      }
+      if (pooled) {
       } else if ((key0 + BKV - 1 > pos0) || (p.window > 0 && key0 <= pos0 + FA_BQ - 1 - p.window) || (key0 + BKV > seq_len)) {
         if (key0 < p.keep_first) {
 #pragma unroll
@@ -450,7 +479,7 @@ fa_prefill_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_const
             float o[8];
 #pragma unroll
             for (int e = 0; e < 8; ++e) o[e] = __uint_as_float(ov[i + e]) * inv;
-            if (MODE == 2 && p.out_cos) {
+            if constexpr (MODE == 2) if (p.out_cos) {
               const size_t at = (size_t)min(qpos, p.out_n - 1) * p.out_half;
               const int m = (cb + i) / 2;
               float co[4], si[4];
@@ -573,7 +602,7 @@ static int launch_fa_split(const void* q, const FaSplit& x, const FaParams& p, i
 // MODE 2: the plain pages and, for the pooled blocks, dense pages [n_dense][n_kv][128][dk / dv].
 struct FaPooled { const void* pk; const void* pv; int n_dense; };
 template <int DK, int DV>
-static int launch_fa_pooled(const void* q, const void* k_cache, const void* v_cache, const FaPooled& x, const FaParams& p, int B, int Tq, int n_blocks,
+static int launch_fa_pooled(const void* q, const void* k_cache, const void* v_cache, const FaPooled& x, const FaPoolParams& p, int B, int Tq, int n_blocks,
                             cudaStream_t st) {
   using L = FaCfg<DK, DV>;
   CUtensorMap tq, tk, tv, tpk, tpv;
@@ -646,7 +675,6 @@ MX_HOST_API int mx_attention_prefill_tc_ext(const void* q, int q_ld, const void*
   p.block_table = block_table; p.rot_table = nullptr; p.seq_lens = seq_lens; p.cu_q = cu_q; p.sinks = sinks; p.out = (__nv_bfloat16*)out;
   p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate ? gate_ld : 0; p.q_scale = q_scale; p.q_scale_n = q_scale_n;
   p.dk = dk; p.dv = dv; p.q_ld = q_ld; p.gate_heads = gate_heads; p.keep_first = window > 0 ? keep_first : 0;
-  p.pool = p.pool_pages = p.out_n = p.out_half = 0; p.out_cos = p.out_sin = nullptr;
   p.n_q = n_q; p.n_kv = n_kv; p.max_blocks = max_blocks; p.window = window; p.scale = scale; p.softcap = softcap;
   p.max_q_tiles = (max_q_len + FA_BQ - 1) / FA_BQ;
   p.status = status_word();
@@ -677,7 +705,7 @@ MX_HOST_API int mx_attention_prefill_pooled(const void* q, int q_ld, const void*
   if (dk < 8 || dv < 8 || dk > 256 || dv > 256 || dk % 8 || dv % 8 || q_ld % 8 || out_half > dv / 2 || pool < 0 || (((uintptr_t)out_cos | (uintptr_t)out_sin) & 15)) return -112;
   if (pool && (window < 1 || !pk || !pv || pool_pages < 1)) return -112;
   if ((gate && (gate_ld % 8 || ((uintptr_t)gate & 15))) || (((uintptr_t)q | (uintptr_t)pk | (uintptr_t)pv) & 15)) return -112;
-  FaParams p;
+  FaPoolParams p;
   p.block_table = block_table; p.rot_table = nullptr; p.seq_lens = seq_lens; p.cu_q = cu_q; p.sinks = sinks; p.out = (__nv_bfloat16*)out;
   p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate ? gate_ld : 0; p.q_scale = nullptr; p.q_scale_n = 0; p.gate_heads = p.keep_first = 0;
   p.dk = dk; p.dv = dv; p.q_ld = q_ld; p.n_q = n_q; p.n_kv = n_kv; p.max_blocks = max_blocks; p.window = window; p.scale = scale; p.softcap = softcap;
@@ -708,7 +736,6 @@ MX_HOST_API int mx_attention_prefill_latent(const void* q, int q_ld, const void*
   FaParams p;
   p.block_table = kv_table; p.rot_table = block_table; p.seq_lens = seq_lens; p.cu_q = cu_q; p.sinks = nullptr; p.out = (__nv_bfloat16*)out;
   p.gate = (const __nv_bfloat16*)gate; p.gate_ld = gate ? gate_ld : 0; p.q_scale = nullptr; p.q_scale_n = 0; p.gate_heads = p.keep_first = 0;
-  p.pool = p.pool_pages = p.out_n = p.out_half = 0; p.out_cos = p.out_sin = nullptr;
   p.dk = dim + rot; p.dv = vdim; p.q_ld = q_ld; p.n_q = n_q; p.n_kv = n_q; p.max_blocks = max_blocks; p.window = window; p.scale = scale; p.softcap = 0.f;
   p.max_q_tiles = (max_q_len + FA_BQ - 1) / FA_BQ;
   p.status = status_word();
